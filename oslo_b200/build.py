@@ -24,7 +24,11 @@ CSRC = os.path.join(HERE, "csrc")
 BUILD = os.path.join(HERE, "csrc", "build")
 
 CUDA_SOURCES = ["gemm_sm100.cu", "elementwise.cu", "attention.cu", "attention_sm100.cu", "attention_bwd_sm100.cu",
-                "decode_sm100.cu", "comm.cu", "fused_comm_gemm.cu", "noalloc_colsum.cu"]
+                "decode_sm100.cu", "comm.cu", "fused_comm_gemm.cu", "noalloc_colsum.cu", "rms_norm.cu",
+                "linear_recurrence.cu", "latent_attention.cu", "moe.cu"]
+# kernels that also serve float32 models and keep routers, norms and recurrences in 32-bit: IEEE division / square root
+# and the accurate exponential
+ACCURATE_SOURCES = ("rms_norm.cu", "linear_recurrence.cu", "latent_attention.cu", "moe.cu")
 CPP_SOURCES = ["bindings.cpp"]
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-std=c++17", "-O3", "-lineinfo",
               "--use_fast_math", "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=hidden",
@@ -85,7 +89,8 @@ def build_kernels(force: bool = False, verbose: bool = True, debug_bounds: bool 
     for src in cu:
         obj = os.path.join(BUILD, os.path.basename(src) + suffix)
         objs.append(obj)
-        jobs.append([nvcc] + NVCC_FLAGS + extra + inc + ["-c", src, "-o", obj])
+        flags = [f for f in NVCC_FLAGS if f != "--use_fast_math" or os.path.basename(src) not in ACCURATE_SOURCES]
+        jobs.append([nvcc] + flags + extra + inc + ["-c", src, "-o", obj])
     abi = int(torch._C._GLIBCXX_USE_CXX11_ABI)
     for src in cpp:
         obj = os.path.join(BUILD, os.path.basename(src) + suffix)

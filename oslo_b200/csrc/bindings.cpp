@@ -713,6 +713,318 @@ void allreduce_oneshot(Tensor x, int64_t peer_ptrs_dev, int64_t mc_ptr, int64_t 
                                   st.err.data_ptr<int>(), cur_stream()), "allreduce_oneshot");
 }
 
+
+// ---------------------------------------------------------------------- RMS norms, residual join, gated MLP
+void check_rows(const Tensor& t, const char* name) {
+  TORCH_CHECK(t.is_cuda() && t.dim() == 2 && t.stride(1) == 1 && t.stride(0) >= t.size(1), name,
+              " must be a 2-D CUDA tensor with a contiguous last dim");
+}
+const uint8_t* keep_ptr(const optional<Tensor>& keep, int64_t rows, int64_t cols, int64_t& ld) {
+  ld = 0;
+  if (!keep.has_value() || !keep->defined()) return nullptr;
+  TORCH_CHECK(keep->is_cuda() && keep->scalar_type() == at::kByte && keep->dim() == 2 && keep->size(0) == rows &&
+                  keep->size(1) >= cols && keep->stride(1) == 1, "keep must be uint8 [rows, positions]");
+  ld = keep->stride(0);
+  return keep->data_ptr<uint8_t>();
+}
+
+Tensor rms_norm(const Tensor& x, const Tensor& w, double eps, double offset) {
+  check_rows(x, "x");
+  TORCH_CHECK(w.is_contiguous() && w.numel() == x.size(1), "rms_norm: weight size");
+  TORCH_CHECK(x.scalar_type() == w.scalar_type() || x.scalar_type() == at::kFloat, "rms_norm: x is fp32 or has the weight's type");
+  c10::cuda::CUDAGuard guard(x.device());
+  Tensor out = at::empty({x.size(0), x.size(1)}, w.options());
+  check_rc(oslo_rms_norm(x.data_ptr(), x.stride(0), x.scalar_type() == at::kFloat, w.data_ptr(), out.data_ptr(), out.stride(0),
+                         x.size(0), static_cast<int>(x.size(1)), static_cast<float>(eps), static_cast<float>(offset), dt_code(w),
+                         cur_stream()), "rms_norm");
+  return out;
+}
+
+std::tuple<Tensor, Tensor> residual_join(const Tensor& x, const Tensor& y, const optional<Tensor>& slots,
+                                         const optional<Tensor>& slot_weights, const Tensor& gate, const Tensor& gate_bias,
+                                         const Tensor& w_post, const optional<Tensor>& w_next, double eps) {
+  check_rows(x, "x"); check_rows(y, "y"); check_rows(gate, "gate");
+  const int64_t rows = x.size(0), cols = x.size(1);
+  TORCH_CHECK(x.scalar_type() == at::kFloat && x.is_contiguous(), "residual_join: the residual stream is contiguous fp32");
+  TORCH_CHECK(y.size(1) == cols && gate.size(0) == rows && gate.size(1) == cols && gate_bias.numel() == cols &&
+                  w_post.numel() == cols, "residual_join: sizes");
+  TORCH_CHECK(y.scalar_type() == w_post.scalar_type() && gate.scalar_type() == y.scalar_type() &&
+                  gate_bias.scalar_type() == y.scalar_type(), "residual_join: dtypes");
+  int top = 1;
+  const float* sw = nullptr;
+  const int* sl = nullptr;
+  if (slot_weights.has_value() && slot_weights->defined()) {
+    TORCH_CHECK(slot_weights->is_contiguous() && slot_weights->scalar_type() == at::kFloat && slot_weights->size(0) == rows, "slot weights");
+    top = static_cast<int>(slot_weights->size(1));
+    sw = slot_weights->data_ptr<float>();
+    if (slots.has_value() && slots->defined()) {
+      TORCH_CHECK(slots->is_contiguous() && slots->scalar_type() == at::kInt && slots->numel() == rows * top, "slots");
+      sl = slots->data_ptr<int>();
+    } else {
+      TORCH_CHECK(y.size(0) == rows * top, "residual_join: one row of y per (token, choice)");
+    }
+  } else {
+    TORCH_CHECK(y.size(0) == rows, "residual_join: rows of y");
+  }
+  const bool next = w_next.has_value() && w_next->defined();
+  if (next) TORCH_CHECK(w_next->numel() == cols && w_next->scalar_type() == w_post.scalar_type(), "residual_join: next weight");
+  c10::cuda::CUDAGuard guard(x.device());
+  Tensor xo = at::empty_like(x);
+  Tensor h = at::empty({next ? rows : 0, cols}, y.options());
+  check_rc(oslo_residual_join(x.data_ptr<float>(), y.data_ptr(), y.stride(0), sl, sw, top, gate.data_ptr(), gate.stride(0),
+                              gate_bias.data_ptr(), w_post.data_ptr(), ptr_or_null(w_next), xo.data_ptr<float>(),
+                              next ? h.data_ptr() : nullptr, rows, static_cast<int>(cols), static_cast<float>(eps), dt_code(y),
+                              cur_stream()), "residual_join");
+  return {xo, h};
+}
+
+Tensor silu_mul(const Tensor& gate, const Tensor& up) {
+  check_rows(gate, "gate"); check_rows(up, "up");
+  TORCH_CHECK(gate.sizes() == up.sizes() && gate.scalar_type() == up.scalar_type(), "silu_mul: operands differ");
+  c10::cuda::CUDAGuard guard(gate.device());
+  Tensor out = at::empty({gate.size(0), gate.size(1)}, gate.options());
+  check_rc(oslo_silu_mul(gate.data_ptr(), gate.stride(0), up.data_ptr(), up.stride(0), out.data_ptr(), gate.size(0),
+                         static_cast<int>(gate.size(1)), dt_code(gate), cur_stream()), "silu_mul");
+  return out;
+}
+
+// ---------------------------------------------------------------------- gated linear recurrence
+void check_recurrence(const Tensor& q, const Tensor& f, const Tensor& v, const Tensor& f_bias, const Tensor& lower, int64_t heads,
+                      int64_t dim, int64_t vdim) {
+  check_rows(q, "q"); check_rows(f, "f"); check_rows(v, "v");
+  TORCH_CHECK(q.size(1) == heads * dim && f.size(1) == heads * dim && v.size(1) == heads * vdim && f.size(0) == q.size(0) &&
+                  v.size(0) == q.size(0), "recurrence: projection sizes");
+  TORCH_CHECK(f_bias.is_contiguous() && lower.is_contiguous() && f_bias.numel() == heads * dim && lower.numel() == heads * dim,
+              "recurrence: gate bias / lower bound sizes");
+  TORCH_CHECK(f.scalar_type() == q.scalar_type() && v.scalar_type() == q.scalar_type() && f_bias.scalar_type() == q.scalar_type() &&
+                  lower.scalar_type() == q.scalar_type(), "recurrence: dtypes");
+}
+
+Tensor recurrence(const Tensor& q, const Tensor& f, const Tensor& v, const Tensor& f_bias, const Tensor& lower,
+                  const optional<Tensor>& keep, const optional<Tensor>& state, int64_t batch, int64_t heads, int64_t dim,
+                  int64_t vdim, int64_t chunks) {
+  check_recurrence(q, f, v, f_bias, lower, heads, dim, vdim);
+  TORCH_CHECK(batch > 0 && q.size(0) % batch == 0, "recurrence: rows are not batch x positions");
+  const int64_t S = q.size(0) / batch;
+  int64_t ld_keep = 0;
+  const uint8_t* kp = keep_ptr(keep, batch, S, ld_keep);
+  float* st = nullptr;
+  if (state.has_value() && state->defined()) {
+    TORCH_CHECK(state->is_contiguous() && state->scalar_type() == at::kFloat && state->numel() == batch * heads * dim * vdim, "recurrence: state");
+    st = state->data_ptr<float>();
+  }
+  c10::cuda::CUDAGuard guard(q.device());
+  const int sms = dev_state(q.get_device()).sms;
+  int nch = chunks > 0 ? static_cast<int>(chunks)
+                       : oslo_recurrence_chunks(static_cast<int>(batch), static_cast<int>(S), static_cast<int>(heads),
+                                                static_cast<int>(dim), static_cast<int>(vdim), sms);
+  const auto f32 = q.options().dtype(at::kFloat);
+  Tensor out = at::empty({batch, S, heads, vdim}, f32);
+  Tensor ws, decay;
+  if (nch > 1) {
+    ws = at::empty({batch, nch, heads, dim, vdim}, f32);
+    decay = at::empty({batch, nch, heads, dim}, f32);
+  }
+  check_rc(oslo_recurrence(q.data_ptr(), q.stride(0), f.data_ptr(), f.stride(0), v.data_ptr(), v.stride(0), f_bias.data_ptr(),
+                           lower.data_ptr(), kp, ld_keep, st, out.data_ptr<float>(), nch > 1 ? ws.data_ptr<float>() : nullptr,
+                           nch > 1 ? decay.data_ptr<float>() : nullptr, nch, static_cast<int>(batch), static_cast<int>(S),
+                           static_cast<int>(heads), static_cast<int>(dim), static_cast<int>(vdim), dt_code(q),
+                           cur_stream(nch > 1 ? 3 : 1)), "recurrence");
+  return out;
+}
+
+Tensor recurrence_step(const Tensor& q, const Tensor& f, const Tensor& v, const Tensor& f_bias, const Tensor& lower,
+                       const Tensor& norm_w, const optional<Tensor>& keep, Tensor state, double eps, int64_t heads, int64_t dim,
+                       int64_t vdim) {
+  check_recurrence(q, f, v, f_bias, lower, heads, dim, vdim);
+  const int64_t B = q.size(0);
+  TORCH_CHECK(state.is_contiguous() && state.scalar_type() == at::kFloat && state.numel() == B * heads * dim * vdim, "recurrence_step: state");
+  TORCH_CHECK(norm_w.is_contiguous() && norm_w.numel() == vdim && norm_w.scalar_type() == q.scalar_type(), "recurrence_step: norm weight");
+  int64_t ld_keep = 0;
+  const uint8_t* kp = keep_ptr(keep, B, 1, ld_keep);
+  c10::cuda::CUDAGuard guard(q.device());
+  Tensor out = at::empty({B, heads * vdim}, q.options());
+  check_rc(oslo_recurrence_step(q.data_ptr(), q.stride(0), f.data_ptr(), f.stride(0), v.data_ptr(), v.stride(0),
+                                f_bias.data_ptr(), lower.data_ptr(), norm_w.data_ptr(), kp, ld_keep, state.data_ptr<float>(), out.data_ptr(),
+                                static_cast<float>(eps), static_cast<int>(B), static_cast<int>(heads), static_cast<int>(dim),
+                                static_cast<int>(vdim), dev_state(q.get_device()).sms, dt_code(q), cur_stream()), "recurrence_step");
+  return out;
+}
+
+// ---------------------------------------------------------------------- latent attention
+Tensor sink_gate(const Tensor& o, const Tensor& lse, const Tensor& sink, const Tensor& gate, int64_t vdim) {
+  // o is [B, H, S, D] (any strides, contiguous D), of which the first vdim columns count
+  TORCH_CHECK(o.is_cuda() && o.dim() == 4 && o.stride(3) == 1 && o.size(3) >= vdim, "sink_gate: o");
+  const int64_t B = o.size(0), H = o.size(1), S = o.size(2);
+  check_rows(gate, "gate");
+  TORCH_CHECK(lse.is_contiguous() && lse.scalar_type() == at::kFloat && lse.numel() == B * H * S && sink.numel() == H &&
+                  gate.size(0) == B * S && gate.size(1) == H && gate.scalar_type() == o.scalar_type() &&
+                  sink.scalar_type() == o.scalar_type(), "sink_gate: operands");
+  c10::cuda::CUDAGuard guard(o.device());
+  Tensor out = at::empty({B * S, H * vdim}, o.options());
+  check_rc(oslo_sink_gate(o.data_ptr(), o.stride(0), o.stride(2), o.stride(1), lse.data_ptr<float>(), sink.data_ptr(),
+                          gate.data_ptr(), gate.stride(0), out.data_ptr(), static_cast<int>(B), static_cast<int>(S),
+                          static_cast<int>(H), static_cast<int>(vdim), dt_code(o), cur_stream()), "sink_gate");
+  return out;
+}
+
+Tensor sink_attention(const Tensor& q, const Tensor& k, const Tensor& v, const optional<Tensor>& keep, const Tensor& sink,
+                      const Tensor& gate, double scale) {
+  // [B, S, H, D] views with contiguous D
+  TORCH_CHECK(q.is_cuda() && q.dim() == 4 && k.dim() == 4 && v.dim() == 4 && q.stride(3) == 1 && k.stride(3) == 1 && v.stride(3) == 1,
+              "sink_attention: q, k, v must be [B, S, H, D] with a contiguous last dim");
+  const int64_t B = q.size(0), Sq = q.size(1), H = q.size(2), D = q.size(3), Sk = k.size(1), Dv = v.size(3);
+  TORCH_CHECK(k.size(0) == B && v.size(0) == B && k.size(2) == H && v.size(2) == H && v.size(1) == Sk && k.size(3) == D && Sk >= Sq,
+              "sink_attention: sizes");
+  check_rows(gate, "gate");
+  TORCH_CHECK(gate.size(0) == B * Sq && gate.size(1) == H && sink.numel() == H, "sink_attention: gate / sink sizes");
+  TORCH_CHECK(k.scalar_type() == q.scalar_type() && v.scalar_type() == q.scalar_type() && gate.scalar_type() == q.scalar_type() &&
+                  sink.scalar_type() == q.scalar_type(), "sink_attention: dtypes");
+  int64_t ld_keep = 0;
+  const uint8_t* kp = keep_ptr(keep, B, Sk, ld_keep);
+  c10::cuda::CUDAGuard guard(q.device());
+  Tensor out = at::empty({B * Sq, H * Dv}, q.options());
+  check_rc(oslo_sink_attention(q.data_ptr(), q.stride(0), q.stride(1), q.stride(2), k.data_ptr(), k.stride(0), k.stride(1),
+                               k.stride(2), v.data_ptr(), v.stride(0), v.stride(1), v.stride(2), kp, ld_keep, sink.data_ptr(),
+                               gate.data_ptr(), gate.stride(0), out.data_ptr(), static_cast<int>(B), static_cast<int>(H),
+                               static_cast<int>(Sq), static_cast<int>(Sk), static_cast<int>(D), static_cast<int>(Dv),
+                               static_cast<float>(scale), dt_code(q), cur_stream()), "sink_attention");
+  return out;
+}
+
+Tensor latent_prep(const Tensor& cq, const Tensor& wq, const optional<Tensor>& ckv, const optional<Tensor>& wkv,
+                   optional<Tensor> cache, const Tensor& lengths, double eps) {
+  check_rows(cq, "cq");
+  const int64_t B = cq.size(0);
+  TORCH_CHECK(wq.is_contiguous() && wq.numel() == cq.size(1) && wq.scalar_type() == cq.scalar_type(), "latent_prep: query norm weight");
+  TORCH_CHECK(lengths.scalar_type() == at::kInt && lengths.is_contiguous() && lengths.numel() == B, "latent_prep: lengths");
+  const bool kv = ckv.has_value() && ckv->defined();
+  int64_t R = 0, T = 0;
+  if (kv) {
+    check_rows(*ckv, "ckv");
+    R = ckv->size(1);
+    TORCH_CHECK(wkv.has_value() && wkv->numel() == R && wkv->is_contiguous() && cache.has_value() && cache->dim() == 3 &&
+                    cache->is_contiguous() && cache->size(0) == B && cache->size(2) == R && ckv->size(0) == B &&
+                    cache->scalar_type() == cq.scalar_type() && ckv->scalar_type() == cq.scalar_type() &&
+                    wkv->scalar_type() == cq.scalar_type(), "latent_prep: key-value operands");
+    T = cache->size(1);
+  }
+  c10::cuda::CUDAGuard guard(cq.device());
+  Tensor out = at::empty({B, cq.size(1)}, cq.options());
+  check_rc(oslo_latent_prep(cq.data_ptr(), cq.stride(0), wq.data_ptr(), static_cast<int>(cq.size(1)), out.data_ptr(),
+                            ptr_or_null(ckv), kv ? ckv->stride(0) : 0, ptr_or_null(wkv), static_cast<int>(R),
+                            kv ? cache->data_ptr() : nullptr, lengths.data_ptr<int>(), static_cast<int>(T),
+                            static_cast<float>(eps), static_cast<int>(B), dt_code(cq),
+                            dev_state(cq.get_device()).err.data_ptr<int>(), cur_stream()), "latent_prep");
+  return out;
+}
+
+Tensor latent_decode(const Tensor& q, const Tensor& w_uk, const Tensor& w_uv, const Tensor& cache, const Tensor& lengths,
+                     const optional<Tensor>& keep, const Tensor& sink, const Tensor& gate, double scale, int64_t heads) {
+  check_rows(q, "q"); check_rows(w_uk, "w_uk"); check_rows(w_uv, "w_uv"); check_rows(gate, "gate");
+  TORCH_CHECK(cache.dim() == 3 && cache.is_contiguous(), "latent_decode: cache must be contiguous [B, T, rank]");
+  const int64_t B = q.size(0), R = cache.size(2), T = cache.size(1);
+  TORCH_CHECK(q.size(1) % heads == 0 && w_uk.size(0) == q.size(1) && w_uv.size(0) % heads == 0 && w_uk.size(1) == R &&
+                  w_uv.size(1) == R && cache.size(0) == B && gate.size(0) == B && gate.size(1) == heads && sink.numel() == heads,
+              "latent_decode: sizes");
+  TORCH_CHECK(w_uk.scalar_type() == q.scalar_type() && w_uv.scalar_type() == q.scalar_type() && cache.scalar_type() == q.scalar_type() &&
+                  gate.scalar_type() == q.scalar_type() && sink.scalar_type() == q.scalar_type(), "latent_decode: dtypes");
+  TORCH_CHECK(lengths.scalar_type() == at::kInt && lengths.is_contiguous() && lengths.numel() == B, "latent_decode: lengths");
+  int64_t ld_keep = 0;
+  const uint8_t* kp = keep_ptr(keep, B, 0, ld_keep);
+  const int64_t dim = q.size(1) / heads, vdim = w_uv.size(0) / heads;
+  c10::cuda::CUDAGuard guard(q.device());
+  auto& st = dev_state(q.get_device());
+  const int groups = static_cast<int>((heads + 15) / 16);
+  int splits = std::max<int>(1, std::min<int>(64, 2 * st.sms / std::max<int>(1, static_cast<int>(B) * groups)));
+  splits = static_cast<int>(std::min<int64_t>(splits, std::max<int64_t>(1, T / 32)));
+  const auto f32 = q.options().dtype(at::kFloat);
+  Tensor qa = at::empty({B, heads, R}, f32);
+  Tensor ws = at::empty({B, heads, splits, R + 2}, f32);
+  Tensor out = at::empty({B, heads * vdim}, q.options());
+  check_rc(oslo_latent_decode(q.data_ptr(), q.stride(0), w_uk.data_ptr(), w_uk.stride(0), w_uv.data_ptr(), w_uv.stride(0),
+                              cache.data_ptr(), lengths.data_ptr<int>(), kp, ld_keep, kp ? static_cast<int>(keep->size(1)) : 0,
+                              sink.data_ptr(), gate.data_ptr(), gate.stride(0), qa.data_ptr<float>(), ws.data_ptr<float>(),
+                              out.data_ptr(), static_cast<int>(B), static_cast<int>(heads), static_cast<int>(dim),
+                              static_cast<int>(vdim), static_cast<int>(R), static_cast<int>(T), splits,
+                              static_cast<float>(scale), dt_code(q), st.err.data_ptr<int>(), cur_stream(3)), "latent_decode");
+  return out;
+}
+
+// ---------------------------------------------------------------------- mixture of experts
+std::tuple<Tensor, Tensor> moe_route(const Tensor& h, const Tensor& w, const Tensor& bias, const optional<Tensor>& logits, int64_t top) {
+  check_rows(h, "h");
+  TORCH_CHECK(w.dim() == 2 && w.is_contiguous() && w.size(1) == h.size(1) && bias.numel() == w.size(0) &&
+                  w.scalar_type() == h.scalar_type() && bias.scalar_type() == h.scalar_type(), "moe_route: router");
+  const int64_t n = h.size(0), E = w.size(0);
+  const float* lg = nullptr;
+  if (logits.has_value() && logits->defined()) {
+    TORCH_CHECK(logits->scalar_type() == at::kFloat && logits->is_contiguous() && logits->numel() == n * E, "moe_route: logits");
+    lg = logits->data_ptr<float>();
+  }
+  c10::cuda::CUDAGuard guard(h.device());
+  Tensor idx = at::empty({n, top}, h.options().dtype(at::kInt));
+  Tensor wgt = at::empty({n, top}, h.options().dtype(at::kFloat));
+  check_rc(oslo_moe_route(h.data_ptr(), h.stride(0), w.data_ptr(), bias.data_ptr(), lg, idx.data_ptr<int>(), wgt.data_ptr<float>(),
+                          n, static_cast<int>(E), static_cast<int>(h.size(1)), static_cast<int>(top), dt_code(h), cur_stream()),
+           "moe_route");
+  return {idx, wgt};
+}
+
+// (slots [n, top], rows sorted by expert, expert of every 128-row tile, tiles in use)
+std::tuple<Tensor, Tensor, Tensor, Tensor> moe_plan(const Tensor& h, const Tensor& idx, int64_t experts) {
+  check_rows(h, "h");
+  TORCH_CHECK(idx.is_contiguous() && idx.scalar_type() == at::kInt && idx.dim() == 2 && idx.size(0) == h.size(0), "moe_plan: idx");
+  const int64_t pairs = idx.numel(), K = h.size(1);
+  const int64_t tiles = (pairs + 127) / 128 + std::min<int64_t>(experts, pairs);   // every expert rounds up by at most one tile
+  c10::cuda::CUDAGuard guard(h.device());
+  const auto i32 = h.options().dtype(at::kInt);
+  Tensor cursor = at::empty({experts}, i32), tg = at::empty({tiles}, i32), nt = at::empty({1}, i32);
+  Tensor slots = at::empty({idx.size(0), idx.size(1)}, i32);
+  Tensor rows = at::empty({tiles * 128, K}, h.options());
+  check_rc(oslo_moe_plan(h.data_ptr(), h.stride(0), idx.data_ptr<int>(), cursor.data_ptr<int>(), tg.data_ptr<int>(),
+                         nt.data_ptr<int>(), slots.data_ptr<int>(), rows.data_ptr(), pairs, static_cast<int>(experts),
+                         static_cast<int>(K), static_cast<int>(idx.size(1)), static_cast<int>(tiles), dt_code(h), cur_stream(2)),
+           "moe_plan");
+  return {slots, rows, tg, nt};
+}
+
+// act(rows . w[expert of the tile]^T): [slots, N]; tcgen05 for 16-bit types with K % 8 == 0 and N % 8 == 0
+Tensor moe_grouped(const Tensor& rows, const Tensor& w, const Tensor& tile_group, const Tensor& n_tiles, bool relu2) {
+  TORCH_CHECK(rows.is_cuda() && rows.dim() == 2 && rows.is_contiguous() && w.dim() == 3 && w.is_contiguous() &&
+                  w.size(2) == rows.size(1) && w.scalar_type() == rows.scalar_type(), "moe_grouped: operands");
+  TORCH_CHECK(tile_group.scalar_type() == at::kInt && tile_group.numel() * 128 == rows.size(0) && n_tiles.scalar_type() == at::kInt,
+              "moe_grouped: plan");
+  const int64_t N = w.size(1), K = w.size(2);
+  c10::cuda::CUDAGuard guard(rows.device());
+  auto& st = dev_state(rows.get_device());
+  Tensor out = at::empty({rows.size(0), N}, rows.options());
+  if (rows.scalar_type() != at::kFloat && K % 8 == 0 && N % 8 == 0 && reinterpret_cast<uintptr_t>(w.data_ptr()) % 16 == 0) {
+    const int fl = (relu2 ? GEMM_FLAG_RELU2 : 0) | (rows.scalar_type() == at::kHalf ? GEMM_FLAG_FP16 : 0);
+    check_rc(oslo_gemm_grouped(rows.data_ptr(), w.data_ptr(), out.data_ptr(), static_cast<int>(rows.size(0)), static_cast<int>(N),
+                               static_cast<int>(K), static_cast<int>(w.size(0)), tile_group.data_ptr<int>(),
+                               n_tiles.data_ptr<int>(), fl, st.err.data_ptr<int>(), usable_sms(st), cur_stream()), "gemm_grouped");
+  } else {
+    check_rc(oslo_moe_grouped(rows.data_ptr(), w.data_ptr(), out.data_ptr(), tile_group.data_ptr<int>(), n_tiles.data_ptr<int>(),
+                              static_cast<int>(tile_group.numel()), static_cast<int>(N), static_cast<int>(K), relu2, dt_code(rows),
+                              cur_stream()), "moe_grouped");
+  }
+  return out;
+}
+
+// one row of the result per (row, choice): act(w[idx] . x[row]); x has one row per `per_row` entries of idx
+Tensor moe_few(const Tensor& x, const Tensor& idx, const Tensor& w, int64_t per_row, bool relu2) {
+  check_rows(x, "x");
+  TORCH_CHECK(w.dim() == 3 && w.is_contiguous() && w.size(2) == x.size(1) && w.scalar_type() == x.scalar_type(), "moe_few: weights");
+  TORCH_CHECK(idx.is_contiguous() && idx.scalar_type() == at::kInt && idx.numel() == x.size(0) * per_row, "moe_few: idx");
+  c10::cuda::CUDAGuard guard(x.device());
+  Tensor out = at::empty({idx.numel(), w.size(1)}, x.options());
+  check_rc(oslo_moe_few(x.data_ptr(), x.stride(0), idx.data_ptr<int>(), w.data_ptr(), out.data_ptr(), static_cast<int>(idx.numel()),
+                        static_cast<int>(per_row), static_cast<int>(w.size(1)), static_cast<int>(w.size(2)), relu2, dt_code(x),
+                        cur_stream()), "moe_few");
+  return out;
+}
+
 }  // namespace
 
 // Schemas. Kernels that take tensors are registered for the CUDA dispatch key (below), which leaves the Meta /
@@ -755,6 +1067,19 @@ TORCH_LIBRARY(oslo_b200, m) {
   m.def("dp_reduce_scatter(Tensor like, int peer_ptrs_dev, int mc_ptr, int signal_ptrs_dev, int lo, int hi, int shard, int rank, int world, bool use_multimem) -> ()");
   m.def("dp_all_gather(Tensor like, int peer_ptrs_dev, int mc_ptr, int signal_ptrs_dev, int lo, int hi, int shard, int rank, int world, bool use_multimem) -> ()");
   m.def("allreduce_symm(int peer_ptrs_dev, int mc_ptr, int signal_ptrs_dev, Tensor(a!) out, int numel, int rank, int world, bool use_multimem) -> ()");
+  m.def("rms_norm(Tensor x, Tensor w, float eps, float offset) -> Tensor");
+  m.def("residual_join(Tensor x, Tensor y, Tensor? slots, Tensor? slot_weights, Tensor gate, Tensor gate_bias, Tensor w_post, Tensor? w_next, float eps) -> (Tensor, Tensor)");
+  m.def("silu_mul(Tensor gate, Tensor up) -> Tensor");
+  m.def("recurrence(Tensor q, Tensor f, Tensor v, Tensor f_bias, Tensor lower, Tensor? keep, Tensor(a!)? state, int batch, int heads, int dim, int vdim, int chunks=0) -> Tensor");
+  m.def("recurrence_step(Tensor q, Tensor f, Tensor v, Tensor f_bias, Tensor lower, Tensor norm_w, Tensor? keep, Tensor(a!) state, float eps, int heads, int dim, int vdim) -> Tensor");
+  m.def("sink_gate(Tensor o, Tensor lse, Tensor sink, Tensor gate, int vdim) -> Tensor");
+  m.def("sink_attention(Tensor q, Tensor k, Tensor v, Tensor? keep, Tensor sink, Tensor gate, float scale) -> Tensor");
+  m.def("latent_prep(Tensor cq, Tensor wq, Tensor? ckv, Tensor? wkv, Tensor(a!)? cache, Tensor lengths, float eps) -> Tensor");
+  m.def("latent_decode(Tensor q, Tensor w_uk, Tensor w_uv, Tensor cache, Tensor lengths, Tensor? keep, Tensor sink, Tensor gate, float scale, int heads) -> Tensor");
+  m.def("moe_route(Tensor h, Tensor w, Tensor bias, Tensor? logits, int top) -> (Tensor, Tensor)");
+  m.def("moe_plan(Tensor h, Tensor idx, int experts) -> (Tensor, Tensor, Tensor, Tensor)");
+  m.def("moe_grouped(Tensor rows, Tensor w, Tensor tile_group, Tensor n_tiles, bool relu2) -> Tensor");
+  m.def("moe_few(Tensor x, Tensor idx, Tensor w, int per_row, bool relu2) -> Tensor");
 }
 
 TORCH_LIBRARY_IMPL(oslo_b200, CUDA, m) {
@@ -792,4 +1117,17 @@ TORCH_LIBRARY_IMPL(oslo_b200, CUDA, m) {
   m.impl("ce_combine", &ce_combine);
   m.impl("dp_reduce_scatter", &dp_reduce_scatter);
   m.impl("dp_all_gather", &dp_all_gather);
+  m.impl("rms_norm", &rms_norm);
+  m.impl("residual_join", &residual_join);
+  m.impl("silu_mul", &silu_mul);
+  m.impl("recurrence", &recurrence);
+  m.impl("recurrence_step", &recurrence_step);
+  m.impl("sink_gate", &sink_gate);
+  m.impl("sink_attention", &sink_attention);
+  m.impl("latent_prep", &latent_prep);
+  m.impl("latent_decode", &latent_decode);
+  m.impl("moe_route", &moe_route);
+  m.impl("moe_plan", &moe_plan);
+  m.impl("moe_grouped", &moe_grouped);
+  m.impl("moe_few", &moe_few);
 }

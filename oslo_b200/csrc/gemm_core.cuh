@@ -58,6 +58,10 @@ struct GemmParams {
   float* ce_stats = nullptr;              // [ceil(N / 128), M, 3]
   const float* ce_lse = nullptr;          // [M]
   const float* ce_scale = nullptr;        // [M]
+  // grouped product (a mixture of experts): A holds rows sorted by group, padded so that a 128-row tile belongs to one
+  // group; B stacks the groups' [N, K] matrices. Both arrays are device data written by an earlier kernel.
+  const int* group_of_tile = nullptr;     // [tiles_m] group of every row tile, or nullptr
+  const int* group_tiles = nullptr;       // [1] row tiles in use (<= tiles_m)
   CommParams comm;
 };
 
@@ -331,6 +335,13 @@ __device__ __forceinline__ void epilogue_chunk(const GemmParams& p, int row, int
 #pragma unroll
       for (int i = 0; i < 32; ++i) v[i] = gelu_tanh_f(v[i]);
     }
+    if (p.flags & GEMM_FLAG_RELU2) {
+#pragma unroll
+      for (int i = 0; i < 32; ++i) {
+        const float x = fmaxf(v[i], 0.f);
+        v[i] = x * x;
+      }
+    }
     if (p.flags & GEMM_FLAG_DGELU) {
       const uint16_t* z = reinterpret_cast<const uint16_t*>(p.aux) + static_cast<size_t>(row) * p.ld_aux + col0;
       if (vec) {
@@ -457,14 +468,15 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_cons
     if (threadIdx.x == 0) trace[0] = globaltimer_ns();
   }
 
-  const int num_tiles = p.tiles_m * p.tiles_n;
+  const int tiles_m = (!COMM && p.group_tiles != nullptr) ? min(*p.group_tiles, p.tiles_m) : p.tiles_m;
+  const int num_tiles = tiles_m * p.tiles_n;
   const int kblocks = (p.K + BK - 1) / BK;
   // work item = (tile, k slice); one slice per tile unless split_k > 1
   const int split_k = COMM ? 1 : p.split_k;
   const int num_items = num_tiles * split_k;
   // all-gather mode walks the row blocks starting with this rank's own shard, which needs no transfer
   auto coords = [&](int tile, int& tm, int& tn) {
-    tile_coords(tile, p.tiles_m, p.tiles_n, tm, tn);
+    tile_coords(tile, tiles_m, p.tiles_n, tm, tn);
     if (COMM && p.comm.mode == COMM_ALLGATHER_A) {
       tm += p.comm.rank * (p.tiles_m / p.comm.world);
       if (tm >= p.tiles_m) tm -= p.tiles_m;
@@ -529,7 +541,9 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_cons
         const int kb0 = ks * kblocks / split_k, kb1 = (ks + 1) * kblocks / split_k;
         int tm, tn;
         coords(tile, tm, tn);
-        const int m0 = tm * BM, n0 = tn * BN;
+        const int m0 = tm * BM;
+        // rows past a group's N belong to the next group (or are zero fill); their columns are never stored
+        const int n0 = tn * BN + ((!COMM && p.group_of_tile != nullptr) ? p.group_of_tile[tm] * p.N : 0);
         for (int kb = kb0; kb < kb1; ++kb) {
           ok = mbar_wait(empty_bar(stage), phase ^ 1, abort_flag, p.err, ERR_WAIT_EMPTY);
           if (!ok) break;

@@ -248,3 +248,27 @@ extern "C" int oslo_gemm_splitk_16bit(const void* A, const void* B, float* D, in
   p.comm = CommParams{};
   return launch_split_k(ta, tb, p, split_k, num_sms, stream);
 }
+
+// D[slot, N] = act(A[slot, :] . B[group of the slot's 128-row tile]^T) for rows sorted by group (see GemmParams)
+extern "C" int oslo_gemm_grouped(const void* A, const void* B, void* D, int M, int N, int K, int groups, const int* group_of_tile,
+                                 const int* group_tiles, int flags, int* err_word, int num_sms, cudaStream_t stream) {
+  using namespace oslo;
+  if (M <= 0 || N <= 0 || K <= 0 || M % BM || groups <= 0 || group_of_tile == nullptr || group_tiles == nullptr) return -1;
+  if (flags & ~(GEMM_FLAG_RELU2 | GEMM_FLAG_FP16 | GEMM_FLAG_OUT_FP32)) return -7;
+  static thread_local bool ctx_bound = false;
+  if (!ctx_bound) { cudaFree(nullptr); ctx_bound = true; }
+  const bool fp16 = (flags & GEMM_FLAG_FP16) != 0;
+  const bool wide = N >= 256 && static_cast<long long>(M / BM) * ((N + 255) / 256) >= num_sms;
+  CUtensorMap ta, tb;
+  int rc = make_tma_2d_16bit(&ta, A, K, M, K, BM, fp16);
+  if (rc) return rc;
+  rc = make_tma_2d_16bit(&tb, B, K, static_cast<uint64_t>(groups) * N, K, wide ? 256 : 128, fp16);
+  if (rc) return rc - 1000;
+  GemmParams p;
+  p.D = D; p.bias = nullptr; p.aux = nullptr; p.aux_out = nullptr;
+  p.M = M; p.N = N; p.K = K; p.ldd = N; p.ld_aux = 0; p.ld_aux_out = 0;
+  p.a_mn_major = 0; p.b_mn_major = 0; p.flags = flags; p.alpha = 1.f; p.err = err_word;
+  p.group_of_tile = group_of_tile; p.group_tiles = group_tiles;
+  p.comm = CommParams{};
+  return wide ? launch<256, 4>(ta, tb, p, num_sms, stream) : launch<128, 6>(ta, tb, p, num_sms, stream);
+}

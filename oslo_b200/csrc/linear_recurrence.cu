@@ -1,0 +1,435 @@
+// Gated linear recurrence (HGRN2 form), state in 32-bit floats:
+//   k = (1 - lower) * sigmoid(-(f + f_bias)),  forget gate = 1 - k  (= lower + (1 - lower) * sigmoid(f + f_bias))
+//   S_t = S_{t-1} + k_t (v_t - S_{t-1})   per row of the state (a key channel) and column (a value channel)
+//   o_t[j] = sum_i silu(q_t)[i] S_t[i, j]
+// `k` is computed from the negated logit, so a gate close to 1 does not lose what it writes to cancellation.
+//
+// Prefill (recurrence_kernel): a thread keeps a 16 x 8 tile of S in registers - rows in pairs, so that every update is
+// a packed two-float FMA - and G lanes share a column group; per token it reads 16 + 16 + 8 floats from shared
+// memory, does 192 packed FMAs and reduces 8 partial outputs over the G lanes. The prompt is cut into chunks when
+// (batch x heads) alone does not fill the GPU: local states of all chunks from zero (no outputs), one elementwise scan
+// over the chunks, then every chunk again from its true initial state. Only products of forget gates (<= 1) ever
+// appear, so no chunk length can overflow.
+// Decode (recurrence_step_kernel): a cluster of CTAs per (row, head), each on a slice of the value channels; the RMS
+// norm over the head's outputs is finished over distributed shared memory, so a step is one launch.
+// Tokens whose `keep` entry is 0 (padding) leave the state as it is and produce zeros.
+#include <cooperative_groups.h>
+
+#include <algorithm>
+
+#include "num.cuh"
+#include "oslo_kernels.h"
+
+namespace cg = cooperative_groups;
+
+namespace oslo {
+
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pack_f2(float lo, float hi) {
+  f32x2 r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+  return r;
+}
+__device__ __forceinline__ void unpack_f2(f32x2 v, float& lo, float& hi) {
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v));
+}
+__device__ __forceinline__ f32x2 fma_f2(f32x2 a, f32x2 b, f32x2 c) {
+  f32x2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+
+__device__ __forceinline__ float write_gate(float logit, float lower) { return (1.0f - lower) * sigmoid_f(-logit); }
+
+struct RecParams {
+  const void *q, *f, *v;             // row (b * S + t) of each has the stride ldq / ldf / ldv
+  long long ldq, ldf, ldv;
+  const void *f_bias, *lower;        // [H * dim]
+  const uint8_t* keep; long long ld_keep;   // [B, S], 0 = padding, or nullptr
+  const float* s_in;                 // initial states, or nullptr (zero)
+  float* s_out;                      // final states, or nullptr
+  float* decay;                      // STATE_ONLY: product of the forget gates of the chunk
+  float* out;                        // [B, S, H, vdim]
+  int B, S, H, dim, vdim;
+  int chunk, nchunks;                // tokens per chunk
+  long long s_batch, s_chunk;        // element strides of s_in / s_out over batch rows and chunks
+};
+
+constexpr int REC_TB = 16;    // tokens staged at a time
+constexpr int REC_COLS = 8;   // state columns per thread
+constexpr int REC_ROWS = 16;  // state rows per thread
+
+// STATE_ONLY: no outputs, start from zero, also the chunk's total decay per row
+template <typename T, int G, bool STATE_ONLY>
+__global__ void __launch_bounds__(128) recurrence_kernel(const RecParams p) {
+  constexpr int DP = REC_ROWS * G;
+  extern __shared__ float4 rec_smem[];
+  const int nt = blockDim.x;
+  const int cols = nt / G * REC_COLS;
+  float* ks = reinterpret_cast<float*>(rec_smem);
+  float* qs = ks + REC_TB * DP;
+  float* vs = qs + (STATE_ONLY ? 0 : REC_TB * DP);
+  const int tid = threadIdx.x, g = tid % G, cgp = tid / G;
+  const int h = blockIdx.y;
+  const int b = blockIdx.z / p.nchunks, ch = blockIdx.z % p.nchunks;
+  const int col0 = blockIdx.x * cols;
+  const int t_begin = ch * p.chunk, t_end = min(p.S, t_begin + p.chunk);
+  const T* q = static_cast<const T*>(p.q) + static_cast<long long>(b) * p.S * p.ldq + static_cast<long long>(h) * p.dim;
+  const T* f = static_cast<const T*>(p.f) + static_cast<long long>(b) * p.S * p.ldf + static_cast<long long>(h) * p.dim;
+  const T* v = static_cast<const T*>(p.v) + static_cast<long long>(b) * p.S * p.ldv + static_cast<long long>(h) * p.vdim + col0;
+  const T* fb = static_cast<const T*>(p.f_bias) + h * p.dim;
+  const T* lw = static_cast<const T*>(p.lower) + h * p.dim;
+  const int my_col = col0 + cgp * REC_COLS;
+
+  // row pair rp of this thread: rows 4 * (g + G * (rp / 2)) + 2 * (rp % 2) and the next one
+  f32x2 s[REC_ROWS / 2][REC_COLS];
+  const float* sin = p.s_in ? p.s_in + b * p.s_batch + ch * p.s_chunk + static_cast<long long>(h) * p.dim * p.vdim : nullptr;
+#pragma unroll
+  for (int rp = 0; rp < REC_ROWS / 2; ++rp) {
+    const int i = 4 * (g + G * (rp / 2)) + 2 * (rp % 2);
+#pragma unroll
+    for (int c = 0; c < REC_COLS; ++c) {
+      float a0 = 0.f, a1 = 0.f;
+      if (!STATE_ONLY && sin && my_col + c < p.vdim) {
+        if (i < p.dim) a0 = sin[static_cast<long long>(i) * p.vdim + my_col + c];
+        if (i + 1 < p.dim) a1 = sin[static_cast<long long>(i + 1) * p.vdim + my_col + c];
+      }
+      s[rp][c] = pack_f2(a0, a1);
+    }
+  }
+  float dec[REC_ROWS];
+#pragma unroll
+  for (int i = 0; i < REC_ROWS; ++i) dec[i] = 1.f;
+  const f32x2 minus1 = pack_f2(-1.f, -1.f);
+
+  for (int t0 = t_begin; t0 < t_end; t0 += REC_TB) {
+    const int n = min(REC_TB, t_end - t0);
+    __syncthreads();
+    for (int e = tid; e < n * DP; e += nt) {
+      const int t = e / DP, i = e % DP;
+      const bool on = i < p.dim && (p.keep == nullptr || p.keep[b * p.ld_keep + t0 + t]);
+      float kk = 0.f, qq = 0.f;
+      if (on) {
+        kk = write_gate(Num<T>::to(f[(t0 + t) * p.ldf + i]) + Num<T>::to(fb[i]), Num<T>::to(lw[i]));
+        if (!STATE_ONLY) qq = silu_f(Num<T>::to(q[(t0 + t) * p.ldq + i]));
+      }
+      ks[t * DP + i] = kk;
+      if (!STATE_ONLY) qs[t * DP + i] = qq;
+    }
+    for (int e = tid; e < n * cols; e += nt) {
+      const int t = e / cols, c = e % cols;
+      vs[t * cols + c] = col0 + c < p.vdim ? Num<T>::to(v[(t0 + t) * p.ldv + c]) : 0.f;
+    }
+    __syncthreads();
+    for (int t = 0; t < n; ++t) {
+      f32x2 v2[REC_COLS];
+      {
+        const float4 a = *reinterpret_cast<const float4*>(vs + t * cols + cgp * REC_COLS);
+        const float4 c = *reinterpret_cast<const float4*>(vs + t * cols + cgp * REC_COLS + 4);
+        v2[0] = pack_f2(a.x, a.x); v2[1] = pack_f2(a.y, a.y); v2[2] = pack_f2(a.z, a.z); v2[3] = pack_f2(a.w, a.w);
+        v2[4] = pack_f2(c.x, c.x); v2[5] = pack_f2(c.y, c.y); v2[6] = pack_f2(c.z, c.z); v2[7] = pack_f2(c.w, c.w);
+      }
+      f32x2 o2[REC_COLS];
+#pragma unroll
+      for (int c = 0; c < REC_COLS; ++c) o2[c] = 0ull;
+#pragma unroll
+      for (int kk = 0; kk < REC_ROWS / 4; ++kk) {
+        const float4 k4 = *reinterpret_cast<const float4*>(ks + t * DP + 4 * (g + G * kk));
+        const f32x2 k2[2] = {pack_f2(k4.x, k4.y), pack_f2(k4.z, k4.w)};
+        f32x2 q2[2] = {0ull, 0ull};
+        if (!STATE_ONLY) {
+          const float4 q4 = *reinterpret_cast<const float4*>(qs + t * DP + 4 * (g + G * kk));
+          q2[0] = pack_f2(q4.x, q4.y);
+          q2[1] = pack_f2(q4.z, q4.w);
+        } else {
+          dec[4 * kk] *= 1.f - k4.x; dec[4 * kk + 1] *= 1.f - k4.y;
+          dec[4 * kk + 2] *= 1.f - k4.z; dec[4 * kk + 3] *= 1.f - k4.w;
+        }
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+#pragma unroll
+          for (int c = 0; c < REC_COLS; ++c) {
+            f32x2& st = s[2 * kk + u][c];
+            const f32x2 d = fma_f2(st, minus1, v2[c]);
+            st = fma_f2(k2[u], d, st);
+            if (!STATE_ONLY) o2[c] = fma_f2(q2[u], st, o2[c]);
+          }
+        }
+      }
+      if (!STATE_ONLY) {
+        float o[REC_COLS];
+#pragma unroll
+        for (int c = 0; c < REC_COLS; ++c) {
+          float lo, hi;
+          unpack_f2(o2[c], lo, hi);
+          o[c] = lo + hi;
+        }
+        // reduce over the G lanes; each halving step also halves the columns a lane is responsible for
+        int first = 0;   // first column this lane still holds
+        int width = REC_COLS;
+#pragma unroll
+        for (int off = G / 2; off > 0; off >>= 1) {
+          if (width > 1) {
+            const int half = width / 2;
+            const bool upper = (g & off) != 0;
+#pragma unroll
+            for (int c = 0; c < REC_COLS / 2; ++c) {
+              if (c < half) {
+                const float mine = upper ? o[c + half] : o[c];
+                const float give = upper ? o[c] : o[c + half];
+                o[c] = mine + __shfl_xor_sync(0xffffffffu, give, off);
+              }
+            }
+            if (upper) first += half;
+            width = half;
+          } else {
+            o[0] += __shfl_xor_sync(0xffffffffu, o[0], off);
+          }
+        }
+        float* orow = p.out + ((static_cast<long long>(b) * p.S + t0 + t) * p.H + h) * p.vdim;
+        const bool writes = G <= REC_COLS || (g % (G / REC_COLS > 0 ? G / REC_COLS : 1)) == 0;
+        if (writes) {
+#pragma unroll
+          for (int c = 0; c < REC_COLS; ++c)
+            if (c < width && my_col + first + c < p.vdim) orow[my_col + first + c] = o[c];
+        }
+      }
+    }
+  }
+  if (p.s_out) {
+    float* so = p.s_out + b * p.s_batch + ch * p.s_chunk + static_cast<long long>(h) * p.dim * p.vdim;
+#pragma unroll
+    for (int rp = 0; rp < REC_ROWS / 2; ++rp) {
+      const int i = 4 * (g + G * (rp / 2)) + 2 * (rp % 2);
+#pragma unroll
+      for (int c = 0; c < REC_COLS; ++c) {
+        float a0, a1;
+        unpack_f2(s[rp][c], a0, a1);
+        if (my_col + c < p.vdim) {
+          if (i < p.dim) so[static_cast<long long>(i) * p.vdim + my_col + c] = a0;
+          if (i + 1 < p.dim) so[static_cast<long long>(i + 1) * p.vdim + my_col + c] = a1;
+        }
+      }
+    }
+  }
+  if (STATE_ONLY && cgp == 0 && blockIdx.x == 0) {
+    float* d = p.decay + ((static_cast<long long>(b) * p.nchunks + ch) * p.H + h) * p.dim;
+#pragma unroll
+    for (int kk = 0; kk < REC_ROWS / 4; ++kk)
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        const int i = 4 * (g + G * kk) + u;
+        if (i < p.dim) d[i] = dec[4 * kk + u];
+      }
+  }
+}
+
+// ws[b, c] holds the local final state of chunk c; replace it by the state at the chunk's start; state <- final state
+__global__ void __launch_bounds__(256) recurrence_chunk_scan_kernel(float* __restrict__ ws, const float* __restrict__ decay,
+                                                                    const float* __restrict__ s_in, float* __restrict__ s_out,
+                                                                    int nchunks, int H, int dim, int vdim) {
+  const long long per = static_cast<long long>(H) * dim * vdim;
+  const long long e = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x;
+  const int b = blockIdx.y;
+  if (e >= per) return;
+  const long long hi = e / vdim;   // head * dim + row
+  float s = s_in ? s_in[b * per + e] : 0.f;
+  for (int c = 0; c < nchunks; ++c) {
+    const long long o = (static_cast<long long>(b) * nchunks + c) * per + e;
+    const float local = ws[o];
+    const float d = decay[(static_cast<long long>(b) * nchunks + c) * H * dim + hi];
+    ws[o] = s;
+    s = fmaf(d, s, local);
+  }
+  if (s_out) s_out[b * per + e] = s;
+}
+
+struct StepParams {
+  const void *q, *f, *v;
+  long long ldq, ldf, ldv;
+  const void *f_bias, *lower, *norm_w;
+  const uint8_t* keep; long long ld_keep;   // [B, 1], 0 = padding, or nullptr
+  float* state;      // [B, H, dim, vdim]
+  void* out;         // [B, H * vdim]
+  int H, dim, vdim, cols;   // cols: value channels per CTA
+  float eps;
+};
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) recurrence_step_kernel(const StepParams p) {
+  extern __shared__ float step_smem[];
+  float* ks = step_smem;            // [dim]
+  float* qs = ks + p.dim;           // [dim]
+  float* part = qs + p.dim;         // [ty][cols]
+  __shared__ float red[32];
+  __shared__ float slice_ss;
+  cg::cluster_group cluster = cg::this_cluster();
+  const int slices = cluster.num_blocks();
+  const int h = blockIdx.y, b = blockIdx.z, c0 = blockIdx.x * p.cols;
+  const int cols = max(0, min(p.cols, p.vdim - c0));
+  const T* q = static_cast<const T*>(p.q) + b * p.ldq + static_cast<long long>(h) * p.dim;
+  const T* f = static_cast<const T*>(p.f) + b * p.ldf + static_cast<long long>(h) * p.dim;
+  const T* v = static_cast<const T*>(p.v) + b * p.ldv + static_cast<long long>(h) * p.vdim;
+  const bool on = p.keep == nullptr || p.keep[b * p.ld_keep];
+  for (int i = threadIdx.x; i < p.dim; i += blockDim.x) {
+    ks[i] = on ? write_gate(Num<T>::to(f[i]) + Num<T>::to(static_cast<const T*>(p.f_bias)[h * p.dim + i]),
+                            Num<T>::to(static_cast<const T*>(p.lower)[h * p.dim + i])) : 0.f;
+    qs[i] = on ? silu_f(Num<T>::to(q[i])) : 0.f;
+  }
+  __syncthreads();
+  const int tx_n = p.cols / VEC;                       // the launcher keeps tx_n <= 256
+  const int ty_n = blockDim.x / tx_n;
+  const int tx = threadIdx.x % tx_n, ty = threadIdx.x / tx_n;
+  float* st = p.state + (static_cast<long long>(b) * p.H + h) * p.dim * p.vdim + c0;
+  if (ty < ty_n) {
+    const int c = tx * VEC;
+    float o[VEC], vv[VEC];
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) { o[i] = 0.f; vv[i] = c + i < cols ? Num<T>::to(v[c0 + c + i]) : 0.f; }
+    if (c < cols) {                                    // VEC > 1: the launcher guarantees vdim % VEC == 0
+#pragma unroll 4
+      for (int i = ty; i < p.dim; i += ty_n) {
+        float s[VEC];
+        load_vec<float, VEC>(st + static_cast<long long>(i) * p.vdim + c, s);
+        const float k = ks[i], qq = qs[i];
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) {
+          s[j] = fmaf(k, vv[j] - s[j], s[j]);
+          o[j] = fmaf(qq, s[j], o[j]);
+        }
+        store_vec<float, VEC>(st + static_cast<long long>(i) * p.vdim + c, s);
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) part[ty * p.cols + c + j] = o[j];
+  }
+  __syncthreads();
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < cols; c += blockDim.x) {
+    float o = 0.f;
+    for (int y = 0; y < ty_n; ++y) o += part[y * p.cols + c];
+    part[c] = o;                                       // row 0, column c: only this thread reads or writes it now
+    ss = fmaf(o, o, ss);
+  }
+  ss = block_sum(ss, red);
+  if (threadIdx.x == 0) slice_ss = ss;
+  cluster.sync();
+  float tot = 0.f;
+  for (int r = 0; r < slices; ++r) tot += *cluster.map_shared_rank(&slice_ss, r);
+  cluster.sync();                                      // no CTA leaves while another still reads its shared memory
+  const float rn = 1.0f / sqrtf(tot / p.vdim + p.eps);
+  T* out = static_cast<T*>(p.out) + (static_cast<long long>(b) * p.H + h) * p.vdim + c0;
+  const T* nw = static_cast<const T*>(p.norm_w) + c0;
+  for (int c = threadIdx.x; c < cols; c += blockDim.x) out[c] = Num<T>::from(part[c] * rn * Num<T>::to(nw[c]));
+}
+
+template <typename T, int G, bool STATE_ONLY>
+static int rec_launch(const RecParams& p, cudaStream_t st) {
+  const int groups = (p.vdim + REC_COLS - 1) / REC_COLS;
+  int nt = std::min(128, (groups * G + 31) / 32 * 32);
+  const int cols = nt / G * REC_COLS;
+  const size_t smem = static_cast<size_t>(REC_TB) * ((STATE_ONLY ? 1 : 2) * REC_ROWS * G + cols) * sizeof(float);
+  if (smem > 48 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(recurrence_kernel<T, G, STATE_ONLY>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                         static_cast<int>(smem));
+    if (e != cudaSuccess) return static_cast<int>(e);
+  }
+  dim3 grid((p.vdim + cols - 1) / cols, p.H, p.B * p.nchunks);
+  recurrence_kernel<T, G, STATE_ONLY><<<grid, nt, smem, st>>>(p);
+  return static_cast<int>(cudaGetLastError());
+}
+template <typename T, bool STATE_ONLY>
+static int rec_dispatch(const RecParams& p, cudaStream_t st) {
+  if (p.dim <= 16) return rec_launch<T, 1, STATE_ONLY>(p, st);
+  if (p.dim <= 32) return rec_launch<T, 2, STATE_ONLY>(p, st);
+  if (p.dim <= 64) return rec_launch<T, 4, STATE_ONLY>(p, st);
+  if (p.dim <= 128) return rec_launch<T, 8, STATE_ONLY>(p, st);
+  if (p.dim <= 256) return rec_launch<T, 16, STATE_ONLY>(p, st);
+  if (p.dim <= 512) return rec_launch<T, 32, STATE_ONLY>(p, st);
+  return -3;
+}
+
+}  // namespace oslo
+
+// how many chunks a prompt of S tokens is cut into so that the recurrence fills the GPU
+extern "C" int oslo_recurrence_chunks(int B, int S, int H, int dim, int vdim, int num_sms) {
+  using namespace oslo;
+  int g = 1;
+  while (16 * g < dim) g *= 2;
+  const int groups = (vdim + REC_COLS - 1) / REC_COLS;
+  const int nt = std::min(128, (groups * g + 31) / 32 * 32);
+  const int cols = nt / g * REC_COLS;
+  const long long ctas = static_cast<long long>(B) * H * ((vdim + cols - 1) / cols);
+  const int resident = 256 / nt * num_sms;             // CTAs of nt threads that keep an SM's register file busy
+  if (ctas * 2 > resident || S < 128) return 1;
+  int n = static_cast<int>(resident / ctas);
+  n = std::min(n, S / 64);
+  return std::max(1, n);
+}
+
+extern "C" int oslo_recurrence(const void* q, long long ldq, const void* f, long long ldf, const void* v, long long ldv,
+                               const void* f_bias, const void* lower, const uint8_t* keep, long long ld_keep, float* state,
+                               float* out, float* ws, float* decay, int nchunks, int B, int S, int H, int dim, int vdim,
+                               int dtype, cudaStream_t stream) {
+  using namespace oslo;
+  if (B <= 0 || S <= 0 || H <= 0) return 0;
+  if (dim <= 0 || vdim <= 0 || dim > 512 || H > 65535 || nchunks < 1 || static_cast<long long>(B) * nchunks > 65535) return -1;
+  RecParams p{};
+  p.q = q; p.f = f; p.v = v; p.ldq = ldq; p.ldf = ldf; p.ldv = ldv; p.f_bias = f_bias; p.lower = lower;
+  p.keep = keep; p.ld_keep = ld_keep; p.out = out;
+  p.B = B; p.S = S; p.H = H; p.dim = dim; p.vdim = vdim;
+  const long long per = static_cast<long long>(H) * dim * vdim;
+  int rc = 0;
+  if (nchunks == 1) {
+    p.chunk = S; p.nchunks = 1; p.s_in = state; p.s_out = state; p.s_batch = per; p.s_chunk = 0;
+    OSLO_DISPATCH_T(dtype, { rc = rec_dispatch<T, false>(p, stream); });
+    return rc;
+  }
+  if (ws == nullptr || decay == nullptr) return -1;
+  p.nchunks = nchunks;
+  p.chunk = ((S + nchunks - 1) / nchunks + REC_TB - 1) / REC_TB * REC_TB;
+  p.s_batch = per * nchunks; p.s_chunk = per;
+  p.s_in = nullptr; p.s_out = ws; p.decay = decay;
+  OSLO_DISPATCH_T(dtype, { rc = rec_dispatch<T, true>(p, stream); });
+  if (rc) return rc;
+  recurrence_chunk_scan_kernel<<<dim3(static_cast<unsigned>((per + 255) / 256), B), 256, 0, stream>>>(ws, decay, state, state,
+                                                                                                     nchunks, H, dim, vdim);
+  rc = static_cast<int>(cudaGetLastError());
+  if (rc) return rc;
+  p.s_in = ws; p.s_out = nullptr;
+  OSLO_DISPATCH_T(dtype, { rc = rec_dispatch<T, false>(p, stream); });
+  return rc;
+}
+
+extern "C" int oslo_recurrence_step(const void* q, long long ldq, const void* f, long long ldf, const void* v, long long ldv,
+                                    const void* f_bias, const void* lower, const void* norm_w, const uint8_t* keep,
+                                    long long ld_keep, float* state, void* out, float eps, int B, int H, int dim, int vdim, int num_sms, int dtype, cudaStream_t stream) {
+  using namespace oslo;
+  if (B <= 0 || H <= 0) return 0;
+  if (dim <= 0 || vdim <= 0 || B > 65535 || H > 65535) return -1;
+  const int vec = vdim % 4 == 0 && aligned_to(state, 16) ? 4 : 1;
+  int slices = 1;   // portable cluster sizes; a slice keeps at least 16 columns
+  while (slices < 8 && static_cast<long long>(B) * H * slices < 2 * num_sms && vdim / (2 * slices) >= 16) slices *= 2;
+  while (slices < 8 && (vdim + slices - 1) / slices > 256 * vec) slices *= 2;
+  int cols = ((vdim + slices - 1) / slices + vec - 1) / vec * vec;
+  if (cols / vec > 256) return -3;
+  StepParams p{q, f, v, ldq, ldf, ldv, f_bias, lower, norm_w, keep, ld_keep, state, out, H, dim, vdim, cols, eps};
+  const int ty = 256 / (cols / vec);
+  const size_t smem = (2 * static_cast<size_t>(dim) + static_cast<size_t>(ty) * cols) * sizeof(float);
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(slices, H, B);
+  cfg.blockDim = dim3(256);
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = stream;
+  cudaLaunchAttribute attr[1];
+  attr[0].id = cudaLaunchAttributeClusterDimension;
+  attr[0].val.clusterDim.x = slices; attr[0].val.clusterDim.y = 1; attr[0].val.clusterDim.z = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = 1;
+  cudaError_t e = cudaSuccess;
+  OSLO_DISPATCH_T(dtype, {
+    if (vec == 4) e = cudaLaunchKernelEx(&cfg, recurrence_step_kernel<T, 4>, p);
+    else e = cudaLaunchKernelEx(&cfg, recurrence_step_kernel<T, 1>, p);
+  });
+  return static_cast<int>(e);
+}

@@ -1,0 +1,317 @@
+// Mixture-of-experts feed-forward: routing, the plan that turns (token, choice) pairs into expert-contiguous rows, and the
+// expert products that do not go through the tcgen05 grouped GEMM (oslo_gemm_grouped, gemm_sm100.cu).
+//
+//   route:   z = W_router h + b (32-bit), the `top` largest, softmax over those only
+//   prefill: moe_plan assigns every (token, choice) a slot; an expert's slots are consecutive and start at a multiple of
+//            128, so a 128-row tile of the grouped GEMM belongs to one expert (tile_group); moe_gather copies the rows.
+//            Everything stays on the device: no counts are read back, grids are sized for the worst case.
+//   decode:  a few rows: one warp per output element of the chosen experts, straight from the expert's weights.
+// The down projection leaves one row per slot; the residual join adds them up with their weights.
+#include <math_constants.h>
+
+#include <algorithm>
+
+#include "num.cuh"
+#include "oslo_kernels.h"
+
+namespace oslo {
+
+constexpr int MOE_TILE = 128;          // rows per grouped-GEMM tile
+constexpr int MOE_MAX_EXPERTS = 2048;
+
+// the `top` largest of z[0..E) (shared memory, overwritten), ties to the lower index; softmax over them. One warp.
+__device__ __forceinline__ void pick_top(float* z, int E, int top, int* idx, float* wgt, int lane) {
+  float first = 0.f, sum = 0.f;
+  for (int j = 0; j < top; ++j) {
+    float best = -CUDART_INF_F;
+    int at = E;
+    for (int e = lane; e < E; e += 32) {
+      const float v = z[e];
+      if (v > best || (at == E && v == best)) { best = v; at = e; }
+    }
+#pragma unroll
+    for (int off = 16; off > 0; off >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, best, off);
+      const int oa = __shfl_xor_sync(0xffffffffu, at, off);
+      if (ov > best || (ov == best && oa < at)) { best = ov; at = oa; }
+    }
+    if (at >= E) { at = 0; best = 0.f; }               // only NaN logits get here
+    if (j == 0) first = best;
+    const float ex = expf(best - first);
+    sum += ex;
+    if (lane == 0) {
+      idx[j] = at;
+      wgt[j] = ex;
+      z[at] = -CUDART_INF_F;
+    }
+    __syncwarp();
+  }
+  if (lane == 0) {
+    const float inv = 1.0f / sum;
+    for (int j = 0; j < top; ++j) wgt[j] *= inv;
+  }
+}
+
+// logits from the kernel itself: one block per row
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) route_kernel(const T* __restrict__ h, long long ldh, const T* __restrict__ w,
+                                                    const T* __restrict__ bias, int* __restrict__ idx, float* __restrict__ wgt,
+                                                    int E, int K, int top) {
+  extern __shared__ float rt_smem[];
+  float* x = rt_smem;                  // [K]
+  float* z = x + K;                    // [E]
+  const long long row = blockIdx.x;
+  for (int k = threadIdx.x; k < K; k += blockDim.x) x[k] = Num<T>::to(h[row * ldh + k]);
+  __syncthreads();
+  const int lane = threadIdx.x & 31;
+  for (int e = threadIdx.x >> 5; e < E; e += blockDim.x >> 5) {
+    const float d = warp_dot<T, VEC>(w + static_cast<long long>(e) * K, x, K, lane);
+    if (lane == 0) z[e] = d + Num<T>::to(bias[e]);
+  }
+  __syncthreads();
+  if (threadIdx.x < 32) pick_top(z, E, top, idx + row * top, wgt + row * top, lane);
+}
+
+// logits [rows, E] (32-bit, without the bias) from a GEMM: one warp per row
+template <typename T>
+__global__ void __launch_bounds__(128) route_logits_kernel(const float* __restrict__ logits, const T* __restrict__ bias,
+                                                           int* __restrict__ idx, float* __restrict__ wgt, long long rows,
+                                                           int E, int top) {
+  extern __shared__ float rl_smem[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long long row = static_cast<long long>(blockIdx.x) * 4 + warp;
+  if (row >= rows) return;
+  float* z = rl_smem + warp * E;
+  for (int e = lane; e < E; e += 32) z[e] = logits[row * E + e] + Num<T>::to(bias[e]);
+  __syncwarp();
+  pick_top(z, E, top, idx + row * top, wgt + row * top, lane);
+}
+
+// counts per expert -> start slot of every expert (multiple of MOE_TILE), expert of every tile, number of tiles
+__global__ void __launch_bounds__(1024) moe_plan_kernel(const int* __restrict__ idx, long long pairs, int E,
+                                                        int* __restrict__ cursor, int* __restrict__ tile_group,
+                                                        int* __restrict__ n_tiles, int max_tiles) {
+  __shared__ int count[MOE_MAX_EXPERTS];
+  __shared__ int start[MOE_MAX_EXPERTS];
+  __shared__ int total;
+  for (int e = threadIdx.x; e < E; e += blockDim.x) count[e] = 0;
+  __syncthreads();
+  for (long long i = threadIdx.x; i < pairs; i += blockDim.x) atomicAdd(&count[idx[i]], 1);
+  __syncthreads();
+  if (threadIdx.x == 0) {
+    int t = 0;
+    for (int e = 0; e < E; ++e) {
+      start[e] = t;
+      t += (count[e] + MOE_TILE - 1) / MOE_TILE;
+    }
+    total = min(t, max_tiles);
+    *n_tiles = total;
+  }
+  __syncthreads();
+  for (int e = threadIdx.x; e < E; e += blockDim.x) {
+    cursor[e] = start[e] * MOE_TILE;
+    const int n = (count[e] + MOE_TILE - 1) / MOE_TILE;
+    for (int i = 0; i < n; ++i)
+      if (start[e] + i < max_tiles) tile_group[start[e] + i] = e;
+  }
+}
+
+// one block per (token, choice): take the next slot of its expert and copy the token's row there
+template <typename T, int VEC>
+__global__ void __launch_bounds__(128) moe_gather_kernel(const T* __restrict__ h, long long ldh, const int* __restrict__ idx,
+                                                         int* __restrict__ cursor, int* __restrict__ slots, T* __restrict__ out,
+                                                         int K, int top, int max_slots) {
+  __shared__ int slot_s;
+  const long long pair = blockIdx.x;
+  if (threadIdx.x == 0) {
+    slot_s = atomicAdd(&cursor[idx[pair]], 1);
+    slots[pair] = slot_s;
+  }
+  __syncthreads();
+  const int slot = slot_s;
+  if (slot >= max_slots) return;
+  const T* src = h + pair / top * ldh;
+  T* dst = out + static_cast<long long>(slot) * K;
+  for (int k = threadIdx.x * VEC; k < K; k += blockDim.x * VEC)
+    *reinterpret_cast<Pack<T, VEC>*>(dst + k) = *reinterpret_cast<const Pack<T, VEC>*>(src + k);
+}
+
+// scalar grouped product for types and sizes outside the tensor-core path: 32 x 64 outputs per block
+template <typename T>
+__global__ void __launch_bounds__(256) moe_grouped_kernel(const T* __restrict__ a, const T* __restrict__ w, T* __restrict__ out,
+                                                          const int* __restrict__ tile_group, const int* __restrict__ n_tiles,
+                                                          int N, int K, int relu2) {
+  constexpr int BMS = 32, BNS = 64, BKS = 16;
+  __shared__ float as[BKS][BMS + 1];
+  __shared__ float bs[BKS][BNS + 1];
+  const int m0 = blockIdx.y * BMS, n0 = blockIdx.x * BNS;
+  const int tile = m0 / MOE_TILE;
+  if (tile >= *n_tiles) return;
+  const T* b = w + static_cast<long long>(tile_group[tile]) * N * K;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  float acc[2][4] = {};
+  for (int k0 = 0; k0 < K; k0 += BKS) {
+    for (int e = threadIdx.x; e < BMS * BKS; e += 256) {
+      const int r = e / BKS, k = e % BKS;
+      as[k][r] = k0 + k < K ? Num<T>::to(a[static_cast<long long>(m0 + r) * K + k0 + k]) : 0.f;
+    }
+    for (int e = threadIdx.x; e < BNS * BKS; e += 256) {
+      const int r = e / BKS, k = e % BKS;
+      bs[k][r] = (k0 + k < K && n0 + r < N) ? Num<T>::to(b[static_cast<long long>(n0 + r) * K + k0 + k]) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < BKS; ++k) {
+      const float a0 = as[k][ty * 2], a1 = as[k][ty * 2 + 1];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float x = bs[k][tx + 16 * j];
+        acc[0][j] = fmaf(a0, x, acc[0][j]);
+        acc[1][j] = fmaf(a1, x, acc[1][j]);
+      }
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 2; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int n = n0 + tx + 16 * j;
+      if (n >= N) continue;
+      float v = acc[i][j];
+      if (relu2) { v = fmaxf(v, 0.f); v *= v; }
+      out[static_cast<long long>(m0 + ty * 2 + i) * N + n] = Num<T>::from(v);
+    }
+}
+
+// few rows: out[pair, n] = act(w[idx[pair]][n, :] . x[row of pair, :]); a warp computes 4 outputs
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) moe_few_kernel(const T* __restrict__ x, long long ldx, const int* __restrict__ idx,
+                                                      const T* __restrict__ w, T* __restrict__ out, int N, int K, int per_row,
+                                                      int relu2) {
+  extern __shared__ float mf_smem[];
+  const int pair = blockIdx.y;
+  const T* src = x + static_cast<long long>(pair / per_row) * ldx;
+  for (int k = threadIdx.x; k < K; k += blockDim.x) mf_smem[k] = Num<T>::to(src[k]);
+  __syncthreads();
+  const T* we = w + static_cast<long long>(idx[pair]) * N * K;
+  const int lane = threadIdx.x & 31;
+  const int n0 = (blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5)) * 4;
+  float acc[4] = {0.f, 0.f, 0.f, 0.f};
+  const int nn = min(4, N - n0);
+  for (int k = lane * VEC; k < K; k += 32 * VEC) {
+    float v[4][VEC];
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+      if (j < nn) load_vec<T, VEC>(we + static_cast<long long>(n0 + j) * K + k, v[j]);
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+      if (j < nn) {
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) acc[j] = fmaf(v[j][i], mf_smem[k + i], acc[j]);
+      }
+  }
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    if (j < nn) {                      // uniform over the warp
+      float v = warp_sum(acc[j]);
+      if (relu2) { v = fmaxf(v, 0.f); v *= v; }
+      if (lane == 0) out[static_cast<long long>(pair) * N + n0 + j] = Num<T>::from(v);
+    }
+  }
+}
+
+}  // namespace oslo
+
+extern "C" int oslo_moe_route(const void* h, long long ldh, const void* w, const void* bias, const float* logits, int* idx,
+                              float* wgt, long long rows, int E, int K, int top, int dtype, cudaStream_t stream) {
+  using namespace oslo;
+  if (rows <= 0) return 0;
+  if (E <= 0 || E > MOE_MAX_EXPERTS || top <= 0 || top > E || rows > 0x7fffffffll) return -1;
+  const size_t te = dtype == OSLO_DT_FP32 ? 4 : 2;
+  if (logits) {
+    OSLO_DISPATCH_T(dtype, {
+      route_logits_kernel<T><<<static_cast<unsigned>((rows + 3) / 4), 128, 4 * E * sizeof(float), stream>>>(
+          logits, static_cast<const T*>(bias), idx, wgt, rows, E, top);
+    });
+    return static_cast<int>(cudaGetLastError());
+  }
+  const size_t smem = (static_cast<size_t>(K) + E) * sizeof(float);
+  if (smem > 227 * 1024) return -3;
+  const bool vec = K % 4 == 0 && aligned_to(w, 4 * te);
+#define ROUTE_GO(V)                                                                                                   \
+  {                                                                                                                   \
+    if (smem > 48 * 1024) {                                                                                           \
+      cudaError_t e = cudaFuncSetAttribute(route_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize,           \
+                                           static_cast<int>(smem));                                                   \
+      if (e != cudaSuccess) return static_cast<int>(e);                                                               \
+    }                                                                                                                 \
+    route_kernel<T, V><<<static_cast<unsigned>(rows), 256, smem, stream>>>(                                           \
+        static_cast<const T*>(h), ldh, static_cast<const T*>(w), static_cast<const T*>(bias), idx, wgt, E, K, top);   \
+  }
+  OSLO_DISPATCH_T(dtype, { if (vec) ROUTE_GO(4) else ROUTE_GO(1) });
+#undef ROUTE_GO
+  return static_cast<int>(cudaGetLastError());
+}
+
+extern "C" int oslo_moe_plan(const void* h, long long ldh, const int* idx, int* cursor, int* tile_group, int* n_tiles, int* slots,
+                             void* rows_out, long long pairs, int E, int K, int top, int max_tiles, int dtype,
+                             cudaStream_t stream) {
+  using namespace oslo;
+  if (pairs <= 0) return 0;
+  if (E <= 0 || E > MOE_MAX_EXPERTS || pairs > 0x7fffffffll) return -1;
+  const size_t te = dtype == OSLO_DT_FP32 ? 4 : 2;
+  moe_plan_kernel<<<1, 1024, 0, stream>>>(idx, pairs, E, cursor, tile_group, n_tiles, max_tiles);
+  const int v = static_cast<int>(16 / te);
+  const bool vec = K % v == 0 && ldh % v == 0 && aligned_to(h, 16) && aligned_to(rows_out, 16);
+  OSLO_DISPATCH_T(dtype, {
+    constexpr int V = 16 / sizeof(T);
+    if (vec)
+      moe_gather_kernel<T, V><<<static_cast<unsigned>(pairs), 128, 0, stream>>>(
+          static_cast<const T*>(h), ldh, idx, cursor, slots, static_cast<T*>(rows_out), K, top, max_tiles * MOE_TILE);
+    else
+      moe_gather_kernel<T, 1><<<static_cast<unsigned>(pairs), 128, 0, stream>>>(
+          static_cast<const T*>(h), ldh, idx, cursor, slots, static_cast<T*>(rows_out), K, top, max_tiles * MOE_TILE);
+  });
+  return static_cast<int>(cudaGetLastError());
+}
+
+extern "C" int oslo_moe_grouped(const void* a, const void* w, void* out, const int* tile_group, const int* n_tiles,
+                                int max_tiles, int N, int K, int relu2, int dtype, cudaStream_t stream) {
+  using namespace oslo;
+  if (max_tiles <= 0 || N <= 0) return 0;
+  if (static_cast<long long>(max_tiles) * (MOE_TILE / 32) > 65535) return -1;
+  OSLO_DISPATCH_T(dtype, {
+    moe_grouped_kernel<T><<<dim3((N + 63) / 64, max_tiles * (MOE_TILE / 32)), 256, 0, stream>>>(
+        static_cast<const T*>(a), static_cast<const T*>(w), static_cast<T*>(out), tile_group, n_tiles, N, K, relu2);
+  });
+  return static_cast<int>(cudaGetLastError());
+}
+
+extern "C" int oslo_moe_few(const void* x, long long ldx, const int* idx, const void* w, void* out, int pairs, int per_row,
+                            int N, int K, int relu2, int dtype, cudaStream_t stream) {
+  using namespace oslo;
+  if (pairs <= 0 || N <= 0) return 0;
+  if (pairs > 65535 || per_row < 1) return -1;
+  const size_t te = dtype == OSLO_DT_FP32 ? 4 : 2;
+  const size_t smem = static_cast<size_t>(K) * sizeof(float);
+  if (smem > 227 * 1024) return -3;
+  const int v = static_cast<int>(16 / te);
+  const bool vec = K % v == 0 && aligned_to(w, 16);
+#define FEW_GO(V)                                                                                                       \
+  {                                                                                                                     \
+    if (smem > 48 * 1024) {                                                                                             \
+      cudaError_t e = cudaFuncSetAttribute(moe_few_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize,           \
+                                           static_cast<int>(smem));                                                     \
+      if (e != cudaSuccess) return static_cast<int>(e);                                                                 \
+    }                                                                                                                   \
+    moe_few_kernel<T, V><<<dim3((N + 31) / 32, pairs), 256, smem, stream>>>(                                            \
+        static_cast<const T*>(x), ldx, idx, static_cast<const T*>(w), static_cast<T*>(out), N, K, per_row, relu2);      \
+  }
+  OSLO_DISPATCH_T(dtype, {
+    constexpr int V = 16 / sizeof(T);
+    if (vec) FEW_GO(V) else FEW_GO(1)
+  });
+#undef FEW_GO
+  return static_cast<int>(cudaGetLastError());
+}

@@ -16,6 +16,7 @@
 #define GEMM_FLAG_CE_STATS 256    // LM head + cross-entropy, forward: no D; per (row, 128-column block) the epilogue emits
                                   // (max, sum exp(x - max), logit of the row's label if it lies in the block)
 #define GEMM_FLAG_CE_GRAD 512     // LM head + cross-entropy, backward: D = (exp(x - lse[row]) - [col == label]) * scale[row]
+#define GEMM_FLAG_RELU2 1024      // square of relu
 #define GEMM_CE_BLOCK 128         // columns per statistics record
 
 #define OSLO_DT_BF16 0
@@ -196,6 +197,61 @@ int oslo_allreduce_oneshot(const void* in, void* out, void* const* peer_ptrs_dev
                            uint32_t* const* signal_ptrs_dev, uint32_t* counters, long long n, long long stage_off,
                            long long half_bytes, int rank, int world, int dtype, int use_multimem, int* err_word,
                            cudaStream_t stream);
+
+// RMS norms and the residual join (rms_norm.cu). x is fp32 when x_fp32, else the storage type; rows have strides
+int oslo_rms_norm(const void* x, long long ldx, int x_fp32, const void* w, void* out, long long ldo, long long rows, int cols,
+                  float eps, float offset, int dtype, cudaStream_t stream);
+// x_out = x + rms(y * sigmoid(gate + gate_bias)) * (1 + w_post); h_out = rms(x_out) * (1 + w_next) unless w_next is null.
+// slot_weights null: y has one row per token, else y = sum_j slot_weights[t, j] * y[slots[t, j]] (slots null: t * top + j)
+int oslo_residual_join(const float* x, const void* y, long long ldy, const int* slots, const float* slot_weights, int top,
+                       const void* gate, long long ldg, const void* gate_bias, const void* w_post, const void* w_next,
+                       float* x_out, void* h_out, long long rows, int cols, float eps, int dtype, cudaStream_t stream);
+int oslo_silu_mul(const void* gate, long long ldg, const void* up, long long ldu, void* out, long long rows, int cols, int dtype,
+                  cudaStream_t stream);
+
+// gated linear recurrence (linear_recurrence.cu): q, f [B * S, H * dim], v [B * S, H * vdim] with row strides; keep [B, S]
+// (0 = padding) or null; state [B, H, dim, vdim] fp32, read and updated, or null; out fp32 [B, S, H, vdim].
+// nchunks > 1 (oslo_recurrence_chunks) needs ws [B, nchunks, H, dim, vdim] and decay [B, nchunks, H, dim] fp32
+int oslo_recurrence_chunks(int B, int S, int H, int dim, int vdim, int num_sms);
+int oslo_recurrence(const void* q, long long ldq, const void* f, long long ldf, const void* v, long long ldv,
+                    const void* f_bias, const void* lower, const uint8_t* keep, long long ld_keep, float* state, float* out,
+                    float* ws, float* decay, int nchunks, int B, int S, int H, int dim, int vdim, int dtype,
+                    cudaStream_t stream);
+// one token per row, the outputs RMS-normed per head with norm_w [vdim]
+int oslo_recurrence_step(const void* q, long long ldq, const void* f, long long ldf, const void* v, long long ldv,
+                         const void* f_bias, const void* lower, const void* norm_w, const uint8_t* keep, long long ld_keep,
+                         float* state, void* out, float eps, int B, int H, int dim, int vdim, int num_sms, int dtype, cudaStream_t stream);
+
+// latent attention (latent_attention.cu). sink_gate: flash output [B, S, H, *] + lse [B, H, S] -> out [B * S, H * vdim]
+int oslo_sink_gate(const void* o, long long o_sb, long long o_ss, long long o_sh, const float* lse, const void* sink,
+                   const void* gate, long long ldg, void* out, int B, int S, int H, int vdim, int dtype, cudaStream_t stream);
+// causal attention with sink and output gate in 32-bit, any head sizes; strides of (batch, position, head)
+int oslo_sink_attention(const void* q, long long q_sb, long long q_ss, long long q_sh, const void* k, long long k_sb,
+                        long long k_ss, long long k_sh, const void* v, long long v_sb, long long v_ss, long long v_sh,
+                        const uint8_t* keep, long long ld_keep, const void* sink, const void* gate, long long ldg, void* out,
+                        int B, int H, int Sq, int Sk, int dim, int vdim, float scale, int dtype, cudaStream_t stream);
+// decode: RMS norm of the query latent -> cq_out; of the key-value latent (null: none) -> cache [B, Tmax, kv_rank] at lengths[b]
+int oslo_latent_prep(const void* cq, long long ldq, const void* wq, int q_rank, void* cq_out, const void* ckv, long long ldkv,
+                     const void* wkv, int kv_rank, void* cache, const int* lengths, int Tmax, float eps, int B, int dtype,
+                     int* err_word, cudaStream_t stream);
+// one query per row over a latent cache; qa fp32 [B, H, R] and ws fp32 [B, H, splits, R + 2] are workspaces
+int oslo_latent_decode(const void* q, long long ldq, const void* w_uk, long long ldk, const void* w_uv, long long ldv,
+                       const void* cache, const int* lengths, const uint8_t* keep, long long ld_keep, int n_keep,
+                       const void* sink, const void* gate, long long ldg, float* qa, float* ws, void* out, int B, int H,
+                       int dim, int vdim, int R, int Tmax, int splits, float scale, int dtype, int* err_word,
+                       cudaStream_t stream);
+
+// mixture of experts (moe.cu, grouped GEMM in gemm_sm100.cu)
+int oslo_moe_route(const void* h, long long ldh, const void* w, const void* bias, const float* logits, int* idx, float* wgt,
+                   long long rows, int E, int K, int top, int dtype, cudaStream_t stream);
+int oslo_moe_plan(const void* h, long long ldh, const int* idx, int* cursor, int* tile_group, int* n_tiles, int* slots,
+                  void* rows_out, long long pairs, int E, int K, int top, int max_tiles, int dtype, cudaStream_t stream);
+int oslo_moe_grouped(const void* a, const void* w, void* out, const int* tile_group, const int* n_tiles, int max_tiles, int N,
+                     int K, int relu2, int dtype, cudaStream_t stream);
+int oslo_moe_few(const void* x, long long ldx, const int* idx, const void* w, void* out, int pairs, int per_row, int N, int K,
+                 int relu2, int dtype, cudaStream_t stream);
+int oslo_gemm_grouped(const void* A, const void* B, void* D, int M, int N, int K, int groups, const int* group_of_tile,
+                      const int* group_tiles, int flags, int* err_word, int num_sms, cudaStream_t stream);
 
 #ifdef __cplusplus
 }

@@ -1,0 +1,248 @@
+// RMS norms with 32-bit arithmetic and the step that joins a sublayer to the residual stream.
+//
+//   rms_norm:      out = x / sqrt(mean(x^2) + eps) * (offset + w)        offset 1: the weight is stored around zero
+//   residual_join: z   = y * sigmoid(gate + gate_bias)
+//                  x'  = x + z / sqrt(mean(z^2) + eps) * (1 + w_post)
+//                  h   = x' / sqrt(mean(x'^2) + eps) * (1 + w_next)      the input of the next sublayer, 16-bit
+// The residual stream x is 32-bit. y is either one row per token or the weighted sum of the `top` rows that a
+// mixture-of-experts layer left in its slot buffer, so that the experts' combine step costs no pass of its own.
+#include <algorithm>
+
+#include "num.cuh"
+#include "oslo_kernels.h"
+
+namespace oslo {
+
+// one warp per row
+template <typename TX, typename T, int VEC>
+__global__ void __launch_bounds__(256) rms_norm_warp_kernel(const TX* __restrict__ x, long long ldx, const T* __restrict__ w,
+                                                            T* __restrict__ out, long long ldo, long long rows, int cols,
+                                                            float eps, float offset) {
+  const long long row = static_cast<long long>(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  if (row >= rows) return;
+  const TX* xr = x + row * ldx;
+  float ss = 0.f;
+  for (int c = lane * VEC; c < cols; c += 32 * VEC) {
+    float v[VEC];
+    load_vec<TX, VEC>(xr + c, v);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) ss = fmaf(v[i], v[i], ss);
+  }
+  ss = warp_sum(ss);
+  const float r = 1.0f / sqrtf(ss / cols + eps);
+  for (int c = lane * VEC; c < cols; c += 32 * VEC) {
+    float v[VEC], g[VEC];
+    load_vec<TX, VEC>(xr + c, v);
+    load_vec<T, VEC>(w + c, g);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[i] = v[i] * r * (offset + g[i]);
+    store_vec<T, VEC>(out + row * ldo + c, v);
+  }
+}
+
+// one block per row
+template <typename TX, typename T, int VEC>
+__global__ void __launch_bounds__(256) rms_norm_block_kernel(const TX* __restrict__ x, long long ldx, const T* __restrict__ w,
+                                                             T* __restrict__ out, long long ldo, int cols, float eps,
+                                                             float offset) {
+  __shared__ float red[32];
+  const TX* xr = x + blockIdx.x * ldx;
+  float ss = 0.f;
+  for (int c = threadIdx.x * VEC; c < cols; c += blockDim.x * VEC) {
+    float v[VEC];
+    load_vec<TX, VEC>(xr + c, v);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) ss = fmaf(v[i], v[i], ss);
+  }
+  ss = block_sum(ss, red);
+  const float r = 1.0f / sqrtf(ss / cols + eps);
+  for (int c = threadIdx.x * VEC; c < cols; c += blockDim.x * VEC) {
+    float v[VEC], g[VEC];
+    load_vec<TX, VEC>(xr + c, v);
+    load_vec<T, VEC>(w + c, g);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[i] = v[i] * r * (offset + g[i]);
+    store_vec<T, VEC>(out + blockIdx.x * ldo + c, v);
+  }
+}
+
+template <typename TX, typename T, int VEC>
+static void rms_norm_launch(const void* x, long long ldx, const void* w, void* out, long long ldo, long long rows, int cols,
+                            float eps, float offset, cudaStream_t st) {
+  if (cols <= 512 && rows >= 64) {
+    rms_norm_warp_kernel<TX, T, VEC><<<static_cast<unsigned>((rows + 7) / 8), 256, 0, st>>>(
+        static_cast<const TX*>(x), ldx, static_cast<const T*>(w), static_cast<T*>(out), ldo, rows, cols, eps, offset);
+  } else {
+    const int threads = cols >= 256 * VEC ? 256 : (cols >= 128 * VEC ? 128 : 64);
+    rms_norm_block_kernel<TX, T, VEC><<<static_cast<unsigned>(rows), threads, 0, st>>>(
+        static_cast<const TX*>(x), ldx, static_cast<const T*>(w), static_cast<T*>(out), ldo, cols, eps, offset);
+  }
+}
+
+struct JoinParams {
+  const float* x;
+  const void* y; long long ldy;
+  const int* slots;            // [rows, top] rows of y, or nullptr: row * top + j
+  const float* slot_weights;   // [rows, top], or nullptr: y has one row per token
+  int top;
+  const void* gate; long long ldg;
+  const void* gate_bias;
+  const void* w_post;
+  const void* w_next;          // nullptr: no second norm
+  float* x_out;
+  void* h_out;
+  int cols;
+  float eps;
+};
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) residual_join_kernel(const JoinParams p) {
+  extern __shared__ float row_s[];
+  __shared__ float red[32];
+  const long long row = blockIdx.x;
+  const T* gate = static_cast<const T*>(p.gate) + row * p.ldg;
+  const T* gb = static_cast<const T*>(p.gate_bias);
+  const T* y = static_cast<const T*>(p.y);
+  float ss = 0.f;
+  for (int c = threadIdx.x * VEC; c < p.cols; c += blockDim.x * VEC) {
+    float z[VEC], g[VEC], b[VEC];
+    if (p.slot_weights == nullptr) {
+      load_vec<T, VEC>(y + row * p.ldy + c, z);
+    } else {
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) z[i] = 0.f;
+      for (int j = 0; j < p.top; ++j) {
+        const long long s = p.slots ? p.slots[row * p.top + j] : row * p.top + j;
+        const float wgt = p.slot_weights[row * p.top + j];
+        float e[VEC];
+        load_vec<T, VEC>(y + s * p.ldy + c, e);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) z[i] = fmaf(wgt, e[i], z[i]);
+      }
+    }
+    load_vec<T, VEC>(gate + c, g);
+    load_vec<T, VEC>(gb + c, b);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) {
+      z[i] *= sigmoid_f(g[i] + b[i]);
+      ss = fmaf(z[i], z[i], ss);
+      row_s[c + i] = z[i];
+    }
+  }
+  ss = block_sum(ss, red);
+  const float r = 1.0f / sqrtf(ss / p.cols + p.eps);
+  const T* wp = static_cast<const T*>(p.w_post);
+  float sx = 0.f;
+  for (int c = threadIdx.x * VEC; c < p.cols; c += blockDim.x * VEC) {   // every thread revisits its own elements
+    float v[VEC], w[VEC];
+    load_vec<float, VEC>(p.x + row * p.cols + c, v);
+    load_vec<T, VEC>(wp + c, w);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) {
+      v[i] += row_s[c + i] * r * (1.0f + w[i]);
+      sx = fmaf(v[i], v[i], sx);
+      row_s[c + i] = v[i];
+    }
+    store_vec<float, VEC>(p.x_out + row * p.cols + c, v);
+  }
+  if (p.w_next == nullptr) return;
+  sx = block_sum(sx, red);
+  const float rn = 1.0f / sqrtf(sx / p.cols + p.eps);
+  const T* wn = static_cast<const T*>(p.w_next);
+  for (int c = threadIdx.x * VEC; c < p.cols; c += blockDim.x * VEC) {
+    float v[VEC], w[VEC];
+    load_vec<T, VEC>(wn + c, w);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[i] = row_s[c + i] * rn * (1.0f + w[i]);
+    store_vec<T, VEC>(static_cast<T*>(p.h_out) + row * p.cols + c, v);
+  }
+}
+
+// y = silu(gate) * up on [rows, cols] slices with row strides
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) silu_mul_kernel(const T* __restrict__ gate, long long ldg, const T* __restrict__ up,
+                                                       long long ldu, T* __restrict__ out, long long rows, int cols) {
+  const long long per_row = cols / VEC;
+  const long long total = rows * per_row;
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const long long r = i / per_row;
+    const int c = static_cast<int>(i - r * per_row) * VEC;
+    float a[VEC], b[VEC];
+    load_vec<T, VEC>(gate + r * ldg + c, a);
+    load_vec<T, VEC>(up + r * ldu + c, b);
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) a[k] = silu_f(a[k]) * b[k];
+    store_vec<T, VEC>(out + r * cols + c, a);
+  }
+}
+
+}  // namespace oslo
+
+extern "C" int oslo_rms_norm(const void* x, long long ldx, int x_fp32, const void* w, void* out, long long ldo, long long rows,
+                             int cols, float eps, float offset, int dtype, cudaStream_t stream) {
+  using namespace oslo;
+  if (rows <= 0 || cols <= 0) return 0;
+  if (rows > 0x7fffffffll) return -1;
+  const size_t xe = x_fp32 ? 4 : (dtype == OSLO_DT_FP32 ? 4 : 2), te = dtype == OSLO_DT_FP32 ? 4 : 2;
+  const bool vec = cols % 4 == 0 && ldx % 4 == 0 && ldo % 4 == 0 && aligned_to(x, 4 * xe) && aligned_to(w, 4 * te) &&
+                   aligned_to(out, 4 * te);
+  OSLO_DISPATCH_T(dtype, {
+    if (x_fp32) {
+      if (vec) rms_norm_launch<float, T, 4>(x, ldx, w, out, ldo, rows, cols, eps, offset, stream);
+      else rms_norm_launch<float, T, 1>(x, ldx, w, out, ldo, rows, cols, eps, offset, stream);
+    } else {
+      if (vec) rms_norm_launch<T, T, 4>(x, ldx, w, out, ldo, rows, cols, eps, offset, stream);
+      else rms_norm_launch<T, T, 1>(x, ldx, w, out, ldo, rows, cols, eps, offset, stream);
+    }
+  });
+  return static_cast<int>(cudaGetLastError());
+}
+
+extern "C" int oslo_residual_join(const float* x, const void* y, long long ldy, const int* slots, const float* slot_weights,
+                                  int top, const void* gate, long long ldg, const void* gate_bias, const void* w_post,
+                                  const void* w_next, float* x_out, void* h_out, long long rows, int cols, float eps,
+                                  int dtype, cudaStream_t stream) {
+  using namespace oslo;
+  if (rows <= 0 || cols <= 0) return 0;
+  if (rows > 0x7fffffffll) return -1;
+  JoinParams p{x, y, ldy, slots, slot_weights, top, gate, ldg, gate_bias, w_post, w_next, x_out, h_out, cols, eps};
+  const size_t te = dtype == OSLO_DT_FP32 ? 4 : 2;
+  const bool vec = cols % 4 == 0 && ldy % 4 == 0 && ldg % 4 == 0 && aligned_to(x, 16) && aligned_to(x_out, 16) &&
+                   aligned_to(y, 4 * te) && aligned_to(gate, 4 * te) && aligned_to(gate_bias, 4 * te) &&
+                   aligned_to(w_post, 4 * te) && (w_next == nullptr || (aligned_to(w_next, 4 * te) && aligned_to(h_out, 4 * te)));
+  const size_t smem = static_cast<size_t>(cols) * sizeof(float);
+  if (smem > 200 * 1024) return -3;
+  const int threads = cols >= 1024 ? 256 : (cols >= 512 ? 128 : 64);
+#define JOIN_GO(V)                                                                                                 \
+  {                                                                                                                \
+    if (smem > 48 * 1024) {                                                                                        \
+      cudaError_t e = cudaFuncSetAttribute(residual_join_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
+                                           static_cast<int>(smem));                                                \
+      if (e != cudaSuccess) return static_cast<int>(e);                                                            \
+    }                                                                                                              \
+    residual_join_kernel<T, V><<<static_cast<unsigned>(rows), threads, smem, stream>>>(p);                         \
+  }
+  OSLO_DISPATCH_T(dtype, { if (vec) JOIN_GO(4) else JOIN_GO(1) });
+#undef JOIN_GO
+  return static_cast<int>(cudaGetLastError());
+}
+
+extern "C" int oslo_silu_mul(const void* gate, long long ldg, const void* up, long long ldu, void* out, long long rows,
+                             int cols, int dtype, cudaStream_t stream) {
+  using namespace oslo;
+  if (rows <= 0 || cols <= 0) return 0;
+  const size_t te = dtype == OSLO_DT_FP32 ? 4 : 2;
+  const bool vec = cols % 4 == 0 && ldg % 4 == 0 && ldu % 4 == 0 && aligned_to(gate, 4 * te) && aligned_to(up, 4 * te) &&
+                   aligned_to(out, 4 * te);
+  const long long work = rows * (vec ? cols / 4 : cols);
+  const unsigned blocks = static_cast<unsigned>(std::min<long long>((work + 255) / 256, 148 * 16));
+  OSLO_DISPATCH_T(dtype, {
+    if (vec) silu_mul_kernel<T, 4><<<blocks, 256, 0, stream>>>(static_cast<const T*>(gate), ldg, static_cast<const T*>(up), ldu,
+                                                               static_cast<T*>(out), rows, cols);
+    else silu_mul_kernel<T, 1><<<blocks, 256, 0, stream>>>(static_cast<const T*>(gate), ldg, static_cast<const T*>(up), ldu,
+                                                           static_cast<T*>(out), rows, cols);
+  });
+  return static_cast<int>(cudaGetLastError());
+}

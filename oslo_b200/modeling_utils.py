@@ -357,9 +357,14 @@ class PreTrainedModel(nn.Module, ParallelizationMixin, FusedKernelMixin, Generat
         model.eval()
         return model
 
+    def convert_checkpoint(self, state_dict: Dict[str, torch.Tensor]) -> Dict[str, torch.Tensor]:
+        """Hook for families whose published checkpoints use other tensor names or layouts than their modules."""
+        return state_dict
+
     def load_checkpoint_state(self, state_dict: Dict[str, torch.Tensor], strict: bool = False):
         """``load_state_dict`` that tolerates the base-model prefix being present or absent and
         drops legacy buffers (``attn.bias`` / ``attn.masked_bias``) found in old HF files."""
+        state_dict = self.convert_checkpoint(state_dict)
         own = self.state_dict()
         prefix = self.base_model_prefix + "."
         has_prefix_model = any(k.startswith(prefix) for k in own)

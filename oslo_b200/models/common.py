@@ -1,4 +1,4 @@
-"""Shared decoder-only transformer machinery for the GPT-2 / GPT-Neo / GPT-J families.
+"""Shared decoder-only transformer machinery of the model families.
 
 Each family supplies its modules under the HF parameter names; this file supplies the attention
 core (eager library path and fused flash / decode-kernel path), the static KV cache, and the
@@ -22,18 +22,26 @@ from ..modeling_utils import (BaseModelOutputWithPast, CausalLMOutputWithPast, P
 
 
 class StaticKVCache:
-    """Pre-allocated key/value cache ``[layers][B, heads, T_max, D]`` written in place.
+    """Pre-allocated cache written in place. Per layer it holds whichever of these the layer's mixer needs:
+
+    * ``k`` / ``v``: keys and values ``[B, heads, T_max, D]``;
+    * ``latent``: one low-rank vector per token ``[B, T_max, rank]`` (latent attention; layers may read another layer's);
+    * ``state``: a recurrent state of fixed size in fp32, first dim ``B`` (linear recurrences).
 
     Replaces the grow-by-``torch.cat`` cache of the reference (oslo/models/gptj/modeling_gptj.py:239-248):
     appends are slice writes, beam reordering is one ``index_select`` per tensor, and the decode
-    attention kernel reads the first ``length`` positions.
+    attention kernels read the first ``length`` positions. ``grow=True``: a full cache is enlarged instead of
+    refusing the append (storage moves, so not under a captured graph).
     """
 
-    def __init__(self, max_len: int) -> None:
+    def __init__(self, max_len: int, grow: bool = False) -> None:
         self.k: Dict[int, Tensor] = {}
         self.v: Dict[int, Tensor] = {}
+        self.latent: Dict[int, Tensor] = {}
+        self.state: Dict[int, Tensor] = {}
         self.length = 0
         self.max_len = int(max_len)
+        self.grow = bool(grow)
         self.lengths_dev: Optional[Tensor] = None
         self.lengths_next: Optional[Tensor] = None
         # device-position mode (CUDA-graph decoding): single-token appends are index_copy_ at a position kept
@@ -61,23 +69,41 @@ class StaticKVCache:
         """Forget the contents (storage is kept) so the cache can take a new prompt."""
         self.length = 0
         self.device_positions = False
+        for s in self.state.values():
+            s.zero_()
         if self.lengths_dev is not None:
             self.lengths_dev.zero_()
             self.lengths_next.fill_(1)
+
+    def _ensure_lengths(self, b: int, device) -> None:
+        if self.lengths_dev is None:
+            self.lengths_dev = torch.full((b,), self.length, dtype=torch.int32, device=device)
+            self.lengths_next = self.lengths_dev + 1
+
+    def _reserve(self, end: int) -> None:
+        if end <= self.max_len:
+            return
+        if not self.grow or self.device_positions:
+            raise RuntimeError(f"KV cache overflow: {end} > {self.max_len}")
+        self.max_len = max(end, 2 * self.max_len)
+        for store, dim in ((self.k, 2), (self.v, 2), (self.latent, 1)):
+            for i, t in store.items():
+                shape = list(t.shape)
+                shape[dim] = self.max_len
+                new = t.new_zeros(shape)
+                new.narrow(dim, 0, t.size(dim)).copy_(t)
+                store[i] = new
 
     def append(self, layer: int, k: Tensor, v: Tensor) -> Tuple[Tensor, Tensor, int]:
         """Write ``k, v`` (``[B, heads, S, D]``) at the current position; returns the whole cache
         tensors of that layer and the new valid length. Storage is allocated on first use per layer."""
         b, h, s, d = k.shape
+        end = self.length + s
+        self._reserve(end)
         if layer not in self.k:
             self.k[layer] = torch.zeros(b, h, self.max_len, d, dtype=k.dtype, device=k.device)
             self.v[layer] = torch.zeros(b, h, self.max_len, d, dtype=v.dtype, device=v.device)
-        if self.lengths_dev is None:
-            self.lengths_dev = torch.full((b,), self.length, dtype=torch.int32, device=k.device)
-            self.lengths_next = self.lengths_dev + 1
-        end = self.length + s
-        if end > self.max_len:
-            raise RuntimeError(f"KV cache overflow: {end} > {self.max_len}")
+        self._ensure_lengths(b, k.device)
         if self.device_positions and s == 1:
             self.k[layer].index_copy_(2, self.write_index, k)
             self.v[layer].index_copy_(2, self.write_index, v)
@@ -86,6 +112,31 @@ class StaticKVCache:
         self.k[layer][:, :, self.length:end].copy_(k)
         self.v[layer][:, :, self.length:end].copy_(v)
         return self.k[layer], self.v[layer], end
+
+    def latent_storage(self, layer: int, b: int, rank: int, dtype: torch.dtype, device, new_tokens: int) -> Tensor:
+        """Latents ``[B, T_max, rank]`` of ``layer`` with room for ``new_tokens`` more; position ``length`` is the next one."""
+        self._reserve(self.length + new_tokens)
+        if layer not in self.latent:
+            self.latent[layer] = torch.zeros(b, self.max_len, rank, dtype=dtype, device=device)
+        self._ensure_lengths(b, device)
+        return self.latent[layer]
+
+    def append_latent(self, layer: int, c: Tensor) -> Tensor:
+        """Write ``c`` (``[B, S, rank]``) at the current position; returns the valid part of the layer's latents."""
+        b, s, r = c.shape
+        store = self.latent_storage(layer, b, r, c.dtype, c.device, s)
+        if self.device_positions and s == 1:
+            store.index_copy_(1, self.write_index, c)
+        else:
+            store[:, self.length:self.length + s].copy_(c)
+        return store[:, :self.length + s]
+
+    def recurrent_state(self, layer: int, shape, device) -> Tensor:
+        """The fp32 state of ``layer`` (zero for a new sequence), to be updated in place."""
+        if layer not in self.state:
+            self.state[layer] = torch.zeros(*shape, dtype=torch.float32, device=device)
+        self._ensure_lengths(shape[0], device)
+        return self.state[layer]
 
     def advance(self, s: int) -> None:
         self.length += s
@@ -98,9 +149,11 @@ class StaticKVCache:
         return self.length
 
     def reorder(self, beam_idx: Tensor) -> "StaticKVCache":
-        for i in list(self.k.keys()):
-            self.k[i] = self.k[i].index_select(0, beam_idx)
-            self.v[i] = self.v[i].index_select(0, beam_idx)
+        """Row ``i`` becomes the old row ``beam_idx[i]``: beams that move, or the rows of a batch that go on while the others
+        have ended (their share of the storage is given back)."""
+        for store in (self.k, self.v, self.latent, self.state):
+            for i in list(store.keys()):
+                store[i] = store[i].index_select(0, beam_idx)
         if self.lengths_dev is not None and beam_idx.numel() != self.lengths_dev.numel():
             self.lengths_dev = self.lengths_dev[:1].expand(beam_idx.numel()).contiguous()
             self.lengths_next = self.lengths_next[:1].expand(beam_idx.numel()).contiguous()

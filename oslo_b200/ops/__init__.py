@@ -70,12 +70,14 @@ def use_kernels(x: Tensor) -> bool:
 from .functional import (  # noqa: E402
     linear, layer_norm, bias_gelu, bias_dropout_residual, rotary_interleaved, attention,
     scaled_upper_triang_masked_softmax, scaled_masked_softmax, cross_entropy, linear_cross_entropy,
-    ban_repeated_ngrams, decode_attention,
+    ban_repeated_ngrams, decode_attention, rms_norm, residual_join, silu_mul, gated_recurrence, sink_attention,
+    latent_decode, moe_route, moe_experts,
 )
 
 __all__ = [
     "reference", "load_ext", "kernels_available", "use_kernels", "linear", "layer_norm", "bias_gelu",
     "bias_dropout_residual", "rotary_interleaved", "attention", "scaled_upper_triang_masked_softmax",
     "scaled_masked_softmax", "cross_entropy", "linear_cross_entropy", "ban_repeated_ngrams",
-    "decode_attention",
+    "decode_attention", "rms_norm", "residual_join", "silu_mul", "gated_recurrence", "sink_attention", "latent_decode",
+    "moe_route", "moe_experts",
 ]

@@ -617,3 +617,95 @@ def ban_repeated_ngrams(tokens: Tensor, lprobs: Tensor, n: int) -> Tensor:
     if lprobs.dtype != torch.float32 or not lprobs.is_contiguous():
         return ref.ban_repeated_ngrams(tokens, lprobs, n)
     return _ext().ngram_ban_(tokens.to(torch.long).contiguous(), lprobs, int(n))
+
+
+# ---------------------------------------------------------------------------------------------------------------
+# RMS norms, residual joins, gated recurrence, latent attention, mixture of experts (forward only)
+def _rows(t: Tensor) -> Tensor:
+    return t if t.stride(-1) == 1 else t.contiguous()
+
+
+def _keep8(keep: Optional[Tensor]) -> Optional[Tensor]:
+    if keep is None or keep.dtype == torch.uint8:
+        return keep
+    return (keep != 0).to(torch.uint8)
+
+
+def rms_norm(x: Tensor, w: Tensor, eps: float, offset: float) -> Tensor:
+    if x.dtype not in (w.dtype, torch.float32):
+        x = x.to(w.dtype)
+    return _ext().rms_norm(_rows(x.reshape(-1, x.size(-1))), w, float(eps), float(offset)).view(x.shape)
+
+
+def residual_join(x: Tensor, y: Tensor, gate: Tensor, gate_bias: Tensor, w_post: Tensor, w_next: Optional[Tensor], eps: float,
+                  slots: Optional[Tensor], slot_weights: Optional[Tensor]):
+    xo, h = _ext().residual_join(x.contiguous(), _rows(y), slots, slot_weights, _rows(gate), gate_bias, w_post, w_next, float(eps))
+    return xo, (h if w_next is not None else None)
+
+
+def silu_mul(gate: Tensor, up: Tensor) -> Tensor:
+    return _ext().silu_mul(_rows(gate), _rows(up))
+
+
+def gated_recurrence(q: Tensor, f: Tensor, v: Tensor, f_bias: Tensor, lower: Tensor, norm_w: Tensor, eps: float, batch: int,
+                     heads: int, keep: Optional[Tensor], state: Optional[Tensor]) -> Tensor:
+    dim, vdim = q.size(1) // heads, v.size(1) // heads
+    if q.size(0) == batch and state is not None:      # one token per sequence
+        return _ext().recurrence_step(_rows(q), _rows(f), _rows(v), f_bias, lower, norm_w, _keep8(keep), state, float(eps), heads,
+                                      dim, vdim)
+    o = _ext().recurrence(_rows(q), _rows(f), _rows(v), f_bias, lower, _keep8(keep), state, batch, heads, dim, vdim)
+    return _ext().rms_norm(o.view(-1, vdim), norm_w, float(eps), 0.0).view(-1, heads * vdim)
+
+
+def flash_head_dim(dim: int, vdim: int) -> int:
+    """Head size at which the tcgen05 flash kernel can run heads of ``dim`` / ``vdim`` (0: none)."""
+    return next((d for d in (64, 128, 256) if d >= max(dim, vdim)), 0)
+
+
+def pad_heads(t: Tensor, d: int) -> Tensor:
+    """``[B, S, H, dim] -> [B, S, H, d]``, zero-padded (no copy when the size already fits)."""
+    return t if t.size(-1) == d else torch.nn.functional.pad(t, (0, d - t.size(-1)))
+
+
+def sink_attention(q: Tensor, k: Tensor, v: Tensor, keep: Optional[Tensor], sink: Tensor, gate: Tensor, scale: float) -> Tensor:
+    """``q``/``k``/``v`` ``[B, S, H, *]``. 16-bit heads run on the tcgen05 flash kernel (zero-padded to the next size it has),
+    whose log-sum-exp the sink and the gate are applied with; everything else in the fp32 kernel."""
+    d = flash_head_dim(q.size(-1), v.size(-1))
+    if q.dtype in _16BIT and d and q.size(1) > 1:
+        qh, kh, vh = (_attn_operand(pad_heads(t, d).permute(0, 2, 1, 3)) for t in (q, k, v))
+        o, lse = _ext().flash_fwd(qh, kh, vh, float(scale), True, 0, _keep8(keep).contiguous() if keep is not None else None,
+                                  _flash_impl())
+        return _ext().sink_gate(o, lse, sink, _rows(gate), v.size(-1))
+    return _ext().sink_attention(*(t if t.stride(-1) == 1 else t.contiguous() for t in (q, k, v)), _keep8(keep), sink,
+                                 _rows(gate), float(scale))
+
+
+def latent_prep(cq: Tensor, wq: Tensor, ckv: Optional[Tensor], wkv: Optional[Tensor], cache: Optional[Tensor], lengths: Tensor,
+                eps: float) -> Tensor:
+    """Decode step: the normed query latent; the normed key-value latent goes into ``cache`` at position ``lengths[row]``."""
+    return _ext().latent_prep(_rows(cq), wq, None if ckv is None else _rows(ckv), wkv, cache, lengths, float(eps))
+
+
+def latent_decode(q: Tensor, w_uk: Tensor, w_uv: Tensor, cache: Tensor, lengths: Tensor, keep: Optional[Tensor], sink: Tensor,
+                  gate: Tensor, scale: float, heads: int) -> Tensor:
+    return _ext().latent_decode(_rows(q), w_uk, w_uv, cache, lengths.to(torch.int32), _keep8(keep), sink, _rows(gate),
+                                float(scale), heads)
+
+
+MOE_FEW_ROWS = 16   # token rows up to which the chosen experts' weights are streamed per (token, choice)
+
+
+def moe_route(h: Tensor, w: Tensor, bias: Tensor, top: int):
+    logits = None
+    if h.size(0) > SMALL_M_ROWS and gemm_ok(h, w) and h.size(1) % 8 == 0:
+        logits = gemm(h, w, flags=FLAG_OUT_FP32)           # 16-bit operands, exact products, fp32 sums and output
+    return _ext().moe_route(_rows(h), w, bias, logits, top)
+
+
+def moe_experts(h: Tensor, idx: Tensor, up: Tensor, down: Tensor):
+    if h.size(0) <= MOE_FEW_ROWS:
+        a = _ext().moe_few(_rows(h), idx, up, idx.size(1), True)
+        return _ext().moe_few(a, idx, down, 1, False), None
+    slots, rows, tile_group, n_tiles = _ext().moe_plan(_rows(h), idx, up.size(0))
+    a = _ext().moe_grouped(rows, up, tile_group, n_tiles, True)
+    return _ext().moe_grouped(a, down, tile_group, n_tiles, False), slots

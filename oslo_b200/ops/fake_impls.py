@@ -173,3 +173,56 @@ def register() -> None:
     def _(like, peer_ptrs_dev, mc_ptr, signal_ptrs_dev, lo, hi, shard, rank, world, use_multimem):
         return None
 
+
+    @reg("oslo_b200::rms_norm")
+    def _(x, w, eps, offset):
+        return w.new_empty(x.shape)
+
+    @reg("oslo_b200::residual_join")
+    def _(x, y, slots, slot_weights, gate, gate_bias, w_post, w_next, eps):
+        return torch.empty_like(x), y.new_empty((x.size(0) if w_next is not None else 0, x.size(1)))
+
+    @reg("oslo_b200::silu_mul")
+    def _(gate, up):
+        return gate.new_empty(gate.shape)
+
+    @reg("oslo_b200::recurrence")
+    def _(q, f, v, f_bias, lower, keep, state, batch, heads, dim, vdim, chunks=0):
+        return q.new_empty((batch, q.size(0) // batch, heads, vdim), dtype=torch.float32)
+
+    @reg("oslo_b200::recurrence_step")
+    def _(q, f, v, f_bias, lower, norm_w, keep, state, eps, heads, dim, vdim):
+        return q.new_empty((q.size(0), heads * vdim))
+
+    @reg("oslo_b200::sink_gate")
+    def _(o, lse, sink, gate, vdim):
+        return o.new_empty((o.size(0) * o.size(2), o.size(1) * vdim))
+
+    @reg("oslo_b200::sink_attention")
+    def _(q, k, v, keep, sink, gate, scale):
+        return q.new_empty((q.size(0) * q.size(1), q.size(2) * v.size(3)))
+
+    @reg("oslo_b200::latent_prep")
+    def _(cq, wq, ckv, wkv, cache, lengths, eps):
+        return cq.new_empty(cq.shape)
+
+    @reg("oslo_b200::latent_decode")
+    def _(q, w_uk, w_uv, cache, lengths, keep, sink, gate, scale, heads):
+        return q.new_empty((q.size(0), w_uv.size(0)))
+
+    @reg("oslo_b200::moe_route")
+    def _(h, w, bias, logits, top):
+        return h.new_empty((h.size(0), top), dtype=torch.int32), h.new_empty((h.size(0), top), dtype=torch.float32)
+
+    @reg("oslo_b200::moe_plan")
+    def _(h, idx, experts):
+        tiles = (idx.numel() + 127) // 128 + min(experts, idx.numel())
+        return (torch.empty_like(idx), h.new_empty((tiles * 128, h.size(1))), idx.new_empty((tiles,)), idx.new_empty((1,)))
+
+    @reg("oslo_b200::moe_grouped")
+    def _(rows, w, tile_group, n_tiles, relu2):
+        return rows.new_empty((rows.size(0), w.size(1)))
+
+    @reg("oslo_b200::moe_few")
+    def _(x, idx, w, per_row, relu2):
+        return x.new_empty((idx.numel(), w.size(1)))

@@ -2,7 +2,7 @@
 from __future__ import annotations
 
 import math
-from typing import Optional
+from typing import Optional, Tuple
 
 import torch
 from torch import Tensor
@@ -145,3 +145,83 @@ def ban_repeated_ngrams(tokens: Tensor, lprobs: Tensor, n: int) -> Tensor:
         from . import cuda_ops
         return cuda_ops.ban_repeated_ngrams(tokens, lprobs, n)
     return ref.ban_repeated_ngrams(tokens, lprobs, n)
+
+
+# ---------------------------------------------------------------------------------------------------------------
+# The kernels behind the functions below have no backward: with gradients on, the differentiable statement runs.
+def _kn(x: Tensor, *others: Optional[Tensor]) -> bool:
+    if torch.is_grad_enabled() and (x.requires_grad or any(t is not None and t.requires_grad for t in others)):
+        return False
+    return _k(x)
+
+
+def rms_norm(x: Tensor, w: Tensor, eps: float, offset: float = 0.0) -> Tensor:
+    """``x / sqrt(mean(x^2) + eps) * (offset + w)`` with fp32 math, in ``w``'s dtype; ``x`` is fp32 or has ``w``'s dtype."""
+    if _kn(x, w):
+        from . import cuda_ops
+        return cuda_ops.rms_norm(x, w, eps, offset)
+    return ref.rms_norm(x, w, eps, offset)
+
+
+def residual_join(x: Tensor, y: Tensor, gate: Tensor, gate_bias: Tensor, w_post: Tensor, w_next: Optional[Tensor],
+                  eps: float, slots: Optional[Tensor] = None,
+                  slot_weights: Optional[Tensor] = None) -> Tuple[Tensor, Optional[Tensor]]:
+    """Gate a sublayer's result, norm it, add it to the fp32 residual stream and norm the sum for the next sublayer: one
+    pass over the rows. See ``reference.residual_join``."""
+    if _kn(x, y, gate, gate_bias, w_post, w_next, slot_weights):
+        from . import cuda_ops
+        return cuda_ops.residual_join(x, y, gate, gate_bias, w_post, w_next, eps, slots, slot_weights)
+    return ref.residual_join(x, y, gate, gate_bias, w_post, w_next, eps, slots, slot_weights)
+
+
+def silu_mul(gate: Tensor, up: Tensor) -> Tensor:
+    if _kn(gate, up):
+        from . import cuda_ops
+        return cuda_ops.silu_mul(gate, up)
+    return ref.silu_mul(gate, up)
+
+
+def gated_recurrence(q: Tensor, f: Tensor, v: Tensor, f_bias: Tensor, lower: Tensor, norm_w: Tensor, eps: float, batch: int,
+                     heads: int, keep: Optional[Tensor] = None, state: Optional[Tensor] = None) -> Tensor:
+    """``reference.recurrence`` followed by the RMS norm of every head's output; ``state`` (fp32, updated in place) carries the
+    sequence on. ``[batch * S, heads * vdim]`` in ``norm_w``'s dtype."""
+    if _kn(q, f, v, f_bias, lower, norm_w):
+        from . import cuda_ops
+        return cuda_ops.gated_recurrence(q, f, v, f_bias, lower, norm_w, eps, batch, heads, keep, state)
+    dim, vdim = q.size(1) // heads, v.size(1) // heads
+    o, final = ref.recurrence(q, f, v, f_bias, lower, keep, state, batch, heads, dim, vdim)
+    if state is not None:
+        state.copy_(final.detach())
+    return ref.rms_norm(o, norm_w, eps).reshape(-1, heads * vdim)
+
+
+def sink_attention(q: Tensor, k: Tensor, v: Tensor, keep: Optional[Tensor], sink: Tensor, gate: Tensor, scale: float) -> Tensor:
+    """``reference.sink_attention`` without the weights."""
+    if _kn(q, k, v, sink, gate):
+        from . import cuda_ops
+        return cuda_ops.sink_attention(q, k, v, keep, sink, gate, scale)
+    return ref.sink_attention(q, k, v, keep, sink, gate, scale)[0]
+
+
+def latent_decode(q: Tensor, w_uk: Tensor, w_uv: Tensor, cache: Tensor, lengths: Tensor, keep: Optional[Tensor], sink: Tensor,
+                  gate: Tensor, scale: float, heads: int) -> Tensor:
+    if _kn(q, w_uk, w_uv, cache, sink, gate):
+        from . import cuda_ops
+        return cuda_ops.latent_decode(q, w_uk, w_uv, cache, lengths, keep, sink, gate, scale, heads)
+    return ref.latent_decode(q, w_uk, w_uv, cache, lengths, keep, sink, gate, scale, heads)
+
+
+def moe_route(h: Tensor, w: Tensor, bias: Tensor, top: int) -> Tuple[Tensor, Tensor]:
+    if _kn(h, w, bias):
+        from . import cuda_ops
+        return cuda_ops.moe_route(h, w, bias, top)
+    return ref.moe_route(h, w, bias, top)
+
+
+def moe_experts(h: Tensor, idx: Tensor, up: Tensor, down: Tensor) -> Tuple[Tensor, Optional[Tensor]]:
+    """``W_down relu(W_up h)^2`` of the chosen experts, one row per (token, choice), and where those rows are
+    (``None``: row ``token * top + choice``); ``residual_join`` adds them up."""
+    if _kn(h, up, down):
+        from . import cuda_ops
+        return cuda_ops.moe_experts(h, idx, up, down)
+    return ref.moe_experts(h, idx, up, down), None

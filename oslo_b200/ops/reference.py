@@ -176,3 +176,116 @@ def ban_repeated_ngrams(tokens: Tensor, lprobs: Tensor, n: int) -> Tensor:
         if banned:
             lprobs[r, banned] = float("-inf")
     return lprobs
+
+
+# ---------------------------------------------------------------------------------------------------------------
+# RMS norms, gated residual joins, gated linear recurrence, latent attention with a sink, mixture of experts. All of them
+# compute in fp32 and are differentiable; rows are tokens ([batch * positions, features]) unless stated otherwise.
+def rms_norm(x: Tensor, w: Tensor, eps: float, offset: float = 0.0) -> Tensor:
+    """``x / sqrt(mean(x^2) + eps) * (offset + w)`` over the last dim, in ``w``'s dtype (``offset=1``: the weight is stored
+    around zero)."""
+    xf = x.to(torch.float32)
+    r = torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps)
+    return (xf * r * (offset + w.to(torch.float32))).to(w.dtype)
+
+
+def residual_join(x: Tensor, y: Tensor, gate: Tensor, gate_bias: Tensor, w_post: Tensor, w_next: Optional[Tensor],
+                  eps: float, slots: Optional[Tensor] = None, slot_weights: Optional[Tensor] = None):
+    """``x + norm(y * sigmoid(gate + gate_bias))`` in fp32, and the norm of that for the next sublayer (or ``None``). With
+    ``slot_weights`` ``[tokens, top]`` the sublayer's result is the weighted sum of ``y``'s rows ``slots``
+    (``token * top + choice`` when ``slots`` is ``None``)."""
+    yf = y.to(torch.float32)
+    if slot_weights is not None:
+        n, top = slot_weights.shape
+        picked = yf.view(n, top, -1) if slots is None else yf[slots.reshape(-1).to(torch.long)].view(n, top, -1)
+        yf = (picked * slot_weights.unsqueeze(-1)).sum(1)
+    z = yf * torch.sigmoid(gate.to(torch.float32) + gate_bias.to(torch.float32))
+    r = torch.rsqrt(z.pow(2).mean(-1, keepdim=True) + eps)
+    x = x + z * r * (1.0 + w_post.to(torch.float32))
+    return x, (rms_norm(x, w_next, eps, 1.0) if w_next is not None else None)
+
+
+def silu_mul(gate: Tensor, up: Tensor) -> Tensor:
+    return F.silu(gate.to(torch.float32)).mul(up.to(torch.float32)).to(up.dtype)
+
+
+def recurrence(q: Tensor, f: Tensor, v: Tensor, f_bias: Tensor, lower: Tensor, keep: Optional[Tensor],
+               state: Optional[Tensor], batch: int, heads: int, dim: int, vdim: int) -> Tuple[Tensor, Tensor]:
+    """Linear attention whose forget gate also decides what is written: per head and key channel
+    ``1 - k = lower + (1 - lower) sigmoid(f + f_bias)``, ``S <- S + k (v - S)``, ``o = S^T silu(q)``.
+
+    ``q``/``f`` ``[batch * S, heads * dim]``, ``v`` ``[batch * S, heads * vdim]``; ``keep`` ``[batch, S]`` (0: the token leaves
+    the state alone and its output is 0); ``state`` ``[batch, heads, dim, vdim]`` fp32 or ``None`` (zero). Returns
+    ``[batch, S, heads, vdim]`` in fp32 and the final state."""
+    lo = lower.to(torch.float32)
+    k = ((1.0 - lo) * torch.sigmoid(-(f.to(torch.float32) + f_bias.to(torch.float32)))).view(batch, -1, heads, dim)
+    qs = F.silu(q.to(torch.float32)).view(batch, -1, heads, dim)
+    vf = v.to(torch.float32).reshape(batch, -1, heads, vdim)
+    if keep is not None:
+        on = (keep != 0).to(torch.float32)[:, :, None, None]
+        k, qs = k * on, qs * on
+    s = torch.zeros(batch, heads, dim, vdim, dtype=torch.float32, device=q.device) if state is None else state
+    out = []
+    for t in range(k.size(1)):
+        s = s + k[:, t].unsqueeze(-1) * (vf[:, t].unsqueeze(-2) - s)
+        out.append(torch.einsum("bhi,bhij->bhj", qs[:, t], s))
+    return torch.stack(out, dim=1), s
+
+
+def sink_attention(q: Tensor, k: Tensor, v: Tensor, keep: Optional[Tensor], sink: Tensor, gate: Tensor, scale: float):
+    """Causal softmax attention whose denominator also holds ``exp(sink[head])``; head ``h``'s output times
+    ``sigmoid(gate[:, h])``. ``q`` ``[B, Sq, H, D]`` are the last positions of ``k``/``v`` ``[B, Sk, H, *]``; ``keep``
+    ``[B, Sk]``; ``gate`` ``[B * Sq, H]``. Returns ``[B * Sq, H * Dv]`` and the weights ``[B, H, Sq, Sk]``."""
+    b, sq, h, _ = q.shape
+    sk = k.size(1)
+    s = torch.einsum("bqhd,bkhd->bhqk", q.to(torch.float32), k.to(torch.float32)) * scale
+    vis = attention_mask_bias(sq, sk, q.device, True, None)[None, None]
+    if keep is not None:
+        vis = vis & (keep != 0)[:, None, None, :]
+    s = s.masked_fill(~vis, float("-inf"))
+    s = torch.cat([s, sink.to(torch.float32)[None, :, None, None].expand(b, h, sq, 1)], dim=-1)
+    p = torch.softmax(s, dim=-1)[..., :sk]
+    o = torch.einsum("bhqk,bkhd->bqhd", p, v.to(torch.float32))
+    o = o * torch.sigmoid(gate.to(torch.float32)).view(b, sq, h, 1)
+    return o.reshape(b * sq, -1).to(q.dtype), p
+
+
+def latent_decode(q: Tensor, w_uk: Tensor, w_uv: Tensor, cache: Tensor, lengths: Tensor, keep: Optional[Tensor],
+                  sink: Tensor, gate: Tensor, scale: float, heads: int) -> Tensor:
+    """One query per row over a cache of latents ``[B, T, rank]`` without expanding keys or values: the query takes
+    ``W_uk``, the weighted sum of latents takes ``W_uv``. ``q`` ``[B, heads * dim]``; returns ``[B, heads * vdim]``."""
+    b, t, r = cache.shape
+    c = cache.to(torch.float32)
+    qa = torch.einsum("bhd,hdr->bhr", q.to(torch.float32).view(b, heads, -1), w_uk.to(torch.float32).view(heads, -1, r)) * scale
+    s = torch.einsum("bhr,btr->bht", qa, c)
+    vis = torch.arange(t, device=q.device)[None, :] < lengths[:, None]
+    if keep is not None:
+        vis = vis.clone()
+        n = min(t, keep.size(1))
+        vis[:, :n] &= keep[:, :n] != 0
+    s = s.masked_fill(~vis[:, None, :], float("-inf"))
+    s = torch.cat([s, sink.to(torch.float32)[None, :, None].expand(b, heads, 1)], dim=-1)
+    p = torch.softmax(s, dim=-1)[..., :t]
+    o = torch.einsum("bhr,hvr->bhv", torch.einsum("bht,btr->bhr", p, c), w_uv.to(torch.float32).view(heads, -1, r))
+    return (o * torch.sigmoid(gate.to(torch.float32)).unsqueeze(-1)).reshape(b, -1).to(q.dtype)
+
+
+def moe_route(h: Tensor, w: Tensor, bias: Tensor, top: int) -> Tuple[Tensor, Tensor]:
+    """The ``top`` experts with the largest ``W h + b`` per token (``[tokens, top]``, int32) and the softmax over those logits."""
+    z = torch.matmul(h.to(torch.float32), w.to(torch.float32).t()) + bias.to(torch.float32)
+    picked, idx = torch.topk(z, top, dim=-1)
+    return idx.to(torch.int32), torch.softmax(picked, dim=-1)
+
+
+def moe_experts(h: Tensor, idx: Tensor, up: Tensor, down: Tensor) -> Tensor:
+    """``W_down relu(W_up h)^2`` of every (token, choice): ``[tokens * top, width]``; ``up`` ``[experts, ff, width]``,
+    ``down`` ``[experts, width, ff]``."""
+    n, top = idx.shape
+    flat = idx.reshape(-1).to(torch.long)
+    rows = h.repeat_interleave(top, dim=0)
+    out = h.new_zeros(n * top, down.size(1))
+    for e in flat.unique().tolist():
+        at = (flat == e).nonzero(as_tuple=True)[0]
+        a = torch.relu(torch.matmul(rows[at], up[e].t())).pow(2)
+        out = out.index_copy(0, at, torch.matmul(a, down[e].t()).to(out.dtype))
+    return out

@@ -8,7 +8,7 @@ oslo/parallelism/engine_tensor.py:439-446).
 """
 from __future__ import annotations
 
-from typing import Optional
+from typing import Dict, Optional
 
 import torch
 import torch.nn as nn
@@ -74,6 +74,57 @@ class LayerNorm(nn.LayerNorm):
         if self.oslo_fused:
             return ops.layer_norm(x, self.weight, self.bias, self.eps)
         return F.layer_norm(x, self.normalized_shape, self.weight, self.bias, self.eps)
+
+
+class RMSNorm(nn.Module):
+    """``x / sqrt(mean(x^2) + eps) * (offset + weight)``, fp32 arithmetic, result in the weight's dtype. ``offset=1``: the
+    weight is stored around zero."""
+
+    oslo_fused = False
+
+    def __init__(self, dim: int, eps: float, offset: float = 0.0) -> None:
+        super().__init__()
+        self.eps, self.offset = float(eps), float(offset)
+        self.weight = nn.Parameter(torch.full((dim,), 1.0 - offset))
+
+    def forward(self, x: Tensor) -> Tensor:
+        fn = ops.rms_norm if self.oslo_fused else ops.reference.rms_norm
+        return fn(x, self.weight, self.eps, self.offset)
+
+
+class PackedLinear(Linear):
+    """Several bias-free projections of one input as one weight ``[sum of sizes, in]`` and one GEMM. Every part starts at a
+    multiple of ``ALIGN`` rows, so that the slices of the result stay aligned; the rows in between are never read.
+    ``forward`` returns ``{name: [..., size]}`` (views)."""
+
+    ALIGN = 8
+
+    def __init__(self, in_features: int, parts: Dict[str, int]) -> None:
+        self_parts, total = {}, 0
+        for name, size in parts.items():
+            self_parts[name] = (total, int(size))
+            total += -(-int(size) // self.ALIGN) * self.ALIGN
+        super().__init__(in_features, total, bias=False)
+        self.parts = self_parts
+
+    def part(self, name: str) -> Tensor:
+        start, size = self.parts[name]
+        return self.weight[start:start + size]
+
+    def pack(self, tensors: Dict[str, Tensor]) -> Tensor:
+        """The packed weight made of one tensor per part."""
+        if set(tensors) != set(self.parts):
+            raise KeyError(f"parts {sorted(self.parts)} expected, got {sorted(tensors)}")
+        out = next(iter(tensors.values())).new_zeros(self.out_features, self.in_features)
+        for name, (start, size) in self.parts.items():
+            if tuple(tensors[name].shape) != (size, self.in_features):
+                raise ValueError(f"{name}: shape {tuple(tensors[name].shape)}, expected {(size, self.in_features)}")
+            out[start:start + size] = tensors[name]
+        return out
+
+    def forward(self, x: Tensor) -> Dict[str, Tensor]:  # type: ignore[override]
+        y = super().forward(x)
+        return {name: y[..., start:start + size] for name, (start, size) in self.parts.items()}
 
 
 class Embedding(nn.Embedding):

@@ -36,6 +36,12 @@ struct FaParams {
   // position of the (seq, head, batch) coordinates inside each 4-D tensor map (dim 0 is always D)
   int q_pos[3], k_pos[3], v_pos[3];
   int* err;
+  // softmax with a sink and an output gate (both null: plain attention): exp(sink[h]) joins the denominator, row s of
+  // head h is multiplied by sigmoid(gate[(b * Sq + s) * ldg + h]); only the first d_out columns are stored
+  const void* sink;
+  const void* gate;
+  long long ldg;
+  int d_out;
 };
 
 // PT = true: P goes back into TMEM (over the S buffer it came from, two bf16 per 32-bit column) and is the
@@ -303,7 +309,16 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
       ok = mbar_wait(bar(14), (nblk - 1) & 1, abort_flag, p.err, ERR_WAIT_TMEM_FULL);
       tc_fence_after();
     }
-    const float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
+    float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
+    if (p.sink != nullptr && row < p.Sq && l_sum > 0.f) {
+      const long long gi = (static_cast<long long>(b) * p.Sq + row) * p.ldg + h;
+      const float snk = fp16 ? __half2float(static_cast<const __half*>(p.sink)[h])
+                             : __bfloat162float(static_cast<const __nv_bfloat16*>(p.sink)[h]);
+      const float gate = fp16 ? __half2float(static_cast<const __half*>(p.gate)[gi])
+                              : __bfloat162float(static_cast<const __nv_bfloat16*>(p.gate)[gi]);
+      // m_ref is the running reference in log2 units; an overflowing sink term gives 1 / inf = 0
+      inv = 1.f / ((l_sum + exp2f(snk * 1.4426950408889634f - m_ref)) * (1.f + exp2f(-gate * 1.4426950408889634f)));
+    }
     uint16_t* orow = reinterpret_cast<uint16_t*>(p.out) + b * p.o_sb + h * p.o_sh + static_cast<long long>(row) * p.o_ss;
 #pragma unroll 1
     for (int c0 = 0; c0 < D; c0 += 32) {
@@ -318,6 +333,7 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
       if (row < p.Sq) {
 #pragma unroll
         for (int i = 0; i < 32; i += 8) {
+          if (c0 + i >= p.d_out) break;
           uint4 v;
           v.x = fa_pack2(__uint_as_float(r[i]) * inv, __uint_as_float(r[i + 1]) * inv, fp16);
           v.y = fa_pack2(__uint_as_float(r[i + 2]) * inv, __uint_as_float(r[i + 3]) * inv, fp16);
@@ -365,13 +381,12 @@ static int fa_launch(const CUtensorMap& tq, const CUtensorMap& tk, const CUtenso
 
 }  // namespace oslo
 
-extern "C" int oslo_flash_fwd_sm100(const void* q, const void* k, const void* v, void* o, float* lse,
-                                    const uint8_t* kpm, int B, int H, int Sq, int Sk, int D, long long q_sb,
-                                    long long q_sh, long long q_ss, long long k_sb, long long k_sh, long long k_ss,
-                                    long long v_sb, long long v_sh, long long v_ss, long long o_sb, long long o_sh,
-                                    long long o_ss, float scale, int causal, int window, int dtype, int* err_word,
-                                    cudaStream_t stream) {
-  using namespace oslo;
+namespace oslo {
+static int flash_fwd_entry(const void* q, const void* k, const void* v, void* o, float* lse, const uint8_t* kpm,
+                           const void* sink, const void* gate, long long ldg, int d_out, int B, int H, int Sq, int Sk, int D,
+                           long long q_sb, long long q_sh, long long q_ss, long long k_sb, long long k_sh, long long k_ss,
+                           long long v_sb, long long v_sh, long long v_ss, long long o_sb, long long o_sh, long long o_ss,
+                           float scale, int causal, int window, int dtype, int* err_word, cudaStream_t stream) {
   if (B <= 0 || H <= 0 || Sq <= 0 || Sk <= 0) return -1;
   if (D != 64 && D != 128 && D != 256) return -2;
   if (dtype != OSLO_DT_BF16 && dtype != OSLO_DT_FP16) return -3;
@@ -382,6 +397,7 @@ extern "C" int oslo_flash_fwd_sm100(const void* q, const void* k, const void* v,
   const int bn = D == 256 ? 64 : 128;
   FaParams p;
   p.out = o; p.lse = lse; p.kpm = kpm;
+  p.sink = sink; p.gate = gate; p.ldg = ldg; p.d_out = d_out;
   p.B = B; p.H = H; p.Sq = Sq; p.Sk = Sk;
   p.o_sb = o_sb; p.o_sh = o_sh; p.o_ss = o_ss;
   p.scale = scale; p.causal = causal; p.window = window; p.fp16 = fp16 ? 1 : 0; p.err = err_word;
@@ -401,4 +417,26 @@ extern "C" int oslo_flash_fwd_sm100(const void* q, const void* k, const void* v,
   if (D == 64) return fa_launch<64, 128, true>(tq, tk, tv, p, stream);
   if (D == 128) return fa_launch<128, 128, true>(tq, tk, tv, p, stream);
   return fa_launch<256, 64, true>(tq, tk, tv, p, stream);
+}
+}  // namespace oslo
+
+extern "C" int oslo_flash_fwd_sm100(const void* q, const void* k, const void* v, void* o, float* lse,
+                                    const uint8_t* kpm, int B, int H, int Sq, int Sk, int D, long long q_sb,
+                                    long long q_sh, long long q_ss, long long k_sb, long long k_sh, long long k_ss,
+                                    long long v_sb, long long v_sh, long long v_ss, long long o_sb, long long o_sh,
+                                    long long o_ss, float scale, int causal, int window, int dtype, int* err_word,
+                                    cudaStream_t stream) {
+  return oslo::flash_fwd_entry(q, k, v, o, lse, kpm, nullptr, nullptr, 0, D, B, H, Sq, Sk, D, q_sb, q_sh, q_ss, k_sb, k_sh,
+                               k_ss, v_sb, v_sh, v_ss, o_sb, o_sh, o_ss, scale, causal, window, dtype, err_word, stream);
+}
+
+extern "C" int oslo_flash_sink_fwd_sm100(const void* q, const void* k, const void* v, void* o, const uint8_t* kpm,
+                                         const void* sink, const void* gate, long long ldg, int d_out, int B, int H, int Sq,
+                                         int Sk, int D, long long q_sb, long long q_sh, long long q_ss, long long k_sb,
+                                         long long k_sh, long long k_ss, long long v_sb, long long v_sh, long long v_ss,
+                                         long long o_sb, long long o_sh, long long o_ss, float scale, int dtype, int* err_word,
+                                         cudaStream_t stream) {
+  if (sink == nullptr || gate == nullptr || d_out <= 0 || d_out > D || d_out % 8) return -1;
+  return oslo::flash_fwd_entry(q, k, v, o, nullptr, kpm, sink, gate, ldg, d_out, B, H, Sq, Sk, D, q_sb, q_sh, q_ss, k_sb, k_sh,
+                               k_ss, v_sb, v_sh, v_ss, o_sb, o_sh, o_ss, scale, 1, 0, dtype, err_word, stream);
 }

@@ -868,6 +868,33 @@ Tensor sink_gate(const Tensor& o, const Tensor& lse, const Tensor& sink, const T
   return out;
 }
 
+// q, k, v [B, H, S, D] (any strides with contiguous D, D one of the flash kernel's sizes) -> [B * Sq, H * vdim]
+Tensor flash_sink_fwd(const Tensor& q, const Tensor& k, const Tensor& v, const optional<Tensor>& kpm, const Tensor& sink,
+                      const Tensor& gate, double scale, int64_t vdim) {
+  TORCH_CHECK(q.is_cuda() && q.dim() == 4 && k.dim() == 4 && v.sizes() == k.sizes() && q.stride(3) == 1 && k.stride(3) == 1 &&
+                  v.stride(3) == 1 && k.size(3) == q.size(3) && k.size(0) == q.size(0) && k.size(1) == q.size(1) &&
+                  k.size(2) >= q.size(2), "flash_sink_fwd: q, k, v");
+  const int64_t B = q.size(0), H = q.size(1), Sq = q.size(2), Sk = k.size(2), D = q.size(3);
+  check_rows(gate, "gate");
+  TORCH_CHECK(vdim > 0 && vdim <= D && vdim % 8 == 0 && gate.size(0) == B * Sq && gate.size(1) == H && sink.numel() == H &&
+                  k.scalar_type() == q.scalar_type() && v.scalar_type() == q.scalar_type() && gate.scalar_type() == q.scalar_type() &&
+                  sink.scalar_type() == q.scalar_type(), "flash_sink_fwd: operands");
+  const uint8_t* kp = nullptr;
+  if (kpm.has_value() && kpm->defined()) {
+    TORCH_CHECK(kpm->is_contiguous() && kpm->scalar_type() == at::kByte && kpm->numel() == B * Sk, "flash_sink_fwd: mask");
+    kp = kpm->data_ptr<uint8_t>();
+  }
+  c10::cuda::CUDAGuard guard(q.device());
+  Tensor out = at::empty({B * Sq, H * vdim}, q.options());
+  check_rc(oslo_flash_sink_fwd_sm100(q.data_ptr(), k.data_ptr(), v.data_ptr(), out.data_ptr(), kp, sink.data_ptr(),
+                                     gate.data_ptr(), gate.stride(0), static_cast<int>(vdim), static_cast<int>(B),
+                                     static_cast<int>(H), static_cast<int>(Sq), static_cast<int>(Sk), static_cast<int>(D),
+                                     q.stride(0), q.stride(1), q.stride(2), k.stride(0), k.stride(1), k.stride(2), v.stride(0),
+                                     v.stride(1), v.stride(2), Sq * H * vdim, vdim, H * vdim, static_cast<float>(scale),
+                                     dt_code(q), dev_state(q.get_device()).err.data_ptr<int>(), cur_stream()), "flash_sink_fwd");
+  return out;
+}
+
 Tensor sink_attention(const Tensor& q, const Tensor& k, const Tensor& v, const optional<Tensor>& keep, const Tensor& sink,
                       const Tensor& gate, double scale) {
   // [B, S, H, D] views with contiguous D
@@ -935,9 +962,7 @@ Tensor latent_decode(const Tensor& q, const Tensor& w_uk, const Tensor& w_uv, co
   const int64_t dim = q.size(1) / heads, vdim = w_uv.size(0) / heads;
   c10::cuda::CUDAGuard guard(q.device());
   auto& st = dev_state(q.get_device());
-  const int groups = static_cast<int>((heads + 15) / 16);
-  int splits = std::max<int>(1, std::min<int>(64, 2 * st.sms / std::max<int>(1, static_cast<int>(B) * groups)));
-  splits = static_cast<int>(std::min<int64_t>(splits, std::max<int64_t>(1, T / 32)));
+  const int splits = oslo_latent_splits(static_cast<int>(B), static_cast<int>(heads), static_cast<int>(T), static_cast<int>(R), st.sms);
   const auto f32 = q.options().dtype(at::kFloat);
   Tensor qa = at::empty({B, heads, R}, f32);
   Tensor ws = at::empty({B, heads, splits, R + 2}, f32);
@@ -947,7 +972,8 @@ Tensor latent_decode(const Tensor& q, const Tensor& w_uk, const Tensor& w_uv, co
                               sink.data_ptr(), gate.data_ptr(), gate.stride(0), qa.data_ptr<float>(), ws.data_ptr<float>(),
                               out.data_ptr(), static_cast<int>(B), static_cast<int>(heads), static_cast<int>(dim),
                               static_cast<int>(vdim), static_cast<int>(R), static_cast<int>(T), splits,
-                              static_cast<float>(scale), dt_code(q), st.err.data_ptr<int>(), cur_stream(3)), "latent_decode");
+                              static_cast<float>(scale), st.sms, dt_code(q), st.err.data_ptr<int>(), cur_stream(3)),
+           "latent_decode");
   return out;
 }
 
@@ -1073,6 +1099,7 @@ TORCH_LIBRARY(oslo_b200, m) {
   m.def("recurrence(Tensor q, Tensor f, Tensor v, Tensor f_bias, Tensor lower, Tensor? keep, Tensor(a!)? state, int batch, int heads, int dim, int vdim, int chunks=0) -> Tensor");
   m.def("recurrence_step(Tensor q, Tensor f, Tensor v, Tensor f_bias, Tensor lower, Tensor norm_w, Tensor? keep, Tensor(a!) state, float eps, int heads, int dim, int vdim) -> Tensor");
   m.def("sink_gate(Tensor o, Tensor lse, Tensor sink, Tensor gate, int vdim) -> Tensor");
+  m.def("flash_sink_fwd(Tensor q, Tensor k, Tensor v, Tensor? kpm, Tensor sink, Tensor gate, float scale, int vdim) -> Tensor");
   m.def("sink_attention(Tensor q, Tensor k, Tensor v, Tensor? keep, Tensor sink, Tensor gate, float scale) -> Tensor");
   m.def("latent_prep(Tensor cq, Tensor wq, Tensor? ckv, Tensor? wkv, Tensor(a!)? cache, Tensor lengths, float eps) -> Tensor");
   m.def("latent_decode(Tensor q, Tensor w_uk, Tensor w_uv, Tensor cache, Tensor lengths, Tensor? keep, Tensor sink, Tensor gate, float scale, int heads) -> Tensor");
@@ -1123,6 +1150,7 @@ TORCH_LIBRARY_IMPL(oslo_b200, CUDA, m) {
   m.impl("recurrence", &recurrence);
   m.impl("recurrence_step", &recurrence_step);
   m.impl("sink_gate", &sink_gate);
+  m.impl("flash_sink_fwd", &flash_sink_fwd);
   m.impl("sink_attention", &sink_attention);
   m.impl("latent_prep", &latent_prep);
   m.impl("latent_decode", &latent_decode);

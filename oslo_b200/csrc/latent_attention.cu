@@ -330,41 +330,264 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentDecodePa
   }
 }
 
+// 16-bit version on the tensor cores for R % 16 == 0: the 16 heads of a group are the 16 rows of an m16n8k16 tile, so the
+// cache streams through shared memory once for all of them. 8 warps; per KT cached vectors:
+//   scores  the warps cover the KT / 8 key columns (and halves of R when KT = 32); q' is split into two 16-bit terms
+//   softmax warp w owns heads 2 w and 2 w + 1 (running max and sum in registers), P is stored as 16-bit
+//   output  a warp owns every eighth pair of 8-column blocks of R; the cached vectors are read transposed
+// The next KT vectors are fetched with cp.async meanwhile.
+template <typename T> struct MmaT;
+template <> struct MmaT<__nv_bfloat16> {
+  static __device__ __forceinline__ void mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+  }
+};
+template <> struct MmaT<__half> {
+  static __device__ __forceinline__ void mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.f16.f16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+  }
+};
+__device__ __forceinline__ void ldsm4(uint32_t addr, uint32_t (&r)[4]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void ldsm2(uint32_t addr, uint32_t& r0, uint32_t& r1) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(r0), "=r"(r1) : "r"(addr));
+}
+__device__ __forceinline__ void ldsm4_t(uint32_t addr, uint32_t (&r)[4]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+
+template <typename T, int KT, int NP>   // KT cached vectors per step (64 or 32), NP pairs of 8-column blocks per warp
+__global__ void __launch_bounds__(256, 1) latent_decode_mma_kernel(const LatentDecodeParams p) {
+  constexpr int KS = KT == 64 ? 1 : 2;  // slices of R in the score product
+  constexpr int PP = KT + 8;            // padded row of P
+  extern __shared__ __align__(16) uint8_t lm_smem[];
+  const int rp = p.R + 8;               // padded row: 16-byte aligned, conflict-free ldmatrix
+  T* q_hi = reinterpret_cast<T*>(lm_smem);          // [16][rp]
+  T* q_lo = q_hi + 16 * rp;
+  T* cs = q_lo + 16 * rp;                           // [2][KT][rp]
+  T* ps = cs + 2 * KT * rp;                         // [16][PP]
+  float* ss = reinterpret_cast<float*>(ps + 16 * PP);   // [KS][16][KT + 1]
+  float* fac = ss + KS * 16 * (KT + 1);             // [16]
+  const int b = blockIdx.z, h0 = blockIdx.y * LD_HEADS, sp = blockIdx.x, tid = threadIdx.x;
+  const int warp = tid >> 5, lane = tid & 31;
+  const int nh = min(LD_HEADS, p.H - h0);
+  int len = p.lengths[b];
+  if (len < 0 || len > p.Tmax) {       // a length that does not fit the cache: never read past it
+    if (tid == 0) OSLO_REPORT_BOUNDS(p.err);
+    len = len < 0 ? 0 : p.Tmax;
+  }
+  const int tiles = (len + KT - 1) / KT, per = (tiles + p.splits - 1) / p.splits * KT;
+  const int t0 = sp * per, t1 = min(len, t0 + per);
+  const T* c = static_cast<const T*>(p.cache) + static_cast<long long>(b) * p.Tmax * p.R;
+  const int vr = p.R / 8;              // 16-byte pieces of a cached vector
+  auto fetch = [&](int k0, int buf) {
+    T* dst = cs + static_cast<size_t>(buf) * KT * rp;
+    for (int e = tid; e < KT * vr; e += 256) {
+      const int t = e / vr, v = e - t * vr;
+      const uint32_t d32 = smem_u32(dst + t * rp + v * 8);
+      const bool in = k0 + t < t1;     // rows past the slice are zero-filled (source size 0)
+      const T* src = c + static_cast<long long>(in ? k0 + t : 0) * p.R + v * 8;
+      const int bytes = in ? 16 : 0;
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d32), "l"(src), "r"(bytes) : "memory");
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  if (t0 < t1) fetch(t0, 0);
+  for (int e = tid; e < 16 * p.R; e += 256) {
+    const int a = e / p.R, r = e - a * p.R;
+    const float x = a < nh ? p.qa[(static_cast<long long>(b) * p.H + h0 + a) * p.R + r] : 0.f;
+    const T hi = Num<T>::from(x);
+    q_hi[a * rp + r] = hi;
+    q_lo[a * rp + r] = Num<T>::from(x - Num<T>::to(hi));
+  }
+  float acc[NP][2][4];
+#pragma unroll
+  for (int j = 0; j < NP; ++j)
+#pragma unroll
+    for (int u = 0; u < 2; ++u)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) acc[j][u][i] = 0.f;
+  float m_run[2] = {-CUDART_INF_F, -CUDART_INF_F}, l_run[2] = {0.f, 0.f};
+  const int arow = lane & 15, acol = (lane >> 4) * 8;      // ldmatrix.x4 source of an A fragment
+  for (int k0 = t0, it = 0; k0 < t1; k0 += KT, ++it) {
+    const int buf = it & 1;
+    if (k0 + KT < t1) {                                    // the other buffer was last read before the closing barrier
+      fetch(k0 + KT, buf ^ 1);
+      asm volatile("cp.async.wait_group 1;" ::: "memory");
+    } else {
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
+    }
+    __syncthreads();
+    const T* ct = cs + static_cast<size_t>(buf) * KT * rp;
+    {
+      const int kg = warp % (KT / 8), ks = warp / (KT / 8);
+      const int n16 = p.R / 16, s_begin = ks * n16 / KS, s_end = (ks + 1) * n16 / KS;
+      float d[4] = {0.f, 0.f, 0.f, 0.f}, e[4] = {0.f, 0.f, 0.f, 0.f};
+      for (int s = s_begin; s < s_end; ++s) {
+        uint32_t ah[4], al[4], b0, b1;
+        ldsm4(smem_u32(q_hi + arow * rp + s * 16 + acol), ah);
+        ldsm4(smem_u32(q_lo + arow * rp + s * 16 + acol), al);
+        ldsm2(smem_u32(ct + (kg * 8 + (lane & 7)) * rp + s * 16 + ((lane >> 3) & 1) * 8), b0, b1);
+        MmaT<T>::mma(d, ah, b0, b1);
+        MmaT<T>::mma(e, al, b0, b1);
+      }
+      float* o = ss + ks * 16 * (KT + 1) + (lane >> 2) * (KT + 1) + kg * 8 + (lane & 3) * 2;
+      o[0] = d[0] + e[0]; o[1] = d[1] + e[1];
+      o[8 * (KT + 1)] = d[2] + e[2]; o[8 * (KT + 1) + 1] = d[3] + e[3];
+    }
+    __syncthreads();
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int a = warp * 2 + u;
+      float x[KT / 32], mx = m_run[u];
+#pragma unroll
+      for (int i = 0; i < KT / 32; ++i) {
+        const int t = lane + 32 * i, pos = k0 + t;
+        float v = ss[a * (KT + 1) + t];
+        if (KS == 2) v += ss[16 * (KT + 1) + a * (KT + 1) + t];
+        const bool vis = pos < t1 && (p.keep == nullptr || pos >= p.n_keep || p.keep[b * p.ld_keep + pos]);
+        x[i] = vis ? v : -CUDART_INF_F;
+        mx = fmaxf(mx, x[i]);
+      }
+#pragma unroll
+      for (int off = 16; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
+      float sum = 0.f;
+#pragma unroll
+      for (int i = 0; i < KT / 32; ++i) {
+        const float pr = x[i] == -CUDART_INF_F ? 0.f : expf(x[i] - mx);
+        sum += pr;
+        ps[a * PP + lane + 32 * i] = Num<T>::from(pr);
+      }
+      sum = warp_sum(sum);
+      const float f = m_run[u] == -CUDART_INF_F ? 0.f : expf(m_run[u] - mx);
+      l_run[u] = l_run[u] * f + sum;
+      m_run[u] = mx;
+      if (lane == 0) fac[a] = f;
+    }
+    __syncthreads();
+    const float f0 = fac[lane >> 2], f1 = fac[(lane >> 2) + 8];
+#pragma unroll
+    for (int j = 0; j < NP; ++j)
+#pragma unroll
+      for (int u = 0; u < 2; ++u) {
+        acc[j][u][0] *= f0; acc[j][u][1] *= f0; acc[j][u][2] *= f1; acc[j][u][3] *= f1;
+      }
+#pragma unroll
+    for (int s = 0; s < KT / 16; ++s) {
+      uint32_t a[4];
+      ldsm4(smem_u32(ps + arow * PP + s * 16 + acol), a);
+#pragma unroll
+      for (int j = 0; j < NP; ++j) {
+        const int col = (warp + 8 * j) * 16;
+        if (col < p.R) {                                   // uniform over the warp
+          uint32_t bb[4];
+          ldsm4_t(smem_u32(ct + (s * 16 + (lane & 15)) * rp + col + (lane >> 4) * 8), bb);
+          MmaT<T>::mma(acc[j][0], a, bb[0], bb[1]);
+          MmaT<T>::mma(acc[j][1], a, bb[2], bb[3]);
+        }
+      }
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int j = 0; j < NP; ++j) {
+    const int col = (warp + 8 * j) * 16;
+    if (col >= p.R) continue;
+#pragma unroll
+    for (int u = 0; u < 2; ++u)
+#pragma unroll
+      for (int hf = 0; hf < 2; ++hf) {
+        const int a = (lane >> 2) + 8 * hf;
+        if (a < nh) {
+          float* w = p.ws + ((static_cast<long long>(b) * p.H + h0 + a) * p.splits + sp) * (p.R + 2) + col + u * 8 + (lane & 3) * 2;
+          w[0] = acc[j][u][hf * 2];
+          w[1] = acc[j][u][hf * 2 + 1];
+        }
+      }
+  }
+#pragma unroll
+  for (int u = 0; u < 2; ++u) {
+    const int a = warp * 2 + u;
+    if (lane == 0 && a < nh) {
+      float* w = p.ws + ((static_cast<long long>(b) * p.H + h0 + a) * p.splits + sp) * (p.R + 2) + p.R;
+      w[0] = m_run[u];
+      w[1] = l_run[u];
+    }
+  }
+}
+static size_t latent_mma_smem(int R, int kt) {
+  const size_t rp = R + 8;
+  return (32 * rp + 2 * kt * rp + 16 * (kt + 8)) * 2 + ((kt == 64 ? 1 : 2) * 16 * (kt + 1) + 16) * sizeof(float);
+}
+
 // out[b, h * vdim + j] = sigmoid(g) * sum_r w_uv[h * vdim + j, r] * o[r],  o = merged slices / (sum + exp(sink))
-template <typename T, int VEC>
+// for NB rows b per block, so that W_uv is read once for all of them
+template <typename T, int VEC, int NB>
 __global__ void __launch_bounds__(256) latent_finish_kernel(const float* __restrict__ ws, const T* __restrict__ w, long long ldw,
                                                             const T* __restrict__ sink, const T* __restrict__ gate,
-                                                            long long ldg, T* __restrict__ out, int H, int R, int vdim,
+                                                            long long ldg, T* __restrict__ out, int B, int H, int R, int vdim,
                                                             int splits, int rows_per_block) {
-  extern __shared__ float fin_smem[];   // [R] then [splits] weights
+  extern __shared__ float fin_smem[];   // [NB][R] then [NB][splits] weights
   float* o = fin_smem;
-  float* wt = fin_smem + R;
-  const int h = blockIdx.y, b = blockIdx.z;
-  const float* base = ws + (static_cast<long long>(b) * H + h) * splits * (R + 2);
+  float* wt = fin_smem + NB * R;
+  const int h = blockIdx.y, b0 = blockIdx.z * NB, nb = min(NB, B - b0);
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const float snk = Num<T>::to(sink[h]);
-  float m = snk;
-  for (int s = 0; s < splits; ++s) m = fmaxf(m, base[static_cast<long long>(s) * (R + 2) + R]);
-  float tot = expf(snk - m);
-  for (int s = 0; s < splits; ++s) {
-    const float ms = base[static_cast<long long>(s) * (R + 2) + R];
-    const float f = ms == -CUDART_INF_F ? 0.f : expf(ms - m);
-    tot += f * base[static_cast<long long>(s) * (R + 2) + R + 1];
-    if (threadIdx.x == 0) wt[s] = f;
+  for (int i = warp; i < nb; i += 8) {  // slice weights of a row, already divided by the denominator and gated
+    const float* st = ws + (static_cast<long long>(b0 + i) * H + h) * splits * (R + 2) + R;
+    float m = snk;
+    for (int s = lane; s < splits; s += 32) m = fmaxf(m, st[static_cast<long long>(s) * (R + 2)]);
+#pragma unroll
+    for (int off = 16; off > 0; off >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, off));
+    float tot = 0.f;
+    for (int s = lane; s < splits; s += 32) {
+      const float ms = st[static_cast<long long>(s) * (R + 2)];
+      const float f = ms == -CUDART_INF_F ? 0.f : expf(ms - m);
+      tot += f * st[static_cast<long long>(s) * (R + 2) + 1];
+      wt[i * splits + s] = f;
+    }
+    tot = warp_sum(tot) + expf(snk - m);
+    const float inv = sigmoid_f(Num<T>::to(gate[(b0 + i) * ldg + h])) / tot;
+    for (int s = lane; s < splits; s += 32) wt[i * splits + s] *= inv;
   }
   __syncthreads();
-  const float inv = sigmoid_f(Num<T>::to(gate[b * ldg + h])) / tot;
-  for (int r = threadIdx.x; r < R; r += blockDim.x) {
+  for (int e = threadIdx.x; e < nb * R; e += blockDim.x) {
+    const int i = e / R, r = e - i * R;
+    const float* base = ws + (static_cast<long long>(b0 + i) * H + h) * splits * (R + 2) + r;
     float v = 0.f;
-    for (int s = 0; s < splits; ++s)
-      if (wt[s] != 0.f) v = fmaf(wt[s], base[static_cast<long long>(s) * (R + 2) + r], v);
-    o[r] = v * inv;
+#pragma unroll 8
+    for (int s = 0; s < splits; ++s) v = fmaf(wt[i * splits + s], base[static_cast<long long>(s) * (R + 2)], v);
+    o[i * R + r] = v;
   }
   __syncthreads();
-  const int lane = threadIdx.x & 31;
   const int j1 = min(vdim, (static_cast<int>(blockIdx.x) + 1) * rows_per_block);
-  for (int j = blockIdx.x * rows_per_block + (threadIdx.x >> 5); j < j1; j += blockDim.x >> 5) {
-    const float d = warp_dot<T, VEC>(w + (static_cast<long long>(h) * vdim + j) * ldw, o, R, lane);
-    if (lane == 0) out[(static_cast<long long>(b) * H + h) * vdim + j] = Num<T>::from(d);
+  for (int j = blockIdx.x * rows_per_block + warp; j < j1; j += 8) {
+    const T* wr = w + (static_cast<long long>(h) * vdim + j) * ldw;
+    float acc[NB];
+#pragma unroll
+    for (int i = 0; i < NB; ++i) acc[i] = 0.f;
+    for (int k = lane * VEC; k < R; k += 32 * VEC) {
+      float x[VEC];
+      load_vec<T, VEC>(wr + k, x);
+#pragma unroll
+      for (int i = 0; i < NB; ++i)
+        if (i < nb) {
+#pragma unroll
+          for (int u = 0; u < VEC; ++u) acc[i] = fmaf(x[u], o[i * R + k + u], acc[i]);
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < NB; ++i) {
+      const float d = warp_sum(acc[i]);
+      if (lane == 0 && i < nb) out[(static_cast<long long>(b0 + i) * H + h) * vdim + j] = Num<T>::from(d);
+    }
   }
 }
 
@@ -425,47 +648,99 @@ extern "C" int oslo_latent_prep(const void* cq, long long ldq, const void* wq, i
   return static_cast<int>(cudaGetLastError());
 }
 
+namespace oslo {
+
+template <typename T>
+static int latent_scan(const LatentDecodeParams& p, int use_mma, cudaStream_t st) {
+  dim3 grid(p.splits, (p.H + LD_HEADS - 1) / LD_HEADS, p.B);
+  if constexpr (sizeof(T) == 2) {
+    if (use_mma) {
+      const int kt = p.R <= 512 ? 64 : 32, np = (p.R + 127) / 128;
+      const size_t smem = latent_mma_smem(p.R, kt);
+#define LM_GO(KT, NP)                                                                                   \
+  {                                                                                                     \
+    const int rc = set_smem(reinterpret_cast<const void*>(&latent_decode_mma_kernel<T, KT, NP>), smem); \
+    if (rc) return rc;                                                                                  \
+    latent_decode_mma_kernel<T, KT, NP><<<grid, 256, smem, st>>>(p);                                    \
+    return static_cast<int>(cudaGetLastError());                                                        \
+  }
+      if (np == 1) LM_GO(64, 1)
+      if (np == 2) LM_GO(64, 2)
+      if (np <= 4) LM_GO(64, 4)
+      LM_GO(32, 8)
+#undef LM_GO
+    }
+  }
+  const size_t smem = (static_cast<size_t>(LD_HEADS + LD_KEYS) * (p.R + 1) + LD_HEADS * LD_KEYS) * sizeof(float);
+#define LD_GO(NR)                                                                             \
+  {                                                                                           \
+    const int rc = set_smem(reinterpret_cast<const void*>(&latent_decode_kernel<T, NR>), smem); \
+    if (rc) return rc;                                                                        \
+    latent_decode_kernel<T, NR><<<grid, 256, smem, st>>>(p);                                  \
+  }
+  if (p.R <= 256) LD_GO(1)
+  else if (p.R <= 512) LD_GO(2)
+  else LD_GO(4)
+#undef LD_GO
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <typename T, int VEC>
+static int latent_finish(const LatentDecodeParams& p, const void* w_uv, long long ldv, const void* sink, const void* gate,
+                         long long ldg, void* out, int vdim, int num_sms, cudaStream_t st) {
+  const int nb = p.B >= 8 ? 8 : (p.B >= 2 ? 2 : 1), zb = (p.B + nb - 1) / nb;
+  int parts = 1;                       // value rows of a head over several blocks while the GPU has room
+  while (parts < 16 && static_cast<long long>(zb) * p.H * parts < num_sms && vdim / (2 * parts) >= 8) parts *= 2;
+  const int rpb = (vdim + parts - 1) / parts;
+  const size_t smem = static_cast<size_t>(nb) * (p.R + p.splits) * sizeof(float);
+  dim3 grid(parts, p.H, zb);
+#define FIN_GO(NB)                                                                                                    \
+  latent_finish_kernel<T, VEC, NB><<<grid, 256, smem, st>>>(p.ws, static_cast<const T*>(w_uv), ldv, static_cast<const T*>(sink), \
+                                                            static_cast<const T*>(gate), ldg, static_cast<T*>(out), p.B, p.H, p.R, \
+                                                            vdim, p.splits, rpb)
+  if (nb == 8) FIN_GO(8);
+  else if (nb == 2) FIN_GO(2);
+  else FIN_GO(1);
+#undef FIN_GO
+  return static_cast<int>(cudaGetLastError());
+}
+
+}  // namespace oslo
+
+// slices of the cache per (row, head group): fewest waves of blocks, then the least work per block
+extern "C" int oslo_latent_splits(int B, int H, int T, int R, int num_sms) {
+  const int groups = (H + oslo::LD_HEADS - 1) / oslo::LD_HEADS, kt = R <= 512 ? 64 : 32, tiles = (T + kt - 1) / kt;
+  int best = 1;
+  double best_cost = 1e30;
+  for (int s = 1; s <= 32 && s <= tiles; ++s) {
+    const long long waves = (static_cast<long long>(B) * groups * s + num_sms - 1) / num_sms;
+    const double cost = static_cast<double>(waves) * ((tiles + s - 1) / s + 1.5) + 0.05 * s;   // set-up and merge of a slice
+    if (cost < best_cost) { best_cost = cost; best = s; }
+  }
+  return best;
+}
+
 extern "C" int oslo_latent_decode(const void* q, long long ldq, const void* w_uk, long long ldk, const void* w_uv, long long ldv,
                                   const void* cache, const int* lengths, const uint8_t* keep, long long ld_keep, int n_keep,
                                   const void* sink, const void* gate, long long ldg, float* qa, float* ws, void* out, int B,
-                                  int H, int dim, int vdim, int R, int Tmax, int splits, float scale, int dtype, int* err_word,
-                                  cudaStream_t stream) {
+                                  int H, int dim, int vdim, int R, int Tmax, int splits, float scale, int num_sms, int dtype,
+                                  int* err_word, cudaStream_t stream) {
   using namespace oslo;
   if (B <= 0 || H <= 0) return 0;
-  if (R <= 0 || R > 1024 || splits < 1 || B > 65535) return -1;
+  if (R <= 0 || R > 1024 || splits < 1 || splits > 64 || B > 65535 || H > 65535) return -1;
   LatentDecodeParams p{qa, cache, lengths, keep, ld_keep, n_keep, ws, B, H, R, Tmax, splits, err_word};
   const size_t te = dtype == OSLO_DT_FP32 ? 4 : 2;
   const size_t ab_smem = (8 * static_cast<size_t>(dim) + 8 * 8 * 64) * sizeof(float);
-  const size_t ld_smem = (static_cast<size_t>(LD_HEADS + LD_KEYS) * (R + 1) + LD_HEADS * LD_KEYS) * sizeof(float);
-  const size_t fin_smem = static_cast<size_t>(R + splits) * sizeof(float);
-  dim3 grid(splits, (H + LD_HEADS - 1) / LD_HEADS, B);
-#define LD_GO(NR)                                                                             \
-  {                                                                                           \
-    rc = set_smem(reinterpret_cast<const void*>(&latent_decode_kernel<T, NR>), ld_smem);      \
-    if (rc) return rc;                                                                        \
-    latent_decode_kernel<T, NR><<<grid, 256, ld_smem, stream>>>(p);                           \
-  }
   OSLO_DISPATCH_T(dtype, {
     int rc = set_smem(reinterpret_cast<const void*>(&latent_absorb_kernel<T>), ab_smem);
     if (rc) return rc;
     latent_absorb_kernel<T><<<dim3((R + 63) / 64, H, (B + 7) / 8), 256, ab_smem, stream>>>(
         static_cast<const T*>(q), ldq, static_cast<const T*>(w_uk), ldk, qa, B, H, dim, R, scale);
-    if (R <= 256) LD_GO(1)
-    else if (R <= 512) LD_GO(2)
-    else LD_GO(4)
-    int parts = 1;                     // value rows of a head over several blocks while the GPU has room
-    while (parts < 8 && static_cast<long long>(B) * H * parts < 148 && vdim / (2 * parts) >= 8) parts *= 2;
-    const int rpb = (vdim + parts - 1) / parts;
+    rc = latent_scan<T>(p, R % 16 == 0 && aligned_to(cache, 16), stream);
+    if (rc) return rc;
     const bool vec = R % 4 == 0 && ldv % 4 == 0 && aligned_to(w_uv, 4 * te);
-    if (vec)
-      latent_finish_kernel<T, 4><<<dim3(parts, H, B), 256, fin_smem, stream>>>(
-          ws, static_cast<const T*>(w_uv), ldv, static_cast<const T*>(sink), static_cast<const T*>(gate), ldg,
-          static_cast<T*>(out), H, R, vdim, splits, rpb);
-    else
-      latent_finish_kernel<T, 1><<<dim3(parts, H, B), 256, fin_smem, stream>>>(
-          ws, static_cast<const T*>(w_uv), ldv, static_cast<const T*>(sink), static_cast<const T*>(gate), ldg,
-          static_cast<T*>(out), H, R, vdim, splits, rpb);
+    return vec ? latent_finish<T, 4>(p, w_uv, ldv, sink, gate, ldg, out, vdim, num_sms, stream)
+               : latent_finish<T, 1>(p, w_uv, ldv, sink, gate, ldg, out, vdim, num_sms, stream);
   });
-#undef LD_GO
-  return static_cast<int>(cudaGetLastError());
+  return -2;
 }

@@ -53,6 +53,8 @@ struct RecParams {
   int B, S, H, dim, vdim;
   int chunk, nchunks;                // tokens per chunk
   long long s_batch, s_chunk;        // element strides of s_in / s_out over batch rows and chunks
+  int dim_pad;                       // dim rounded up so that every row of a raw stage starts at a 16-byte boundary
+  int vec16;                         // q, f, v rows and head slices start at 16-byte boundaries
 };
 
 constexpr int REC_TB = 16;    // tokens staged at a time
@@ -102,23 +104,68 @@ __global__ void __launch_bounds__(128) recurrence_kernel(const RecParams p) {
   for (int i = 0; i < REC_ROWS; ++i) dec[i] = 1.f;
   const f32x2 minus1 = pack_f2(-1.f, -1.f);
 
-  for (int t0 = t_begin; t0 < t_end; t0 += REC_TB) {
+  // raw [REC_TB][raw_ld] stages in the storage type, fetched one step ahead: q (unless STATE_ONLY), f, v slice
+  const int f_at = STATE_ONLY ? 0 : p.dim_pad, v_at = f_at + p.dim_pad, raw_ld = v_at + cols;
+  T* raw = reinterpret_cast<T*>(vs + REC_TB * cols);
+  auto fetch = [&](int t0, int buf) {
+    T* dst = raw + static_cast<size_t>(buf) * REC_TB * raw_ld;
     const int n = min(REC_TB, t_end - t0);
-    __syncthreads();
-    for (int e = tid; e < n * DP; e += nt) {
-      const int t = e / DP, i = e % DP;
-      const bool on = i < p.dim && (p.keep == nullptr || p.keep[b * p.ld_keep + t0 + t]);
-      float kk = 0.f, qq = 0.f;
-      if (on) {
-        kk = write_gate(Num<T>::to(f[(t0 + t) * p.ldf + i]) + Num<T>::to(fb[i]), Num<T>::to(lw[i]));
-        if (!STATE_ONLY) qq = silu_f(Num<T>::to(q[(t0 + t) * p.ldq + i]));
+    if (p.vec16) {
+      constexpr int V = 16 / sizeof(T);
+      const int per_dim = p.dim / V, per_v = min(cols, p.vdim - col0) / V;
+      const int per_row = (STATE_ONLY ? 1 : 2) * per_dim + per_v;
+      for (int e = tid; e < n * per_row; e += nt) {
+        const int t = e / per_row;
+        int c = e - t * per_row;
+        const T* src;
+        int at;
+        if (!STATE_ONLY && c < per_dim) {
+          src = q + (t0 + t) * p.ldq + c * V; at = c * V;
+        } else {
+          if (!STATE_ONLY) c -= per_dim;
+          if (c < per_dim) { src = f + (t0 + t) * p.ldf + c * V; at = f_at + c * V; }
+          else { c -= per_dim; src = v + (t0 + t) * p.ldv + c * V; at = v_at + c * V; }
+        }
+        const uint32_t d32 = static_cast<uint32_t>(__cvta_generic_to_shared(dst + t * raw_ld + at));
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(d32), "l"(src) : "memory");
       }
-      ks[t * DP + i] = kk;
-      if (!STATE_ONLY) qs[t * DP + i] = qq;
+    } else {
+      const int nv = min(cols, p.vdim - col0);
+      for (int t = 0; t < n; ++t) {
+        for (int i = tid; i < p.dim; i += nt) {
+          if (!STATE_ONLY) dst[t * raw_ld + i] = q[(t0 + t) * p.ldq + i];
+          dst[t * raw_ld + f_at + i] = f[(t0 + t) * p.ldf + i];
+        }
+        for (int c = tid; c < nv; c += nt) dst[t * raw_ld + v_at + c] = v[(t0 + t) * p.ldv + c];
+      }
     }
-    for (int e = tid; e < n * cols; e += nt) {
-      const int t = e / cols, c = e % cols;
-      vs[t * cols + c] = col0 + c < p.vdim ? Num<T>::to(v[(t0 + t) * p.ldv + c]) : 0.f;
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  if (t_begin < t_end) fetch(t_begin, 0);
+  for (int t0 = t_begin, it = 0; t0 < t_end; t0 += REC_TB, ++it) {
+    const int n = min(REC_TB, t_end - t0);
+    if (t0 + REC_TB < t_end) {                         // every thread read the other stage before the last barrier
+      fetch(t0 + REC_TB, (it + 1) & 1);
+      asm volatile("cp.async.wait_group 1;" ::: "memory");
+    } else {
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
+    }
+    __syncthreads();
+    const T* src = raw + static_cast<size_t>(it & 1) * REC_TB * raw_ld;
+    for (int i = tid; i < DP; i += nt) {
+      const bool real = i < p.dim;
+      const float bias = real ? Num<T>::to(fb[i]) : 0.f, low = real ? Num<T>::to(lw[i]) : 1.f;
+#pragma unroll 4
+      for (int t = 0; t < n; ++t) {
+        const bool on = real && (p.keep == nullptr || p.keep[b * p.ld_keep + t0 + t]);
+        ks[t * DP + i] = on ? write_gate(Num<T>::to(src[t * raw_ld + f_at + i]) + bias, low) : 0.f;
+        if (!STATE_ONLY) qs[t * DP + i] = on ? silu_f(Num<T>::to(src[t * raw_ld + i])) : 0.f;
+      }
+    }
+    for (int c = tid; c < cols; c += nt) {
+      const bool real = col0 + c < p.vdim;
+#pragma unroll 4
+      for (int t = 0; t < n; ++t) vs[t * cols + c] = real ? Num<T>::to(src[t * raw_ld + v_at + c]) : 0.f;
     }
     __syncthreads();
     for (int t = 0; t < n; ++t) {
@@ -328,7 +375,8 @@ static int rec_launch(const RecParams& p, cudaStream_t st) {
   const int groups = (p.vdim + REC_COLS - 1) / REC_COLS;
   int nt = std::min(128, (groups * G + 31) / 32 * 32);
   const int cols = nt / G * REC_COLS;
-  const size_t smem = static_cast<size_t>(REC_TB) * ((STATE_ONLY ? 1 : 2) * REC_ROWS * G + cols) * sizeof(float);
+  const size_t smem = static_cast<size_t>(REC_TB) * (((STATE_ONLY ? 1 : 2) * REC_ROWS * G + cols) * sizeof(float) +
+                                                     2 * ((STATE_ONLY ? 1 : 2) * p.dim_pad + cols) * sizeof(T));
   if (smem > 48 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(recurrence_kernel<T, G, STATE_ONLY>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          static_cast<int>(smem));
@@ -379,6 +427,10 @@ extern "C" int oslo_recurrence(const void* q, long long ldq, const void* f, long
   p.keep = keep; p.ld_keep = ld_keep; p.out = out;
   p.B = B; p.S = S; p.H = H; p.dim = dim; p.vdim = vdim;
   const long long per = static_cast<long long>(H) * dim * vdim;
+  const int te = dtype == OSLO_DT_FP32 ? 4 : 2, v16 = 16 / te;
+  p.dim_pad = (dim + 7) / 8 * 8;
+  p.vec16 = dim % v16 == 0 && vdim % v16 == 0 && ldq % v16 == 0 && ldf % v16 == 0 && ldv % v16 == 0 && aligned_to(q, 16) &&
+            aligned_to(f, 16) && aligned_to(v, 16);
   int rc = 0;
   if (nchunks == 1) {
     p.chunk = S; p.nchunks = 1; p.s_in = state; p.s_out = state; p.s_batch = per; p.s_chunk = 0;

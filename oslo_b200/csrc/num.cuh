@@ -39,7 +39,7 @@ __device__ __forceinline__ void store_vec(T* p, const float (&v)[VEC]) {
   *reinterpret_cast<Pack<T, VEC>*>(p) = k;
 }
 
-__device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float sigmoid_f(float z) { return __fdividef(1.0f, 1.0f + expf(-z)); }   // 2 ulp; 0 when expf overflows
 __device__ __forceinline__ float silu_f(float z) { return z * sigmoid_f(z); }
 
 __device__ __forceinline__ float warp_sum(float v) {

@@ -120,6 +120,12 @@ int oslo_flash_fwd_sm100(const void* q, const void* k, const void* v, void* o, f
                          long long k_sh, long long k_ss, long long v_sb, long long v_sh, long long v_ss, long long o_sb,
                          long long o_sh, long long o_ss, float scale, int causal, int window, int dtype, int* err_word,
                          cudaStream_t stream);
+// causal, with exp(sink[h]) in the denominator and a sigmoid output gate per (position, head); stores the first d_out columns
+int oslo_flash_sink_fwd_sm100(const void* q, const void* k, const void* v, void* o, const uint8_t* kpm, const void* sink,
+                              const void* gate, long long ldg, int d_out, int B, int H, int Sq, int Sk, int D, long long q_sb,
+                              long long q_sh, long long q_ss, long long k_sb, long long k_sh, long long k_ss, long long v_sb,
+                              long long v_sh, long long v_ss, long long o_sb, long long o_sh, long long o_ss, float scale,
+                              int dtype, int* err_word, cudaStream_t stream);
 int oslo_flash_bwd(const void* q, const void* k, const void* v, const void* o, const void* dout, const float* lse,
                    float* delta, float* dq_acc, void* dq, void* dk, void* dv, const uint8_t* kpm, int B, int H,
                    int Sq, int Sk, int D, long long q_sb, long long q_sh, long long q_ss, long long k_sb,
@@ -238,8 +244,9 @@ int oslo_latent_prep(const void* cq, long long ldq, const void* wq, int q_rank, 
 int oslo_latent_decode(const void* q, long long ldq, const void* w_uk, long long ldk, const void* w_uv, long long ldv,
                        const void* cache, const int* lengths, const uint8_t* keep, long long ld_keep, int n_keep,
                        const void* sink, const void* gate, long long ldg, float* qa, float* ws, void* out, int B, int H,
-                       int dim, int vdim, int R, int Tmax, int splits, float scale, int dtype, int* err_word,
+                       int dim, int vdim, int R, int Tmax, int splits, float scale, int num_sms, int dtype, int* err_word,
                        cudaStream_t stream);
+int oslo_latent_splits(int B, int H, int T, int R, int num_sms);
 
 // mixture of experts (moe.cu, grouped GEMM in gemm_sm100.cu)
 int oslo_moe_route(const void* h, long long ldh, const void* w, const void* bias, const float* logits, int* idx, float* wgt,

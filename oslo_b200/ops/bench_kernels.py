@@ -3,6 +3,10 @@
 ``python -m oslo_b200.ops.bench_kernels --op gemm``       tcgen05 GEMM vs ``torch.matmul`` (cuBLAS), GPT-J shapes
 ``python -m oslo_b200.ops.bench_kernels --op attention``  tcgen05 flash attention (forward, backward) vs the
                                                            mma.sync kernels of this package
+``python -m oslo_b200.ops.bench_kernels --op mixers``      the prompt and decode kernels of the recurrence, latent-attention,
+                                                           expert and norm layers, each with its bound (HBM bytes, bf16
+                                                           tensor-core or fp32 FMA throughput, whichever is slowest),
+                                                           beside the like kernels of GPT-J at the same sizes
 ``--case i`` restricts the run to one shape and ``--iters n --warmup w`` bound the number of launches, which is
 what a profiler capture wants. Every line is JSON; ``frac_of_measured`` divides by the bf16 GEMM throughput in
 ``MEASURED_PEAKS.json`` at the repository root when that file exists (else by 1590 TFLOP/s).
@@ -64,6 +68,25 @@ class _Timer:
         return ts[len(ts) // 2]
 
 
+class _GraphTimer(_Timer):
+    """The same timing with ``fn`` captured once into a CUDA graph and replayed, which is how decode steps run: without the
+    host's launch work, that takes longer than a small kernel."""
+
+    def __call__(self, fn) -> float:
+        side = torch.cuda.Stream()
+        side.wait_stream(torch.cuda.current_stream())
+        with torch.cuda.stream(side):
+            for _ in range(2):
+                fn()
+        torch.cuda.current_stream().wait_stream(side)
+        graph = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(graph):
+            fn()
+        ms = super().__call__(graph.replay)
+        del graph
+        return ms
+
+
 def bench_gemm(args, timer: _Timer) -> None:
     peak = _peak_tflops()
     cases = GEMM_CASES if args.case is None else [GEMM_CASES[args.case]]
@@ -108,18 +131,140 @@ def bench_attention(args, timer: _Timer) -> None:
             print(json.dumps(rec), flush=True)
 
 
+# width, heads, head dim, q_rank, kv_rank, experts, top, ff of an expert
+MIXER_CASES = [(2048, 16, 128, 1024, 512, 16, 2, 1024), (4096, 32, 128, 1536, 512, 32, 4, 1536)]
+FP32_TFLOPS = 148 * 128 * 2 * 1.965e9 / 1e12       # FMA pipes at the maximum SM clock (nominal; nothing measures it)
+
+
+def _measured_hbm() -> float:
+    path = os.path.join(os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__)))), "MEASURED_PEAKS.json")
+    try:
+        with open(path) as f:
+            return float(json.load(f)["hbm_gbs"])
+    except Exception:
+        return 6650.0
+
+
+def bench_mixers(args, timer: _Timer) -> None:
+    ext = load_ext(required=True)
+    timer = _GraphTimer(args.iters, args.warmup, not args.no_flush)
+    peak, hbm = _peak_tflops(), _measured_hbm()
+    bf = torch.bfloat16
+    mk = lambda *s: (torch.randn(*s, device="cuda") * 0.5).to(bf)                                          # noqa: E731
+
+    def report(case, op, fn, gbytes=0.0, tflop=0.0, fp32_tflop=0.0, like=""):
+        if args.only and args.only not in op:
+            return
+        ms = timer(fn)
+        bound = {"hbm": gbytes / hbm * 1e3, "bf16": tflop / peak * 1e3, "fp32": fp32_tflop / FP32_TFLOPS * 1e3}
+        by = max(bound, key=bound.get)
+        print(json.dumps(dict(case=case, op=op, us=round(ms * 1e3, 2), bound_us=round(bound[by] * 1e3, 2), bound_by=by,
+                              times_bound=round(ms / bound[by], 2), like=like)), flush=True)
+
+    for case, (w, h, d, qr, kr, e, top, ff) in enumerate(MIXER_CASES):
+        if args.case is not None and args.case != case:
+            continue
+        # ------------------------------------------------ prompts: 4 x 2048 tokens
+        b, s = 4, 2048
+        n = b * s
+        p = mk(n, 3 * h * d)
+        q, f, v = p[:, :h * d], p[:, h * d:2 * h * d], p[:, 2 * h * d:]
+        fb, lo, nw = mk(h * d), mk(h * d).abs().clamp(max=0.9), mk(d)
+        state = torch.zeros(b, h, d, d, device="cuda")
+        report(case, "prompt recurrence", lambda: ext.recurrence(q, f, v, fb, lo, None, state, b, h, d, d),
+               gbytes=n * h * d * (3 * 2 + 4) / 1e9, fp32_tflop=6.0 * n * h * d * d / 1e12, like="prompt attention (GPT-J)")
+        st1 = torch.zeros(1, h, d, d, device="cuda")
+        report(case, "prompt recurrence, 1 x 2048", lambda: ext.recurrence(q[:s], f[:s], v[:s], fb, lo, None, st1, 1, h, d, d),
+               gbytes=s * h * d * (3 * 2 + 4) / 1e9, fp32_tflop=6.0 * s * h * d * d / 1e12, like="prompt attention (GPT-J)")
+        o = torch.randn(n * h, d, device="cuda")
+        report(case, "prompt head norm", lambda: ext.rms_norm(o, nw, 1e-5, 0.0), gbytes=n * h * d * 6 / 1e9, like="layer norm")
+        qa, ka, va = (mk(b, s, h, d).permute(0, 2, 1, 3) for _ in range(3))
+        fl = 4.0 * b * h * s * s * d * 0.5 / 1e12
+        report(case, "prompt attention (GPT-J)", lambda: ext.flash_fwd(qa, ka, va, d ** -0.5, True, 0, None, 1),
+               gbytes=4 * n * h * d * 2 / 1e9, tflop=fl)
+        oa, lse = ext.flash_fwd(qa, ka, va, d ** -0.5, True, 0, None, 1)
+        g, sink = mk(n, h), mk(h)
+        report(case, "prompt sink + gate", lambda: ext.sink_gate(oa, lse, sink, g, d), gbytes=n * h * d * 4 / 1e9, like="layer norm")
+        x, y, gate, vec = torch.randn(n, w, device="cuda"), mk(n, w), mk(n, w), mk(w)
+        report(case, "prompt residual join", lambda: ext.residual_join(x, y, None, None, gate, vec, vec, vec, 1e-5),
+               gbytes=n * w * (4 + 2 + 2 + 4 + 2) / 1e9, like="layer norm")
+        hb = mk(n, w)
+        report(case, "layer norm (GPT-J)", lambda: ext.layernorm_fwd(hb, vec, vec, 1e-5), gbytes=n * w * 4 / 1e9)
+        rw, rb = mk(e, w), mk(e)
+        up, down = mk(e, ff, w), mk(e, w, ff)
+        report(case, "prompt route", lambda: co.moe_route(hb, rw, rb, top), gbytes=n * w * 2 / 1e9, like="layer norm")
+        idx, wgt = co.moe_route(hb, rw, rb, top)
+        slots, rows, tg, nt = ext.moe_plan(hb, idx, e)
+        report(case, "prompt plan + gather", lambda: ext.moe_plan(hb, idx, e), gbytes=n * w * (1 + top) * 2 / 1e9, like="layer norm")
+        report(case, "prompt experts up", lambda: ext.moe_grouped(rows, up, tg, nt, True), tflop=2.0 * n * top * w * ff / 1e12,
+               gbytes=(n * top * (w + ff) + e * w * ff) * 2 / 1e9, like="MLP GEMM (GPT-J)")
+        a = ext.moe_grouped(rows, up, tg, nt, True)
+        report(case, "prompt experts down", lambda: ext.moe_grouped(a, down, tg, nt, False), tflop=2.0 * n * top * w * ff / 1e12,
+               gbytes=(n * top * (w + ff) + e * w * ff) * 2 / 1e9, like="MLP GEMM (GPT-J)")
+        ye = ext.moe_grouped(a, down, tg, nt, False)
+        report(case, "prompt residual join of experts", lambda: ext.residual_join(x, ye, slots, wgt, gate, vec, vec, vec, 1e-5),
+               gbytes=n * w * (4 + 2 * top + 2 + 4 + 2) / 1e9, like="layer norm")
+        wm = mk(top * ff, w)
+        report(case, "MLP GEMM (GPT-J)", lambda: co.gemm(hb, wm), tflop=2.0 * n * w * top * ff / 1e12)
+        gu = mk(n, 2 * top * ff)
+        report(case, "prompt silu_mul", lambda: ext.silu_mul(gu[:, :top * ff], gu[:, top * ff:]), gbytes=n * top * ff * 6 / 1e9,
+               like="layer norm")
+        del p, o, qa, ka, va, oa, x, y, gate, hb, rows, a, ye, gu
+        # ------------------------------------------------ decode: 1 and 8 rows over 4096 cached tokens
+        for rows_n in (1, 8, 64):
+            t = 4096
+            p = mk(rows_n, 3 * h * d)
+            q, f, v = p[:, :h * d], p[:, h * d:2 * h * d], p[:, 2 * h * d:]
+            state = torch.zeros(rows_n, h, d, d, device="cuda")
+            report(case, f"decode {rows_n} recurrence step", lambda: ext.recurrence_step(q, f, v, fb, lo, nw, None, state, 1e-5, h, d, d),
+                   gbytes=rows_n * h * d * d * 8 / 1e9, like="decode attention (GPT-J)")
+            cache = mk(rows_n, t, kr)
+            lengths = torch.full((rows_n,), t, dtype=torch.int32, device="cuda")
+            uk, uv, qd, gd = mk(h * d, kr), mk(h * d, kr), mk(rows_n, h * d), mk(rows_n, h)
+            report(case, f"decode {rows_n} latent attention (3 launches)",
+                   lambda: ext.latent_decode(qd, uk, uv, cache, lengths, None, sink, gd, d ** -0.5, h),
+                   gbytes=(rows_n * t * kr + 2 * h * d * kr) * 2 / 1e9,
+                   tflop=4.0 * rows_n * t * h * kr / 1e12, like="decode attention (GPT-J)")
+            dq, dkv, wq, wkv = mk(rows_n, qr), mk(rows_n, kr), mk(qr), mk(kr)
+            l0 = torch.zeros(rows_n, dtype=torch.int32, device="cuda")
+            report(case, f"decode {rows_n} latent norms + append", lambda: ext.latent_prep(dq, wq, dkv, wkv, cache, l0, 1e-5),
+                   gbytes=rows_n * (qr + kr) * 4 / 1e9, like="layer norm")
+            if rows_n * t * h * d * 4 < 20e9:
+                kc, vc = mk(rows_n, h, t, d), mk(rows_n, h, t, d)
+                q3 = mk(rows_n, h, d)
+                report(case, f"decode {rows_n} attention (GPT-J, 2 launches)", lambda: ext.decode_attn(q3, kc, vc, lengths, d ** -0.5, 0),
+                       gbytes=2 * rows_n * t * h * d * 2 / 1e9)
+                del kc, vc
+            x, y, gate = torch.randn(rows_n, w, device="cuda"), mk(rows_n, w), mk(rows_n, w)
+            report(case, f"decode {rows_n} residual join", lambda: ext.residual_join(x, y, None, None, gate, vec, vec, vec, 1e-5),
+                   gbytes=rows_n * w * 14 / 1e9, like="layer norm")
+            hb = mk(rows_n, w)
+            report(case, f"decode {rows_n} layer norm (GPT-J)", lambda: ext.layernorm_fwd(hb, vec, vec, 1e-5), gbytes=rows_n * w * 4 / 1e9)
+            report(case, f"decode {rows_n} route", lambda: co.moe_route(hb, rw, rb, top), gbytes=e * w * 2 / 1e9, like="MLP GEMV (GPT-J)")
+            idx, wgt = co.moe_route(hb, rw, rb, top)
+            used = int(idx.unique().numel())
+            report(case, f"decode {rows_n} experts up + down", lambda: co.moe_experts(hb, idx, up, down),
+                   gbytes=used * w * ff * 4 / 1e9, like="MLP GEMV (GPT-J)")
+            wm, wm2 = mk(top * ff, w), mk(w, top * ff)
+            report(case, f"decode {rows_n} MLP GEMV x 2 (GPT-J)", lambda: co.linear(co.linear(hb, wm, None, False, None), wm2, None, False, None),
+                   gbytes=2 * w * top * ff * 2 / 1e9)
+            del cache
+
+
 def main() -> None:
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
-    ap.add_argument("--op", choices=["gemm", "attention"], required=True)
+    ap.add_argument("--op", choices=["gemm", "attention", "mixers"], required=True)
     ap.add_argument("--case", type=int, default=None, help="index into the op's shape list")
     ap.add_argument("--iters", type=int, default=20)
     ap.add_argument("--warmup", type=int, default=5)
     ap.add_argument("--causal", type=int, default=None, help="attention: 1 / 0 to run only one mask")
     ap.add_argument("--no-baseline", action="store_true", help="skip the library / legacy-kernel baseline")
     ap.add_argument("--no-flush", action="store_true", help="do not write a 256 MB buffer between timed calls")
+    ap.add_argument("--only", default="", help="mixers: only the entries whose name contains this")
     args = ap.parse_args()
     timer = _Timer(args.iters, args.warmup, not args.no_flush)
-    (bench_gemm if args.op == "gemm" else bench_attention)(args, timer)
+    with torch.no_grad():
+        {"gemm": bench_gemm, "attention": bench_attention, "mixers": bench_mixers}[args.op](args, timer)
 
 
 if __name__ == "__main__":

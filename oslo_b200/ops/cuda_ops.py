@@ -669,12 +669,14 @@ def pad_heads(t: Tensor, d: int) -> Tensor:
 
 def sink_attention(q: Tensor, k: Tensor, v: Tensor, keep: Optional[Tensor], sink: Tensor, gate: Tensor, scale: float) -> Tensor:
     """``q``/``k``/``v`` ``[B, S, H, *]``. 16-bit heads run on the tcgen05 flash kernel (zero-padded to the next size it has),
-    whose log-sum-exp the sink and the gate are applied with; everything else in the fp32 kernel."""
+    with sink and gate in its epilogue (value sizes that are no multiple of 8: from its log-sum-exp); everything else in the fp32 kernel."""
     d = flash_head_dim(q.size(-1), v.size(-1))
     if q.dtype in _16BIT and d and q.size(1) > 1:
         qh, kh, vh = (_attn_operand(pad_heads(t, d).permute(0, 2, 1, 3)) for t in (q, k, v))
-        o, lse = _ext().flash_fwd(qh, kh, vh, float(scale), True, 0, _keep8(keep).contiguous() if keep is not None else None,
-                                  _flash_impl())
+        kpm = _keep8(keep).contiguous() if keep is not None else None
+        if v.size(-1) % 8 == 0:
+            return _ext().flash_sink_fwd(qh, kh, vh, kpm, sink, _rows(gate), float(scale), v.size(-1))
+        o, lse = _ext().flash_fwd(qh, kh, vh, float(scale), True, 0, kpm, _flash_impl())
         return _ext().sink_gate(o, lse, sink, _rows(gate), v.size(-1))
     return _ext().sink_attention(*(t if t.stride(-1) == 1 else t.contiguous() for t in (q, k, v)), _keep8(keep), sink,
                                  _rows(gate), float(scale))

@@ -198,6 +198,10 @@ def register() -> None:
     def _(o, lse, sink, gate, vdim):
         return o.new_empty((o.size(0) * o.size(2), o.size(1) * vdim))
 
+    @reg("oslo_b200::flash_sink_fwd")
+    def _(q, k, v, kpm, sink, gate, scale, vdim):
+        return q.new_empty((q.size(0) * q.size(2), q.size(1) * vdim))
+
     @reg("oslo_b200::sink_attention")
     def _(q, k, v, keep, sink, gate, scale):
         return q.new_empty((q.size(0) * q.size(1), q.size(2) * v.size(3)))

@@ -962,15 +962,16 @@ Tensor latent_decode(const Tensor& q, const Tensor& w_uk, const Tensor& w_uv, co
   const int64_t dim = q.size(1) / heads, vdim = w_uv.size(0) / heads;
   c10::cuda::CUDAGuard guard(q.device());
   auto& st = dev_state(q.get_device());
-  const int splits = oslo_latent_splits(static_cast<int>(B), static_cast<int>(heads), static_cast<int>(T), static_cast<int>(R), st.sms);
+  const int splits = oslo_latent_splits(static_cast<int>(B), static_cast<int>(heads), static_cast<int>(T), st.sms);
   const auto f32 = q.options().dtype(at::kFloat);
   Tensor qa = at::empty({B, heads, R}, f32);
-  Tensor ws = at::empty({B, heads, splits, R + 2}, f32);
+  Tensor ws = at::empty({B, heads, splits, (R + 3) / 4 * 4}, f32);
+  Tensor stat = at::empty({B, heads, splits, 2}, f32);
   Tensor out = at::empty({B, heads * vdim}, q.options());
   check_rc(oslo_latent_decode(q.data_ptr(), q.stride(0), w_uk.data_ptr(), w_uk.stride(0), w_uv.data_ptr(), w_uv.stride(0),
                               cache.data_ptr(), lengths.data_ptr<int>(), kp, ld_keep, kp ? static_cast<int>(keep->size(1)) : 0,
                               sink.data_ptr(), gate.data_ptr(), gate.stride(0), qa.data_ptr<float>(), ws.data_ptr<float>(),
-                              out.data_ptr(), static_cast<int>(B), static_cast<int>(heads), static_cast<int>(dim),
+                              stat.data_ptr<float>(), out.data_ptr(), static_cast<int>(B), static_cast<int>(heads), static_cast<int>(dim),
                               static_cast<int>(vdim), static_cast<int>(R), static_cast<int>(T), splits,
                               static_cast<float>(scale), st.sms, dt_code(q), st.err.data_ptr<int>(), cur_stream(3)),
            "latent_decode");

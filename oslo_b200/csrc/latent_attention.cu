@@ -173,56 +173,55 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const T* __restrict__ 
   for (int c = threadIdx.x; c < n; c += blockDim.x) out[c] = Num<T>::from(Num<T>::to(x[c]) * r * Num<T>::to(w[c]));
 }
 
-// qa[b, h, r] = scale * sum_d q[b, h * dim + d] * w_uk[h * dim + d, r]; block = (64 columns r, head, 8 rows b)
-template <typename T>
+// qa[b, h, r] = scale * sum_d q[b, h * dim + d] * w_uk[h * dim + d, r]; block = (64 columns r, head, NB rows b)
+template <typename T, int VEC, int NB>
 __global__ void __launch_bounds__(256) latent_absorb_kernel(const T* __restrict__ q, long long ldq, const T* __restrict__ w,
                                                             long long ldw, float* __restrict__ qa, int B, int H, int dim,
                                                             int R, float scale) {
-  constexpr int RB = 8, CW = 64, DG = 8;
+  constexpr int CW = 64, CP = CW / VEC, DG = 256 / CP;   // VEC columns per thread, DG groups of rows d
   extern __shared__ float ab_smem[];
-  float* qs = ab_smem;                 // [RB][dim]
-  float* part = qs + RB * dim;         // [DG][RB][CW]
-  const int h = blockIdx.y, r0 = blockIdx.x * CW, b0 = blockIdx.z * RB;
-  const int nb = min(RB, B - b0);
-  for (int e = threadIdx.x; e < nb * dim; e += 256) {
-    const int b = e / dim, d = e % dim;
-    qs[b * dim + d] = Num<T>::to(q[(b0 + b) * ldq + static_cast<long long>(h) * dim + d]) * scale;
-  }
+  float* qs = ab_smem;                 // [NB][dim]
+  float* part = qs + NB * dim;         // [DG][CW], one row b at a time
+  const int h = blockIdx.y, r0 = blockIdx.x * CW, b0 = blockIdx.z * NB;
+  const int nb = min(NB, B - b0);
+  for (int b = 0; b < nb; ++b)
+    for (int d = threadIdx.x; d < dim; d += 256)
+      qs[b * dim + d] = Num<T>::to(q[(b0 + b) * ldq + static_cast<long long>(h) * dim + d]) * scale;
   __syncthreads();
-  const int cp = threadIdx.x & 31, dg = threadIdx.x >> 5;
-  const int r = r0 + cp * 2;
-  float acc[RB][2];
+  const int cp = threadIdx.x % CP, dg = threadIdx.x / CP;
+  const int r = r0 + cp * VEC;
+  float acc[NB][VEC];
 #pragma unroll
-  for (int b = 0; b < RB; ++b) acc[b][0] = acc[b][1] = 0.f;
-  if (r < R) {
-    const bool two = r + 1 < R;
-#pragma unroll 8
+  for (int b = 0; b < NB; ++b)
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) acc[b][i] = 0.f;
+  if (r < R) {                         // VEC > 1: the launcher guarantees R % VEC == 0
+    const T* wr = w + static_cast<long long>(h) * dim * ldw + r;
+#pragma unroll 4
     for (int d = dg; d < dim; d += DG) {
-      const T* wr = w + (static_cast<long long>(h) * dim + d) * ldw + r;
-      const float w0 = Num<T>::to(wr[0]), w1 = two ? Num<T>::to(wr[1]) : 0.f;
+      float v[VEC];
+      load_vec<T, VEC>(wr + d * ldw, v);
 #pragma unroll
-      for (int b = 0; b < RB; ++b) {
-        if (b < nb) {
-          const float x = qs[b * dim + d];
-          acc[b][0] = fmaf(x, w0, acc[b][0]);
-          acc[b][1] = fmaf(x, w1, acc[b][1]);
-        }
+      for (int b = 0; b < NB; ++b) {
+        const float x = b < nb ? qs[b * dim + d] : 0.f;
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) acc[b][i] = fmaf(x, v[i], acc[b][i]);
       }
     }
   }
 #pragma unroll
-  for (int b = 0; b < RB; ++b) {
-    part[(dg * RB + b) * CW + cp * 2] = acc[b][0];
-    part[(dg * RB + b) * CW + cp * 2 + 1] = acc[b][1];
-  }
-  __syncthreads();
-  for (int e = threadIdx.x; e < nb * CW; e += 256) {
-    const int b = e / CW, c = e % CW;
-    if (r0 + c >= R) continue;
-    float t = 0.f;
+  for (int b = 0; b < NB; ++b) {
+    if (b >= nb) break;                // uniform over the block
+    __syncthreads();
 #pragma unroll
-    for (int g = 0; g < DG; ++g) t += part[(g * RB + b) * CW + c];
-    qa[((static_cast<long long>(b0 + b)) * H + h) * R + r0 + c] = t;
+    for (int i = 0; i < VEC; ++i) part[dg * CW + cp * VEC + i] = acc[b][i];
+    __syncthreads();
+    if (threadIdx.x < CW && r0 + threadIdx.x < R) {
+      float t = 0.f;
+#pragma unroll
+      for (int g = 0; g < DG; ++g) t += part[g * CW + threadIdx.x];
+      qa[(static_cast<long long>(b0 + b) * H + h) * R + r0 + threadIdx.x] = t;
+    }
   }
 }
 
@@ -231,8 +230,9 @@ struct LatentDecodeParams {
   const void* cache;                   // [B, Tmax, R]
   const int* lengths;                  // [B] valid positions
   const uint8_t* keep; long long ld_keep; int n_keep;   // [B, n_keep], 0 = padded, or nullptr
-  float* ws;                           // [B, H, splits, R + 2]: sum p c, max, sum p
-  int B, H, R, Tmax, splits;
+  float* ws;                           // [B, H, splits, ldw]: sum p c; ldw = R rounded up to a multiple of 4
+  float* stat;                         // [B, H, splits, 2]: max, sum p
+  int B, H, R, ldw, Tmax, splits;
   int* err;
 };
 
@@ -315,7 +315,8 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentDecodePa
   }
   __syncthreads();
   for (int a = 0; a < nh; ++a) {
-    float* w = p.ws + ((static_cast<long long>(b) * p.H + h0 + a) * p.splits + sp) * (p.R + 2);
+    const long long at = (static_cast<long long>(b) * p.H + h0 + a) * p.splits + sp;
+    float* w = p.ws + at * p.ldw;
 #pragma unroll
     for (int j = 0; j < NR; ++j) {
       const int r = tid + j * 256;
@@ -326,16 +327,16 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentDecodePa
         w[r] = v;
       }
     }
-    if (tid == 0) { w[p.R] = ms[a]; w[p.R + 1] = ls[a]; }
+    if (tid == 0) { p.stat[at * 2] = ms[a]; p.stat[at * 2 + 1] = ls[a]; }
   }
 }
 
-// 16-bit version on the tensor cores for R % 16 == 0: the 16 heads of a group are the 16 rows of an m16n8k16 tile, so the
-// cache streams through shared memory once for all of them. 8 warps; per KT cached vectors:
-//   scores  the warps cover the KT / 8 key columns (and halves of R when KT = 32); q' is split into two 16-bit terms
-//   softmax warp w owns heads 2 w and 2 w + 1 (running max and sum in registers), P is stored as 16-bit
+// 16-bit version on the tensor cores for R % 16 == 0: MT x 16 heads are the rows of m16n8k16 tiles, so the cache streams
+// through shared memory once for all of them. 8 warps, LM_KT cached vectors per step:
+//   scores  warp = (16 heads) x (16 of the keys) x (a half or a quarter of R); q' as 16-bit, 32-bit sums
+//   softmax warp w owns heads 2 MT w ..; lane = key; running max and sum in registers, P is stored as 16-bit
 //   output  a warp owns every eighth pair of 8-column blocks of R; the cached vectors are read transposed
-// The next KT vectors are fetched with cp.async meanwhile.
+// The next vectors are fetched with cp.async meanwhile, and two blocks per SM overlap each other's phases.
 template <typename T> struct MmaT;
 template <> struct MmaT<__nv_bfloat16> {
   static __device__ __forceinline__ void mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
@@ -355,238 +356,400 @@ __device__ __forceinline__ void ldsm4(uint32_t addr, uint32_t (&r)[4]) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
 }
-__device__ __forceinline__ void ldsm2(uint32_t addr, uint32_t& r0, uint32_t& r1) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(r0), "=r"(r1) : "r"(addr));
+__device__ __forceinline__ void ldsm2_t(uint32_t addr, uint32_t& r0, uint32_t& r1) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];" : "=r"(r0), "=r"(r1) : "r"(addr));
 }
 __device__ __forceinline__ void ldsm4_t(uint32_t addr, uint32_t (&r)[4]) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
 }
 
-template <typename T, int KT, int NP>   // KT cached vectors per step (64 or 32), NP pairs of 8-column blocks per warp
-__global__ void __launch_bounds__(256, 1) latent_decode_mma_kernel(const LatentDecodeParams p) {
-  constexpr int KS = KT == 64 ? 1 : 2;  // slices of R in the score product
-  constexpr int PP = KT + 8;            // padded row of P
+// 16-bit, 16 rows b at a time on the tensor cores: qa[b, h, r] = scale * sum_d q[b, d] w_uk[d, r]. Block = (64 columns r, head,
+// 16 rows); W_uk's [dim, 64] tile goes through shared memory and is read transposed; dim % 16 == 0, R % 8 == 0.
+template <typename T>
+__global__ void __launch_bounds__(256) latent_absorb_mma_kernel(const T* __restrict__ q, long long ldq, const T* __restrict__ w,
+                                                                long long ldw, float* __restrict__ qa, int B, int H, int dim,
+                                                                int R, float scale) {
+  constexpr int CW = 64, WP = CW + 8;
+  extern __shared__ __align__(16) uint8_t am_smem[];
+  const int qp = dim + 8;
+  T* qs = reinterpret_cast<T*>(am_smem);   // [16][qp]
+  T* wsm = qs + 16 * qp;                   // [dim][WP]
+  const int h = blockIdx.y, r0 = blockIdx.x * CW, b0 = blockIdx.z * 16;
+  const int nb = min(16, B - b0), nc = min(CW, R - r0) / 8;   // 16-byte pieces of a tile row
+  for (int e = threadIdx.x; e < dim * 8; e += 256) {
+    const int d = e >> 3, v = e & 7;
+    const bool in = v < nc;                // columns past R are zero-filled
+    const T* src = w + (static_cast<long long>(h) * dim + d) * ldw + r0 + (in ? v * 8 : 0);
+    const int bytes = in ? 16 : 0;
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(wsm + d * WP + v * 8)), "l"(src), "r"(bytes) : "memory");
+  }
+  asm volatile("cp.async.commit_group;" ::: "memory");
+  for (int e = threadIdx.x; e < 16 * dim; e += 256) {
+    const int b = e / dim, d = e - b * dim;
+    qs[b * qp + d] = b < nb ? q[(b0 + b) * ldq + static_cast<long long>(h) * dim + d] : Num<T>::from(0.f);
+  }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  __syncthreads();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  float acc[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 4
+  for (int s = 0; s < dim / 16; ++s) {
+    uint32_t a[4], b0r, b1r;
+    ldsm4(smem_u32(qs + (lane & 15) * qp + s * 16 + (lane >> 4) * 8), a);
+    ldsm2_t(smem_u32(wsm + (s * 16 + (lane & 15)) * WP + warp * 8), b0r, b1r);
+    MmaT<T>::mma(acc, a, b0r, b1r);
+  }
+  const int col = r0 + warp * 8 + (lane & 3) * 2;
+  if (col < R) {                           // R is even
+#pragma unroll
+    for (int hf = 0; hf < 2; ++hf) {
+      const int b = (lane >> 2) + 8 * hf;
+      if (b < nb)
+        *reinterpret_cast<float2*>(qa + (static_cast<long long>(b0 + b) * H + h) * R + col) =
+            make_float2(acc[hf * 2] * scale, acc[hf * 2 + 1] * scale);
+    }
+  }
+}
+
+constexpr int LM_KT = 32;
+
+template <typename T, int MT, int NP>   // MT groups of 16 heads, NP pairs of 8-column blocks per warp
+__global__ void __launch_bounds__(256, NP <= 4 ? 2 : 1) latent_decode_mma_kernel(const LatentDecodeParams p) {
+  constexpr int HM = 16 * MT, PP = LM_KT + 8, SP = LM_KT + 1, KS = 4 / MT;
   extern __shared__ __align__(16) uint8_t lm_smem[];
   const int rp = p.R + 8;               // padded row: 16-byte aligned, conflict-free ldmatrix
-  T* q_hi = reinterpret_cast<T*>(lm_smem);          // [16][rp]
-  T* q_lo = q_hi + 16 * rp;
-  T* cs = q_lo + 16 * rp;                           // [2][KT][rp]
-  T* ps = cs + 2 * KT * rp;                         // [16][PP]
-  float* ss = reinterpret_cast<float*>(ps + 16 * PP);   // [KS][16][KT + 1]
-  float* fac = ss + KS * 16 * (KT + 1);             // [16]
-  const int b = blockIdx.z, h0 = blockIdx.y * LD_HEADS, sp = blockIdx.x, tid = threadIdx.x;
+  T* qs = reinterpret_cast<T*>(lm_smem);            // [HM][rp]
+  T* cs = qs + HM * rp;                             // [2][LM_KT][rp]
+  T* ps = cs + 2 * LM_KT * rp;                      // [HM][PP]
+  float* ss = reinterpret_cast<float*>(ps + HM * PP);   // [KS][HM][SP]
+  float* fac = ss + KS * HM * SP;                // [HM]
+  const int b = blockIdx.z, h0 = blockIdx.y * HM, sp = blockIdx.x, tid = threadIdx.x;
   const int warp = tid >> 5, lane = tid & 31;
-  const int nh = min(LD_HEADS, p.H - h0);
+  const int nh = min(HM, p.H - h0);
   int len = p.lengths[b];
   if (len < 0 || len > p.Tmax) {       // a length that does not fit the cache: never read past it
     if (tid == 0) OSLO_REPORT_BOUNDS(p.err);
     len = len < 0 ? 0 : p.Tmax;
   }
-  const int tiles = (len + KT - 1) / KT, per = (tiles + p.splits - 1) / p.splits * KT;
+  const int tiles = (len + LM_KT - 1) / LM_KT, per = (tiles + p.splits - 1) / p.splits * LM_KT;
   const int t0 = sp * per, t1 = min(len, t0 + per);
   const T* c = static_cast<const T*>(p.cache) + static_cast<long long>(b) * p.Tmax * p.R;
   const int vr = p.R / 8;              // 16-byte pieces of a cached vector
+  const int dt = 256 / vr, dv = 256 % vr, ft = tid / vr, fv = tid % vr;
   auto fetch = [&](int k0, int buf) {
-    T* dst = cs + static_cast<size_t>(buf) * KT * rp;
-    for (int e = tid; e < KT * vr; e += 256) {
-      const int t = e / vr, v = e - t * vr;
+    T* dst = cs + static_cast<size_t>(buf) * LM_KT * rp;
+    int t = ft, v = fv;
+    while (t < LM_KT) {
       const uint32_t d32 = smem_u32(dst + t * rp + v * 8);
       const bool in = k0 + t < t1;     // rows past the slice are zero-filled (source size 0)
       const T* src = c + static_cast<long long>(in ? k0 + t : 0) * p.R + v * 8;
       const int bytes = in ? 16 : 0;
       asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d32), "l"(src), "r"(bytes) : "memory");
+      t += dt;
+      v += dv;
+      if (v >= vr) { v -= vr; ++t; }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   if (t0 < t1) fetch(t0, 0);
-  for (int e = tid; e < 16 * p.R; e += 256) {
-    const int a = e / p.R, r = e - a * p.R;
-    const float x = a < nh ? p.qa[(static_cast<long long>(b) * p.H + h0 + a) * p.R + r] : 0.f;
-    const T hi = Num<T>::from(x);
-    q_hi[a * rp + r] = hi;
-    q_lo[a * rp + r] = Num<T>::from(x - Num<T>::to(hi));
+  for (int a = warp; a < HM; a += 8) {
+    const float* src = p.qa + (static_cast<long long>(b) * p.H + h0 + a) * p.R;
+#pragma unroll 4
+    for (int r = lane * 4; r < p.R; r += 128) {
+      float x[4] = {0.f, 0.f, 0.f, 0.f};
+      if (a < nh) load_vec<float, 4>(src + r, x);
+      store_vec<T, 4>(qs + a * rp + r, x);
+    }
   }
-  float acc[NP][2][4];
+  float acc[MT][NP][2][4];
 #pragma unroll
-  for (int j = 0; j < NP; ++j)
+  for (int m = 0; m < MT; ++m)
 #pragma unroll
-    for (int u = 0; u < 2; ++u)
+    for (int j = 0; j < NP; ++j)
 #pragma unroll
-      for (int i = 0; i < 4; ++i) acc[j][u][i] = 0.f;
-  float m_run[2] = {-CUDART_INF_F, -CUDART_INF_F}, l_run[2] = {0.f, 0.f};
+      for (int u = 0; u < 2; ++u)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) acc[m][j][u][i] = 0.f;
+  float m_run[2 * MT], l_run[2 * MT];
+#pragma unroll
+  for (int u = 0; u < 2 * MT; ++u) { m_run[u] = -CUDART_INF_F; l_run[u] = 0.f; }
   const int arow = lane & 15, acol = (lane >> 4) * 8;      // ldmatrix.x4 source of an A fragment
-  for (int k0 = t0, it = 0; k0 < t1; k0 += KT, ++it) {
+  const int kg = warp & 1, mt = (warp >> 1) % MT, ks = (warp >> 1) / MT;
+  const int n16 = p.R / 16, s_begin = ks * n16 / KS, s_end = (ks + 1) * n16 / KS;
+  // B fragments of 16 keys x 16 columns: matrices (keys 0-7, cols 0-7), (keys 0-7, cols 8-15), (keys 8-15, ...)
+  const int brow = kg * 16 + (lane & 7) + ((lane >> 4) << 3), bcol = ((lane >> 3) & 1) * 8;
+  for (int k0 = t0, it = 0; k0 < t1; k0 += LM_KT, ++it) {
     const int buf = it & 1;
-    if (k0 + KT < t1) {                                    // the other buffer was last read before the closing barrier
-      fetch(k0 + KT, buf ^ 1);
+    if (k0 + LM_KT < t1) {                                 // the other buffer was last read before the closing barrier
+      fetch(k0 + LM_KT, buf ^ 1);
       asm volatile("cp.async.wait_group 1;" ::: "memory");
     } else {
       asm volatile("cp.async.wait_group 0;" ::: "memory");
     }
     __syncthreads();
-    const T* ct = cs + static_cast<size_t>(buf) * KT * rp;
+    const T* ct = cs + static_cast<size_t>(buf) * LM_KT * rp;
     {
-      const int kg = warp % (KT / 8), ks = warp / (KT / 8);
-      const int n16 = p.R / 16, s_begin = ks * n16 / KS, s_end = (ks + 1) * n16 / KS;
-      float d[4] = {0.f, 0.f, 0.f, 0.f}, e[4] = {0.f, 0.f, 0.f, 0.f};
+      float d[2][4];
+#pragma unroll
+      for (int u = 0; u < 2; ++u)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) d[u][i] = 0.f;
+#pragma unroll 4
       for (int s = s_begin; s < s_end; ++s) {
-        uint32_t ah[4], al[4], b0, b1;
-        ldsm4(smem_u32(q_hi + arow * rp + s * 16 + acol), ah);
-        ldsm4(smem_u32(q_lo + arow * rp + s * 16 + acol), al);
-        ldsm2(smem_u32(ct + (kg * 8 + (lane & 7)) * rp + s * 16 + ((lane >> 3) & 1) * 8), b0, b1);
-        MmaT<T>::mma(d, ah, b0, b1);
-        MmaT<T>::mma(e, al, b0, b1);
+        uint32_t a[4], bb[4];
+        ldsm4(smem_u32(ct + brow * rp + s * 16 + bcol), bb);
+        ldsm4(smem_u32(qs + (mt * 16 + arow) * rp + s * 16 + acol), a);
+        MmaT<T>::mma(d[0], a, bb[0], bb[1]);
+        MmaT<T>::mma(d[1], a, bb[2], bb[3]);
       }
-      float* o = ss + ks * 16 * (KT + 1) + (lane >> 2) * (KT + 1) + kg * 8 + (lane & 3) * 2;
-      o[0] = d[0] + e[0]; o[1] = d[1] + e[1];
-      o[8 * (KT + 1)] = d[2] + e[2]; o[8 * (KT + 1) + 1] = d[3] + e[3];
-    }
-    __syncthreads();
-#pragma unroll
-    for (int u = 0; u < 2; ++u) {
-      const int a = warp * 2 + u;
-      float x[KT / 32], mx = m_run[u];
-#pragma unroll
-      for (int i = 0; i < KT / 32; ++i) {
-        const int t = lane + 32 * i, pos = k0 + t;
-        float v = ss[a * (KT + 1) + t];
-        if (KS == 2) v += ss[16 * (KT + 1) + a * (KT + 1) + t];
-        const bool vis = pos < t1 && (p.keep == nullptr || pos >= p.n_keep || p.keep[b * p.ld_keep + pos]);
-        x[i] = vis ? v : -CUDART_INF_F;
-        mx = fmaxf(mx, x[i]);
-      }
-#pragma unroll
-      for (int off = 16; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
-      float sum = 0.f;
-#pragma unroll
-      for (int i = 0; i < KT / 32; ++i) {
-        const float pr = x[i] == -CUDART_INF_F ? 0.f : expf(x[i] - mx);
-        sum += pr;
-        ps[a * PP + lane + 32 * i] = Num<T>::from(pr);
-      }
-      sum = warp_sum(sum);
-      const float f = m_run[u] == -CUDART_INF_F ? 0.f : expf(m_run[u] - mx);
-      l_run[u] = l_run[u] * f + sum;
-      m_run[u] = mx;
-      if (lane == 0) fac[a] = f;
-    }
-    __syncthreads();
-    const float f0 = fac[lane >> 2], f1 = fac[(lane >> 2) + 8];
-#pragma unroll
-    for (int j = 0; j < NP; ++j)
 #pragma unroll
       for (int u = 0; u < 2; ++u) {
-        acc[j][u][0] *= f0; acc[j][u][1] *= f0; acc[j][u][2] *= f1; acc[j][u][3] *= f1;
+        float* o = ss + (ks * HM + mt * 16 + (lane >> 2)) * SP + kg * 16 + u * 8 + (lane & 3) * 2;
+        o[0] = d[u][0]; o[1] = d[u][1];
+        o[8 * SP] = d[u][2]; o[8 * SP + 1] = d[u][3];
+      }
+    }
+    __syncthreads();
+    {
+      const int pos = k0 + lane;
+      const bool vis = pos < t1 && (p.keep == nullptr || pos >= p.n_keep || p.keep[b * p.ld_keep + pos]);
+      float x[2 * MT], mx[2 * MT], sum[2 * MT];
+#pragma unroll
+      for (int u = 0; u < 2 * MT; ++u) {
+        const float* o = ss + (warp * 2 * MT + u) * SP + lane;
+        float v = o[0];
+#pragma unroll
+        for (int k = 1; k < KS; ++k) v += o[k * HM * SP];
+        x[u] = vis ? v : -CUDART_INF_F;
+        mx[u] = fmaxf(m_run[u], x[u]);
       }
 #pragma unroll
-    for (int s = 0; s < KT / 16; ++s) {
-      uint32_t a[4];
-      ldsm4(smem_u32(ps + arow * PP + s * 16 + acol), a);
+      for (int off = 16; off > 0; off >>= 1)
+#pragma unroll
+        for (int u = 0; u < 2 * MT; ++u) mx[u] = fmaxf(mx[u], __shfl_xor_sync(0xffffffffu, mx[u], off));
+#pragma unroll
+      for (int u = 0; u < 2 * MT; ++u) {
+        sum[u] = x[u] == -CUDART_INF_F ? 0.f : expf(x[u] - mx[u]);
+        ps[(warp * 2 * MT + u) * PP + lane] = Num<T>::from(sum[u]);
+      }
+#pragma unroll
+      for (int off = 16; off > 0; off >>= 1)
+#pragma unroll
+        for (int u = 0; u < 2 * MT; ++u) sum[u] += __shfl_xor_sync(0xffffffffu, sum[u], off);
+#pragma unroll
+      for (int u = 0; u < 2 * MT; ++u) {
+        const float f = m_run[u] == -CUDART_INF_F ? 0.f : expf(m_run[u] - mx[u]);
+        l_run[u] = l_run[u] * f + sum[u];
+        m_run[u] = mx[u];
+        if (lane == 0) fac[warp * 2 * MT + u] = f;
+      }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int m = 0; m < MT; ++m) {
+      const float f0 = fac[m * 16 + (lane >> 2)], f1 = fac[m * 16 + (lane >> 2) + 8];
+#pragma unroll
+      for (int j = 0; j < NP; ++j)
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+          acc[m][j][u][0] *= f0; acc[m][j][u][1] *= f0; acc[m][j][u][2] *= f1; acc[m][j][u][3] *= f1;
+        }
+    }
+#pragma unroll
+    for (int s = 0; s < LM_KT / 16; ++s) {
+      uint32_t a[MT][4];
+#pragma unroll
+      for (int m = 0; m < MT; ++m) ldsm4(smem_u32(ps + (m * 16 + arow) * PP + s * 16 + acol), a[m]);
 #pragma unroll
       for (int j = 0; j < NP; ++j) {
         const int col = (warp + 8 * j) * 16;
         if (col < p.R) {                                   // uniform over the warp
           uint32_t bb[4];
           ldsm4_t(smem_u32(ct + (s * 16 + (lane & 15)) * rp + col + (lane >> 4) * 8), bb);
-          MmaT<T>::mma(acc[j][0], a, bb[0], bb[1]);
-          MmaT<T>::mma(acc[j][1], a, bb[2], bb[3]);
+#pragma unroll
+          for (int m = 0; m < MT; ++m) {
+            MmaT<T>::mma(acc[m][j][0], a[m], bb[0], bb[1]);
+            MmaT<T>::mma(acc[m][j][1], a[m], bb[2], bb[3]);
+          }
         }
       }
     }
     __syncthreads();
   }
 #pragma unroll
-  for (int j = 0; j < NP; ++j) {
-    const int col = (warp + 8 * j) * 16;
-    if (col >= p.R) continue;
+  for (int m = 0; m < MT; ++m)
 #pragma unroll
-    for (int u = 0; u < 2; ++u)
+    for (int j = 0; j < NP; ++j) {
+      const int col = (warp + 8 * j) * 16;
+      if (col >= p.R) continue;
 #pragma unroll
-      for (int hf = 0; hf < 2; ++hf) {
-        const int a = (lane >> 2) + 8 * hf;
-        if (a < nh) {
-          float* w = p.ws + ((static_cast<long long>(b) * p.H + h0 + a) * p.splits + sp) * (p.R + 2) + col + u * 8 + (lane & 3) * 2;
-          w[0] = acc[j][u][hf * 2];
-          w[1] = acc[j][u][hf * 2 + 1];
+      for (int u = 0; u < 2; ++u)
+#pragma unroll
+        for (int hf = 0; hf < 2; ++hf) {
+          const int a = m * 16 + (lane >> 2) + 8 * hf;
+          if (a < nh) {
+            float* w = p.ws + ((static_cast<long long>(b) * p.H + h0 + a) * p.splits + sp) * p.ldw + col + u * 8 + (lane & 3) * 2;
+            *reinterpret_cast<float2*>(w) = make_float2(acc[m][j][u][hf * 2], acc[m][j][u][hf * 2 + 1]);
+          }
         }
-      }
-  }
+    }
 #pragma unroll
-  for (int u = 0; u < 2; ++u) {
-    const int a = warp * 2 + u;
+  for (int u = 0; u < 2 * MT; ++u) {
+    const int a = warp * 2 * MT + u;
     if (lane == 0 && a < nh) {
-      float* w = p.ws + ((static_cast<long long>(b) * p.H + h0 + a) * p.splits + sp) * (p.R + 2) + p.R;
+      float* w = p.stat + ((static_cast<long long>(b) * p.H + h0 + a) * p.splits + sp) * 2;
       w[0] = m_run[u];
       w[1] = l_run[u];
     }
   }
 }
-static size_t latent_mma_smem(int R, int kt) {
-  const size_t rp = R + 8;
-  return (32 * rp + 2 * kt * rp + 16 * (kt + 8)) * 2 + ((kt == 64 ? 1 : 2) * 16 * (kt + 1) + 16) * sizeof(float);
+static size_t latent_mma_smem(int R, int mt) {
+  const size_t rp = R + 8, hm = 16 * mt;
+  return (hm * rp + 2 * LM_KT * rp + hm * (LM_KT + 8)) * 2 + (4 / mt * hm * (LM_KT + 1) + hm) * sizeof(float);
+}
+
+// the slice weights of one row (all lanes of a warp): wt[s] = exp(max_s - max) * gate / denominator
+template <typename T>
+__device__ __forceinline__ void slice_weights(const LatentDecodeParams& p, int b, int h, float snk, float gate, float* wt, int lane) {
+  const float2* st = reinterpret_cast<const float2*>(p.stat) + (static_cast<long long>(b) * p.H + h) * p.splits;
+  float m = snk;
+  for (int s = lane; s < p.splits; s += 32) m = fmaxf(m, st[s].x);
+#pragma unroll
+  for (int off = 16; off > 0; off >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, off));
+  float tot = 0.f;
+  for (int s = lane; s < p.splits; s += 32) {
+    const float2 ml = st[s];
+    const float f = ml.x == -CUDART_INF_F ? 0.f : expf(ml.x - m);
+    tot += f * ml.y;
+    wt[s] = f;
+  }
+  const float g = sigmoid_f(gate) / (warp_sum(tot) + expf(snk - m));
+  for (int s = lane; s < p.splits; s += 32) wt[s] *= g;
 }
 
 // out[b, h * vdim + j] = sigmoid(g) * sum_r w_uv[h * vdim + j, r] * o[r],  o = merged slices / (sum + exp(sink))
-// for NB rows b per block, so that W_uv is read once for all of them
+// for NB rows b per block, so that W_uv is read once for all of them; a warp computes 4 of the j at a time
 template <typename T, int VEC, int NB>
-__global__ void __launch_bounds__(256) latent_finish_kernel(const float* __restrict__ ws, const T* __restrict__ w, long long ldw,
+__global__ void __launch_bounds__(256) latent_finish_kernel(const LatentDecodeParams p, const T* __restrict__ w, long long ldw,
                                                             const T* __restrict__ sink, const T* __restrict__ gate,
-                                                            long long ldg, T* __restrict__ out, int B, int H, int R, int vdim,
-                                                            int splits, int rows_per_block) {
-  extern __shared__ float fin_smem[];   // [NB][R] then [NB][splits] weights
+                                                            long long ldg, T* __restrict__ out, int vdim, int rows_per_block) {
+  extern __shared__ __align__(16) float fin_smem[];   // [NB][p.ldw] then [NB][splits] weights
   float* o = fin_smem;
-  float* wt = fin_smem + NB * R;
-  const int h = blockIdx.y, b0 = blockIdx.z * NB, nb = min(NB, B - b0);
+  float* wt = fin_smem + NB * p.ldw;
+  const int h = blockIdx.y, b0 = blockIdx.z * NB, nb = min(NB, p.B - b0), R = p.R, splits = p.splits;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const float snk = Num<T>::to(sink[h]);
-  for (int i = warp; i < nb; i += 8) {  // slice weights of a row, already divided by the denominator and gated
-    const float* st = ws + (static_cast<long long>(b0 + i) * H + h) * splits * (R + 2) + R;
-    float m = snk;
-    for (int s = lane; s < splits; s += 32) m = fmaxf(m, st[static_cast<long long>(s) * (R + 2)]);
-#pragma unroll
-    for (int off = 16; off > 0; off >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, off));
-    float tot = 0.f;
-    for (int s = lane; s < splits; s += 32) {
-      const float ms = st[static_cast<long long>(s) * (R + 2)];
-      const float f = ms == -CUDART_INF_F ? 0.f : expf(ms - m);
-      tot += f * st[static_cast<long long>(s) * (R + 2) + 1];
-      wt[i * splits + s] = f;
-    }
-    tot = warp_sum(tot) + expf(snk - m);
-    const float inv = sigmoid_f(Num<T>::to(gate[(b0 + i) * ldg + h])) / tot;
-    for (int s = lane; s < splits; s += 32) wt[i * splits + s] *= inv;
-  }
+  for (int i = warp; i < nb; i += 8)
+    slice_weights<T>(p, b0 + i, h, snk, Num<T>::to(gate[(b0 + i) * ldg + h]), wt + i * splits, lane);
   __syncthreads();
-  for (int e = threadIdx.x; e < nb * R; e += blockDim.x) {
-    const int i = e / R, r = e - i * R;
-    const float* base = ws + (static_cast<long long>(b0 + i) * H + h) * splits * (R + 2) + r;
-    float v = 0.f;
+  const int quads = p.ldw / 4;
+  for (int e = threadIdx.x; e < nb * quads; e += 256) {
+    const int i = e / quads, c = e - i * quads;
+    const float* base = p.ws + (static_cast<long long>(b0 + i) * p.H + h) * splits * p.ldw + c * 4;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll 8
-    for (int s = 0; s < splits; ++s) v = fmaf(wt[i * splits + s], base[static_cast<long long>(s) * (R + 2)], v);
-    o[i * R + r] = v;
+    for (int s = 0; s < splits; ++s) {
+      const float4 x = *reinterpret_cast<const float4*>(base + static_cast<long long>(s) * p.ldw);
+      const float f = wt[i * splits + s];
+      v.x = fmaf(f, x.x, v.x); v.y = fmaf(f, x.y, v.y); v.z = fmaf(f, x.z, v.z); v.w = fmaf(f, x.w, v.w);
+    }
+    *reinterpret_cast<float4*>(o + i * p.ldw + c * 4) = v;   // columns past R are never read below
   }
   __syncthreads();
+  constexpr int JR = 4;
   const int j1 = min(vdim, (static_cast<int>(blockIdx.x) + 1) * rows_per_block);
-  for (int j = blockIdx.x * rows_per_block + warp; j < j1; j += 8) {
+  for (int j = blockIdx.x * rows_per_block + warp * JR; j < j1; j += 8 * JR) {
     const T* wr = w + (static_cast<long long>(h) * vdim + j) * ldw;
-    float acc[NB];
+    const int nj = min(JR, j1 - j);
+    float acc[JR][NB];
 #pragma unroll
-    for (int i = 0; i < NB; ++i) acc[i] = 0.f;
+    for (int a = 0; a < JR; ++a)
+#pragma unroll
+      for (int i = 0; i < NB; ++i) acc[a][i] = 0.f;
+#pragma unroll 2
     for (int k = lane * VEC; k < R; k += 32 * VEC) {
-      float x[VEC];
-      load_vec<T, VEC>(wr + k, x);
+      float x[JR][VEC];
+#pragma unroll
+      for (int a = 0; a < JR; ++a)
+        if (a < nj) load_vec<T, VEC>(wr + a * ldw + k, x[a]);
+        else {
+#pragma unroll
+          for (int u = 0; u < VEC; ++u) x[a][u] = 0.f;
+        }
 #pragma unroll
       for (int i = 0; i < NB; ++i)
         if (i < nb) {
 #pragma unroll
-          for (int u = 0; u < VEC; ++u) acc[i] = fmaf(x[u], o[i * R + k + u], acc[i]);
+          for (int u = 0; u < VEC; ++u) {
+            const float y = o[i * p.ldw + k + u];
+#pragma unroll
+            for (int a = 0; a < JR; ++a) acc[a][i] = fmaf(x[a][u], y, acc[a][i]);
+          }
         }
     }
 #pragma unroll
-    for (int i = 0; i < NB; ++i) {
-      const float d = warp_sum(acc[i]);
-      if (lane == 0 && i < nb) out[(static_cast<long long>(b0 + i) * H + h) * vdim + j] = Num<T>::from(d);
+    for (int a = 0; a < JR; ++a)
+#pragma unroll
+      for (int i = 0; i < NB; ++i) {
+        const float d = warp_sum(acc[a][i]);
+        if (lane == 0 && i < nb && a < nj) out[(static_cast<long long>(b0 + i) * p.H + h) * vdim + j + a] = Num<T>::from(d);
+      }
+  }
+}
+
+// 16-bit, 16 rows b at a time on the tensor cores; R % 32 == 0, vdim % 8 == 0. A lane fetches 8 consecutive elements of its
+// column's W_uv row with one load and uses them as two k steps; the A operand is permuted alike, so no shuffles are needed.
+template <typename T>
+__global__ void __launch_bounds__(256) latent_finish_mma_kernel(const LatentDecodeParams p, const T* __restrict__ w, long long ldw,
+                                                                const T* __restrict__ sink, const T* __restrict__ gate,
+                                                                long long ldg, T* __restrict__ out, int vdim) {
+  extern __shared__ __align__(16) uint8_t fm_smem[];
+  const int op = p.R + 8, quads = p.R / 4;
+  T* o = reinterpret_cast<T*>(fm_smem);                    // [16][op]
+  float* wt = reinterpret_cast<float*>(o + 16 * op);       // [16][splits]
+  const int h = blockIdx.y, b0 = blockIdx.z * 16, nb = min(16, p.B - b0);
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const float snk = Num<T>::to(sink[h]);
+  for (int i = warp; i < nb; i += 8)
+    slice_weights<T>(p, b0 + i, h, snk, Num<T>::to(gate[(b0 + i) * ldg + h]), wt + i * p.splits, lane);
+  __syncthreads();
+#pragma unroll 2
+  for (int e = threadIdx.x; e < 16 * quads; e += 256) {
+    const int i = e / quads, c = e - i * quads;
+    float v[4] = {0.f, 0.f, 0.f, 0.f};
+    if (i < nb) {
+      const float* base = p.ws + (static_cast<long long>(b0 + i) * p.H + h) * p.splits * p.ldw + c * 4;
+#pragma unroll 4
+      for (int s = 0; s < p.splits; ++s) {
+        const float4 x = *reinterpret_cast<const float4*>(base + static_cast<long long>(s) * p.ldw);
+        const float f = wt[i * p.splits + s];
+        v[0] = fmaf(f, x.x, v[0]); v[1] = fmaf(f, x.y, v[1]); v[2] = fmaf(f, x.z, v[2]); v[3] = fmaf(f, x.w, v[3]);
+      }
+    }
+    store_vec<T, 4>(o + i * op + c * 4, v);
+  }
+  __syncthreads();
+  const int g = lane >> 2, t = lane & 3;
+  for (int j0 = (blockIdx.x * 8 + warp) * 8; j0 < vdim; j0 += gridDim.x * 64) {
+    const T* wr = w + (static_cast<long long>(h) * vdim + j0 + g) * ldw + t * 8;
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 8
+    for (int k = 0; k < p.R; k += 32) {
+      const uint4 bv = *reinterpret_cast<const uint4*>(wr + k);
+      const uint4 a0 = *reinterpret_cast<const uint4*>(o + g * op + k + t * 8);
+      const uint4 a1 = *reinterpret_cast<const uint4*>(o + (g + 8) * op + k + t * 8);
+      const uint32_t s0[4] = {a0.x, a1.x, a0.y, a1.y}, s1[4] = {a0.z, a1.z, a0.w, a1.w};
+      MmaT<T>::mma(acc, s0, bv.x, bv.y);
+      MmaT<T>::mma(acc, s1, bv.z, bv.w);
+    }
+#pragma unroll
+    for (int hf = 0; hf < 2; ++hf) {
+      const int b = g + 8 * hf;
+      if (b < nb) {
+        const float v[2] = {acc[hf * 2], acc[hf * 2 + 1]};
+        store_vec<T, 2>(out + (static_cast<long long>(b0 + b) * p.H + h) * vdim + j0 + t * 2, v);
+      }
     }
   }
 }
@@ -652,31 +815,38 @@ namespace oslo {
 
 template <typename T>
 static int latent_scan(const LatentDecodeParams& p, int use_mma, cudaStream_t st) {
-  dim3 grid(p.splits, (p.H + LD_HEADS - 1) / LD_HEADS, p.B);
   if constexpr (sizeof(T) == 2) {
     if (use_mma) {
-      const int kt = p.R <= 512 ? 64 : 32, np = (p.R + 127) / 128;
-      const size_t smem = latent_mma_smem(p.R, kt);
-#define LM_GO(KT, NP)                                                                                   \
+      const int mt = p.H > LD_HEADS ? 2 : 1, np = (p.R + 127) / 128;
+      const size_t smem = latent_mma_smem(p.R, mt);
+      dim3 grid(p.splits, (p.H + 16 * mt - 1) / (16 * mt), p.B);
+#define LM_GO(MT, NP)                                                                                   \
   {                                                                                                     \
-    const int rc = set_smem(reinterpret_cast<const void*>(&latent_decode_mma_kernel<T, KT, NP>), smem); \
+    const int rc = set_smem(reinterpret_cast<const void*>(&latent_decode_mma_kernel<T, MT, NP>), smem); \
     if (rc) return rc;                                                                                  \
-    latent_decode_mma_kernel<T, KT, NP><<<grid, 256, smem, st>>>(p);                                    \
+    latent_decode_mma_kernel<T, MT, NP><<<grid, 256, smem, st>>>(p);                                    \
     return static_cast<int>(cudaGetLastError());                                                        \
   }
-      if (np == 1) LM_GO(64, 1)
-      if (np == 2) LM_GO(64, 2)
-      if (np <= 4) LM_GO(64, 4)
-      LM_GO(32, 8)
+      if (mt == 1) {
+        if (np == 1) LM_GO(1, 1)
+        if (np == 2) LM_GO(1, 2)
+        if (np <= 4) LM_GO(1, 4)
+        LM_GO(1, 8)
+      }
+      if (np == 1) LM_GO(2, 1)
+      if (np == 2) LM_GO(2, 2)
+      if (np <= 4) LM_GO(2, 4)
+      LM_GO(2, 8)
 #undef LM_GO
     }
   }
+  dim3 grid(p.splits, (p.H + LD_HEADS - 1) / LD_HEADS, p.B);
   const size_t smem = (static_cast<size_t>(LD_HEADS + LD_KEYS) * (p.R + 1) + LD_HEADS * LD_KEYS) * sizeof(float);
-#define LD_GO(NR)                                                                             \
-  {                                                                                           \
+#define LD_GO(NR)                                                                               \
+  {                                                                                             \
     const int rc = set_smem(reinterpret_cast<const void*>(&latent_decode_kernel<T, NR>), smem); \
-    if (rc) return rc;                                                                        \
-    latent_decode_kernel<T, NR><<<grid, 256, smem, st>>>(p);                                  \
+    if (rc) return rc;                                                                          \
+    latent_decode_kernel<T, NR><<<grid, 256, smem, st>>>(p);                                    \
   }
   if (p.R <= 256) LD_GO(1)
   else if (p.R <= 512) LD_GO(2)
@@ -686,18 +856,60 @@ static int latent_scan(const LatentDecodeParams& p, int use_mma, cudaStream_t st
 }
 
 template <typename T, int VEC>
+static int latent_absorb(const LatentDecodeParams& p, const void* q, long long ldq, const void* w, long long ldw, float* qa,
+                         int dim, float scale, cudaStream_t st) {
+  if constexpr (sizeof(T) == 2 && VEC == 8) {
+    if (p.B > 2 && dim % 16 == 0) {
+      const size_t smem = (16 * static_cast<size_t>(dim + 8) + static_cast<size_t>(dim) * 72) * 2;
+      const int rc = set_smem(reinterpret_cast<const void*>(&latent_absorb_mma_kernel<T>), smem);
+      if (rc) return rc;
+      latent_absorb_mma_kernel<T><<<dim3((p.R + 63) / 64, p.H, (p.B + 15) / 16), 256, smem, st>>>(
+          static_cast<const T*>(q), ldq, static_cast<const T*>(w), ldw, qa, p.B, p.H, dim, p.R, scale);
+      return static_cast<int>(cudaGetLastError());
+    }
+  }
+  const int nb = p.B >= 8 ? 8 : (p.B >= 2 ? 2 : 1);
+  const size_t smem = (static_cast<size_t>(nb) * dim + 256 * VEC) * sizeof(float);
+  dim3 grid((p.R + 63) / 64, p.H, (p.B + nb - 1) / nb);
+#define AB_GO(NB)                                                                                                       \
+  {                                                                                                                     \
+    const int rc = set_smem(reinterpret_cast<const void*>(&latent_absorb_kernel<T, VEC, NB>), smem);                    \
+    if (rc) return rc;                                                                                                  \
+    latent_absorb_kernel<T, VEC, NB><<<grid, 256, smem, st>>>(static_cast<const T*>(q), ldq, static_cast<const T*>(w), ldw, qa, \
+                                                              p.B, p.H, dim, p.R, scale);                               \
+  }
+  if (nb == 8) AB_GO(8)
+  else if (nb == 2) AB_GO(2)
+  else AB_GO(1)
+#undef AB_GO
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <typename T, int VEC>
 static int latent_finish(const LatentDecodeParams& p, const void* w_uv, long long ldv, const void* sink, const void* gate,
                          long long ldg, void* out, int vdim, int num_sms, cudaStream_t st) {
+  if constexpr (sizeof(T) == 2 && VEC == 8) {
+    if (p.B > 2 && p.R % 32 == 0 && vdim % 8 == 0) {
+      const size_t smem = 16 * (static_cast<size_t>(p.R + 8) * 2 + p.splits * sizeof(float));
+      const int rc = set_smem(reinterpret_cast<const void*>(&latent_finish_mma_kernel<T>), smem);
+      if (rc) return rc;
+      const int zb = (p.B + 15) / 16, tiles = (vdim / 8 + 7) / 8;   // one 8-column block per warp while the GPU has room
+      const int parts = static_cast<long long>(zb) * p.H * tiles <= 2 * num_sms ? tiles : 1;
+      latent_finish_mma_kernel<T><<<dim3(parts, p.H, zb), 256, smem, st>>>(p, static_cast<const T*>(w_uv), ldv,
+                                                                           static_cast<const T*>(sink), static_cast<const T*>(gate),
+                                                                           ldg, static_cast<T*>(out), vdim);
+      return static_cast<int>(cudaGetLastError());
+    }
+  }
   const int nb = p.B >= 8 ? 8 : (p.B >= 2 ? 2 : 1), zb = (p.B + nb - 1) / nb;
   int parts = 1;                       // value rows of a head over several blocks while the GPU has room
-  while (parts < 16 && static_cast<long long>(zb) * p.H * parts < num_sms && vdim / (2 * parts) >= 8) parts *= 2;
+  while (parts < 16 && static_cast<long long>(zb) * p.H * parts < num_sms && vdim / (2 * parts) >= 16) parts *= 2;
   const int rpb = (vdim + parts - 1) / parts;
-  const size_t smem = static_cast<size_t>(nb) * (p.R + p.splits) * sizeof(float);
+  const size_t smem = static_cast<size_t>(nb) * (p.ldw + p.splits) * sizeof(float);
   dim3 grid(parts, p.H, zb);
 #define FIN_GO(NB)                                                                                                    \
-  latent_finish_kernel<T, VEC, NB><<<grid, 256, smem, st>>>(p.ws, static_cast<const T*>(w_uv), ldv, static_cast<const T*>(sink), \
-                                                            static_cast<const T*>(gate), ldg, static_cast<T*>(out), p.B, p.H, p.R, \
-                                                            vdim, p.splits, rpb)
+  latent_finish_kernel<T, VEC, NB><<<grid, 256, smem, st>>>(p, static_cast<const T*>(w_uv), ldv, static_cast<const T*>(sink), \
+                                                            static_cast<const T*>(gate), ldg, static_cast<T*>(out), vdim, rpb)
   if (nb == 8) FIN_GO(8);
   else if (nb == 2) FIN_GO(2);
   else FIN_GO(1);
@@ -707,14 +919,15 @@ static int latent_finish(const LatentDecodeParams& p, const void* w_uv, long lon
 
 }  // namespace oslo
 
-// slices of the cache per (row, head group): fewest waves of blocks, then the least work per block
-extern "C" int oslo_latent_splits(int B, int H, int T, int R, int num_sms) {
-  const int groups = (H + oslo::LD_HEADS - 1) / oslo::LD_HEADS, kt = R <= 512 ? 64 : 32, tiles = (T + kt - 1) / kt;
+// slices of the cache per (row, head group): fewest waves of blocks (two per SM), then the least work per block
+extern "C" int oslo_latent_splits(int B, int H, int T, int num_sms) {
+  const int per_block = H > oslo::LD_HEADS ? 2 * oslo::LD_HEADS : oslo::LD_HEADS, groups = (H + per_block - 1) / per_block;
+  const int tiles = (T + oslo::LM_KT - 1) / oslo::LM_KT;
   int best = 1;
   double best_cost = 1e30;
-  for (int s = 1; s <= 32 && s <= tiles; ++s) {
-    const long long waves = (static_cast<long long>(B) * groups * s + num_sms - 1) / num_sms;
-    const double cost = static_cast<double>(waves) * ((tiles + s - 1) / s + 1.5) + 0.05 * s;   // set-up and merge of a slice
+  for (int s = 1; s <= 64 && s <= tiles; ++s) {
+    const long long blocks = static_cast<long long>(B) * groups * s, waves = (blocks + 2 * num_sms - 1) / (2 * num_sms);
+    const double cost = static_cast<double>(waves) * ((tiles + s - 1) / s + 2.0) + 0.08 * s;   // set-up and merge of a slice
     if (cost < best_cost) { best_cost = cost; best = s; }
   }
   return best;
@@ -722,25 +935,26 @@ extern "C" int oslo_latent_splits(int B, int H, int T, int R, int num_sms) {
 
 extern "C" int oslo_latent_decode(const void* q, long long ldq, const void* w_uk, long long ldk, const void* w_uv, long long ldv,
                                   const void* cache, const int* lengths, const uint8_t* keep, long long ld_keep, int n_keep,
-                                  const void* sink, const void* gate, long long ldg, float* qa, float* ws, void* out, int B,
-                                  int H, int dim, int vdim, int R, int Tmax, int splits, float scale, int num_sms, int dtype,
-                                  int* err_word, cudaStream_t stream) {
+                                  const void* sink, const void* gate, long long ldg, float* qa, float* ws, float* stat, void* out,
+                                  int B, int H, int dim, int vdim, int R, int Tmax, int splits, float scale, int num_sms,
+                                  int dtype, int* err_word, cudaStream_t stream) {
   using namespace oslo;
   if (B <= 0 || H <= 0) return 0;
   if (R <= 0 || R > 1024 || splits < 1 || splits > 64 || B > 65535 || H > 65535) return -1;
-  LatentDecodeParams p{qa, cache, lengths, keep, ld_keep, n_keep, ws, B, H, R, Tmax, splits, err_word};
+  LatentDecodeParams p{qa, cache, lengths, keep, ld_keep, n_keep, ws, stat, B, H, R, (R + 3) / 4 * 4, Tmax, splits, err_word};
   const size_t te = dtype == OSLO_DT_FP32 ? 4 : 2;
-  const size_t ab_smem = (8 * static_cast<size_t>(dim) + 8 * 8 * 64) * sizeof(float);
+  const int v16 = static_cast<int>(16 / te);
+  const bool kv = R % v16 == 0 && ldk % v16 == 0 && aligned_to(w_uk, 16);
+  const bool vv = R % v16 == 0 && ldv % v16 == 0 && aligned_to(w_uv, 16);
   OSLO_DISPATCH_T(dtype, {
-    int rc = set_smem(reinterpret_cast<const void*>(&latent_absorb_kernel<T>), ab_smem);
+    constexpr int V = 16 / sizeof(T);
+    int rc = kv ? latent_absorb<T, V>(p, q, ldq, w_uk, ldk, qa, dim, scale, stream)
+                : latent_absorb<T, 1>(p, q, ldq, w_uk, ldk, qa, dim, scale, stream);
     if (rc) return rc;
-    latent_absorb_kernel<T><<<dim3((R + 63) / 64, H, (B + 7) / 8), 256, ab_smem, stream>>>(
-        static_cast<const T*>(q), ldq, static_cast<const T*>(w_uk), ldk, qa, B, H, dim, R, scale);
     rc = latent_scan<T>(p, R % 16 == 0 && aligned_to(cache, 16), stream);
     if (rc) return rc;
-    const bool vec = R % 4 == 0 && ldv % 4 == 0 && aligned_to(w_uv, 4 * te);
-    return vec ? latent_finish<T, 4>(p, w_uv, ldv, sink, gate, ldg, out, vdim, num_sms, stream)
-               : latent_finish<T, 1>(p, w_uv, ldv, sink, gate, ldg, out, vdim, num_sms, stream);
+    return vv ? latent_finish<T, V>(p, w_uv, ldv, sink, gate, ldg, out, vdim, num_sms, stream)
+              : latent_finish<T, 1>(p, w_uv, ldv, sink, gate, ldg, out, vdim, num_sms, stream);
   });
   return -2;
 }

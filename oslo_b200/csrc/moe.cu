@@ -7,12 +7,15 @@
 //            Everything stays on the device: no counts are read back, grids are sized for the worst case.
 //   decode:  a few rows: one warp per output element of the chosen experts, straight from the expert's weights.
 // The down projection leaves one row per slot; the residual join adds them up with their weights.
+#include <cooperative_groups.h>
 #include <math_constants.h>
 
 #include <algorithm>
 
 #include "num.cuh"
 #include "oslo_kernels.h"
+
+namespace cg = cooperative_groups;
 
 namespace oslo {
 
@@ -52,24 +55,36 @@ __device__ __forceinline__ void pick_top(float* z, int E, int top, int* idx, flo
   }
 }
 
-// logits from the kernel itself: one block per row
+// logits from the kernel itself: a cluster of RT_CLUSTER blocks per row shares the experts, the first block collects the
+// logits over distributed shared memory and picks
+constexpr int RT_CLUSTER = 8;
 template <typename T, int VEC>
-__global__ void __launch_bounds__(256) route_kernel(const T* __restrict__ h, long long ldh, const T* __restrict__ w,
-                                                    const T* __restrict__ bias, int* __restrict__ idx, float* __restrict__ wgt,
-                                                    int E, int K, int top) {
-  extern __shared__ float rt_smem[];
-  float* x = rt_smem;                  // [K]
-  float* z = x + K;                    // [E]
-  const long long row = blockIdx.x;
-  for (int k = threadIdx.x; k < K; k += blockDim.x) x[k] = Num<T>::to(h[row * ldh + k]);
-  __syncthreads();
+__global__ void __cluster_dims__(RT_CLUSTER, 1, 1) __launch_bounds__(256)
+route_kernel(const T* __restrict__ h, long long ldh, const T* __restrict__ w, const T* __restrict__ bias, int* __restrict__ idx,
+             float* __restrict__ wgt, int E, int K, int top) {
+  extern __shared__ float z[];         // [E], used in the first block
+  cg::cluster_group cluster = cg::this_cluster();
+  const int rank = static_cast<int>(cluster.block_rank());
+  float* z0 = cluster.map_shared_rank(z, 0);
+  const long long row = blockIdx.y;
+  const T* x = h + row * ldh;
   const int lane = threadIdx.x & 31;
-  for (int e = threadIdx.x >> 5; e < E; e += blockDim.x >> 5) {
-    const float d = warp_dot<T, VEC>(w + static_cast<long long>(e) * K, x, K, lane);
-    if (lane == 0) z[e] = d + Num<T>::to(bias[e]);
+  for (int e = rank + RT_CLUSTER * (threadIdx.x >> 5); e < E; e += RT_CLUSTER * (blockDim.x >> 5)) {
+    const T* we = w + static_cast<long long>(e) * K;
+    float acc = 0.f;
+#pragma unroll 8
+    for (int k = lane * VEC; k < K; k += 32 * VEC) {
+      float a[VEC], b[VEC];
+      load_vec<T, VEC>(we + k, a);
+      load_vec<T, VEC>(x + k, b);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) acc = fmaf(a[i], b[i], acc);
+    }
+    acc = warp_sum(acc);
+    if (lane == 0) z0[e] = acc + Num<T>::to(bias[e]);
   }
-  __syncthreads();
-  if (threadIdx.x < 32) pick_top(z, E, top, idx + row * top, wgt + row * top, lane);
+  cluster.sync();                      // also keeps the first block's shared memory alive until all have written
+  if (rank == 0 && threadIdx.x < 32) pick_top(z, E, top, idx + row * top, wgt + row * top, lane);
 }
 
 // logits [rows, E] (32-bit, without the bias) from a GEMM: one warp per row
@@ -184,39 +199,47 @@ __global__ void __launch_bounds__(256) moe_grouped_kernel(const T* __restrict__ 
     }
 }
 
-// few rows: out[pair, n] = act(w[idx[pair]][n, :] . x[row of pair, :]); a warp computes 4 outputs
+// few rows: out[pair, n] = act(w[idx[pair]][n, :] . x[row of pair, :]); groups of `wg` warps share the k range of 4 outputs
+// and walk over the output groups, so that the chosen expert is looked up once per block
 template <typename T, int VEC>
-__global__ void __launch_bounds__(256) moe_few_kernel(const T* __restrict__ x, long long ldx, const int* __restrict__ idx,
-                                                      const T* __restrict__ w, T* __restrict__ out, int N, int K, int per_row,
-                                                      int relu2) {
-  extern __shared__ float mf_smem[];
-  const int pair = blockIdx.y;
+__global__ void __launch_bounds__(256, 4) moe_few_kernel(const T* __restrict__ x, long long ldx, const int* __restrict__ idx,
+                                                         const T* __restrict__ w, T* __restrict__ out, int N, int K,
+                                                         int per_row, int relu2, int wg) {
+  __shared__ float red[2][8][4];
+  const int pair = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const T* src = x + static_cast<long long>(pair / per_row) * ldx;
-  for (int k = threadIdx.x; k < K; k += blockDim.x) mf_smem[k] = Num<T>::to(src[k]);
-  __syncthreads();
   const T* we = w + static_cast<long long>(idx[pair]) * N * K;
-  const int lane = threadIdx.x & 31;
-  const int n0 = (blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5)) * 4;
-  float acc[4] = {0.f, 0.f, 0.f, 0.f};
-  const int nn = min(4, N - n0);
-  for (int k = lane * VEC; k < K; k += 32 * VEC) {
-    float v[4][VEC];
+  const int group = warp / wg, gw = warp % wg, per_block = 8 / wg * 4;
+  for (int nb = blockIdx.x * per_block, it = 0; nb < N; nb += gridDim.x * per_block, ++it) {
+    const int n0 = nb + group * 4, nn = min(4, N - n0);      // nn may be <= 0 for the last groups
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    for (int k = (gw * 32 + lane) * VEC; k < K; k += wg * 32 * VEC) {
+      Pack<T, VEC> v[4];
 #pragma unroll
-    for (int j = 0; j < 4; ++j)
-      if (j < nn) load_vec<T, VEC>(we + static_cast<long long>(n0 + j) * K + k, v[j]);
+      for (int j = 0; j < 4; ++j)
+        if (j < nn) v[j] = *reinterpret_cast<const Pack<T, VEC>*>(we + static_cast<long long>(n0 + j) * K + k);
+      float xv[VEC];
+      load_vec<T, VEC>(src + k, xv);
 #pragma unroll
-    for (int j = 0; j < 4; ++j)
-      if (j < nn) {
+      for (int j = 0; j < 4; ++j)
+        if (j < nn) {
 #pragma unroll
-        for (int i = 0; i < VEC; ++i) acc[j] = fmaf(v[j][i], mf_smem[k + i], acc[j]);
-      }
-  }
+          for (int i = 0; i < VEC; ++i) acc[j] = fmaf(Num<T>::to(v[j].e[i]), xv[i], acc[j]);
+        }
+    }
 #pragma unroll
-  for (int j = 0; j < 4; ++j) {
-    if (j < nn) {                      // uniform over the warp
-      float v = warp_sum(acc[j]);
-      if (relu2) { v = fmaxf(v, 0.f); v *= v; }
-      if (lane == 0) out[static_cast<long long>(pair) * N + n0 + j] = Num<T>::from(v);
+    for (int j = 0; j < 4; ++j) acc[j] = warp_sum(acc[j]);
+    float(*r)[4] = red[it & 1];
+    if (lane == 0) {
+#pragma unroll
+      for (int j = 0; j < 4; ++j) r[warp][j] = acc[j];
+    }
+    __syncthreads();                   // the other half of `red` is free again: it was read before this barrier
+    if (gw == 0 && lane < nn) {
+      float s = 0.f;
+      for (int g = 0; g < wg; ++g) s += r[warp + g][lane];
+      if (relu2) { s = fmaxf(s, 0.f); s *= s; }
+      out[static_cast<long long>(pair) * N + n0 + lane] = Num<T>::from(s);
     }
   }
 }
@@ -236,21 +259,19 @@ extern "C" int oslo_moe_route(const void* h, long long ldh, const void* w, const
     });
     return static_cast<int>(cudaGetLastError());
   }
-  const size_t smem = (static_cast<size_t>(K) + E) * sizeof(float);
-  if (smem > 227 * 1024) return -3;
-  const bool vec = K % 4 == 0 && aligned_to(w, 4 * te);
-#define ROUTE_GO(V)                                                                                                   \
-  {                                                                                                                   \
-    if (smem > 48 * 1024) {                                                                                           \
-      cudaError_t e = cudaFuncSetAttribute(route_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize,           \
-                                           static_cast<int>(smem));                                                   \
-      if (e != cudaSuccess) return static_cast<int>(e);                                                               \
-    }                                                                                                                 \
-    route_kernel<T, V><<<static_cast<unsigned>(rows), 256, smem, stream>>>(                                           \
-        static_cast<const T*>(h), ldh, static_cast<const T*>(w), static_cast<const T*>(bias), idx, wgt, E, K, top);   \
-  }
-  OSLO_DISPATCH_T(dtype, { if (vec) ROUTE_GO(4) else ROUTE_GO(1) });
-#undef ROUTE_GO
+  if (rows > 65535) return -1;         // larger batches bring their logits
+  const int v = static_cast<int>(16 / te);
+  const bool vec = K % v == 0 && ldh % v == 0 && aligned_to(w, 16) && aligned_to(h, 16);
+  const dim3 grid(RT_CLUSTER, static_cast<unsigned>(rows));
+  OSLO_DISPATCH_T(dtype, {
+    constexpr int V = 16 / sizeof(T);
+    if (vec)
+      route_kernel<T, V><<<grid, 256, E * sizeof(float), stream>>>(static_cast<const T*>(h), ldh, static_cast<const T*>(w),
+                                                                   static_cast<const T*>(bias), idx, wgt, E, K, top);
+    else
+      route_kernel<T, 1><<<grid, 256, E * sizeof(float), stream>>>(static_cast<const T*>(h), ldh, static_cast<const T*>(w),
+                                                                   static_cast<const T*>(bias), idx, wgt, E, K, top);
+  });
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -294,24 +315,21 @@ extern "C" int oslo_moe_few(const void* x, long long ldx, const int* idx, const 
   if (pairs <= 0 || N <= 0) return 0;
   if (pairs > 65535 || per_row < 1) return -1;
   const size_t te = dtype == OSLO_DT_FP32 ? 4 : 2;
-  const size_t smem = static_cast<size_t>(K) * sizeof(float);
-  if (smem > 227 * 1024) return -3;
   const int v = static_cast<int>(16 / te);
-  const bool vec = K % v == 0 && aligned_to(w, 16);
-#define FEW_GO(V)                                                                                                       \
-  {                                                                                                                     \
-    if (smem > 48 * 1024) {                                                                                             \
-      cudaError_t e = cudaFuncSetAttribute(moe_few_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize,           \
-                                           static_cast<int>(smem));                                                     \
-      if (e != cudaSuccess) return static_cast<int>(e);                                                                 \
-    }                                                                                                                   \
-    moe_few_kernel<T, V><<<dim3((N + 31) / 32, pairs), 256, smem, stream>>>(                                            \
-        static_cast<const T*>(x), ldx, idx, static_cast<const T*>(w), static_cast<T*>(out), N, K, per_row, relu2);      \
-  }
+  const bool vec = K % v == 0 && ldx % v == 0 && aligned_to(w, 16) && aligned_to(x, 16);
+  int wg = 8;                          // warps on one output group: at least one full stride each
+  while (wg > 1 && K < wg * 32 * (vec ? v : 1)) wg /= 2;
+  const int per_block = 8 / wg * 4;
+  const int want = (148 * 4 + pairs - 1) / pairs;
+  const dim3 grid(std::min((N + per_block - 1) / per_block, want), pairs);
   OSLO_DISPATCH_T(dtype, {
     constexpr int V = 16 / sizeof(T);
-    if (vec) FEW_GO(V) else FEW_GO(1)
+    if (vec)
+      moe_few_kernel<T, V><<<grid, 256, 0, stream>>>(static_cast<const T*>(x), ldx, idx, static_cast<const T*>(w),
+                                                     static_cast<T*>(out), N, K, per_row, relu2, wg);
+    else
+      moe_few_kernel<T, 1><<<grid, 256, 0, stream>>>(static_cast<const T*>(x), ldx, idx, static_cast<const T*>(w),
+                                                     static_cast<T*>(out), N, K, per_row, relu2, wg);
   });
-#undef FEW_GO
   return static_cast<int>(cudaGetLastError());
 }

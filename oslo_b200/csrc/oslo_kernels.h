@@ -240,13 +240,14 @@ int oslo_sink_attention(const void* q, long long q_sb, long long q_ss, long long
 int oslo_latent_prep(const void* cq, long long ldq, const void* wq, int q_rank, void* cq_out, const void* ckv, long long ldkv,
                      const void* wkv, int kv_rank, void* cache, const int* lengths, int Tmax, float eps, int B, int dtype,
                      int* err_word, cudaStream_t stream);
-// one query per row over a latent cache; qa fp32 [B, H, R] and ws fp32 [B, H, splits, R + 2] are workspaces
+// one query per row over a latent cache; fp32 workspaces qa [B, H, R], ws [B, H, splits, R rounded up to
+// a multiple of 4] and stat [B, H, splits, 2]
 int oslo_latent_decode(const void* q, long long ldq, const void* w_uk, long long ldk, const void* w_uv, long long ldv,
                        const void* cache, const int* lengths, const uint8_t* keep, long long ld_keep, int n_keep,
-                       const void* sink, const void* gate, long long ldg, float* qa, float* ws, void* out, int B, int H,
-                       int dim, int vdim, int R, int Tmax, int splits, float scale, int num_sms, int dtype, int* err_word,
-                       cudaStream_t stream);
-int oslo_latent_splits(int B, int H, int T, int R, int num_sms);
+                       const void* sink, const void* gate, long long ldg, float* qa, float* ws, float* stat, void* out,
+                       int B, int H, int dim, int vdim, int R, int Tmax, int splits, float scale, int num_sms, int dtype,
+                       int* err_word, cudaStream_t stream);
+int oslo_latent_splits(int B, int H, int T, int num_sms);
 
 // mixture of experts (moe.cu, grouped GEMM in gemm_sm100.cu)
 int oslo_moe_route(const void* h, long long ldh, const void* w, const void* bias, const float* logits, int* idx, float* wgt,

@@ -694,18 +694,20 @@ def latent_decode(q: Tensor, w_uk: Tensor, w_uv: Tensor, cache: Tensor, lengths:
                                 float(scale), heads)
 
 
-MOE_FEW_ROWS = 16   # token rows up to which the chosen experts' weights are streamed per (token, choice)
+MOE_FEW_PAIRS = 8   # (token, choice) pairs up to which the chosen experts' weights are streamed per pair
 
 
 def moe_route(h: Tensor, w: Tensor, bias: Tensor, top: int):
     logits = None
     if h.size(0) > SMALL_M_ROWS and gemm_ok(h, w) and h.size(1) % 8 == 0:
         logits = gemm(h, w, flags=FLAG_OUT_FP32)           # 16-bit operands, exact products, fp32 sums and output
+    elif h.size(0) > 65535:                                # no tensor-core path for these sizes or types: 32-bit library product
+        logits = torch.matmul(h.float(), w.float().t())
     return _ext().moe_route(_rows(h), w, bias, logits, top)
 
 
 def moe_experts(h: Tensor, idx: Tensor, up: Tensor, down: Tensor):
-    if h.size(0) <= MOE_FEW_ROWS:
+    if idx.numel() <= MOE_FEW_PAIRS:
         a = _ext().moe_few(_rows(h), idx, up, idx.size(1), True)
         return _ext().moe_few(a, idx, down, 1, False), None
     slots, rows, tile_group, n_tiles = _ext().moe_plan(_rows(h), idx, up.size(0))

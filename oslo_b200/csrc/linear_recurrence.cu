@@ -4,12 +4,12 @@
 //   o_t[j] = sum_i silu(q_t)[i] S_t[i, j]
 // `k` is computed from the negated logit, so a gate close to 1 does not lose what it writes to cancellation.
 //
-// Prefill (recurrence_kernel): a thread keeps a 16 x 8 tile of S in registers - rows in pairs, so that every update is
-// a packed two-float FMA - and G lanes share a column group; per token it reads 16 + 16 + 8 floats from shared
-// memory, does 192 packed FMAs and reduces 8 partial outputs over the G lanes. The prompt is cut into chunks when
-// (batch x heads) alone does not fill the GPU: local states of all chunks from zero (no outputs), one elementwise scan
-// over the chunks, then every chunk again from its true initial state. Only products of forget gates (<= 1) ever
-// appear, so no chunk length can overflow.
+// Prefill (recurrence_kernel): a thread keeps a 16 x 4 tile of S in registers - rows in pairs, so that every update is a
+// packed two-float FMA - and G lanes share a column group; per token it reads 16 + 16 + 4 floats from shared memory,
+// does 96 packed FMAs and reduces 4 partial outputs over the G lanes. The prompt is
+// cut into chunks when (batch x heads) alone does not fill the GPU: local states of all chunks but the last from zero
+// (no outputs), one elementwise scan over the chunks, then every chunk again from its true initial state. Only
+// products of forget gates (<= 1) ever appear, so no chunk length can overflow.
 // Decode (recurrence_step_kernel): a cluster of CTAs per (row, head), each on a slice of the value channels; the RMS
 // norm over the head's outputs is finished over distributed shared memory, so a step is one launch.
 // Tokens whose `keep` entry is 0 (padding) leave the state as it is and produce zeros.
@@ -39,7 +39,14 @@ __device__ __forceinline__ f32x2 fma_f2(f32x2 a, f32x2 b, f32x2 c) {
   return r;
 }
 
-__device__ __forceinline__ float write_gate(float logit, float lower) { return (1.0f - lower) * sigmoid_f(-logit); }
+// 32-bit models get the accurate exponential; logits that come from 16-bit projections the hardware one (2^-21)
+template <typename T> __device__ __forceinline__ float sigmoid_t(float z) {
+  return sizeof(T) == 4 ? sigmoid_f(z) : __fdividef(1.0f, 1.0f + __expf(-z));
+}
+template <typename T> __device__ __forceinline__ float write_gate(float logit, float lower) {
+  return (1.0f - lower) * sigmoid_t<T>(-logit);
+}
+template <typename T> __device__ __forceinline__ float silu_t(float z) { return z * sigmoid_t<T>(z); }
 
 struct RecParams {
   const void *q, *f, *v;             // row (b * S + t) of each has the stride ldq / ldf / ldv
@@ -51,20 +58,23 @@ struct RecParams {
   float* decay;                      // STATE_ONLY: product of the forget gates of the chunk
   float* out;                        // [B, S, H, vdim]
   int B, S, H, dim, vdim;
-  int chunk, nchunks;                // tokens per chunk
+  int chunk, nchunks;                // tokens per chunk; chunks of this launch per batch row
+  float* s_end;                      // last chunk only: final states [B, H, dim, vdim], or nullptr
   long long s_batch, s_chunk;        // element strides of s_in / s_out over batch rows and chunks
   int dim_pad;                       // dim rounded up so that every row of a raw stage starts at a 16-byte boundary
   int vec16;                         // q, f, v rows and head slices start at 16-byte boundaries
 };
 
 constexpr int REC_TB = 16;    // tokens staged at a time
-constexpr int REC_COLS = 8;   // state columns per thread
-constexpr int REC_ROWS = 16;  // state rows per thread
+constexpr int REC_COLS = 4;   // state columns per thread
+constexpr int REC_ROWS = 16;      // state rows per thread
 
-// STATE_ONLY: no outputs, start from zero, also the chunk's total decay per row
+// G lanes per column group. STATE_ONLY: no outputs, start from zero, also the chunk's total decay per row
 template <typename T, int G, bool STATE_ONLY>
-__global__ void __launch_bounds__(128) recurrence_kernel(const RecParams p) {
+__global__ void __launch_bounds__(256, 2) recurrence_kernel(const RecParams p) {
   constexpr int DP = REC_ROWS * G;
+  constexpr int CONV = DP >= 256 ? 1 : 256 / DP;
+  constexpr int WIDTH = G >= REC_COLS ? 1 : REC_COLS / G;    // output columns a lane holds after the reduction
   extern __shared__ float4 rec_smem[];
   const int nt = blockDim.x;
   const int cols = nt / G * REC_COLS;
@@ -103,6 +113,15 @@ __global__ void __launch_bounds__(128) recurrence_kernel(const RecParams p) {
 #pragma unroll
   for (int i = 0; i < REC_ROWS; ++i) dec[i] = 1.f;
   const f32x2 minus1 = pack_f2(-1.f, -1.f);
+  // where this lane's share of an output row goes, and how many of its WIDTH columns exist (0: another lane writes them)
+  int first = 0;
+#pragma unroll
+  for (int off = G / 2, w = REC_COLS; off > 0 && w > 1; off >>= 1, w /= 2)
+    if (g & off) first += w / 2;
+  const int out_cols = (G <= REC_COLS || g % (G / REC_COLS > 0 ? G / REC_COLS : 1) == 0) ? min(WIDTH, p.vdim - my_col - first) : 0;
+  const long long out_step = static_cast<long long>(p.H) * p.vdim;
+  float* out = STATE_ONLY ? nullptr
+                          : p.out + ((static_cast<long long>(b) * p.S + t_begin) * p.H + h) * p.vdim + my_col + first;
 
   // raw [REC_TB][raw_ld] stages in the storage type, fetched one step ahead: q (unless STATE_ONLY), f, v slice
   const int f_at = STATE_ONLY ? 0 : p.dim_pad, v_at = f_at + p.dim_pad, raw_ld = v_at + cols;
@@ -152,29 +171,27 @@ __global__ void __launch_bounds__(128) recurrence_kernel(const RecParams p) {
     }
     __syncthreads();
     const T* src = raw + static_cast<size_t>(it & 1) * REC_TB * raw_ld;
-    for (int i = tid; i < DP; i += nt) {
+    for (int e = tid; e < DP * CONV; e += nt) {          // CONV threads share a channel's tokens
+      const int i = e % DP;
       const bool real = i < p.dim;
       const float bias = real ? Num<T>::to(fb[i]) : 0.f, low = real ? Num<T>::to(lw[i]) : 1.f;
 #pragma unroll 4
-      for (int t = 0; t < n; ++t) {
+      for (int t = e / DP; t < n; t += CONV) {
         const bool on = real && (p.keep == nullptr || p.keep[b * p.ld_keep + t0 + t]);
-        ks[t * DP + i] = on ? write_gate(Num<T>::to(src[t * raw_ld + f_at + i]) + bias, low) : 0.f;
-        if (!STATE_ONLY) qs[t * DP + i] = on ? silu_f(Num<T>::to(src[t * raw_ld + i])) : 0.f;
+        ks[t * DP + i] = on ? write_gate<T>(Num<T>::to(src[t * raw_ld + f_at + i]) + bias, low) : 0.f;
+        if (!STATE_ONLY) qs[t * DP + i] = on ? silu_t<T>(Num<T>::to(src[t * raw_ld + i])) : 0.f;
       }
     }
-    for (int c = tid; c < cols; c += nt) {
-      const bool real = col0 + c < p.vdim;
-#pragma unroll 4
-      for (int t = 0; t < n; ++t) vs[t * cols + c] = real ? Num<T>::to(src[t * raw_ld + v_at + c]) : 0.f;
+    for (int e = tid; e < n * cols; e += nt) {
+      const int t = e / cols, c = e - t * cols;
+      vs[e] = col0 + c < p.vdim ? Num<T>::to(src[t * raw_ld + v_at + c]) : 0.f;
     }
     __syncthreads();
     for (int t = 0; t < n; ++t) {
       f32x2 v2[REC_COLS];
       {
         const float4 a = *reinterpret_cast<const float4*>(vs + t * cols + cgp * REC_COLS);
-        const float4 c = *reinterpret_cast<const float4*>(vs + t * cols + cgp * REC_COLS + 4);
         v2[0] = pack_f2(a.x, a.x); v2[1] = pack_f2(a.y, a.y); v2[2] = pack_f2(a.z, a.z); v2[3] = pack_f2(a.w, a.w);
-        v2[4] = pack_f2(c.x, c.x); v2[5] = pack_f2(c.y, c.y); v2[6] = pack_f2(c.z, c.z); v2[7] = pack_f2(c.w, c.w);
       }
       f32x2 o2[REC_COLS];
 #pragma unroll
@@ -212,7 +229,6 @@ __global__ void __launch_bounds__(128) recurrence_kernel(const RecParams p) {
           o[c] = lo + hi;
         }
         // reduce over the G lanes; each halving step also halves the columns a lane is responsible for
-        int first = 0;   // first column this lane still holds
         int width = REC_COLS;
 #pragma unroll
         for (int off = G / 2; off > 0; off >>= 1) {
@@ -227,24 +243,19 @@ __global__ void __launch_bounds__(128) recurrence_kernel(const RecParams p) {
                 o[c] = mine + __shfl_xor_sync(0xffffffffu, give, off);
               }
             }
-            if (upper) first += half;
             width = half;
           } else {
             o[0] += __shfl_xor_sync(0xffffffffu, o[0], off);
           }
         }
-        float* orow = p.out + ((static_cast<long long>(b) * p.S + t0 + t) * p.H + h) * p.vdim;
-        const bool writes = G <= REC_COLS || (g % (G / REC_COLS > 0 ? G / REC_COLS : 1)) == 0;
-        if (writes) {
 #pragma unroll
-          for (int c = 0; c < REC_COLS; ++c)
-            if (c < width && my_col + first + c < p.vdim) orow[my_col + first + c] = o[c];
-        }
+        for (int c = 0; c < WIDTH; ++c)
+          if (c < out_cols) out[c] = o[c];
+        out += out_step;
       }
     }
   }
-  if (p.s_out) {
-    float* so = p.s_out + b * p.s_batch + ch * p.s_chunk + static_cast<long long>(h) * p.dim * p.vdim;
+  auto store_state = [&](float* so) {
 #pragma unroll
     for (int rp = 0; rp < REC_ROWS / 2; ++rp) {
       const int i = 4 * (g + G * (rp / 2)) + 2 * (rp % 2);
@@ -258,6 +269,12 @@ __global__ void __launch_bounds__(128) recurrence_kernel(const RecParams p) {
         }
       }
     }
+  };
+  if (p.s_end && ch == p.nchunks - 1) {
+    store_state(p.s_end + (static_cast<long long>(b) * p.H + h) * p.dim * p.vdim);
+  }
+  if (p.s_out) {
+    store_state(p.s_out + b * p.s_batch + ch * p.s_chunk + static_cast<long long>(h) * p.dim * p.vdim);
   }
   if (STATE_ONLY && cgp == 0 && blockIdx.x == 0) {
     float* d = p.decay + ((static_cast<long long>(b) * p.nchunks + ch) * p.H + h) * p.dim;
@@ -271,24 +288,25 @@ __global__ void __launch_bounds__(128) recurrence_kernel(const RecParams p) {
   }
 }
 
-// ws[b, c] holds the local final state of chunk c; replace it by the state at the chunk's start; state <- final state
+// ws[b, c] (c < nchunks - 1) holds the local final state of chunk c; replace every ws[b, c] by the state at the chunk's start
 __global__ void __launch_bounds__(256) recurrence_chunk_scan_kernel(float* __restrict__ ws, const float* __restrict__ decay,
-                                                                    const float* __restrict__ s_in, float* __restrict__ s_out,
-                                                                    int nchunks, int H, int dim, int vdim) {
+                                                                    const float* __restrict__ s_in, int nchunks, int H, int dim,
+                                                                    int vdim) {
   const long long per = static_cast<long long>(H) * dim * vdim;
   const long long e = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x;
   const int b = blockIdx.y;
   if (e >= per) return;
   const long long hi = e / vdim;   // head * dim + row
   float s = s_in ? s_in[b * per + e] : 0.f;
+#pragma unroll 4
   for (int c = 0; c < nchunks; ++c) {
     const long long o = (static_cast<long long>(b) * nchunks + c) * per + e;
-    const float local = ws[o];
-    const float d = decay[(static_cast<long long>(b) * nchunks + c) * H * dim + hi];
+    const bool more = c + 1 < nchunks;
+    const float local = more ? ws[o] : 0.f;
+    const float d = more ? decay[(static_cast<long long>(b) * (nchunks - 1) + c) * H * dim + hi] : 0.f;
     ws[o] = s;
     s = fmaf(d, s, local);
   }
-  if (s_out) s_out[b * per + e] = s;
 }
 
 struct StepParams {
@@ -319,9 +337,9 @@ __global__ void __launch_bounds__(256) recurrence_step_kernel(const StepParams p
   const T* v = static_cast<const T*>(p.v) + b * p.ldv + static_cast<long long>(h) * p.vdim;
   const bool on = p.keep == nullptr || p.keep[b * p.ld_keep];
   for (int i = threadIdx.x; i < p.dim; i += blockDim.x) {
-    ks[i] = on ? write_gate(Num<T>::to(f[i]) + Num<T>::to(static_cast<const T*>(p.f_bias)[h * p.dim + i]),
+    ks[i] = on ? write_gate<T>(Num<T>::to(f[i]) + Num<T>::to(static_cast<const T*>(p.f_bias)[h * p.dim + i]),
                             Num<T>::to(static_cast<const T*>(p.lower)[h * p.dim + i])) : 0.f;
-    qs[i] = on ? silu_f(Num<T>::to(q[i])) : 0.f;
+    qs[i] = on ? silu_t<T>(Num<T>::to(q[i])) : 0.f;
   }
   __syncthreads();
   const int tx_n = p.cols / VEC;                       // the launcher keeps tx_n <= 256
@@ -370,11 +388,15 @@ __global__ void __launch_bounds__(256) recurrence_step_kernel(const StepParams p
   for (int c = threadIdx.x; c < cols; c += blockDim.x) out[c] = Num<T>::from(part[c] * rn * Num<T>::to(nw[c]));
 }
 
+// threads of a block: the column groups of a head, at most 256
+static int rec_threads(int g, int vdim) {
+  const int groups = (vdim + REC_COLS - 1) / REC_COLS;
+  return std::min(256, (groups * g + 31) / 32 * 32);
+}
+
 template <typename T, int G, bool STATE_ONLY>
 static int rec_launch(const RecParams& p, cudaStream_t st) {
-  const int groups = (p.vdim + REC_COLS - 1) / REC_COLS;
-  int nt = std::min(128, (groups * G + 31) / 32 * 32);
-  const int cols = nt / G * REC_COLS;
+  const int nt = rec_threads(G, p.vdim), cols = nt / G * REC_COLS;
   const size_t smem = static_cast<size_t>(REC_TB) * (((STATE_ONLY ? 1 : 2) * REC_ROWS * G + cols) * sizeof(float) +
                                                      2 * ((STATE_ONLY ? 1 : 2) * p.dim_pad + cols) * sizeof(T));
   if (smem > 48 * 1024) {
@@ -403,16 +425,22 @@ static int rec_dispatch(const RecParams& p, cudaStream_t st) {
 extern "C" int oslo_recurrence_chunks(int B, int S, int H, int dim, int vdim, int num_sms) {
   using namespace oslo;
   int g = 1;
-  while (16 * g < dim) g *= 2;
-  const int groups = (vdim + REC_COLS - 1) / REC_COLS;
-  const int nt = std::min(128, (groups * g + 31) / 32 * 32);
-  const int cols = nt / g * REC_COLS;
+  while (REC_ROWS * g < dim && g < 32) g *= 2;
+  const int nt = rec_threads(g, vdim), cols = nt / g * REC_COLS;
   const long long ctas = static_cast<long long>(B) * H * ((vdim + cols - 1) / cols);
-  const int resident = 256 / nt * num_sms;             // CTAs of nt threads that keep an SM's register file busy
-  if (ctas * 2 > resident || S < 128) return 1;
-  int n = static_cast<int>(resident / ctas);
-  n = std::min(n, S / 64);
-  return std::max(1, n);
+  if (S < 128) return 1;
+  // an SM's blocks share its FMA pipes: time ~ (blocks of the fullest SM) x (tokens per chunk); more than one chunk adds the
+  // local states (two thirds of the work, all chunks but the last) and the scan
+  int best = 1;
+  double best_cost = 1e30;
+  for (int n = 1; n <= S / 64 && n <= 64; ++n) {
+    const double per = static_cast<double>(S) / n;
+    const auto fullest = [&](long long blocks) { return static_cast<double>((blocks + num_sms - 1) / num_sms); };
+    // fewer than two blocks on an SM leave its pipes partly idle
+    const double c3 = std::max(1.4, fullest(ctas * n)) * per, c1 = n > 1 ? std::max(1.4, fullest(ctas * (n - 1))) * per * 0.67 + 16.0 + n : 0.0;
+    if (c3 + c1 < best_cost) { best_cost = c3 + c1; best = n; }
+  }
+  return best;
 }
 
 extern "C" int oslo_recurrence(const void* q, long long ldq, const void* f, long long ldf, const void* v, long long ldv,
@@ -442,13 +470,15 @@ extern "C" int oslo_recurrence(const void* q, long long ldq, const void* f, long
   p.chunk = ((S + nchunks - 1) / nchunks + REC_TB - 1) / REC_TB * REC_TB;
   p.s_batch = per * nchunks; p.s_chunk = per;
   p.s_in = nullptr; p.s_out = ws; p.decay = decay;
+  p.nchunks = nchunks - 1;             // nobody starts from the last chunk's state
   OSLO_DISPATCH_T(dtype, { rc = rec_dispatch<T, true>(p, stream); });
   if (rc) return rc;
-  recurrence_chunk_scan_kernel<<<dim3(static_cast<unsigned>((per + 255) / 256), B), 256, 0, stream>>>(ws, decay, state, state,
-                                                                                                     nchunks, H, dim, vdim);
+  recurrence_chunk_scan_kernel<<<dim3(static_cast<unsigned>((per + 255) / 256), B), 256, 0, stream>>>(ws, decay, state, nchunks, H,
+                                                                                                     dim, vdim);
   rc = static_cast<int>(cudaGetLastError());
   if (rc) return rc;
-  p.s_in = ws; p.s_out = nullptr;
+  p.nchunks = nchunks;
+  p.s_in = ws; p.s_out = nullptr; p.s_end = state;
   OSLO_DISPATCH_T(dtype, { rc = rec_dispatch<T, false>(p, stream); });
   return rc;
 }

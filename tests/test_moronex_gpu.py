@@ -5,7 +5,12 @@ import torch
 
 import oslo_b200 as ob
 from oslo_b200 import ops
+from oslo_b200.generation import BatchSteps, GraphedGreedyDecoder
+from oslo_b200.models.common import StaticKVCache
 from oslo_b200.ops import reference as ref
+
+from . import plain_moronex as plain
+from .moronex_cases import CASES, case, dense, far_key_weights, hgrn2, latent, make_tensors, moe, write_model
 
 pytestmark = pytest.mark.gpu
 DTYPES = [torch.float32, torch.bfloat16, torch.float16]
@@ -183,3 +188,183 @@ def test_moe_when_one_expert_takes_everything():
         idx = torch.full((600, 1), 4, dtype=torch.int32, device="cuda")
         y, slots = ops.moe_experts(h, idx, up, down)
         close(y[slots.reshape(-1).long()], ref.moe_experts(h, idx, up, down), dtype)
+
+
+# ---------------------------------------------------------------------------------------------------- the whole model
+MODEL_TOL = {torch.float32: 5e-5, torch.bfloat16: 0.08}
+WIDE = {
+    # chunked recurrences, several key tiles, the grouped expert product, cluster sizes above 1
+    "wide": case(200, 256, 1e-5, hgrn2(4, 128, 64, moe(128, 6, 2)), latent(6, 64, 64, 128, 128, 0.125, moe(96, 4, 3)),
+                 latent(18, 32, 48, 96, 128, 0.2, dense(320), kv_from=1), hgrn2(2, 24, 136, None)),
+}
+ALL = {**CASES, **WIDE}
+
+
+def load(tmp_path, cfg, tensors=None, dtype=torch.float32):
+    tensors = make_tensors(cfg) if tensors is None else tensors
+    write_model(str(tmp_path), cfg, tensors)
+    model = ob.load_causal_lm(str(tmp_path), torch_dtype=dtype).cuda().fuse().eval()
+    return model, tensors
+
+
+def ids(n, vocab, seed=1):
+    return torch.randint(0, vocab, (n,), generator=torch.Generator().manual_seed(seed)).tolist()
+
+
+class Want:
+    """The plain model's logits of a sequence, and the positions that 16-bit rounding does not blow up (a router's close call, a
+    post-norm of next to nothing): those where weights off by a fraction of a 16-bit step change little."""
+
+    def __init__(self, cfg, tensors, seq):
+        self.logits = plain.forward(cfg, tensors, seq)
+        g = torch.Generator().manual_seed(77)
+        self.clear = torch.ones(len(seq), dtype=torch.bool)
+        for _ in range(2):
+            off = {k: t.double() * (1 + 2.0 ** -9 * torch.randn(t.shape, generator=g)) for k, t in tensors.items()}
+            d = (plain.forward(cfg, off, seq) - self.logits).pow(2).mean(-1).sqrt() / self.logits.pow(2).mean().sqrt()
+            self.clear &= d < 0.03
+        assert self.clear.double().mean() > 0.5
+
+
+def errors(got, want, dtype, at=slice(None)):
+    """Per position: root mean square over the vocabulary, relative to the logits' own."""
+    ref_rows, clear = want.logits[at], want.clear[at]
+    got = got.double().cpu()
+    assert torch.isfinite(got).all() and got.shape == ref_rows.shape
+    d = (got - ref_rows).pow(2).mean(-1).sqrt() / want.logits.pow(2).mean().sqrt()
+    return d if dtype == torch.float32 else d[clear]
+
+
+def small(d, dtype, factor=1.0):
+    """In 32-bit every position counts; in 16-bit one position in thirty may be one that rounding blows up all the same."""
+    over = int((d > factor * MODEL_TOL[dtype]).sum())
+    assert over <= (0 if dtype == torch.float32 else -(-d.numel() // 30)), (over, d.numel(), float(d.max()))
+
+
+def same(got, want, dtype, at=slice(None), factor=1.0):
+    small(errors(got, want, dtype, at), dtype, factor)
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("name", sorted(ALL))
+def test_model_prompts_decoding_and_portions(tmp_path, dtype, name):
+    cfg = ALL[name]
+    model, tensors = load(tmp_path, cfg, dtype=dtype)
+    n = 150 if name == "wide" else 70
+    seq = ids(n, cfg["vocab"])
+    want = Want(cfg, tensors, seq)
+    x = torch.tensor([seq], device="cuda")
+    before = ops.load_ext(required=True).launch_count()
+    with torch.no_grad():
+        same(model(input_ids=x).logits[0], want, dtype)
+        assert ops.load_ext().launch_count() > before
+        for portions in ([n - 12] + [1] * 12, [1] * 20, [2] * 6 + [n - 13, 1], [n // 2, 2, n - n // 2 - 2]):
+            cache, at = StaticKVCache(16, grow=True), 0
+            for m in portions:
+                out = model(input_ids=x[:, at:at + m], past_key_values=cache, use_cache=True).logits[0]
+                same(out, want, dtype, slice(at, at + m))
+                at += m
+    assert int(ops.load_ext().error_word(x).item()) == 0
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("name", ["mixed", "odd", "wide"])
+def test_model_batches_of_unequal_requests(tmp_path, dtype, name):
+    cfg = ALL[name]
+    model, tensors = load(tmp_path, cfg, dtype=dtype)
+    lens, tails = (40, 1, 23, 70), (6, 9, 3, 2)
+    seqs = [ids(a + b, cfg["vocab"], seed=a) for a, b in zip(lens, tails)]
+    want = [Want(cfg, tensors, s) for s in seqs]
+    steps = BatchSteps(model, reserve=1)
+    out = steps.start([s[:a] for s, a in zip(seqs, lens)])
+    for r in range(4):
+        same(out[r, steps.pad[r]:], want[r], dtype, slice(0, lens[r]))
+    live, at, d = [0, 1, 2, 3], list(lens), []
+    while True:
+        rows = [i for i, r in enumerate(live) if at[r] < len(seqs[r])]
+        if not rows:
+            break
+        steps.keep(rows)
+        live = [live[i] for i in rows]
+        out = steps.advance([seqs[r][at[r]] for r in live])
+        for i, r in enumerate(live):
+            d.append(errors(out[i, 0][None], want[r], dtype, slice(at[r], at[r] + 1)))
+            at[r] += 1
+    small(torch.cat(d), dtype, 1.5)
+
+
+def test_model_many_rows_decode_like_few(tmp_path):
+    """The decode kernels for batches (tensor-core projections, grouped experts) against one row at a time."""
+    cfg = WIDE["wide"]
+    model, tensors = load(tmp_path, cfg, dtype=torch.bfloat16)
+    seqs = [ids(30, 200, seed=s) for s in range(21)]
+    want = [Want(cfg, tensors, s) for s in seqs[:3]]
+    x = torch.tensor(seqs, device="cuda")
+    cache, d = StaticKVCache(40), []
+    with torch.no_grad():
+        model(input_ids=x[:, :26], past_key_values=cache)
+        for t in range(26, 30):
+            out = model(input_ids=x[:, t:t + 1], past_key_values=cache).logits
+            for r in range(3):
+                d.append(errors(out[r], want[r], torch.bfloat16, slice(t, t + 1)))
+    small(torch.cat(d), torch.bfloat16, 1.5)
+
+
+def test_model_far_keys_on_the_gpu(tmp_path):
+    cfg = case(64, 64, 1e-5, latent(2, 64, 64, 64, 64, 1.0, None), latent(3, 32, 64, 64, 64, 1.0, None, kv_from=0),
+               hgrn2(2, 16, 32, dense(48)))
+    tensors = far_key_weights(cfg, 0, make_tensors(cfg, 3))
+    seq = [t % 60 for t in ids(420, 60, 8)]
+    for at in (0, 1, 127, 128, 255):
+        seq[at] = 63
+    want = Want(cfg, tensors, seq)
+    other = plain.forward(cfg, tensors, [62] + seq[1:])
+    model, _ = load(tmp_path, cfg, tensors)
+    x = torch.tensor([seq], device="cuda")
+    with torch.no_grad():
+        same(model(input_ids=x).logits[0], want, torch.float32, factor=2.0)
+        cache = StaticKVCache(420)
+        model(input_ids=x[:, :400], past_key_values=cache)
+        got = torch.cat([model(input_ids=x[:, t:t + 1], past_key_values=cache).logits[0] for t in range(400, 420)])
+    same(got, want, torch.float32, slice(400, None), 2.0)
+    moved = (other[400:] - want.logits[400:]).pow(2).mean(-1).sqrt().max() / want.logits.pow(2).mean().sqrt()
+    assert float(moved) > 20 * MODEL_TOL[torch.float32]   # the first token is seen from the end
+
+
+@pytest.mark.parametrize("name", ["mixed", "wide"])
+def test_model_greedy_generation_and_captured_decoding(tmp_path, name):
+    cfg = ALL[name]
+    model, tensors = load(tmp_path, cfg)
+    prompts = [ids(9, cfg["vocab"], 11), ids(9, cfg["vocab"], 12)]
+    want = []
+    for p in prompts:
+        seq = list(p)
+        for _ in range(10):
+            seq.append(int(plain.forward(cfg, tensors, seq)[-1].argmax()))
+        want.append(seq)
+    want = torch.tensor(want)
+    x = torch.tensor(prompts, device="cuda")
+    kw = dict(max_new_tokens=10, eos_token_id=None, pad_token_id=None)
+    assert torch.equal(model.generate(x, **kw).cpu(), want)
+    assert torch.equal(model.generate(x, cuda_graph=True, **kw).cpu(), want)
+    dec = GraphedGreedyDecoder(model, max_len=32)
+    for _ in range(2):                                    # the captured step, the cache and the states are used again
+        assert torch.equal(dec.generate(x, 10).cpu(), want)
+    assert dec.replays > 0
+    # the 16-bit model decodes the same tokens eagerly and from the captured step
+    half, _ = load(tmp_path, cfg, tensors, dtype=torch.bfloat16)
+    assert torch.equal(half.generate(x, **kw), half.generate(x, cuda_graph=True, **kw))
+
+
+def test_long_decoding_keeps_agreeing_with_the_prompt_form(tmp_path):
+    cfg = CASES["heads64"]
+    for dtype in (torch.float32, torch.bfloat16):
+        model, tensors = load(tmp_path, cfg, dtype=dtype)
+        seq = ids(400, 128, 5)
+        want = Want(cfg, tensors, seq)
+        x = torch.tensor([seq], device="cuda")
+        cache = StaticKVCache(400)
+        with torch.no_grad():
+            model(input_ids=x[:, :3], past_key_values=cache)
+            got = torch.cat([model(input_ids=x[:, t:t + 1], past_key_values=cache).logits[0] for t in range(3, 400)])
+        same(got, want, dtype, slice(3, None), 1.5)

@@ -66,8 +66,9 @@ def parse_args():
                          "least; the limit grows to 1.5 x the headline configuration's own run time per extra block)")
     ap.add_argument("--checkpoint-activations", action="store_true")
     ap.add_argument("--no-e2e", action="store_true")
-    ap.add_argument("--mode", default="train", choices=["train", "decode", "fusion"],
+    ap.add_argument("--mode", default="train", choices=["train", "decode", "fusion", "serving"],
                     help="train: tokens/s of a training step; decode: ms/token of greedy generation with a KV cache; "
+                         "serving: prompt and decode throughput of Moronex beside GPT-J at equal width, heads and layers; "
                          "fusion: seconds of one GPT-2 small beam-search generate() call before and after fuse() (the "
                          "benchmark behind the reference's published numbers)")
     ap.add_argument("--fusion-dtype", default="fp32", choices=["fp32", "bf16"],
@@ -361,6 +362,9 @@ def main() -> None:
     if args.mode == "fusion":
         fusion_main(args)
         return
+    if args.mode == "serving":
+        serving_main(args)
+        return
 
     import torch
     import torch.distributed as dist
@@ -564,6 +568,103 @@ def fusion_main(args) -> None:
     if world > 1:
         dist.barrier()
         dist.destroy_process_group()
+
+
+SERVING_SIZES = {   # width, heads, layers, q_rank, kv_rank, experts
+    "w2048": (2048, 16, 12, 1024, 512, 16),
+    "w4096": (4096, 32, 8, 1536, 512, 16),
+}
+
+
+def serving_config(width, heads, layers, q_rank, kv_rank, experts, vocab=50400):
+    """Layers in groups of four: two recurrent ones, latent attention, latent attention over the latents before it; the first
+    feed-forward is dense, the others are mixtures of experts whose 4 active experts have as many weights as GPT-J's MLP."""
+    dim = width // heads
+    out = []
+    for i in range(layers):
+        mlp = ({"kind": "dense", "ff": 8 * width // 3 // 64 * 64} if i == 0 else
+               {"kind": "moe", "expert": {"ff": width}, "router": {"experts": experts, "top": 4}})
+        mixer = {"heads": heads, "dim": dim, "vdim": dim}
+        if i % 4 >= 2:
+            mixer.update(q_rank=q_rank, kv_rank=kv_rank, scale=dim ** -0.5)
+            if i % 4 == 3:
+                mixer["kv_from"] = i - 1
+        out.append({"type": "latent_attention" if i % 4 >= 2 else "hgrn2", "mixer": mixer, "mlp": mlp})
+    return dict(vocab=vocab, width=width, norm={"eps": 1e-5}, layers=out)
+
+
+def serving_main(args) -> None:
+    """One GPU, random weights, bf16: prompt throughput (4 x 2048 tokens) and greedy decoding after 2048-token prompts with 1, 8
+    and 64 sequences (one CUDA-graph replay per token) of Moronex and of GPT-J with the same width, heads and number of
+    layers. A "step" is one ``GraphedGreedyDecoder.generate`` call; CUDA events around its prompt and its token loop; weights
+    and caches are larger than L2. ``--layers`` shortens both models (debug)."""
+    import gc
+
+    import torch
+
+    import oslo_b200 as ob
+    from oslo_b200.generation import GraphedGreedyDecoder
+
+    if args.gpus != 1:
+        raise SystemExit("--mode serving runs on one GPU")
+    torch.cuda.set_device(0)
+    dev = torch.device("cuda", 0)
+    ext = ob.ops.load_ext(required=True)
+    sampler = ClockSampler(0)
+    sampler.start()
+    l0, results = ext.launch_count(), {}
+    for size, (width, heads, layers, q_rank, kv_rank, experts) in SERVING_SIZES.items():
+        layers = args.layers or layers
+        for name in ("moronex", "gptj"):
+            if name == "moronex":
+                cls, cfg = ob.MoronexForCausalLM, ob.MoronexConfig(**serving_config(width, heads, layers, q_rank, kv_rank, experts),
+                                                                   torch_dtype=torch.bfloat16)
+            else:
+                cls, cfg = ob.GPTJForCausalLM, ob.GPTJConfig(vocab_size=50400, n_positions=4096, n_embd=width, n_layer=layers,
+                                                             n_head=heads, rotary_dim=64, torch_dtype=torch.bfloat16)
+            torch.manual_seed(1234)
+            with torch.device(dev):
+                model = cls._from_config(cfg, torch_dtype=torch.bfloat16)
+            model.fuse().eval()
+            rec = {"parameters": model.num_parameters()}
+            gen = torch.Generator().manual_seed(77)
+            for rows, prompt, new in ((4, 2048, 4), (1, 2048, 64), (8, 2048, 64), (64, 2048, 32)):
+                ids = torch.randint(0, 50400, (rows, prompt), generator=gen).to(dev)
+                dec = GraphedGreedyDecoder(model, max_len=prompt + new)
+                dec.record_events = True
+                pre, tok = [], []
+                for i in range(args.warmup + args.steps):
+                    dec.generate(ids, new)
+                    torch.cuda.synchronize()
+                    if i >= args.warmup:
+                        e = dec.events
+                        pre.append(e[0].elapsed_time(e[1]))
+                        tok.append(e[1].elapsed_time(e[2]) / (new - 1))
+                pre.sort(), tok.sort()
+                if rows == 4:
+                    rec["prompt_tokens_per_s"] = round(rows * prompt / pre[len(pre) // 2] * 1e3)
+                else:
+                    rec[f"decode_{rows}_ms_per_token"] = round(tok[len(tok) // 2], 4)
+                    rec[f"decode_{rows}_tokens_per_s"] = round(rows / tok[len(tok) // 2] * 1e3)
+                dec.release()
+                del dec, ids
+                torch.cuda.empty_cache()
+            results[f"{size}_{name}"] = rec
+            del model
+            gc.collect()
+            torch.cuda.empty_cache()
+    clocks = sampler.stop()
+    main_rec = results["w2048_moronex"]
+    print(json.dumps({
+        "metric": "Moronex prompt tokens/sec (width 2048)" + (" (debug)" if args.layers else ""), "value": main_rec["prompt_tokens_per_s"],
+        "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
+        "ms_per_step": 4 * 2048 / main_rec["prompt_tokens_per_s"] * 1e3, "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
+        "dtype": "bf16", "data": "synthetic uniform token ids, random-init weights", "impl": "oslo_b200",
+        "config": {"model": "moronex beside gptj", "global_batch": 4, "seq_len": 2048, "parallelism": "single",
+                   "sizes": {k: dict(zip(("width", "heads", "layers", "q_rank", "kv_rank", "experts"), v)) for k, v in SERVING_SIZES.items()},
+                   "l2": "weights + caches per step >> 126 MB L2, no explicit flush"},
+        "results": results, "clocks": clocks, "e2e": None, "gpu_launches": ext.launch_count() - l0,
+    }), flush=True)
 
 
 def decode_deployment_main(args) -> None:

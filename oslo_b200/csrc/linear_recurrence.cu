@@ -6,10 +6,11 @@
 //
 // Prefill (recurrence_kernel): a thread keeps a 16 x 4 tile of S in registers - rows in pairs, so that every update is a
 // packed two-float FMA - and G lanes share a column group; per token it reads 16 + 16 + 4 floats from shared memory,
-// does 96 packed FMAs and reduces 4 partial outputs over the G lanes. The prompt is
-// cut into chunks when (batch x heads) alone does not fill the GPU: local states of all chunks but the last from zero
-// (no outputs), one elementwise scan over the chunks, then every chunk again from its true initial state. Only
-// products of forget gates (<= 1) ever appear, so no chunk length can overflow.
+// does 96 packed FMAs and reduces 4 partial outputs over the G lanes. The prompt is cut into chunks when
+// (batch x heads) alone does not fill the GPU: local states of all chunks but the last from zero (no outputs), one
+// elementwise scan over the chunks, then every chunk again from its true initial state. Only products of forget gates
+// (<= 1) ever appear, so no chunk length can overflow. Three FMAs per state element and token bound the kernel: scalar
+// and packed FMAs take the same time here, half the nominal rate, and two resident blocks come close to that.
 // Decode (recurrence_step_kernel): a cluster of CTAs per (row, head), each on a slice of the value channels; the RMS
 // norm over the head's outputs is finished over distributed shared memory, so a step is one launch.
 // Tokens whose `keep` entry is 0 (padding) leave the state as it is and produce zeros.
@@ -437,7 +438,9 @@ extern "C" int oslo_recurrence_chunks(int B, int S, int H, int dim, int vdim, in
     const double per = static_cast<double>(S) / n;
     const auto fullest = [&](long long blocks) { return static_cast<double>((blocks + num_sms - 1) / num_sms); };
     // fewer than two blocks on an SM leave its pipes partly idle
-    const double c3 = std::max(1.4, fullest(ctas * n)) * per, c1 = n > 1 ? std::max(1.4, fullest(ctas * (n - 1))) * per * 0.67 + 16.0 + n : 0.0;
+    const double c3 = std::max(1.4, fullest(ctas * n)) * per;
+    // ... and the states' four trips through memory (16 bytes per element, in units of one token's update)
+    const double c1 = n > 1 ? std::max(1.4, fullest(ctas * (n - 1))) * per * 0.67 + 40.0 + 0.094 * B * H * n : 0.0;
     if (c3 + c1 < best_cost) { best_cost = c3 + c1; best = n; }
   }
   return best;

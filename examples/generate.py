@@ -5,6 +5,7 @@ greedy decoder, optionally tensor-parallel or through the deployment launcher.
     python -m torch.distributed.run --nproc-per-node 4 --master-addr 127.0.0.1 examples/generate.py \
         --model gptj --checkpoint out --tp 4 --num-beams 5 --no-repeat-ngram-size 2
     python examples/generate.py --model gptj --checkpoint out/merged --tp 4 --deployment    # one parent, 4 GPU workers
+    python examples/generate.py --model auto --checkpoint moronex --dtype bfloat16 --cuda-graph  # family from config.json
 
 Mirrors the reference's ``tests/*/ *_test_kernel_fusion.py`` / ``*_test_deployment.py`` usage. Prompts are encoded
 as UTF-8 bytes unless ``--tokenizer`` names a Hugging Face tokenizer directory.
@@ -12,6 +13,7 @@ as UTF-8 bytes unless ``--tokenizer`` names a Hugging Face tokenizer directory.
 from __future__ import annotations
 
 import argparse
+import json
 import os
 import sys
 import time
@@ -22,16 +24,18 @@ sys.path.insert(0, os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
 
 import oslo_b200 as ob  # noqa: E402
 
-CLASSES = {"gpt2": ob.GPT2LMHeadModel, "gpt_neo": ob.GPTNeoForCausalLM, "gptj": ob.GPTJForCausalLM}
+CLASSES = {name: entry.causal_lm for name, entry in ob.MODELS.items()}
 
 
 def main() -> None:
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
-    ap.add_argument("--model", default="gptj", choices=sorted(CLASSES))
+    ap.add_argument("--model", default="gptj", choices=sorted(CLASSES) + ["auto"],
+                    help="auto: the family the checkpoint's config.json names")
     ap.add_argument("--checkpoint", required=True)
+    ap.add_argument("--dtype", choices=["float32", "bfloat16", "float16"], help="parameter dtype (default: float32)")
     ap.add_argument("--tp", type=int, default=1)
     ap.add_argument("--deployment", action="store_true")
-    ap.add_argument("--prompt", default="Hello")
+    ap.add_argument("--prompt", nargs="+", default=["Hello"], help="one or more prompts; several run as one left-padded batch")
     ap.add_argument("--tokenizer")
     ap.add_argument("--max-new-tokens", type=int, default=32)
     ap.add_argument("--num-beams", type=int, default=1)
@@ -52,22 +56,31 @@ def main() -> None:
         decode = lambda ids: bytes(int(i) for i in ids if 0 <= int(i) < 256).decode("utf-8", "replace")  # noqa: E731
 
     on_gpu = torch.cuda.is_available() and os.environ.get("OSLO_B200_BACKEND", "nccl") != "gloo"
-    cls = CLASSES[args.model]
+    if args.model == "auto":
+        with open(os.path.join(args.checkpoint, "config.json"), encoding="utf-8") as f:
+            cls = ob.find_model(json.load(f)).causal_lm
+    else:
+        cls = CLASSES[args.model]
+    dtype = {"torch_dtype": getattr(torch, args.dtype)} if args.dtype else {}
     if args.tp > 1 or args.deployment:
         model = cls.from_pretrained_with_parallel(args.checkpoint, tensor_parallel_size=args.tp,
-                                                  deployment=args.deployment or None)
+                                                  deployment=args.deployment or None, **dtype)
         device = torch.device("cpu") if args.deployment else model.mpu.device
     else:
-        model = cls.from_pretrained(args.checkpoint)
+        model = cls.from_pretrained(args.checkpoint, **dtype)
         device = torch.device("cuda") if on_gpu else torch.device("cpu")
         model = model.to(device)
     if on_gpu and not args.deployment:
         model.fuse()
     model.eval()
-    ids = torch.tensor([encode(args.prompt)], dtype=torch.long, device=device)
+    rows = [encode(p) for p in args.prompt]
+    longest = max(len(r) for r in rows)
+    ids = torch.tensor([[0] * (longest - len(r)) + r for r in rows], dtype=torch.long, device=device)
     kw = dict(max_new_tokens=args.max_new_tokens, num_beams=args.num_beams, do_sample=args.do_sample,
               top_k=args.top_k, top_p=args.top_p, temperature=args.temperature,
               no_repeat_ngram_size=args.no_repeat_ngram_size)
+    if any(len(r) != longest for r in rows):
+        kw["attention_mask"] = torch.tensor([[0] * (longest - len(r)) + [1] * len(r) for r in rows], device=device)
     if args.cuda_graph:
         kw["cuda_graph"] = True
     if on_gpu and args.no_repeat_ngram_size:
@@ -76,9 +89,10 @@ def main() -> None:
     out = model.generate(ids, **{k: v for k, v in kw.items() if v is not None})
     dt = time.perf_counter() - t0
     if int(os.environ.get("RANK", "0")) == 0:
-        new = out[0, ids.size(1):].tolist()
-        print(decode(out[0].tolist()))
-        print(f"[{len(new)} new tokens in {dt:.2f} s]", file=sys.stderr)
+        for i in range(out.size(0)):
+            r = i * len(rows) // out.size(0)
+            print(decode(out[i, longest - len(rows[r]):].tolist()))
+        print(f"[{out.size(1) - longest} new tokens in {dt:.2f} s]", file=sys.stderr)
 
 
 if __name__ == "__main__":

@@ -451,3 +451,18 @@ def test_trace_runner(tmp_path):
         r.step({"step": 1, "entries": [{"id": "a", "tokens": a[7:8]}, {"id": "new", "tokens": [1]}], "end": []})
     with pytest.raises(ValueError):
         r.step({"step": 1, "entries": [{"id": "a", "tokens": a[7:9]}], "end": []})
+
+
+def test_generate_command_line(tmp_path):
+    cfg = case(256, 24, 1e-5, hgrn2(2, 8, 12, moe(16, 3, 2)), latent(2, 8, 12, 16, 16, 0.3, dense(32)))
+    model, _ = load(tmp_path, cfg)
+    prompts = ["a b", "longer prompt"]
+    run = subprocess.run(["python3", os.path.join(ROOT, "examples", "generate.py"), "--model", "auto", "--checkpoint", str(tmp_path),
+                          "--prompt", *prompts, "--max-new-tokens", "6"], capture_output=True,
+                         env={**os.environ, "CUDA_VISIBLE_DEVICES": "", "PYTHONPATH": ROOT})
+    assert run.returncode == 0, run.stderr.decode()[-600:]
+    want = b""
+    for p in prompts:
+        row = model.generate(torch.tensor([list(p.encode())]), max_new_tokens=6, eos_token_id=None, pad_token_id=None)[0]
+        want += bytes(row.tolist()).decode("utf-8", "replace").encode() + b"\n"
+    assert run.stdout == want

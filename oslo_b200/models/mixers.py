@@ -70,11 +70,12 @@ class LatentAttention(nn.Module):
                 latent: Optional[Tensor], keep: Optional[Tensor], output_attentions: bool = False) -> MixerOutput:
         """``h`` ``[batch * S, width]``; ``latent``: the latents of ``kv_layer`` when there is no cache; ``keep``
         ``[batch, past + S]`` marks real tokens (0 = padding)."""
+        from ..ops.cuda_ops import LATENT_MAX_RANK
         p = self.in_proj(h)
         side = {n: p[n] for n in self.side}
         s = h.size(0) // batch
         if (cache is not None and s == 1 and not output_attentions and self.oslo_fused and _inference(h, self.sink)
-                and ops.use_kernels(h)):
+                and ops.use_kernels(h) and self.kv_rank <= LATENT_MAX_RANK):
             return MixerOutput(self._decode(p, batch, kv_layer, cache, keep), side)
         q = self.uq(self.q_norm(p["dq"])).view(batch, s, self.heads, self.dim)
         if not self.shared_latents:

@@ -647,13 +647,29 @@ def silu_mul(gate: Tensor, up: Tensor) -> Tensor:
     return _ext().silu_mul(_rows(gate), _rows(up))
 
 
+RECURRENCE_MAX_DIM = 512   # key channels per head that one launch of the prompt kernel covers
+LATENT_MAX_RANK = 1024     # latent sizes that the decode kernel covers
+
+
 def gated_recurrence(q: Tensor, f: Tensor, v: Tensor, f_bias: Tensor, lower: Tensor, norm_w: Tensor, eps: float, batch: int,
                      heads: int, keep: Optional[Tensor], state: Optional[Tensor]) -> Tensor:
     dim, vdim = q.size(1) // heads, v.size(1) // heads
     if q.size(0) == batch and state is not None:      # one token per sequence
         return _ext().recurrence_step(_rows(q), _rows(f), _rows(v), f_bias, lower, norm_w, _keep8(keep), state, float(eps), heads,
                                       dim, vdim)
-    o = _ext().recurrence(_rows(q), _rows(f), _rows(v), f_bias, lower, _keep8(keep), state, batch, heads, dim, vdim)
+    if dim > RECURRENCE_MAX_DIM:      # key channels are independent of one another: sum the outputs of blocks of them
+        o = None
+        for a in range(0, dim, RECURRENCE_MAX_DIM):
+            b = min(dim, a + RECURRENCE_MAX_DIM)
+            cut = lambda t: t.reshape(-1, heads, dim)[:, :, a:b].reshape(t.size(0), -1)            # noqa: E731
+            part = state[:, :, a:b].contiguous() if state is not None else None
+            ob = _ext().recurrence(cut(q), cut(f), _rows(v), cut(f_bias[None])[0].contiguous(), cut(lower[None])[0].contiguous(),
+                                   _keep8(keep), part, batch, heads, b - a, vdim)
+            if state is not None:
+                state[:, :, a:b] = part
+            o = ob if o is None else o + ob
+    else:
+        o = _ext().recurrence(_rows(q), _rows(f), _rows(v), f_bias, lower, _keep8(keep), state, batch, heads, dim, vdim)
     return _ext().rms_norm(o.view(-1, vdim), norm_w, float(eps), 0.0).view(-1, heads * vdim)
 
 

@@ -31,6 +31,16 @@ def test_argument_defaults_finish_quickly():
     assert a.model == "gptj-6b" and a.seq == 2048
 
 
+def test_serving_sizes_are_valid_configurations():
+    sys.path.insert(0, ROOT)
+    import bench
+    import oslo_b200 as ob
+    for size in bench.SERVING_SIZES.values():
+        cfg = ob.MoronexConfig(**bench.serving_config(*size))
+        assert cfg.num_hidden_layers == size[2] and {l["type"] for l in cfg.layers} == {"latent_attention", "hgrn2"}
+        assert any(l["mixer"].get("kv_from") is not None for l in cfg.layers)
+
+
 def _reference_installed() -> bool:
     return os.path.isdir(os.path.join(ROOT, "baseline", "_ref", "oslo"))
 

@@ -82,7 +82,7 @@ def recurrence_inputs(batch, s, heads, dim, vdim, dtype, seed=0):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("batch,s,heads,dim,vdim", [(2, 37, 3, 48, 64), (1, 1, 2, 16, 8), (1, 200, 1, 12, 20), (2, 17, 2, 100, 33),
+@pytest.mark.parametrize("batch,s,heads,dim,vdim", [(2, 37, 3, 40, 72), (1, 1, 2, 16, 8), (1, 200, 1, 12, 20), (2, 17, 2, 100, 33),
                                                     (1, 150, 2, 128, 128), (3, 5, 1, 256, 24), (1, 9, 1, 300, 40), (2, 64, 2, 30, 72)])
 def test_recurrence(dtype, batch, s, heads, dim, vdim):
     q, f, v, fb, lower = recurrence_inputs(batch, s, heads, dim, vdim, dtype)
@@ -100,7 +100,7 @@ def test_recurrence(dtype, batch, s, heads, dim, vdim):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("batch,heads,dim,vdim", [(1, 4, 48, 64), (5, 3, 20, 30), (2, 16, 128, 128), (70, 2, 64, 256), (1, 1, 7, 2100)])
+@pytest.mark.parametrize("batch,heads,dim,vdim", [(1, 5, 40, 72), (5, 3, 20, 30), (2, 16, 128, 128), (70, 2, 64, 256), (1, 1, 7, 2100)])
 def test_recurrence_step_is_one_token_of_the_recurrence(dtype, batch, heads, dim, vdim):
     q, f, v, fb, lower = recurrence_inputs(batch, 1, heads, dim, vdim, dtype)
     w = rnd(vdim, dtype=dtype)
@@ -127,7 +127,7 @@ def test_sink_attention(dtype, batch, sq, sk, heads, dim, vdim):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("batch,heads,dim,vdim,rank,tmax,length", [(2, 4, 64, 64, 96, 200, 131), (1, 3, 20, 12, 40, 64, 1),
+@pytest.mark.parametrize("batch,heads,dim,vdim,rank,tmax,length", [(2, 6, 64, 72, 112, 200, 131), (1, 3, 20, 12, 40, 64, 1),
                                                                    (3, 17, 48, 80, 100, 96, 96), (1, 16, 128, 128, 512, 1500, 1400),
                                                                    (2, 8, 32, 64, 1000, 300, 290), (9, 2, 16, 24, 64, 33, 20),
                                                                    (1, 40, 64, 64, 256, 700, 641), (2, 5, 64, 64, 320, 400, 390)])
@@ -161,7 +161,7 @@ def test_latent_prep_norms_and_appends():
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("rows,width,ff,experts,top", [(1, 64, 32, 4, 2), (5, 40, 24, 3, 3), (16, 256, 96, 8, 2), (17, 256, 96, 8, 2),
+@pytest.mark.parametrize("rows,width,ff,experts,top", [(1, 64, 32, 4, 2), (5, 40, 24, 3, 3), (4, 192, 104, 9, 2), (17, 192, 104, 9, 2),
                                                        (200, 128, 300, 5, 1), (300, 36, 20, 7, 3), (700, 512, 256, 16, 4)])
 def test_moe(dtype, rows, width, ff, experts, top):
     h = rnd(rows, width, dtype=dtype)
@@ -354,6 +354,18 @@ def test_model_greedy_generation_and_captured_decoding(tmp_path, name):
     # the 16-bit model decodes the same tokens eagerly and from the captured step
     half, _ = load(tmp_path, cfg, tensors, dtype=torch.bfloat16)
     assert torch.equal(half.generate(x, **kw), half.generate(x, cuda_graph=True, **kw))
+
+
+def test_model_with_heads_and_latents_beyond_one_kernel(tmp_path):
+    cfg = case(40, 32, 1e-5, hgrn2(1, 700, 16, None), latent(2, 20, 300, 24, 1100, 0.2, None))
+    model, tensors = load(tmp_path, cfg)
+    seq = ids(24, 40)
+    want = Want(cfg, tensors, seq)
+    x = torch.tensor([seq], device="cuda")
+    cache = StaticKVCache(24)
+    with torch.no_grad():
+        got = [model(input_ids=x[:, a:b], past_key_values=cache).logits[0] for a, b in ((0, 15), (15, 20), (20, 21), (21, 22))]
+    same(torch.cat(got), want, torch.float32, slice(0, 22), 2.0)
 
 
 def test_long_decoding_keeps_agreeing_with_the_prompt_form(tmp_path):

@@ -36,7 +36,9 @@ struct FaParams {
   // position of the (seq, head, batch) coordinates inside each 4-D tensor map (dim 0 is always D)
   int q_pos[3], k_pos[3], v_pos[3];
   int* err;
-  // softmax with a sink and an output gate (both null: plain attention): exp(sink[h]) joins the denominator, row s of
+  int group;            // query heads per key / value head
+  float softcap;        // CAP kernels: scores become softcap * tanh(score / softcap)
+  // softmax with a sink and an output gate (null: without): exp(sink[h]) joins the denominator, row s of
   // head h is multiplied by sigmoid(gate[(b * Sq + s) * ldg + h]); only the first d_out columns are stored
   const void* sink;
   const void* gate;
@@ -46,7 +48,9 @@ struct FaParams {
 
 // PT = true: P goes back into TMEM (over the S buffer it came from, two bf16 per 32-bit column) and is the
 // A operand of P V straight from tensor memory; PT = false: P goes through a swizzled shared-memory tile.
-template <int D, int BN, bool PT>
+// CAP = true: capped scores, tanh(u) = 1 - 2 / (exp(2u) + 1) in 32-bit (absolute error about 2^-23 of the cap).
+// Head sizes below D: the tensor maps are as wide as the heads, TMA fills the rest of a tile with zeros.
+template <int D, int BN, bool PT, bool CAP>
 __global__ void __launch_bounds__(FA_THREADS, 1)
 fa_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUtensorMap tk,
               const __grid_constant__ CUtensorMap tv, const FaParams p) {
@@ -108,6 +112,7 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
 #pragma unroll
       for (int c = 0; c < DC; ++c) tma_load_rows(q_s + c * Q_SUB, &tq, bar(0), c * 64, q0, h, b, p.q_pos);
       bool ok = true;
+      const int hk = h / p.group;
       for (int j = 0; j < nblk && ok; ++j) {
         const int st = j & 1;
         const uint32_t ph = (j >> 1) & 1;
@@ -116,12 +121,12 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
         if (!ok) break;
         mbar_expect_tx(bar(1 + st), KV_BYTES);
 #pragma unroll
-        for (int c = 0; c < DC; ++c) tma_load_rows(k_s + st * KV_BYTES + c * KV_SUB, &tk, bar(1 + st), c * 64, n0, h, b, p.k_pos);
+        for (int c = 0; c < DC; ++c) tma_load_rows(k_s + st * KV_BYTES + c * KV_SUB, &tk, bar(1 + st), c * 64, n0, hk, b, p.k_pos);
         ok = mbar_wait(bar(7 + st), ph ^ 1, abort_flag, p.err, ERR_WAIT_EMPTY);
         if (!ok) break;
         mbar_expect_tx(bar(5 + st), KV_BYTES);
 #pragma unroll
-        for (int c = 0; c < DC; ++c) tma_load_rows(v_s + st * KV_BYTES + c * KV_SUB, &tv, bar(5 + st), c * 64, n0, h, b, p.v_pos);
+        for (int c = 0; c < DC; ++c) tma_load_rows(v_s + st * KV_BYTES + c * KV_SUB, &tv, bar(5 + st), c * 64, n0, hk, b, p.v_pos);
       }
     }
   } else if (warp == 1) {
@@ -181,7 +186,8 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
     const int row = q0 + row_l;
     const uint32_t t_lane = tmem_base + (static_cast<uint32_t>(quad * 32) << 16);
     const uint8_t* kpm_row = p.kpm ? p.kpm + static_cast<long long>(b) * p.Sk : nullptr;
-    const float sc = p.scale * FA_LOG2E;
+    const float sc = CAP ? 2.f * FA_LOG2E * p.scale / p.softcap : p.scale * FA_LOG2E;
+    const float cap = p.softcap * FA_LOG2E;
     const bool fp16 = p.fp16 != 0;
     float m_ref = -CUDART_INF_F, l_sum = 0.f;
     bool ok = true;
@@ -198,7 +204,10 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
         tmem_ld_32x32(t_lane + st * BN + c0, r);
         tmem_wait_ld();
 #pragma unroll
-        for (int i = 0; i < 32; ++i) s[c0 + i] = __uint_as_float(r[i]) * sc;
+        for (int i = 0; i < 32; ++i) {
+          s[c0 + i] = __uint_as_float(r[i]) * sc;
+          if (CAP) s[c0 + i] = cap - __fdividef(2.f * cap, exp2f(s[c0 + i]) + 1.f);
+        }
       }
       tc_fence_before();
       __syncwarp();
@@ -314,10 +323,14 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
       const long long gi = (static_cast<long long>(b) * p.Sq + row) * p.ldg + h;
       const float snk = fp16 ? __half2float(static_cast<const __half*>(p.sink)[h])
                              : __bfloat162float(static_cast<const __nv_bfloat16*>(p.sink)[h]);
-      const float gate = fp16 ? __half2float(static_cast<const __half*>(p.gate)[gi])
-                              : __bfloat162float(static_cast<const __nv_bfloat16*>(p.gate)[gi]);
       // m_ref is the running reference in log2 units; an overflowing sink term gives 1 / inf = 0
-      inv = 1.f / ((l_sum + exp2f(snk * 1.4426950408889634f - m_ref)) * (1.f + exp2f(-gate * 1.4426950408889634f)));
+      inv = l_sum + exp2f(snk * 1.4426950408889634f - m_ref);
+      if (p.gate != nullptr) {
+        const float gate = fp16 ? __half2float(static_cast<const __half*>(p.gate)[gi])
+                                : __bfloat162float(static_cast<const __nv_bfloat16*>(p.gate)[gi]);
+        inv *= 1.f + exp2f(-gate * 1.4426950408889634f);
+      }
+      inv = 1.f / inv;
     }
     uint16_t* orow = reinterpret_cast<uint16_t*>(p.out) + b * p.o_sb + h * p.o_sh + static_cast<long long>(row) * p.o_ss;
 #pragma unroll 1
@@ -363,19 +376,19 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
 }
 
 // ---------------------------------------------------------------------- host side
-template <int D, int BN, bool PT>
+template <int D, int BN, bool PT, bool CAP = false>
 static int fa_launch(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const FaParams& p,
                      cudaStream_t stream) {
   constexpr size_t smem = FA_BM * D * 2 + 4 * BN * D * 2 + (PT ? 0 : FA_BM * BN * 2) + 16 * 8 + 16 + 1024;
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(fa_fwd_kernel<D, BN, PT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    cudaError_t e = cudaFuncSetAttribute(fa_fwd_kernel<D, BN, PT, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          static_cast<int>(smem));
     if (e != cudaSuccess) return static_cast<int>(e);
     configured = true;
   }
   dim3 grid((p.Sq + FA_BM - 1) / FA_BM, p.H, p.B);
-  fa_fwd_kernel<D, BN, PT><<<grid, FA_THREADS, smem, stream>>>(tq, tk, tv, p);
+  fa_fwd_kernel<D, BN, PT, CAP><<<grid, FA_THREADS, smem, stream>>>(tq, tk, tv, p);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -383,12 +396,14 @@ static int fa_launch(const CUtensorMap& tq, const CUtensorMap& tk, const CUtenso
 
 namespace oslo {
 static int flash_fwd_entry(const void* q, const void* k, const void* v, void* o, float* lse, const uint8_t* kpm,
-                           const void* sink, const void* gate, long long ldg, int d_out, int B, int H, int Sq, int Sk, int D,
+                           const void* sink, const void* gate, long long ldg, int B, int H, int G, int Sq, int Sk, int dim, int vdim,
                            long long q_sb, long long q_sh, long long q_ss, long long k_sb, long long k_sh, long long k_ss,
                            long long v_sb, long long v_sh, long long v_ss, long long o_sb, long long o_sh, long long o_ss,
-                           float scale, int causal, int window, int dtype, int* err_word, cudaStream_t stream) {
-  if (B <= 0 || H <= 0 || Sq <= 0 || Sk <= 0) return -1;
-  if (D != 64 && D != 128 && D != 256) return -2;
+                           float scale, float softcap, int causal, int window, int dtype, int* err_word, cudaStream_t stream) {
+  if (B <= 0 || H <= 0 || Sq <= 0 || Sk <= 0 || G <= 0 || H % G) return -1;
+  const int widest = std::max(dim, vdim);
+  const int D = widest <= 64 ? 64 : (widest <= 128 ? 128 : 256);
+  if (dim <= 0 || vdim <= 0 || widest > 256 || dim % 8 || vdim % 8) return -2;
   if (dtype != OSLO_DT_BF16 && dtype != OSLO_DT_FP16) return -3;
   if ((reinterpret_cast<uintptr_t>(o) & 15) || (o_sb % 8) || (o_sh % 8) || (o_ss % 8)) return -4;
   static thread_local bool ctx_bound = false;
@@ -397,17 +412,22 @@ static int flash_fwd_entry(const void* q, const void* k, const void* v, void* o,
   const int bn = D == 256 ? 64 : 128;
   FaParams p;
   p.out = o; p.lse = lse; p.kpm = kpm;
-  p.sink = sink; p.gate = gate; p.ldg = ldg; p.d_out = d_out;
+  p.sink = sink; p.gate = gate; p.ldg = ldg; p.d_out = vdim; p.group = H / G; p.softcap = softcap;
   p.B = B; p.H = H; p.Sq = Sq; p.Sk = Sk;
   p.o_sb = o_sb; p.o_sh = o_sh; p.o_ss = o_ss;
   p.scale = scale; p.causal = causal; p.window = window; p.fp16 = fp16 ? 1 : 0; p.err = err_word;
   CUtensorMap tq, tk, tv;
-  int rc = make_qkv_map(&tq, q, B, H, Sq, D, q_sb, q_sh, q_ss, FA_BM, fp16, p.q_pos);
+  int rc = make_qkv_map(&tq, q, B, H, Sq, dim, q_sb, q_sh, q_ss, FA_BM, fp16, p.q_pos);
   if (rc) return rc;
-  rc = make_qkv_map(&tk, k, B, H, Sk, D, k_sb, k_sh, k_ss, bn, fp16, p.k_pos);
+  rc = make_qkv_map(&tk, k, B, G, Sk, dim, k_sb, k_sh, k_ss, bn, fp16, p.k_pos);
   if (rc) return rc - 1000;
-  rc = make_qkv_map(&tv, v, B, H, Sk, D, v_sb, v_sh, v_ss, bn, fp16, p.v_pos);
+  rc = make_qkv_map(&tv, v, B, G, Sk, vdim, v_sb, v_sh, v_ss, bn, fp16, p.v_pos);
   if (rc) return rc - 2000;
+  if (softcap > 0.f) {
+    if (D == 64) return fa_launch<64, 128, true, true>(tq, tk, tv, p, stream);
+    if (D == 128) return fa_launch<128, 128, true, true>(tq, tk, tv, p, stream);
+    return fa_launch<256, 64, true, true>(tq, tk, tv, p, stream);
+  }
   static const bool p_smem = [] { const char* e = getenv("OSLO_B200_ATTN_P_SMEM"); return e && e[0] == '1'; }();
   if (p_smem) {
     if (D == 64) return fa_launch<64, 128, false>(tq, tk, tv, p, stream);
@@ -426,17 +446,18 @@ extern "C" int oslo_flash_fwd_sm100(const void* q, const void* k, const void* v,
                                     long long v_sb, long long v_sh, long long v_ss, long long o_sb, long long o_sh,
                                     long long o_ss, float scale, int causal, int window, int dtype, int* err_word,
                                     cudaStream_t stream) {
-  return oslo::flash_fwd_entry(q, k, v, o, lse, kpm, nullptr, nullptr, 0, D, B, H, Sq, Sk, D, q_sb, q_sh, q_ss, k_sb, k_sh,
-                               k_ss, v_sb, v_sh, v_ss, o_sb, o_sh, o_ss, scale, causal, window, dtype, err_word, stream);
+  if (D != 64 && D != 128 && D != 256) return -2;
+  return oslo::flash_fwd_entry(q, k, v, o, lse, kpm, nullptr, nullptr, 0, B, H, H, Sq, Sk, D, D, q_sb, q_sh, q_ss, k_sb, k_sh,
+                               k_ss, v_sb, v_sh, v_ss, o_sb, o_sh, o_ss, scale, 0.f, causal, window, dtype, err_word, stream);
 }
 
 extern "C" int oslo_flash_sink_fwd_sm100(const void* q, const void* k, const void* v, void* o, const uint8_t* kpm,
-                                         const void* sink, const void* gate, long long ldg, int d_out, int B, int H, int Sq,
-                                         int Sk, int D, long long q_sb, long long q_sh, long long q_ss, long long k_sb,
+                                         const void* sink, const void* gate, long long ldg, int B, int H, int G, int Sq, int Sk,
+                                         int dim, int vdim, long long q_sb, long long q_sh, long long q_ss, long long k_sb,
                                          long long k_sh, long long k_ss, long long v_sb, long long v_sh, long long v_ss,
-                                         long long o_sb, long long o_sh, long long o_ss, float scale, int dtype, int* err_word,
-                                         cudaStream_t stream) {
-  if (sink == nullptr || gate == nullptr || d_out <= 0 || d_out > D || d_out % 8) return -1;
-  return oslo::flash_fwd_entry(q, k, v, o, nullptr, kpm, sink, gate, ldg, d_out, B, H, Sq, Sk, D, q_sb, q_sh, q_ss, k_sb, k_sh,
-                               k_ss, v_sb, v_sh, v_ss, o_sb, o_sh, o_ss, scale, 1, 0, dtype, err_word, stream);
+                                         long long o_sb, long long o_sh, long long o_ss, float scale, float softcap, int dtype,
+                                         int* err_word, cudaStream_t stream) {
+  if (sink == nullptr) return -1;
+  return oslo::flash_fwd_entry(q, k, v, o, nullptr, kpm, sink, gate, ldg, B, H, G, Sq, Sk, dim, vdim, q_sb, q_sh, q_ss, k_sb, k_sh,
+                               k_ss, v_sb, v_sh, v_ss, o_sb, o_sh, o_ss, scale, softcap, 1, 0, dtype, err_word, stream);
 }

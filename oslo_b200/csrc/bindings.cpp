@@ -788,7 +788,79 @@ Tensor silu_mul(const Tensor& gate, const Tensor& up) {
   return out;
 }
 
-// ---------------------------------------------------------------------- gated linear recurrence
+Tensor clamped_glu(const Tensor& gate, const Tensor& up, double limit, double alpha) {
+  check_rows(gate, "gate"); check_rows(up, "up");
+  TORCH_CHECK(gate.sizes() == up.sizes() && gate.scalar_type() == up.scalar_type(), "clamped_glu: operands differ");
+  c10::cuda::CUDAGuard guard(gate.device());
+  Tensor out = at::empty({gate.size(0), gate.size(1)}, gate.options());
+  check_rc(oslo_clamped_glu(gate.data_ptr(), gate.stride(0), up.data_ptr(), up.stride(0), out.data_ptr(), gate.size(0),
+                            static_cast<int>(gate.size(1)), static_cast<float>(limit), static_cast<float>(alpha), dt_code(gate),
+                            cur_stream()), "clamped_glu");
+  return out;
+}
+
+// up to three results join the stream; h1 / h2: the sum normed with w1 / w2 (empty without them)
+std::tuple<Tensor, Tensor, Tensor> branch_join(const Tensor& x, const Tensor& y0, const optional<Tensor>& n0, double f0,
+                                               const optional<Tensor>& y1, const optional<Tensor>& n1, double f1,
+                                               const optional<Tensor>& y2, const optional<Tensor>& n2, double f2, double mult,
+                                               double eps, const optional<Tensor>& w1, const optional<Tensor>& w2) {
+  check_rows(x, "x");
+  const int64_t rows = x.size(0), cols = x.size(1);
+  TORCH_CHECK(x.scalar_type() == at::kFloat && x.is_contiguous(), "branch_join: the residual stream is contiguous fp32");
+  const void *y[3], *w[3];
+  long long ldy[3];
+  float f[3];
+  int n = 0;
+  auto vec_ok = [&](const optional<Tensor>& v) {
+    return !(v.has_value() && v->defined()) || (v->is_contiguous() && v->numel() == cols && v->scalar_type() == y0.scalar_type());
+  };
+  auto add = [&](const Tensor& t, const optional<Tensor>& norm, double factor) {
+    check_rows(t, "y");
+    TORCH_CHECK(t.size(0) == rows && t.size(1) == cols && t.scalar_type() == y0.scalar_type() && vec_ok(norm), "branch_join: branch");
+    y[n] = t.data_ptr(); ldy[n] = t.stride(0); w[n] = ptr_or_null(norm); f[n] = static_cast<float>(factor);
+    ++n;
+  };
+  add(y0, n0, f0);
+  if (y1.has_value() && y1->defined()) add(*y1, n1, f1);
+  if (y2.has_value() && y2->defined()) add(*y2, n2, f2);
+  TORCH_CHECK(vec_ok(w1) && vec_ok(w2) && (ptr_or_null(w1) || !ptr_or_null(w2)), "branch_join: norm weights");
+  c10::cuda::CUDAGuard guard(x.device());
+  Tensor xo = at::empty_like(x);
+  Tensor h1 = at::empty({ptr_or_null(w1) ? rows : 0, cols}, y0.options()), h2 = at::empty({ptr_or_null(w2) ? rows : 0, cols}, y0.options());
+  check_rc(oslo_branch_join(x.data_ptr<float>(), n, y, ldy, w, f, static_cast<float>(mult), static_cast<float>(eps), ptr_or_null(w1),
+                            ptr_or_null(w2), xo.data_ptr<float>(), ptr_or_null(w1) ? h1.data_ptr() : nullptr,
+                            ptr_or_null(w2) ? h2.data_ptr() : nullptr, rows, static_cast<int>(cols), dt_code(y0), cur_stream()),
+           "branch_join");
+  return {xo, h1, h2};
+}
+
+Tensor gated_rms_norm(const Tensor& o, const Tensor& w, const Tensor& gate, double eps, int64_t group, int64_t act) {
+  check_rows(o, "o"); check_rows(gate, "gate");
+  TORCH_CHECK(o.scalar_type() == at::kFloat && o.is_contiguous() && w.is_contiguous() && w.numel() == o.size(1) &&
+                  gate.size(0) == o.size(0) && gate.size(1) == o.size(1) && gate.scalar_type() == w.scalar_type() && group > 0 &&
+                  o.size(1) % group == 0, "gated_rms_norm: operands");
+  c10::cuda::CUDAGuard guard(o.device());
+  Tensor out = at::empty({o.size(0), o.size(1)}, w.options());
+  check_rc(oslo_gated_rms_norm(o.data_ptr<float>(), w.data_ptr(), gate.data_ptr(), gate.stride(0), out.data_ptr(), o.size(0),
+                               static_cast<int>(o.size(1)), static_cast<int>(group), static_cast<float>(eps), static_cast<int>(act),
+                               dt_code(w), cur_stream()), "gated_rms_norm");
+  return out;
+}
+
+// x [P, M <= 4, K] (rows of a part contiguous in K), w [P, N, K] -> [P, M, N]
+Tensor gemv_stacked(const Tensor& x, const Tensor& w) {
+  TORCH_CHECK(x.is_cuda() && x.dim() == 3 && w.dim() == 3 && x.stride(2) == 1 && w.is_contiguous() && x.size(0) == w.size(0) &&
+                  x.size(2) == w.size(2) && x.scalar_type() == w.scalar_type(), "gemv_stacked: operands");
+  c10::cuda::CUDAGuard guard(x.device());
+  Tensor out = at::empty({x.size(0), x.size(1), w.size(1)}, x.options());
+  check_rc(oslo_gemv_stacked(x.data_ptr(), static_cast<int>(x.stride(1)), x.stride(0), w.data_ptr(), static_cast<int>(w.size(2)),
+                             w.size(1) * w.size(2), out.data_ptr(), static_cast<int>(x.size(0)), static_cast<int>(x.size(1)),
+                             static_cast<int>(w.size(1)), static_cast<int>(w.size(2)), dt_code(x), dev_state(x.get_device()).sms,
+                             cur_stream()), "gemv_stacked");
+  return out;
+}
+
+// ---------------------------------------------------------------------- linear recurrences
 void check_recurrence(const Tensor& q, const Tensor& f, const Tensor& v, const Tensor& f_bias, const Tensor& lower, int64_t heads,
                       int64_t dim, int64_t vdim) {
   check_rows(q, "q"); check_rows(f, "f"); check_rows(v, "v");
@@ -800,10 +872,13 @@ void check_recurrence(const Tensor& q, const Tensor& f, const Tensor& v, const T
                   lower.scalar_type() == q.scalar_type(), "recurrence: dtypes");
 }
 
-Tensor recurrence(const Tensor& q, const Tensor& f, const Tensor& v, const Tensor& f_bias, const Tensor& lower,
-                  const optional<Tensor>& keep, const optional<Tensor>& state, int64_t batch, int64_t heads, int64_t dim,
-                  int64_t vdim, int64_t chunks) {
-  check_recurrence(q, f, v, f_bias, lower, heads, dim, vdim);
+struct RecurrenceRule {
+  int rule = 0;
+  const Tensor *f_bias = nullptr, *lower = nullptr, *z = nullptr, *head_decay = nullptr;
+};
+
+Tensor run_recurrence(const RecurrenceRule& r, const Tensor& q, const Tensor& f, const Tensor& v, const optional<Tensor>& keep,
+                      const optional<Tensor>& state, int64_t batch, int64_t heads, int64_t dim, int64_t vdim, int64_t chunks) {
   TORCH_CHECK(batch > 0 && q.size(0) % batch == 0, "recurrence: rows are not batch x positions");
   const int64_t S = q.size(0) / batch;
   int64_t ld_keep = 0;
@@ -825,11 +900,103 @@ Tensor recurrence(const Tensor& q, const Tensor& f, const Tensor& v, const Tenso
     ws = at::empty({batch, nch, heads, dim, vdim}, f32);
     decay = at::empty({batch, nch, heads, dim}, f32);
   }
-  check_rc(oslo_recurrence(q.data_ptr(), q.stride(0), f.data_ptr(), f.stride(0), v.data_ptr(), v.stride(0), f_bias.data_ptr(),
-                           lower.data_ptr(), kp, ld_keep, st, out.data_ptr<float>(), nch > 1 ? ws.data_ptr<float>() : nullptr,
-                           nch > 1 ? decay.data_ptr<float>() : nullptr, nch, static_cast<int>(batch), static_cast<int>(S),
-                           static_cast<int>(heads), static_cast<int>(dim), static_cast<int>(vdim), dt_code(q),
-                           cur_stream(nch > 1 ? 3 : 1)), "recurrence");
+  check_rc(oslo_recurrence(r.rule, q.data_ptr(), q.stride(0), f.data_ptr(), f.stride(0), v.data_ptr(), v.stride(0),
+                           r.f_bias ? r.f_bias->data_ptr() : nullptr, r.lower ? r.lower->data_ptr() : nullptr,
+                           r.z ? r.z->data_ptr<float>() : nullptr, r.z ? r.z->stride(0) : 0,
+                           r.head_decay ? r.head_decay->data_ptr<float>() : nullptr, kp, ld_keep, st, out.data_ptr<float>(),
+                           nch > 1 ? ws.data_ptr<float>() : nullptr, nch > 1 ? decay.data_ptr<float>() : nullptr, nch,
+                           static_cast<int>(batch), static_cast<int>(S), static_cast<int>(heads), static_cast<int>(dim),
+                           static_cast<int>(vdim), dt_code(q), cur_stream(nch > 1 ? 3 : 1)), "recurrence");
+  return out;
+}
+
+Tensor recurrence(const Tensor& q, const Tensor& f, const Tensor& v, const Tensor& f_bias, const Tensor& lower,
+                  const optional<Tensor>& keep, const optional<Tensor>& state, int64_t batch, int64_t heads, int64_t dim,
+                  int64_t vdim, int64_t chunks) {
+  check_recurrence(q, f, v, f_bias, lower, heads, dim, vdim);
+  RecurrenceRule r;
+  r.f_bias = &f_bias; r.lower = &lower;
+  return run_recurrence(r, q, f, v, keep, state, batch, heads, dim, vdim, chunks);
+}
+
+void check_qkv_rows(const Tensor& q, const Tensor& k, const Tensor& v, int64_t heads, int64_t dim, int64_t vdim) {
+  check_rows(q, "q"); check_rows(k, "k"); check_rows(v, "v");
+  TORCH_CHECK(q.size(1) == heads * dim && k.sizes() == q.sizes() && v.size(1) == heads * vdim && v.size(0) == q.size(0) &&
+                  k.scalar_type() == q.scalar_type() && v.scalar_type() == q.scalar_type(), "recurrence: projections");
+}
+void check_head_decay(const Tensor& decay, int64_t heads) {
+  TORCH_CHECK(decay.is_cuda() && decay.is_contiguous() && decay.scalar_type() == at::kFloat && decay.numel() == heads, "head decays: fp32 [heads]");
+}
+
+Tensor decayed_recurrence(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& decay, const optional<Tensor>& keep,
+                          const optional<Tensor>& state, int64_t batch, int64_t heads, int64_t dim, int64_t vdim, int64_t chunks) {
+  check_qkv_rows(q, k, v, heads, dim, vdim);
+  check_head_decay(decay, heads);
+  RecurrenceRule r;
+  r.rule = 1; r.head_decay = &decay;
+  return run_recurrence(r, q, k, v, keep, state, batch, heads, dim, vdim, chunks);
+}
+
+void check_channels(const Tensor& t, int64_t n, const Tensor& like, const char* what) {
+  TORCH_CHECK(t.is_cuda() && t.is_contiguous() && t.numel() == n && t.scalar_type() == like.scalar_type(), what);
+}
+
+Tensor bonus_recurrence(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& z, const Tensor& w0, const Tensor& u,
+                        const optional<Tensor>& keep, const optional<Tensor>& state, int64_t batch, int64_t heads, int64_t dim,
+                        int64_t vdim, int64_t chunks) {
+  check_qkv_rows(q, k, v, heads, dim, vdim);
+  check_rows(z, "z");
+  TORCH_CHECK(z.scalar_type() == at::kFloat && z.sizes() == q.sizes(), "bonus_recurrence: decay logits are fp32 [rows, heads * dim]");
+  check_channels(w0, heads * dim, q, "bonus_recurrence: w0");
+  check_channels(u, heads * dim, q, "bonus_recurrence: u");
+  RecurrenceRule r;
+  r.rule = 2; r.f_bias = &w0; r.lower = &u; r.z = &z;
+  return run_recurrence(r, q, k, v, keep, state, batch, heads, dim, vdim, chunks);
+}
+
+void check_state(const Tensor& state, int64_t n) {
+  TORCH_CHECK(state.is_cuda() && state.is_contiguous() && state.scalar_type() == at::kFloat && state.numel() == n, "state: contiguous fp32 of the right size");
+}
+
+Tensor decayed_step(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& decay, const optional<Tensor>& keep, Tensor state,
+                    int64_t heads, int64_t dim, int64_t vdim) {
+  check_qkv_rows(q, k, v, heads, dim, vdim);
+  check_head_decay(decay, heads);
+  const int64_t B = q.size(0);
+  check_state(state, B * heads * dim * vdim);
+  int64_t ld_keep = 0;
+  const uint8_t* kp = keep_ptr(keep, B, 1, ld_keep);
+  c10::cuda::CUDAGuard guard(q.device());
+  Tensor out = at::empty({B, heads * vdim}, q.options().dtype(at::kFloat));
+  check_rc(oslo_decayed_step(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), decay.data_ptr<float>(),
+                             kp, ld_keep, state.data_ptr<float>(), out.data_ptr<float>(), static_cast<int>(B),
+                             static_cast<int>(heads), static_cast<int>(dim), static_cast<int>(vdim),
+                             dev_state(q.get_device()).sms, dt_code(q), cur_stream()), "decayed_step");
+  return out;
+}
+
+Tensor bonus_step(const Tensor& r, const Tensor& k, const Tensor& v, const Tensor& t, const Tensor& w2, const Tensor& w0, const Tensor& u,
+                  const Tensor& norm_w, const Tensor& gate, const optional<Tensor>& keep, Tensor state, double eps, int64_t heads,
+                  int64_t dim, int64_t vdim) {
+  check_qkv_rows(r, k, v, heads, dim, vdim);
+  check_rows(t, "t"); check_rows(gate, "gate");
+  const int64_t B = r.size(0);
+  check_state(state, B * heads * dim * vdim);
+  check_channels(w0, heads * dim, r, "bonus_step: w0");
+  check_channels(u, heads * dim, r, "bonus_step: u");
+  check_channels(norm_w, heads * vdim, r, "bonus_step: norm weight");
+  check_channels(w2, heads * dim * t.size(1), r, "bonus_step: w2");
+  TORCH_CHECK(t.size(0) == B && gate.size(0) == B && gate.size(1) == heads * vdim && t.scalar_type() == r.scalar_type() &&
+                  gate.scalar_type() == r.scalar_type(), "bonus_step: operands");
+  int64_t ld_keep = 0;
+  const uint8_t* kp = keep_ptr(keep, B, 1, ld_keep);
+  c10::cuda::CUDAGuard guard(r.device());
+  Tensor out = at::empty({B, heads * vdim}, r.options());
+  check_rc(oslo_bonus_step(r.data_ptr(), r.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), t.data_ptr(), t.stride(0),
+                           w2.data_ptr(), static_cast<int>(t.size(1)), w0.data_ptr(), u.data_ptr(), norm_w.data_ptr(),
+                           gate.data_ptr(), gate.stride(0), kp, ld_keep, state.data_ptr<float>(), out.data_ptr(),
+                           static_cast<float>(eps), static_cast<int>(B), static_cast<int>(heads), static_cast<int>(dim),
+                           static_cast<int>(vdim), dev_state(r.get_device()).sms, dt_code(r), cur_stream()), "bonus_step");
   return out;
 }
 
@@ -868,17 +1035,20 @@ Tensor sink_gate(const Tensor& o, const Tensor& lse, const Tensor& sink, const T
   return out;
 }
 
-// q, k, v [B, H, S, D] (any strides with contiguous D, D one of the flash kernel's sizes) -> [B * Sq, H * vdim]
+// q [B, H, Sq, dim], k [B, G, Sk, dim], v [B, G, Sk, vdim] (any strides that TMA takes, contiguous last dim) -> [B * Sq, H * vdim]
 Tensor flash_sink_fwd(const Tensor& q, const Tensor& k, const Tensor& v, const optional<Tensor>& kpm, const Tensor& sink,
-                      const Tensor& gate, double scale, int64_t vdim) {
-  TORCH_CHECK(q.is_cuda() && q.dim() == 4 && k.dim() == 4 && v.sizes() == k.sizes() && q.stride(3) == 1 && k.stride(3) == 1 &&
-                  v.stride(3) == 1 && k.size(3) == q.size(3) && k.size(0) == q.size(0) && k.size(1) == q.size(1) &&
-                  k.size(2) >= q.size(2), "flash_sink_fwd: q, k, v");
-  const int64_t B = q.size(0), H = q.size(1), Sq = q.size(2), Sk = k.size(2), D = q.size(3);
-  check_rows(gate, "gate");
-  TORCH_CHECK(vdim > 0 && vdim <= D && vdim % 8 == 0 && gate.size(0) == B * Sq && gate.size(1) == H && sink.numel() == H &&
-                  k.scalar_type() == q.scalar_type() && v.scalar_type() == q.scalar_type() && gate.scalar_type() == q.scalar_type() &&
+                      const optional<Tensor>& gate, double scale, double softcap) {
+  TORCH_CHECK(q.is_cuda() && q.dim() == 4 && k.dim() == 4 && v.dim() == 4 && q.stride(3) == 1 && k.stride(3) == 1 && v.stride(3) == 1 &&
+                  k.size(3) == q.size(3) && k.size(0) == q.size(0) && v.size(0) == q.size(0) && v.size(1) == k.size(1) &&
+                  v.size(2) == k.size(2) && q.size(1) % k.size(1) == 0 && k.size(2) >= q.size(2), "flash_sink_fwd: q, k, v");
+  const int64_t B = q.size(0), H = q.size(1), G = k.size(1), Sq = q.size(2), Sk = k.size(2), dim = q.size(3), vdim = v.size(3);
+  TORCH_CHECK(sink.is_contiguous() && sink.numel() == H && k.scalar_type() == q.scalar_type() && v.scalar_type() == q.scalar_type() &&
                   sink.scalar_type() == q.scalar_type(), "flash_sink_fwd: operands");
+  const bool gated = gate.has_value() && gate->defined();
+  if (gated) {
+    check_rows(*gate, "gate");
+    TORCH_CHECK(gate->size(0) == B * Sq && gate->size(1) == H && gate->scalar_type() == q.scalar_type(), "flash_sink_fwd: gate");
+  }
   const uint8_t* kp = nullptr;
   if (kpm.has_value() && kpm->defined()) {
     TORCH_CHECK(kpm->is_contiguous() && kpm->scalar_type() == at::kByte && kpm->numel() == B * Sk, "flash_sink_fwd: mask");
@@ -887,35 +1057,197 @@ Tensor flash_sink_fwd(const Tensor& q, const Tensor& k, const Tensor& v, const o
   c10::cuda::CUDAGuard guard(q.device());
   Tensor out = at::empty({B * Sq, H * vdim}, q.options());
   check_rc(oslo_flash_sink_fwd_sm100(q.data_ptr(), k.data_ptr(), v.data_ptr(), out.data_ptr(), kp, sink.data_ptr(),
-                                     gate.data_ptr(), gate.stride(0), static_cast<int>(vdim), static_cast<int>(B),
-                                     static_cast<int>(H), static_cast<int>(Sq), static_cast<int>(Sk), static_cast<int>(D),
-                                     q.stride(0), q.stride(1), q.stride(2), k.stride(0), k.stride(1), k.stride(2), v.stride(0),
-                                     v.stride(1), v.stride(2), Sq * H * vdim, vdim, H * vdim, static_cast<float>(scale),
-                                     dt_code(q), dev_state(q.get_device()).err.data_ptr<int>(), cur_stream()), "flash_sink_fwd");
+                                     ptr_or_null(gate), gated ? gate->stride(0) : 0, static_cast<int>(B), static_cast<int>(H),
+                                     static_cast<int>(G), static_cast<int>(Sq), static_cast<int>(Sk), static_cast<int>(dim),
+                                     static_cast<int>(vdim), q.stride(0), q.stride(1), q.stride(2), k.stride(0), k.stride(1),
+                                     k.stride(2), v.stride(0), v.stride(1), v.stride(2), Sq * H * vdim, vdim, H * vdim,
+                                     static_cast<float>(scale), static_cast<float>(softcap), dt_code(q),
+                                     dev_state(q.get_device()).err.data_ptr<int>(), cur_stream()), "flash_sink_fwd");
   return out;
 }
 
 Tensor sink_attention(const Tensor& q, const Tensor& k, const Tensor& v, const optional<Tensor>& keep, const Tensor& sink,
-                      const Tensor& gate, double scale) {
-  // [B, S, H, D] views with contiguous D
+                      const optional<Tensor>& gate, double scale, double softcap) {
+  // [B, S, heads, D] views with contiguous D
   TORCH_CHECK(q.is_cuda() && q.dim() == 4 && k.dim() == 4 && v.dim() == 4 && q.stride(3) == 1 && k.stride(3) == 1 && v.stride(3) == 1,
               "sink_attention: q, k, v must be [B, S, H, D] with a contiguous last dim");
-  const int64_t B = q.size(0), Sq = q.size(1), H = q.size(2), D = q.size(3), Sk = k.size(1), Dv = v.size(3);
-  TORCH_CHECK(k.size(0) == B && v.size(0) == B && k.size(2) == H && v.size(2) == H && v.size(1) == Sk && k.size(3) == D && Sk >= Sq,
+  const int64_t B = q.size(0), Sq = q.size(1), H = q.size(2), G = k.size(2), D = q.size(3), Sk = k.size(1), Dv = v.size(3);
+  TORCH_CHECK(k.size(0) == B && v.size(0) == B && H % G == 0 && v.size(2) == G && v.size(1) == Sk && k.size(3) == D && Sk >= Sq,
               "sink_attention: sizes");
-  check_rows(gate, "gate");
-  TORCH_CHECK(gate.size(0) == B * Sq && gate.size(1) == H && sink.numel() == H, "sink_attention: gate / sink sizes");
-  TORCH_CHECK(k.scalar_type() == q.scalar_type() && v.scalar_type() == q.scalar_type() && gate.scalar_type() == q.scalar_type() &&
-                  sink.scalar_type() == q.scalar_type(), "sink_attention: dtypes");
+  TORCH_CHECK(sink.is_contiguous() && sink.numel() == H && k.scalar_type() == q.scalar_type() && v.scalar_type() == q.scalar_type() &&
+                  sink.scalar_type() == q.scalar_type(), "sink_attention: operands");
+  const bool gated = gate.has_value() && gate->defined();
+  if (gated) {
+    check_rows(*gate, "gate");
+    TORCH_CHECK(gate->size(0) == B * Sq && gate->size(1) == H && gate->scalar_type() == q.scalar_type(), "sink_attention: gate");
+  }
   int64_t ld_keep = 0;
   const uint8_t* kp = keep_ptr(keep, B, Sk, ld_keep);
   c10::cuda::CUDAGuard guard(q.device());
   Tensor out = at::empty({B * Sq, H * Dv}, q.options());
   check_rc(oslo_sink_attention(q.data_ptr(), q.stride(0), q.stride(1), q.stride(2), k.data_ptr(), k.stride(0), k.stride(1),
                                k.stride(2), v.data_ptr(), v.stride(0), v.stride(1), v.stride(2), kp, ld_keep, sink.data_ptr(),
-                               gate.data_ptr(), gate.stride(0), out.data_ptr(), static_cast<int>(B), static_cast<int>(H),
-                               static_cast<int>(Sq), static_cast<int>(Sk), static_cast<int>(D), static_cast<int>(Dv),
-                               static_cast<float>(scale), dt_code(q), cur_stream()), "sink_attention");
+                               ptr_or_null(gate), gated ? gate->stride(0) : 0, out.data_ptr(), static_cast<int>(B),
+                               static_cast<int>(H), static_cast<int>(G), static_cast<int>(Sq), static_cast<int>(Sk),
+                               static_cast<int>(D), static_cast<int>(Dv), static_cast<float>(scale), static_cast<float>(softcap),
+                               dt_code(q), cur_stream()), "sink_attention");
+  return out;
+}
+
+// ---------------------------------------------------------------------- grouped-query attention
+Tensor qkv_prep(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& wq, const Tensor& wk, double eps, const Tensor& positions,
+                const Tensor& freq, Tensor kc, Tensor vc, const Tensor& lengths) {
+  check_rows(q, "q"); check_rows(k, "k"); check_rows(v, "v");
+  TORCH_CHECK(kc.dim() == 4 && vc.dim() == 4 && kc.is_contiguous() && vc.is_contiguous() && vc.size(0) == kc.size(0) &&
+                  vc.size(1) == kc.size(1) && vc.size(2) == kc.size(2), "qkv_prep: caches");
+  const int64_t B = kc.size(0), G = kc.size(1), T = kc.size(2), dim = kc.size(3), vdim = vc.size(3);
+  TORCH_CHECK(q.size(0) % B == 0 && q.size(1) % dim == 0 && k.size(0) == q.size(0) && v.size(0) == q.size(0) && k.size(1) == G * dim &&
+                  v.size(1) == G * vdim, "qkv_prep: projections");
+  const int64_t S = q.size(0) / B, H = q.size(1) / dim;
+  for (const Tensor* t : {&k, &v, static_cast<const Tensor*>(&kc), static_cast<const Tensor*>(&vc)})
+    TORCH_CHECK(t->scalar_type() == q.scalar_type(), "qkv_prep: dtypes");
+  check_channels(wq, dim, q, "qkv_prep: query norm weight");
+  check_channels(wk, dim, q, "qkv_prep: key norm weight");
+  TORCH_CHECK(positions.is_cuda() && positions.dim() == 2 && positions.size(0) == B && positions.size(1) == S && positions.scalar_type() == at::kLong, "qkv_prep: positions");
+  TORCH_CHECK(freq.is_cuda() && freq.is_contiguous() && freq.scalar_type() == at::kFloat && 2 * freq.numel() <= dim, "qkv_prep: frequencies");
+  TORCH_CHECK(lengths.scalar_type() == at::kInt && lengths.is_contiguous() && lengths.numel() == B, "qkv_prep: lengths");
+  c10::cuda::CUDAGuard guard(q.device());
+  Tensor out = at::empty({B, S, H, dim}, q.options());
+  check_rc(oslo_qkv_prep(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), wq.data_ptr(), wk.data_ptr(),
+                         static_cast<float>(eps), reinterpret_cast<const long long*>(positions.data_ptr<int64_t>()), positions.stride(0),
+                         positions.stride(1), freq.numel() ? freq.data_ptr<float>() : nullptr, static_cast<int>(freq.numel()),
+                         out.data_ptr(), kc.data_ptr(), vc.data_ptr(), lengths.data_ptr<int>(), static_cast<int>(B),
+                         static_cast<int>(S), static_cast<int>(H), static_cast<int>(G), static_cast<int>(dim),
+                         static_cast<int>(vdim), static_cast<int>(T), dt_code(q), dev_state(q.get_device()).err.data_ptr<int>(),
+                         cur_stream()), "qkv_prep");
+  return out;
+}
+
+Tensor grouped_decode(const Tensor& q, const Tensor& kc, const Tensor& vc, const Tensor& lengths, const optional<Tensor>& keep,
+                      const Tensor& sink, double scale, double softcap) {
+  TORCH_CHECK(q.is_cuda() && q.dim() == 3 && q.is_contiguous() && kc.dim() == 4 && vc.dim() == 4 && kc.is_contiguous() && vc.is_contiguous() &&
+                  vc.size(0) == kc.size(0) && vc.size(1) == kc.size(1) && vc.size(2) == kc.size(2) && kc.size(0) == q.size(0) &&
+                  kc.size(3) == q.size(2) && q.size(1) % kc.size(1) == 0, "grouped_decode: q [B, H, dim], caches [B, G, T, *]");
+  const int64_t B = q.size(0), H = q.size(1), G = kc.size(1), T = kc.size(2), vdim = vc.size(3);
+  TORCH_CHECK(sink.is_contiguous() && sink.numel() == H && kc.scalar_type() == q.scalar_type() && vc.scalar_type() == q.scalar_type() &&
+                  sink.scalar_type() == q.scalar_type(), "grouped_decode: operands");
+  TORCH_CHECK(lengths.scalar_type() == at::kInt && lengths.is_contiguous() && lengths.numel() == B, "grouped_decode: lengths");
+  int64_t ld_keep = 0;
+  const uint8_t* kp = keep_ptr(keep, B, 0, ld_keep);
+  c10::cuda::CUDAGuard guard(q.device());
+  auto& st = dev_state(q.get_device());
+  const int splits = oslo_grouped_splits(static_cast<int>(B), static_cast<int>(H), static_cast<int>(G), static_cast<int>(T), st.sms);
+  const auto f32 = q.options().dtype(at::kFloat);
+  Tensor ws = at::empty({B, H, splits, (vdim + 3) / 4 * 4}, f32);
+  Tensor stat = at::empty({B, H, splits, 2}, f32);
+  Tensor out = at::empty({B, H * vdim}, q.options());
+  check_rc(oslo_grouped_decode(q.data_ptr(), kc.data_ptr(), vc.data_ptr(), lengths.data_ptr<int>(), kp, ld_keep,
+                               kp ? static_cast<int>(keep->size(1)) : 0, sink.data_ptr(), ws.data_ptr<float>(), stat.data_ptr<float>(),
+                               out.data_ptr(), static_cast<int>(B), static_cast<int>(H), static_cast<int>(G),
+                               static_cast<int>(q.size(2)), static_cast<int>(vdim), static_cast<int>(T), splits,
+                               static_cast<float>(scale), static_cast<float>(softcap), dt_code(q), st.err.data_ptr<int>(),
+                               cur_stream(2)), "grouped_decode");
+  return out;
+}
+
+// ---------------------------------------------------------------------- token shift, convolution, selective scan
+float* carried_ptr(const optional<Tensor>& t, int64_t n) {
+  if (!(t.has_value() && t->defined())) return nullptr;
+  check_state(*t, n);
+  return t->data_ptr<float>();
+}
+
+Tensor token_shift(const Tensor& h, const Tensor& mu, int64_t batch, const optional<Tensor>& keep, optional<Tensor> prev) {
+  check_rows(h, "h");
+  TORCH_CHECK(batch > 0 && h.size(0) % batch == 0 && mu.dim() == 2 && mu.is_contiguous() && mu.size(1) == h.size(1) &&
+                  mu.scalar_type() == h.scalar_type(), "token_shift: operands");
+  const int64_t S = h.size(0) / batch, width = h.size(1), P = mu.size(0);
+  int64_t ld_keep = 0;
+  const uint8_t* kp = keep_ptr(keep, batch, S, ld_keep);
+  c10::cuda::CUDAGuard guard(h.device());
+  Tensor out = at::empty({P, h.size(0), width}, h.options());
+  check_rc(oslo_token_shift(h.data_ptr(), h.stride(0), mu.data_ptr(), kp, ld_keep, carried_ptr(prev, batch * width), out.data_ptr(),
+                            static_cast<int>(batch), static_cast<int>(S), static_cast<int>(width), static_cast<int>(P), dt_code(h),
+                            cur_stream()), "token_shift");
+  return out;
+}
+
+Tensor causal_conv_silu(const Tensor& x, const Tensor& w, const Tensor& bias, int64_t batch, const optional<Tensor>& keep,
+                        optional<Tensor> prev) {
+  check_rows(x, "x");
+  const int64_t C = x.size(1);
+  TORCH_CHECK(batch > 0 && x.size(0) % batch == 0 && w.dim() == 2 && w.is_contiguous() && w.size(0) == C && w.scalar_type() == x.scalar_type(),
+              "causal_conv_silu: operands");
+  check_channels(bias, C, x, "causal_conv_silu: bias");
+  const int64_t S = x.size(0) / batch, taps = w.size(1);
+  int64_t ld_keep = 0;
+  const uint8_t* kp = keep_ptr(keep, batch, S, ld_keep);
+  c10::cuda::CUDAGuard guard(x.device());
+  Tensor out = at::empty({x.size(0), C}, x.options());
+  check_rc(oslo_causal_conv_silu(x.data_ptr(), x.stride(0), w.data_ptr(), bias.data_ptr(), kp, ld_keep,
+                                 carried_ptr(prev, batch * (taps - 1) * C), out.data_ptr(), static_cast<int>(batch),
+                                 static_cast<int>(S), static_cast<int>(C), static_cast<int>(taps), dt_code(x), cur_stream()),
+           "causal_conv_silu");
+  return out;
+}
+
+void check_scan(const Tensor& x, const Tensor& dt_bias, const Tensor& a_log, const Tensor& b, const Tensor& c, const Tensor& d, const Tensor& z) {
+  check_rows(x, "x"); check_rows(b, "b"); check_rows(c, "c"); check_rows(z, "z");
+  const int64_t C = x.size(1);
+  TORCH_CHECK(a_log.dim() == 2 && a_log.size(0) == C, "selective_scan: a_log is [channels, states]");
+  const int64_t N = a_log.size(1);
+  check_channels(a_log, C * N, x, "selective_scan: a_log");
+  check_channels(dt_bias, C, x, "selective_scan: dt bias");
+  check_channels(d, C, x, "selective_scan: d");
+  TORCH_CHECK(z.sizes() == x.sizes() && b.size(0) == x.size(0) && c.size(0) == x.size(0) && b.size(1) == N && c.size(1) == N &&
+                  z.scalar_type() == x.scalar_type() && b.scalar_type() == x.scalar_type() && c.scalar_type() == x.scalar_type(),
+              "selective_scan: operands");
+}
+
+Tensor selective_scan(const Tensor& x, const Tensor& dt, const Tensor& dt_bias, const Tensor& a_log, const Tensor& b, const Tensor& c,
+                      const Tensor& d, const Tensor& z, int64_t batch, const optional<Tensor>& keep, optional<Tensor> state,
+                      int64_t chunks) {
+  check_scan(x, dt_bias, a_log, b, c, d, z);
+  check_rows(dt, "dt");
+  TORCH_CHECK(batch > 0 && x.size(0) % batch == 0 && dt.sizes() == x.sizes() && dt.scalar_type() == at::kFloat, "selective_scan: dt is fp32 [rows, channels]");
+  const int64_t S = x.size(0) / batch, C = x.size(1), N = a_log.size(1);
+  int64_t ld_keep = 0;
+  const uint8_t* kp = keep_ptr(keep, batch, S, ld_keep);
+  c10::cuda::CUDAGuard guard(x.device());
+  const int nch = chunks > 0 ? static_cast<int>(chunks)
+                             : oslo_scan_chunks(static_cast<int>(batch), static_cast<int>(S), static_cast<int>(C),
+                                                static_cast<int>(N), dev_state(x.get_device()).sms);
+  const auto f32 = x.options().dtype(at::kFloat);
+  Tensor out = at::empty({x.size(0), C}, x.options());
+  Tensor ws, steps;
+  if (nch > 1) {
+    ws = at::empty({batch, nch, C, N}, f32);
+    steps = at::empty({batch, nch, C}, f32);
+  }
+  check_rc(oslo_selective_scan(x.data_ptr(), x.stride(0), dt.data_ptr<float>(), dt.stride(0), dt_bias.data_ptr(), a_log.data_ptr(),
+                               b.data_ptr(), b.stride(0), c.data_ptr(), c.stride(0), d.data_ptr(), z.data_ptr(), z.stride(0), kp,
+                               ld_keep, carried_ptr(state, batch * C * N), out.data_ptr(), nch > 1 ? ws.data_ptr<float>() : nullptr,
+                               nch > 1 ? steps.data_ptr<float>() : nullptr, nch, static_cast<int>(batch), static_cast<int>(S),
+                               static_cast<int>(C), static_cast<int>(N), dt_code(x), cur_stream(nch > 1 ? 3 : 1)), "selective_scan");
+  return out;
+}
+
+Tensor scan_step(const Tensor& x, const Tensor& dt, const Tensor& w_dt, const Tensor& dt_bias, const Tensor& a_log, const Tensor& b,
+                 const Tensor& c, const Tensor& d, const Tensor& z, const optional<Tensor>& keep, Tensor state) {
+  check_scan(x, dt_bias, a_log, b, c, d, z);
+  check_rows(dt, "dt");
+  const int64_t B = x.size(0), C = x.size(1), N = a_log.size(1);
+  TORCH_CHECK(dt.size(0) == B && dt.scalar_type() == x.scalar_type(), "scan_step: dt");
+  check_channels(w_dt, C * dt.size(1), x, "scan_step: step projection");
+  check_state(state, B * C * N);
+  int64_t ld_keep = 0;
+  const uint8_t* kp = keep_ptr(keep, B, 1, ld_keep);
+  c10::cuda::CUDAGuard guard(x.device());
+  Tensor out = at::empty({B, C}, x.options());
+  check_rc(oslo_scan_step(x.data_ptr(), x.stride(0), dt.data_ptr(), dt.stride(0), w_dt.data_ptr(), static_cast<int>(dt.size(1)),
+                          dt_bias.data_ptr(), a_log.data_ptr(), b.data_ptr(), b.stride(0), c.data_ptr(), c.stride(0), d.data_ptr(),
+                          z.data_ptr(), z.stride(0), kp, ld_keep, state.data_ptr<float>(), out.data_ptr(), static_cast<int>(B),
+                          static_cast<int>(C), static_cast<int>(N), dt_code(x), cur_stream()), "scan_step");
   return out;
 }
 
@@ -1100,14 +1432,28 @@ TORCH_LIBRARY(oslo_b200, m) {
   m.def("recurrence(Tensor q, Tensor f, Tensor v, Tensor f_bias, Tensor lower, Tensor? keep, Tensor(a!)? state, int batch, int heads, int dim, int vdim, int chunks=0) -> Tensor");
   m.def("recurrence_step(Tensor q, Tensor f, Tensor v, Tensor f_bias, Tensor lower, Tensor norm_w, Tensor? keep, Tensor(a!) state, float eps, int heads, int dim, int vdim) -> Tensor");
   m.def("sink_gate(Tensor o, Tensor lse, Tensor sink, Tensor gate, int vdim) -> Tensor");
-  m.def("flash_sink_fwd(Tensor q, Tensor k, Tensor v, Tensor? kpm, Tensor sink, Tensor gate, float scale, int vdim) -> Tensor");
-  m.def("sink_attention(Tensor q, Tensor k, Tensor v, Tensor? keep, Tensor sink, Tensor gate, float scale) -> Tensor");
+  m.def("flash_sink_fwd(Tensor q, Tensor k, Tensor v, Tensor? kpm, Tensor sink, Tensor? gate, float scale, float softcap) -> Tensor");
+  m.def("sink_attention(Tensor q, Tensor k, Tensor v, Tensor? keep, Tensor sink, Tensor? gate, float scale, float softcap) -> Tensor");
   m.def("latent_prep(Tensor cq, Tensor wq, Tensor? ckv, Tensor? wkv, Tensor(a!)? cache, Tensor lengths, float eps) -> Tensor");
   m.def("latent_decode(Tensor q, Tensor w_uk, Tensor w_uv, Tensor cache, Tensor lengths, Tensor? keep, Tensor sink, Tensor gate, float scale, int heads) -> Tensor");
   m.def("moe_route(Tensor h, Tensor w, Tensor bias, Tensor? logits, int top) -> (Tensor, Tensor)");
   m.def("moe_plan(Tensor h, Tensor idx, int experts) -> (Tensor, Tensor, Tensor, Tensor)");
   m.def("moe_grouped(Tensor rows, Tensor w, Tensor tile_group, Tensor n_tiles, bool relu2) -> Tensor");
   m.def("moe_few(Tensor x, Tensor idx, Tensor w, int per_row, bool relu2) -> Tensor");
+  m.def("clamped_glu(Tensor gate, Tensor up, float limit, float alpha) -> Tensor");
+  m.def("branch_join(Tensor x, Tensor y0, Tensor? n0, float f0, Tensor? y1, Tensor? n1, float f1, Tensor? y2, Tensor? n2, float f2, float mult, float eps, Tensor? w1, Tensor? w2) -> (Tensor, Tensor, Tensor)");
+  m.def("gated_rms_norm(Tensor o, Tensor w, Tensor gate, float eps, int group, int act) -> Tensor");
+  m.def("gemv_stacked(Tensor x, Tensor w) -> Tensor");
+  m.def("decayed_recurrence(Tensor q, Tensor k, Tensor v, Tensor decay, Tensor? keep, Tensor(a!)? state, int batch, int heads, int dim, int vdim, int chunks=0) -> Tensor");
+  m.def("bonus_recurrence(Tensor q, Tensor k, Tensor v, Tensor z, Tensor w0, Tensor u, Tensor? keep, Tensor(a!)? state, int batch, int heads, int dim, int vdim, int chunks=0) -> Tensor");
+  m.def("decayed_step(Tensor q, Tensor k, Tensor v, Tensor decay, Tensor? keep, Tensor(a!) state, int heads, int dim, int vdim) -> Tensor");
+  m.def("bonus_step(Tensor r, Tensor k, Tensor v, Tensor t, Tensor w2, Tensor w0, Tensor u, Tensor norm_w, Tensor gate, Tensor? keep, Tensor(a!) state, float eps, int heads, int dim, int vdim) -> Tensor");
+  m.def("qkv_prep(Tensor q, Tensor k, Tensor v, Tensor wq, Tensor wk, float eps, Tensor positions, Tensor freq, Tensor(a!) kc, Tensor(b!) vc, Tensor lengths) -> Tensor");
+  m.def("grouped_decode(Tensor q, Tensor kc, Tensor vc, Tensor lengths, Tensor? keep, Tensor sink, float scale, float softcap) -> Tensor");
+  m.def("token_shift(Tensor h, Tensor mu, int batch, Tensor? keep, Tensor(a!)? prev) -> Tensor");
+  m.def("causal_conv_silu(Tensor x, Tensor w, Tensor bias, int batch, Tensor? keep, Tensor(a!)? prev) -> Tensor");
+  m.def("selective_scan(Tensor x, Tensor dt, Tensor dt_bias, Tensor a_log, Tensor b, Tensor c, Tensor d, Tensor z, int batch, Tensor? keep, Tensor(a!)? state, int chunks=0) -> Tensor");
+  m.def("scan_step(Tensor x, Tensor dt, Tensor w_dt, Tensor dt_bias, Tensor a_log, Tensor b, Tensor c, Tensor d, Tensor z, Tensor? keep, Tensor(a!) state) -> Tensor");
 }
 
 TORCH_LIBRARY_IMPL(oslo_b200, CUDA, m) {
@@ -1159,4 +1505,18 @@ TORCH_LIBRARY_IMPL(oslo_b200, CUDA, m) {
   m.impl("moe_plan", &moe_plan);
   m.impl("moe_grouped", &moe_grouped);
   m.impl("moe_few", &moe_few);
+  m.impl("clamped_glu", &clamped_glu);
+  m.impl("branch_join", &branch_join);
+  m.impl("gated_rms_norm", &gated_rms_norm);
+  m.impl("gemv_stacked", &gemv_stacked);
+  m.impl("decayed_recurrence", &decayed_recurrence);
+  m.impl("bonus_recurrence", &bonus_recurrence);
+  m.impl("decayed_step", &decayed_step);
+  m.impl("bonus_step", &bonus_step);
+  m.impl("qkv_prep", &qkv_prep);
+  m.impl("grouped_decode", &grouped_decode);
+  m.impl("token_shift", &token_shift);
+  m.impl("causal_conv_silu", &causal_conv_silu);
+  m.impl("selective_scan", &selective_scan);
+  m.impl("scan_step", &scan_step);
 }

@@ -98,7 +98,11 @@ __global__ void __launch_bounds__(GV_THREADS) gemv_rows_kernel(const T* __restri
                                                                const T* __restrict__ W, int ldw,
                                                                const T* __restrict__ bias,
                                                                const T* __restrict__ res, int ldr, T* __restrict__ out,
-                                                               int ldo, int N, int m_valid, int gelu_from) {
+                                                               int ldo, int N, int m_valid, int gelu_from,
+                                                               long long sx, long long sw, long long so) {
+  x1 += blockIdx.y * sx;                        // stacked products: one per blockIdx.y
+  W += blockIdx.y * sw;
+  out += blockIdx.y * so;
   __shared__ float red[GV_THREADS / 32][GV_COLS * MR];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int k_begin = threadIdx.x * 8, k_step = GV_THREADS * 8;
@@ -181,13 +185,13 @@ __global__ void rotary_append_kernel(const T* __restrict__ q, const T* __restric
 template <typename T>
 static int gemv_launch(const void* x1, int ld1, int K1, const void* x2, int ld2, int K2, const void* W, int ldw,
                        const void* bias, const void* res, int ldr, void* out, int ldo, int M, int N, int gelu_from,
-                       int num_sms, cudaStream_t st) {
+                       int num_sms, cudaStream_t st, int parts = 1, long long sx = 0, long long sw = 0, long long so = 0) {
   int blocks = N / GV_COLS;                   // one block per column group, at most 8 resident blocks per SM's worth
-  if (blocks > num_sms * 8) blocks = num_sms * 8;
+  if (blocks > num_sms * 8 / parts) blocks = num_sms * 8 / parts;
   if (blocks < 1) blocks = 1;
 #define GV_CASE(MR)                                                                                               \
-  gemv_rows_kernel<T, MR><<<blocks, GV_THREADS, 0, st>>>((const T*)x1, ld1, K1, (const T*)x2, ld2, K2, (const T*)W, ldw, \
-                                                         (const T*)bias, (const T*)res, ldr, (T*)out, ldo, N, M, gelu_from)
+  gemv_rows_kernel<T, MR><<<dim3(blocks, parts), GV_THREADS, 0, st>>>((const T*)x1, ld1, K1, (const T*)x2, ld2, K2, (const T*)W, ldw, \
+                                                         (const T*)bias, (const T*)res, ldr, (T*)out, ldo, N, M, gelu_from, sx, sw, so)
   if (M <= 1) GV_CASE(1);
   else if (M <= 2) GV_CASE(2);
   else GV_CASE(4);
@@ -211,6 +215,20 @@ extern "C" int oslo_gemv_rows(const void* x1, int ld1, int K1, const void* x2, i
     return gemv_launch<__nv_bfloat16>(x1, ld1, K1, x2, ld2, x2 ? K2 : 0, W, ldw, bias, res, ldr, out, ldo, M, N, gelu_from, num_sms, stream);
   if (dtype == OSLO_DT_FP16)
     return gemv_launch<__half>(x1, ld1, K1, x2, ld2, x2 ? K2 : 0, W, ldw, bias, res, ldr, out, ldo, M, N, gelu_from, num_sms, stream);
+  return -2;
+}
+
+extern "C" int oslo_gemv_stacked(const void* x, int ldx, long long sx, const void* W, int ldw, long long sw, void* out, int P, int M,
+                                 int N, int K, int dtype, int num_sms, cudaStream_t stream) {
+  using namespace oslo;
+  if (P <= 0 || M <= 0 || N <= 0) return 0;
+  if (M > 4 || P > 64 || N % GV_COLS || K <= 0 || K % 8 || ldx % 8 || ldw % 8 || sx % 8 || sw % 8) return -1;
+  if ((reinterpret_cast<uintptr_t>(x) & 15) || (reinterpret_cast<uintptr_t>(W) & 15)) return -4;
+  const long long so = static_cast<long long>(M) * N;
+  if (dtype == OSLO_DT_BF16)
+    return gemv_launch<__nv_bfloat16>(x, ldx, K, nullptr, 0, 0, W, ldw, nullptr, nullptr, 0, out, N, M, N, -1, num_sms, stream, P, sx, sw, so);
+  if (dtype == OSLO_DT_FP16)
+    return gemv_launch<__half>(x, ldx, K, nullptr, 0, 0, W, ldw, nullptr, nullptr, 0, out, N, M, N, -1, num_sms, stream, P, sx, sw, so);
   return -2;
 }
 

@@ -54,10 +54,10 @@ struct SinkAttnParams {
   long long q_sb, q_ss, q_sh, k_sb, k_ss, k_sh, v_sb, v_ss, v_sh;
   const uint8_t* keep; long long ld_keep;   // [B, Sk], 0 = padded key
   const void* sink;
-  const void* gate; long long ldg;     // row b * Sq + s
+  const void* gate; long long ldg;     // row b * Sq + s; nullptr: no output gate
   void* out;                           // [B * Sq, H * vdim]
-  int B, H, Sq, Sk, dim, vdim;
-  float scale;
+  int B, H, G, Sq, Sk, dim, vdim;      // query head h reads key / value head h / (H / G)
+  float scale, softcap;                // softcap > 0: scores become softcap * tanh(score / softcap)
 };
 
 constexpr int SA_Q = 16, SA_K = 32;
@@ -76,8 +76,9 @@ __global__ void __launch_bounds__(128) sink_attention_kernel(const SinkAttnParam
   const int tid = threadIdx.x, qi = tid >> 3, l8 = tid & 7;
   const int past = p.Sk - p.Sq;
   const T* q = static_cast<const T*>(p.q) + b * p.q_sb + h * p.q_sh;
-  const T* k = static_cast<const T*>(p.k) + b * p.k_sb + h * p.k_sh;
-  const T* v = static_cast<const T*>(p.v) + b * p.v_sb + h * p.v_sh;
+  const int kv = h / (p.H / p.G);
+  const T* k = static_cast<const T*>(p.k) + b * p.k_sb + kv * p.k_sh;
+  const T* v = static_cast<const T*>(p.v) + b * p.v_sb + kv * p.v_sh;
   for (int e = tid; e < SA_Q * p.dim; e += 128) {
     const int r = e / p.dim, c = e % p.dim;
     qs[r * dp + c] = q0 + r < p.Sq ? Num<T>::to(q[(q0 + r) * p.q_ss + c]) : 0.f;
@@ -104,7 +105,9 @@ __global__ void __launch_bounds__(128) sink_attention_kernel(const SinkAttnParam
       float d = 0.f;
       for (int c = 0; c < p.dim; ++c) d = fmaf(qs[qi * dp + c], ks[kj * dp + c], d);
       const bool vis = pos < k_end && pos <= past + q0 + qi && (p.keep == nullptr || p.keep[b * p.ld_keep + pos]);
-      sc[u] = vis ? d * p.scale : -CUDART_INF_F;
+      d *= p.scale;
+      if (p.softcap > 0.f) d = p.softcap * tanhf(d / p.softcap);
+      sc[u] = vis ? d : -CUDART_INF_F;
       mx = fmaxf(mx, sc[u]);
     }
 #pragma unroll
@@ -131,7 +134,7 @@ __global__ void __launch_bounds__(128) sink_attention_kernel(const SinkAttnParam
   }
   if (q0 + qi < p.Sq) {
     const long long row = static_cast<long long>(b) * p.Sq + q0 + qi;
-    const float fac = sigmoid_f(Num<T>::to(static_cast<const T*>(p.gate)[row * p.ldg + h])) / s;
+    const float fac = (p.gate ? sigmoid_f(Num<T>::to(static_cast<const T*>(p.gate)[row * p.ldg + h])) : 1.0f) / s;
     T* out = static_cast<T*>(p.out) + row * (static_cast<long long>(p.H) * p.vdim) + static_cast<long long>(h) * p.vdim;
     for (int c = l8; c < p.vdim; c += 8) out[c] = Num<T>::from(os[qi * vp + c] * fac);
   }
@@ -781,13 +784,13 @@ extern "C" int oslo_sink_gate(const void* o, long long o_sb, long long o_ss, lon
 extern "C" int oslo_sink_attention(const void* q, long long q_sb, long long q_ss, long long q_sh, const void* k, long long k_sb,
                                    long long k_ss, long long k_sh, const void* v, long long v_sb, long long v_ss,
                                    long long v_sh, const uint8_t* keep, long long ld_keep, const void* sink, const void* gate,
-                                   long long ldg, void* out, int B, int H, int Sq, int Sk, int dim, int vdim, float scale,
-                                   int dtype, cudaStream_t stream) {
+                                   long long ldg, void* out, int B, int H, int G, int Sq, int Sk, int dim, int vdim, float scale,
+                                   float softcap, int dtype, cudaStream_t stream) {
   using namespace oslo;
   if (B <= 0 || H <= 0 || Sq <= 0) return 0;
-  if (Sk < Sq || B > 65535 || H > 65535) return -1;
+  if (Sk < Sq || B > 65535 || H > 65535 || G <= 0 || H % G) return -1;
   SinkAttnParams p{q, k, v, q_sb, q_ss, q_sh, k_sb, k_ss, k_sh, v_sb, v_ss, v_sh, keep, ld_keep, sink, gate, ldg, out,
-                   B, H, Sq, Sk, dim, vdim, scale};
+                   B, H, G, Sq, Sk, dim, vdim, scale, softcap};
   const size_t smem = (static_cast<size_t>(SA_Q + SA_K) * (dim + 1 + vdim + 1) + SA_Q * (SA_K + 1)) * sizeof(float);
   dim3 grid((Sq + SA_Q - 1) / SA_Q, H, B);
   OSLO_DISPATCH_T(dtype, {

@@ -1,8 +1,15 @@
-// Gated linear recurrence (HGRN2 form), state in 32-bit floats:
-//   k = (1 - lower) * sigmoid(-(f + f_bias)),  forget gate = 1 - k  (= lower + (1 - lower) * sigmoid(f + f_bias))
+// Linear recurrences with a matrix state S (key channels x value channels) per head, in 32-bit floats. Three rules:
+//
+// RULE_GATED (HGRN2 form): k = (1 - lower) * sigmoid(-(f + f_bias)),  forget gate = 1 - k  (= lower + (1 - lower) * sigmoid(f + f_bias))
 //   S_t = S_{t-1} + k_t (v_t - S_{t-1})   per row of the state (a key channel) and column (a value channel)
 //   o_t[j] = sum_i silu(q_t)[i] S_t[i, j]
-// `k` is computed from the negated logit, so a gate close to 1 does not lose what it writes to cancellation.
+//   `k` is computed from the negated logit, so a gate close to 1 does not lose what it writes to cancellation.
+// RULE_DECAY: q, k, v are silu of what is given, S_t = d S_{t-1} + k_t v_t^T with one constant d per head, o_t = S_t^T q_t.
+//   Within a period of tokens the state is kept relative to the period's decay: with P_t the product of d over the tokens
+//   after the period's first, k_t / P_t is written and P_t q_t reads, which leaves two FMAs per state element and token; the
+//   state is multiplied once per period. The period is short enough for 1 / P_t to stay far from overflow, whatever d is.
+// RULE_BONUS (RWKV form): decay w_t = exp(-exp(z_t + w0)) per key channel, o_t = S_{t-1}^T r_t + (r_t . (u k_t)) v_t, then
+//   S_t = diag(w_t) S_{t-1} + k_t v_t^T.
 //
 // Prefill (recurrence_kernel): a thread keeps a 16 x 4 tile of S in registers - rows in pairs, so that every update is a
 // packed two-float FMA - and G lanes share a column group; per token it reads 16 + 16 + 4 floats from shared memory,
@@ -25,6 +32,8 @@ namespace cg = cooperative_groups;
 
 namespace oslo {
 
+enum { RULE_GATED = 0, RULE_DECAY = 1, RULE_BONUS = 2 };
+
 typedef unsigned long long f32x2;
 __device__ __forceinline__ f32x2 pack_f2(float lo, float hi) {
   f32x2 r;
@@ -40,6 +49,12 @@ __device__ __forceinline__ f32x2 fma_f2(f32x2 a, f32x2 b, f32x2 c) {
   return r;
 }
 
+__device__ __forceinline__ f32x2 mul_f2(f32x2 a, f32x2 b) {
+  f32x2 r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+
 // 32-bit models get the accurate exponential; logits that come from 16-bit projections the hardware one (2^-21)
 template <typename T> __device__ __forceinline__ float sigmoid_t(float z) {
   return sizeof(T) == 4 ? sigmoid_f(z) : __fdividef(1.0f, 1.0f + __expf(-z));
@@ -48,40 +63,52 @@ template <typename T> __device__ __forceinline__ float write_gate(float logit, f
   return (1.0f - lower) * sigmoid_t<T>(-logit);
 }
 template <typename T> __device__ __forceinline__ float silu_t(float z) { return z * sigmoid_t<T>(z); }
+template <typename T> __device__ __forceinline__ float channel_decay(float logit) {
+  return sizeof(T) == 4 ? expf(-expf(logit)) : __expf(-__expf(logit));
+}
 
 struct RecParams {
-  const void *q, *f, *v;             // row (b * S + t) of each has the stride ldq / ldf / ldv
+  const void *q, *f, *v;             // row (b * S + t) of each has the stride ldq / ldf / ldv; f: gate logits, or the keys
   long long ldq, ldf, ldv;
-  const void *f_bias, *lower;        // [H * dim]
+  const void *f_bias, *lower;        // [H * dim]; RULE_BONUS: w0 and u
+  const float* z; long long ldz;     // RULE_BONUS: decay logits [B * S, H * dim]
+  const float* head_decay;           // RULE_DECAY: [H]
   const uint8_t* keep; long long ld_keep;   // [B, S], 0 = padding, or nullptr
   const float* s_in;                 // initial states, or nullptr (zero)
   float* s_out;                      // final states, or nullptr
-  float* decay;                      // STATE_ONLY: product of the forget gates of the chunk
+  float* decay;                      // STATE_ONLY: product of the forget gates or decays of the chunk
   float* out;                        // [B, S, H, vdim]
   int B, S, H, dim, vdim;
   int chunk, nchunks;                // tokens per chunk; chunks of this launch per batch row
   float* s_end;                      // last chunk only: final states [B, H, dim, vdim], or nullptr
   long long s_batch, s_chunk;        // element strides of s_in / s_out over batch rows and chunks
   int dim_pad;                       // dim rounded up so that every row of a raw stage starts at a 16-byte boundary
-  int vec16;                         // q, f, v rows and head slices start at 16-byte boundaries
+  int vec16;                         // q, f, v (and z) rows and head slices start at 16-byte boundaries
 };
 
 constexpr int REC_TB = 16;    // tokens staged at a time
 constexpr int REC_COLS = 4;   // state columns per thread
 constexpr int REC_ROWS = 16;      // state rows per thread
 
+constexpr float REC_MIN_PERIOD = 1e-15f;   // RULE_DECAY: the smallest product of decays within a period
+
 // G lanes per column group. STATE_ONLY: no outputs, start from zero, also the chunk's total decay per row
-template <typename T, int G, bool STATE_ONLY>
+template <typename T, int G, bool STATE_ONLY, int RULE>
 __global__ void __launch_bounds__(256, 2) recurrence_kernel(const RecParams p) {
   constexpr int DP = REC_ROWS * G;
   constexpr int CONV = DP >= 256 ? 1 : 256 / DP;
+  constexpr int PARTS = DP > 32 ? DP / 32 : 1;               // RULE_BONUS: partial sums of r . (u k) per token
   constexpr int WIDTH = G >= REC_COLS ? 1 : REC_COLS / G;    // output columns a lane holds after the reduction
   extern __shared__ float4 rec_smem[];
   const int nt = blockDim.x;
   const int cols = nt / G * REC_COLS;
   float* ks = reinterpret_cast<float*>(rec_smem);
   float* qs = ks + REC_TB * DP;
-  float* vs = qs + (STATE_ONLY ? 0 : REC_TB * DP);
+  float* ws = qs + (STATE_ONLY ? 0 : REC_TB * DP);            // RULE_BONUS: decays
+  float* vs = ws + (RULE == RULE_BONUS ? REC_TB * DP : 0);
+  __shared__ float bonus_s[RULE == RULE_BONUS && !STATE_ONLY ? REC_TB * PARTS : 1];
+  __shared__ float read_s[RULE == RULE_DECAY ? REC_TB : 1], write_s[RULE == RULE_DECAY ? REC_TB : 1];   // P_t, 1 / P_t
+  __shared__ float period_s[RULE == RULE_DECAY ? 2 * REC_TB : 1];   // [stage parity][period]: d^(real tokens - 1), negative: none
   const int tid = threadIdx.x, g = tid % G, cgp = tid / G;
   const int h = blockIdx.y;
   const int b = blockIdx.z / p.nchunks, ch = blockIdx.z % p.nchunks;
@@ -114,6 +141,18 @@ __global__ void __launch_bounds__(256, 2) recurrence_kernel(const RecParams p) {
 #pragma unroll
   for (int i = 0; i < REC_ROWS; ++i) dec[i] = 1.f;
   const f32x2 minus1 = pack_f2(-1.f, -1.f);
+  const float hd = RULE == RULE_DECAY ? p.head_decay[h] : 1.f;
+  int period = REC_TB;                                   // RULE_DECAY: tokens between two multiplications of the state
+  if (RULE == RULE_DECAY) {
+    float least = hd;
+    for (int i = 0; i < 4; ++i) least *= least;          // d^16
+    while (period > 1 && !(least >= REC_MIN_PERIOD)) {
+      period /= 2;
+      least = 1.f;
+      for (int i = 0; i < period; ++i) least *= hd;
+    }
+  }
+  float pending = 1.f;                                   // what the state still has to be multiplied by
   // where this lane's share of an output row goes, and how many of its WIDTH columns exist (0: another lane writes them)
   int first = 0;
 #pragma unroll
@@ -126,10 +165,26 @@ __global__ void __launch_bounds__(256, 2) recurrence_kernel(const RecParams p) {
 
   // raw [REC_TB][raw_ld] stages in the storage type, fetched one step ahead: q (unless STATE_ONLY), f, v slice
   const int f_at = STATE_ONLY ? 0 : p.dim_pad, v_at = f_at + p.dim_pad, raw_ld = v_at + cols;
-  T* raw = reinterpret_cast<T*>(vs + REC_TB * cols);
+  float* zraw = vs + REC_TB * cols;                      // RULE_BONUS: [2][REC_TB][dim_pad]
+  T* raw = reinterpret_cast<T*>(zraw + (RULE == RULE_BONUS ? 2 * REC_TB * p.dim_pad : 0));
+  const float* z = RULE == RULE_BONUS ? p.z + static_cast<long long>(b) * p.S * p.ldz + static_cast<long long>(h) * p.dim : nullptr;
   auto fetch = [&](int t0, int buf) {
     T* dst = raw + static_cast<size_t>(buf) * REC_TB * raw_ld;
     const int n = min(REC_TB, t_end - t0);
+    if (RULE == RULE_BONUS) {
+      float* zd = zraw + static_cast<size_t>(buf) * REC_TB * p.dim_pad;
+      if (p.vec16) {
+        const int per = p.dim / 4;
+        for (int e = tid; e < n * per; e += nt) {
+          const int t = e / per, c = (e - t * per) * 4;
+          const uint32_t d32 = static_cast<uint32_t>(__cvta_generic_to_shared(zd + t * p.dim_pad + c));
+          asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(d32), "l"(z + (t0 + t) * p.ldz + c) : "memory");
+        }
+      } else {
+        for (int t = 0; t < n; ++t)
+          for (int i = tid; i < p.dim; i += nt) zd[t * p.dim_pad + i] = z[(t0 + t) * p.ldz + i];
+      }
+    }
     if (p.vec16) {
       constexpr int V = 16 / sizeof(T);
       const int per_dim = p.dim / V, per_v = min(cols, p.vdim - col0) / V;
@@ -170,25 +225,85 @@ __global__ void __launch_bounds__(256, 2) recurrence_kernel(const RecParams p) {
     } else {
       asm volatile("cp.async.wait_group 0;" ::: "memory");
     }
+    if (RULE == RULE_DECAY) {                            // read before the second barrier, periods until the stage after next
+      for (int s0 = tid * period; s0 < n; s0 += nt * period) {
+        float pr = 1.f, ip = 1.f;
+        int real = 0;
+        const int s1 = min(n, s0 + period);
+        for (int t = s0; t < s1; ++t) {
+          if (p.keep == nullptr || p.keep[b * p.ld_keep + t0 + t]) {
+            if (real++) { pr *= hd; ip = 1.f / pr; }
+          }
+          read_s[t] = pr;
+          write_s[t] = ip;
+        }
+        period_s[(it & 1) * REC_TB + s0 / period] = real ? pr : -1.f;
+      }
+    }
     __syncthreads();
     const T* src = raw + static_cast<size_t>(it & 1) * REC_TB * raw_ld;
     for (int e = tid; e < DP * CONV; e += nt) {          // CONV threads share a channel's tokens
       const int i = e % DP;
       const bool real = i < p.dim;
-      const float bias = real ? Num<T>::to(fb[i]) : 0.f, low = real ? Num<T>::to(lw[i]) : 1.f;
+      if constexpr (RULE == RULE_GATED) {
+        const float bias = real ? Num<T>::to(fb[i]) : 0.f, low = real ? Num<T>::to(lw[i]) : 1.f;
 #pragma unroll 4
-      for (int t = e / DP; t < n; t += CONV) {
-        const bool on = real && (p.keep == nullptr || p.keep[b * p.ld_keep + t0 + t]);
-        ks[t * DP + i] = on ? write_gate<T>(Num<T>::to(src[t * raw_ld + f_at + i]) + bias, low) : 0.f;
-        if (!STATE_ONLY) qs[t * DP + i] = on ? silu_t<T>(Num<T>::to(src[t * raw_ld + i])) : 0.f;
+        for (int t = e / DP; t < n; t += CONV) {
+          const bool on = real && (p.keep == nullptr || p.keep[b * p.ld_keep + t0 + t]);
+          ks[t * DP + i] = on ? write_gate<T>(Num<T>::to(src[t * raw_ld + f_at + i]) + bias, low) : 0.f;
+          if (!STATE_ONLY) qs[t * DP + i] = on ? silu_t<T>(Num<T>::to(src[t * raw_ld + i])) : 0.f;
+        }
+      } else if constexpr (RULE == RULE_DECAY) {
+#pragma unroll 4
+        for (int t = e / DP; t < n; t += CONV) {
+          const bool on = real && (p.keep == nullptr || p.keep[b * p.ld_keep + t0 + t]);
+          ks[t * DP + i] = on ? silu_t<T>(Num<T>::to(src[t * raw_ld + f_at + i])) * write_s[t] : 0.f;
+          if (!STATE_ONLY) qs[t * DP + i] = on ? silu_t<T>(Num<T>::to(src[t * raw_ld + i])) * read_s[t] : 0.f;
+        }
+      } else {
+        const float w0 = real ? Num<T>::to(fb[i]) : 0.f, u = real ? Num<T>::to(lw[i]) : 0.f;
+        const float* zs = zraw + static_cast<size_t>(it & 1) * REC_TB * p.dim_pad;
+        // a warp's threads are at one token (or, with 16 channels, at two); the loop below makes as many turns in each of them
+        for (int tt = 0; tt < (REC_TB + CONV - 1) / CONV; ++tt) {
+          const int t = e / DP + tt * CONV;
+          const bool on = t < n && real && (p.keep == nullptr || p.keep[b * p.ld_keep + t0 + t]);
+          const float k = on ? Num<T>::to(src[t * raw_ld + f_at + i]) : 0.f;
+          if (t < n) {
+            ks[t * DP + i] = k;
+            ws[t * DP + i] = on ? channel_decay<T>(zs[t * p.dim_pad + i] + w0) : 1.f;
+          }
+          if (!STATE_ONLY) {
+            const float r = on ? Num<T>::to(src[t * raw_ld + i]) : 0.f;
+            if (t < n) qs[t * DP + i] = r;
+            float a = r * u * k;
+            constexpr int RED = DP < 32 ? DP : 32;
+#pragma unroll
+            for (int off = RED / 2; off > 0; off >>= 1) a += __shfl_xor_sync(0xffffffffu, a, off);
+            if (t < n && i % RED == 0) bonus_s[t * PARTS + i / RED] = a;
+          }
+        }
       }
     }
     for (int e = tid; e < n * cols; e += nt) {
       const int t = e / cols, c = e - t * cols;
-      vs[e] = col0 + c < p.vdim ? Num<T>::to(src[t * raw_ld + v_at + c]) : 0.f;
+      const float v = col0 + c < p.vdim ? Num<T>::to(src[t * raw_ld + v_at + c]) : 0.f;
+      vs[e] = RULE == RULE_DECAY ? silu_t<T>(v) : v;
     }
     __syncthreads();
     for (int t = 0; t < n; ++t) {
+      if (RULE == RULE_DECAY && (t & (period - 1)) == 0) {    // a period begins: its first real token's decay and what is pending
+        const float in_period = period_s[(it & 1) * REC_TB + t / period];
+        if (in_period >= 0.f) {
+          const float f = hd * pending;
+          const f32x2 f2 = pack_f2(f, f);
+#pragma unroll
+          for (int rp = 0; rp < REC_ROWS / 2; ++rp)
+#pragma unroll
+            for (int c = 0; c < REC_COLS; ++c) s[rp][c] = mul_f2(s[rp][c], f2);
+          pending = in_period;
+          if (STATE_ONLY) dec[0] *= hd * in_period;
+        }
+      }
       f32x2 v2[REC_COLS];
       {
         const float4 a = *reinterpret_cast<const float4*>(vs + t * cols + cgp * REC_COLS);
@@ -197,6 +312,11 @@ __global__ void __launch_bounds__(256, 2) recurrence_kernel(const RecParams p) {
       f32x2 o2[REC_COLS];
 #pragma unroll
       for (int c = 0; c < REC_COLS; ++c) o2[c] = 0ull;
+      if (RULE == RULE_BONUS && !STATE_ONLY) {               // this lane's share of (r . (u k)) v
+        const f32x2 a2 = g < PARTS ? pack_f2(bonus_s[t * PARTS + g], 0.f) : 0ull;
+#pragma unroll
+        for (int c = 0; c < REC_COLS; ++c) o2[c] = mul_f2(a2, v2[c]);
+      }
 #pragma unroll
       for (int kk = 0; kk < REC_ROWS / 4; ++kk) {
         const float4 k4 = *reinterpret_cast<const float4*>(ks + t * DP + 4 * (g + G * kk));
@@ -206,18 +326,33 @@ __global__ void __launch_bounds__(256, 2) recurrence_kernel(const RecParams p) {
           const float4 q4 = *reinterpret_cast<const float4*>(qs + t * DP + 4 * (g + G * kk));
           q2[0] = pack_f2(q4.x, q4.y);
           q2[1] = pack_f2(q4.z, q4.w);
-        } else {
+        } else if (RULE == RULE_GATED) {
           dec[4 * kk] *= 1.f - k4.x; dec[4 * kk + 1] *= 1.f - k4.y;
           dec[4 * kk + 2] *= 1.f - k4.z; dec[4 * kk + 3] *= 1.f - k4.w;
+        }
+        f32x2 w2[2] = {0ull, 0ull};
+        if (RULE == RULE_BONUS) {
+          const float4 w4 = *reinterpret_cast<const float4*>(ws + t * DP + 4 * (g + G * kk));
+          w2[0] = pack_f2(w4.x, w4.y);
+          w2[1] = pack_f2(w4.z, w4.w);
+          if (STATE_ONLY) { dec[4 * kk] *= w4.x; dec[4 * kk + 1] *= w4.y; dec[4 * kk + 2] *= w4.z; dec[4 * kk + 3] *= w4.w; }
         }
 #pragma unroll
         for (int u = 0; u < 2; ++u) {
 #pragma unroll
           for (int c = 0; c < REC_COLS; ++c) {
             f32x2& st = s[2 * kk + u][c];
-            const f32x2 d = fma_f2(st, minus1, v2[c]);
-            st = fma_f2(k2[u], d, st);
-            if (!STATE_ONLY) o2[c] = fma_f2(q2[u], st, o2[c]);
+            if (RULE == RULE_GATED) {
+              const f32x2 d = fma_f2(st, minus1, v2[c]);
+              st = fma_f2(k2[u], d, st);
+              if (!STATE_ONLY) o2[c] = fma_f2(q2[u], st, o2[c]);
+            } else if (RULE == RULE_DECAY) {
+              st = fma_f2(k2[u], v2[c], st);
+              if (!STATE_ONLY) o2[c] = fma_f2(q2[u], st, o2[c]);
+            } else {
+              if (!STATE_ONLY) o2[c] = fma_f2(q2[u], st, o2[c]);
+              st = fma_f2(w2[u], st, mul_f2(k2[u], v2[c]));
+            }
           }
         }
       }
@@ -256,6 +391,13 @@ __global__ void __launch_bounds__(256, 2) recurrence_kernel(const RecParams p) {
       }
     }
   }
+  if (RULE == RULE_DECAY) {
+    const f32x2 f2 = pack_f2(pending, pending);
+#pragma unroll
+    for (int rp = 0; rp < REC_ROWS / 2; ++rp)
+#pragma unroll
+      for (int c = 0; c < REC_COLS; ++c) s[rp][c] = mul_f2(s[rp][c], f2);
+  }
   auto store_state = [&](float* so) {
 #pragma unroll
     for (int rp = 0; rp < REC_ROWS / 2; ++rp) {
@@ -284,7 +426,7 @@ __global__ void __launch_bounds__(256, 2) recurrence_kernel(const RecParams p) {
 #pragma unroll
       for (int u = 0; u < 4; ++u) {
         const int i = 4 * (g + G * kk) + u;
-        if (i < p.dim) d[i] = dec[4 * kk + u];
+        if (i < p.dim) d[i] = RULE == RULE_DECAY ? dec[0] : dec[4 * kk + u];
       }
   }
 }
@@ -313,20 +455,26 @@ __global__ void __launch_bounds__(256) recurrence_chunk_scan_kernel(float* __res
 struct StepParams {
   const void *q, *f, *v;
   long long ldq, ldf, ldv;
-  const void *f_bias, *lower, *norm_w;
+  const void *f_bias, *lower, *norm_w;      // RULE_BONUS: w0, u, and a norm weight per channel [H * vdim]
+  const float* head_decay;                  // RULE_DECAY
+  const void* t; long long ldt;             // RULE_BONUS: W_w1 mix [B, rank]
+  const void* w2; int rank;                 // ... W_w2 [H * dim, rank]
+  const void* gate; long long ldg;          // ... gate logits [B, H * vdim]
   const uint8_t* keep; long long ld_keep;   // [B, 1], 0 = padding, or nullptr
   float* state;      // [B, H, dim, vdim]
-  void* out;         // [B, H * vdim]
+  void* out;         // [B, H * vdim]; RULE_DECAY: fp32, not normed
   int H, dim, vdim, cols;   // cols: value channels per CTA
   float eps;
 };
 
-template <typename T, int VEC>
+template <typename T, int VEC, int RULE>
 __global__ void __launch_bounds__(256) recurrence_step_kernel(const StepParams p) {
   extern __shared__ float step_smem[];
   float* ks = step_smem;            // [dim]
   float* qs = ks + p.dim;           // [dim]
-  float* part = qs + p.dim;         // [ty][cols]
+  float* ws = qs + p.dim;           // [dim], RULE_BONUS
+  float* ts = ws + (RULE == RULE_BONUS ? p.dim : 0);   // [rank], RULE_BONUS
+  float* part = ts + (RULE == RULE_BONUS ? p.rank : 0);   // [ty][cols]
   __shared__ float red[32];
   __shared__ float slice_ss;
   cg::cluster_group cluster = cg::this_cluster();
@@ -337,12 +485,40 @@ __global__ void __launch_bounds__(256) recurrence_step_kernel(const StepParams p
   const T* f = static_cast<const T*>(p.f) + b * p.ldf + static_cast<long long>(h) * p.dim;
   const T* v = static_cast<const T*>(p.v) + b * p.ldv + static_cast<long long>(h) * p.vdim;
   const bool on = p.keep == nullptr || p.keep[b * p.ld_keep];
-  for (int i = threadIdx.x; i < p.dim; i += blockDim.x) {
-    ks[i] = on ? write_gate<T>(Num<T>::to(f[i]) + Num<T>::to(static_cast<const T*>(p.f_bias)[h * p.dim + i]),
-                            Num<T>::to(static_cast<const T*>(p.lower)[h * p.dim + i])) : 0.f;
-    qs[i] = on ? silu_t<T>(Num<T>::to(q[i])) : 0.f;
+  float bonus = 0.f;
+  if constexpr (RULE == RULE_BONUS) {
+    const T* t = static_cast<const T*>(p.t) + b * p.ldt;
+    for (int i = threadIdx.x; i < p.rank; i += blockDim.x) ts[i] = Num<T>::to(Num<T>::from(tanhf(Num<T>::to(t[i]))));
+    __syncthreads();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const T* w2 = static_cast<const T*>(p.w2) + static_cast<long long>(h) * p.dim * p.rank;
+    const T* w0 = static_cast<const T*>(p.f_bias) + h * p.dim;
+    const bool vec = p.rank % 4 == 0;
+#pragma unroll 2
+    for (int i = warp; i < p.dim; i += 8) {
+      const T* row = w2 + static_cast<long long>(i) * p.rank;
+      const float z = vec ? warp_dot<T, 4>(row, ts, p.rank, lane) : warp_dot<T, 1>(row, ts, p.rank, lane);
+      if (lane == 0) ws[i] = on ? channel_decay<T>(z + Num<T>::to(w0[i])) : 1.f;
+    }
+    for (int i = threadIdx.x; i < p.dim; i += blockDim.x) {
+      ks[i] = on ? Num<T>::to(f[i]) : 0.f;
+      qs[i] = on ? Num<T>::to(q[i]) : 0.f;
+      bonus = fmaf(qs[i] * Num<T>::to(static_cast<const T*>(p.lower)[h * p.dim + i]), ks[i], bonus);
+    }
+    bonus = block_sum(bonus, red);
+  } else {
+    for (int i = threadIdx.x; i < p.dim; i += blockDim.x) {
+      if (RULE == RULE_GATED) {
+        ks[i] = on ? write_gate<T>(Num<T>::to(f[i]) + Num<T>::to(static_cast<const T*>(p.f_bias)[h * p.dim + i]),
+                                Num<T>::to(static_cast<const T*>(p.lower)[h * p.dim + i])) : 0.f;
+      } else {
+        ks[i] = on ? silu_t<T>(Num<T>::to(f[i])) : 0.f;
+      }
+      qs[i] = on ? silu_t<T>(Num<T>::to(q[i])) : 0.f;
+    }
   }
   __syncthreads();
+  const float hd = RULE == RULE_DECAY && on ? p.head_decay[h] : 1.f;
   const int tx_n = p.cols / VEC;                       // the launcher keeps tx_n <= 256
   const int ty_n = blockDim.x / tx_n;
   const int tx = threadIdx.x % tx_n, ty = threadIdx.x / tx_n;
@@ -351,17 +527,29 @@ __global__ void __launch_bounds__(256) recurrence_step_kernel(const StepParams p
     const int c = tx * VEC;
     float o[VEC], vv[VEC];
 #pragma unroll
-    for (int i = 0; i < VEC; ++i) { o[i] = 0.f; vv[i] = c + i < cols ? Num<T>::to(v[c0 + c + i]) : 0.f; }
+    for (int i = 0; i < VEC; ++i) {
+      vv[i] = c + i < cols ? Num<T>::to(v[c0 + c + i]) : 0.f;
+      if (RULE == RULE_DECAY) vv[i] = silu_t<T>(vv[i]);
+      o[i] = RULE == RULE_BONUS && ty == 0 ? bonus * vv[i] : 0.f;
+    }
     if (c < cols) {                                    // VEC > 1: the launcher guarantees vdim % VEC == 0
 #pragma unroll 4
       for (int i = ty; i < p.dim; i += ty_n) {
         float s[VEC];
         load_vec<float, VEC>(st + static_cast<long long>(i) * p.vdim + c, s);
-        const float k = ks[i], qq = qs[i];
+        const float k = ks[i], qq = qs[i], w = RULE == RULE_BONUS ? ws[i] : hd;
 #pragma unroll
         for (int j = 0; j < VEC; ++j) {
-          s[j] = fmaf(k, vv[j] - s[j], s[j]);
-          o[j] = fmaf(qq, s[j], o[j]);
+          if (RULE == RULE_GATED) {
+            s[j] = fmaf(k, vv[j] - s[j], s[j]);
+            o[j] = fmaf(qq, s[j], o[j]);
+          } else if (RULE == RULE_DECAY) {
+            s[j] = fmaf(w, s[j], k * vv[j]);
+            o[j] = fmaf(qq, s[j], o[j]);
+          } else {
+            o[j] = fmaf(qq, s[j], o[j]);
+            s[j] = fmaf(w, s[j], k * vv[j]);
+          }
         }
         store_vec<float, VEC>(st + static_cast<long long>(i) * p.vdim + c, s);
       }
@@ -376,7 +564,9 @@ __global__ void __launch_bounds__(256) recurrence_step_kernel(const StepParams p
     for (int y = 0; y < ty_n; ++y) o += part[y * p.cols + c];
     part[c] = o;                                       // row 0, column c: only this thread reads or writes it now
     ss = fmaf(o, o, ss);
+    if (RULE == RULE_DECAY) static_cast<float*>(p.out)[(static_cast<long long>(b) * p.H + h) * p.vdim + c0 + c] = o;
   }
+  if (RULE == RULE_DECAY) return;                      // the norm runs over all heads
   ss = block_sum(ss, red);
   if (threadIdx.x == 0) slice_ss = ss;
   cluster.sync();
@@ -385,8 +575,13 @@ __global__ void __launch_bounds__(256) recurrence_step_kernel(const StepParams p
   cluster.sync();                                      // no CTA leaves while another still reads its shared memory
   const float rn = 1.0f / sqrtf(tot / p.vdim + p.eps);
   T* out = static_cast<T*>(p.out) + (static_cast<long long>(b) * p.H + h) * p.vdim + c0;
-  const T* nw = static_cast<const T*>(p.norm_w) + c0;
-  for (int c = threadIdx.x; c < cols; c += blockDim.x) out[c] = Num<T>::from(part[c] * rn * Num<T>::to(nw[c]));
+  const T* nw = static_cast<const T*>(p.norm_w) + (RULE == RULE_BONUS ? static_cast<long long>(h) * p.vdim : 0) + c0;
+  const T* gate = RULE == RULE_BONUS ? static_cast<const T*>(p.gate) + b * p.ldg + static_cast<long long>(h) * p.vdim + c0 : nullptr;
+  for (int c = threadIdx.x; c < cols; c += blockDim.x) {
+    float y = part[c] * rn * Num<T>::to(nw[c]);
+    if (RULE == RULE_BONUS) y *= silu_t<T>(Num<T>::to(gate[c]));
+    out[c] = Num<T>::from(y);
+  }
 }
 
 // threads of a block: the column groups of a head, at most 256
@@ -395,29 +590,38 @@ static int rec_threads(int g, int vdim) {
   return std::min(256, (groups * g + 31) / 32 * 32);
 }
 
-template <typename T, int G, bool STATE_ONLY>
+template <typename T, int G, bool STATE_ONLY, int RULE>
 static int rec_launch(const RecParams& p, cudaStream_t st) {
   const int nt = rec_threads(G, p.vdim), cols = nt / G * REC_COLS;
-  const size_t smem = static_cast<size_t>(REC_TB) * (((STATE_ONLY ? 1 : 2) * REC_ROWS * G + cols) * sizeof(float) +
+  const int rows = (STATE_ONLY ? 1 : 2) + (RULE == RULE_BONUS ? 1 : 0);
+  const size_t smem = static_cast<size_t>(REC_TB) * ((rows * REC_ROWS * G + cols + (RULE == RULE_BONUS ? 2 * p.dim_pad : 0)) * sizeof(float) +
                                                      2 * ((STATE_ONLY ? 1 : 2) * p.dim_pad + cols) * sizeof(T));
-  if (smem > 48 * 1024) {
-    cudaError_t e = cudaFuncSetAttribute(recurrence_kernel<T, G, STATE_ONLY>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+  if (smem > 44 * 1024) {      // static arrays come on top
+    cudaError_t e = cudaFuncSetAttribute(recurrence_kernel<T, G, STATE_ONLY, RULE>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          static_cast<int>(smem));
     if (e != cudaSuccess) return static_cast<int>(e);
   }
   dim3 grid((p.vdim + cols - 1) / cols, p.H, p.B * p.nchunks);
-  recurrence_kernel<T, G, STATE_ONLY><<<grid, nt, smem, st>>>(p);
+  recurrence_kernel<T, G, STATE_ONLY, RULE><<<grid, nt, smem, st>>>(p);
   return static_cast<int>(cudaGetLastError());
 }
-template <typename T, bool STATE_ONLY>
-static int rec_dispatch(const RecParams& p, cudaStream_t st) {
-  if (p.dim <= 16) return rec_launch<T, 1, STATE_ONLY>(p, st);
-  if (p.dim <= 32) return rec_launch<T, 2, STATE_ONLY>(p, st);
-  if (p.dim <= 64) return rec_launch<T, 4, STATE_ONLY>(p, st);
-  if (p.dim <= 128) return rec_launch<T, 8, STATE_ONLY>(p, st);
-  if (p.dim <= 256) return rec_launch<T, 16, STATE_ONLY>(p, st);
-  if (p.dim <= 512) return rec_launch<T, 32, STATE_ONLY>(p, st);
+template <typename T, bool STATE_ONLY, int RULE>
+static int rec_dispatch_rule(const RecParams& p, cudaStream_t st) {
+  if (p.dim <= 16) return rec_launch<T, 1, STATE_ONLY, RULE>(p, st);
+  if (p.dim <= 32) return rec_launch<T, 2, STATE_ONLY, RULE>(p, st);
+  if (p.dim <= 64) return rec_launch<T, 4, STATE_ONLY, RULE>(p, st);
+  if (p.dim <= 128) return rec_launch<T, 8, STATE_ONLY, RULE>(p, st);
+  if (p.dim <= 256) return rec_launch<T, 16, STATE_ONLY, RULE>(p, st);
+  if constexpr (RULE != RULE_BONUS)                     // the bonus rule's stages of 512 channels exceed the shared memory
+    if (p.dim <= 512) return rec_launch<T, 32, STATE_ONLY, RULE>(p, st);
   return -3;
+}
+template <typename T, bool STATE_ONLY>
+static int rec_dispatch(const RecParams& p, int rule, cudaStream_t st) {
+  if (rule == RULE_GATED) return rec_dispatch_rule<T, STATE_ONLY, RULE_GATED>(p, st);
+  if (rule == RULE_DECAY) return rec_dispatch_rule<T, STATE_ONLY, RULE_DECAY>(p, st);
+  if (rule == RULE_BONUS) return rec_dispatch_rule<T, STATE_ONLY, RULE_BONUS>(p, st);
+  return -1;
 }
 
 }  // namespace oslo
@@ -446,26 +650,29 @@ extern "C" int oslo_recurrence_chunks(int B, int S, int H, int dim, int vdim, in
   return best;
 }
 
-extern "C" int oslo_recurrence(const void* q, long long ldq, const void* f, long long ldf, const void* v, long long ldv,
-                               const void* f_bias, const void* lower, const uint8_t* keep, long long ld_keep, float* state,
-                               float* out, float* ws, float* decay, int nchunks, int B, int S, int H, int dim, int vdim,
-                               int dtype, cudaStream_t stream) {
+// f_bias / lower: the gate bias and lower bound (RULE_GATED), or w0 and u (RULE_BONUS); z: decay logits (RULE_BONUS);
+// head_decay: RULE_DECAY
+extern "C" int oslo_recurrence(int rule, const void* q, long long ldq, const void* f, long long ldf, const void* v, long long ldv,
+                               const void* f_bias, const void* lower, const float* z, long long ldz, const float* head_decay,
+                               const uint8_t* keep, long long ld_keep, float* state, float* out, float* ws, float* decay, int nchunks,
+                               int B, int S, int H, int dim, int vdim, int dtype, cudaStream_t stream) {
   using namespace oslo;
   if (B <= 0 || S <= 0 || H <= 0) return 0;
   if (dim <= 0 || vdim <= 0 || dim > 512 || H > 65535 || nchunks < 1 || static_cast<long long>(B) * nchunks > 65535) return -1;
   RecParams p{};
   p.q = q; p.f = f; p.v = v; p.ldq = ldq; p.ldf = ldf; p.ldv = ldv; p.f_bias = f_bias; p.lower = lower;
+  p.z = z; p.ldz = ldz; p.head_decay = head_decay;
   p.keep = keep; p.ld_keep = ld_keep; p.out = out;
   p.B = B; p.S = S; p.H = H; p.dim = dim; p.vdim = vdim;
   const long long per = static_cast<long long>(H) * dim * vdim;
   const int te = dtype == OSLO_DT_FP32 ? 4 : 2, v16 = 16 / te;
   p.dim_pad = (dim + 7) / 8 * 8;
   p.vec16 = dim % v16 == 0 && vdim % v16 == 0 && ldq % v16 == 0 && ldf % v16 == 0 && ldv % v16 == 0 && aligned_to(q, 16) &&
-            aligned_to(f, 16) && aligned_to(v, 16);
+            aligned_to(f, 16) && aligned_to(v, 16) && (rule != RULE_BONUS || (ldz % 4 == 0 && aligned_to(z, 16)));
   int rc = 0;
   if (nchunks == 1) {
     p.chunk = S; p.nchunks = 1; p.s_in = state; p.s_out = state; p.s_batch = per; p.s_chunk = 0;
-    OSLO_DISPATCH_T(dtype, { rc = rec_dispatch<T, false>(p, stream); });
+    OSLO_DISPATCH_T(dtype, { rc = rec_dispatch<T, false>(p, rule, stream); });
     return rc;
   }
   if (ws == nullptr || decay == nullptr) return -1;
@@ -474,7 +681,7 @@ extern "C" int oslo_recurrence(const void* q, long long ldq, const void* f, long
   p.s_batch = per * nchunks; p.s_chunk = per;
   p.s_in = nullptr; p.s_out = ws; p.decay = decay;
   p.nchunks = nchunks - 1;             // nobody starts from the last chunk's state
-  OSLO_DISPATCH_T(dtype, { rc = rec_dispatch<T, true>(p, stream); });
+  OSLO_DISPATCH_T(dtype, { rc = rec_dispatch<T, true>(p, rule, stream); });
   if (rc) return rc;
   recurrence_chunk_scan_kernel<<<dim3(static_cast<unsigned>((per + 255) / 256), B), 256, 0, stream>>>(ws, decay, state, nchunks, H,
                                                                                                      dim, vdim);
@@ -482,25 +689,24 @@ extern "C" int oslo_recurrence(const void* q, long long ldq, const void* f, long
   if (rc) return rc;
   p.nchunks = nchunks;
   p.s_in = ws; p.s_out = nullptr; p.s_end = state;
-  OSLO_DISPATCH_T(dtype, { rc = rec_dispatch<T, false>(p, stream); });
+  OSLO_DISPATCH_T(dtype, { rc = rec_dispatch<T, false>(p, rule, stream); });
   return rc;
 }
 
-extern "C" int oslo_recurrence_step(const void* q, long long ldq, const void* f, long long ldf, const void* v, long long ldv,
-                                    const void* f_bias, const void* lower, const void* norm_w, const uint8_t* keep,
-                                    long long ld_keep, float* state, void* out, float eps, int B, int H, int dim, int vdim, int num_sms, int dtype, cudaStream_t stream) {
+static int step_launch(int rule, oslo::StepParams p, int B, int num_sms, int dtype, cudaStream_t stream) {
   using namespace oslo;
-  if (B <= 0 || H <= 0) return 0;
-  if (dim <= 0 || vdim <= 0 || B > 65535 || H > 65535) return -1;
-  const int vec = vdim % 4 == 0 && aligned_to(state, 16) ? 4 : 1;
+  if (B <= 0 || p.H <= 0) return 0;
+  if (p.dim <= 0 || p.vdim <= 0 || B > 65535 || p.H > 65535) return -1;
+  const int H = p.H, vdim = p.vdim;
+  const int vec = vdim % 4 == 0 && aligned_to(p.state, 16) ? 4 : 1;
   int slices = 1;   // portable cluster sizes; a slice keeps at least 16 columns
   while (slices < 8 && static_cast<long long>(B) * H * slices < 2 * num_sms && vdim / (2 * slices) >= 16) slices *= 2;
   while (slices < 8 && (vdim + slices - 1) / slices > 256 * vec) slices *= 2;
-  int cols = ((vdim + slices - 1) / slices + vec - 1) / vec * vec;
-  if (cols / vec > 256) return -3;
-  StepParams p{q, f, v, ldq, ldf, ldv, f_bias, lower, norm_w, keep, ld_keep, state, out, H, dim, vdim, cols, eps};
-  const int ty = 256 / (cols / vec);
-  const size_t smem = (2 * static_cast<size_t>(dim) + static_cast<size_t>(ty) * cols) * sizeof(float);
+  p.cols = ((vdim + slices - 1) / slices + vec - 1) / vec * vec;
+  if (p.cols / vec > 256) return -3;
+  const int ty = 256 / (p.cols / vec);
+  const size_t smem = ((rule == RULE_BONUS ? 3 : 2) * static_cast<size_t>(p.dim) + p.rank + static_cast<size_t>(ty) * p.cols) * sizeof(float);
+  if (smem > 48 * 1024) return -3;
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3(slices, H, B);
   cfg.blockDim = dim3(256);
@@ -512,9 +718,44 @@ extern "C" int oslo_recurrence_step(const void* q, long long ldq, const void* f,
   cfg.attrs = attr;
   cfg.numAttrs = 1;
   cudaError_t e = cudaSuccess;
+#define STEP_GO(R)                                                                    \
+  if (vec == 4) e = cudaLaunchKernelEx(&cfg, recurrence_step_kernel<T, 4, R>, p);     \
+  else e = cudaLaunchKernelEx(&cfg, recurrence_step_kernel<T, 1, R>, p);
   OSLO_DISPATCH_T(dtype, {
-    if (vec == 4) e = cudaLaunchKernelEx(&cfg, recurrence_step_kernel<T, 4>, p);
-    else e = cudaLaunchKernelEx(&cfg, recurrence_step_kernel<T, 1>, p);
+    if (rule == RULE_GATED) { STEP_GO(RULE_GATED) }
+    else if (rule == RULE_DECAY) { STEP_GO(RULE_DECAY) }
+    else { STEP_GO(RULE_BONUS) }
   });
+#undef STEP_GO
   return static_cast<int>(e);
+}
+
+extern "C" int oslo_recurrence_step(const void* q, long long ldq, const void* f, long long ldf, const void* v, long long ldv,
+                                    const void* f_bias, const void* lower, const void* norm_w, const uint8_t* keep,
+                                    long long ld_keep, float* state, void* out, float eps, int B, int H, int dim, int vdim, int num_sms, int dtype, cudaStream_t stream) {
+  oslo::StepParams p{};
+  p.q = q; p.f = f; p.v = v; p.ldq = ldq; p.ldf = ldf; p.ldv = ldv;
+  p.f_bias = f_bias; p.lower = lower; p.norm_w = norm_w; p.keep = keep; p.ld_keep = ld_keep;
+  p.state = state; p.out = out; p.H = H; p.dim = dim; p.vdim = vdim; p.eps = eps;
+  return step_launch(oslo::RULE_GATED, p, B, num_sms, dtype, stream);
+}
+
+extern "C" int oslo_decayed_step(const void* q, long long ldq, const void* k, long long ldk, const void* v, long long ldv,
+                                 const float* head_decay, const uint8_t* keep, long long ld_keep, float* state, float* out, int B,
+                                 int H, int dim, int vdim, int num_sms, int dtype, cudaStream_t stream) {
+  oslo::StepParams p{};
+  p.q = q; p.f = k; p.v = v; p.ldq = ldq; p.ldf = ldk; p.ldv = ldv; p.head_decay = head_decay; p.keep = keep; p.ld_keep = ld_keep;
+  p.state = state; p.out = out; p.H = H; p.dim = dim; p.vdim = vdim;
+  return step_launch(oslo::RULE_DECAY, p, B, num_sms, dtype, stream);
+}
+
+extern "C" int oslo_bonus_step(const void* r, long long ldr, const void* k, long long ldk, const void* v, long long ldv, const void* t,
+                               long long ldt, const void* w2, int rank, const void* w0, const void* u, const void* norm_w,
+                               const void* gate, long long ldg, const uint8_t* keep, long long ld_keep, float* state, void* out,
+                               float eps, int B, int H, int dim, int vdim, int num_sms, int dtype, cudaStream_t stream) {
+  oslo::StepParams p{};
+  p.q = r; p.f = k; p.v = v; p.ldq = ldr; p.ldf = ldk; p.ldv = ldv; p.f_bias = w0; p.lower = u; p.norm_w = norm_w;
+  p.t = t; p.ldt = ldt; p.w2 = w2; p.rank = rank; p.gate = gate; p.ldg = ldg;
+  p.keep = keep; p.ld_keep = ld_keep; p.state = state; p.out = out; p.H = H; p.dim = dim; p.vdim = vdim; p.eps = eps;
+  return step_launch(oslo::RULE_BONUS, p, B, num_sms, dtype, stream);
 }

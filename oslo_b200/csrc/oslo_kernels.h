@@ -122,10 +122,10 @@ int oslo_flash_fwd_sm100(const void* q, const void* k, const void* v, void* o, f
                          cudaStream_t stream);
 // causal, with exp(sink[h]) in the denominator and a sigmoid output gate per (position, head); stores the first d_out columns
 int oslo_flash_sink_fwd_sm100(const void* q, const void* k, const void* v, void* o, const uint8_t* kpm, const void* sink,
-                              const void* gate, long long ldg, int d_out, int B, int H, int Sq, int Sk, int D, long long q_sb,
-                              long long q_sh, long long q_ss, long long k_sb, long long k_sh, long long k_ss, long long v_sb,
-                              long long v_sh, long long v_ss, long long o_sb, long long o_sh, long long o_ss, float scale,
-                              int dtype, int* err_word, cudaStream_t stream);
+                              const void* gate, long long ldg, int B, int H, int G, int Sq, int Sk, int dim, int vdim,
+                              long long q_sb, long long q_sh, long long q_ss, long long k_sb, long long k_sh, long long k_ss,
+                              long long v_sb, long long v_sh, long long v_ss, long long o_sb, long long o_sh, long long o_ss,
+                              float scale, float softcap, int dtype, int* err_word, cudaStream_t stream);
 int oslo_flash_bwd(const void* q, const void* k, const void* v, const void* o, const void* dout, const float* lse,
                    float* delta, float* dq_acc, void* dq, void* dk, void* dv, const uint8_t* kpm, int B, int H,
                    int Sq, int Sk, int D, long long q_sb, long long q_sh, long long q_ss, long long k_sb,
@@ -178,6 +178,9 @@ int oslo_ce_combine(const float* mx, const float* se, const float* tg, float* ou
 // decode-step kernels (decode_sm100.cu). gemv_rows: out[m, n] = act([x1 | x2][m, :] . W[n, :] + bias[n]) for M <= 4
 // rows, W [N, K1 + K2] K-major, tanh-GeLU on columns >= gelu_from (-1 = none); x2 may be null.
 // `res` [M, N] (row stride ldr) is added after the activation; bias and res may be null.
+// P of them at once: x [P, M, K] and W [P, N, K] (strides sx, sw between parts) -> out [P, M, N]
+int oslo_gemv_stacked(const void* x, int ldx, long long sx, const void* W, int ldw, long long sw, void* out, int P, int M, int N, int K,
+                      int dtype, int num_sms, cudaStream_t stream);
 int oslo_gemv_rows(const void* x1, int ld1, int K1, const void* x2, int ld2, int K2, const void* W, int ldw,
                    const void* bias, const void* res, int ldr, void* out, int ldo, int M, int N, int gelu_from,
                    int dtype, int num_sms, cudaStream_t stream);
@@ -214,28 +217,53 @@ int oslo_residual_join(const float* x, const void* y, long long ldy, const int* 
                        float* x_out, void* h_out, long long rows, int cols, float eps, int dtype, cudaStream_t stream);
 int oslo_silu_mul(const void* gate, long long ldg, const void* up, long long ldu, void* out, long long rows, int cols, int dtype,
                   cudaStream_t stream);
+// g sigmoid(alpha g) (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit)
+int oslo_clamped_glu(const void* gate, long long ldg, const void* up, long long ldu, void* out, long long rows, int cols,
+                     float limit, float alpha, int dtype, cudaStream_t stream);
+// x_out = x + mult * sum_i factor[i] * (w[i] ? rms(y[i]) * w[i] : y[i]), n <= 3; h1 = rms(x_out) * w1, h2 = rms(x_out) * w2 (or null)
+int oslo_branch_join(const float* x, int n, const void* const* y, const long long* ldy, const void* const* w, const float* factor,
+                     float mult, float eps, const void* w1, const void* w2, float* x_out, void* h1, void* h2, long long rows,
+                     int cols, int dtype, cudaStream_t stream);
+// out = o / rms(runs of `group` columns) * w * act(gate); act 0: sigmoid, 1: silu; o fp32 [rows, cols]
+int oslo_gated_rms_norm(const float* o, const void* w, const void* gate, long long ldg, void* out, long long rows, int cols,
+                        int group, float eps, int act, int dtype, cudaStream_t stream);
 
-// gated linear recurrence (linear_recurrence.cu): q, f [B * S, H * dim], v [B * S, H * vdim] with row strides; keep [B, S]
+// linear recurrences (linear_recurrence.cu): q, f [B * S, H * dim], v [B * S, H * vdim] with row strides; keep [B, S]
 // (0 = padding) or null; state [B, H, dim, vdim] fp32, read and updated, or null; out fp32 [B, S, H, vdim].
-// nchunks > 1 (oslo_recurrence_chunks) needs ws [B, nchunks, H, dim, vdim] and decay [B, nchunks, H, dim] fp32
+// nchunks > 1 (oslo_recurrence_chunks) needs ws [B, nchunks, H, dim, vdim] and decay [B, nchunks, H, dim] fp32.
+// rule 0: f are forget-gate logits with f_bias and lower bounds [H * dim]; 1: f are keys, head_decay [H] fp32; 2: f are keys,
+// f_bias = w0 and lower = u [H * dim], z the decay logits fp32 [B * S, H * dim]
 int oslo_recurrence_chunks(int B, int S, int H, int dim, int vdim, int num_sms);
-int oslo_recurrence(const void* q, long long ldq, const void* f, long long ldf, const void* v, long long ldv,
-                    const void* f_bias, const void* lower, const uint8_t* keep, long long ld_keep, float* state, float* out,
-                    float* ws, float* decay, int nchunks, int B, int S, int H, int dim, int vdim, int dtype,
-                    cudaStream_t stream);
+int oslo_recurrence(int rule, const void* q, long long ldq, const void* f, long long ldf, const void* v, long long ldv,
+                    const void* f_bias, const void* lower, const float* z, long long ldz, const float* head_decay,
+                    const uint8_t* keep, long long ld_keep, float* state, float* out, float* ws, float* decay, int nchunks, int B,
+                    int S, int H, int dim, int vdim, int dtype, cudaStream_t stream);
 // one token per row, the outputs RMS-normed per head with norm_w [vdim]
 int oslo_recurrence_step(const void* q, long long ldq, const void* f, long long ldf, const void* v, long long ldv,
                          const void* f_bias, const void* lower, const void* norm_w, const uint8_t* keep, long long ld_keep,
                          float* state, void* out, float eps, int B, int H, int dim, int vdim, int num_sms, int dtype, cudaStream_t stream);
 
+// rule 1, one token per row: out fp32 [B, H * vdim], not normed
+int oslo_decayed_step(const void* q, long long ldq, const void* k, long long ldk, const void* v, long long ldv,
+                      const float* head_decay, const uint8_t* keep, long long ld_keep, float* state, float* out, int B, int H,
+                      int dim, int vdim, int num_sms, int dtype, cudaStream_t stream);
+// rule 2, one token per row: decay logits W_w2 tanh(t) (t [B, rank], w2 [H * dim, rank]), heads RMS-normed, times norm_w
+// [H * vdim] and silu(gate)
+int oslo_bonus_step(const void* r, long long ldr, const void* k, long long ldk, const void* v, long long ldv, const void* t,
+                    long long ldt, const void* w2, int rank, const void* w0, const void* u, const void* norm_w, const void* gate,
+                    long long ldg, const uint8_t* keep, long long ld_keep, float* state, void* out, float eps, int B, int H, int dim,
+                    int vdim, int num_sms, int dtype, cudaStream_t stream);
+
 // latent attention (latent_attention.cu). sink_gate: flash output [B, S, H, *] + lse [B, H, S] -> out [B * S, H * vdim]
 int oslo_sink_gate(const void* o, long long o_sb, long long o_ss, long long o_sh, const float* lse, const void* sink,
                    const void* gate, long long ldg, void* out, int B, int S, int H, int vdim, int dtype, cudaStream_t stream);
-// causal attention with sink and output gate in 32-bit, any head sizes; strides of (batch, position, head)
+// causal attention with sink and output gate (or null) in 32-bit, any head sizes; strides of (batch, position, head); G key /
+// value heads; softcap > 0: scores become softcap * tanh(score / softcap)
 int oslo_sink_attention(const void* q, long long q_sb, long long q_ss, long long q_sh, const void* k, long long k_sb,
                         long long k_ss, long long k_sh, const void* v, long long v_sb, long long v_ss, long long v_sh,
                         const uint8_t* keep, long long ld_keep, const void* sink, const void* gate, long long ldg, void* out,
-                        int B, int H, int Sq, int Sk, int dim, int vdim, float scale, int dtype, cudaStream_t stream);
+                        int B, int H, int G, int Sq, int Sk, int dim, int vdim, float scale, float softcap, int dtype,
+                        cudaStream_t stream);
 // decode: RMS norm of the query latent -> cq_out; of the key-value latent (null: none) -> cache [B, Tmax, kv_rank] at lengths[b]
 int oslo_latent_prep(const void* cq, long long ldq, const void* wq, int q_rank, void* cq_out, const void* ckv, long long ldkv,
                      const void* wkv, int kv_rank, void* cache, const int* lengths, int Tmax, float eps, int B, int dtype,
@@ -248,6 +276,39 @@ int oslo_latent_decode(const void* q, long long ldq, const void* w_uk, long long
                        int B, int H, int dim, int vdim, int R, int Tmax, int splits, float scale, int num_sms, int dtype,
                        int* err_word, cudaStream_t stream);
 int oslo_latent_splits(int B, int H, int T, int num_sms);
+
+// grouped-query attention (grouped_attention.cu). qkv_prep: RMS norm of every query / key head (weights wq, wk [dim]), rotation of
+// the first 2 * n_freq dims by pos[b, t] * freq, q -> q_out [B, S, H, dim], k / v -> caches [B, G, Tmax, *] at lengths[b] + t
+int oslo_qkv_prep(const void* q, long long ldq, const void* k, long long ldk, const void* v, long long ldv, const void* wq,
+                  const void* wk, float eps, const long long* pos, long long pos_sb, long long pos_ss, const float* freq, int n_freq,
+                  void* q_out, void* kc, void* vc, const int* lengths, int B, int S, int H, int G, int dim, int vdim, int Tmax,
+                  int dtype, int* err_word, cudaStream_t stream);
+// one query per row: q [B, H, dim], caches [B, G, Tmax, *], of which lengths[b] positions count; keep [B, n_keep] (0 = padded) or
+// null; fp32 workspaces ws [B, H, splits, vdim rounded up to a multiple of 4] and stat [B, H, splits, 2]; out [B, H * vdim]
+int oslo_grouped_splits(int B, int H, int G, int T, int num_sms);
+int oslo_grouped_decode(const void* q, const void* kc, const void* vc, const int* lengths, const uint8_t* keep, long long ld_keep,
+                        int n_keep, const void* sink, float* ws, float* stat, void* out, int B, int H, int G, int dim, int vdim,
+                        int Tmax, int splits, float scale, float softcap, int dtype, int* err_word, cudaStream_t stream);
+
+// token shift, causal convolution and selective scan (selective_scan.cu)
+// out[i] = h + (h' - h) * mu[i], i < P; prev fp32 [B, width] (the row before the first; read and updated) or null
+int oslo_token_shift(const void* h, long long ldh, const void* mu, const uint8_t* keep, long long ld_keep, float* prev, void* out,
+                     int B, int S, int width, int P, int dtype, cudaStream_t stream);
+// out [B * S, C] = silu(conv(x) + bias); prev fp32 [B, taps - 1, C] (read and updated) or null
+int oslo_causal_conv_silu(const void* x, long long ldx, const void* w, const void* bias, const uint8_t* keep, long long ld_keep,
+                          float* prev, void* out, int B, int S, int C, int taps, int dtype, cudaStream_t stream);
+// dt fp32 logits [B * S, C]; state fp32 [B, C, N] (read and updated) or null; out [B * S, C]. nchunks > 1 (oslo_scan_chunks) needs
+// ws [B, nchunks, C, N] and steps [B, nchunks, C] fp32
+int oslo_scan_chunks(int B, int S, int C, int N, int num_sms);
+int oslo_selective_scan(const void* x, long long ldx, const float* dt, long long lddt, const void* dt_bias, const void* a_log,
+                        const void* b, long long ldb, const void* c, long long ldc, const void* d, const void* z, long long ldz,
+                        const uint8_t* keep, long long ld_keep, float* state, void* out, float* ws, float* steps, int nchunks, int B,
+                        int S, int C, int N, int dtype, cudaStream_t stream);
+// one token per row; the step logits are w_dt [C, rank] . dt [B, rank]
+int oslo_scan_step(const void* x, long long ldx, const void* dt, long long lddt, const void* w_dt, int rank, const void* dt_bias,
+                   const void* a_log, const void* b, long long ldb, const void* c, long long ldc, const void* d, const void* z,
+                   long long ldz, const uint8_t* keep, long long ld_keep, float* state, void* out, int B, int C, int N, int dtype,
+                   cudaStream_t stream);
 
 // mixture of experts (moe.cu, grouped GEMM in gemm_sm100.cu)
 int oslo_moe_route(const void* h, long long ldh, const void* w, const void* bias, const float* logits, int* idx, float* wgt,

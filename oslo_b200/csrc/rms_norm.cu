@@ -1,6 +1,9 @@
 // RMS norms with 32-bit arithmetic and the step that joins a sublayer to the residual stream.
 //
 //   rms_norm:      out = x / sqrt(mean(x^2) + eps) * (offset + w)        offset 1: the weight is stored around zero
+//   gated_rms_norm: out = o / sqrt(mean(o^2 of a run of columns) + eps) * w * act(gate)
+//   branch_join:   x'  = x + mult * sum of the (possibly normed) results of parallel branches
+//                  h_i = x' / sqrt(mean(x'^2) + eps) * w_i, i = 1, 2    the inputs of the next layer's branches
 //   residual_join: z   = y * sigmoid(gate + gate_bias)
 //                  x'  = x + z / sqrt(mean(z^2) + eps) * (1 + w_post)
 //                  h   = x' / sqrt(mean(x'^2) + eps) * (1 + w_next)      the input of the next sublayer, 16-bit
@@ -159,10 +162,141 @@ __global__ void __launch_bounds__(256) residual_join_kernel(const JoinParams p) 
   }
 }
 
-// y = silu(gate) * up on [rows, cols] slices with row strides
+struct BranchParams {
+  const float* x;
+  int n;
+  const void* y[3]; long long ldy[3];
+  const void* w[3];            // norm weight of the branch, or nullptr
+  float factor[3];
+  float mult, eps;
+  const void *w1, *w2;         // nullptr: no such output
+  float* x_out;
+  void *h1, *h2;
+  int cols;
+};
+
 template <typename T, int VEC>
-__global__ void __launch_bounds__(256) silu_mul_kernel(const T* __restrict__ gate, long long ldg, const T* __restrict__ up,
-                                                       long long ldu, T* __restrict__ out, long long rows, int cols) {
+__global__ void __launch_bounds__(256) branch_join_kernel(const BranchParams p) {
+  extern __shared__ float row_s[];
+  __shared__ float red[32];
+  const long long row = blockIdx.x;
+  float f[3];
+#pragma unroll
+  for (int b = 0; b < 3; ++b) {
+    if (b >= p.n) break;
+    f[b] = p.mult * p.factor[b];
+    if (p.w[b] == nullptr) continue;             // uniform over the block
+    const T* y = static_cast<const T*>(p.y[b]) + row * p.ldy[b];
+    float ss = 0.f;
+    for (int c = threadIdx.x * VEC; c < p.cols; c += blockDim.x * VEC) {
+      float v[VEC];
+      load_vec<T, VEC>(y + c, v);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) ss = fmaf(v[i], v[i], ss);
+    }
+    ss = block_sum(ss, red);
+    f[b] *= 1.0f / sqrtf(ss / p.cols + p.eps);
+  }
+  float sx = 0.f;
+  for (int c = threadIdx.x * VEC; c < p.cols; c += blockDim.x * VEC) {
+    float v[VEC];
+    load_vec<float, VEC>(p.x + row * p.cols + c, v);
+#pragma unroll
+    for (int b = 0; b < 3; ++b) {
+      if (b >= p.n) break;
+      float y[VEC];
+      load_vec<T, VEC>(static_cast<const T*>(p.y[b]) + row * p.ldy[b] + c, y);
+      if (p.w[b] != nullptr) {
+        float w[VEC];
+        load_vec<T, VEC>(static_cast<const T*>(p.w[b]) + c, w);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) v[i] = fmaf(f[b] * y[i], w[i], v[i]);
+      } else {
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) v[i] = fmaf(f[b], y[i], v[i]);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) {
+      sx = fmaf(v[i], v[i], sx);
+      row_s[c + i] = v[i];
+    }
+    store_vec<float, VEC>(p.x_out + row * p.cols + c, v);
+  }
+  if (p.w1 == nullptr) return;
+  sx = block_sum(sx, red);
+  const float rn = 1.0f / sqrtf(sx / p.cols + p.eps);
+  for (int c = threadIdx.x * VEC; c < p.cols; c += blockDim.x * VEC) {   // every thread revisits its own elements
+    float v[VEC], w[VEC];
+    load_vec<T, VEC>(static_cast<const T*>(p.w1) + c, w);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[i] = row_s[c + i] * rn * w[i];
+    store_vec<T, VEC>(static_cast<T*>(p.h1) + row * p.cols + c, v);
+    if (p.w2 != nullptr) {
+      load_vec<T, VEC>(static_cast<const T*>(p.w2) + c, w);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) v[i] = row_s[c + i] * rn * w[i];
+      store_vec<T, VEC>(static_cast<T*>(p.h2) + row * p.cols + c, v);
+    }
+  }
+}
+
+template <typename T, int VEC>
+__device__ __forceinline__ void gate_run(const float* o, const T* w, const T* gate, T* out, int c, float r, int act) {
+  float v[VEC], g[VEC], ww[VEC];
+  load_vec<float, VEC>(o + c, v);
+  load_vec<T, VEC>(w + c, ww);
+  load_vec<T, VEC>(gate + c, g);
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) v[i] = v[i] * r * ww[i] * (act ? silu_f(g[i]) : sigmoid_f(g[i]));
+  store_vec<T, VEC>(out + c, v);
+}
+
+// one warp (WARP) or one block per run of `group` columns
+template <typename T, int VEC, bool WARP>
+__global__ void __launch_bounds__(256) gated_rms_norm_kernel(const float* __restrict__ o, const T* __restrict__ w,
+                                                             const T* __restrict__ gate, long long ldg, T* __restrict__ out,
+                                                             long long runs, int cols, int group, float eps, int act) {
+  __shared__ float red[32];
+  const long long run = WARP ? static_cast<long long>(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5) : blockIdx.x;
+  if (run >= runs) return;                                 // WARP: whole warps leave, and no barrier follows
+  const int per_row = cols / group;
+  const long long row = run / per_row;
+  const int c0 = static_cast<int>(run - row * per_row) * group;
+  const int lane = WARP ? threadIdx.x & 31 : threadIdx.x, step = WARP ? 32 : blockDim.x;
+  o += row * cols + c0;
+  w += c0;
+  gate += row * ldg + c0;
+  out += row * cols + c0;
+  float ss = 0.f;
+  for (int c = lane * VEC; c < group; c += step * VEC) {
+    float v[VEC];
+    load_vec<float, VEC>(o + c, v);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) ss = fmaf(v[i], v[i], ss);
+  }
+  ss = WARP ? warp_sum(ss) : block_sum(ss, red);
+  const float r = 1.0f / sqrtf(ss / group + eps);
+  for (int c = lane * VEC; c < group; c += step * VEC) gate_run<T, VEC>(o, w, gate, out, c, r, act);
+}
+
+struct SiluUnit {
+  __device__ __forceinline__ float operator()(float g, float u) const { return silu_f(g) * u; }
+};
+struct ClampedUnit {
+  float limit, alpha;
+  __device__ __forceinline__ float operator()(float g, float u) const {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g * sigmoid_f(alpha * g) * (u + 1.0f);
+  }
+};
+
+// y = unit(gate, up) on [rows, cols] slices with row strides
+template <typename T, int VEC, typename Unit>
+__global__ void __launch_bounds__(256) gated_unit_kernel(const T* __restrict__ gate, long long ldg, const T* __restrict__ up,
+                                                         long long ldu, T* __restrict__ out, long long rows, int cols,
+                                                         const Unit unit) {
   const long long per_row = cols / VEC;
   const long long total = rows * per_row;
   for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total;
@@ -173,9 +307,27 @@ __global__ void __launch_bounds__(256) silu_mul_kernel(const T* __restrict__ gat
     load_vec<T, VEC>(gate + r * ldg + c, a);
     load_vec<T, VEC>(up + r * ldu + c, b);
 #pragma unroll
-    for (int k = 0; k < VEC; ++k) a[k] = silu_f(a[k]) * b[k];
+    for (int k = 0; k < VEC; ++k) a[k] = unit(a[k], b[k]);
     store_vec<T, VEC>(out + r * cols + c, a);
   }
+}
+
+template <typename Unit>
+static int gated_unit(const void* gate, long long ldg, const void* up, long long ldu, void* out, long long rows, int cols,
+                      const Unit& unit, int dtype, cudaStream_t stream) {
+  if (rows <= 0 || cols <= 0) return 0;
+  const size_t te = dtype == OSLO_DT_FP32 ? 4 : 2;
+  const bool vec = cols % 4 == 0 && ldg % 4 == 0 && ldu % 4 == 0 && aligned_to(gate, 4 * te) && aligned_to(up, 4 * te) &&
+                   aligned_to(out, 4 * te);
+  const long long work = rows * (vec ? cols / 4 : cols);
+  const unsigned blocks = static_cast<unsigned>(std::min<long long>((work + 255) / 256, 148 * 16));
+  OSLO_DISPATCH_T(dtype, {
+    if (vec) gated_unit_kernel<T, 4, Unit><<<blocks, 256, 0, stream>>>(static_cast<const T*>(gate), ldg, static_cast<const T*>(up),
+                                                                       ldu, static_cast<T*>(out), rows, cols, unit);
+    else gated_unit_kernel<T, 1, Unit><<<blocks, 256, 0, stream>>>(static_cast<const T*>(gate), ldg, static_cast<const T*>(up), ldu,
+                                                                   static_cast<T*>(out), rows, cols, unit);
+  });
+  return static_cast<int>(cudaGetLastError());
 }
 
 }  // namespace oslo
@@ -231,18 +383,65 @@ extern "C" int oslo_residual_join(const float* x, const void* y, long long ldy, 
 
 extern "C" int oslo_silu_mul(const void* gate, long long ldg, const void* up, long long ldu, void* out, long long rows,
                              int cols, int dtype, cudaStream_t stream) {
+  return oslo::gated_unit(gate, ldg, up, ldu, out, rows, cols, oslo::SiluUnit{}, dtype, stream);
+}
+
+extern "C" int oslo_clamped_glu(const void* gate, long long ldg, const void* up, long long ldu, void* out, long long rows,
+                                int cols, float limit, float alpha, int dtype, cudaStream_t stream) {
+  return oslo::gated_unit(gate, ldg, up, ldu, out, rows, cols, oslo::ClampedUnit{limit, alpha}, dtype, stream);
+}
+
+extern "C" int oslo_branch_join(const float* x, int n, const void* const* y, const long long* ldy, const void* const* w,
+                                const float* factor, float mult, float eps, const void* w1, const void* w2, float* x_out, void* h1,
+                                void* h2, long long rows, int cols, int dtype, cudaStream_t stream) {
   using namespace oslo;
   if (rows <= 0 || cols <= 0) return 0;
+  if (rows > 0x7fffffffll || n < 1 || n > 3) return -1;
   const size_t te = dtype == OSLO_DT_FP32 ? 4 : 2;
-  const bool vec = cols % 4 == 0 && ldg % 4 == 0 && ldu % 4 == 0 && aligned_to(gate, 4 * te) && aligned_to(up, 4 * te) &&
+  BranchParams p{};
+  bool vec = cols % 4 == 0 && aligned_to(x, 16) && aligned_to(x_out, 16);
+  for (const void* t : {w1, w2, static_cast<const void*>(h1), static_cast<const void*>(h2)}) vec = vec && (t == nullptr || aligned_to(t, 4 * te));
+  p.x = x; p.n = n;
+  for (int i = 0; i < n; ++i) {
+    p.y[i] = y[i]; p.ldy[i] = ldy[i]; p.w[i] = w[i]; p.factor[i] = factor[i];
+    vec = vec && ldy[i] % 4 == 0 && aligned_to(y[i], 4 * te) && (w[i] == nullptr || aligned_to(w[i], 4 * te));
+  }
+  p.mult = mult; p.eps = eps; p.w1 = w1; p.w2 = w2; p.x_out = x_out; p.h1 = h1; p.h2 = h2; p.cols = cols;
+  const size_t smem = static_cast<size_t>(cols) * sizeof(float);
+  if (smem > 200 * 1024) return -3;
+  const int threads = cols >= 1024 ? 256 : (cols >= 512 ? 128 : 64);
+#define BRANCH_GO(V)                                                                                             \
+  {                                                                                                              \
+    if (smem > 48 * 1024) {                                                                                      \
+      cudaError_t e = cudaFuncSetAttribute(branch_join_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
+                                           static_cast<int>(smem));                                              \
+      if (e != cudaSuccess) return static_cast<int>(e);                                                          \
+    }                                                                                                            \
+    branch_join_kernel<T, V><<<static_cast<unsigned>(rows), threads, smem, stream>>>(p);                         \
+  }
+  OSLO_DISPATCH_T(dtype, { if (vec) BRANCH_GO(4) else BRANCH_GO(1) });
+#undef BRANCH_GO
+  return static_cast<int>(cudaGetLastError());
+}
+
+extern "C" int oslo_gated_rms_norm(const float* o, const void* w, const void* gate, long long ldg, void* out, long long rows,
+                                   int cols, int group, float eps, int act, int dtype, cudaStream_t stream) {
+  using namespace oslo;
+  if (rows <= 0 || cols <= 0) return 0;
+  if (group <= 0 || cols % group) return -1;
+  const long long runs = rows * (cols / group);
+  if (runs > 0x7fffffffll) return -1;
+  const size_t te = dtype == OSLO_DT_FP32 ? 4 : 2;
+  const bool vec = group % 4 == 0 && ldg % 4 == 0 && aligned_to(o, 16) && aligned_to(w, 4 * te) && aligned_to(gate, 4 * te) &&
                    aligned_to(out, 4 * te);
-  const long long work = rows * (vec ? cols / 4 : cols);
-  const unsigned blocks = static_cast<unsigned>(std::min<long long>((work + 255) / 256, 148 * 16));
-  OSLO_DISPATCH_T(dtype, {
-    if (vec) silu_mul_kernel<T, 4><<<blocks, 256, 0, stream>>>(static_cast<const T*>(gate), ldg, static_cast<const T*>(up), ldu,
-                                                               static_cast<T*>(out), rows, cols);
-    else silu_mul_kernel<T, 1><<<blocks, 256, 0, stream>>>(static_cast<const T*>(gate), ldg, static_cast<const T*>(up), ldu,
-                                                           static_cast<T*>(out), rows, cols);
-  });
+#define GATED_GO(V)                                                                                                         \
+  if (group <= 512)                                                                                                         \
+    gated_rms_norm_kernel<T, V, true><<<static_cast<unsigned>((runs + 7) / 8), 256, 0, stream>>>(                           \
+        o, static_cast<const T*>(w), static_cast<const T*>(gate), ldg, static_cast<T*>(out), runs, cols, group, eps, act);  \
+  else                                                                                                                      \
+    gated_rms_norm_kernel<T, V, false><<<static_cast<unsigned>(runs), 256, 0, stream>>>(                                    \
+        o, static_cast<const T*>(w), static_cast<const T*>(gate), ldg, static_cast<T*>(out), runs, cols, group, eps, act);
+  OSLO_DISPATCH_T(dtype, { if (vec) { GATED_GO(4) } else { GATED_GO(1) } });
+#undef GATED_GO
   return static_cast<int>(cudaGetLastError());
 }

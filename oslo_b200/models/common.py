@@ -24,9 +24,10 @@ from ..modeling_utils import (BaseModelOutputWithPast, CausalLMOutputWithPast, P
 class StaticKVCache:
     """Pre-allocated cache written in place. Per layer it holds whichever of these the layer's mixer needs:
 
-    * ``k`` / ``v``: keys and values ``[B, heads, T_max, D]``;
+    * ``k`` / ``v``: keys and values ``[B, heads, T_max, D]`` (the two may differ in ``D``);
     * ``latent``: one low-rank vector per token ``[B, T_max, rank]`` (latent attention; layers may read another layer's);
-    * ``state``: a recurrent state of fixed size in fp32, first dim ``B`` (linear recurrences).
+    * ``state``: states of fixed size in fp32, first dim ``B`` (linear recurrences, scans, the inputs a convolution or token
+      shift looks back to); keyed by layer, or by ``(layer, name)`` where a layer has several.
 
     Replaces the grow-by-``torch.cat`` cache of the reference (oslo/models/gptj/modeling_gptj.py:239-248):
     appends are slice writes, beam reordering is one ``index_select`` per tensor, and the decode
@@ -38,7 +39,7 @@ class StaticKVCache:
         self.k: Dict[int, Tensor] = {}
         self.v: Dict[int, Tensor] = {}
         self.latent: Dict[int, Tensor] = {}
-        self.state: Dict[int, Tensor] = {}
+        self.state: Dict[Any, Tensor] = {}
         self.length = 0
         self.max_len = int(max_len)
         self.grow = bool(grow)
@@ -94,16 +95,23 @@ class StaticKVCache:
                 new.narrow(dim, 0, t.size(dim)).copy_(t)
                 store[i] = new
 
+    def kv_storage(self, layer: int, b: int, heads: int, dim: int, vdim: int, dtype: torch.dtype, device,
+                   new_tokens: int) -> Tuple[Tensor, Tensor]:
+        """Keys ``[B, heads, T_max, dim]`` and values ``[B, heads, T_max, vdim]`` of ``layer`` with room for ``new_tokens`` more;
+        position ``length`` is the next one. Storage is allocated on first use per layer."""
+        self._reserve(self.length + new_tokens)
+        if layer not in self.k:
+            self.k[layer] = torch.zeros(b, heads, self.max_len, dim, dtype=dtype, device=device)
+            self.v[layer] = torch.zeros(b, heads, self.max_len, vdim, dtype=dtype, device=device)
+        self._ensure_lengths(b, device)
+        return self.k[layer], self.v[layer]
+
     def append(self, layer: int, k: Tensor, v: Tensor) -> Tuple[Tensor, Tensor, int]:
         """Write ``k, v`` (``[B, heads, S, D]``) at the current position; returns the whole cache
-        tensors of that layer and the new valid length. Storage is allocated on first use per layer."""
+        tensors of that layer and the new valid length."""
         b, h, s, d = k.shape
         end = self.length + s
-        self._reserve(end)
-        if layer not in self.k:
-            self.k[layer] = torch.zeros(b, h, self.max_len, d, dtype=k.dtype, device=k.device)
-            self.v[layer] = torch.zeros(b, h, self.max_len, d, dtype=v.dtype, device=v.device)
-        self._ensure_lengths(b, k.device)
+        self.kv_storage(layer, b, h, d, v.size(-1), k.dtype, k.device, s)
         if self.device_positions and s == 1:
             self.k[layer].index_copy_(2, self.write_index, k)
             self.v[layer].index_copy_(2, self.write_index, v)
@@ -131,12 +139,14 @@ class StaticKVCache:
             store[:, self.length:self.length + s].copy_(c)
         return store[:, :self.length + s]
 
-    def recurrent_state(self, layer: int, shape, device) -> Tensor:
-        """The fp32 state of ``layer`` (zero for a new sequence), to be updated in place."""
-        if layer not in self.state:
-            self.state[layer] = torch.zeros(*shape, dtype=torch.float32, device=device)
+    def recurrent_state(self, layer: int, shape, device, name: Optional[str] = None) -> Tensor:
+        """The fp32 state of ``layer`` (zero for a new sequence), to be updated in place; ``name`` tells several states of a layer
+        apart."""
+        key = layer if name is None else (layer, name)
+        if key not in self.state:
+            self.state[key] = torch.zeros(*shape, dtype=torch.float32, device=device)
         self._ensure_lengths(shape[0], device)
-        return self.state[layer]
+        return self.state[key]
 
     def advance(self, s: int) -> None:
         self.length += s

@@ -10,6 +10,7 @@ import os
 from typing import Any, Dict, NamedTuple, Type
 
 from ..modeling_utils import CONFIG_NAME, PretrainedConfig, PreTrainedModel, _resolve_hub_file
+from .begovik import BegovikConfig, BegovikForCausalLM
 from .gpt2 import GPT2Config, GPT2LMHeadModel
 from .gpt_neo import GPTNeoConfig, GPTNeoForCausalLM
 from .gptj import GPTJConfig, GPTJForCausalLM
@@ -26,6 +27,7 @@ MODELS: Dict[str, ModelEntry] = {
     "gpt_neo": ModelEntry(GPTNeoConfig, GPTNeoForCausalLM),
     "gptj": ModelEntry(GPTJConfig, GPTJForCausalLM),
     "moronex": ModelEntry(MoronexConfig, MoronexForCausalLM),
+    "begovik": ModelEntry(BegovikConfig, BegovikForCausalLM),
 }
 
 

@@ -648,7 +648,26 @@ def silu_mul(gate: Tensor, up: Tensor) -> Tensor:
 
 
 RECURRENCE_MAX_DIM = 512   # key channels per head that one launch of the prompt kernel covers
+BONUS_MAX_DIM = 256        # ... under the rule with a decay per channel
 LATENT_MAX_RANK = 1024     # latent sizes that the decode kernel covers
+GROUPED_MAX_VDIM = 1024    # value sizes that the grouped decode kernel covers
+
+
+def _channel_blocks(run, dim: int, limit: int, heads: int, state: Optional[Tensor], rows, vectors) -> Tensor:
+    """``run(rows, vectors, state, dim)`` over blocks of at most ``limit`` key channels per head, outputs summed (key channels are
+    independent of one another). ``rows`` ``[n, heads * dim]``, ``vectors`` ``[heads * dim]``."""
+    if dim <= limit:
+        return run(rows, vectors, state, dim)
+    out = None
+    for a in range(0, dim, limit):
+        b = min(dim, a + limit)
+        cut = lambda t: t.reshape(-1, heads, dim)[:, :, a:b].reshape(t.size(0), -1)            # noqa: E731
+        part = state[:, :, a:b].contiguous() if state is not None else None
+        o = run([cut(t) for t in rows], [cut(t[None])[0].contiguous() for t in vectors], part, b - a)
+        if state is not None:
+            state[:, :, a:b] = part
+        out = o if out is None else out + o
+    return out
 
 
 def gated_recurrence(q: Tensor, f: Tensor, v: Tensor, f_bias: Tensor, lower: Tensor, norm_w: Tensor, eps: float, batch: int,
@@ -657,20 +676,111 @@ def gated_recurrence(q: Tensor, f: Tensor, v: Tensor, f_bias: Tensor, lower: Ten
     if q.size(0) == batch and state is not None:      # one token per sequence
         return _ext().recurrence_step(_rows(q), _rows(f), _rows(v), f_bias, lower, norm_w, _keep8(keep), state, float(eps), heads,
                                       dim, vdim)
-    if dim > RECURRENCE_MAX_DIM:      # key channels are independent of one another: sum the outputs of blocks of them
-        o = None
-        for a in range(0, dim, RECURRENCE_MAX_DIM):
-            b = min(dim, a + RECURRENCE_MAX_DIM)
-            cut = lambda t: t.reshape(-1, heads, dim)[:, :, a:b].reshape(t.size(0), -1)            # noqa: E731
-            part = state[:, :, a:b].contiguous() if state is not None else None
-            ob = _ext().recurrence(cut(q), cut(f), _rows(v), cut(f_bias[None])[0].contiguous(), cut(lower[None])[0].contiguous(),
-                                   _keep8(keep), part, batch, heads, b - a, vdim)
-            if state is not None:
-                state[:, :, a:b] = part
-            o = ob if o is None else o + ob
-    else:
-        o = _ext().recurrence(_rows(q), _rows(f), _rows(v), f_bias, lower, _keep8(keep), state, batch, heads, dim, vdim)
+    run = lambda r, w, s, d: _ext().recurrence(r[0], r[1], _rows(v), w[0], w[1], _keep8(keep), s, batch, heads, d, vdim)   # noqa: E731
+    o = _channel_blocks(run, dim, RECURRENCE_MAX_DIM, heads, state, [_rows(q), _rows(f)], [f_bias, lower])
     return _ext().rms_norm(o.view(-1, vdim), norm_w, float(eps), 0.0).view(-1, heads * vdim)
+
+
+def decayed_attention(q: Tensor, k: Tensor, v: Tensor, decay: Tensor, keep: Optional[Tensor], state: Optional[Tensor], batch: int,
+                      heads: int) -> Tensor:
+    dim, vdim = q.size(1) // heads, v.size(1) // heads
+    q, k, v, keep = _rows(q), _rows(k), _rows(v), _keep8(keep)
+    if q.size(0) == batch and state is not None:
+        return _ext().decayed_step(q, k, v, decay, keep, state, heads, dim, vdim)
+    run = lambda r, w, s, d: _ext().decayed_recurrence(r[0], r[1], v, decay, keep, s, batch, heads, d, vdim)                # noqa: E731
+    return _channel_blocks(run, dim, RECURRENCE_MAX_DIM, heads, state, [q, k], []).view(q.size(0), -1)
+
+
+def bonus_recurrence(r: Tensor, k: Tensor, v: Tensor, z: Tensor, w0: Tensor, u: Tensor, keep: Optional[Tensor],
+                     state: Optional[Tensor], batch: int, heads: int) -> Tensor:
+    dim, vdim = r.size(1) // heads, v.size(1) // heads
+    v, keep = _rows(v), _keep8(keep)
+    run = lambda x, w, s, d: _ext().bonus_recurrence(x[0], x[1], v, x[2], w[0], w[1], keep, s, batch, heads, d, vdim)       # noqa: E731
+    return _channel_blocks(run, dim, BONUS_MAX_DIM, heads, state, [_rows(r), _rows(k), _rows(z)], [w0, u]).view(r.size(0), -1)
+
+
+def bonus_step(r: Tensor, k: Tensor, v: Tensor, t: Tensor, w2: Tensor, w0: Tensor, u: Tensor, norm_w: Tensor, gate: Tensor,
+               keep: Optional[Tensor], state: Tensor, eps: float, heads: int) -> Tensor:
+    """Decode step: decay projection, recurrence, head norms and gate in one launch; ``t`` is ``W_w1 mix`` before its tanh."""
+    return _ext().bonus_step(_rows(r), _rows(k), _rows(v), _rows(t), w2, w0, u, norm_w, _rows(gate), _keep8(keep), state, float(eps),
+                             heads, r.size(1) // heads, v.size(1) // heads)
+
+
+def linear_fp32(x: Tensor, weight: Tensor) -> Tensor:
+    if gemm_ok(x, weight) and weight.dtype == x.dtype:
+        return gemm(x, weight, flags=FLAG_OUT_FP32)
+    return torch.matmul(x.float(), weight.float().t())
+
+
+def stacked_linear(x: Tensor, weight: Tensor) -> Tensor:
+    parts, rows, _ = x.shape
+    if gemm_ok(x[0], weight[0]) and weight.size(1) % 8 == 0:
+        if rows <= GEMV_ROWS:
+            return _ext().gemv_stacked(x, weight)
+        out = torch.empty(parts, rows, weight.size(1), dtype=x.dtype, device=x.device)
+        for i in range(parts):
+            if rows <= SMALL_M_ROWS:
+                out[i] = _ext().gemm_small_m(x[i], weight[i], 0, None, -1)
+            else:
+                gemm(x[i], weight[i], out=out[i])
+        return out
+    return torch.matmul(x, weight.transpose(1, 2))
+
+
+def branch_join(x: Tensor, branches, mult: float, eps: float, w_next):
+    args = [a for y, w, factor in branches for a in (_rows(y), w, float(factor))]
+    args += [None, None, 1.0] * (3 - len(branches))
+    w = list(w_next) + [None] * (2 - len(w_next))
+    xo, h1, h2 = _ext().branch_join(x.contiguous(), *args, float(mult), float(eps), w[0], w[1])
+    return xo, [h1, h2][:len(w_next)]
+
+
+def clamped_glu(gate: Tensor, up: Tensor, limit: float, alpha: float) -> Tensor:
+    return _ext().clamped_glu(_rows(gate), _rows(up), float(limit), float(alpha))
+
+
+def gated_rms_norm(o: Tensor, w: Tensor, gate: Tensor, eps: float, group: int, act: str) -> Tensor:
+    return _ext().gated_rms_norm(o.contiguous(), w, _rows(gate), float(eps), int(group), {"sigmoid": 0, "silu": 1}[act])
+
+
+def token_shift(h: Tensor, mu: Tensor, batch: int, keep: Optional[Tensor], prev: Optional[Tensor]) -> Tensor:
+    return _ext().token_shift(_rows(h), mu, batch, _keep8(keep), prev)
+
+
+def causal_conv_silu(x: Tensor, w: Tensor, bias: Tensor, batch: int, keep: Optional[Tensor], prev: Optional[Tensor]) -> Tensor:
+    return _ext().causal_conv_silu(_rows(x), w, bias, batch, _keep8(keep), prev)
+
+
+SCAN_MAX_STATES = 256   # states per channel that one launch of the prompt scan covers
+
+
+def selective_scan(x: Tensor, dt: Tensor, dt_bias: Tensor, a_log: Tensor, b: Tensor, c: Tensor, d: Tensor, z: Tensor, batch: int,
+                   keep: Optional[Tensor], state: Optional[Tensor]) -> Tensor:
+    if a_log.size(1) > SCAN_MAX_STATES:
+        y, final = ref.selective_scan(x, dt, dt_bias, a_log, b, c, d, z, batch, keep, state)
+        if state is not None:
+            state.copy_(final)
+        return y
+    return _ext().selective_scan(_rows(x), _rows(dt), dt_bias, a_log, _rows(b), _rows(c), d, _rows(z), batch, _keep8(keep), state)
+
+
+def scan_step(x: Tensor, dt: Tensor, w_dt: Tensor, dt_bias: Tensor, a_log: Tensor, b: Tensor, c: Tensor, d: Tensor, z: Tensor,
+              keep: Optional[Tensor], state: Tensor) -> Tensor:
+    """Decode step: step projection ``w_dt dt``, state update, gate in one launch."""
+    return _ext().scan_step(_rows(x), _rows(dt), w_dt, dt_bias, a_log, _rows(b), _rows(c), d, _rows(z), _keep8(keep), state)
+
+
+def qkv_prep(q: Tensor, k: Tensor, v: Tensor, wq: Tensor, wk: Tensor, eps: float, positions: Tensor, freq: Tensor, k_store: Tensor,
+             v_store: Tensor, lengths: Tensor) -> Tensor:
+    """Head norms and rotation of queries and keys; keys and values go into the caches at ``lengths[row]``. Returns ``[B, S, H, dim]``."""
+    return _ext().qkv_prep(_rows(q), _rows(k), _rows(v), wq, wk, float(eps), positions, freq, k_store, v_store, lengths)
+
+
+def grouped_decode(q: Tensor, k: Tensor, v: Tensor, lengths: Tensor, keep: Optional[Tensor], sink: Tensor, scale: float,
+                   softcap: float) -> Tensor:
+    if v.size(-1) > GROUPED_MAX_VDIM:
+        return ref.grouped_decode(q, k, v, lengths, keep, sink, scale, softcap)
+    return _ext().grouped_decode(q.contiguous(), k, v, lengths, _keep8(keep), sink, float(scale), float(softcap))
 
 
 def flash_head_dim(dim: int, vdim: int) -> int:
@@ -683,19 +793,24 @@ def pad_heads(t: Tensor, d: int) -> Tensor:
     return t if t.size(-1) == d else torch.nn.functional.pad(t, (0, d - t.size(-1)))
 
 
-def sink_attention(q: Tensor, k: Tensor, v: Tensor, keep: Optional[Tensor], sink: Tensor, gate: Tensor, scale: float) -> Tensor:
-    """``q``/``k``/``v`` ``[B, S, H, *]``. 16-bit heads run on the tcgen05 flash kernel (zero-padded to the next size it has),
-    with sink and gate in its epilogue (value sizes that are no multiple of 8: from its log-sum-exp); everything else in the fp32 kernel."""
-    d = flash_head_dim(q.size(-1), v.size(-1))
+def sink_attention(q: Tensor, k: Tensor, v: Tensor, keep: Optional[Tensor], sink: Tensor, gate: Optional[Tensor], scale: float,
+                   softcap: float = 0.0) -> Tensor:
+    """``q`` ``[B, Sq, H, dim]``, ``k``/``v`` ``[B, Sk, G, *]``. 16-bit heads run on the tcgen05 flash kernel, with sink, gate and cap
+    in its softmax and epilogue (gated value sizes that are no multiple of 8: zero-padded heads, sink and gate from its
+    log-sum-exp); everything else in the fp32 kernel."""
+    dim, vdim = q.size(-1), v.size(-1)
+    d = flash_head_dim(dim, vdim)
     if q.dtype in _16BIT and d and q.size(1) > 1:
-        qh, kh, vh = (_attn_operand(pad_heads(t, d).permute(0, 2, 1, 3)) for t in (q, k, v))
         kpm = _keep8(keep).contiguous() if keep is not None else None
-        if v.size(-1) % 8 == 0:
-            return _ext().flash_sink_fwd(qh, kh, vh, kpm, sink, _rows(gate), float(scale), v.size(-1))
-        o, lse = _ext().flash_fwd(qh, kh, vh, float(scale), True, 0, kpm, _flash_impl())
-        return _ext().sink_gate(o, lse, sink, _rows(gate), v.size(-1))
+        if dim % 8 == 0 and vdim % 8 == 0:
+            qh, kh, vh = (_attn_operand(t.permute(0, 2, 1, 3)) for t in (q, k, v))
+            return _ext().flash_sink_fwd(qh, kh, vh, kpm, sink, None if gate is None else _rows(gate), float(scale), float(softcap))
+        if gate is not None and not softcap and k.size(2) == q.size(2):
+            qh, kh, vh = (_attn_operand(pad_heads(t, d).permute(0, 2, 1, 3)) for t in (q, k, v))
+            o, lse = _ext().flash_fwd(qh, kh, vh, float(scale), True, 0, kpm, _flash_impl())
+            return _ext().sink_gate(o, lse, sink, _rows(gate), vdim)
     return _ext().sink_attention(*(t if t.stride(-1) == 1 else t.contiguous() for t in (q, k, v)), _keep8(keep), sink,
-                                 _rows(gate), float(scale))
+                                 None if gate is None else _rows(gate), float(scale), float(softcap))
 
 
 def latent_prep(cq: Tensor, wq: Tensor, ckv: Optional[Tensor], wkv: Optional[Tensor], cache: Optional[Tensor], lengths: Tensor,

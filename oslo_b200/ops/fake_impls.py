@@ -199,11 +199,11 @@ def register() -> None:
         return o.new_empty((o.size(0) * o.size(2), o.size(1) * vdim))
 
     @reg("oslo_b200::flash_sink_fwd")
-    def _(q, k, v, kpm, sink, gate, scale, vdim):
-        return q.new_empty((q.size(0) * q.size(2), q.size(1) * vdim))
+    def _(q, k, v, kpm, sink, gate, scale, softcap):
+        return q.new_empty((q.size(0) * q.size(2), q.size(1) * v.size(3)))
 
     @reg("oslo_b200::sink_attention")
-    def _(q, k, v, keep, sink, gate, scale):
+    def _(q, k, v, keep, sink, gate, scale, softcap):
         return q.new_empty((q.size(0) * q.size(1), q.size(2) * v.size(3)))
 
     @reg("oslo_b200::latent_prep")
@@ -230,3 +230,61 @@ def register() -> None:
     @reg("oslo_b200::moe_few")
     def _(x, idx, w, per_row, relu2):
         return x.new_empty((idx.numel(), w.size(1)))
+
+    @reg("oslo_b200::clamped_glu")
+    def _(gate, up, limit, alpha):
+        return gate.new_empty(gate.shape)
+
+    @reg("oslo_b200::branch_join")
+    def _(x, y0, n0, f0, y1, n1, f1, y2, n2, f2, mult, eps, w1, w2):
+        rows, cols = x.shape
+        return (torch.empty_like(x), y0.new_empty((rows if w1 is not None else 0, cols)),
+                y0.new_empty((rows if w2 is not None else 0, cols)))
+
+    @reg("oslo_b200::gated_rms_norm")
+    def _(o, w, gate, eps, group, act):
+        return w.new_empty(o.shape)
+
+    @reg("oslo_b200::gemv_stacked")
+    def _(x, w):
+        return x.new_empty((x.size(0), x.size(1), w.size(1)))
+
+    @reg("oslo_b200::decayed_recurrence")
+    def _(q, k, v, decay, keep, state, batch, heads, dim, vdim, chunks=0):
+        return q.new_empty((batch, q.size(0) // batch, heads, vdim), dtype=torch.float32)
+
+    @reg("oslo_b200::bonus_recurrence")
+    def _(q, k, v, z, w0, u, keep, state, batch, heads, dim, vdim, chunks=0):
+        return q.new_empty((batch, q.size(0) // batch, heads, vdim), dtype=torch.float32)
+
+    @reg("oslo_b200::decayed_step")
+    def _(q, k, v, decay, keep, state, heads, dim, vdim):
+        return q.new_empty((q.size(0), heads * vdim), dtype=torch.float32)
+
+    @reg("oslo_b200::bonus_step")
+    def _(r, k, v, t, w2, w0, u, norm_w, gate, keep, state, eps, heads, dim, vdim):
+        return r.new_empty((r.size(0), heads * vdim))
+
+    @reg("oslo_b200::qkv_prep")
+    def _(q, k, v, wq, wk, eps, positions, freq, kc, vc, lengths):
+        return q.new_empty((kc.size(0), q.size(0) // kc.size(0), q.size(1) // kc.size(3), kc.size(3)))
+
+    @reg("oslo_b200::grouped_decode")
+    def _(q, kc, vc, lengths, keep, sink, scale, softcap):
+        return q.new_empty((q.size(0), q.size(1) * vc.size(3)))
+
+    @reg("oslo_b200::token_shift")
+    def _(h, mu, batch, keep, prev):
+        return h.new_empty((mu.size(0), h.size(0), h.size(1)))
+
+    @reg("oslo_b200::causal_conv_silu")
+    def _(x, w, bias, batch, keep, prev):
+        return x.new_empty(x.shape)
+
+    @reg("oslo_b200::selective_scan")
+    def _(x, dt, dt_bias, a_log, b, c, d, z, batch, keep, state, chunks=0):
+        return x.new_empty(x.shape)
+
+    @reg("oslo_b200::scan_step")
+    def _(x, dt, w_dt, dt_bias, a_log, b, c, d, z, keep, state):
+        return x.new_empty(x.shape)

@@ -195,12 +195,13 @@ def gated_recurrence(q: Tensor, f: Tensor, v: Tensor, f_bias: Tensor, lower: Ten
     return ref.rms_norm(o, norm_w, eps).reshape(-1, heads * vdim)
 
 
-def sink_attention(q: Tensor, k: Tensor, v: Tensor, keep: Optional[Tensor], sink: Tensor, gate: Tensor, scale: float) -> Tensor:
+def sink_attention(q: Tensor, k: Tensor, v: Tensor, keep: Optional[Tensor], sink: Tensor, gate: Optional[Tensor], scale: float,
+                   softcap: float = 0.0) -> Tensor:
     """``reference.sink_attention`` without the weights."""
     if _kn(q, k, v, sink, gate):
         from . import cuda_ops
-        return cuda_ops.sink_attention(q, k, v, keep, sink, gate, scale)
-    return ref.sink_attention(q, k, v, keep, sink, gate, scale)[0]
+        return cuda_ops.sink_attention(q, k, v, keep, sink, gate, scale, softcap)
+    return ref.sink_attention(q, k, v, keep, sink, gate, scale, softcap)[0]
 
 
 def latent_decode(q: Tensor, w_uk: Tensor, w_uv: Tensor, cache: Tensor, lengths: Tensor, keep: Optional[Tensor], sink: Tensor,
@@ -225,3 +226,99 @@ def moe_experts(h: Tensor, idx: Tensor, up: Tensor, down: Tensor) -> Tuple[Tenso
         from . import cuda_ops
         return cuda_ops.moe_experts(h, idx, up, down)
     return ref.moe_experts(h, idx, up, down), None
+
+
+def linear_fp32(x: Tensor, weight: Tensor, fused: bool = True) -> Tensor:
+    """``x @ W.T`` with a 32-bit result whatever the storage type: what enters a decay or a step size is not rounded to 16 bits."""
+    if fused and _kn(x, weight):
+        from . import cuda_ops
+        return cuda_ops.linear_fp32(x, weight)
+    return torch.matmul(x, weight.t()).to(torch.float32)
+
+
+def stacked_linear(x: Tensor, weight: Tensor, fused: bool = True) -> Tensor:
+    """``x[i] @ W[i].T``: ``x`` ``[P, rows, in]``, ``weight`` ``[P, out, in]``."""
+    if fused and _kn(x, weight):
+        from . import cuda_ops
+        return cuda_ops.stacked_linear(x, weight)
+    return torch.matmul(x, weight.transpose(1, 2))
+
+
+def branch_join(x: Tensor, branches, mult: float, eps: float, w_next, fused: bool = True):
+    """Add the results of parallel branches to the fp32 residual stream and norm the sum once per weight of ``w_next``: one pass
+    over the rows. See ``reference.branch_join``."""
+    if fused and _kn(x, *(t for b in branches for t in b[:2]), *w_next):
+        from . import cuda_ops
+        return cuda_ops.branch_join(x, branches, mult, eps, w_next)
+    return ref.branch_join(x, branches, mult, eps, w_next)
+
+
+def clamped_glu(gate: Tensor, up: Tensor, limit: float, alpha: float, fused: bool = True) -> Tensor:
+    if fused and _kn(gate, up):
+        from . import cuda_ops
+        return cuda_ops.clamped_glu(gate, up, limit, alpha)
+    return ref.clamped_glu(gate, up, limit, alpha)
+
+
+def gated_rms_norm(o: Tensor, w: Tensor, gate: Tensor, eps: float, group: int, act: str, fused: bool = True) -> Tensor:
+    if fused and _kn(o, w, gate):
+        from . import cuda_ops
+        return cuda_ops.gated_rms_norm(o, w, gate, eps, group, act)
+    return ref.gated_rms_norm(o, w, gate, eps, group, act)
+
+
+# ``state`` / ``prev`` of the functions below (fp32) carry a sequence on: read, and updated in place.
+def decayed_attention(q: Tensor, k: Tensor, v: Tensor, decay: Tensor, keep: Optional[Tensor], state: Optional[Tensor], batch: int,
+                      heads: int, fused: bool = True) -> Tensor:
+    """``reference.decayed_attention``: ``[B * S, heads * vdim]`` in fp32."""
+    if fused and _kn(q, k, v):
+        from . import cuda_ops
+        return cuda_ops.decayed_attention(q, k, v, decay, keep, state, batch, heads)
+    o, final = ref.decayed_attention(q, k, v, decay, keep, state, batch, heads)
+    if state is not None:
+        state.copy_(final.detach())
+    return o.reshape(q.size(0), -1)
+
+
+def bonus_recurrence(r: Tensor, k: Tensor, v: Tensor, z: Tensor, w0: Tensor, u: Tensor, keep: Optional[Tensor],
+                     state: Optional[Tensor], batch: int, heads: int, fused: bool = True) -> Tensor:
+    """``reference.bonus_recurrence``: ``[B * S, heads * vdim]`` in fp32."""
+    if fused and _kn(r, k, v, z, w0, u):
+        from . import cuda_ops
+        return cuda_ops.bonus_recurrence(r, k, v, z, w0, u, keep, state, batch, heads)
+    o, final = ref.bonus_recurrence(r, k, v, z, w0, u, keep, state, batch, heads)
+    if state is not None:
+        state.copy_(final.detach())
+    return o.reshape(r.size(0), -1)
+
+
+def token_shift(h: Tensor, mu: Tensor, batch: int, keep: Optional[Tensor], prev: Optional[Tensor], fused: bool = True) -> Tensor:
+    if fused and _kn(h, mu):
+        from . import cuda_ops
+        return cuda_ops.token_shift(h, mu, batch, keep, prev)
+    mixed, last = ref.token_shift(h, mu, batch, keep, prev)
+    if prev is not None:
+        prev.copy_(last.detach())
+    return mixed
+
+
+def causal_conv_silu(x: Tensor, w: Tensor, bias: Tensor, batch: int, keep: Optional[Tensor], prev: Optional[Tensor],
+                     fused: bool = True) -> Tensor:
+    if fused and _kn(x, w, bias):
+        from . import cuda_ops
+        return cuda_ops.causal_conv_silu(x, w, bias, batch, keep, prev)
+    y, last = ref.causal_conv_silu(x, w, bias, batch, keep, prev)
+    if prev is not None:
+        prev.copy_(last.detach())
+    return y
+
+
+def selective_scan(x: Tensor, dt: Tensor, dt_bias: Tensor, a_log: Tensor, b: Tensor, c: Tensor, d: Tensor, z: Tensor, batch: int,
+                   keep: Optional[Tensor], state: Optional[Tensor], fused: bool = True) -> Tensor:
+    if fused and _kn(x, dt, dt_bias, a_log, b, c, d, z):
+        from . import cuda_ops
+        return cuda_ops.selective_scan(x, dt, dt_bias, a_log, b, c, d, z, batch, keep, state)
+    y, final = ref.selective_scan(x, dt, dt_bias, a_log, b, c, d, z, batch, keep, state)
+    if state is not None:
+        state.copy_(final.detach())
+    return y

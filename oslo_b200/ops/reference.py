@@ -232,13 +232,19 @@ def recurrence(q: Tensor, f: Tensor, v: Tensor, f_bias: Tensor, lower: Tensor, k
     return torch.stack(out, dim=1), s
 
 
-def sink_attention(q: Tensor, k: Tensor, v: Tensor, keep: Optional[Tensor], sink: Tensor, gate: Tensor, scale: float):
-    """Causal softmax attention whose denominator also holds ``exp(sink[head])``; head ``h``'s output times
-    ``sigmoid(gate[:, h])``. ``q`` ``[B, Sq, H, D]`` are the last positions of ``k``/``v`` ``[B, Sk, H, *]``; ``keep``
-    ``[B, Sk]``; ``gate`` ``[B * Sq, H]``. Returns ``[B * Sq, H * Dv]`` and the weights ``[B, H, Sq, Sk]``."""
+def sink_attention(q: Tensor, k: Tensor, v: Tensor, keep: Optional[Tensor], sink: Tensor, gate: Optional[Tensor], scale: float,
+                   softcap: float = 0.0):
+    """Causal softmax attention whose denominator also holds ``exp(sink[head])``; with ``gate`` ``[B * Sq, H]`` head ``h``'s
+    output is multiplied by ``sigmoid(gate[:, h])``, with ``softcap`` scores become ``softcap * tanh(score / softcap)``. ``q``
+    ``[B, Sq, H, D]`` are the last positions of ``k``/``v`` ``[B, Sk, G, *]``; query head ``h`` reads key head ``h // (H / G)``;
+    ``keep`` ``[B, Sk]``. Returns ``[B * Sq, H * Dv]`` and the weights ``[B, H, Sq, Sk]``."""
     b, sq, h, _ = q.shape
-    sk = k.size(1)
+    sk, per = k.size(1), h // k.size(2)
+    if per > 1:
+        k, v = k.repeat_interleave(per, dim=2), v.repeat_interleave(per, dim=2)
     s = torch.einsum("bqhd,bkhd->bhqk", q.to(torch.float32), k.to(torch.float32)) * scale
+    if softcap:
+        s = softcap * torch.tanh(s / softcap)
     vis = attention_mask_bias(sq, sk, q.device, True, None)[None, None]
     if keep is not None:
         vis = vis & (keep != 0)[:, None, None, :]
@@ -246,7 +252,8 @@ def sink_attention(q: Tensor, k: Tensor, v: Tensor, keep: Optional[Tensor], sink
     s = torch.cat([s, sink.to(torch.float32)[None, :, None, None].expand(b, h, sq, 1)], dim=-1)
     p = torch.softmax(s, dim=-1)[..., :sk]
     o = torch.einsum("bhqk,bkhd->bqhd", p, v.to(torch.float32))
-    o = o * torch.sigmoid(gate.to(torch.float32)).view(b, sq, h, 1)
+    if gate is not None:
+        o = o * torch.sigmoid(gate.to(torch.float32)).view(b, sq, h, 1)
     return o.reshape(b * sq, -1).to(q.dtype), p
 
 
@@ -289,3 +296,161 @@ def moe_experts(h: Tensor, idx: Tensor, up: Tensor, down: Tensor) -> Tensor:
         a = torch.relu(torch.matmul(rows[at], up[e].t())).pow(2)
         out = out.index_copy(0, at, torch.matmul(a, down[e].t()).to(out.dtype))
     return out
+
+
+# ---------------------------------------------------------------------------------------------------------------
+# Residual joins of parallel branches, grouped-query attention, linear recurrences with decays of their own, token shift,
+# causal convolution, selective scan, clamped gated units.
+def branch_join(x: Tensor, branches, mult: float, eps: float, w_next) -> Tuple[Tensor, list]:
+    """``x + mult * sum(factor * y)`` over ``branches`` ``[(y, w, factor), ...]`` in fp32, ``y`` first RMS-normed with weight ``w``
+    unless that is ``None``; and the RMS norms of the sum with every weight of ``w_next``."""
+    total = None
+    for y, w, factor in branches:
+        yf = y.to(torch.float32)
+        if w is not None:
+            yf = yf * torch.rsqrt(yf.pow(2).mean(-1, keepdim=True) + eps) * w.to(torch.float32)
+        yf = yf if factor == 1.0 else yf * factor
+        total = yf if total is None else total + yf
+    x = x + mult * total
+    return x, [rms_norm(x, w, eps) for w in w_next]
+
+
+def clamped_glu(gate: Tensor, up: Tensor, limit: float, alpha: float) -> Tensor:
+    """``g sigmoid(alpha g) (u + 1)`` with ``g = min(gate, limit)``, ``u = clamp(up, -limit, limit)``."""
+    g = gate.to(torch.float32).clamp(max=limit)
+    u = up.to(torch.float32).clamp(-limit, limit)
+    return (g * torch.sigmoid(alpha * g) * (u + 1.0)).to(up.dtype)
+
+
+def rotary_frequencies(rot_dims: int, base: float):
+    """``base^(-2i / rot_dims)`` for the pairs of the rotated dims, as 32-bit floats rounded once."""
+    return [base ** (-2.0 * i / rot_dims) for i in range(rot_dims // 2)]
+
+
+def norm_rotate(x: Tensor, w: Optional[Tensor], eps: float, positions: Tensor, freq: Optional[Tensor]) -> Tensor:
+    """Per head of ``x`` ``[B, S, heads, D]``: RMS norm with weight ``w`` ``[D]`` (shared by the heads), then the interleaved
+    rotation of the first ``2 * len(freq)`` dims by ``positions * freq`` (fp32); ``positions`` ``[B, S]``."""
+    y = x.to(torch.float32)
+    if w is not None:
+        y = y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + eps) * w.to(torch.float32)
+    if freq is not None and freq.numel():
+        r = 2 * freq.numel()
+        ang = (positions.to(torch.float32).unsqueeze(-1) * freq).unsqueeze(2)
+        sin, cos = torch.sin(ang), torch.cos(ang)
+        a, b = y[..., :r:2], y[..., 1:r:2]
+        y = torch.cat((torch.stack((a * cos - b * sin, b * cos + a * sin), dim=-1).flatten(-2), y[..., r:]), dim=-1)
+    return y.to(x.dtype)
+
+
+def grouped_decode(q: Tensor, k: Tensor, v: Tensor, lengths: Tensor, keep: Optional[Tensor], sink: Tensor, scale: float,
+                   softcap: float = 0.0) -> Tensor:
+    """One query per row: ``q`` ``[B, H, D]`` over caches ``[B, G, T, *]`` of which the first ``lengths[b]`` positions count;
+    ``keep`` ``[B, <= T]``. Softmax with a sink as in ``sink_attention``. Returns ``[B, H * Dv]``."""
+    b, h, _ = q.shape
+    g, t = k.size(1), k.size(2)
+    vis = torch.arange(t, device=q.device)[None, :] < lengths[:, None]
+    if keep is not None:
+        n = min(t, keep.size(1))
+        vis[:, :n] &= keep[:, :n] != 0
+    qg = q.to(torch.float32).view(b, g, h // g, -1)
+    s = torch.einsum("bgrd,bgtd->bgrt", qg, k.to(torch.float32)) * scale
+    if softcap:
+        s = softcap * torch.tanh(s / softcap)
+    s = s.masked_fill(~vis[:, None, None, :], float("-inf"))
+    s = torch.cat([s, sink.to(torch.float32).view(1, g, h // g, 1).expand(b, g, h // g, 1)], dim=-1)
+    p = torch.softmax(s, dim=-1)[..., :t]
+    # positions beyond the length may hold anything
+    vf = torch.where(vis[:, None, :, None], v.to(torch.float32), torch.zeros((), device=v.device))
+    return torch.einsum("bgrt,bgtd->bgrd", p, vf).reshape(b, -1).to(q.dtype)
+
+
+def gated_rms_norm(o: Tensor, w: Tensor, gate: Tensor, eps: float, group: int, act: str) -> Tensor:
+    """Every run of ``group`` columns of ``o`` ``[rows, n]`` divided by its root mean square, times ``w`` ``[n]``, times
+    ``sigmoid(gate)`` or ``silu(gate)`` (``act``); in ``w``'s dtype."""
+    of = o.to(torch.float32).reshape(o.size(0), -1, group)
+    of = (of * torch.rsqrt(of.pow(2).mean(-1, keepdim=True) + eps)).view(o.size(0), -1)
+    g = gate.to(torch.float32)
+    g = torch.sigmoid(g) if act == "sigmoid" else F.silu(g)
+    return (of * w.to(torch.float32) * g).to(w.dtype)
+
+
+def decayed_attention(q: Tensor, k: Tensor, v: Tensor, decay: Tensor, keep: Optional[Tensor], state: Optional[Tensor],
+                      batch: int, heads: int) -> Tuple[Tensor, Tensor]:
+    """Linear attention with one constant decay per head: ``S <- decay S + silu(k) silu(v)^T``, ``o = S^T silu(q)``. ``q``, ``k``
+    ``[B * S, heads * dim]``, ``v`` ``[B * S, heads * vdim]``; ``keep`` ``[B, S]``: a padded token leaves the state as it is.
+    Returns ``o`` ``[B, S, heads, vdim]`` (fp32) and the final state ``[B, heads, dim, vdim]``."""
+    qf, kf, vf = (F.silu(t.to(torch.float32)).view(batch, -1, heads, t.size(1) // heads) for t in (q, k, v))
+    s = torch.zeros(batch, heads, kf.size(-1), vf.size(-1), device=q.device) if state is None else state
+    dec = decay.to(torch.float32).view(1, heads, 1, 1)
+    out = []
+    for t in range(kf.size(1)):
+        new = dec * s + kf[:, t].unsqueeze(-1) * vf[:, t].unsqueeze(-2)
+        s = new if keep is None else torch.where((keep[:, t] != 0).view(-1, 1, 1, 1), new, s)
+        out.append(torch.einsum("bhi,bhij->bhj", qf[:, t], s))
+    o = torch.stack(out, dim=1)
+    return (o if keep is None else o * (keep != 0).to(torch.float32)[:, :, None, None]), s
+
+
+def bonus_recurrence(r: Tensor, k: Tensor, v: Tensor, z: Tensor, w0: Tensor, u: Tensor, keep: Optional[Tensor],
+                     state: Optional[Tensor], batch: int, heads: int) -> Tuple[Tensor, Tensor]:
+    """Linear attention with a decay per token, head and key channel, ``w = exp(-exp(z + w0))``: a token reads the state before it
+    and itself with a bonus, ``o = S^T r + (r . (u k)) v``, then ``S <- diag(w) S + k v^T``. ``r``, ``k``, ``z`` ``[B * S, heads *
+    dim]``, ``v`` ``[B * S, heads * vdim]``, ``w0``, ``u`` ``[heads * dim]``. Returns as ``decayed_attention``."""
+    rf, kf, vf = (t.to(torch.float32).view(batch, -1, heads, t.size(1) // heads) for t in (r, k, v))
+    w = torch.exp(-torch.exp(z.to(torch.float32) + w0.to(torch.float32))).view(kf.shape)
+    s = torch.zeros(batch, heads, kf.size(-1), vf.size(-1), device=r.device) if state is None else state
+    bonus = (rf * u.to(torch.float32).view(heads, -1) * kf).sum(-1, keepdim=True) * vf
+    out = []
+    for t in range(kf.size(1)):
+        out.append(torch.einsum("bhi,bhij->bhj", rf[:, t], s) + bonus[:, t])
+        new = w[:, t].unsqueeze(-1) * s + kf[:, t].unsqueeze(-1) * vf[:, t].unsqueeze(-2)
+        s = new if keep is None else torch.where((keep[:, t] != 0).view(-1, 1, 1, 1), new, s)
+    o = torch.stack(out, dim=1)
+    return (o if keep is None else o * (keep != 0).to(torch.float32)[:, :, None, None]), s
+
+
+def token_shift(h: Tensor, mu: Tensor, batch: int, keep: Optional[Tensor], prev: Optional[Tensor]) -> Tuple[Tensor, Tensor]:
+    """``h + (h' - h) mu[i]`` for every row of ``mu`` ``[P, width]``, with ``h'`` the row of the token before (``prev`` ``[B, width]``
+    before the first one; zeros at the start of a sequence and after padding). Returns ``[P, B * S, width]`` and the last rows."""
+    hb = h.view(batch, -1, h.size(-1)).to(torch.float32)
+    if keep is not None:
+        hb = hb * (keep != 0).to(torch.float32).unsqueeze(-1)
+    first = torch.zeros_like(hb[:, 0]) if prev is None else prev
+    before = torch.cat([first.unsqueeze(1), hb[:, :-1]], dim=1)
+    m = mu.to(torch.float32).view(mu.size(0), 1, 1, -1)
+    return (hb + (before - hb) * m).to(h.dtype).view(mu.size(0), h.size(0), -1), hb[:, -1]
+
+
+def causal_conv_silu(x: Tensor, w: Tensor, bias: Tensor, batch: int, keep: Optional[Tensor],
+                     prev: Optional[Tensor]) -> Tuple[Tensor, Tensor]:
+    """``silu`` of a causal convolution per channel: ``x`` ``[B * S, C]``, ``w`` ``[C, taps]`` with the current token's tap last,
+    ``prev`` ``[B, taps - 1, C]`` the inputs before (zeros when ``None``). Returns the result and the last ``taps - 1`` inputs."""
+    taps = w.size(1)
+    xb = x.view(batch, -1, x.size(-1)).to(torch.float32)
+    if keep is not None:
+        xb = xb * (keep != 0).to(torch.float32).unsqueeze(-1)
+    s = xb.size(1)
+    head = xb.new_zeros(batch, taps - 1, xb.size(-1)) if prev is None else prev
+    full = torch.cat([head, xb], dim=1)
+    y = bias.to(torch.float32) + sum(w[:, j].to(torch.float32) * full[:, j:j + s] for j in range(taps))
+    return F.silu(y).to(x.dtype).reshape(x.shape), full[:, s:]
+
+
+def selective_scan(x: Tensor, dt: Tensor, dt_bias: Tensor, a_log: Tensor, b: Tensor, c: Tensor, d: Tensor, z: Tensor, batch: int,
+                   keep: Optional[Tensor], state: Optional[Tensor]) -> Tuple[Tensor, Tensor]:
+    """Per channel ``i`` and state ``n``: ``S <- exp(t A) S + t x B_n`` with the step ``t = softplus(dt + dt_bias)`` and ``A =
+    -exp(a_log)``; ``y = sum_n S C_n + d x``, times ``silu(z)``. ``x``, ``dt``, ``z`` ``[B * S, C]``, ``b``, ``c`` ``[B * S, N]``,
+    ``a_log`` ``[C, N]``. A padded token leaves the state as it is. Returns ``[B * S, C]`` and the state ``[B, C, N]``."""
+    step = F.softplus(dt.to(torch.float32) + dt_bias.to(torch.float32), threshold=30.0).view(batch, -1, x.size(-1))
+    if keep is not None:
+        step = step * (keep != 0).to(torch.float32).unsqueeze(-1)
+    a = -torch.exp(a_log.to(torch.float32))
+    xf = x.to(torch.float32).view(step.shape)
+    bf, cf = (t.to(torch.float32).view(batch, -1, t.size(-1)) for t in (b, c))
+    s = torch.zeros(batch, *a_log.shape, device=x.device) if state is None else state
+    out = []
+    for t in range(step.size(1)):
+        s = torch.exp(step[:, t].unsqueeze(-1) * a) * s + (step[:, t] * xf[:, t]).unsqueeze(-1) * bf[:, t].unsqueeze(1)
+        out.append(torch.einsum("bcn,bn->bc", s, cf[:, t]))
+    y = torch.stack(out, dim=1) + d.to(torch.float32) * xf
+    return (y.reshape(x.shape) * F.silu(z.to(torch.float32))).to(x.dtype), s

@@ -127,6 +127,19 @@ class PackedLinear(Linear):
         return {name: y[..., start:start + size] for name, (start, size) in self.parts.items()}
 
 
+class StackedLinear(nn.Module):
+    """Bias-free projections of equal size whose inputs differ: weight ``[parts, out, in]``, ``x`` ``[parts, rows, in]``."""
+
+    oslo_fused = False
+
+    def __init__(self, parts: int, in_features: int, out_features: int) -> None:
+        super().__init__()
+        self.weight = nn.Parameter(torch.empty(parts, out_features, in_features).normal_(std=0.02))
+
+    def forward(self, x: Tensor) -> Tensor:
+        return ops.stacked_linear(x, self.weight, fused=self.oslo_fused)
+
+
 class Embedding(nn.Embedding):
     oslo_fused = False
 

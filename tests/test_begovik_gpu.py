@@ -1,0 +1,285 @@
+"""The kernels behind Begovik against the fp32 PyTorch statements of the same ops, over sizes that do and do not fit the
+vector widths and tiles, and the whole model on the GPU against the plain implementation in ``plain_begovik.py``."""
+import math
+
+import pytest
+import torch
+
+import oslo_b200 as ob
+from oslo_b200 import ops
+from oslo_b200.generation import BatchSteps, GraphedGreedyDecoder
+from oslo_b200.models.common import StaticKVCache
+from oslo_b200.ops import reference as ref
+
+from . import plain_begovik as plain
+from .begovik_cases import CASES, attn, case, dense, far_key_weights, lin, make_tensors, mamba, parallel, wkv, write_model
+
+pytestmark = pytest.mark.gpu
+DTYPES = [torch.float32, torch.bfloat16, torch.float16]
+TOL = {torch.float32: 2e-5, torch.bfloat16: 2e-2, torch.float16: 3e-3}
+
+
+def rnd(*shape, dtype=torch.float32, scale=1.0, seed=0):
+    g = torch.Generator().manual_seed(seed + 7919 * len(shape) + sum(shape))
+    return (torch.randn(*shape, generator=g) * scale).to(dtype).cuda()
+
+
+def close(got, want, dtype, factor=1.0):
+    got, want = got.float(), want.float()
+    assert got.shape == want.shape
+    assert torch.isfinite(got).all()
+    scale = want.abs().amax().clamp(min=1e-3)
+    err = ((got - want).abs().amax() / scale).item()
+    assert err < factor * TOL[dtype], err
+
+
+def some_padding(batch, s):
+    """The last row as it is, the others with padding on the left."""
+    keep = torch.ones(batch, s, dtype=torch.uint8, device="cuda")
+    for b in range(batch - 1):
+        keep[b, :min(s - 1, 3 + 14 * b)] = 0
+    return keep
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("rows,cols", [(1, 256), (7, 100), (33, 1024), (5, 37), (129, 512), (3, 4096)])
+def test_branch_join(dtype, rows, cols):
+    x = rnd(rows, cols)
+    ys = [rnd(rows, cols + 8, dtype=dtype, seed=i, scale=1.0 + i)[:, :cols] for i in range(3)]
+    ws = [rnd(cols, dtype=dtype, seed=9 + i) for i in range(4)]
+    for branches in ([(ys[0], None, 1.0)], [(ys[0], None, 1.0), (ys[1], None, 1.0)],
+                     [(ys[0], ws[0], 0.5), (ys[1], ws[1], 0.5), (ys[2], None, 1.0)], [(ys[2], ws[1], 0.5), (ys[1], ws[0], 0.5)]):
+        for nxt in ([], [ws[2]], [ws[2], ws[3]]):
+            x1, h1 = ops.branch_join(x, branches, 0.3, 1e-4, nxt)
+            x2, h2 = ref.branch_join(x, branches, 0.3, 1e-4, nxt)
+            assert x1.dtype == torch.float32 and len(h1) == len(nxt)
+            close(x1, x2, torch.float32)                  # the stream is 32-bit whatever the storage type
+            for a, b in zip(h1, h2):
+                close(a, b, dtype)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("cols", [96, 50, 2048])
+def test_clamped_glu(dtype, cols):
+    t = rnd(9, 2 * cols + 8, dtype=dtype, scale=2.0)
+    for limit in (0.5, 7.0):
+        close(ops.clamped_glu(t[:, :cols], t[:, cols:2 * cols], limit, 1.702), ref.clamped_glu(t[:, :cols], t[:, cols:2 * cols], limit, 1.702), dtype)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("rows,groups,group", [(1, 3, 64), (70, 2, 128), (5, 7, 9), (3, 1, 2048), (11, 2, 700), (9, 4, 24)])
+def test_gated_rms_norm(dtype, rows, groups, group):
+    n = groups * group
+    o, w, gate = rnd(rows, n), rnd(n, dtype=dtype), rnd(rows, n + 8, dtype=dtype)[:, :n]
+    for act in ("sigmoid", "silu"):
+        close(ops.gated_rms_norm(o, w, gate, 1e-3, group, act), ref.gated_rms_norm(o, w, gate, 1e-3, group, act), dtype)
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("batch,s,heads,dim,vdim", [(2, 37, 3, 40, 72), (1, 1, 2, 16, 8), (1, 200, 1, 12, 20), (2, 17, 2, 100, 33),
+                                                    (1, 150, 2, 128, 128), (3, 50, 1, 256, 24), (1, 9, 1, 300, 40), (2, 64, 2, 64, 64)])
+def test_recurrences_with_decays_of_their_own(dtype, batch, s, heads, dim, vdim):
+    n = batch * s
+    p = rnd(n, 2 * heads * dim + heads * vdim + 8, dtype=dtype)
+    q, k, v = p[:, :heads * dim], p[:, heads * dim:2 * heads * dim], p[:, 2 * heads * dim:2 * heads * dim + heads * vdim]
+    ext = ops.load_ext(required=True)
+    s0 = rnd(batch, heads, dim, vdim, scale=0.5)
+    z, w0, u = rnd(n, heads * dim, scale=2.0), rnd(heads * dim, dtype=dtype) - 2.0, rnd(heads * dim, dtype=dtype)
+    decay = torch.tensor([0.999, 0.3, 0.0, 1e-3, 0.05, 1.0][:heads], device="cuda")
+    for kp in (None, some_padding(batch, s)):
+        for start in (None, s0):
+            for name in ("decayed", "bonus"):
+                if name == "decayed":
+                    want, end = ref.decayed_attention(q, k, v, decay, kp, start, batch, heads)
+                    run = lambda st, ch: ext.decayed_recurrence(q, k, v, decay, kp, st, batch, heads, dim, vdim, ch)           # noqa: E731
+                else:
+                    want, end = ref.bonus_recurrence(q, k, v, z, w0, u, kp, start, batch, heads)
+                    run = lambda st, ch: ext.bonus_recurrence(q, k, v, z, w0, u, kp, st, batch, heads, dim, vdim, ch)          # noqa: E731
+                for chunks in (0, 1, 2, 5):
+                    if name == "bonus" and dim > 256:     # blocks of key channels
+                        st = start.clone() if start is not None else torch.zeros_like(s0)
+                        got = ops.bonus_recurrence(q, k, v, z, w0, u, kp, st, batch, heads).view(want.shape)
+                    else:
+                        st = start.clone() if start is not None else torch.zeros_like(s0)
+                        got = run(st, chunks)
+                    close(got, want, torch.float32, 2.0)
+                    close(st, end, torch.float32, 2.0)
+
+
+def test_every_decay_keeps_its_precision_in_the_scaled_form():
+    """Decays from 0 to 1: the periods within which the state is kept relative differ, the result does not."""
+    ext = ops.load_ext(required=True)
+    for d in (0.0, 1e-30, 1e-9, 1e-4, 0.01, 0.1, 0.12, 0.5, 0.9, 0.9999, 1.0):
+        q, k, v = (rnd(1 * 100, 32, seed=i) for i in range(3))
+        decay = torch.tensor([d, d], device="cuda")
+        st, want = torch.zeros(1, 2, 16, 16, device="cuda"), None
+        want, end = ref.decayed_attention(q, k, v, decay, None, None, 1, 2)
+        for chunks in (1, 3):
+            st.zero_()
+            close(ext.decayed_recurrence(q, k, v, decay, None, st, 1, 2, 16, 16, chunks), want, torch.float32)
+            close(st, end, torch.float32)
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("batch,heads,dim,vdim,rank", [(1, 5, 40, 72, 24), (5, 3, 20, 30, 7), (2, 16, 128, 128, 64), (70, 2, 64, 256, 33),
+                                                       (1, 1, 7, 2100, 1)])
+def test_steps_are_one_token_of_the_recurrences(dtype, batch, heads, dim, vdim, rank):
+    from oslo_b200.ops import cuda_ops
+    p = rnd(batch, 2 * heads * dim + heads * vdim + 8, dtype=dtype)
+    q, k, v = p[:, :heads * dim], p[:, heads * dim:2 * heads * dim], p[:, 2 * heads * dim:2 * heads * dim + heads * vdim]
+    s0 = rnd(batch, heads, dim, vdim)
+    decay = torch.linspace(0.0, 1.0, heads, device="cuda")
+    t, w2 = rnd(batch, rank, dtype=dtype), rnd(heads * dim, rank, dtype=dtype, scale=rank ** -0.5)
+    w0, u = rnd(heads * dim, dtype=dtype) - 1.0, rnd(heads * dim, dtype=dtype)
+    nw, gate = rnd(heads * vdim, dtype=dtype), rnd(batch, heads * vdim, dtype=dtype, seed=4)
+    z = torch.tanh(t.float()).to(dtype).float() @ w2.float().t()
+    for keep in (None, (torch.arange(batch, device="cuda") % 2 == 0).to(torch.uint8)[:, None]):
+        want, end = ref.decayed_attention(q, k, v, decay, keep, s0, batch, heads)
+        st = s0.clone()
+        close(ops.decayed_attention(q, k, v, decay, keep, st, batch, heads), want.view(batch, -1), torch.float32)
+        close(st, end, torch.float32)
+        want, end = ref.bonus_recurrence(q, k, v, z, w0, u, keep, s0, batch, heads)
+        st = s0.clone()
+        got = cuda_ops.bonus_step(q, k, v, t, w2, w0, u, nw, gate, keep, st, 1e-5, heads)
+        close(got, ref.gated_rms_norm(want.view(batch, -1), nw, gate, 1e-5, vdim, "silu"), dtype)
+        close(st, end, torch.float32, 2.0)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("batch,s,width", [(1, 1, 64), (2, 40, 100), (3, 17, 37), (1, 16, 1024)])
+def test_token_shift(dtype, batch, s, width):
+    h, mu = rnd(batch * s, width + 8, dtype=dtype)[:, :width], torch.rand(5, width, device="cuda").to(dtype)
+    start = rnd(batch, width)
+    for kp in (None, some_padding(batch, s)):
+        for prev in (None, start):
+            want, last = ref.token_shift(h, mu, batch, kp, prev)
+            st = prev.clone() if prev is not None else torch.zeros_like(start)
+            close(ops.token_shift(h, mu, batch, kp, st), want, dtype)
+            close(st, last, torch.float32)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("batch,s,channels,taps", [(1, 1, 64, 4), (2, 40, 100, 4), (3, 17, 37, 4), (2, 2, 64, 4), (1, 50, 40, 3), (2, 33, 24, 1),
+                                                   (1, 70, 32, 21), (1, 3, 9, 7)])
+def test_causal_conv(dtype, batch, s, channels, taps):
+    x = rnd(batch * s, channels + 8, dtype=dtype)[:, :channels]
+    w, b = rnd(channels, taps, dtype=dtype, scale=taps ** -0.5), rnd(channels, dtype=dtype)
+    start = rnd(batch, taps - 1, channels)
+    for kp in (None, some_padding(batch, s)):
+        for prev in (None, start):
+            want, last = ref.causal_conv_silu(x, w, b, batch, kp, prev)
+            st = prev.clone() if prev is not None else torch.zeros_like(start)
+            close(ops.causal_conv_silu(x, w, b, batch, kp, st), want, dtype)
+            if taps > 1:
+                close(st, last, torch.float32)
+
+
+def scan_inputs(n, channels, states, dtype):
+    x, z = rnd(n, channels + 8, dtype=dtype)[:, :channels], rnd(n, channels, dtype=dtype, seed=1)
+    dt, bias = rnd(n, channels, scale=2.0), rnd(channels, dtype=dtype) - 2.0
+    a_log = (torch.rand(channels, states, generator=torch.Generator().manual_seed(3)) * 3.0 - 1.0).to(dtype).cuda()
+    bc = rnd(n, 2 * states + 5, dtype=dtype)
+    return x, dt, bias, a_log, bc[:, :states], bc[:, states + 2:2 * states + 2], rnd(channels, dtype=dtype, seed=2), z
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("batch,s,channels,states", [(2, 37, 72, 16), (1, 1, 8, 1), (1, 200, 20, 5), (2, 50, 130, 24), (1, 150, 256, 64),
+                                                     (3, 20, 33, 100), (1, 19, 16, 256), (2, 64, 512, 8)])
+def test_selective_scan(dtype, batch, s, channels, states):
+    args = scan_inputs(batch * s, channels, states, dtype)
+    ext = ops.load_ext(required=True)
+    start = rnd(batch, channels, states, scale=0.5)
+    for kp in (None, some_padding(batch, s)):
+        for s0 in (None, start):
+            want, end = ref.selective_scan(*args, batch, kp, s0)
+            real = torch.ones(batch * s, dtype=torch.bool, device="cuda") if kp is None else kp.view(-1).bool()
+            for chunks in (0, 1, 2, 5):
+                st = s0.clone() if s0 is not None else torch.zeros_like(start)
+                got = ext.selective_scan(*args, batch, kp, st, chunks)
+                close(got[real], want[real], dtype)
+                close(st, end, torch.float32, 2.0)
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("batch,channels,states,rank", [(1, 72, 16, 8), (9, 40, 24, 5), (70, 256, 16, 128), (3, 33, 7, 33)])
+def test_scan_step_is_one_token_of_the_scan(dtype, batch, channels, states, rank):
+    from oslo_b200.ops import cuda_ops
+    x, _, bias, a_log, b, c, d, z = scan_inputs(batch, channels, states, dtype)
+    low, w = rnd(batch, rank, dtype=dtype), rnd(channels, rank, dtype=dtype, scale=rank ** -0.5)
+    dt = low.float() @ w.float().t()
+    s0 = rnd(batch, channels, states)
+    for keep in (None, (torch.arange(batch, device="cuda") % 2 == 0).to(torch.uint8)[:, None]):
+        want, end = ref.selective_scan(x, dt, bias, a_log, b, c, d, z, batch, keep, s0)
+        st = s0.clone()
+        close(cuda_ops.scan_step(x, low, w, bias, a_log, b, c, d, z, keep, st), want, dtype)
+        close(st, end, torch.float32, 2.0)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("batch,s,heads,groups,dim,vdim,rot", [(2, 9, 6, 2, 64, 32, 32), (1, 1, 4, 1, 128, 128, 128), (3, 5, 5, 5, 9, 11, 6),
+                                                               (2, 3, 3, 1, 40, 7, 0), (1, 7, 2, 1, 320, 24, 320)])
+def test_qkv_prep(dtype, batch, s, heads, groups, dim, vdim, rot):
+    from oslo_b200.ops import cuda_ops
+    n, past, tmax = batch * s, 4, s + 9
+    p = rnd(n, heads * dim + groups * (dim + vdim) + 8, dtype=dtype)
+    q, k, v = p[:, :heads * dim], p[:, heads * dim:(heads + groups) * dim], p[:, (heads + groups) * dim:(heads + groups) * dim + groups * vdim]
+    wq, wk = rnd(dim, dtype=dtype), rnd(dim, dtype=dtype, seed=1)
+    pos = torch.stack([torch.arange(past, past + s) + 1000 * b for b in range(batch)]).cuda()
+    freq = torch.tensor(ref.rotary_frequencies(rot, 5e5), device="cuda")
+    kc, vc = torch.zeros(batch, groups, tmax, dim, dtype=dtype, device="cuda"), torch.zeros(batch, groups, tmax, vdim, dtype=dtype, device="cuda")
+    lengths = torch.full((batch,), past, dtype=torch.int32, device="cuda")
+    got = cuda_ops.qkv_prep(q, k, v, wq, wk, 1e-4, pos, freq, kc, vc, lengths)
+    close(got, ref.norm_rotate(q.reshape(batch, s, heads, dim), wq, 1e-4, pos, freq), dtype)
+    close(kc[:, :, past:past + s].transpose(1, 2), ref.norm_rotate(k.reshape(batch, s, groups, dim), wk, 1e-4, pos, freq), dtype)
+    assert torch.equal(vc[:, :, past:past + s].transpose(1, 2), v.reshape(batch, s, groups, vdim))
+    for t in (kc, vc):
+        t[:, :, past:past + s] = 0
+        assert not t.any()
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("batch,sq,sk,heads,groups,dim,vdim", [
+    (2, 50, 50, 4, 1, 64, 64), (1, 2, 9, 4, 2, 24, 16), (2, 33, 70, 6, 3, 48, 80), (1, 140, 300, 4, 2, 128, 128), (1, 19, 19, 2, 1, 300, 20),
+    (2, 130, 130, 4, 2, 192, 128), (1, 37, 37, 5, 1, 9, 11), (2, 200, 257, 8, 2, 64, 32), (1, 257, 257, 2, 2, 32, 136)])
+def test_grouped_capped_attention(dtype, batch, sq, sk, heads, groups, dim, vdim):
+    q, k, v = (rnd(batch, n, h, d, dtype=dtype, seed=i) for i, (n, h, d) in enumerate(((sq, heads, dim), (sk, groups, dim), (sk, groups, vdim))))
+    k[:, 1] *= 6.0                                        # scores beyond the cap
+    sink = torch.zeros(heads, dtype=dtype, device="cuda")
+    keep = torch.ones(batch, sk, dtype=torch.uint8, device="cuda")
+    keep[0, :min(7, sk - sq)] = 0
+    for kp in (None, keep):
+        for cap in (0.0, 2.0, 50.0):
+            want, _ = ref.sink_attention(q, k, v, kp, sink, None, dim ** -0.5, cap)
+            close(ops.sink_attention(q, k, v, kp, sink, None, dim ** -0.5, cap), want, dtype)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("batch,heads,groups,dim,vdim,tmax,length", [
+    (2, 6, 2, 64, 72, 200, 131), (1, 3, 1, 20, 12, 64, 1), (3, 17, 1, 48, 80, 96, 96), (1, 16, 4, 128, 128, 1500, 1400), (2, 8, 8, 32, 64, 300, 290),
+    (9, 2, 1, 9, 11, 33, 20), (1, 40, 4, 64, 64, 700, 641), (2, 5, 5, 256, 256, 400, 390), (1, 4, 2, 16, 600, 50, 49), (40, 16, 2, 64, 32, 300, 257),
+    (1, 8, 1, 320, 40, 300, 255)])
+def test_grouped_decode(dtype, batch, heads, groups, dim, vdim, tmax, length):
+    q = rnd(batch, heads, dim, dtype=dtype)
+    k, v = rnd(batch, groups, tmax, dim, dtype=dtype), rnd(batch, groups, tmax, vdim, dtype=dtype, seed=2)
+    k[:, :, 0] *= 5.0
+    k[:, :, length:], v[:, :, length:] = float("nan"), float("nan")        # nothing beyond the valid length may be touched
+    lengths = torch.full((batch,), length, dtype=torch.int32, device="cuda")
+    lengths[0] = max(1, length - 3)
+    sink = torch.zeros(heads, dtype=dtype, device="cuda")
+    keep = torch.ones(batch, length, dtype=torch.uint8, device="cuda")
+    keep[-1, :min(5, length - 1)] = 0
+    from oslo_b200.ops import cuda_ops
+    for kp in (None, keep):
+        for cap in (0.0, 2.0, 50.0):
+            want = ref.grouped_decode(q, torch.nan_to_num(k), torch.nan_to_num(v), lengths, kp, sink, dim ** -0.5, cap)
+            close(cuda_ops.grouped_decode(q, k, v, lengths, kp, sink, dim ** -0.5, cap), want, dtype)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_products_for_few_and_many_rows(dtype):
+    for rows, k, n in ((1, 64, 40), (3, 128, 96), (20, 64, 48), (70, 64, 24), (200, 72, 13), (5, 30, 9)):
+        x, w = rnd(4, rows, k, dtype=dtype), rnd(4, n, k, dtype=dtype, scale=k ** -0.5)
+        close(ops.stacked_linear(x, w), torch.matmul(x.float(), w.float().transpose(1, 2)), dtype)
+        y = ops.linear_fp32(x[0], w[0])
+        assert y.dtype == torch.float32
+        close(y, x[0].float() @ w[0].float().t(), torch.float32)

@@ -251,20 +251,165 @@ def bench_mixers(args, timer: _Timer) -> None:
             del cache
 
 
+# width, wkv heads x dim, decay rank, inner channels, states, dt_rank, attention heads, kv heads, head dim, linear heads x dim, ff
+BRANCH_CASES = [(2048, 32, 64, 64, 4096, 16, 128, 16, 4, 128, 16, 128, 5504), (4096, 64, 64, 128, 8192, 16, 256, 32, 8, 128, 32, 128, 11008)]
+SFU_TERAOPS = 148 * 16 * 1.965e9 / 1e12            # exponentials, reciprocals: 16 per cycle and SM (nominal)
+
+
+def bench_branches(args, timer: _Timer) -> None:
+    """The kernels of grouped-query attention, the linear recurrences, the selective scan and the joins (Begovik layers) beside the
+    like kernels of the other families."""
+    ext = load_ext(required=True)
+    timer = _GraphTimer(args.iters, args.warmup, not args.no_flush)
+    peak, hbm = _peak_tflops(), _measured_hbm()
+    bf = torch.bfloat16
+    mk = lambda *s: (torch.randn(*s, device="cuda") * 0.5).to(bf)                                          # noqa: E731
+
+    def report(case, op, fn, gbytes=0.0, tflop=0.0, fp32_tflop=0.0, sfu=0.0, like=""):
+        if args.only and args.only not in op:
+            return
+        ms = timer(fn)
+        bound = {"hbm": gbytes / hbm * 1e3, "bf16": tflop / peak * 1e3, "fp32": fp32_tflop / FP32_TFLOPS * 1e3, "sfu": sfu / SFU_TERAOPS / 1e9}
+        by = max(bound, key=bound.get)
+        print(json.dumps(dict(case=case, op=op, us=round(ms * 1e3, 2), bound_us=round(bound[by] * 1e3, 2), bound_by=by,
+                              times_bound=round(ms / bound[by], 2), like=like)), flush=True)
+
+    for case, (w, rh, rd, rank, inner, ns, dtr, h, g, d, lh, ld, ff) in enumerate(BRANCH_CASES):
+        if args.case is not None and args.case != case:
+            continue
+        vec, nr = mk(w), rh * rd
+        w0, u, nw = mk(nr) - 3.0, mk(nr), mk(nr)
+        a_log, dtb, dd = mk(inner, ns), mk(inner) - 2.0, mk(inner)
+        conv, convb, w_dt = mk(inner, 4), mk(inner), mk(inner, dtr)
+        mu, w2 = mk(5, w), mk(nr, rank)
+        decay = torch.linspace(0.5, 0.999, lh, device="cuda")
+        hw, freq, sink = mk(d), torch.rand(d // 2, device="cuda"), torch.zeros(h, dtype=bf, device="cuda")
+        lower = mk(lh * ld).abs().clamp(max=0.9)
+        # ------------------------------------------------ prompts: 4 x 2048 and 1 x 2048 tokens
+        for b, s in ((4, 2048), (1, 2048)):
+            n, tag = b * s, f"prompt {b} x {s} "
+            r, k, v, z = mk(n, nr), mk(n, nr), mk(n, nr), torch.randn(n, nr, device="cuda")
+            st = torch.zeros(b, rh, rd, rd, device="cuda")
+            report(case, tag + "bonus recurrence", lambda: ext.bonus_recurrence(r, k, v, z, w0, u, None, st, b, rh, rd, rd),
+                   gbytes=n * nr * 14 / 1e9, fp32_tflop=6.0 * n * nr * rd / 1e12, like="gated recurrence (Moronex)")
+            report(case, tag + "gated recurrence, same sizes (Moronex)", lambda: ext.recurrence(r, k, v, w0, w0.sigmoid(), None, st, b, rh, rd, rd),
+                   gbytes=n * nr * 10 / 1e9, fp32_tflop=6.0 * n * nr * rd / 1e12)
+            q, k, v = mk(n, lh * ld), mk(n, lh * ld), mk(n, lh * ld)
+            st2 = torch.zeros(b, lh, ld, ld, device="cuda")
+            report(case, tag + "decayed recurrence", lambda: ext.decayed_recurrence(q, k, v, decay, None, st2, b, lh, ld, ld),
+                   gbytes=n * lh * ld * 10 / 1e9, fp32_tflop=4.0 * n * lh * ld * ld / 1e12, like="gated recurrence (Moronex)")
+            report(case, tag + "gated recurrence (Moronex)", lambda: ext.recurrence(q, k, v, lower, lower, None, st2, b, lh, ld, ld),
+                   gbytes=n * lh * ld * 10 / 1e9, fp32_tflop=6.0 * n * lh * ld * ld / 1e12)
+            x, zz, dt = mk(n, inner), mk(n, inner), torch.randn(n, inner, device="cuda")
+            bc = mk(n, 2 * ns)
+            st3 = torch.zeros(b, inner, ns, device="cuda")
+            report(case, tag + "selective scan", lambda: ext.selective_scan(x, dt, dtb, a_log, bc[:, :ns], bc[:, ns:], dd, zz, b, None, st3),
+                   gbytes=n * inner * 10 / 1e9, fp32_tflop=6.0 * n * inner * ns / 1e12, sfu=1.0 * n * inner * ns, like="gated recurrence (Moronex)")
+            qa, ka, va = mk(b, h, s, d), mk(b, g, s, d), mk(b, g, s, d)
+            fl = 4.0 * b * h * s * s * d * 0.5 / 1e12
+            report(case, tag + "capped attention", lambda: ext.flash_sink_fwd(qa, ka, va, None, sink, None, d ** -0.5, 50.0),
+                   gbytes=2 * n * (h + g) * d * 2 / 1e9, tflop=fl, sfu=1.5 * b * h * s * s, like="attention (GPT-J)")
+            kf, vf = mk(b, h, s, d), mk(b, h, s, d)
+            report(case, tag + "attention (GPT-J)", lambda: ext.flash_fwd(qa, kf, vf, d ** -0.5, True, 0, None, 1),
+                   gbytes=4 * n * h * d * 2 / 1e9, tflop=fl)
+            del kf, vf
+            if b == 1:
+                continue
+            o, gate = torch.randn(n, nr, device="cuda"), mk(n, nr)
+            report(case, tag + "head norm + silu gate", lambda: ext.gated_rms_norm(o, nw, gate, 1e-5, rd, 1), gbytes=n * nr * 8 / 1e9, like="layer norm")
+            lw = mk(lh * ld)
+            report(case, tag + "norm over heads + sigmoid gate", lambda: ext.gated_rms_norm(o, lw, gate, 1e-5, lh * ld, 0), gbytes=n * nr * 8 / 1e9,
+                   like="layer norm")
+            hb = mk(n, w)
+            report(case, tag + "token shift", lambda: ext.token_shift(hb, mu, b, None, None), gbytes=n * w * 12 / 1e9, like="layer norm")
+            report(case, tag + "convolution", lambda: ext.causal_conv_silu(x, conv, convb, b, None, None), gbytes=n * inner * 4 / 1e9, like="layer norm")
+            p = mk(n, (h + 2 * g) * d)
+            kc, vc, l0 = mk(b, g, s, d), mk(b, g, s, d), torch.zeros(b, dtype=torch.int32, device="cuda")
+            pos = torch.arange(s, device="cuda")[None].expand(b, s)
+            report(case, tag + "norms + rotation + append", lambda: ext.qkv_prep(p[:, :h * d], p[:, h * d:(h + g) * d], p[:, (h + g) * d:], hw, hw, 1e-5,
+                                                                              pos, freq, kc, vc, l0), gbytes=n * (h + 2 * g) * d * 4 / 1e9, like="layer norm")
+            xs, y1, y2, y3 = torch.randn(n, w, device="cuda"), mk(n, w), mk(n, w), mk(n, w)
+            report(case, tag + "join, 2 branches", lambda: ext.branch_join(xs, y1, None, 1.0, y2, None, 1.0, None, None, 1.0, 0.3, 1e-5, vec, vec),
+                   gbytes=n * w * 16 / 1e9, like="residual join (Moronex)")
+            report(case, tag + "join, 3 branches, 2 normed", lambda: ext.branch_join(xs, y1, vec, 0.5, y2, vec, 0.5, y3, None, 1.0, 0.3, 1e-5, vec, vec),
+                   gbytes=n * w * 18 / 1e9, like="residual join (Moronex)")
+            report(case, tag + "residual join (Moronex)", lambda: ext.residual_join(xs, y1, None, None, y2, vec, vec, vec, 1e-5), gbytes=n * w * 14 / 1e9)
+            report(case, tag + "layer norm (GPT-J)", lambda: ext.layernorm_fwd(hb, vec, vec, 1e-5), gbytes=n * w * 4 / 1e9)
+            gu = mk(n, 2 * ff)
+            report(case, tag + "clamped unit", lambda: ext.clamped_glu(gu[:, :ff], gu[:, ff:], 7.0, 1.702), gbytes=n * ff * 6 / 1e9, like="silu * up (Moronex)")
+            report(case, tag + "silu * up (Moronex)", lambda: ext.silu_mul(gu[:, :ff], gu[:, ff:]), gbytes=n * ff * 6 / 1e9)
+            wx, wz = mk(dtr + 2 * ns, inner), mk(inner, dtr)
+            report(case, tag + "dt product, fp32 result", lambda: co.linear_fp32(x[:, :dtr], wz), gbytes=n * (inner * 4 + dtr * 2) / 1e9,
+                   tflop=2.0 * n * inner * dtr / 1e12, like="MLP GEMM (GPT-J)")
+            report(case, tag + "x product", lambda: co.linear(x, wx, None, False, None), gbytes=n * inner * 2 / 1e9, tflop=2.0 * n * inner * (dtr + 2 * ns) / 1e12,
+                   like="MLP GEMM (GPT-J)")
+            ws = mk(4, nr, w)
+            xm = mk(4, n, w)
+            report(case, tag + "r, k, v, g products", lambda: co.stacked_linear(xm, ws), tflop=8.0 * n * nr * w / 1e12, like="MLP GEMM (GPT-J)")
+            wm = mk(4 * w, w)
+            report(case, tag + "MLP GEMM (GPT-J)", lambda: co.gemm(hb, wm), tflop=8.0 * n * w * w / 1e12)
+            del o, gate, hb, p, xs, y1, y2, y3, gu, xm
+        # ------------------------------------------------ decode over 4096 cached tokens
+        for n in (1, 8, 64):
+            t, tag = 4096, f"decode {n} "
+            r, k, v, lo, gate = mk(n, nr), mk(n, nr), mk(n, nr), mk(n, rank), mk(n, nr)
+            st = torch.zeros(n, rh, rd, rd, device="cuda")
+            report(case, tag + "bonus step", lambda: ext.bonus_step(r, k, v, lo, w2, w0, u, nw, gate, None, st, 1e-5, rh, rd, rd),
+                   gbytes=n * nr * rd * 8 / 1e9 + nr * rank * 2 / 1e9, like="recurrence step (Moronex)")
+            q, k2, v2 = mk(n, lh * ld), mk(n, lh * ld), mk(n, lh * ld)
+            st2 = torch.zeros(n, lh, ld, ld, device="cuda")
+            report(case, tag + "decayed step", lambda: ext.decayed_step(q, k2, v2, decay, None, st2, lh, ld, ld), gbytes=n * lh * ld * ld * 8 / 1e9,
+                   like="recurrence step (Moronex)")
+            nv = mk(ld)
+            report(case, tag + "recurrence step (Moronex)", lambda: ext.recurrence_step(q, k2, v2, lower, lower, nv, None, st2, 1e-5, lh, ld, ld),
+                   gbytes=n * lh * ld * ld * 8 / 1e9)
+            x, zz, dl, bc = mk(n, inner), mk(n, inner), mk(n, dtr), mk(n, 2 * ns)
+            st3 = torch.zeros(n, inner, ns, device="cuda")
+            report(case, tag + "scan step", lambda: ext.scan_step(x, dl, w_dt, dtb, a_log, bc[:, :ns], bc[:, ns:], dd, zz, None, st3),
+                   gbytes=(n * inner * ns * 8 + inner * (dtr + ns) * 2) / 1e9, like="recurrence step (Moronex)")
+            cst = torch.zeros(n, 3, inner, device="cuda")
+            report(case, tag + "convolution step", lambda: ext.causal_conv_silu(x, conv, convb, n, None, cst), gbytes=n * inner * 28 / 1e9, like="layer norm")
+            hb, sh = mk(n, w), torch.zeros(n, w, device="cuda")
+            report(case, tag + "token shift step", lambda: ext.token_shift(hb, mu, n, None, sh), gbytes=n * w * 20 / 1e9, like="layer norm")
+            q3 = mk(n, h, d)
+            lengths = torch.full((n,), t, dtype=torch.int32, device="cuda")
+            kc, vc = mk(n, g, t, d), mk(n, g, t, d)
+            report(case, tag + "capped attention (2 launches)", lambda: ext.grouped_decode(q3, kc, vc, lengths, None, sink, d ** -0.5, 50.0),
+                   gbytes=2 * n * t * g * d * 2 / 1e9, like="attention (GPT-J)")
+            l1 = torch.full((n,), t - 1, dtype=torch.int32, device="cuda")
+            p, pos = mk(n, (h + 2 * g) * d), torch.full((n, 1), t - 1, dtype=torch.long, device="cuda")
+            report(case, tag + "norms + rotation + append", lambda: ext.qkv_prep(p[:, :h * d], p[:, h * d:(h + g) * d], p[:, (h + g) * d:], hw, hw, 1e-5, pos,
+                                                                              freq, kc, vc, l1), gbytes=n * (h + 2 * g) * d * 4 / 1e9, like="layer norm")
+            del kc, vc
+            if n * t * h * d * 4 < 20e9:
+                kf, vf = mk(n, h, t, d), mk(n, h, t, d)
+                report(case, tag + "attention (GPT-J, 2 launches)", lambda: ext.decode_attn(q3, kf, vf, lengths, d ** -0.5, 0), gbytes=2 * n * t * h * d * 2 / 1e9)
+                del kf, vf
+            xs, y1, y2, y3 = torch.randn(n, w, device="cuda"), mk(n, w), mk(n, w), mk(n, w)
+            report(case, tag + "join, 3 branches, 2 normed", lambda: ext.branch_join(xs, y1, vec, 0.5, y2, vec, 0.5, y3, None, 1.0, 0.3, 1e-5, vec, vec),
+                   gbytes=n * w * 18 / 1e9, like="layer norm")
+            report(case, tag + "layer norm (GPT-J)", lambda: ext.layernorm_fwd(hb, vec, vec, 1e-5), gbytes=n * w * 4 / 1e9)
+            ws, xm, wx, wm = mk(4, nr, w), mk(4, n, w), mk(dtr + 2 * ns, inner), mk(4 * w, w)
+            report(case, tag + "r, k, v, g products", lambda: co.stacked_linear(xm, ws), gbytes=4 * nr * w * 2 / 1e9, like="MLP GEMV (GPT-J)")
+            report(case, tag + "x product", lambda: co.linear(x, wx, None, False, None), gbytes=inner * (dtr + 2 * ns) * 2 / 1e9, like="MLP GEMV (GPT-J)")
+            report(case, tag + "MLP GEMV (GPT-J)", lambda: co.linear(hb, wm, None, False, None), gbytes=4 * w * w * 2 / 1e9)
+            del ws, wm
+
+
 def main() -> None:
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
-    ap.add_argument("--op", choices=["gemm", "attention", "mixers"], required=True)
+    ap.add_argument("--op", choices=["gemm", "attention", "mixers", "branches"], required=True)
     ap.add_argument("--case", type=int, default=None, help="index into the op's shape list")
     ap.add_argument("--iters", type=int, default=20)
     ap.add_argument("--warmup", type=int, default=5)
     ap.add_argument("--causal", type=int, default=None, help="attention: 1 / 0 to run only one mask")
     ap.add_argument("--no-baseline", action="store_true", help="skip the library / legacy-kernel baseline")
     ap.add_argument("--no-flush", action="store_true", help="do not write a 256 MB buffer between timed calls")
-    ap.add_argument("--only", default="", help="mixers: only the entries whose name contains this")
+    ap.add_argument("--only", default="", help="mixers, branches: only the entries whose name contains this")
     args = ap.parse_args()
     timer = _Timer(args.iters, args.warmup, not args.no_flush)
     with torch.no_grad():
-        {"gemm": bench_gemm, "attention": bench_attention, "mixers": bench_mixers}[args.op](args, timer)
+        {"gemm": bench_gemm, "attention": bench_attention, "mixers": bench_mixers, "branches": bench_branches}[args.op](args, timer)
 
 
 if __name__ == "__main__":

@@ -1,6 +1,5 @@
 """The kernels behind Begovik against the fp32 PyTorch statements of the same ops, over sizes that do and do not fit the
 vector widths and tiles, and the whole model on the GPU against the plain implementation in ``plain_begovik.py``."""
-import math
 
 import pytest
 import torch
@@ -283,3 +282,170 @@ def test_products_for_few_and_many_rows(dtype):
         y = ops.linear_fp32(x[0], w[0])
         assert y.dtype == torch.float32
         close(y, x[0].float() @ w[0].float().t(), torch.float32)
+
+
+# ---------------------------------------------------------------------------------------------------- the whole model
+MODEL_TOL = {torch.float32: 5e-5, torch.bfloat16: 0.06}
+WIDE = {
+    # chunked recurrences and scans, several key tiles, cluster sizes above 1, more than one tile of query heads per key head
+    "wide": case(200, 256, 1e-5, wkv(4, 64, dense(320), 32), mamba(512, 16, 16, 4, dense(192)),
+                 parallel(attn(20, 2, 64, 64, 0.125, 20.0, 32), lin(4, 128, 64, (0.6, 0.9, 0.97, 0.999)), dense(256)),
+                 mamba(384, 40, 24, 4, None), parallel(attn(4, 4, 128, 128, 0.1, 50.0, 128, 5e5), lin(8, 32, 96, [0.5 + 0.06 * i for i in range(8)]), None)),
+}
+ALL = {**{k: v for k, v in CASES.items() if k != "ones"}, **WIDE}
+
+
+def load(tmp_path, cfg, tensors=None, dtype=torch.float32):
+    tensors = make_tensors(cfg) if tensors is None else tensors
+    write_model(str(tmp_path), cfg, tensors)
+    model = ob.load_causal_lm(str(tmp_path), torch_dtype=dtype).cuda().fuse().eval()
+    return model, tensors
+
+
+def ids(n, vocab, seed=1):
+    return torch.randint(0, vocab, (n,), generator=torch.Generator().manual_seed(seed)).tolist()
+
+
+def same(got, want, dtype, at=slice(None), factor=1.0):
+    """Per position: root mean square over the vocabulary, relative to the logits' own."""
+    got = got.double().cpu()
+    assert torch.isfinite(got).all() and got.shape == want[at].shape
+    d = (got - want[at]).pow(2).mean(-1).sqrt() / want.pow(2).mean().sqrt()
+    assert float(d.max()) < factor * MODEL_TOL[dtype], float(d.max())
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("name", sorted(ALL))
+def test_model_prompts_decoding_and_portions(tmp_path, dtype, name):
+    cfg = ALL[name]
+    model, tensors = load(tmp_path, cfg, dtype=dtype)
+    n = 200 if name == "wide" else 70
+    seq = ids(n, cfg["vocab"])
+    want = plain.forward(cfg, tensors, seq)
+    x = torch.tensor([seq], device="cuda")
+    before = ops.load_ext(required=True).launch_count()
+    with torch.no_grad():
+        same(model(input_ids=x).logits[0], want, dtype)
+        same(model(input_ids=x, use_cache=False).logits[0], want, dtype)
+        assert ops.load_ext().launch_count() > before
+        for portions in ([n - 12] + [1] * 12, [1] * 20, [2] * 6 + [n - 13, 1], [n // 2, 2, n - n // 2 - 2]):
+            cache, at = StaticKVCache(16, grow=True), 0
+            for m in portions:
+                out = model(input_ids=x[:, at:at + m], past_key_values=cache, use_cache=True).logits[0]
+                same(out, want, dtype, slice(at, at + m))
+                at += m
+    assert int(ops.load_ext().error_word(x).item()) == 0
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("name", ["mixed", "odd", "wide"])
+def test_model_batches_of_unequal_requests(tmp_path, dtype, name):
+    cfg = ALL[name]
+    model, tensors = load(tmp_path, cfg, dtype=dtype)
+    lens, tails = (40, 1, 23, 150), (6, 9, 3, 2)
+    seqs = [ids(a + b, cfg["vocab"], seed=a) for a, b in zip(lens, tails)]
+    want = [plain.forward(cfg, tensors, s) for s in seqs]
+    steps = BatchSteps(model, reserve=1)
+    out = steps.start([s[:a] for s, a in zip(seqs, lens)])
+    for r in range(4):
+        same(out[r, steps.pad[r]:], want[r], dtype, slice(0, lens[r]))
+    live, at = [0, 1, 2, 3], list(lens)
+    while True:
+        rows = [i for i, r in enumerate(live) if at[r] < len(seqs[r])]
+        if not rows:
+            break
+        steps.keep(rows)
+        live = [live[i] for i in rows]
+        out = steps.advance([seqs[r][at[r]] for r in live])
+        for i, r in enumerate(live):
+            same(out[i, 0][None], want[r], dtype, slice(at[r], at[r] + 1))
+            at[r] += 1
+
+
+def test_model_many_rows_decode_like_few(tmp_path):
+    cfg = WIDE["wide"]
+    model, tensors = load(tmp_path, cfg, dtype=torch.bfloat16)
+    seqs = [ids(30, 200, seed=s) for s in range(21)]
+    want = [plain.forward(cfg, tensors, s) for s in seqs[:3]]
+    x = torch.tensor(seqs, device="cuda")
+    cache = StaticKVCache(40)
+    with torch.no_grad():
+        model(input_ids=x[:, :26], past_key_values=cache)
+        for t in range(26, 30):
+            out = model(input_ids=x[:, t:t + 1], past_key_values=cache).logits
+            for r in range(3):
+                same(out[r], want[r], torch.bfloat16, slice(t, t + 1))
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_model_far_keys_on_the_gpu(tmp_path, dtype):
+    cfg = case(64, 64, 1e-5, parallel(attn(4, 2, 64, 64, 0.125, 30.0, 16, 1e6), lin(1, 16, 16, (0.5,)), None), mamba(32, 8, 4, 4, dense(48)))
+    tensors = far_key_weights(0, make_tensors(cfg, 3), 2.0)
+    seq = [t % 60 for t in ids(420, 60, 8)]
+    for at in (0, 1, 127, 128, 255):
+        seq[at] = 63
+    want = plain.forward(cfg, tensors, seq)
+    other = plain.forward(cfg, tensors, [62] + seq[1:])
+    model, _ = load(tmp_path, cfg, tensors, dtype)
+    x = torch.tensor([seq], device="cuda")
+    factor = 2.0 if dtype == torch.float32 else 1.0
+    with torch.no_grad():
+        same(model(input_ids=x).logits[0], want, dtype, factor=factor)
+        cache = StaticKVCache(420)
+        model(input_ids=x[:, :400], past_key_values=cache)
+        got = torch.cat([model(input_ids=x[:, t:t + 1], past_key_values=cache).logits[0] for t in range(400, 420)])
+    same(got, want, dtype, slice(400, None), factor)
+    moved = (other[400:] - want[400:]).pow(2).mean(-1).sqrt().max() / want.pow(2).mean().sqrt()
+    assert float(moved) > 20 * MODEL_TOL[torch.float32]   # the first token is seen from the end
+
+
+@pytest.mark.parametrize("name", ["mixed", "wide"])
+def test_model_greedy_generation_and_captured_decoding(tmp_path, name):
+    cfg = ALL[name]
+    model, tensors = load(tmp_path, cfg)
+    prompts = [ids(9, cfg["vocab"], 11), ids(9, cfg["vocab"], 12)]
+    want = []
+    for p in prompts:
+        seq = list(p)
+        for _ in range(10):
+            seq.append(int(plain.forward(cfg, tensors, seq)[-1].argmax()))
+        want.append(seq)
+    want = torch.tensor(want)
+    x = torch.tensor(prompts, device="cuda")
+    kw = dict(max_new_tokens=10, eos_token_id=None, pad_token_id=None)
+    assert torch.equal(model.generate(x, **kw).cpu(), want)
+    assert torch.equal(model.generate(x, cuda_graph=True, **kw).cpu(), want)
+    dec = GraphedGreedyDecoder(model, max_len=32)
+    for _ in range(2):                                    # the captured step, the cache and the states are used again
+        assert torch.equal(dec.generate(x, 10).cpu(), want)
+    assert dec.replays > 0
+    # the 16-bit model decodes the same tokens eagerly and from the captured step
+    half, _ = load(tmp_path, cfg, tensors, dtype=torch.bfloat16)
+    assert torch.equal(half.generate(x, **kw), half.generate(x, cuda_graph=True, **kw))
+
+
+def test_model_with_sizes_beyond_one_kernel(tmp_path):
+    cfg = case(40, 32, 1e-5, wkv(1, 300, None, 4), parallel(attn(2, 1, 300, 24, 0.06, 9.0, 300), lin(1, 700, 16, (0.9,)), None),
+               mamba(16, 130, 3, 9, dense(24)))
+    model, tensors = load(tmp_path, cfg)
+    seq = ids(24, 40)
+    want = plain.forward(cfg, tensors, seq)
+    x = torch.tensor([seq], device="cuda")
+    cache = StaticKVCache(24)
+    with torch.no_grad():
+        got = [model(input_ids=x[:, a:b], past_key_values=cache).logits[0] for a, b in ((0, 15), (15, 20), (20, 21), (21, 22))]
+    same(torch.cat(got), want, torch.float32, slice(0, 22), 2.0)
+
+
+def test_long_decoding_keeps_agreeing_with_the_prompt_form(tmp_path):
+    cfg = CASES["heads64"]
+    for dtype in (torch.float32, torch.bfloat16):
+        model, tensors = load(tmp_path, cfg, dtype=dtype)
+        seq = ids(400, 128, 5)
+        want = plain.forward(cfg, tensors, seq)
+        x = torch.tensor([seq], device="cuda")
+        cache = StaticKVCache(400)
+        with torch.no_grad():
+            model(input_ids=x[:, :3], past_key_values=cache)
+            got = torch.cat([model(input_ids=x[:, t:t + 1], past_key_values=cache).logits[0] for t in range(3, 400)])
+        same(got, want, dtype, slice(3, None), 1.5)

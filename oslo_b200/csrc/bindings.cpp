@@ -1136,7 +1136,8 @@ Tensor grouped_decode(const Tensor& q, const Tensor& kc, const Tensor& vc, const
   const uint8_t* kp = keep_ptr(keep, B, 0, ld_keep);
   c10::cuda::CUDAGuard guard(q.device());
   auto& st = dev_state(q.get_device());
-  const int splits = oslo_grouped_splits(static_cast<int>(B), static_cast<int>(H), static_cast<int>(G), static_cast<int>(T), st.sms);
+  const int splits = oslo_grouped_splits(static_cast<int>(B), static_cast<int>(H), static_cast<int>(G), static_cast<int>(T),
+                                         static_cast<int>(q.size(2)), static_cast<int>(vdim), dt_code(q), st.sms);
   const auto f32 = q.options().dtype(at::kFloat);
   Tensor ws = at::empty({B, H, splits, (vdim + 3) / 4 * 4}, f32);
   Tensor stat = at::empty({B, H, splits, 2}, f32);

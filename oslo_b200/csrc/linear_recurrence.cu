@@ -469,12 +469,12 @@ struct StepParams {
 
 template <typename T, int VEC, int RULE>
 __global__ void __launch_bounds__(256) recurrence_step_kernel(const StepParams p) {
-  extern __shared__ float step_smem[];
-  float* ks = step_smem;            // [dim]
+  extern __shared__ __align__(16) float step_smem[];
+  float* ts = step_smem;            // [rank], RULE_BONUS
+  float* ks = ts + (RULE == RULE_BONUS ? p.rank : 0);   // [dim]
   float* qs = ks + p.dim;           // [dim]
   float* ws = qs + p.dim;           // [dim], RULE_BONUS
-  float* ts = ws + (RULE == RULE_BONUS ? p.dim : 0);   // [rank], RULE_BONUS
-  float* part = ts + (RULE == RULE_BONUS ? p.rank : 0);   // [ty][cols]
+  float* part = ws + (RULE == RULE_BONUS ? p.dim : 0);   // [ty][cols]
   __shared__ float red[32];
   __shared__ float slice_ss;
   cg::cluster_group cluster = cg::this_cluster();
@@ -485,20 +485,46 @@ __global__ void __launch_bounds__(256) recurrence_step_kernel(const StepParams p
   const T* f = static_cast<const T*>(p.f) + b * p.ldf + static_cast<long long>(h) * p.dim;
   const T* v = static_cast<const T*>(p.v) + b * p.ldv + static_cast<long long>(h) * p.vdim;
   const bool on = p.keep == nullptr || p.keep[b * p.ld_keep];
+  const int tx_n = p.cols / VEC;                       // the launcher keeps tx_n <= 256
+  const int ty_n = blockDim.x / tx_n;
+  const int tx = threadIdx.x % tx_n, ty = threadIdx.x / tx_n;
+  float* st = p.state + (static_cast<long long>(b) * p.H + h) * p.dim * p.vdim + c0;
+  const bool mine = ty < ty_n && tx * VEC < cols;      // VEC > 1: the launcher guarantees vdim % VEC == 0
+  constexpr int AHEAD = 4;                             // state rows that are on their way while the gates are computed
+  float ahead[AHEAD][VEC];
+#pragma unroll
+  for (int a = 0; a < AHEAD; ++a)
+    if (mine && ty + a * ty_n < p.dim) load_vec<float, VEC>(st + static_cast<long long>(ty + a * ty_n) * p.vdim + tx * VEC, ahead[a]);
   float bonus = 0.f;
   if constexpr (RULE == RULE_BONUS) {
     const T* t = static_cast<const T*>(p.t) + b * p.ldt;
     for (int i = threadIdx.x; i < p.rank; i += blockDim.x) ts[i] = Num<T>::to(Num<T>::from(tanhf(Num<T>::to(t[i]))));
     __syncthreads();
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const T* w2 = static_cast<const T*>(p.w2) + static_cast<long long>(h) * p.dim * p.rank;
     const T* w0 = static_cast<const T*>(p.f_bias) + h * p.dim;
+    int tpr = 1;                                       // threads that share a channel's row of W_w2
+    while (tpr < 32 && 2 * tpr * p.dim <= 256) tpr *= 2;
+    const int j = threadIdx.x % tpr;
     const bool vec = p.rank % 4 == 0;
-#pragma unroll 2
-    for (int i = warp; i < p.dim; i += 8) {
-      const T* row = w2 + static_cast<long long>(i) * p.rank;
-      const float z = vec ? warp_dot<T, 4>(row, ts, p.rank, lane) : warp_dot<T, 1>(row, ts, p.rank, lane);
-      if (lane == 0) ws[i] = on ? channel_decay<T>(z + Num<T>::to(w0[i])) : 1.f;
+    for (int i0 = 0; i0 < p.dim; i0 += 256 / tpr) {    // whole warps stay together
+      const int i = i0 + threadIdx.x / tpr;
+      float z = 0.f;
+      if (i < p.dim) {
+        const T* row = w2 + static_cast<long long>(i) * p.rank;
+        if (vec) {
+#pragma unroll 4
+          for (int k = j * 4; k < p.rank; k += 4 * tpr) {
+            float w[4];
+            load_vec<T, 4>(row + k, w);
+            const float4 t4 = *reinterpret_cast<const float4*>(ts + k);
+            z = fmaf(w[0], t4.x, fmaf(w[1], t4.y, fmaf(w[2], t4.z, fmaf(w[3], t4.w, z))));
+          }
+        } else {
+          for (int k = j; k < p.rank; k += tpr) z = fmaf(Num<T>::to(row[k]), ts[k], z);
+        }
+      }
+      for (int off = tpr / 2; off > 0; off >>= 1) z += __shfl_xor_sync(0xffffffffu, z, off);
+      if (i < p.dim && j == 0) ws[i] = on ? channel_decay<T>(z + Num<T>::to(w0[i])) : 1.f;
     }
     for (int i = threadIdx.x; i < p.dim; i += blockDim.x) {
       ks[i] = on ? Num<T>::to(f[i]) : 0.f;
@@ -519,10 +545,6 @@ __global__ void __launch_bounds__(256) recurrence_step_kernel(const StepParams p
   }
   __syncthreads();
   const float hd = RULE == RULE_DECAY && on ? p.head_decay[h] : 1.f;
-  const int tx_n = p.cols / VEC;                       // the launcher keeps tx_n <= 256
-  const int ty_n = blockDim.x / tx_n;
-  const int tx = threadIdx.x % tx_n, ty = threadIdx.x / tx_n;
-  float* st = p.state + (static_cast<long long>(b) * p.H + h) * p.dim * p.vdim + c0;
   if (ty < ty_n) {
     const int c = tx * VEC;
     float o[VEC], vv[VEC];
@@ -532,26 +554,32 @@ __global__ void __launch_bounds__(256) recurrence_step_kernel(const StepParams p
       if (RULE == RULE_DECAY) vv[i] = silu_t<T>(vv[i]);
       o[i] = RULE == RULE_BONUS && ty == 0 ? bonus * vv[i] : 0.f;
     }
-    if (c < cols) {                                    // VEC > 1: the launcher guarantees vdim % VEC == 0
+    auto update = [&](int i, float (&s)[VEC]) {
+      const float k = ks[i], qq = qs[i], w = RULE == RULE_BONUS ? ws[i] : hd;
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) {
+        if (RULE == RULE_GATED) {
+          s[j] = fmaf(k, vv[j] - s[j], s[j]);
+          o[j] = fmaf(qq, s[j], o[j]);
+        } else if (RULE == RULE_DECAY) {
+          s[j] = fmaf(w, s[j], k * vv[j]);
+          o[j] = fmaf(qq, s[j], o[j]);
+        } else {
+          o[j] = fmaf(qq, s[j], o[j]);
+          s[j] = fmaf(w, s[j], k * vv[j]);
+        }
+      }
+      store_vec<float, VEC>(st + static_cast<long long>(i) * p.vdim + c, s);
+    };
+    if (mine) {
+#pragma unroll
+      for (int a = 0; a < AHEAD; ++a)
+        if (ty + a * ty_n < p.dim) update(ty + a * ty_n, ahead[a]);
 #pragma unroll 4
-      for (int i = ty; i < p.dim; i += ty_n) {
+      for (int i = ty + AHEAD * ty_n; i < p.dim; i += ty_n) {
         float s[VEC];
         load_vec<float, VEC>(st + static_cast<long long>(i) * p.vdim + c, s);
-        const float k = ks[i], qq = qs[i], w = RULE == RULE_BONUS ? ws[i] : hd;
-#pragma unroll
-        for (int j = 0; j < VEC; ++j) {
-          if (RULE == RULE_GATED) {
-            s[j] = fmaf(k, vv[j] - s[j], s[j]);
-            o[j] = fmaf(qq, s[j], o[j]);
-          } else if (RULE == RULE_DECAY) {
-            s[j] = fmaf(w, s[j], k * vv[j]);
-            o[j] = fmaf(qq, s[j], o[j]);
-          } else {
-            o[j] = fmaf(qq, s[j], o[j]);
-            s[j] = fmaf(w, s[j], k * vv[j]);
-          }
-        }
-        store_vec<float, VEC>(st + static_cast<long long>(i) * p.vdim + c, s);
+        update(i, s);
       }
     }
 #pragma unroll
@@ -640,8 +668,9 @@ extern "C" int oslo_recurrence_chunks(int B, int S, int H, int dim, int vdim, in
   double best_cost = 1e30;
   for (int n = 1; n <= S / 64 && n <= 64; ++n) {
     const double per = static_cast<double>(S) / n;
-    const auto fullest = [&](long long blocks) { return static_cast<double>((blocks + num_sms - 1) / num_sms); };
-    // fewer than two blocks on an SM leave its pipes partly idle
+    // in units of 256 threads
+    const auto fullest = [&](long long blocks) { return static_cast<double>((blocks + num_sms - 1) / num_sms) * nt / 256.0; };
+    // fewer than 512 threads on an SM leave its pipes partly idle
     const double c3 = std::max(1.4, fullest(ctas * n)) * per;
     // ... and the states' four trips through memory (16 bytes per element, in units of one token's update)
     const double c1 = n > 1 ? std::max(1.4, fullest(ctas * (n - 1))) * per * 0.67 + 40.0 + 0.094 * B * H * n : 0.0;

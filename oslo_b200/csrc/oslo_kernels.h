@@ -285,7 +285,7 @@ int oslo_qkv_prep(const void* q, long long ldq, const void* k, long long ldk, co
                   int dtype, int* err_word, cudaStream_t stream);
 // one query per row: q [B, H, dim], caches [B, G, Tmax, *], of which lengths[b] positions count; keep [B, n_keep] (0 = padded) or
 // null; fp32 workspaces ws [B, H, splits, vdim rounded up to a multiple of 4] and stat [B, H, splits, 2]; out [B, H * vdim]
-int oslo_grouped_splits(int B, int H, int G, int T, int num_sms);
+int oslo_grouped_splits(int B, int H, int G, int T, int dim, int vdim, int dtype, int num_sms);
 int oslo_grouped_decode(const void* q, const void* kc, const void* vc, const int* lengths, const uint8_t* keep, long long ld_keep,
                         int n_keep, const void* sink, float* ws, float* stat, void* out, int B, int H, int G, int dim, int vdim,
                         int Tmax, int splits, float scale, float softcap, int dtype, int* err_word, cudaStream_t stream);

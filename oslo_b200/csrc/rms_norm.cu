@@ -252,18 +252,21 @@ __device__ __forceinline__ void gate_run(const float* o, const T* w, const T* ga
   store_vec<T, VEC>(out + c, v);
 }
 
-// one warp (WARP) or one block per run of `group` columns
-template <typename T, int VEC, bool WARP>
+// LANES lanes of a warp per run of `group` columns, or (LANES 0) one block
+template <typename T, int VEC, int LANES>
 __global__ void __launch_bounds__(256) gated_rms_norm_kernel(const float* __restrict__ o, const T* __restrict__ w,
                                                              const T* __restrict__ gate, long long ldg, T* __restrict__ out,
                                                              long long runs, int cols, int group, float eps, int act) {
   __shared__ float red[32];
-  const long long run = WARP ? static_cast<long long>(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5) : blockIdx.x;
-  if (run >= runs) return;                                 // WARP: whole warps leave, and no barrier follows
+  constexpr bool WARP = LANES > 0;
+  constexpr int L = WARP ? LANES : 32;
+  const bool real = !WARP || static_cast<long long>(blockIdx.x) * (blockDim.x / L) + threadIdx.x / L < runs;
+  // lanes past the last run repeat it without storing, so that their warp stays whole
+  const long long run = WARP ? (real ? static_cast<long long>(blockIdx.x) * (blockDim.x / L) + threadIdx.x / L : runs - 1) : blockIdx.x;
   const int per_row = cols / group;
   const long long row = run / per_row;
   const int c0 = static_cast<int>(run - row * per_row) * group;
-  const int lane = WARP ? threadIdx.x & 31 : threadIdx.x, step = WARP ? 32 : blockDim.x;
+  const int lane = WARP ? threadIdx.x % L : threadIdx.x, step = WARP ? L : blockDim.x;
   o += row * cols + c0;
   w += c0;
   gate += row * ldg + c0;
@@ -275,7 +278,13 @@ __global__ void __launch_bounds__(256) gated_rms_norm_kernel(const float* __rest
 #pragma unroll
     for (int i = 0; i < VEC; ++i) ss = fmaf(v[i], v[i], ss);
   }
-  ss = WARP ? warp_sum(ss) : block_sum(ss, red);
+  if (WARP) {
+#pragma unroll
+    for (int off = L / 2; off > 0; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
+  } else {
+    ss = block_sum(ss, red);
+  }
+  if (!real) return;
   const float r = 1.0f / sqrtf(ss / group + eps);
   for (int c = lane * VEC; c < group; c += step * VEC) gate_run<T, VEC>(o, w, gate, out, c, r, act);
 }
@@ -434,14 +443,16 @@ extern "C" int oslo_gated_rms_norm(const float* o, const void* w, const void* ga
   const size_t te = dtype == OSLO_DT_FP32 ? 4 : 2;
   const bool vec = group % 4 == 0 && ldg % 4 == 0 && aligned_to(o, 16) && aligned_to(w, 4 * te) && aligned_to(gate, 4 * te) &&
                    aligned_to(out, 4 * te);
-#define GATED_GO(V)                                                                                                         \
-  if (group <= 512)                                                                                                         \
-    gated_rms_norm_kernel<T, V, true><<<static_cast<unsigned>((runs + 7) / 8), 256, 0, stream>>>(                           \
-        o, static_cast<const T*>(w), static_cast<const T*>(gate), ldg, static_cast<T*>(out), runs, cols, group, eps, act);  \
-  else                                                                                                                      \
-    gated_rms_norm_kernel<T, V, false><<<static_cast<unsigned>(runs), 256, 0, stream>>>(                                    \
-        o, static_cast<const T*>(w), static_cast<const T*>(gate), ldg, static_cast<T*>(out), runs, cols, group, eps, act);
+#define GATED_LAUNCH(V, L, BLOCKS)                                                                  \
+  gated_rms_norm_kernel<T, V, L><<<static_cast<unsigned>(BLOCKS), 256, 0, stream>>>(                \
+      o, static_cast<const T*>(w), static_cast<const T*>(gate), ldg, static_cast<T*>(out), runs, cols, group, eps, act)
+#define GATED_GO(V)                                                         \
+  if (group <= 8 * V) GATED_LAUNCH(V, 8, (runs + 31) / 32);                 \
+  else if (group <= 16 * V) GATED_LAUNCH(V, 16, (runs + 15) / 16);          \
+  else if (group <= 512) GATED_LAUNCH(V, 32, (runs + 7) / 8);               \
+  else GATED_LAUNCH(V, 0, runs);
   OSLO_DISPATCH_T(dtype, { if (vec) { GATED_GO(4) } else { GATED_GO(1) } });
+#undef GATED_LAUNCH
 #undef GATED_GO
   return static_cast<int>(cudaGetLastError());
 }

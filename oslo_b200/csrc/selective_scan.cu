@@ -119,21 +119,30 @@ __global__ void __launch_bounds__(128) causal_conv_kernel(const ConvParams p) {
       for (int i = 0; i < VEC; ++i) wr[j][i] = Num<T>::to(w[i * TAPS + j]);
 #pragma unroll
     for (int j = 0; j < TAPS - 1; ++j) input(t0 - TAPS + 1 + j, win[j + 1]);
-    for (int t = t0; t < t1; ++t) {
-      float y[VEC];
+    constexpr int AHEAD = 4;                 // tokens whose inputs are on their way
+    for (int tb = t0; tb < t1; tb += AHEAD) {
+      float now[AHEAD][VEC];
 #pragma unroll
-      for (int j = 0; j < TAPS - 1; ++j)
+      for (int a = 0; a < AHEAD; ++a)
+        if (tb + a < t1) input(tb + a, now[a]);
 #pragma unroll
-        for (int i = 0; i < VEC; ++i) win[j][i] = win[j + 1][i];
-      input(t, win[TAPS - 1]);
+      for (int a = 0; a < AHEAD; ++a) {
+        if (tb + a >= t1) break;
+        float y[VEC];
 #pragma unroll
-      for (int i = 0; i < VEC; ++i) {
-        y[i] = bias[i];
+        for (int j = 0; j < TAPS - 1; ++j)
 #pragma unroll
-        for (int j = 0; j < TAPS; ++j) y[i] = fmaf(wr[j][i], win[j][i], y[i]);
-        y[i] = silu_f(y[i]);
+          for (int i = 0; i < VEC; ++i) win[j][i] = win[j + 1][i];
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) {
+          win[TAPS - 1][i] = now[a][i];
+          y[i] = bias[i];
+#pragma unroll
+          for (int j = 0; j < TAPS; ++j) y[i] = fmaf(wr[j][i], win[j][i], y[i]);
+          y[i] = sizeof(T) == 4 ? silu_f(y[i]) : y[i] * __fdividef(1.0f, 1.0f + __expf(-y[i]));
+        }
+        store_vec<T, VEC>(out + static_cast<long long>(tb + a) * p.C, y);
       }
-      store_vec<T, VEC>(out + static_cast<long long>(t) * p.C, y);
     }
   } else {
     for (int t = t0; t < t1; ++t) {
@@ -390,61 +399,62 @@ struct ScanStepParams {
   int B, C, N;
 };
 
+// thread = (row, channel)
 template <typename T, int VEC, int SVEC>
 __global__ void __launch_bounds__(256) scan_step_kernel(const ScanStepParams p) {
-  extern __shared__ float st_smem[];
-  float* dts = st_smem;                      // [ST_ROWS][rank]
-  float* bs = dts + ST_ROWS * p.rank;        // [ST_ROWS][N]
-  float* cs = bs + ST_ROWS * p.N;            // [ST_ROWS][N]
-  __shared__ float step_s[ST_ROWS][ST_CH];
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int c0 = blockIdx.x * ST_CH, b0 = blockIdx.y * ST_ROWS, nb = min(ST_ROWS, p.B - b0);
-  for (int e = tid; e < nb * p.rank; e += 256)
-    dts[e] = Num<T>::to(static_cast<const T*>(p.dt)[(b0 + e / p.rank) * p.lddt + e % p.rank]);
-  for (int e = tid; e < nb * p.N; e += 256) {
-    bs[e] = Num<T>::to(static_cast<const T*>(p.b)[(b0 + e / p.N) * p.ldb + e % p.N]);
-    cs[e] = Num<T>::to(static_cast<const T*>(p.c)[(b0 + e / p.N) * p.ldc + e % p.N]);
-  }
-  __syncthreads();
-  for (int j = warp; j < ST_CH; j += 8) {    // a warp per channel: its row of W_dt against every row's dt
-    if (c0 + j >= p.C) break;
-    const T* w = static_cast<const T*>(p.w_dt) + static_cast<long long>(c0 + j) * p.rank;
-    float acc[ST_ROWS];
-#pragma unroll
-    for (int r = 0; r < ST_ROWS; ++r) acc[r] = 0.f;
-    for (int k = lane * VEC; k < p.rank; k += 32 * VEC) {
-      float v[VEC];
-      load_vec<T, VEC>(w + k, v);
-#pragma unroll
-      for (int r = 0; r < ST_ROWS; ++r) {
-        if (r < nb) {
-#pragma unroll
-          for (int i = 0; i < VEC; ++i) acc[r] = fmaf(v[i], dts[r * p.rank + k + i], acc[r]);
-        }
-      }
-    }
-    const float bias = Num<T>::to(static_cast<const T*>(p.dt_bias)[c0 + j]);
-#pragma unroll
-    for (int r = 0; r < ST_ROWS; ++r) {
-      if (r < nb) {
-        const float t = warp_sum(acc[r]);
-        if (lane == 0) step_s[r][j] = softplus_t<T>(t + bias);
-      }
-    }
-  }
-  __syncthreads();
-  const int c = c0 + lane, r = warp, b = b0 + r;     // a thread per (row, channel)
-  if (r >= nb || c >= p.C) return;
-  const bool on = p.keep == nullptr || p.keep[b * p.ld_keep];
-  const float st = on ? step_s[r][lane] : 0.f;
-  const float x = Num<T>::to(static_cast<const T*>(p.x)[b * p.ldx + c]), sx = st * x;
+  extern __shared__ float4 st_smem[];
+  const int ldd = (p.rank + 3) / 4 * 4, ldw = ldd + 4;   // reads of four elements by 32 rows without conflicts
+  float* dts = reinterpret_cast<float*>(st_smem);        // [ST_ROWS][ldd]
+  T* ws = reinterpret_cast<T*>(dts + ST_ROWS * ldd);     // [ST_CH][ldw]
+  float* bs = reinterpret_cast<float*>(ws + ST_CH * ldw);   // [ST_ROWS][N]
+  float* cs = bs + ST_ROWS * p.N;                        // [ST_ROWS][N]
+  const int tid = threadIdx.x, lane = tid & 31, r = tid >> 5;
+  const int c0 = blockIdx.x * ST_CH, b0 = blockIdx.y * ST_ROWS, nb = min(ST_ROWS, p.B - b0), nc = min(ST_CH, p.C - c0);
+  const int c = c0 + lane, b = b0 + r;
+  const bool mine = r < nb && c < p.C;
+  constexpr int AHEAD = 16 / SVEC;                       // states that are on their way while the step is computed
   float* s = p.state + (static_cast<long long>(b) * p.C + c) * p.N;
+  float ahead[AHEAD][SVEC];
+#pragma unroll
+  for (int a = 0; a < AHEAD; ++a)
+    if (mine && a * SVEC < p.N) load_vec<float, SVEC>(s + a * SVEC, ahead[a]);
+  for (int j = tid / 8; j < nc; j += 32) {               // eight threads per row of the step projection
+    const T* w = static_cast<const T*>(p.w_dt) + static_cast<long long>(c0 + j) * p.rank;
+#pragma unroll 4
+    for (int k = tid % 8 * VEC; k < p.rank; k += 8 * VEC)
+      *reinterpret_cast<Pack<T, VEC>*>(ws + j * ldw + k) = *reinterpret_cast<const Pack<T, VEC>*>(w + k);
+  }
+  if (r < nb) {                                          // a warp per row
+    for (int k = lane; k < ldd; k += 32) dts[r * ldd + k] = k < p.rank ? Num<T>::to(static_cast<const T*>(p.dt)[b * p.lddt + k]) : 0.f;
+    for (int k = lane; k < p.N; k += 32) {
+      bs[r * p.N + k] = Num<T>::to(static_cast<const T*>(p.b)[b * p.ldb + k]);
+      cs[r * p.N + k] = Num<T>::to(static_cast<const T*>(p.c)[b * p.ldc + k]);
+    }
+  }
+  __syncthreads();
+  if (!mine) return;
+  float st = 0.f;
+  if (p.keep == nullptr || p.keep[b * p.ld_keep]) {
+    float z0 = 0.f, z1 = 0.f;
+    int k = 0;
+    if (VEC >= 4) {
+#pragma unroll 4
+      for (; k + 4 <= p.rank; k += 4) {
+        float w[4];
+        load_vec<T, 4>(ws + lane * ldw + k, w);
+        const float4 d4 = *reinterpret_cast<const float4*>(dts + r * ldd + k);
+        z0 = fmaf(w[0], d4.x, fmaf(w[1], d4.y, z0));
+        z1 = fmaf(w[2], d4.z, fmaf(w[3], d4.w, z1));
+      }
+    }
+    for (; k < p.rank; ++k) z0 = fmaf(Num<T>::to(ws[lane * ldw + k]), dts[r * ldd + k], z0);
+    st = softplus_t<T>(z0 + z1 + Num<T>::to(static_cast<const T*>(p.dt_bias)[c]));
+  }
+  const float x = Num<T>::to(static_cast<const T*>(p.x)[b * p.ldx + c]), sx = st * x;
   const T* al = static_cast<const T*>(p.a_log) + static_cast<long long>(c) * p.N;
   float y = 0.f;
-#pragma unroll 4
-  for (int n = 0; n < p.N; n += SVEC) {
-    float sv[SVEC], av[SVEC];
-    load_vec<float, SVEC>(s + n, sv);
+  auto update = [&](int n, float (&sv)[SVEC]) {
+    float av[SVEC];
     load_vec<T, SVEC>(al + n, av);
 #pragma unroll
     for (int i = 0; i < SVEC; ++i) {
@@ -452,6 +462,15 @@ __global__ void __launch_bounds__(256) scan_step_kernel(const ScanStepParams p) 
       y = fmaf(sv[i], cs[r * p.N + n + i], y);
     }
     store_vec<float, SVEC>(s + n, sv);
+  };
+#pragma unroll
+  for (int a = 0; a < AHEAD; ++a)
+    if (a * SVEC < p.N) update(a * SVEC, ahead[a]);
+#pragma unroll 2
+  for (int n = 16; n < p.N; n += SVEC) {
+    float sv[SVEC];
+    load_vec<float, SVEC>(s + n, sv);
+    update(n, sv);
   }
   y = fmaf(Num<T>::to(static_cast<const T*>(p.d)[c]), x, y);
   static_cast<T*>(p.out)[static_cast<long long>(b) * p.C + c] = Num<T>::from(y * silu_f(Num<T>::to(static_cast<const T*>(p.z)[b * p.ldz + c])));
@@ -533,8 +552,11 @@ extern "C" int oslo_causal_conv_silu(const void* x, long long ldx, const void* w
   const size_t te = dtype == OSLO_DT_FP32 ? 4 : 2;
   const bool vec = C % 4 == 0 && ldx % 4 == 0 && aligned_to(x, 4 * te) && aligned_to(bias, 4 * te) && aligned_to(out, 4 * te);
 #define CV_GO(V, N) causal_conv_kernel<T, V, N><<<dim3((C + 128 * V - 1) / (128 * V), runs, B), 128, 0, stream>>>(p)
+  const bool wide = vec && te == 2 && C % 8 == 0 && ldx % 8 == 0 && aligned_to(x, 16) && aligned_to(bias, 16) && aligned_to(out, 16) &&
+                    static_cast<long long>(B) * runs * C >= 148 * 1024 * 8;
   OSLO_DISPATCH_T(dtype, {
-    if (taps == 4 && vec) CV_GO(4, 4);
+    if (taps == 4 && wide) CV_GO(8, 4);
+    else if (taps == 4 && vec) CV_GO(4, 4);
     else if (taps == 3 && vec) CV_GO(4, 3);
     else if (vec) CV_GO(4, 0);
     else CV_GO(1, 0);
@@ -609,9 +631,10 @@ extern "C" int oslo_scan_step(const void* x, long long ldx, const void* dt, long
   if (B <= 0 || C <= 0) return 0;
   if (N <= 0 || rank <= 0 || (B + ST_ROWS - 1) / ST_ROWS > 65535) return -1;
   ScanStepParams p{x, ldx, dt, lddt, w_dt, rank, dt_bias, a_log, d, b, c, ldb, ldc, z, ldz, keep, ld_keep, state, out, B, C, N};
-  const size_t smem = static_cast<size_t>(ST_ROWS) * (rank + 2 * N) * sizeof(float);
-  if (smem > 200 * 1024) return -3;
   const size_t te = dtype == OSLO_DT_FP32 ? 4 : 2;
+  const size_t ldd = (rank + 3) / 4 * 4;
+  const size_t smem = (ST_ROWS * (ldd + 2 * static_cast<size_t>(N))) * sizeof(float) + ST_CH * (ldd + 4) * te;
+  if (smem > 200 * 1024) return -3;
   const bool vec = rank % 4 == 0 && aligned_to(w_dt, 4 * te), svec = N % 4 == 0 && aligned_to(state, 16) && aligned_to(a_log, 4 * te);
 #define SS_GO(V, SV)                                                                                              \
   {                                                                                                               \

@@ -337,7 +337,7 @@ class BonusRecurrence(nn.Module):
             prev = cache.recurrent_state(layer_id, (batch, h.size(1)), h.device, "shift")
             state = cache.recurrent_state(layer_id, (batch, self.heads, self.dim, self.dim), h.device)
         mixed = ops.token_shift(h, self.mu, batch, keep, prev, fused=self.oslo_fused)
-        r, k, v, g = self.rkvg(mixed[:4]).unbind(0)
+        r, k, v, g = self.rkvg(mixed[:4])
         t = self.w1(mixed[4])
         if s == 1 and state is not None and self.oslo_fused and _inference(h, self.w0) and ops.use_kernels(h):
             from ..ops import cuda_ops

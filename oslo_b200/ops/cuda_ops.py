@@ -712,19 +712,20 @@ def linear_fp32(x: Tensor, weight: Tensor) -> Tensor:
     return torch.matmul(x.float(), weight.float().t())
 
 
-def stacked_linear(x: Tensor, weight: Tensor) -> Tensor:
-    parts, rows, _ = x.shape
-    if gemm_ok(x[0], weight[0]) and weight.size(1) % 8 == 0:
-        if rows <= GEMV_ROWS:
-            return _ext().gemv_stacked(x, weight)
-        out = torch.empty(parts, rows, weight.size(1), dtype=x.dtype, device=x.device)
-        for i in range(parts):
-            if rows <= SMALL_M_ROWS:
-                out[i] = _ext().gemm_small_m(x[i], weight[i], 0, None, -1)
-            else:
-                gemm(x[i], weight[i], out=out[i])
-        return out
-    return torch.matmul(x, weight.transpose(1, 2))
+def stacked_linear(x: Tensor, weight: Tensor):
+    """A few rows: all parts' rows against all parts' weights in one weight-streaming product, of which the diagonal blocks are
+    kept - reading the weights is what takes time there."""
+    parts, rows, k = x.shape
+    n = weight.size(1)
+    if not (gemm_ok(x[0], weight[0]) and n % 8 == 0):
+        return torch.matmul(x, weight.transpose(1, 2)).unbind(0)
+    if rows <= GEMV_ROWS:
+        return _ext().gemv_stacked(x, weight).unbind(0)
+    if rows <= SMALL_M_ROWS and x.is_contiguous() and weight.is_contiguous():
+        flat, w = x.view(parts * rows, k), weight.view(parts * n, k)
+        y = _ext().gemm_small_m(flat, w, 0, None, -1) if parts * rows <= SMALL_M_ROWS else gemm(flat, w)
+        return tuple(y[i * rows:(i + 1) * rows, i * n:(i + 1) * n] for i in range(parts))
+    return tuple(gemm(x[i], weight[i]) for i in range(parts))
 
 
 def branch_join(x: Tensor, branches, mult: float, eps: float, w_next):

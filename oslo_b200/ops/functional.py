@@ -236,12 +236,12 @@ def linear_fp32(x: Tensor, weight: Tensor, fused: bool = True) -> Tensor:
     return torch.matmul(x, weight.t()).to(torch.float32)
 
 
-def stacked_linear(x: Tensor, weight: Tensor, fused: bool = True) -> Tensor:
-    """``x[i] @ W[i].T``: ``x`` ``[P, rows, in]``, ``weight`` ``[P, out, in]``."""
+def stacked_linear(x: Tensor, weight: Tensor, fused: bool = True) -> Tuple[Tensor, ...]:
+    """``x[i] @ W[i].T`` for every part ``i``: ``x`` ``[P, rows, in]``, ``weight`` ``[P, out, in]``."""
     if fused and _kn(x, weight):
         from . import cuda_ops
         return cuda_ops.stacked_linear(x, weight)
-    return torch.matmul(x, weight.transpose(1, 2))
+    return torch.matmul(x, weight.transpose(1, 2)).unbind(0)
 
 
 def branch_join(x: Tensor, branches, mult: float, eps: float, w_next, fused: bool = True):

@@ -128,7 +128,8 @@ class PackedLinear(Linear):
 
 
 class StackedLinear(nn.Module):
-    """Bias-free projections of equal size whose inputs differ: weight ``[parts, out, in]``, ``x`` ``[parts, rows, in]``."""
+    """Bias-free projections of equal size whose inputs differ: weight ``[parts, out, in]``, ``x`` ``[parts, rows, in]``; one result
+    per part."""
 
     oslo_fused = False
 
@@ -136,7 +137,7 @@ class StackedLinear(nn.Module):
         super().__init__()
         self.weight = nn.Parameter(torch.empty(parts, out_features, in_features).normal_(std=0.02))
 
-    def forward(self, x: Tensor) -> Tensor:
+    def forward(self, x: Tensor):
         return ops.stacked_linear(x, self.weight, fused=self.oslo_fused)
 
 

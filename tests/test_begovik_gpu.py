@@ -276,9 +276,9 @@ def test_grouped_decode(dtype, batch, heads, groups, dim, vdim, tmax, length):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_products_for_few_and_many_rows(dtype):
-    for rows, k, n in ((1, 64, 40), (3, 128, 96), (20, 64, 48), (70, 64, 24), (200, 72, 13), (5, 30, 9)):
+    for rows, k, n in ((1, 64, 40), (3, 128, 96), (9, 64, 48), (20, 64, 48), (70, 64, 24), (200, 72, 13), (5, 30, 9)):
         x, w = rnd(4, rows, k, dtype=dtype), rnd(4, n, k, dtype=dtype, scale=k ** -0.5)
-        close(ops.stacked_linear(x, w), torch.matmul(x.float(), w.float().transpose(1, 2)), dtype)
+        close(torch.stack(ops.stacked_linear(x, w)), torch.matmul(x.float(), w.float().transpose(1, 2)), dtype)
         y = ops.linear_fp32(x[0], w[0])
         assert y.dtype == torch.float32
         close(y, x[0].float() @ w[0].float().t(), torch.float32)

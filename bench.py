@@ -68,7 +68,7 @@ def parse_args():
     ap.add_argument("--no-e2e", action="store_true")
     ap.add_argument("--mode", default="train", choices=["train", "decode", "fusion", "serving"],
                     help="train: tokens/s of a training step; decode: ms/token of greedy generation with a KV cache; "
-                         "serving: prompt and decode throughput of Moronex beside GPT-J at equal width, heads and layers; "
+                         "serving: prompt and decode throughput of Moronex and Begovik beside GPT-J at equal width, heads and layers; "
                          "fusion: seconds of one GPT-2 small beam-search generate() call before and after fuse() (the "
                          "benchmark behind the reference's published numbers)")
     ap.add_argument("--fusion-dtype", default="fp32", choices=["fp32", "bf16"],
@@ -593,9 +593,23 @@ def serving_config(width, heads, layers, q_rank, kv_rank, experts, vocab=50400):
     return dict(vocab=vocab, width=width, norm={"eps": 1e-5}, layers=out)
 
 
+def begovik_config(width, heads, layers, vocab=50400):
+    """Layers in groups of three: recurrence with a bonus (heads of 64), selective scan over 2 x width channels, attention (4 query
+    heads per key / value head) beside linear attention with constant decays; feed-forwards with as many weights as GPT-J's."""
+    dim = width // heads
+    mlp = {"kind": "dense", "ff": 8 * width // 3 // 64 * 64, "limit": 7.0}
+    left = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": dim, "vdim": dim, "scale": dim ** -0.5, "softcap": 50.0,
+            "rot": {"base": 500000.0, "dims": dim // 2}}
+    right = {"heads": heads, "dim": dim, "vdim": dim, "decay": [1.0 - 2.0 ** (-1 - 9 * i / heads) for i in range(heads)]}
+    kinds = [("wkv", {"heads": width // 64, "dim": 64, "decay_rank": 64}),
+             ("mamba1", {"inner": 2 * width, "state": 16, "dt_rank": width // 16, "conv": 4}), ("parallel", {"left": left, "right": right})]
+    return dict(vocab=vocab, width=width, norm={"eps": 1e-5}, embedding={"scale": width ** 0.5}, residual_mult=0.5,
+                layers=[{"type": kinds[i % 3][0], "mixer": kinds[i % 3][1], "mlp": mlp} for i in range(layers)])
+
+
 def serving_main(args) -> None:
     """One GPU, random weights, bf16: prompt throughput (4 x 2048 tokens) and greedy decoding after 2048-token prompts with 1, 8
-    and 64 sequences (one CUDA-graph replay per token) of Moronex and of GPT-J with the same width, heads and number of
+    and 64 sequences (one CUDA-graph replay per token) of Moronex, Begovik and GPT-J with the same width, heads and number of
     layers. A "step" is one ``GraphedGreedyDecoder.generate`` call; CUDA events around its prompt and its token loop; weights
     and caches are larger than L2. ``--layers`` shortens both models (debug)."""
     import gc
@@ -615,8 +629,10 @@ def serving_main(args) -> None:
     l0, results = ext.launch_count(), {}
     for size, (width, heads, layers, q_rank, kv_rank, experts) in SERVING_SIZES.items():
         layers = args.layers or layers
-        for name in ("moronex", "gptj"):
-            if name == "moronex":
+        for name in ("moronex", "begovik", "gptj"):
+            if name == "begovik":
+                cls, cfg = ob.BegovikForCausalLM, ob.BegovikConfig(**begovik_config(width, heads, layers), torch_dtype=torch.bfloat16)
+            elif name == "moronex":
                 cls, cfg = ob.MoronexForCausalLM, ob.MoronexConfig(**serving_config(width, heads, layers, q_rank, kv_rank, experts),
                                                                    torch_dtype=torch.bfloat16)
             else:
@@ -660,7 +676,7 @@ def serving_main(args) -> None:
         "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
         "ms_per_step": 4 * 2048 / main_rec["prompt_tokens_per_s"] * 1e3, "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
         "dtype": "bf16", "data": "synthetic uniform token ids, random-init weights", "impl": "oslo_b200",
-        "config": {"model": "moronex beside gptj", "global_batch": 4, "seq_len": 2048, "parallelism": "single",
+        "config": {"model": "moronex and begovik beside gptj", "global_batch": 4, "seq_len": 2048, "parallelism": "single",
                    "sizes": {k: dict(zip(("width", "heads", "layers", "q_rank", "kv_rank", "experts"), v)) for k, v in SERVING_SIZES.items()},
                    "l2": "weights + caches per step >> 126 MB L2, no explicit flush"},
         "results": results, "clocks": clocks, "e2e": None, "gpu_launches": ext.launch_count() - l0,

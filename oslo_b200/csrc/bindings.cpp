@@ -891,7 +891,7 @@ Tensor run_recurrence(const RecurrenceRule& r, const Tensor& q, const Tensor& f,
   c10::cuda::CUDAGuard guard(q.device());
   const int sms = dev_state(q.get_device()).sms;
   int nch = chunks > 0 ? static_cast<int>(chunks)
-                       : oslo_recurrence_chunks(static_cast<int>(batch), static_cast<int>(S), static_cast<int>(heads),
+                       : oslo_recurrence_chunks(r.rule, static_cast<int>(batch), static_cast<int>(S), static_cast<int>(heads),
                                                 static_cast<int>(dim), static_cast<int>(vdim), sms);
   const auto f32 = q.options().dtype(at::kFloat);
   Tensor out = at::empty({batch, S, heads, vdim}, f32);
@@ -1229,7 +1229,8 @@ Tensor selective_scan(const Tensor& x, const Tensor& dt, const Tensor& dt_bias, 
                                b.data_ptr(), b.stride(0), c.data_ptr(), c.stride(0), d.data_ptr(), z.data_ptr(), z.stride(0), kp,
                                ld_keep, carried_ptr(state, batch * C * N), out.data_ptr(), nch > 1 ? ws.data_ptr<float>() : nullptr,
                                nch > 1 ? steps.data_ptr<float>() : nullptr, nch, static_cast<int>(batch), static_cast<int>(S),
-                               static_cast<int>(C), static_cast<int>(N), dt_code(x), cur_stream(nch > 1 ? 3 : 1)), "selective_scan");
+                               static_cast<int>(C), static_cast<int>(N), dev_state(x.get_device()).sms, dt_code(x),
+                               cur_stream(nch > 1 ? 3 : 1)), "selective_scan");
   return out;
 }
 

@@ -266,6 +266,13 @@ template <> struct GdMma<__half> {
   }
 };
 
+constexpr float GD_LOG2E = 1.4426950408889634f, GD_LN2 = 0.6931471805599453f;
+__device__ __forceinline__ float gd_exp2(float x) {
+  float r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+  return r;
+}
+
 constexpr int GM_HEADS = 16, GM_KEYS = 64;   // rows of a product; keys per stage, 16 of them per warp
 
 template <int D> constexpr size_t gd_mma_smem() { return static_cast<size_t>(GM_HEADS + 4 * GM_KEYS) * (D + 8) * 2; }
@@ -299,25 +306,29 @@ __global__ void __launch_bounds__(128) grouped_decode_mma_kernel(const GroupedPa
     const int a = e / (p.dim / 8), c = e % (p.dim / 8) * 8;
     *reinterpret_cast<uint4*>(qs + a * PITCH + c) = *reinterpret_cast<const uint4*>(q + a * p.dim + c);
   }
-  auto copy = [&](T* dst, const T* src, int width, int k0) {
-    const int per_row = width / 8;
-    for (int e = tid; e < GM_KEYS * per_row; e += 128) {
-      const int t = e / per_row, c = (e - t * per_row) * 8;
+  // a thread copies the same 16-byte column of every `rows`-th key
+  auto copy = [&](T* dst, const T* src, int width, int rows, int t_first, int c, int k0) {
+    if (t_first >= rows) return;
+#pragma unroll 4
+    for (int t = t_first; t < GM_KEYS; t += rows) {
       const bool ok = k0 + t < t1;
       const uint32_t d32 = smem_u32(dst + t * PITCH + c);
       const int bytes = ok ? 16 : 0;         // 0: the 16 bytes are filled with zeros
       asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d32), "l"(src + static_cast<long long>(ok ? k0 + t : t0) * width + c), "r"(bytes) : "memory");
     }
   };
+  const int k_rows = 128 / (p.dim / 8), k_first = tid / (p.dim / 8), k_col = tid % (p.dim / 8) * 8;
+  const int v_rows = 128 / (p.vdim / 8), v_first = tid / (p.vdim / 8), v_col = tid % (p.vdim / 8) * 8;
   auto fetch = [&](int k0, int buf) {
-    copy(ks + buf * GM_KEYS * PITCH, kb, p.dim, k0);
-    copy(vs + buf * GM_KEYS * PITCH, vb, p.vdim, k0);
+    copy(ks + buf * GM_KEYS * PITCH, kb, p.dim, k_rows, k_first, k_col, k0);
+    copy(vs + buf * GM_KEYS * PITCH, vb, p.vdim, v_rows, v_first, v_col, k0);
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   float o[D / 8][4];
 #pragma unroll
   for (int i = 0; i < D / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
-  float m[2] = {-CUDART_INF_F, -CUDART_INF_F}, s[2] = {0.f, 0.f};     // rows l / 4 and l / 4 + 8
+  float m[2] = {-CUDART_INF_F, -CUDART_INF_F}, s[2] = {0.f, 0.f};     // rows l / 4 and l / 4 + 8; scores in log2 units
+  const float cap = p.softcap * GD_LOG2E, scale = p.softcap > 0.f ? 2.f * p.scale / p.softcap * GD_LOG2E : p.scale * GD_LOG2E;
   if (t0 < t1) fetch(t0, 0);
   for (int k0 = t0, it = 0; k0 < t1; k0 += GM_KEYS, ++it) {
     const int buf = it & 1;
@@ -346,8 +357,8 @@ __global__ void __launch_bounds__(128) grouped_decode_mma_kernel(const GroupedPa
       for (int e = 0; e < 4; ++e) {
         const int pos = k0 + w * 16 + nt * 8 + (l & 3) * 2 + (e & 1);
         const bool vis = pos < t1 && (p.keep == nullptr || pos >= p.n_keep || p.keep[b * p.ld_keep + pos]);
-        float d = c[nt][e] * p.scale;
-        if (p.softcap > 0.f) d = p.softcap - __fdividef(2.f * p.softcap, __expf(2.f * d / p.softcap) + 1.f);   // cap * tanh(d / cap)
+        float d = c[nt][e] * scale;                    // capped: twice the score over the cap, in log2 units
+        if (p.softcap > 0.f) d = cap - __fdividef(2.f * cap, gd_exp2(d) + 1.f);   // cap * tanh(score / cap)
         c[nt][e] = vis ? d : -CUDART_INF_F;
         mx[e >> 1] = fmaxf(mx[e >> 1], c[nt][e]);
       }
@@ -358,7 +369,7 @@ __global__ void __launch_bounds__(128) grouped_decode_mma_kernel(const GroupedPa
       mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 1));
       mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 2));
       ref[i] = mx[i] == -CUDART_INF_F ? 0.f : mx[i];
-      alpha[i] = __expf(m[i] - ref[i]);                // exp(-inf) = 0
+      alpha[i] = gd_exp2(m[i] - ref[i]);               // 2^-inf = 0
       m[i] = mx[i];
       s[i] *= alpha[i];
     }
@@ -366,7 +377,7 @@ __global__ void __launch_bounds__(128) grouped_decode_mma_kernel(const GroupedPa
     for (int nt = 0; nt < 2; ++nt) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        c[nt][e] = __expf(c[nt][e] - ref[e >> 1]);
+        c[nt][e] = gd_exp2(c[nt][e] - ref[e >> 1]);
         s[e >> 1] += c[nt][e];
       }
     }
@@ -397,7 +408,7 @@ __global__ void __launch_bounds__(128) grouped_decode_mma_kernel(const GroupedPa
   for (int i = 0; i < 2; ++i) {
     const int row = (l >> 2) + 8 * i;
     const float top = fmaxf(fmaxf(ms[0][row], ms[1][row]), fmaxf(ms[2][row], ms[3][row]));
-    const float f = m[i] == -CUDART_INF_F ? 0.f : __expf(m[i] - top);
+    const float f = m[i] == -CUDART_INF_F ? 0.f : gd_exp2(m[i] - top);
 #pragma unroll
     for (int dt = 0; dt < D / 8; ++dt)
       *reinterpret_cast<float2*>(red + (w * GM_HEADS + row) * D + dt * 8 + (l & 3) * 2) = make_float2(o[dt][2 * i] * f, o[dt][2 * i + 1] * f);
@@ -412,9 +423,9 @@ __global__ void __launch_bounds__(128) grouped_decode_mma_kernel(const GroupedPa
     const float top = fmaxf(fmaxf(ms[0][tid], ms[1][tid]), fmaxf(ms[2][tid], ms[3][tid]));
     float tot = 0.f;
 #pragma unroll
-    for (int i = 0; i < 4; ++i) tot += ms[i][tid] == -CUDART_INF_F ? 0.f : ls[i][tid] * __expf(ms[i][tid] - top);
+    for (int i = 0; i < 4; ++i) tot += ms[i][tid] == -CUDART_INF_F ? 0.f : ls[i][tid] * gd_exp2(ms[i][tid] - top);
     const long long at = (static_cast<long long>(b) * p.H + h0 + tid) * p.splits + sp;
-    p.stat[at * 2] = top;
+    p.stat[at * 2] = top * GD_LN2;
     p.stat[at * 2 + 1] = tot;
   }
 }

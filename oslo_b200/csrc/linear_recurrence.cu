@@ -94,7 +94,7 @@ constexpr float REC_MIN_PERIOD = 1e-15f;   // RULE_DECAY: the smallest product o
 
 // G lanes per column group. STATE_ONLY: no outputs, start from zero, also the chunk's total decay per row
 template <typename T, int G, bool STATE_ONLY, int RULE>
-__global__ void __launch_bounds__(256, 2) recurrence_kernel(const RecParams p) {
+__global__ void __launch_bounds__(RULE == RULE_BONUS ? 128 : 256, RULE == RULE_BONUS ? 3 : 2) recurrence_kernel(const RecParams p) {
   constexpr int DP = REC_ROWS * G;
   constexpr int CONV = DP >= 256 ? 1 : 256 / DP;
   constexpr int PARTS = DP > 32 ? DP / 32 : 1;               // RULE_BONUS: partial sums of r . (u k) per token
@@ -612,15 +612,15 @@ __global__ void __launch_bounds__(256) recurrence_step_kernel(const StepParams p
   }
 }
 
-// threads of a block: the column groups of a head, at most 256
-static int rec_threads(int g, int vdim) {
+// threads of a block: the column groups of a head, at most 256 (128 with the bonus rule, whose decays need more registers)
+static int rec_threads(int g, int vdim, int rule) {
   const int groups = (vdim + REC_COLS - 1) / REC_COLS;
-  return std::min(256, (groups * g + 31) / 32 * 32);
+  return std::min(rule == RULE_BONUS ? 128 : 256, (groups * g + 31) / 32 * 32);
 }
 
 template <typename T, int G, bool STATE_ONLY, int RULE>
 static int rec_launch(const RecParams& p, cudaStream_t st) {
-  const int nt = rec_threads(G, p.vdim), cols = nt / G * REC_COLS;
+  const int nt = rec_threads(G, p.vdim, RULE), cols = nt / G * REC_COLS;
   const int rows = (STATE_ONLY ? 1 : 2) + (RULE == RULE_BONUS ? 1 : 0);
   const size_t smem = static_cast<size_t>(REC_TB) * ((rows * REC_ROWS * G + cols + (RULE == RULE_BONUS ? 2 * p.dim_pad : 0)) * sizeof(float) +
                                                      2 * ((STATE_ONLY ? 1 : 2) * p.dim_pad + cols) * sizeof(T));
@@ -655,11 +655,11 @@ static int rec_dispatch(const RecParams& p, int rule, cudaStream_t st) {
 }  // namespace oslo
 
 // how many chunks a prompt of S tokens is cut into so that the recurrence fills the GPU
-extern "C" int oslo_recurrence_chunks(int B, int S, int H, int dim, int vdim, int num_sms) {
+extern "C" int oslo_recurrence_chunks(int rule, int B, int S, int H, int dim, int vdim, int num_sms) {
   using namespace oslo;
   int g = 1;
   while (REC_ROWS * g < dim && g < 32) g *= 2;
-  const int nt = rec_threads(g, vdim), cols = nt / g * REC_COLS;
+  const int nt = rec_threads(g, vdim, rule), cols = nt / g * REC_COLS;
   const long long ctas = static_cast<long long>(B) * H * ((vdim + cols - 1) / cols);
   if (S < 128) return 1;
   // an SM's blocks share its FMA pipes: time ~ (blocks of the fullest SM) x (tokens per chunk); more than one chunk adds the

@@ -233,7 +233,7 @@ int oslo_gated_rms_norm(const float* o, const void* w, const void* gate, long lo
 // nchunks > 1 (oslo_recurrence_chunks) needs ws [B, nchunks, H, dim, vdim] and decay [B, nchunks, H, dim] fp32.
 // rule 0: f are forget-gate logits with f_bias and lower bounds [H * dim]; 1: f are keys, head_decay [H] fp32; 2: f are keys,
 // f_bias = w0 and lower = u [H * dim], z the decay logits fp32 [B * S, H * dim]
-int oslo_recurrence_chunks(int B, int S, int H, int dim, int vdim, int num_sms);
+int oslo_recurrence_chunks(int rule, int B, int S, int H, int dim, int vdim, int num_sms);
 int oslo_recurrence(int rule, const void* q, long long ldq, const void* f, long long ldf, const void* v, long long ldv,
                     const void* f_bias, const void* lower, const float* z, long long ldz, const float* head_decay,
                     const uint8_t* keep, long long ld_keep, float* state, float* out, float* ws, float* decay, int nchunks, int B,
@@ -303,7 +303,7 @@ int oslo_scan_chunks(int B, int S, int C, int N, int num_sms);
 int oslo_selective_scan(const void* x, long long ldx, const float* dt, long long lddt, const void* dt_bias, const void* a_log,
                         const void* b, long long ldb, const void* c, long long ldc, const void* d, const void* z, long long ldz,
                         const uint8_t* keep, long long ld_keep, float* state, void* out, float* ws, float* steps, int nchunks, int B,
-                        int S, int C, int N, int dtype, cudaStream_t stream);
+                        int S, int C, int N, int num_sms, int dtype, cudaStream_t stream);
 // one token per row; the step logits are w_dt [C, rank] . dt [B, rank]
 int oslo_scan_step(const void* x, long long ldx, const void* dt, long long lddt, const void* w_dt, int rank, const void* dt_bias,
                    const void* a_log, const void* b, long long ldb, const void* c, long long ldc, const void* d, const void* z,

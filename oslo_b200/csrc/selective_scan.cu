@@ -5,7 +5,8 @@
 //   scan:         s_t = softplus(dt_t + dt_bias),  S[n] <- exp(s_t A[n]) S[n] + s_t x_t B_t[n],  A = -exp(a_log)
 //                 out_t = (sum_n S[n] C_t[n] + d x_t) * silu(z_t)
 //
-// Scan over a prompt (selective_scan_kernel): G lanes share a channel, each keeps NS of its states in registers. A stage of
+// Scan over a prompt (selective_scan_kernel): G lanes share a channel, each keeps NS of its states in registers (more lanes than
+// needed when there are few channels). A stage of
 // tokens is fetched one stage ahead with cp.async; step sizes and s_t x_t are computed once per (token, channel), B and C are
 // broadcast from shared memory, the outputs pass through shared memory to the gated, coalesced store. One exponential per
 // state and token bounds it (16 per cycle and SM). When the channels do not fill the GPU the prompt is cut into chunks:
@@ -476,10 +477,12 @@ __global__ void __launch_bounds__(256) scan_step_kernel(const ScanStepParams p) 
   static_cast<T*>(p.out)[static_cast<long long>(b) * p.C + c] = Num<T>::from(y * silu_f(Num<T>::to(static_cast<const T*>(p.z)[b * p.ldz + c])));
 }
 
-// lanes per channel and states per lane
-static void scan_split(int N, int& g, int& ns) {
+// lanes per channel and states per lane: as few lanes as hold the states, more of them when the channels alone leave fewer than
+// four warps for each of an SM's four schedulers (a token's exponentials are too few to hide their own latency)
+static void scan_split(long long channels, int N, int num_sms, int& g, int& ns) {
   g = 1;
-  while (g < 32 && N > 16 * g) g *= 2;
+  while (N > 16 * g) g *= 2;
+  while (g < 16 && channels * g < 512ll * num_sms && (N + 2 * g - 1) / (2 * g) >= 3) g *= 2;
   ns = ((N + g - 1) / g + 3) / 4 * 4;
 }
 
@@ -498,18 +501,14 @@ static int scan_launch(const ScanParams& p, cudaStream_t st) {
 }
 template <typename T, int G, bool STATE_ONLY>
 static int scan_states(const ScanParams& p, int ns, cudaStream_t st) {
-  if constexpr (G == 1) {                    // with more lanes every lane holds more than half of 16
-    if (ns == 4) return scan_launch<T, 4, G, STATE_ONLY>(p, st);
-    if (ns == 8) return scan_launch<T, 8, G, STATE_ONLY>(p, st);
-  }
+  if (ns == 4) return scan_launch<T, 4, G, STATE_ONLY>(p, st);
+  if (ns == 8) return scan_launch<T, 8, G, STATE_ONLY>(p, st);
   if (ns == 12) return scan_launch<T, 12, G, STATE_ONLY>(p, st);
   if (ns == 16) return scan_launch<T, 16, G, STATE_ONLY>(p, st);
   return -3;
 }
 template <typename T, bool STATE_ONLY>
-static int scan_dispatch(const ScanParams& p, cudaStream_t st) {
-  int g, ns;
-  scan_split(p.N, g, ns);
+static int scan_dispatch(const ScanParams& p, int g, int ns, cudaStream_t st) {
   if (g == 1) return scan_states<T, 1, STATE_ONLY>(p, ns, st);
   if (g == 2) return scan_states<T, 2, STATE_ONLY>(p, ns, st);
   if (g == 4) return scan_states<T, 4, STATE_ONLY>(p, ns, st);
@@ -552,11 +551,8 @@ extern "C" int oslo_causal_conv_silu(const void* x, long long ldx, const void* w
   const size_t te = dtype == OSLO_DT_FP32 ? 4 : 2;
   const bool vec = C % 4 == 0 && ldx % 4 == 0 && aligned_to(x, 4 * te) && aligned_to(bias, 4 * te) && aligned_to(out, 4 * te);
 #define CV_GO(V, N) causal_conv_kernel<T, V, N><<<dim3((C + 128 * V - 1) / (128 * V), runs, B), 128, 0, stream>>>(p)
-  const bool wide = vec && te == 2 && C % 8 == 0 && ldx % 8 == 0 && aligned_to(x, 16) && aligned_to(bias, 16) && aligned_to(out, 16) &&
-                    static_cast<long long>(B) * runs * C >= 148 * 1024 * 8;
   OSLO_DISPATCH_T(dtype, {
-    if (taps == 4 && wide) CV_GO(8, 4);
-    else if (taps == 4 && vec) CV_GO(4, 4);
+    if (taps == 4 && vec) CV_GO(4, 4);
     else if (taps == 3 && vec) CV_GO(4, 3);
     else if (vec) CV_GO(4, 0);
     else CV_GO(1, 0);
@@ -568,18 +564,18 @@ extern "C" int oslo_causal_conv_silu(const void* x, long long ldx, const void* w
 extern "C" int oslo_scan_chunks(int B, int S, int C, int N, int num_sms) {
   using namespace oslo;
   int g, ns;
-  scan_split(N, g, ns);
+  scan_split(static_cast<long long>(B) * C, N, num_sms, g, ns);
   const int ch = SC_THREADS / g;
   const long long ctas = static_cast<long long>(B) * ((C + ch - 1) / ch);
   if (S < 128) return 1;
-  // an SM's blocks share its exponential units; one block (a warp per quarter) keeps them about 60 % busy
+  // an SM's blocks share its exponential units, which fewer than four blocks do not keep busy
   int best = 1;
   double best_cost = 1e30;
   for (int n = 1; n <= S / 64 && n <= 64; ++n) {
     const double per = static_cast<double>(S) / n;
     const auto fullest = [&](long long blocks) { return static_cast<double>((blocks + num_sms - 1) / num_sms); };
-    const double c3 = std::max(1.6, fullest(ctas * n)) * per;
-    const double c1 = n > 1 ? std::max(1.6, fullest(ctas * (n - 1))) * per * 0.8 + 40.0 : 0.0;
+    const double c3 = std::max(3.5, fullest(ctas * n)) * per;
+    const double c1 = n > 1 ? std::max(3.5, fullest(ctas * (n - 1))) * per * 0.8 + 160.0 : 0.0;
     if (c3 + c1 < best_cost) { best_cost = c3 + c1; best = n; }
   }
   return best;
@@ -588,7 +584,8 @@ extern "C" int oslo_scan_chunks(int B, int S, int C, int N, int num_sms) {
 extern "C" int oslo_selective_scan(const void* x, long long ldx, const float* dt, long long lddt, const void* dt_bias,
                                    const void* a_log, const void* b, long long ldb, const void* c, long long ldc, const void* d,
                                    const void* z, long long ldz, const uint8_t* keep, long long ld_keep, float* state, void* out,
-                                   float* ws, float* steps, int nchunks, int B, int S, int C, int N, int dtype, cudaStream_t stream) {
+                                   float* ws, float* steps, int nchunks, int B, int S, int C, int N, int num_sms, int dtype,
+                                   cudaStream_t stream) {
   using namespace oslo;
   if (B <= 0 || S <= 0 || C <= 0) return 0;
   if (N <= 0 || N > 256 || nchunks < 1 || static_cast<long long>(B) * nchunks > 65535) return -1;
@@ -598,10 +595,11 @@ extern "C" int oslo_selective_scan(const void* x, long long ldx, const float* dt
   p.B = B; p.S = S; p.C = C; p.N = N;
   p.vec16 = C % 8 == 0 && ldx % 8 == 0 && ldz % 8 == 0 && lddt % 4 == 0 && aligned_to(x, 16) && aligned_to(z, 16) && aligned_to(dt, 16);
   const long long per = static_cast<long long>(C) * N;
-  int rc = 0;
+  int rc = 0, g, ns;
+  scan_split(static_cast<long long>(B) * C, N, num_sms, g, ns);
   if (nchunks == 1) {
     p.chunk = S; p.nchunks = 1; p.s_in = state; p.s_out = state; p.s_batch = per;
-    OSLO_DISPATCH_T(dtype, { rc = scan_dispatch<T, false>(p, stream); });
+    OSLO_DISPATCH_T(dtype, { rc = scan_dispatch<T, false>(p, g, ns, stream); });
     return rc;
   }
   if (ws == nullptr || steps == nullptr) return -1;
@@ -609,7 +607,7 @@ extern "C" int oslo_selective_scan(const void* x, long long ldx, const float* dt
   p.s_batch = per * nchunks; p.s_chunk = per;
   p.s_out = ws; p.steps = steps;
   p.nchunks = nchunks - 1;             // nobody starts from the last chunk's state
-  OSLO_DISPATCH_T(dtype, { rc = scan_dispatch<T, true>(p, stream); });
+  OSLO_DISPATCH_T(dtype, { rc = scan_dispatch<T, true>(p, g, ns, stream); });
   if (rc) return rc;
   OSLO_DISPATCH_T(dtype, {
     scan_chunks_kernel<T><<<dim3(static_cast<unsigned>((per + 255) / 256), B), 256, 0, stream>>>(
@@ -619,7 +617,7 @@ extern "C" int oslo_selective_scan(const void* x, long long ldx, const float* dt
   if (rc) return rc;
   p.nchunks = nchunks;
   p.s_in = ws; p.s_out = nullptr; p.s_end = state;
-  OSLO_DISPATCH_T(dtype, { rc = scan_dispatch<T, false>(p, stream); });
+  OSLO_DISPATCH_T(dtype, { rc = scan_dispatch<T, false>(p, g, ns, stream); });
   return rc;
 }
 

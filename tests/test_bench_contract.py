@@ -39,6 +39,8 @@ def test_serving_sizes_are_valid_configurations():
         cfg = ob.MoronexConfig(**bench.serving_config(*size))
         assert cfg.num_hidden_layers == size[2] and {l["type"] for l in cfg.layers} == {"latent_attention", "hgrn2"}
         assert any(l["mixer"].get("kv_from") is not None for l in cfg.layers)
+        cfg = ob.BegovikConfig(**bench.begovik_config(*size[:3]))
+        assert cfg.num_hidden_layers == size[2] and {l["type"] for l in cfg.layers} == {"wkv", "mamba1", "parallel"}
 
 
 def _reference_installed() -> bool:

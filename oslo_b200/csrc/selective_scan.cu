@@ -178,8 +178,18 @@ constexpr float SC_LOG2E = 1.4426950408889634f;
 
 // 32-bit models get the accurate functions
 template <typename T> __device__ __forceinline__ float softplus_t(float z) {
-  if (z > 20.f) return z;
-  return sizeof(T) == 4 ? log1pf(expf(z)) : log1pf(__expf(z));
+  if (sizeof(T) == 4) return z > 20.f ? z : log1pf(expf(z));
+  // max(z, 0) + log(1 + e), e = exp(-|z|): log(1 + e) = 2 atanh(r), r = e / (2 + e) <= 1/3, by the series of atanh (the first term
+  // left out is below 1e-8 of the sum); small e keep their relative precision
+  const float e = __expf(-fabsf(z)), r = __fdividef(e, 2.f + e), q = r * r;
+  float s = fmaf(q, 1.f / 15.f, 1.f / 13.f);
+  s = fmaf(q, s, 1.f / 11.f);
+  s = fmaf(q, s, 1.f / 9.f);
+  s = fmaf(q, s, 1.f / 7.f);
+  s = fmaf(q, s, 1.f / 5.f);
+  s = fmaf(q, s, 1.f / 3.f);
+  s = fmaf(q, s, 1.f);
+  return fmaf(2.f * r, s, fmaxf(z, 0.f));
 }
 // exp(a): 16-bit models pass a * log2(e)
 template <typename T> __device__ __forceinline__ float decay_t(float a) {
@@ -189,7 +199,7 @@ template <typename T> __device__ __forceinline__ float decay_t(float a) {
   return r;
 }
 template <typename T> __device__ __forceinline__ float decay_rate(float a_log) {
-  return sizeof(T) == 4 ? -expf(a_log) : -expf(a_log) * SC_LOG2E;
+  return sizeof(T) == 4 ? -expf(a_log) : -__expf(a_log) * SC_LOG2E;
 }
 
 struct ScanParams {
@@ -208,6 +218,7 @@ struct ScanParams {
   long long s_batch, s_chunk;                // element strides of s_in / s_out over batch rows and chunks
   float* steps;                              // STATE_ONLY: sum of the chunk's steps [B, nchunks, C]
   int vec16;                                 // rows of dt, x and z start at 16-byte boundaries, C is a multiple of 8
+  int bc16;                                  // rows of b and c start at 16-byte boundaries, N is a multiple of 8
 };
 
 template <typename T, int NS, int G, bool STATE_ONLY>
@@ -221,7 +232,10 @@ __global__ void __launch_bounds__(SC_THREADS) selective_scan_kernel(const ScanPa
   float* y_s = sx_s + SC_TB * CH;                        // [SC_TB][CH], not STATE_ONLY
   float* draw = y_s + (STATE_ONLY ? 0 : SC_TB * CH);     // [2][SC_TB][CH] raw step logits
   T* xraw = reinterpret_cast<T*>(draw + 2 * SC_TB * CH); // [2][SC_TB][CH]
-  T* zraw = xraw + 2 * SC_TB * CH;                       // [2][SC_TB][CH], not STATE_ONLY
+  T* braw = xraw + 2 * SC_TB * CH;                       // [2][SC_TB][NP8]
+  constexpr int NP8 = (NP + 7) / 8 * 8;
+  T* craw = braw + 2 * SC_TB * NP8;                      // [2][SC_TB][NP8], not STATE_ONLY
+  T* zraw = craw + (STATE_ONLY ? 0 : 2 * SC_TB * NP8);   // [2][SC_TB][CH], not STATE_ONLY
   const int tid = threadIdx.x, g = tid % G, ch = tid / G;
   const int b = blockIdx.y / p.nchunks, ck = blockIdx.y % p.nchunks;
   const int c0 = blockIdx.x * CH, nc = min(CH, p.C - c0), my_c = c0 + ch;
@@ -276,6 +290,30 @@ __global__ void __launch_bounds__(SC_THREADS) selective_scan_kernel(const ScanPa
         }
       }
     }
+    T* bd = braw + buf * SC_TB * NP8;
+    T* cd = craw + buf * SC_TB * NP8;
+    if (p.bc16) {
+      constexpr int V = 16 / sizeof(T);
+      for (int e = tid; e < n * (NP8 / V); e += SC_THREADS) {
+        const int t = e / (NP8 / V), i = e % (NP8 / V) * V;
+        if (i < p.N) {
+          const uint32_t b32 = static_cast<uint32_t>(__cvta_generic_to_shared(bd + t * NP8 + i));
+          asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(b32), "l"(bt + (t0 + t) * p.ldb + i) : "memory");
+          if (!STATE_ONLY) {
+            const uint32_t c32 = static_cast<uint32_t>(__cvta_generic_to_shared(cd + t * NP8 + i));
+            asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(c32), "l"(ct + (t0 + t) * p.ldc + i) : "memory");
+          }
+        }
+      }
+    } else {
+      for (int e = tid; e < n * NP8; e += SC_THREADS) {
+        const int t = e / NP8, i = e % NP8;
+        if (i < p.N) {
+          bd[e] = bt[(t0 + t) * p.ldb + i];
+          if (!STATE_ONLY) cd[e] = ct[(t0 + t) * p.ldc + i];
+        }
+      }
+    }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   float total = 0.f;
@@ -288,12 +326,12 @@ __global__ void __launch_bounds__(SC_THREADS) selective_scan_kernel(const ScanPa
     } else {
       asm volatile("cp.async.wait_group 0;" ::: "memory");
     }
+    __syncthreads();
     for (int e = tid; e < n * NP; e += SC_THREADS) {
       const int t = e / NP, i = e % NP;
-      bs[e] = i < p.N ? Num<T>::to(bt[(t0 + t) * p.ldb + i]) : 0.f;
-      if (!STATE_ONLY) cs[e] = i < p.N ? Num<T>::to(ct[(t0 + t) * p.ldc + i]) : 0.f;
+      bs[e] = i < p.N ? Num<T>::to(braw[(buf * SC_TB + t) * NP8 + i]) : 0.f;
+      if (!STATE_ONLY) cs[e] = i < p.N ? Num<T>::to(craw[(buf * SC_TB + t) * NP8 + i]) : 0.f;
     }
-    __syncthreads();
     {
       const int c = tid % CH;
       const float bias = c < nc ? Num<T>::to(static_cast<const T*>(p.dt_bias)[c0 + c]) : 0.f;
@@ -386,6 +424,18 @@ __global__ void __launch_bounds__(256) scan_chunks_kernel(float* __restrict__ ws
 
 // ------------------------------------------------------------------ selective scan, one token per row
 constexpr int ST_CH = 32, ST_ROWS = 8;   // channels and rows of a block
+constexpr int ST_PARTS = 4;              // MMA: warps that share the step projection of 16 channels
+
+// D[channel][row] += W[channel][k] dt[row][k] for 16 channels, 8 rows and 16 k
+__device__ __forceinline__ void st_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1, __nv_bfloat16) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void st_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1, __half) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.f16.f16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void st_mma(float (&)[4], const uint32_t (&)[4], uint32_t, uint32_t, float) {}
 
 struct ScanStepParams {
   const void* x; long long ldx;
@@ -400,15 +450,16 @@ struct ScanStepParams {
   int B, C, N;
 };
 
-// thread = (row, channel)
-template <typename T, int VEC, int SVEC>
+// thread = (row, channel). MMA (16-bit types, rank a multiple of 16, even strides): the step projection on tensor cores
+template <typename T, int VEC, int SVEC, bool MMA>
 __global__ void __launch_bounds__(256) scan_step_kernel(const ScanStepParams p) {
   extern __shared__ float4 st_smem[];
+  __shared__ float part[MMA ? ST_PARTS : 1][MMA ? ST_CH : 1][MMA ? ST_ROWS + 1 : 1];
   const int ldd = (p.rank + 3) / 4 * 4, ldw = ldd + 4;   // reads of four elements by 32 rows without conflicts
-  float* dts = reinterpret_cast<float*>(st_smem);        // [ST_ROWS][ldd]
-  T* ws = reinterpret_cast<T*>(dts + ST_ROWS * ldd);     // [ST_CH][ldw]
-  float* bs = reinterpret_cast<float*>(ws + ST_CH * ldw);   // [ST_ROWS][N]
+  float* bs = reinterpret_cast<float*>(st_smem);         // [ST_ROWS][N]
   float* cs = bs + ST_ROWS * p.N;                        // [ST_ROWS][N]
+  float* dts = cs + ST_ROWS * p.N;                       // [ST_ROWS][ldd], not MMA
+  T* ws = reinterpret_cast<T*>(dts + ST_ROWS * ldd);     // [ST_CH][ldw], not MMA
   const int tid = threadIdx.x, lane = tid & 31, r = tid >> 5;
   const int c0 = blockIdx.x * ST_CH, b0 = blockIdx.y * ST_ROWS, nb = min(ST_ROWS, p.B - b0), nc = min(ST_CH, p.C - c0);
   const int c = c0 + lane, b = b0 + r;
@@ -419,14 +470,34 @@ __global__ void __launch_bounds__(256) scan_step_kernel(const ScanStepParams p) 
 #pragma unroll
   for (int a = 0; a < AHEAD; ++a)
     if (mine && a * SVEC < p.N) load_vec<float, SVEC>(s + a * SVEC, ahead[a]);
-  for (int j = tid / 8; j < nc; j += 32) {               // eight threads per row of the step projection
-    const T* w = static_cast<const T*>(p.w_dt) + static_cast<long long>(c0 + j) * p.rank;
+  if constexpr (MMA) {
+    const int j = (r & 1) * 16 + lane / 4, k2 = lane % 4 * 2;             // channels j and j + 8 of the fragments; row lane / 4
+    const T* w0 = static_cast<const T*>(p.w_dt) + static_cast<long long>(c0 + j) * p.rank + k2;
+    const T* w1 = w0 + 8ll * p.rank;
+    const T* d = static_cast<const T*>(p.dt) + (b0 + lane / 4) * p.lddt + k2;
+    const bool on0 = j < nc, on1 = j + 8 < nc, row = lane / 4 < nb;
+    float z[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 2
+    for (int k = r / 2 * 16; k < p.rank; k += 16 * ST_PARTS) {
+      auto pair = [&](bool ok, const T* at) { return ok ? *reinterpret_cast<const uint32_t*>(at + k) : 0u; };
+      const uint32_t a[4] = {pair(on0, w0), pair(on1, w1), pair(on0, w0 + 8), pair(on1, w1 + 8)};
+      st_mma(z, a, pair(row, d), pair(row, d + 8), T());
+    }
+    part[r / 2][j][k2] = z[0];
+    part[r / 2][j][k2 + 1] = z[1];
+    part[r / 2][j + 8][k2] = z[2];
+    part[r / 2][j + 8][k2 + 1] = z[3];
+  } else {
+    for (int j = tid / 8; j < nc; j += 32) {             // eight threads per row of the step projection
+      const T* w = static_cast<const T*>(p.w_dt) + static_cast<long long>(c0 + j) * p.rank;
 #pragma unroll 4
-    for (int k = tid % 8 * VEC; k < p.rank; k += 8 * VEC)
-      *reinterpret_cast<Pack<T, VEC>*>(ws + j * ldw + k) = *reinterpret_cast<const Pack<T, VEC>*>(w + k);
+      for (int k = tid % 8 * VEC; k < p.rank; k += 8 * VEC)
+        *reinterpret_cast<Pack<T, VEC>*>(ws + j * ldw + k) = *reinterpret_cast<const Pack<T, VEC>*>(w + k);
+    }
   }
   if (r < nb) {                                          // a warp per row
-    for (int k = lane; k < ldd; k += 32) dts[r * ldd + k] = k < p.rank ? Num<T>::to(static_cast<const T*>(p.dt)[b * p.lddt + k]) : 0.f;
+    if (!MMA)
+      for (int k = lane; k < ldd; k += 32) dts[r * ldd + k] = k < p.rank ? Num<T>::to(static_cast<const T*>(p.dt)[b * p.lddt + k]) : 0.f;
     for (int k = lane; k < p.N; k += 32) {
       bs[r * p.N + k] = Num<T>::to(static_cast<const T*>(p.b)[b * p.ldb + k]);
       cs[r * p.N + k] = Num<T>::to(static_cast<const T*>(p.c)[b * p.ldc + k]);
@@ -438,7 +509,11 @@ __global__ void __launch_bounds__(256) scan_step_kernel(const ScanStepParams p) 
   if (p.keep == nullptr || p.keep[b * p.ld_keep]) {
     float z0 = 0.f, z1 = 0.f;
     int k = 0;
-    if (VEC >= 4) {
+    if constexpr (MMA) {
+#pragma unroll
+      for (int u = 0; u < ST_PARTS; ++u) z0 += part[u][lane][r];
+      k = p.rank;
+    } else if (VEC >= 4) {
 #pragma unroll 4
       for (; k + 4 <= p.rank; k += 4) {
         float w[4];
@@ -455,12 +530,14 @@ __global__ void __launch_bounds__(256) scan_step_kernel(const ScanStepParams p) 
   const T* al = static_cast<const T*>(p.a_log) + static_cast<long long>(c) * p.N;
   float y = 0.f;
   auto update = [&](int n, float (&sv)[SVEC]) {
-    float av[SVEC];
+    float av[SVEC], bv[SVEC], cv[SVEC];
     load_vec<T, SVEC>(al + n, av);
+    load_vec<float, SVEC>(bs + r * p.N + n, bv);
+    load_vec<float, SVEC>(cs + r * p.N + n, cv);
 #pragma unroll
     for (int i = 0; i < SVEC; ++i) {
-      sv[i] = fmaf(decay_t<T>(st * decay_rate<T>(av[i])), sv[i], sx * bs[r * p.N + n + i]);
-      y = fmaf(sv[i], cs[r * p.N + n + i], y);
+      sv[i] = fmaf(decay_t<T>(st * decay_rate<T>(av[i])), sv[i], sx * bv[i]);
+      y = fmaf(sv[i], cv[i], y);
     }
     store_vec<float, SVEC>(s + n, sv);
   };
@@ -490,7 +567,7 @@ template <typename T, int NS, int G, bool STATE_ONLY>
 static int scan_launch(const ScanParams& p, cudaStream_t st) {
   constexpr int CH = SC_THREADS / G;
   const size_t smem = static_cast<size_t>(SC_TB) * ((STATE_ONLY ? 1 : 2) * NS * G + (STATE_ONLY ? 2 : 3) * CH + 2 * CH) * sizeof(float) +
-                      static_cast<size_t>(2) * SC_TB * CH * (STATE_ONLY ? 1 : 2) * sizeof(T);
+                      static_cast<size_t>(2) * SC_TB * (CH + (NS * G + 7) / 8 * 8) * (STATE_ONLY ? 1 : 2) * sizeof(T);
   if (smem > 44 * 1024) {      // static arrays come on top
     cudaError_t e = cudaFuncSetAttribute(selective_scan_kernel<T, NS, G, STATE_ONLY>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          static_cast<int>(smem));
@@ -594,6 +671,7 @@ extern "C" int oslo_selective_scan(const void* x, long long ldx, const float* dt
   p.b = b; p.ldb = ldb; p.c = c; p.ldc = ldc; p.z = z; p.ldz = ldz; p.keep = keep; p.ld_keep = ld_keep; p.out = out;
   p.B = B; p.S = S; p.C = C; p.N = N;
   p.vec16 = C % 8 == 0 && ldx % 8 == 0 && ldz % 8 == 0 && lddt % 4 == 0 && aligned_to(x, 16) && aligned_to(z, 16) && aligned_to(dt, 16);
+  p.bc16 = N % 8 == 0 && ldb % 8 == 0 && ldc % 8 == 0 && aligned_to(b, 16) && aligned_to(c, 16);
   const long long per = static_cast<long long>(C) * N;
   int rc = 0, g, ns;
   scan_split(static_cast<long long>(B) * C, N, num_sms, g, ns);
@@ -631,23 +709,26 @@ extern "C" int oslo_scan_step(const void* x, long long ldx, const void* dt, long
   ScanStepParams p{x, ldx, dt, lddt, w_dt, rank, dt_bias, a_log, d, b, c, ldb, ldc, z, ldz, keep, ld_keep, state, out, B, C, N};
   const size_t te = dtype == OSLO_DT_FP32 ? 4 : 2;
   const size_t ldd = (rank + 3) / 4 * 4;
-  const size_t smem = (ST_ROWS * (ldd + 2 * static_cast<size_t>(N))) * sizeof(float) + ST_CH * (ldd + 4) * te;
+  const bool mma = te == 2 && rank % 16 == 0 && lddt % 2 == 0 && aligned_to(w_dt, 4) && aligned_to(dt, 4);
+  const size_t smem = ST_ROWS * 2 * static_cast<size_t>(N) * sizeof(float) + (mma ? 0 : ST_ROWS * ldd * sizeof(float) + ST_CH * (ldd + 4) * te);
   if (smem > 200 * 1024) return -3;
   const bool vec = rank % 4 == 0 && aligned_to(w_dt, 4 * te), svec = N % 4 == 0 && aligned_to(state, 16) && aligned_to(a_log, 4 * te);
-#define SS_GO(V, SV)                                                                                              \
-  {                                                                                                               \
-    if (smem > 40 * 1024) {                                                                                       \
-      cudaError_t e = cudaFuncSetAttribute(scan_step_kernel<T, V, SV>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
-                                           static_cast<int>(smem));                                               \
-      if (e != cudaSuccess) return static_cast<int>(e);                                                           \
-    }                                                                                                             \
-    scan_step_kernel<T, V, SV><<<dim3((C + ST_CH - 1) / ST_CH, (B + ST_ROWS - 1) / ST_ROWS), 256, smem, stream>>>(p); \
+#define SS_GO(V, SV, M)                                                                                              \
+  {                                                                                                                  \
+    if (smem > 40 * 1024) {                                                                                          \
+      cudaError_t e = cudaFuncSetAttribute(scan_step_kernel<T, V, SV, M>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
+                                           static_cast<int>(smem));                                                  \
+      if (e != cudaSuccess) return static_cast<int>(e);                                                              \
+    }                                                                                                                \
+    scan_step_kernel<T, V, SV, M><<<dim3((C + ST_CH - 1) / ST_CH, (B + ST_ROWS - 1) / ST_ROWS), 256, smem, stream>>>(p); \
   }
   OSLO_DISPATCH_T(dtype, {
-    if (vec && svec) SS_GO(4, 4)
-    else if (vec) SS_GO(4, 1)
-    else if (svec) SS_GO(1, 4)
-    else SS_GO(1, 1)
+    if (mma && svec) SS_GO(1, 4, true)
+    else if (mma) SS_GO(1, 1, true)
+    else if (vec && svec) SS_GO(4, 4, false)
+    else if (vec) SS_GO(4, 1, false)
+    else if (svec) SS_GO(1, 4, false)
+    else SS_GO(1, 1, false)
   });
 #undef SS_GO
   return static_cast<int>(cudaGetLastError());

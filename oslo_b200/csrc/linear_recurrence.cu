@@ -668,12 +668,16 @@ extern "C" int oslo_recurrence_chunks(int rule, int B, int S, int H, int dim, in
   double best_cost = 1e30;
   for (int n = 1; n <= S / 64 && n <= 64; ++n) {
     const double per = static_cast<double>(S) / n;
-    // in units of 256 threads
-    const auto fullest = [&](long long blocks) { return static_cast<double>((blocks + num_sms - 1) / num_sms) * nt / 256.0; };
-    // fewer than 512 threads on an SM leave its pipes partly idle
-    const double c3 = std::max(1.4, fullest(ctas * n)) * per;
+    // the fullest SM runs its blocks in waves of as many as fit; in units of 256 threads, of which too few leave its pipes partly idle
+    const int fit = std::max(1, (rule == RULE_BONUS ? 384 : 512) / nt);
+    const auto time = [&](long long blocks) {
+      const int most = static_cast<int>((blocks + num_sms - 1) / num_sms), waves = most / fit, rest = most % fit;
+      const double unit = nt / 256.0;
+      return waves * fit * unit + (rest ? std::max(waves ? 1.0 : 1.4, rest * unit) : 0.0);
+    };
+    const double c3 = time(ctas * n) * per;
     // ... and the states' four trips through memory (16 bytes per element, in units of one token's update)
-    const double c1 = n > 1 ? std::max(1.4, fullest(ctas * (n - 1))) * per * 0.67 + 40.0 + 0.094 * B * H * n : 0.0;
+    const double c1 = n > 1 ? time(ctas * (n - 1)) * per * 0.67 + 40.0 + 0.094 * B * H * n : 0.0;
     if (c3 + c1 < best_cost) { best_cost = c3 + c1; best = n; }
   }
   return best;

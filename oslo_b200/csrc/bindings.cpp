@@ -107,6 +107,11 @@ Tensor gemm(const Tensor& a, const Tensor& b, int64_t a_mn, int64_t b_mn, const 
     d = at::empty({M, N}, a.options().dtype(out_f32 ? at::kFloat : a.scalar_type()));
   }
   if (M == 0 || N == 0) return d;
+  // the epilogue moves 32 columns of a row in 16-byte pieces
+  const auto rows16 = [&](const Tensor& t) {
+    return N < 32 || (t.stride(0) * t.element_size() % 16 == 0 && reinterpret_cast<uintptr_t>(t.data_ptr()) % 16 == 0);
+  };
+  TORCH_CHECK(rows16(d), "gemm: rows of a result with 32 or more columns must start at 16-byte boundaries");
   if (fl & GEMM_FLAG_BIAS) {
     TORCH_CHECK(bias.has_value() && bias->numel() == N && bias->scalar_type() == a.scalar_type() && bias->is_contiguous(),
                 "bias must be a contiguous [N] tensor of the input dtype");
@@ -117,11 +122,12 @@ Tensor gemm(const Tensor& a, const Tensor& b, int64_t a_mn, int64_t b_mn, const 
     TORCH_CHECK(aux.has_value() && aux->dim() == 2 && aux->size(0) == M && aux->size(1) == N && aux->stride(1) == 1, "bad aux");
     const auto want = (fl & GEMM_FLAG_RESIDUAL) ? d.scalar_type() : a.scalar_type();
     TORCH_CHECK(aux->scalar_type() == want, "aux dtype mismatch");
+    TORCH_CHECK(rows16(*aux), "gemm: rows of aux must start at 16-byte boundaries");
     ld_aux = static_cast<int>(aux->stride(0));
   }
   if (fl & GEMM_FLAG_SAVE_PREACT) {
     TORCH_CHECK(aux_out.has_value() && aux_out->dim() == 2 && aux_out->size(0) == M && aux_out->size(1) == N &&
-                    aux_out->stride(1) == 1 && aux_out->scalar_type() == a.scalar_type(), "bad aux_out");
+                    aux_out->stride(1) == 1 && aux_out->scalar_type() == a.scalar_type() && rows16(*aux_out), "bad aux_out");
     ld_aux_out = static_cast<int>(aux_out->stride(0));
   }
   auto& st = dev_state(a.get_device());

@@ -708,7 +708,9 @@ def bonus_step(r: Tensor, k: Tensor, v: Tensor, t: Tensor, w2: Tensor, w0: Tenso
 
 def linear_fp32(x: Tensor, weight: Tensor) -> Tensor:
     if gemm_ok(x, weight) and weight.dtype == x.dtype:
-        return gemm(x, weight, flags=FLAG_OUT_FP32)
+        n = weight.size(0)
+        out = torch.empty(x.size(0), -(-n // 4) * 4, dtype=torch.float32, device=x.device)[:, :n]   # rows at 16-byte boundaries
+        return gemm(x, weight, out=out, flags=FLAG_OUT_FP32)
     return torch.matmul(x.float(), weight.float().t())
 
 
@@ -831,7 +833,7 @@ MOE_FEW_PAIRS = 8   # (token, choice) pairs up to which the chosen experts' weig
 
 def moe_route(h: Tensor, w: Tensor, bias: Tensor, top: int):
     logits = None
-    if h.size(0) > SMALL_M_ROWS and gemm_ok(h, w) and h.size(1) % 8 == 0:
+    if h.size(0) > SMALL_M_ROWS and gemm_ok(h, w) and h.size(1) % 8 == 0 and (w.size(0) < 32 or w.size(0) % 4 == 0):
         logits = gemm(h, w, flags=FLAG_OUT_FP32)           # 16-bit operands, exact products, fp32 sums and output
     elif h.size(0) > 65535:                                # no tensor-core path for these sizes or types: 32-bit library product
         logits = torch.matmul(h.float(), w.float().t())

@@ -276,12 +276,19 @@ def test_grouped_decode(dtype, batch, heads, groups, dim, vdim, tmax, length):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_products_for_few_and_many_rows(dtype):
-    for rows, k, n in ((1, 64, 40), (3, 128, 96), (9, 64, 48), (20, 64, 48), (70, 64, 24), (200, 72, 13), (5, 30, 9)):
+    for rows, k, n in ((1, 64, 40), (3, 128, 96), (9, 64, 48), (20, 64, 48), (70, 64, 24), (200, 72, 13), (5, 30, 9), (200, 64, 45), (70, 32, 434), (3, 64, 33)):
         x, w = rnd(4, rows, k, dtype=dtype), rnd(4, n, k, dtype=dtype, scale=k ** -0.5)
         close(torch.stack(ops.stacked_linear(x, w)), torch.matmul(x.float(), w.float().transpose(1, 2)), dtype)
         y = ops.linear_fp32(x[0], w[0])
         assert y.dtype == torch.float32
         close(y, x[0].float() @ w[0].float().t(), torch.float32)
+
+
+def test_products_refuse_results_with_unaligned_rows():
+    x, w = rnd(80, 64, dtype=torch.bfloat16), rnd(45, 64, dtype=torch.bfloat16)
+    ext = ops.load_ext(required=True)
+    with pytest.raises(RuntimeError, match="16-byte"):
+        ext.gemm(x, w, 0, 0, None, None, None, None, 32, 1.0)          # 45 fp32 columns, rows without padding
 
 
 # ---------------------------------------------------------------------------------------------------- the whole model

@@ -162,7 +162,7 @@ def test_latent_prep_norms_and_appends():
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("rows,width,ff,experts,top", [(1, 64, 32, 4, 2), (5, 40, 24, 3, 3), (4, 192, 104, 9, 2), (17, 192, 104, 9, 2),
-                                                       (200, 128, 300, 5, 1), (300, 36, 20, 7, 3), (700, 512, 256, 16, 4)])
+                                                       (200, 128, 300, 5, 1), (300, 36, 20, 7, 3), (700, 512, 256, 16, 4), (300, 64, 24, 37, 3)])
 def test_moe(dtype, rows, width, ff, experts, top):
     h = rnd(rows, width, dtype=dtype)
     w, b = rnd(experts, width, dtype=dtype, scale=width ** -0.5), rnd(experts, dtype=dtype)

@@ -1,6 +1,7 @@
-"""Token mixers and feed-forwards that are not tied to one model family: latent attention with a sink, grouped-query attention
-with query / key norms and capped scores, gated linear recurrence (HGRN2), linear attention with constant decays, linear
-recurrence with a bonus (WKV), selective scan (Mamba), two mixers side by side; gated MLPs, mixture of experts.
+"""Token mixers and feed-forwards that are not tied to one model family: latent attention (with or without a sink and a rotated
+part), grouped-query attention with query / key norms, capped scores, windows and gates, gated linear recurrence (HGRN2),
+linear attention with constant decays, linear recurrence with a bonus (WKV), matrix memory (mLSTM), selective scan (Mamba), two
+mixers side by side; gated MLPs, mixtures of experts; residual streams with hyper-connections.
 
 They take their sizes and constants as arguments and work on token rows ``[batch * positions, width]``. A mixer or
 feed-forward can carry ``side`` projections: further linear maps of the same input (a block's residual gate, say) that
@@ -42,6 +43,9 @@ class FeedForwardOutput(NamedTuple):
     side: Dict[str, Tensor]
     slots: Optional[Tensor] = None         # where a (token, choice)'s row of ``y`` is; None: in order
     weights: Optional[Tensor] = None       # [rows, top] weights of those rows; None: ``y`` has one row per token
+    choice: Optional[Tensor] = None        # [rows, top] chosen router outputs, when some of them are no experts
+    shared: Optional[Tensor] = None        # [rows, width] of a shared expert, to be added times sigmoid(shared_gate)
+    shared_gate: Optional[Tensor] = None   # [rows, 1]
 
 
 def _inference(*ts: Tensor) -> bool:
@@ -53,73 +57,124 @@ def _last(keep: Optional[Tensor], s: int) -> Optional[Tensor]:
     return None if keep is None else keep[:, -s:]
 
 
-class LatentAttention(nn.Module):
-    """Attention over low-rank latents, without positions.
+class _Constants:
+    """Vectors that the configuration fixes, as fp32 tensors on whatever device they are asked for (not parameters: neither
+    saved nor converted to the model's storage type)."""
 
-    ``c = norm(W_dkv h)`` (``kv_rank``) is all that is cached; per head ``k = W_uk c`` (``dim``), ``v = W_uv c`` (``vdim``),
-    ``q = W_uq norm(W_dq h)`` (through ``q_rank``), scores ``(q . k) * scale``, causal. The softmax denominator also
-    holds ``exp(sink[head])``; head ``h``'s output is multiplied by ``sigmoid(W_g h)[head]`` before ``W_o``. With
+    def _constant(self, name: str, values: Sequence[float], device) -> Tensor:
+        table = self.__dict__.setdefault("_constant_tensors", {})
+        key = (name, str(device))
+        if key not in table:
+            table[key] = torch.tensor(list(values), dtype=torch.float32, device=device)
+        return table[key]
+
+
+class LatentAttention(nn.Module, _Constants):
+    """Attention over low-rank latents.
+
+    ``c = norm(W_dkv h)`` (``kv_rank``) is what is cached; per head ``k = W_uk c`` (``dim``), ``v = W_uv c`` (``vdim``), ``q = W_uq
+    norm(W_dq h)`` (through ``q_rank``), scores ``(q . k) * scale``, causal. With ``rot_dim`` a head's query has ``rot_dim`` further
+    dimensions and ``W_dkv h`` as many further rows, one key part for all heads (not normed, cached with ``c``); both are rotated
+    (halves, ``rot_base``) and their product joins the score. With ``sink`` the softmax denominator also holds ``exp(sink[head])``. The
+    output is multiplied by ``sigmoid(W_g h)`` before ``W_o``: one number per head, or (``gate="element"``) one per element. With
     ``shared_latents`` the module has no ``W_dkv`` and reads the latents of another layer (``kv_layer``).
     """
 
     oslo_fused = False
 
     def __init__(self, width: int, heads: int, dim: int, vdim: int, q_rank: int, kv_rank: int, scale: float, eps: float,
-                 shared_latents: bool = False, side: Optional[Dict[str, int]] = None) -> None:
+                 shared_latents: bool = False, side: Optional[Dict[str, int]] = None, rot_dim: int = 0, rot_base: float = 10000.0,
+                 sink: bool = True, gate: str = "head") -> None:
         super().__init__()
+        if gate not in ("head", "element"):
+            raise ValueError(f"output gate per {gate!r}")
         self.heads, self.dim, self.vdim, self.kv_rank, self.scale = heads, dim, vdim, kv_rank, float(scale)
+        self.rot_dim = rot_dim
+        self.frequencies = ops.reference.rotary_frequencies(rot_dim, rot_base)
         self.shared_latents = shared_latents
         self.side = dict(side or {})
-        parts = {"dq": q_rank, "g": heads, **self.side}
+        parts = {"dq": q_rank, "g": heads if gate == "head" else heads * vdim, **self.side}
         if not shared_latents:
-            parts["dkv"] = kv_rank
+            parts["dkv"] = kv_rank + rot_dim
         self.in_proj = PackedLinear(width, parts)
         self.q_norm = RMSNorm(q_rank, eps)
         self.kv_norm = None if shared_latents else RMSNorm(kv_rank, eps)
-        self.uq = Linear(q_rank, heads * dim, bias=False)
+        self.uq = Linear(q_rank, heads * (dim + rot_dim), bias=False)
         self.kv_up = PackedLinear(kv_rank, {"k": heads * dim, "v": heads * vdim})
-        self.sink = nn.Parameter(torch.zeros(heads))
+        self.sink = nn.Parameter(torch.zeros(heads)) if sink else None
         self.out_proj = Linear(heads * vdim, width, bias=False)
 
     def forward(self, h: Tensor, batch: int, layer_id: int, kv_layer: int, cache: Optional[StaticKVCache],
-                latent: Optional[Tensor], keep: Optional[Tensor], output_attentions: bool = False) -> MixerOutput:
+                latent: Optional[Tensor], keep: Optional[Tensor], output_attentions: bool = False,
+                positions: Optional[Tensor] = None) -> MixerOutput:
         """``h`` ``[batch * S, width]``; ``latent``: the latents of ``kv_layer`` when there is no cache; ``keep``
-        ``[batch, past + S]`` marks real tokens (0 = padding)."""
+        ``[batch, past + S]`` marks real tokens (0 = padding); ``positions`` ``[batch, S]`` where something is rotated."""
         from ..ops.cuda_ops import LATENT_MAX_RANK
         p = self.in_proj(h)
         side = {n: p[n] for n in self.side}
         s = h.size(0) // batch
-        if (cache is not None and s == 1 and not output_attentions and self.oslo_fused and _inference(h, self.sink)
-                and ops.use_kernels(h) and self.kv_rank <= LATENT_MAX_RANK):
-            return MixerOutput(self._decode(p, batch, kv_layer, cache, keep), side)
-        q = self.uq(self.q_norm(p["dq"])).view(batch, s, self.heads, self.dim)
-        if not self.shared_latents:
-            latent = self.kv_norm(p["dkv"]).view(batch, s, self.kv_rank)
-            if cache is not None:
-                latent = cache.append_latent(layer_id, latent)
-        elif cache is not None:
-            latent = cache.latent[kv_layer][:, :cache.length + s]
+        kernels = self.oslo_fused and not output_attentions and _inference(h, self.out_proj.weight) and ops.use_kernels(h)
+        if cache is not None and s == 1 and kernels and self.kv_rank <= LATENT_MAX_RANK:
+            return MixerOutput(self._decode(p, batch, kv_layer, cache, keep, positions), side)
+        if self.rot_dim and kernels and not self.shared_latents:
+            q, latent, c = self._prompt(p, batch, s, layer_id, cache, positions)
+        else:
+            q = self.uq(self.q_norm(p["dq"])).view(batch, s, self.heads, self.dim + self.rot_dim)
+            if self.rot_dim:
+                freq = self._constant("freq", self.frequencies, h.device)
+                turned = ops.reference.rotate_halves(q[..., self.dim:], positions, freq)
+                q = torch.cat([q[..., :self.dim], turned], dim=-1)
+            if not self.shared_latents:
+                latent = self.kv_norm(p["dkv"][:, :self.kv_rank]).view(batch, s, self.kv_rank)
+                if self.rot_dim:
+                    shared = p["dkv"][:, self.kv_rank:].reshape(batch, s, 1, self.rot_dim)
+                    latent = torch.cat([latent, ops.reference.rotate_halves(shared, positions, freq)[:, :, 0]], dim=-1)
+                if cache is not None:
+                    latent = cache.append_latent(layer_id, latent)
+            elif cache is not None:
+                latent = cache.latent[kv_layer][:, :cache.length + s]
+            c = latent[..., :self.kv_rank].reshape(-1, self.kv_rank)
         t = latent.size(1)
-        kv = self.kv_up(latent.reshape(batch * t, self.kv_rank))
+        kv = self.kv_up(c)
         k = kv["k"].view(batch, t, self.heads, self.dim)
         v = kv["v"].view(batch, t, self.heads, self.vdim)
+        rotated = (q[..., self.dim:], latent[..., self.kv_rank:]) if self.rot_dim else (None, None)
+        args = (q[..., :self.dim], k, v, keep, self.sink, p["g"], self.scale, 0.0, 0, 0, None, *rotated)
         probs = None
         if output_attentions or not self.oslo_fused:
-            o, probs = ops.reference.sink_attention(q, k, v, keep, self.sink, p["g"], self.scale)
+            o, probs = ops.reference.sink_attention(*args)
         else:
-            o = ops.sink_attention(q, k, v, keep, self.sink, p["g"], self.scale)
+            o = ops.sink_attention(*args)
         return MixerOutput(self.out_proj(o), side, latent, probs if output_attentions else None)
 
-    def _decode(self, p: Dict[str, Tensor], batch: int, kv_layer: int, cache: StaticKVCache, keep: Optional[Tensor]) -> Tensor:
-        """One token per row: norms + cache append, query projection, attention over the latents, output projection."""
+    def _prompt(self, p: Dict[str, Tensor], batch: int, s: int, layer_id: int, cache: Optional[StaticKVCache], positions: Tensor):
+        """Norms, rotations and cache append of a prompt: queries ``[batch, S, heads, *]``, what the cache holds now, and the latents of
+        that as contiguous rows."""
         from ..ops import cuda_ops
         dq = p["dq"]
-        store = cache.latent_storage(kv_layer, batch, self.kv_rank, dq.dtype, dq.device, 1)
+        freq = self._constant("freq", self.frequencies, dq.device)
+        holder = cache if cache is not None else StaticKVCache(s)
+        store = holder.latent_storage(layer_id, batch, self.kv_rank + self.rot_dim, dq.dtype, dq.device, s)
+        cq, c = cuda_ops.latent_prep(dq, self.q_norm.weight, p["dkv"], self.kv_norm.weight, store, holder.lengths_dev, self.q_norm.eps,
+                                     positions, freq, rows=True)
+        q = cuda_ops.rotate_halves_(self.uq(cq).view(batch, s, self.heads, self.dim + self.rot_dim), positions, freq)
+        latent = store[:, :holder.length + s]
+        if holder.length:
+            c = latent[..., :self.kv_rank].reshape(-1, self.kv_rank)
+        return q, latent, c
+
+    def _decode(self, p: Dict[str, Tensor], batch: int, kv_layer: int, cache: StaticKVCache, keep: Optional[Tensor],
+                positions: Optional[Tensor]) -> Tensor:
+        """One token per row: norms + rotation + cache append, query projection, attention over the latents, output projection."""
+        from ..ops import cuda_ops
+        dq = p["dq"]
+        store = cache.latent_storage(kv_layer, batch, self.kv_rank + self.rot_dim, dq.dtype, dq.device, 1)
         own = not self.shared_latents
-        cq = cuda_ops.latent_prep(dq, self.q_norm.weight, p["dkv"] if own else None, self.kv_norm.weight if own else None,
-                                  store if own else None, cache.lengths_dev, self.q_norm.eps)
+        freq = self._constant("freq", self.frequencies, dq.device) if self.rot_dim else None
+        cq, _ = cuda_ops.latent_prep(dq, self.q_norm.weight, p["dkv"] if own else None, self.kv_norm.weight if own else None,
+                                     store if own else None, cache.lengths_dev, self.q_norm.eps, positions, freq)
         o = cuda_ops.latent_decode(self.uq(cq), self.kv_up.part("k"), self.kv_up.part("v"), store, cache.lengths_next, keep,
-                                   self.sink, p["g"], self.scale, self.heads)
+                                   self.sink, p["g"], self.scale, self.heads, positions, freq)
         return self.out_proj(o)
 
 
@@ -162,88 +217,91 @@ def _plain_recurrence(q, f, v, f_bias, lower, norm_w, eps, batch, heads, keep, s
     return ops.reference.rms_norm(o, norm_w, eps).reshape(-1, heads * vdim)
 
 
-class _Constants:
-    """Vectors that the configuration fixes, as fp32 tensors on whatever device they are asked for (not parameters: neither
-    saved nor converted to the model's storage type)."""
-
-    def _constant(self, name: str, values: Sequence[float], device) -> Tensor:
-        table = self.__dict__.setdefault("_constant_tensors", {})
-        key = (name, str(device))
-        if key not in table:
-            table[key] = torch.tensor(list(values), dtype=torch.float32, device=device)
-        return table[key]
-
-
 class GroupedQueryAttention(nn.Module, _Constants):
     """Causal softmax attention with ``heads`` query heads over ``kv_heads`` key / value heads.
 
-    Queries and keys are RMS-normed per head (weights ``[dim]``, shared by the heads), then the first ``rot_dims`` dims are rotated
-    (interleaved pairs, ``rot_base``); scores ``(q . k) * scale`` pass through ``softcap * tanh(score / softcap)`` (0: they do
-    not); the softmax denominator holds an additional 1 (a sink with score 0). Keys (after norm and rotation) and values are
-    cached. ``in_proj=False``: the projections come from the caller's packed GEMM (``parts``)."""
+    Queries and keys are RMS-normed per head (weights ``[dim]``, shared by the heads; ``norm_weights=False``: without weights), then
+    the first ``rot_dims`` dims are rotated (interleaved pairs, ``rot_base``); scores ``(q . k) * scale`` pass through ``softcap *
+    tanh(score / softcap)`` (0: they do not). With ``sink`` the softmax denominator holds an additional 1 (a sink with score 0). With a
+    ``window`` > 0 a position reads the last ``window`` positions and the first ``keep_first`` of the sequence. ``value_is_key``: values
+    are the projected keys, before norm and rotation. ``gate``: head ``h``'s output is multiplied by ``sigmoid(W_g x)[h]``. Keys (after
+    norm and rotation) and values are cached. ``in_proj=False``: the projections come from the caller's packed GEMM (``parts``)."""
 
     oslo_fused = False
 
     def __init__(self, width: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, eps: float, rot_dims: int = 0,
-                 rot_base: float = 10000.0, softcap: float = 0.0, in_proj: bool = True) -> None:
+                 rot_base: float = 10000.0, softcap: float = 0.0, in_proj: bool = True, norm_weights: bool = True, sink: bool = True,
+                 window: int = 0, keep_first: int = 0, value_is_key: bool = False, gate: bool = False) -> None:
         super().__init__()
         if heads % kv_heads:
             raise ValueError(f"{heads} query heads do not divide into {kv_heads} groups")
-        self.heads, self.kv_heads, self.dim, self.vdim = heads, kv_heads, dim, vdim
+        if value_is_key and vdim != dim:
+            raise ValueError(f"values are the keys, but have size {vdim} and not {dim}")
+        self.heads, self.kv_heads, self.dim, self.vdim, self.eps = heads, kv_heads, dim, vdim, float(eps)
         self.scale, self.softcap = float(scale), float(softcap)
+        self.sink, self.window, self.keep_first = bool(sink), int(window), int(keep_first)
         self.frequencies = ops.reference.rotary_frequencies(rot_dims, rot_base)
-        self.parts = {"q": heads * dim, "k": kv_heads * dim, "v": kv_heads * vdim}
+        self.parts = {"q": heads * dim, "k": kv_heads * dim}
+        if not value_is_key:
+            self.parts["v"] = kv_heads * vdim
+        if gate:
+            self.parts["g"] = heads
         self.in_proj = PackedLinear(width, self.parts) if in_proj else None
-        self.q_norm = RMSNorm(dim, eps)
-        self.k_norm = RMSNorm(dim, eps)
+        self.q_norm = RMSNorm(dim, eps) if norm_weights else None
+        self.k_norm = RMSNorm(dim, eps) if norm_weights else None
         self.out_proj = Linear(heads * vdim, width, bias=False)
 
     def forward(self, h: Tensor, batch: int, layer_id: int, cache: Optional[StaticKVCache], keep: Optional[Tensor],
-                positions: Tensor, output_attentions: bool = False) -> MixerOutput:
-        return self.mix(self.in_proj(h), batch, layer_id, cache, keep, positions, output_attentions)
+                positions: Tensor, output_attentions: bool = False, lead: Optional[Tensor] = None) -> MixerOutput:
+        return self.mix(self.in_proj(h), batch, layer_id, cache, keep, positions, output_attentions, lead)
 
     def mix(self, p: Dict[str, Tensor], batch: int, layer_id: int, cache: Optional[StaticKVCache], keep: Optional[Tensor],
-            positions: Tensor, output_attentions: bool = False) -> MixerOutput:
-        """``keep`` ``[batch, past + S]`` marks real tokens, ``positions`` ``[batch, S]``."""
+            positions: Tensor, output_attentions: bool = False, lead: Optional[Tensor] = None) -> MixerOutput:
+        """``keep`` ``[batch, past + S]`` marks real tokens, ``positions`` ``[batch, S]``; ``lead`` ``[batch]`` int32: padding ahead of a
+        sequence's first token (``None``: none anywhere)."""
         rows = p["q"].size(0)
         s = rows // batch
         freq = self._constant("freq", self.frequencies, p["q"].device)
-        sink = self._sink(p["q"])
-        if (self.oslo_fused and not output_attentions and _inference(p["q"], self.q_norm.weight) and ops.use_kernels(p["q"])):
-            o = self._kernels(p, batch, s, layer_id, cache, keep, positions, freq, sink)
+        sink, gate, values = self._sink(p["q"]), p.get("g"), p.get("v", p["k"])
+        wq, wk = (None, None) if self.q_norm is None else (self.q_norm.weight, self.k_norm.weight)
+        mask = (self.window, self.keep_first, lead)
+        if (self.oslo_fused and not output_attentions and _inference(p["q"], self.out_proj.weight) and ops.use_kernels(p["q"])):
+            o = self._kernels(p, values, batch, s, layer_id, cache, keep, positions, freq, sink, gate, mask)
             return MixerOutput(self.out_proj(o), {})
-        q = ops.reference.norm_rotate(p["q"].reshape(batch, s, self.heads, self.dim), self.q_norm.weight, self.q_norm.eps, positions, freq)
-        k = ops.reference.norm_rotate(p["k"].reshape(batch, s, self.kv_heads, self.dim), self.k_norm.weight, self.k_norm.eps, positions, freq)
-        v = p["v"].reshape(batch, s, self.kv_heads, self.vdim)
+        q = ops.reference.norm_rotate(p["q"].reshape(batch, s, self.heads, self.dim), wq, self.eps, positions, freq)
+        k = ops.reference.norm_rotate(p["k"].reshape(batch, s, self.kv_heads, self.dim), wk, self.eps, positions, freq)
+        v = values.reshape(batch, s, self.kv_heads, self.vdim)
         if cache is not None:
             k, v, end = cache.append(layer_id, k.transpose(1, 2), v.transpose(1, 2))
             if s == 1 and not output_attentions:
-                o = ops.reference.grouped_decode(q[:, 0], k, v, cache.lengths_next, keep, sink, self.scale, self.softcap)
+                o = ops.reference.grouped_decode(q[:, 0], k, v, cache.lengths_next, keep, sink, self.scale, self.softcap, gate, *mask)
                 return MixerOutput(self.out_proj(o), {})
             k, v = k[:, :, :end].transpose(1, 2), v[:, :, :end].transpose(1, 2)
-        o, probs = ops.reference.sink_attention(q, k, v, keep, sink, None, self.scale, self.softcap)
+        o, probs = ops.reference.sink_attention(q, k, v, keep, sink, gate, self.scale, self.softcap, *mask)
         return MixerOutput(self.out_proj(o), {}, probs=probs if output_attentions else None)
 
-    def _sink(self, like: Tensor) -> Tensor:
+    def _sink(self, like: Tensor) -> Optional[Tensor]:
+        if not self.sink:
+            return None
         table = self.__dict__.setdefault("_constant_tensors", {})
         key = ("sink", str(like.device), like.dtype)
         if key not in table:
             table[key] = torch.zeros(self.heads, dtype=like.dtype, device=like.device)
         return table[key]
 
-    def _kernels(self, p, batch, s, layer_id, cache, keep, positions, freq, sink) -> Tensor:
+    def _kernels(self, p, values, batch, s, layer_id, cache, keep, positions, freq, sink, gate, mask) -> Tensor:
         """Norms, rotation and cache append in one launch, then the prompt or the decode kernel on the cached keys."""
         from ..ops import cuda_ops
         q = p["q"]
         holder = cache if cache is not None else StaticKVCache(s)
         ks, vs = holder.kv_storage(layer_id, batch, self.kv_heads, self.dim, self.vdim, q.dtype, q.device, s)
-        q = cuda_ops.qkv_prep(q, p["k"], p["v"], self.q_norm.weight, self.k_norm.weight, self.q_norm.eps, positions, freq, ks, vs,
-                              holder.lengths_dev)
+        wq, wk = (None, None) if self.q_norm is None else (self.q_norm.weight, self.k_norm.weight)
+        q = cuda_ops.qkv_prep(q, p["k"], values, wq, wk, self.eps, positions, freq, ks, vs, holder.lengths_dev)
         if s == 1 and cache is not None:
-            return cuda_ops.grouped_decode(q[:, 0], ks, vs, holder.lengths_next, keep, sink, self.scale, self.softcap)
+            return cuda_ops.grouped_decode(q[:, 0], ks, vs, holder.lengths_next, keep, sink, self.scale, self.softcap, gate, *mask)
         end = holder.length + s
-        return cuda_ops.sink_attention(q, ks[:, :, :end].transpose(1, 2), vs[:, :, :end].transpose(1, 2), keep, sink, None, self.scale,
-                                       self.softcap)
+        return cuda_ops.sink_attention(q, ks[:, :, :end].transpose(1, 2), vs[:, :, :end].transpose(1, 2), keep, sink, gate, self.scale,
+                                       self.softcap, *mask)
 
 
 class DecayedLinearAttention(nn.Module, _Constants):
@@ -349,6 +407,42 @@ class BonusRecurrence(nn.Module):
         return MixerOutput(self.out_proj(o), {})
 
 
+class MatrixMemory(nn.Module):
+    """mLSTM: per head a matrix memory ``S`` and a normaliser ``n`` with one input gate and one forget gate per token in the exponent,
+    ``cap`` bounding both, and a running maximum that keeps them in range (``reference.matrix_memory``). A head's ``S^T q`` is divided by
+    ``max(|n . q|, exp(-m)) + 1e-6`` and by its root mean square, then times a weight, times ``sigmoid(W_g h)``, and projected."""
+
+    oslo_fused = False
+
+    def __init__(self, width: int, heads: int, dim: int, vdim: int, cap: float, eps: float) -> None:
+        super().__init__()
+        self.heads, self.dim, self.vdim, self.cap, self.eps = heads, dim, vdim, float(cap), float(eps)
+        self.in_proj = PackedLinear(width, {"q": heads * dim, "k": heads * dim, "v": heads * vdim, "g": heads * vdim})
+        self.gates = Linear(width, 2 * heads)              # input gates, then forget gates; applied with 32-bit results
+        self.o_norm = nn.Parameter(torch.ones(heads * vdim))
+        self.out_proj = Linear(heads * vdim, width, bias=False)
+
+    def forward(self, h: Tensor, batch: int, layer_id: int, cache: Optional[StaticKVCache], keep: Optional[Tensor]) -> MixerOutput:
+        s = h.size(0) // batch
+        keep = _last(keep, s)
+        state = top = None
+        if cache is not None:
+            width = ops.reference.memory_state_width(self.vdim)
+            state = cache.recurrent_state(layer_id, (batch, self.heads, self.dim, width), h.device)
+            top = cache.recurrent_state(layer_id, (batch, self.heads), h.device, "max")
+        p = self.in_proj(h)
+        if s == 1 and state is not None and self.oslo_fused and _inference(h, self.o_norm) and ops.use_kernels(h):
+            from ..ops import cuda_ops
+            o = cuda_ops.memory_step(p["q"], p["k"], p["v"], h, self.gates.weight, self.gates.bias, self.cap, p["g"], self.o_norm, keep,
+                                     state, top, self.eps, self.heads)
+            return MixerOutput(self.out_proj(o), {})
+        z = ops.linear_fp32(h, self.gates.weight, fused=self.oslo_fused)
+        o, n, m = ops.matrix_memory(p["q"], p["k"], p["v"], z, self.gates.bias, self.cap, keep, state, top, batch, self.heads,
+                                    fused=self.oslo_fused)
+        o = ops.gated_rms_norm(o, self.o_norm, p["g"], self.eps, self.vdim, "sigmoid", (n, m), fused=self.oslo_fused)
+        return MixerOutput(self.out_proj(o), {})
+
+
 class SelectiveScan(nn.Module):
     """Mamba: ``x`` and ``z`` from one projection; ``x`` through a causal convolution per channel and ``silu``; steps ``dt`` and the
     token's ``B``, ``C`` from ``x``; ``S <- exp(dt A) S + dt x B`` per channel and state (fp32), ``y = S C + D x``, times ``silu(z)``."""
@@ -413,27 +507,62 @@ class GatedMLP(nn.Module):
 
 
 class MixtureOfExperts(nn.Module):
-    """``experts`` small feed-forwards ``W_down relu(W_up h)^2``; a token's router logits ``W_r h + b`` (fp32) choose ``top`` of
-    them, weighted by the softmax over the chosen logits only. No capacity limit: every choice is computed. The result keeps
-    one row per (token, choice); whoever adds it to the residual stream sums the rows."""
+    """``experts`` small feed-forwards, of which a token uses ``top``. No capacity limit: every choice is computed. The result keeps one
+    row per (token, choice); whoever adds it to the residual stream sums the rows.
+
+    ``unit="relu2"``: ``W_down relu(W_up h)^2``; ``"silu"``: ``W_down (silu(W_gate h) * W_up h)``. The router's logits are fp32: ``W_r h + b``
+    choose, weighted by the softmax over the chosen ones; ``scored``: scores are the softmax of ``W_r h`` over all outputs, ``score +
+    correction`` choose, the weights are the chosen scores divided by their sum. ``identity`` further router outputs stand for the
+    input itself. ``shared``: size of an expert that every token uses, weighted by a sigmoid projection of its own."""
 
     oslo_fused = False
 
-    def __init__(self, width: int, ff: int, experts: int, top: int, side: Optional[Dict[str, int]] = None) -> None:
+    def __init__(self, width: int, ff: int, experts: int, top: int, side: Optional[Dict[str, int]] = None, unit: str = "relu2",
+                 scored: bool = False, identity: int = 0, shared: Optional[int] = None) -> None:
         super().__init__()
-        self.experts, self.top = experts, top
+        if unit not in ("relu2", "silu"):
+            raise ValueError(f"unknown expert unit {unit!r}")
+        self.experts, self.top, self.unit, self.scored, self.identity = experts, top, unit, scored, identity
         self.side = dict(side or {})
         self.in_proj = PackedLinear(width, self.side) if self.side else None
-        self.router = Linear(width, experts)
-        self.up = nn.Parameter(torch.empty(experts, ff, width).normal_(std=0.02))
+        outputs = experts + identity
+        self.router = Linear(width, outputs, bias=not scored)
+        self.correction = nn.Parameter(torch.zeros(outputs)) if scored else None
+        self.up = nn.Parameter(torch.empty(experts, ff * (2 if unit == "silu" else 1), width).normal_(std=0.02))
         self.down = nn.Parameter(torch.empty(experts, width, ff).normal_(std=0.02))
+        self.shared = GatedMLP(width, shared, side={"sg": 1}) if shared is not None else None
+
+    @staticmethod
+    def interleave(gate: Tensor, up: Tensor) -> Tensor:
+        """``up`` of a ``"silu"`` expert from its two matrices ``[ff, width]``: rows in turns, so that one tile holds both factors."""
+        return torch.stack([gate, up], dim=1).reshape(2 * gate.size(0), gate.size(1))
 
     def forward(self, h: Tensor) -> FeedForwardOutput:
         side = self.in_proj(h) if self.in_proj is not None else {}
-        if self.oslo_fused:
-            idx, weights = ops.moe_route(h, self.router.weight, self.router.bias, self.top)
-            y, slots = ops.moe_experts(h, idx, self.up, self.down)
-        else:
-            idx, weights = ops.reference.moe_route(h, self.router.weight, self.router.bias, self.top)
-            y, slots = ops.reference.moe_experts(h, idx, self.up, self.down), None
-        return FeedForwardOutput(y, side, slots, weights)
+        bias = self.correction if self.scored else self.router.bias
+        idx, weights = ops.moe_route(h, self.router.weight, bias, self.top, self.scored, fused=self.oslo_fused)
+        y, slots = ops.moe_experts(h, idx, self.up, self.down, self.unit, fused=self.oslo_fused)
+        shared, gate = None, None
+        if self.shared is not None:
+            out = self.shared(h)
+            shared, gate = out.y, out.side["sg"]
+        return FeedForwardOutput(y, side, slots, weights, idx if self.identity else None, shared, gate)
+
+
+class HyperConnections(nn.Module):
+    """What ties one sublayer to ``streams`` residual streams: it reads ``sum_s w_in[s] x_s``; afterwards ``x_t <- sum_s mix[s, t] x_s +
+    w_out[t] y`` (``reference.hyper_join``)."""
+
+    oslo_fused = False
+
+    def __init__(self, streams: int) -> None:
+        super().__init__()
+        self.w_in = nn.Parameter(torch.full((streams,), 1.0 / streams))
+        self.w_out = nn.Parameter(torch.ones(streams))
+        self.mix = nn.Parameter(torch.eye(streams))
+
+    def forward(self, x: Tensor, result: Optional[ops.reference.SublayerResult], w_in: Optional[Tensor], norm: RMSNorm,
+                scale: float = 1.0) -> Tuple[Tensor, Tensor]:
+        """``x`` ``[rows, streams, width]`` with the sublayer's ``result``, and the input of the next sublayer, which reads with ``w_in``
+        (``None``: the sum of the streams) through ``norm`` (weights around zero)."""
+        return ops.hyper_join(x, result, self.w_out, self.mix, w_in, norm.weight, norm.eps, scale, fused=self.oslo_fused)

@@ -11,6 +11,7 @@ from typing import Any, Dict, NamedTuple, Type
 
 from ..modeling_utils import CONFIG_NAME, PretrainedConfig, PreTrainedModel, _resolve_hub_file
 from .begovik import BegovikConfig, BegovikForCausalLM
+from .dekutar import DekutarConfig, DekutarForCausalLM
 from .gpt2 import GPT2Config, GPT2LMHeadModel
 from .gpt_neo import GPTNeoConfig, GPTNeoForCausalLM
 from .gptj import GPTJConfig, GPTJForCausalLM
@@ -28,6 +29,7 @@ MODELS: Dict[str, ModelEntry] = {
     "gptj": ModelEntry(GPTJConfig, GPTJForCausalLM),
     "moronex": ModelEntry(MoronexConfig, MoronexForCausalLM),
     "begovik": ModelEntry(BegovikConfig, BegovikForCausalLM),
+    "dekutar": ModelEntry(DekutarConfig, DekutarForCausalLM),
 }
 
 

@@ -195,37 +195,51 @@ def gated_recurrence(q: Tensor, f: Tensor, v: Tensor, f_bias: Tensor, lower: Ten
     return ref.rms_norm(o, norm_w, eps).reshape(-1, heads * vdim)
 
 
-def sink_attention(q: Tensor, k: Tensor, v: Tensor, keep: Optional[Tensor], sink: Tensor, gate: Optional[Tensor], scale: float,
-                   softcap: float = 0.0) -> Tensor:
+def sink_attention(q: Tensor, k: Tensor, v: Tensor, keep: Optional[Tensor], sink: Optional[Tensor], gate: Optional[Tensor],
+                   scale: float, softcap: float = 0.0, window: int = 0, keep_first: int = 0, lead: Optional[Tensor] = None,
+                   q_rot: Optional[Tensor] = None, k_rot: Optional[Tensor] = None) -> Tensor:
     """``reference.sink_attention`` without the weights."""
-    if _kn(q, k, v, sink, gate):
+    if _kn(q, k, v, sink, gate, q_rot, k_rot):
         from . import cuda_ops
-        return cuda_ops.sink_attention(q, k, v, keep, sink, gate, scale, softcap)
-    return ref.sink_attention(q, k, v, keep, sink, gate, scale, softcap)[0]
+        return cuda_ops.sink_attention(q, k, v, keep, sink, gate, scale, softcap, window, keep_first, lead, q_rot, k_rot)
+    return ref.sink_attention(q, k, v, keep, sink, gate, scale, softcap, window, keep_first, lead, q_rot, k_rot)[0]
 
 
-def latent_decode(q: Tensor, w_uk: Tensor, w_uv: Tensor, cache: Tensor, lengths: Tensor, keep: Optional[Tensor], sink: Tensor,
-                  gate: Tensor, scale: float, heads: int) -> Tensor:
+def latent_decode(q: Tensor, w_uk: Tensor, w_uv: Tensor, cache: Tensor, lengths: Tensor, keep: Optional[Tensor],
+                  sink: Optional[Tensor], gate: Tensor, scale: float, heads: int, positions: Optional[Tensor] = None,
+                  freq: Optional[Tensor] = None) -> Tensor:
     if _kn(q, w_uk, w_uv, cache, sink, gate):
         from . import cuda_ops
-        return cuda_ops.latent_decode(q, w_uk, w_uv, cache, lengths, keep, sink, gate, scale, heads)
-    return ref.latent_decode(q, w_uk, w_uv, cache, lengths, keep, sink, gate, scale, heads)
+        return cuda_ops.latent_decode(q, w_uk, w_uv, cache, lengths, keep, sink, gate, scale, heads, positions, freq)
+    return ref.latent_decode(q, w_uk, w_uv, cache, lengths, keep, sink, gate, scale, heads, positions, freq)
 
 
-def moe_route(h: Tensor, w: Tensor, bias: Tensor, top: int) -> Tuple[Tensor, Tensor]:
-    if _kn(h, w, bias):
+def moe_route(h: Tensor, w: Tensor, bias: Tensor, top: int, scored: bool = False, fused: bool = True) -> Tuple[Tensor, Tensor]:
+    if fused and _kn(h, w, bias):
         from . import cuda_ops
-        return cuda_ops.moe_route(h, w, bias, top)
-    return ref.moe_route(h, w, bias, top)
+        return cuda_ops.moe_route(h, w, bias, top, scored)
+    return ref.moe_route(h, w, bias, top, scored)
 
 
-def moe_experts(h: Tensor, idx: Tensor, up: Tensor, down: Tensor) -> Tuple[Tensor, Optional[Tensor]]:
-    """``W_down relu(W_up h)^2`` of the chosen experts, one row per (token, choice), and where those rows are
-    (``None``: row ``token * top + choice``); ``residual_join`` adds them up."""
-    if _kn(h, up, down):
+def moe_experts(h: Tensor, idx: Tensor, up: Tensor, down: Tensor, unit: str = "relu2",
+                fused: bool = True) -> Tuple[Tensor, Optional[Tensor]]:
+    """The chosen experts' results (``reference.moe_experts``), one row per (token, choice), and where those rows are (``None``: row
+    ``token * top + choice``); the step that joins the residual stream adds them up. Rows of choices that are no expert hold anything."""
+    if fused and _kn(h, up, down):
         from . import cuda_ops
-        return cuda_ops.moe_experts(h, idx, up, down)
-    return ref.moe_experts(h, idx, up, down), None
+        return cuda_ops.moe_experts(h, idx, up, down, unit)
+    return ref.moe_experts(h, idx, up, down, unit), None
+
+
+def hyper_join(x: Tensor, result: Optional[ref.SublayerResult], w_out: Optional[Tensor], mix: Optional[Tensor],
+               w_in: Optional[Tensor], w_norm: Tensor, eps: float, scale: float = 1.0, fused: bool = True) -> Tuple[Tensor, Tensor]:
+    """Residual streams take a sublayer's result and the next sublayer's input is read from them: one pass over the rows. See
+    ``reference.hyper_join``."""
+    mine = () if result is None else (result.y, result.weights, result.h, result.shared, result.shared_gate)
+    if fused and _kn(x, w_out, mix, w_in, w_norm, *mine):
+        from . import cuda_ops
+        return cuda_ops.hyper_join(x, result, w_out, mix, w_in, w_norm, eps, scale)
+    return ref.hyper_join(x, result, w_out, mix, w_in, w_norm, eps, scale)
 
 
 def linear_fp32(x: Tensor, weight: Tensor, fused: bool = True) -> Tensor:
@@ -260,11 +274,12 @@ def clamped_glu(gate: Tensor, up: Tensor, limit: float, alpha: float, fused: boo
     return ref.clamped_glu(gate, up, limit, alpha)
 
 
-def gated_rms_norm(o: Tensor, w: Tensor, gate: Tensor, eps: float, group: int, act: str, fused: bool = True) -> Tensor:
+def gated_rms_norm(o: Tensor, w: Tensor, gate: Tensor, eps: float, group: int, act: str,
+                   normalizer: Optional[Tuple[Tensor, Tensor]] = None, fused: bool = True) -> Tensor:
     if fused and _kn(o, w, gate):
         from . import cuda_ops
-        return cuda_ops.gated_rms_norm(o, w, gate, eps, group, act)
-    return ref.gated_rms_norm(o, w, gate, eps, group, act)
+        return cuda_ops.gated_rms_norm(o, w, gate, eps, group, act, normalizer)
+    return ref.gated_rms_norm(o, w, gate, eps, group, act, normalizer)
 
 
 # ``state`` / ``prev`` of the functions below (fp32) carry a sequence on: read, and updated in place.
@@ -290,6 +305,20 @@ def bonus_recurrence(r: Tensor, k: Tensor, v: Tensor, z: Tensor, w0: Tensor, u: 
     if state is not None:
         state.copy_(final.detach())
     return o.reshape(r.size(0), -1)
+
+
+def matrix_memory(q: Tensor, k: Tensor, v: Tensor, z: Tensor, bias: Tensor, cap: float, keep: Optional[Tensor],
+                  state: Optional[Tensor], top: Optional[Tensor], batch: int, heads: int,
+                  fused: bool = True) -> Tuple[Tensor, Tensor, Tensor]:
+    """``reference.matrix_memory``: ``S^T q``, ``n . q`` and the running maximum of every token (fp32)."""
+    if fused and _kn(q, k, v, z, bias):
+        from . import cuda_ops
+        return cuda_ops.matrix_memory(q, k, v, z, bias, cap, keep, state, top, batch, heads)
+    o, nq, m, final, last = ref.matrix_memory(q, k, v, z, bias, cap, keep, state, top, batch, heads)
+    if state is not None:
+        state.copy_(final.detach())
+        top.copy_(last.detach())
+    return o, nq, m
 
 
 def token_shift(h: Tensor, mu: Tensor, batch: int, keep: Optional[Tensor], prev: Optional[Tensor], fused: bool = True) -> Tensor:

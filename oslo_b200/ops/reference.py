@@ -9,7 +9,7 @@ includes/fused_softmax.h:111-229; n-gram ban: fused_ngram_repeat_block.cu:18-49)
 from __future__ import annotations
 
 import math
-from typing import Optional, Tuple
+from typing import NamedTuple, Optional, Tuple
 
 import torch
 import torch.nn.functional as F
@@ -232,70 +232,180 @@ def recurrence(q: Tensor, f: Tensor, v: Tensor, f_bias: Tensor, lower: Tensor, k
     return torch.stack(out, dim=1), s
 
 
-def sink_attention(q: Tensor, k: Tensor, v: Tensor, keep: Optional[Tensor], sink: Tensor, gate: Optional[Tensor], scale: float,
-                   softcap: float = 0.0):
-    """Causal softmax attention whose denominator also holds ``exp(sink[head])``; with ``gate`` ``[B * Sq, H]`` head ``h``'s
-    output is multiplied by ``sigmoid(gate[:, h])``, with ``softcap`` scores become ``softcap * tanh(score / softcap)``. ``q``
-    ``[B, Sq, H, D]`` are the last positions of ``k``/``v`` ``[B, Sk, G, *]``; query head ``h`` reads key head ``h // (H / G)``;
-    ``keep`` ``[B, Sk]``. Returns ``[B * Sq, H * Dv]`` and the weights ``[B, H, Sq, Sk]``."""
+def visible_keys(qpos: Tensor, kpos: Tensor, window: int, keep_first: int, lead: Optional[Tensor]) -> Tensor:
+    """Which of the columns ``kpos`` a query at column ``qpos`` may read (both broadcast; ``lead`` has the shape of a batch of them):
+    those up to its own, with a ``window`` > 0 only the last ``window`` of them and the sequence's first ``keep_first``, whose
+    columns start behind ``lead`` columns of padding."""
+    vis = kpos <= qpos
+    if window > 0:
+        near = qpos - kpos < window
+        if keep_first > 0:
+            near = near | ((kpos if lead is None else kpos - lead) < keep_first)
+        vis = vis & near
+    return vis
+
+
+def output_gate(o: Tensor, gate: Optional[Tensor]) -> Tensor:
+    """``o`` ``[rows, heads, vdim]`` times the sigmoid of ``gate`` ``[rows, heads]`` (one factor per head) or ``[rows, heads * vdim]``."""
+    if gate is None:
+        return o
+    g = torch.sigmoid(gate.to(torch.float32))
+    return o * (g.unsqueeze(-1) if g.size(-1) == o.size(1) else g.view(o.shape))
+
+
+def sink_attention(q: Tensor, k: Tensor, v: Tensor, keep: Optional[Tensor], sink: Optional[Tensor], gate: Optional[Tensor],
+                   scale: float, softcap: float = 0.0, window: int = 0, keep_first: int = 0, lead: Optional[Tensor] = None,
+                   q_rot: Optional[Tensor] = None, k_rot: Optional[Tensor] = None):
+    """Causal softmax attention; with ``sink`` the denominator also holds ``exp(sink[head])``; with ``gate`` ``[B * Sq, H]`` or
+    ``[B * Sq, H * Dv]`` the output is multiplied by its sigmoid, with ``softcap`` scores become ``softcap * tanh(score / softcap)``.
+    ``q`` ``[B, Sq, H, D]`` are the last positions of ``k``/``v`` ``[B, Sk, G, *]``; query head ``h`` reads key head ``h // (H / G)``;
+    ``keep`` ``[B, Sk]``; ``window``, ``keep_first``, ``lead`` ``[B]``: ``visible_keys``. ``q_rot`` ``[B, Sq, H, R]`` and ``k_rot`` ``[B, Sk,
+    R]``, a part of the keys that all heads share, add ``q_rot . k_rot`` to the scores before the scale. Returns ``[B * Sq, H * Dv]``
+    and the weights ``[B, H, Sq, Sk]``."""
     b, sq, h, _ = q.shape
     sk, per = k.size(1), h // k.size(2)
     if per > 1:
         k, v = k.repeat_interleave(per, dim=2), v.repeat_interleave(per, dim=2)
-    s = torch.einsum("bqhd,bkhd->bhqk", q.to(torch.float32), k.to(torch.float32)) * scale
+    s = torch.einsum("bqhd,bkhd->bhqk", q.to(torch.float32), k.to(torch.float32))
+    if q_rot is not None:
+        s = s + torch.einsum("bqhd,bkd->bhqk", q_rot.to(torch.float32), k_rot.to(torch.float32))
+    s = s * scale
     if softcap:
         s = softcap * torch.tanh(s / softcap)
-    vis = attention_mask_bias(sq, sk, q.device, True, None)[None, None]
+    qpos = torch.arange(sk - sq, sk, device=q.device)[None, None, :, None]
+    kpos = torch.arange(sk, device=q.device)[None, None, None, :]
+    vis = visible_keys(qpos, kpos, window, keep_first, None if lead is None else lead.view(-1, 1, 1, 1))
     if keep is not None:
         vis = vis & (keep != 0)[:, None, None, :]
     s = s.masked_fill(~vis, float("-inf"))
-    s = torch.cat([s, sink.to(torch.float32)[None, :, None, None].expand(b, h, sq, 1)], dim=-1)
-    p = torch.softmax(s, dim=-1)[..., :sk]
+    if sink is not None:
+        s = torch.cat([s, sink.to(torch.float32)[None, :, None, None].expand(b, h, sq, 1)], dim=-1)
+        p = torch.softmax(s, dim=-1)[..., :sk]
+    else:
+        some = vis.any(-1, keepdim=True)               # a padded query may see nothing: its row is zero
+        p = torch.softmax(s.masked_fill(~some, 0.0), dim=-1) * some
     o = torch.einsum("bhqk,bkhd->bqhd", p, v.to(torch.float32))
-    if gate is not None:
-        o = o * torch.sigmoid(gate.to(torch.float32)).view(b, sq, h, 1)
+    o = output_gate(o.reshape(b * sq, h, -1), gate)
     return o.reshape(b * sq, -1).to(q.dtype), p
 
 
+def rotate_halves(x: Tensor, positions: Tensor, freq: Tensor) -> Tensor:
+    """``x`` ``[B, S, heads, 2 n]``: dim ``i`` and dim ``i + n`` turn by ``positions * freq[i]`` (fp32); ``positions`` ``[B, S]``."""
+    n = freq.numel()
+    xf = x.to(torch.float32)
+    ang = (positions.to(torch.float32).unsqueeze(-1) * freq).unsqueeze(2)
+    sin, cos = torch.sin(ang), torch.cos(ang)
+    a, b = xf[..., :n], xf[..., n:]
+    return torch.cat((a * cos - b * sin, b * cos + a * sin), dim=-1).to(x.dtype)
+
+
 def latent_decode(q: Tensor, w_uk: Tensor, w_uv: Tensor, cache: Tensor, lengths: Tensor, keep: Optional[Tensor],
-                  sink: Tensor, gate: Tensor, scale: float, heads: int) -> Tensor:
-    """One query per row over a cache of latents ``[B, T, rank]`` without expanding keys or values: the query takes
-    ``W_uk``, the weighted sum of latents takes ``W_uv``. ``q`` ``[B, heads * dim]``; returns ``[B, heads * vdim]``."""
-    b, t, r = cache.shape
+                  sink: Optional[Tensor], gate: Tensor, scale: float, heads: int, positions: Optional[Tensor] = None,
+                  freq: Optional[Tensor] = None) -> Tensor:
+    """One query per row over a cache of latents ``[B, T, rank + rot]`` without expanding keys or values: the query takes
+    ``W_uk``, the weighted sum of latents takes ``W_uv``. ``q`` ``[B, heads * (dim + rot)]``; the last ``rot`` = ``2 * len(freq)`` dims of a
+    head are rotated (``rotate_halves``) by ``positions`` ``[B, 1]`` and meet the last ``rot`` of a cached row. Returns ``[B, heads *
+    vdim]``."""
+    b, t, _ = cache.shape
+    r = w_uk.size(1)
+    rot = cache.size(2) - r
     c = cache.to(torch.float32)
-    qa = torch.einsum("bhd,hdr->bhr", q.to(torch.float32).view(b, heads, -1), w_uk.to(torch.float32).view(heads, -1, r)) * scale
-    s = torch.einsum("bhr,btr->bht", qa, c)
+    qh = q.to(torch.float32).view(b, heads, -1)
+    dim = qh.size(-1) - rot
+    qa = torch.einsum("bhd,hdr->bhr", qh[..., :dim], w_uk.to(torch.float32).view(heads, dim, r))
+    if rot:
+        qa = torch.cat([qa, rotate_halves(qh[..., dim:].unsqueeze(1), positions, freq)[:, 0]], dim=-1)
+    s = torch.einsum("bhr,btr->bht", qa * scale, c)
     vis = torch.arange(t, device=q.device)[None, :] < lengths[:, None]
     if keep is not None:
         vis = vis.clone()
         n = min(t, keep.size(1))
         vis[:, :n] &= keep[:, :n] != 0
     s = s.masked_fill(~vis[:, None, :], float("-inf"))
-    s = torch.cat([s, sink.to(torch.float32)[None, :, None].expand(b, heads, 1)], dim=-1)
+    if sink is not None:
+        s = torch.cat([s, sink.to(torch.float32)[None, :, None].expand(b, heads, 1)], dim=-1)
     p = torch.softmax(s, dim=-1)[..., :t]
-    o = torch.einsum("bhr,hvr->bhv", torch.einsum("bht,btr->bhr", p, c), w_uv.to(torch.float32).view(heads, -1, r))
-    return (o * torch.sigmoid(gate.to(torch.float32)).unsqueeze(-1)).reshape(b, -1).to(q.dtype)
+    o = torch.einsum("bhr,hvr->bhv", torch.einsum("bht,btr->bhr", p, c[..., :r]), w_uv.to(torch.float32).view(heads, -1, r))
+    return output_gate(o, gate).reshape(b, -1).to(q.dtype)
 
 
-def moe_route(h: Tensor, w: Tensor, bias: Tensor, top: int) -> Tuple[Tensor, Tensor]:
-    """The ``top`` experts with the largest ``W h + b`` per token (``[tokens, top]``, int32) and the softmax over those logits."""
-    z = torch.matmul(h.to(torch.float32), w.to(torch.float32).t()) + bias.to(torch.float32)
-    picked, idx = torch.topk(z, top, dim=-1)
+def moe_route(h: Tensor, w: Tensor, bias: Tensor, top: int, scored: bool = False) -> Tuple[Tensor, Tensor]:
+    """The ``top`` experts with the largest ``W h + b`` per token (``[tokens, top]``, int32) and the softmax over those logits.
+    ``scored``: scores are the softmax of ``W h`` over all experts, the largest ``score + b`` are chosen, and the weights are the
+    chosen scores without ``b``, divided by their sum."""
+    z = torch.matmul(h.to(torch.float32), w.to(torch.float32).t())
+    if scored:
+        score = torch.softmax(z, dim=-1)
+        idx = torch.topk(score + bias.to(torch.float32), top, dim=-1).indices
+        picked = score.gather(-1, idx)
+        return idx.to(torch.int32), picked / (picked.sum(-1, keepdim=True) + 1e-20)
+    picked, idx = torch.topk(z + bias.to(torch.float32), top, dim=-1)
     return idx.to(torch.int32), torch.softmax(picked, dim=-1)
 
 
-def moe_experts(h: Tensor, idx: Tensor, up: Tensor, down: Tensor) -> Tensor:
-    """``W_down relu(W_up h)^2`` of every (token, choice): ``[tokens * top, width]``; ``up`` ``[experts, ff, width]``,
-    ``down`` ``[experts, width, ff]``."""
+def moe_experts(h: Tensor, idx: Tensor, up: Tensor, down: Tensor, unit: str = "relu2") -> Tensor:
+    """Every (token, choice): ``[tokens * top, width]``; ``down`` ``[experts, width, ff]``. ``unit`` ``"relu2"``: ``W_down relu(W_up h)^2``
+    with ``up`` ``[experts, ff, width]``; ``"silu"``: ``W_down (silu(W_gate h) * W_up h)`` with ``up`` ``[experts, 2 ff, width]``, rows of the
+    two matrices in turns. Rows of choices that are no expert (``idx >= experts``) are zeros."""
     n, top = idx.shape
     flat = idx.reshape(-1).to(torch.long)
     rows = h.repeat_interleave(top, dim=0)
     out = h.new_zeros(n * top, down.size(1))
     for e in flat.unique().tolist():
+        if e >= up.size(0):
+            continue
         at = (flat == e).nonzero(as_tuple=True)[0]
-        a = torch.relu(torch.matmul(rows[at], up[e].t())).pow(2)
+        a = torch.matmul(rows[at], up[e].t())
+        a = silu_mul(a[:, 0::2], a[:, 1::2]) if unit == "silu" else torch.relu(a).pow(2)
         out = out.index_copy(0, at, torch.matmul(a, down[e].t()).to(out.dtype))
     return out
+
+
+# ---------------------------------------------------------------------------------------------------------------
+# Hyper-connections: several residual streams, mixed by every sublayer.
+class SublayerResult(NamedTuple):
+    """What a sublayer hands to ``hyper_join``: ``y`` ``[tokens, width]``, or with ``weights`` ``[tokens, top]`` the weighted sum of
+    ``y``'s rows ``slots`` (``token * top + choice`` when ``None``), where a choice ``>= experts`` stands for the sublayer's input ``h``
+    itself; plus ``sigmoid(shared_gate) * shared`` (``shared_gate`` ``[tokens, 1]``) when there is a ``shared``."""
+    y: Tensor
+    slots: Optional[Tensor] = None
+    weights: Optional[Tensor] = None
+    choice: Optional[Tensor] = None
+    experts: int = 0
+    h: Optional[Tensor] = None
+    shared: Optional[Tensor] = None
+    shared_gate: Optional[Tensor] = None
+
+
+def collect_result(r: SublayerResult) -> Tensor:
+    """The sublayer's result as fp32 rows ``[tokens, width]``."""
+    y = r.y.to(torch.float32)
+    if r.weights is not None:
+        n, top = r.weights.shape
+        if r.choice is not None:
+            own = (r.choice.to(torch.long) < r.experts)
+        slots = torch.arange(n * top, device=y.device).view(n, top) if r.slots is None else r.slots.to(torch.long)
+        if r.choice is None:
+            picked = y[slots]
+        else:
+            picked = torch.where(own.unsqueeze(-1), y[torch.where(own, slots, torch.zeros_like(slots))], r.h.to(torch.float32).unsqueeze(1))
+        y = (picked * r.weights.unsqueeze(-1)).sum(1)
+    if r.shared is not None:
+        y = y + torch.sigmoid(r.shared_gate.to(torch.float32)) * r.shared.to(torch.float32)
+    return y
+
+
+def hyper_join(x: Tensor, result: Optional[SublayerResult], w_out: Optional[Tensor], mix: Optional[Tensor], w_in: Optional[Tensor],
+               w_norm: Tensor, eps: float, scale: float = 1.0) -> Tuple[Tensor, Tensor]:
+    """Streams ``x`` ``[tokens, streams, width]`` (fp32) take a sublayer's result ``y``: ``x_t <- sum_s mix[s, t] x_s + w_out[t] y`` (all
+    streams from the old ones; no ``result``: they stay), and what the next sublayer reads: ``u = sum_t w_in[t] x_t`` (``None``: their
+    plain sum), normed with weight ``1 + w_norm`` and multiplied by ``scale``."""
+    if result is not None:
+        y = collect_result(result)
+        x = torch.einsum("nsw,st->ntw", x, mix.to(torch.float32)) + w_out.to(torch.float32)[None, :, None] * y.unsqueeze(1)
+    u = x.sum(1) if w_in is None else (x * w_in.to(torch.float32)[None, :, None]).sum(1)
+    r = torch.rsqrt(u.pow(2).mean(-1, keepdim=True) + eps)
+    return x, (u * r * ((1.0 + w_norm.to(torch.float32)) * scale)).to(w_norm.dtype)
 
 
 # ---------------------------------------------------------------------------------------------------------------
@@ -328,11 +438,13 @@ def rotary_frequencies(rot_dims: int, base: float):
 
 
 def norm_rotate(x: Tensor, w: Optional[Tensor], eps: float, positions: Tensor, freq: Optional[Tensor]) -> Tensor:
-    """Per head of ``x`` ``[B, S, heads, D]``: RMS norm with weight ``w`` ``[D]`` (shared by the heads), then the interleaved
-    rotation of the first ``2 * len(freq)`` dims by ``positions * freq`` (fp32); ``positions`` ``[B, S]``."""
+    """Per head of ``x`` ``[B, S, heads, D]``: RMS norm with weight ``w`` ``[D]`` (shared by the heads; ``None``: without a weight, and
+    then before or after the rotation is the same), then the interleaved rotation of the first ``2 * len(freq)`` dims by
+    ``positions * freq`` (fp32); ``positions`` ``[B, S]``."""
     y = x.to(torch.float32)
+    y = y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + eps)
     if w is not None:
-        y = y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + eps) * w.to(torch.float32)
+        y = y * w.to(torch.float32)
     if freq is not None and freq.numel():
         r = 2 * freq.numel()
         ang = (positions.to(torch.float32).unsqueeze(-1) * freq).unsqueeze(2)
@@ -342,13 +454,15 @@ def norm_rotate(x: Tensor, w: Optional[Tensor], eps: float, positions: Tensor, f
     return y.to(x.dtype)
 
 
-def grouped_decode(q: Tensor, k: Tensor, v: Tensor, lengths: Tensor, keep: Optional[Tensor], sink: Tensor, scale: float,
-                   softcap: float = 0.0) -> Tensor:
+def grouped_decode(q: Tensor, k: Tensor, v: Tensor, lengths: Tensor, keep: Optional[Tensor], sink: Optional[Tensor], scale: float,
+                   softcap: float = 0.0, gate: Optional[Tensor] = None, window: int = 0, keep_first: int = 0,
+                   lead: Optional[Tensor] = None) -> Tensor:
     """One query per row: ``q`` ``[B, H, D]`` over caches ``[B, G, T, *]`` of which the first ``lengths[b]`` positions count;
-    ``keep`` ``[B, <= T]``. Softmax with a sink as in ``sink_attention``. Returns ``[B, H * Dv]``."""
+    ``keep`` ``[B, <= T]``. Sink, gate ``[B, H]`` and window as in ``sink_attention``. Returns ``[B, H * Dv]``."""
     b, h, _ = q.shape
     g, t = k.size(1), k.size(2)
-    vis = torch.arange(t, device=q.device)[None, :] < lengths[:, None]
+    at = torch.arange(t, device=q.device)[None, :]
+    vis = visible_keys(lengths[:, None] - 1, at, window, keep_first, None if lead is None else lead[:, None])
     if keep is not None:
         n = min(t, keep.size(1))
         vis[:, :n] &= keep[:, :n] != 0
@@ -357,21 +471,64 @@ def grouped_decode(q: Tensor, k: Tensor, v: Tensor, lengths: Tensor, keep: Optio
     if softcap:
         s = softcap * torch.tanh(s / softcap)
     s = s.masked_fill(~vis[:, None, None, :], float("-inf"))
-    s = torch.cat([s, sink.to(torch.float32).view(1, g, h // g, 1).expand(b, g, h // g, 1)], dim=-1)
+    if sink is not None:
+        s = torch.cat([s, sink.to(torch.float32).view(1, g, h // g, 1).expand(b, g, h // g, 1)], dim=-1)
     p = torch.softmax(s, dim=-1)[..., :t]
     # positions beyond the length may hold anything
     vf = torch.where(vis[:, None, :, None], v.to(torch.float32), torch.zeros((), device=v.device))
-    return torch.einsum("bgrt,bgtd->bgrd", p, vf).reshape(b, -1).to(q.dtype)
+    o = torch.einsum("bgrt,bgtd->bgrd", p, vf).reshape(b, h, -1)
+    return output_gate(o, gate).reshape(b, -1).to(q.dtype)
 
 
-def gated_rms_norm(o: Tensor, w: Tensor, gate: Tensor, eps: float, group: int, act: str) -> Tensor:
+def gated_rms_norm(o: Tensor, w: Tensor, gate: Tensor, eps: float, group: int, act: str,
+                   normalizer: Optional[Tuple[Tensor, Tensor]] = None) -> Tensor:
     """Every run of ``group`` columns of ``o`` ``[rows, n]`` divided by its root mean square, times ``w`` ``[n]``, times
-    ``sigmoid(gate)`` or ``silu(gate)`` (``act``); in ``w``'s dtype."""
+    ``sigmoid(gate)`` or ``silu(gate)`` (``act``); in ``w``'s dtype. ``normalizer`` ``(z, m)``, both ``[rows, n / group]``: the runs are first
+    divided by ``max(|z|, exp(-m)) + 1e-6``."""
     of = o.to(torch.float32).reshape(o.size(0), -1, group)
+    if normalizer is not None:
+        z, m = (t.reshape(o.size(0), -1, 1) for t in normalizer)
+        of = of / (torch.maximum(z.abs(), torch.exp(-m)) + 1e-6)
     of = (of * torch.rsqrt(of.pow(2).mean(-1, keepdim=True) + eps)).view(o.size(0), -1)
     g = gate.to(torch.float32)
     g = torch.sigmoid(g) if act == "sigmoid" else F.silu(g)
     return (of * w.to(torch.float32) * g).to(w.dtype)
+
+
+def memory_state_width(vdim: int) -> int:
+    """Columns of a matrix-memory state: ``vdim`` values, the normaliser, and padding to a multiple of 4."""
+    return (vdim + 1 + 3) // 4 * 4
+
+
+def matrix_memory(q: Tensor, k: Tensor, v: Tensor, z: Tensor, bias: Tensor, cap: float, keep: Optional[Tensor], state: Optional[Tensor],
+                  top: Optional[Tensor], batch: int, heads: int):
+    """Linear attention with one input and one forget gate per head and token in the exponent (mLSTM). ``z`` ``[B * S, 2 * heads]`` and
+    ``bias`` ``[2 * heads]``, input gates first: ``i = cap tanh((z_i + b_i) / cap)``, ``f = log sigmoid(cap tanh((z_f + b_f) / cap))``. With
+    the running maximum ``m = max(f + m', i)`` (``m' = 0`` before the first token): ``S <- exp(f + m' - m) S + exp(i - m) k v^T``, ``n``
+    likewise from ``k`` alone. ``q`` is scaled by ``dim^-1/2``. ``state`` ``[B, heads, dim, memory_state_width(vdim)]`` holds ``S`` and, in
+    column ``vdim``, ``n``; ``top`` ``[B, heads]`` holds ``m``. A padded token leaves all of it as it is.
+    Returns ``S^T q`` ``[B * S, heads * vdim]``, ``n . q`` and ``m`` ``[B * S, heads]`` (fp32), the final state and maximum."""
+    dim, vdim = q.size(1) // heads, v.size(1) // heads
+    qf, kf, vf = (t.to(torch.float32).reshape(batch, -1, heads, t.size(1) // heads) for t in (q, k, v))
+    qf = qf * dim ** -0.5
+    g = cap * torch.tanh((z.to(torch.float32) + bias.to(torch.float32)) / cap)
+    i, f = g[:, :heads].reshape(batch, -1, heads), F.logsigmoid(g[:, heads:]).reshape(batch, -1, heads)
+    v1 = F.pad(torch.cat([vf, torch.ones_like(vf[..., :1])], dim=-1), (0, memory_state_width(vdim) - vdim - 1))
+    s = torch.zeros(batch, heads, dim, v1.size(-1), device=q.device) if state is None else state
+    m = torch.zeros(batch, heads, device=q.device) if top is None else top
+    out, tops = [], []
+    for t in range(qf.size(1)):
+        new_m = torch.maximum(f[:, t] + m, i[:, t])
+        forget, write = torch.exp(f[:, t] + m - new_m), torch.exp(i[:, t] - new_m)
+        new = forget[..., None, None] * s + (write[..., None] * kf[:, t]).unsqueeze(-1) * v1[:, t].unsqueeze(-2)
+        on = None if keep is None else keep[:, t] != 0
+        s = new if on is None else torch.where(on.view(-1, 1, 1, 1), new, s)
+        m = new_m if on is None else torch.where(on.view(-1, 1), new_m, m)
+        o = torch.einsum("bhi,bhij->bhj", qf[:, t], s)
+        out.append(o if on is None else o * on.to(torch.float32).view(-1, 1, 1))
+        tops.append(m)
+    o = torch.stack(out, dim=1).reshape(q.size(0), heads, -1)
+    return o[..., :vdim].reshape(q.size(0), heads * vdim), o[..., vdim], torch.stack(tops, dim=1).reshape(q.size(0), heads), s, m
 
 
 def decayed_attention(q: Tensor, k: Tensor, v: Tensor, decay: Tensor, keep: Optional[Tensor], state: Optional[Tensor],

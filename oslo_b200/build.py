@@ -25,11 +25,12 @@ BUILD = os.path.join(HERE, "csrc", "build")
 
 CUDA_SOURCES = ["gemm_sm100.cu", "elementwise.cu", "attention.cu", "attention_sm100.cu", "attention_bwd_sm100.cu",
                 "decode_sm100.cu", "comm.cu", "fused_comm_gemm.cu", "noalloc_colsum.cu", "rms_norm.cu",
-                "linear_recurrence.cu", "latent_attention.cu", "moe.cu", "grouped_attention.cu", "selective_scan.cu"]
+                "linear_recurrence.cu", "latent_attention.cu", "moe.cu", "grouped_attention.cu", "selective_scan.cu",
+                "matrix_memory.cu", "hyper_connections.cu"]
 # kernels that also serve float32 models and keep routers, norms and recurrences in 32-bit: IEEE division / square root
 # and the accurate exponential
 ACCURATE_SOURCES = ("rms_norm.cu", "linear_recurrence.cu", "latent_attention.cu", "moe.cu", "grouped_attention.cu",
-                    "selective_scan.cu")
+                    "selective_scan.cu", "matrix_memory.cu", "hyper_connections.cu")
 CPP_SOURCES = ["bindings.cpp"]
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-std=c++17", "-O3", "-lineinfo",
               "--use_fast_math", "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=hidden",

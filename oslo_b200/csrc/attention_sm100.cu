@@ -39,26 +39,37 @@ struct FaParams {
   int group;            // query heads per key / value head
   float softcap;        // CAP kernels: scores become softcap * tanh(score / softcap)
   // softmax with a sink and an output gate (null: without): exp(sink[h]) joins the denominator, row s of
-  // head h is multiplied by sigmoid(gate[(b * Sq + s) * ldg + h]); only the first d_out columns are stored
+  // head h is multiplied by sigmoid(gate[(b * Sq + s) * ldg + h]), or (gate_wide) every element by that of
+  // gate[(b * Sq + s) * ldg + h * d_out + column]; only the first d_out columns are stored
   const void* sink;
   const void* gate;
   long long ldg;
-  int d_out;
+  int d_out, gate_wide;
+  // a window that also sees the sequence's first keep_first keys; lead [B] (or nullptr): padding ahead of a sequence
+  int keep_first;
+  const int* lead;
+  // 64-column sub-tiles of the query and key operands that come from tq / tk; the others come from tq2 / tk2 (a part
+  // of the keys that all heads share)
+  int sub_first;
+  int q2_pos[3], k2_pos[3];
 };
 
 // PT = true: P goes back into TMEM (over the S buffer it came from, two bf16 per 32-bit column) and is the
 // A operand of P V straight from tensor memory; PT = false: P goes through a swizzled shared-memory tile.
 // CAP = true: capped scores, tanh(u) = 1 - 2 / (exp(2u) + 1) in 32-bit (absolute error about 2^-23 of the cap).
 // Head sizes below D: the tensor maps are as wide as the heads, TMA fills the rest of a tile with zeros.
-template <int D, int BN, bool PT, bool CAP>
+// DQ: columns of the query and key tiles, D: of the value tiles and the result. PARTS = true: the last sub-tiles of
+// queries and keys have tensor maps of their own.
+template <int DQ, int D, int BN, bool PT, bool CAP, bool PARTS>
 __global__ void __launch_bounds__(FA_THREADS, 1)
 fa_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUtensorMap tk,
-              const __grid_constant__ CUtensorMap tv, const FaParams p) {
-  constexpr int DC = D / 64;                     // 64-column sub-tiles per row operand
+              const __grid_constant__ CUtensorMap tv, const __grid_constant__ CUtensorMap tq2,
+              const __grid_constant__ CUtensorMap tk2, const FaParams p) {
+  constexpr int DC = DQ / 64, VC = D / 64;       // 64-column sub-tiles per row operand
   constexpr uint32_t Q_SUB = FA_BM * 128;        // bytes of one [128 x 64] sub-tile (Q and P)
   constexpr uint32_t KV_SUB = BN * 128;          // bytes of one [BN x 64] sub-tile (K and V)
   constexpr uint32_t Q_BYTES = DC * Q_SUB;
-  constexpr uint32_t KV_BYTES = DC * KV_SUB;
+  constexpr uint32_t K_BYTES = DC * KV_SUB, V_BYTES = VC * KV_SUB;
   constexpr uint32_t P_BYTES = PT ? 0u : (BN / 64) * Q_SUB;
   constexpr uint32_t TMEM_COLS = 512;
   constexpr uint32_t O_COL = 2 * BN;             // S buffers at columns [0, BN) and [BN, 2 BN)
@@ -68,9 +79,9 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(fa_smem_raw) + 1023) & ~uintptr_t(1023));
   const uint32_t q_s = smem_u32(smem);
   const uint32_t k_s = q_s + Q_BYTES;            // 2 stages
-  const uint32_t v_s = k_s + 2 * KV_BYTES;       // 2 stages
-  const uint32_t p_s = v_s + 2 * KV_BYTES;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + Q_BYTES + 4 * KV_BYTES + P_BYTES);
+  const uint32_t v_s = k_s + 2 * K_BYTES;        // 2 stages
+  const uint32_t p_s = v_s + 2 * V_BYTES;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + Q_BYTES + 2 * (K_BYTES + V_BYTES) + P_BYTES);
   const uint32_t bar0 = smem_u32(bars);
   // 0 q_full | 1,2 k_full | 3,4 k_empty | 5,6 v_full | 7,8 v_empty | 9,10 s_full | 11,12 s_empty | 13 p_ready[0] |
   // 14 pv_done | 15 p_ready[1] (PT only: one per S/P buffer)
@@ -85,7 +96,12 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
   int key_hi = p.Sk, key_lo = 0;
   if (p.causal) key_hi = min(p.Sk, q0 + FA_BM + offset);
   if (p.window > 0) key_lo = max(0, q0 + offset - p.window + 1) / BN * BN;
-  const int nblk = key_hi > key_lo ? (key_hi - key_lo + BN - 1) / BN : 0;
+  // the kept keys' blocks ahead of the window's come first
+  const int lead = p.lead ? p.lead[b] : 0;
+  const int kept_lo = max(0, lead) / BN * BN, kept_hi = min(key_lo, lead + p.keep_first);
+  const int nkept = kept_hi > kept_lo ? (kept_hi - kept_lo + BN - 1) / BN : 0;
+  const int nblk = nkept + (key_hi > key_lo ? (key_hi - key_lo + BN - 1) / BN : 0);
+  auto block_start = [&](int j) { return j < nkept ? kept_lo + j * BN : key_lo + (j - nkept) * BN; };
 
   if (threadIdx.x == 0) {
     for (int i = 0; i < 16; ++i) {
@@ -110,23 +126,30 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
       tma_prefetch_desc(&tq); tma_prefetch_desc(&tk); tma_prefetch_desc(&tv);
       mbar_expect_tx(bar(0), Q_BYTES);
 #pragma unroll
-      for (int c = 0; c < DC; ++c) tma_load_rows(q_s + c * Q_SUB, &tq, bar(0), c * 64, q0, h, b, p.q_pos);
+      for (int c = 0; c < DC; ++c) {
+        if (PARTS && c >= p.sub_first) tma_load_rows(q_s + c * Q_SUB, &tq2, bar(0), (c - p.sub_first) * 64, q0, h, b, p.q2_pos);
+        else tma_load_rows(q_s + c * Q_SUB, &tq, bar(0), c * 64, q0, h, b, p.q_pos);
+      }
       bool ok = true;
       const int hk = h / p.group;
       for (int j = 0; j < nblk && ok; ++j) {
         const int st = j & 1;
         const uint32_t ph = (j >> 1) & 1;
-        const int n0 = key_lo + j * BN;
+        const int n0 = block_start(j);
         ok = mbar_wait(bar(3 + st), ph ^ 1, abort_flag, p.err, ERR_WAIT_EMPTY);
         if (!ok) break;
-        mbar_expect_tx(bar(1 + st), KV_BYTES);
+        mbar_expect_tx(bar(1 + st), K_BYTES);
 #pragma unroll
-        for (int c = 0; c < DC; ++c) tma_load_rows(k_s + st * KV_BYTES + c * KV_SUB, &tk, bar(1 + st), c * 64, n0, hk, b, p.k_pos);
+        for (int c = 0; c < DC; ++c) {
+          const uint32_t dst = k_s + st * K_BYTES + c * KV_SUB;
+          if (PARTS && c >= p.sub_first) tma_load_rows(dst, &tk2, bar(1 + st), (c - p.sub_first) * 64, n0, 0, b, p.k2_pos);
+          else tma_load_rows(dst, &tk, bar(1 + st), c * 64, n0, hk, b, p.k_pos);
+        }
         ok = mbar_wait(bar(7 + st), ph ^ 1, abort_flag, p.err, ERR_WAIT_EMPTY);
         if (!ok) break;
-        mbar_expect_tx(bar(5 + st), KV_BYTES);
+        mbar_expect_tx(bar(5 + st), V_BYTES);
 #pragma unroll
-        for (int c = 0; c < DC; ++c) tma_load_rows(v_s + st * KV_BYTES + c * KV_SUB, &tv, bar(5 + st), c * 64, n0, hk, b, p.v_pos);
+        for (int c = 0; c < VC; ++c) tma_load_rows(v_s + st * V_BYTES + c * KV_SUB, &tv, bar(5 + st), c * 64, n0, hk, b, p.v_pos);
       }
     }
   } else if (warp == 1) {
@@ -143,9 +166,9 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
         if (!mbar_wait(bar(11 + st), ph ^ 1, abort_flag, p.err, ERR_WAIT_TMEM_EMPTY)) return false;
         tc_fence_after();
 #pragma unroll
-        for (int kk = 0; kk < D / 16; ++kk) {
+        for (int kk = 0; kk < DQ / 16; ++kk) {
           const uint64_t da = make_smem_desc(q_s + (kk >> 2) * Q_SUB + (kk & 3) * 32, 16, 1024);
-          const uint64_t db = make_smem_desc(k_s + st * KV_BYTES + (kk >> 2) * KV_SUB + (kk & 3) * 32, 16, 1024);
+          const uint64_t db = make_smem_desc(k_s + st * K_BYTES + (kk >> 2) * KV_SUB + (kk & 3) * 32, 16, 1024);
           umma_f16(tmem_base + st * BN, da, db, idesc_qk, kk != 0);
         }
         umma_commit(bar(3 + st));   // K stage may be refilled once these MMAs have read it
@@ -167,7 +190,7 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
         tc_fence_after();
 #pragma unroll
         for (int ks = 0; ks < BN / 16; ++ks) {
-          const uint64_t db = make_smem_desc(v_s + st * KV_BYTES + ks * 2048, KV_SUB, 1024);
+          const uint64_t db = make_smem_desc(v_s + st * V_BYTES + ks * 2048, KV_SUB, 1024);
           if (PT) {
             umma_f16_ts(tmem_base + O_COL, tmem_base + st * BN + ks * 8, db, idesc_pv, (j | ks) != 0);
           } else {
@@ -193,7 +216,7 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
     bool ok = true;
     for (int j = 0; j < nblk && ok; ++j) {
       const int st = j & 1;
-      const int n0 = key_lo + j * BN;
+      const int n0 = block_start(j);
       ok = mbar_wait(bar(9 + st), (j >> 1) & 1, abort_flag, p.err, ERR_WAIT_TMEM_FULL);
       if (!ok) break;
       tc_fence_after();
@@ -223,7 +246,7 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
           const int col = n0 + i;
           bool vis = col < p.Sk;
           if (p.causal && col > qpos) vis = false;
-          if (p.window > 0 && col <= qpos - p.window) vis = false;
+          if (p.window > 0 && col <= qpos - p.window && col - lead >= p.keep_first) vis = false;
           if (vis && kpm_row && !kpm_row[col]) vis = false;
           if (!vis) s[i] = -CUDART_INF_F;
         }
@@ -319,13 +342,18 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
       tc_fence_after();
     }
     float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
-    if (p.sink != nullptr && row < p.Sq && l_sum > 0.f) {
-      const long long gi = (static_cast<long long>(b) * p.Sq + row) * p.ldg + h;
-      const float snk = fp16 ? __half2float(static_cast<const __half*>(p.sink)[h])
-                             : __bfloat162float(static_cast<const __nv_bfloat16*>(p.sink)[h]);
-      // m_ref is the running reference in log2 units; an overflowing sink term gives 1 / inf = 0
-      inv = l_sum + exp2f(snk * 1.4426950408889634f - m_ref);
-      if (p.gate != nullptr) {
+    const long long gate_row = (static_cast<long long>(b) * p.Sq + row) * p.ldg;
+    const bool wide = p.gate != nullptr && p.gate_wide;
+    if ((p.sink != nullptr || p.gate != nullptr) && row < p.Sq && l_sum > 0.f) {
+      const long long gi = gate_row + h;
+      inv = l_sum;
+      if (p.sink != nullptr) {
+        const float snk = fp16 ? __half2float(static_cast<const __half*>(p.sink)[h])
+                               : __bfloat162float(static_cast<const __nv_bfloat16*>(p.sink)[h]);
+        // m_ref is the running reference in log2 units; an overflowing sink term gives 1 / inf = 0
+        inv += exp2f(snk * 1.4426950408889634f - m_ref);
+      }
+      if (p.gate != nullptr && !wide) {
         const float gate = fp16 ? __half2float(static_cast<const __half*>(p.gate)[gi])
                                 : __bfloat162float(static_cast<const __nv_bfloat16*>(p.gate)[gi]);
         inv *= 1.f + exp2f(-gate * 1.4426950408889634f);
@@ -347,6 +375,17 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
 #pragma unroll
         for (int i = 0; i < 32; i += 8) {
           if (c0 + i >= p.d_out) break;
+          if (wide) {
+            const uint4 g4 = *reinterpret_cast<const uint4*>(static_cast<const uint16_t*>(p.gate) + gate_row + h * p.d_out + c0 + i);
+            const uint32_t gw[4] = {g4.x, g4.y, g4.z, g4.w};
+#pragma unroll
+            for (int u = 0; u < 4; ++u) {
+              const float2 g = fp16 ? __half22float2(*reinterpret_cast<const __half2*>(&gw[u]))
+                                    : __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gw[u]));
+              r[i + 2 * u] = __float_as_uint(__fdividef(__uint_as_float(r[i + 2 * u]), 1.f + exp2f(-g.x * 1.4426950408889634f)));
+              r[i + 2 * u + 1] = __float_as_uint(__fdividef(__uint_as_float(r[i + 2 * u + 1]), 1.f + exp2f(-g.y * 1.4426950408889634f)));
+            }
+          }
           uint4 v;
           v.x = fa_pack2(__uint_as_float(r[i]) * inv, __uint_as_float(r[i + 1]) * inv, fp16);
           v.y = fa_pack2(__uint_as_float(r[i + 2]) * inv, __uint_as_float(r[i + 3]) * inv, fp16);
@@ -376,32 +415,53 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
 }
 
 // ---------------------------------------------------------------------- host side
-template <int D, int BN, bool PT, bool CAP = false>
-static int fa_launch(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const FaParams& p,
-                     cudaStream_t stream) {
-  constexpr size_t smem = FA_BM * D * 2 + 4 * BN * D * 2 + (PT ? 0 : FA_BM * BN * 2) + 16 * 8 + 16 + 1024;
+struct FaMaps {
+  CUtensorMap q, k, v, q2, k2;                   // q2, k2: copies of q, k where there is no second part
+};
+template <int DQ, int D, int BN, bool PT, bool CAP, bool PARTS>
+static int fa_launch_parts(const FaMaps& t, const FaParams& p, cudaStream_t stream) {
+  constexpr size_t smem = FA_BM * DQ * 2 + 2 * BN * (DQ + D) * 2 + (PT ? 0 : FA_BM * BN * 2) + 16 * 8 + 16 + 1024;
+  static_assert(smem <= 232448, "shared memory budget of one CTA");
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(fa_fwd_kernel<D, BN, PT, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    cudaError_t e = cudaFuncSetAttribute(fa_fwd_kernel<DQ, D, BN, PT, CAP, PARTS>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          static_cast<int>(smem));
     if (e != cudaSuccess) return static_cast<int>(e);
     configured = true;
   }
   dim3 grid((p.Sq + FA_BM - 1) / FA_BM, p.H, p.B);
-  fa_fwd_kernel<D, BN, PT, CAP><<<grid, FA_THREADS, smem, stream>>>(tq, tk, tv, p);
+  fa_fwd_kernel<DQ, D, BN, PT, CAP, PARTS><<<grid, FA_THREADS, smem, stream>>>(t.q, t.k, t.v, t.q2, t.k2, p);
   return static_cast<int>(cudaGetLastError());
+}
+template <int D, int BN, bool PT, bool CAP = false>
+static int fa_launch(const FaMaps& t, const FaParams& p, cudaStream_t stream) {
+  return fa_launch_parts<D, D, BN, PT, CAP, false>(t, p, stream);
 }
 
 }  // namespace oslo
 
 namespace oslo {
+// what only some models have: a window's kept first keys, and a second part of queries and keys, q2 [B, H, Sq, rot] and
+// k2 [B, Sk, rot] (one for all heads)
+struct FaExtras {
+  int keep_first = 0;
+  const int* lead = nullptr;
+  int gate_wide = 0;
+  const void *q2 = nullptr, *k2 = nullptr;
+  int rot = 0;
+  long long q2_sb = 0, q2_sh = 0, q2_ss = 0, k2_sb = 0, k2_ss = 0;
+};
+
 static int flash_fwd_entry(const void* q, const void* k, const void* v, void* o, float* lse, const uint8_t* kpm,
                            const void* sink, const void* gate, long long ldg, int B, int H, int G, int Sq, int Sk, int dim, int vdim,
                            long long q_sb, long long q_sh, long long q_ss, long long k_sb, long long k_sh, long long k_ss,
                            long long v_sb, long long v_sh, long long v_ss, long long o_sb, long long o_sh, long long o_ss,
-                           float scale, float softcap, int causal, int window, int dtype, int* err_word, cudaStream_t stream) {
+                           float scale, float softcap, int causal, int window, int dtype, int* err_word, cudaStream_t stream,
+                           const FaExtras& x = FaExtras()) {
   if (B <= 0 || H <= 0 || Sq <= 0 || Sk <= 0 || G <= 0 || H % G) return -1;
-  const int widest = std::max(dim, vdim);
+  const bool parts = x.rot > 0;
+  const int sub_first = (dim + 63) / 64, sub_all = sub_first + (x.rot + 63) / 64;
+  const int widest = std::max(parts ? sub_all * 64 : dim, vdim);
   const int D = widest <= 64 ? 64 : (widest <= 128 ? 128 : 256);
   if (dim <= 0 || vdim <= 0 || widest > 256 || dim % 8 || vdim % 8) return -2;
   if (dtype != OSLO_DT_BF16 && dtype != OSLO_DT_FP16) return -3;
@@ -409,34 +469,51 @@ static int flash_fwd_entry(const void* q, const void* k, const void* v, void* o,
   static thread_local bool ctx_bound = false;
   if (!ctx_bound) { cudaFree(nullptr); ctx_bound = true; }
   const bool fp16 = dtype == OSLO_DT_FP16;
-  const int bn = D == 256 ? 64 : 128;
+  const bool narrow = parts && sub_all == 3 && vdim <= 128;    // 192 query and key columns, 128 value columns
+  const int bn = D == 256 && !narrow ? 64 : 128;
+  if (parts && (x.rot % 8 || softcap > 0.f)) return -2;
+  if (x.gate_wide && (ldg % 8 || (reinterpret_cast<uintptr_t>(gate) & 15))) return -4;
   FaParams p;
   p.out = o; p.lse = lse; p.kpm = kpm;
-  p.sink = sink; p.gate = gate; p.ldg = ldg; p.d_out = vdim; p.group = H / G; p.softcap = softcap;
+  p.sink = sink; p.gate = gate; p.ldg = ldg; p.d_out = vdim; p.gate_wide = x.gate_wide;
+  p.keep_first = window > 0 ? x.keep_first : 0; p.lead = x.lead; p.sub_first = sub_first;
+  p.group = H / G; p.softcap = softcap;
   p.B = B; p.H = H; p.Sq = Sq; p.Sk = Sk;
   p.o_sb = o_sb; p.o_sh = o_sh; p.o_ss = o_ss;
   p.scale = scale; p.causal = causal; p.window = window; p.fp16 = fp16 ? 1 : 0; p.err = err_word;
-  CUtensorMap tq, tk, tv;
-  int rc = make_qkv_map(&tq, q, B, H, Sq, dim, q_sb, q_sh, q_ss, FA_BM, fp16, p.q_pos);
+  FaMaps t;
+  int rc = make_qkv_map(&t.q, q, B, H, Sq, dim, q_sb, q_sh, q_ss, FA_BM, fp16, p.q_pos);
   if (rc) return rc;
-  rc = make_qkv_map(&tk, k, B, G, Sk, dim, k_sb, k_sh, k_ss, bn, fp16, p.k_pos);
+  rc = make_qkv_map(&t.k, k, B, G, Sk, dim, k_sb, k_sh, k_ss, bn, fp16, p.k_pos);
   if (rc) return rc - 1000;
-  rc = make_qkv_map(&tv, v, B, G, Sk, vdim, v_sb, v_sh, v_ss, bn, fp16, p.v_pos);
+  rc = make_qkv_map(&t.v, v, B, G, Sk, vdim, v_sb, v_sh, v_ss, bn, fp16, p.v_pos);
   if (rc) return rc - 2000;
+  t.q2 = t.q;
+  t.k2 = t.k;
+  if (parts) {
+    rc = make_qkv_map(&t.q2, x.q2, B, H, Sq, x.rot, x.q2_sb, x.q2_sh, x.q2_ss, FA_BM, fp16, p.q2_pos);
+    if (rc) return rc - 3000;
+    // one head, so its stride only has to be valid
+    rc = make_qkv_map(&t.k2, x.k2, B, 1, Sk, x.rot, x.k2_sb, x.k2_ss, x.k2_ss, bn, fp16, p.k2_pos);
+    if (rc) return rc - 4000;
+    if (D == 128) return fa_launch_parts<128, 128, 128, true, false, true>(t, p, stream);
+    if (narrow) return fa_launch_parts<192, 128, 128, true, false, true>(t, p, stream);
+    return fa_launch_parts<256, 256, 64, true, false, true>(t, p, stream);
+  }
   if (softcap > 0.f) {
-    if (D == 64) return fa_launch<64, 128, true, true>(tq, tk, tv, p, stream);
-    if (D == 128) return fa_launch<128, 128, true, true>(tq, tk, tv, p, stream);
-    return fa_launch<256, 64, true, true>(tq, tk, tv, p, stream);
+    if (D == 64) return fa_launch<64, 128, true, true>(t, p, stream);
+    if (D == 128) return fa_launch<128, 128, true, true>(t, p, stream);
+    return fa_launch<256, 64, true, true>(t, p, stream);
   }
   static const bool p_smem = [] { const char* e = getenv("OSLO_B200_ATTN_P_SMEM"); return e && e[0] == '1'; }();
   if (p_smem) {
-    if (D == 64) return fa_launch<64, 128, false>(tq, tk, tv, p, stream);
-    if (D == 128) return fa_launch<128, 128, false>(tq, tk, tv, p, stream);
-    return fa_launch<256, 64, false>(tq, tk, tv, p, stream);
+    if (D == 64) return fa_launch<64, 128, false>(t, p, stream);
+    if (D == 128) return fa_launch<128, 128, false>(t, p, stream);
+    return fa_launch<256, 64, false>(t, p, stream);
   }
-  if (D == 64) return fa_launch<64, 128, true>(tq, tk, tv, p, stream);
-  if (D == 128) return fa_launch<128, 128, true>(tq, tk, tv, p, stream);
-  return fa_launch<256, 64, true>(tq, tk, tv, p, stream);
+  if (D == 64) return fa_launch<64, 128, true>(t, p, stream);
+  if (D == 128) return fa_launch<128, 128, true>(t, p, stream);
+  return fa_launch<256, 64, true>(t, p, stream);
 }
 }  // namespace oslo
 
@@ -455,9 +532,13 @@ extern "C" int oslo_flash_sink_fwd_sm100(const void* q, const void* k, const voi
                                          const void* sink, const void* gate, long long ldg, int B, int H, int G, int Sq, int Sk,
                                          int dim, int vdim, long long q_sb, long long q_sh, long long q_ss, long long k_sb,
                                          long long k_sh, long long k_ss, long long v_sb, long long v_sh, long long v_ss,
-                                         long long o_sb, long long o_sh, long long o_ss, float scale, float softcap, int dtype,
-                                         int* err_word, cudaStream_t stream) {
-  if (sink == nullptr) return -1;
+                                         long long o_sb, long long o_sh, long long o_ss, float scale, float softcap, int window,
+                                         int keep_first, const int* lead, int gate_wide, const void* q2, long long q2_sb,
+                                         long long q2_sh, long long q2_ss, const void* k2, long long k2_sb, long long k2_ss, int rot,
+                                         int dtype, int* err_word, cudaStream_t stream) {
+  oslo::FaExtras x;
+  x.keep_first = keep_first; x.lead = lead; x.gate_wide = gate_wide; x.q2 = q2; x.k2 = k2; x.rot = q2 ? rot : 0;
+  x.q2_sb = q2_sb; x.q2_sh = q2_sh; x.q2_ss = q2_ss; x.k2_sb = k2_sb; x.k2_ss = k2_ss;
   return oslo::flash_fwd_entry(q, k, v, o, nullptr, kpm, sink, gate, ldg, B, H, G, Sq, Sk, dim, vdim, q_sb, q_sh, q_ss, k_sb, k_sh,
-                               k_ss, v_sb, v_sh, v_ss, o_sb, o_sh, o_ss, scale, softcap, 1, 0, dtype, err_word, stream);
+                               k_ss, v_sb, v_sh, v_ss, o_sb, o_sh, o_ss, scale, softcap, 1, window, dtype, err_word, stream, x);
 }

@@ -840,17 +840,73 @@ std::tuple<Tensor, Tensor, Tensor> branch_join(const Tensor& x, const Tensor& y0
   return {xo, h1, h2};
 }
 
-Tensor gated_rms_norm(const Tensor& o, const Tensor& w, const Tensor& gate, double eps, int64_t group, int64_t act) {
+Tensor gated_rms_norm(const Tensor& o, const Tensor& w, const Tensor& gate, double eps, int64_t group, int64_t act,
+                      const optional<Tensor>& z, const optional<Tensor>& m) {
   check_rows(o, "o"); check_rows(gate, "gate");
   TORCH_CHECK(o.scalar_type() == at::kFloat && o.is_contiguous() && w.is_contiguous() && w.numel() == o.size(1) &&
                   gate.size(0) == o.size(0) && gate.size(1) == o.size(1) && gate.scalar_type() == w.scalar_type() && group > 0 &&
                   o.size(1) % group == 0, "gated_rms_norm: operands");
+  for (const optional<Tensor>* t : {&z, &m})
+    TORCH_CHECK(!ptr_or_null(*t) || ((*t)->is_contiguous() && (*t)->scalar_type() == at::kFloat && (*t)->numel() == o.size(0) * (o.size(1) / group)),
+                "gated_rms_norm: normalizer");
   c10::cuda::CUDAGuard guard(o.device());
   Tensor out = at::empty({o.size(0), o.size(1)}, w.options());
-  check_rc(oslo_gated_rms_norm(o.data_ptr<float>(), w.data_ptr(), gate.data_ptr(), gate.stride(0), out.data_ptr(), o.size(0),
+  check_rc(oslo_gated_rms_norm(o.data_ptr<float>(), w.data_ptr(), gate.data_ptr(), gate.stride(0), out.data_ptr(),
+                               static_cast<const float*>(ptr_or_null(z)), static_cast<const float*>(ptr_or_null(m)), o.size(0),
                                static_cast<int>(o.size(1)), static_cast<int>(group), static_cast<float>(eps), static_cast<int>(act),
                                dt_code(w), cur_stream()), "gated_rms_norm");
   return out;
+}
+
+// residual streams take a sublayer's result (y, ...; none: they stay) and the next sublayer's input is read from them
+std::tuple<Tensor, Tensor> hyper_join(const Tensor& x, const optional<Tensor>& y, const optional<Tensor>& slots,
+                                      const optional<Tensor>& weights, const optional<Tensor>& choice, int64_t experts,
+                                      const optional<Tensor>& own, const optional<Tensor>& shared, const optional<Tensor>& gate,
+                                      const optional<Tensor>& w_out, const optional<Tensor>& mix, const optional<Tensor>& w_in,
+                                      const Tensor& w_norm, double eps, double scale) {
+  TORCH_CHECK(x.is_cuda() && x.dim() == 3 && x.stride(2) == 1 && x.scalar_type() == at::kFloat, "hyper_join: streams are fp32 [rows, streams, cols]");
+  const int64_t rows = x.size(0), n = x.size(1), cols = x.size(2);
+  auto has = [](const optional<Tensor>& t) { return t.has_value() && t->defined(); };
+  auto param = [&](const optional<Tensor>& t, int64_t numel, const char* what) {
+    TORCH_CHECK(!has(t) || (t->is_contiguous() && t->numel() == numel && t->scalar_type() == w_norm.scalar_type()), what);
+  };
+  auto matrix = [&](const optional<Tensor>& t, int64_t width, const char* what) {
+    if (has(t)) {
+      check_rows(*t, what);
+      TORCH_CHECK(t->size(0) == rows && t->size(1) == width && t->scalar_type() == w_norm.scalar_type(), what);
+    }
+  };
+  TORCH_CHECK(w_norm.is_contiguous() && w_norm.numel() == cols, "hyper_join: norm weight");
+  param(w_in, n, "hyper_join: w_in"); param(w_out, n, "hyper_join: w_out"); param(mix, n * n, "hyper_join: mix");
+  matrix(shared, cols, "hyper_join: shared"); matrix(own, cols, "hyper_join: own rows"); matrix(gate, 1, "hyper_join: gate");
+  TORCH_CHECK(has(shared) == has(gate) && (!has(choice) || has(own)), "hyper_join: operands that belong together");
+  int top = 0;
+  if (has(y)) {
+    check_rows(*y, "y");
+    TORCH_CHECK(has(w_out) && has(mix) && y->size(1) == cols && y->scalar_type() == w_norm.scalar_type(), "hyper_join: result");
+    if (has(weights)) {
+      TORCH_CHECK(weights->is_contiguous() && weights->scalar_type() == at::kFloat && weights->dim() == 2 && weights->size(0) == rows, "hyper_join: weights");
+      top = static_cast<int>(weights->size(1));
+      for (const optional<Tensor>* t : {&slots, &choice})
+        TORCH_CHECK(!has(*t) || ((*t)->is_contiguous() && (*t)->scalar_type() == at::kInt && (*t)->numel() == rows * top), "hyper_join: slots / choices");
+      TORCH_CHECK(has(slots) || y->size(0) == rows * top, "hyper_join: one row of y per (token, choice)");
+    } else {
+      TORCH_CHECK(y->size(0) == rows, "hyper_join: rows of y");
+    }
+  }
+  c10::cuda::CUDAGuard guard(x.device());
+  Tensor xo = at::empty({has(y) ? rows : 0, n, cols}, x.options());
+  Tensor h = at::empty({rows, cols}, w_norm.options());
+  const bool experts_rows = has(y) && has(weights);
+  check_rc(oslo_hyper_join(x.data_ptr<float>(), x.stride(0), x.stride(1), ptr_or_null(y), has(y) ? y->stride(0) : 0,
+                           experts_rows && has(slots) ? slots->data_ptr<int>() : nullptr, experts_rows ? weights->data_ptr<float>() : nullptr,
+                           top, experts_rows && has(choice) ? choice->data_ptr<int>() : nullptr, static_cast<int>(experts),
+                           ptr_or_null(own), has(own) ? own->stride(0) : 0, ptr_or_null(shared), has(shared) ? shared->stride(0) : 0,
+                           ptr_or_null(gate), has(gate) ? gate->stride(0) : 0, ptr_or_null(w_out), ptr_or_null(mix), ptr_or_null(w_in),
+                           w_norm.data_ptr(), has(y) ? xo.data_ptr<float>() : nullptr, h.data_ptr(), rows, static_cast<int>(n),
+                           static_cast<int>(cols), static_cast<float>(eps), static_cast<float>(scale), dt_code(w_norm), cur_stream()),
+           "hyper_join");
+  return {xo, h};
 }
 
 // x [P, M <= 4, K] (rows of a part contiguous in K), w [P, N, K] -> [P, M, N]
@@ -960,6 +1016,88 @@ Tensor bonus_recurrence(const Tensor& q, const Tensor& k, const Tensor& v, const
   return run_recurrence(r, q, k, v, keep, state, batch, heads, dim, vdim, chunks);
 }
 
+void check_state(const Tensor& state, int64_t n);
+
+// z fp32 [B * S, 2 heads] -> read, write, start [B, heads, S], running maximum [B * S, heads]
+std::tuple<Tensor, Tensor, Tensor, Tensor> memory_gates(const Tensor& z, const Tensor& bias, double cap, const optional<Tensor>& keep,
+                                                        optional<Tensor> top, int64_t batch) {
+  check_rows(z, "z");
+  const int64_t H = z.size(1) / 2;
+  TORCH_CHECK(batch > 0 && z.size(0) % batch == 0 && z.size(1) % 2 == 0 && z.scalar_type() == at::kFloat && bias.is_contiguous() &&
+                  bias.numel() == 2 * H && cap > 0.0, "memory_gates: operands");
+  const int64_t S = z.size(0) / batch;
+  const bool has = top.has_value() && top->defined();
+  if (has) check_state(*top, batch * H);
+  int64_t ld_keep = 0;
+  const uint8_t* kp = keep_ptr(keep, batch, S, ld_keep);
+  c10::cuda::CUDAGuard guard(z.device());
+  Tensor rd = at::empty({batch, H, S}, z.options()), wr = at::empty({batch, H, S}, z.options()), st = at::empty({batch, H, S}, z.options());
+  Tensor m = at::empty({batch * S, H}, z.options());
+  check_rc(oslo_memory_gates(z.data_ptr<float>(), z.stride(0), bias.data_ptr(), static_cast<float>(cap), kp, ld_keep,
+                             has ? top->data_ptr<float>() : nullptr, rd.data_ptr<float>(), wr.data_ptr<float>(), st.data_ptr<float>(),
+                             m.data_ptr<float>(), static_cast<int>(batch), static_cast<int>(S), static_cast<int>(H), dt_code(bias),
+                             cur_stream()), "memory_gates");
+  return {rd, wr, st, m};
+}
+
+// S^T q [B * S, heads * vdim] and n . q [B * S, heads], fp32
+std::tuple<Tensor, Tensor> memory_recurrence(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& read, const Tensor& write,
+                                             const Tensor& start, double q_scale, const optional<Tensor>& keep, optional<Tensor> state,
+                                             int64_t batch, int64_t heads, int64_t dim, int64_t vdim, int64_t chunks) {
+  check_qkv_rows(q, k, v, heads, dim, vdim);
+  TORCH_CHECK(batch > 0 && q.size(0) % batch == 0, "memory_recurrence: rows are not batch x positions");
+  const int64_t S = q.size(0) / batch, lds = (vdim + 1 + 3) / 4 * 4;
+  for (const Tensor* t : {&read, &write, &start})
+    TORCH_CHECK(t->is_cuda() && t->is_contiguous() && t->scalar_type() == at::kFloat && t->numel() == batch * heads * S, "memory_recurrence: gates");
+  const bool has = state.has_value() && state->defined();
+  if (has) check_state(*state, batch * heads * dim * lds);
+  int64_t ld_keep = 0;
+  const uint8_t* kp = keep_ptr(keep, batch, S, ld_keep);
+  c10::cuda::CUDAGuard guard(q.device());
+  const int nch = chunks > 0 ? static_cast<int>(chunks)
+                             : oslo_recurrence_chunks(3, static_cast<int>(batch), static_cast<int>(S), static_cast<int>(heads),
+                                                      static_cast<int>(dim), static_cast<int>(vdim), dev_state(q.get_device()).sms);
+  const auto f32 = q.options().dtype(at::kFloat);
+  Tensor out = at::empty({q.size(0), heads * vdim}, f32), norm = at::empty({q.size(0), heads}, f32);
+  Tensor ws, decay;
+  if (nch > 1) {
+    ws = at::empty({batch, nch, heads, dim, lds}, f32);
+    decay = at::empty({batch, nch, heads, dim}, f32);
+  }
+  check_rc(oslo_memory_recurrence(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0),
+                                  read.data_ptr<float>(), write.data_ptr<float>(), start.data_ptr<float>(), static_cast<float>(q_scale),
+                                  kp, ld_keep, has ? state->data_ptr<float>() : nullptr, out.data_ptr<float>(), norm.data_ptr<float>(),
+                                  nch > 1 ? ws.data_ptr<float>() : nullptr, nch > 1 ? decay.data_ptr<float>() : nullptr, nch,
+                                  static_cast<int>(batch), static_cast<int>(S), static_cast<int>(heads), static_cast<int>(dim),
+                                  static_cast<int>(vdim), dt_code(q), cur_stream(nch > 1 ? 3 : 1)), "memory_recurrence");
+  return {out, norm};
+}
+
+Tensor memory_step(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& x, const Tensor& w, const Tensor& bias, double cap,
+                   const Tensor& gate, const Tensor& norm_w, const optional<Tensor>& keep, Tensor state, Tensor top, double q_scale,
+                   double eps, int64_t heads, int64_t dim, int64_t vdim) {
+  check_qkv_rows(q, k, v, heads, dim, vdim);
+  check_rows(x, "x"); check_rows(gate, "gate");
+  const int64_t B = q.size(0);
+  check_state(state, B * heads * dim * ((vdim + 1 + 3) / 4 * 4));
+  check_state(top, B * heads);
+  for (const Tensor* t : {&x, &w, &bias, &gate, &norm_w}) TORCH_CHECK(t->scalar_type() == q.scalar_type(), "memory_step: dtypes");
+  TORCH_CHECK(x.size(0) == B && w.is_contiguous() && w.dim() == 2 && w.size(0) == 2 * heads && w.size(1) == x.size(1) && bias.is_contiguous() &&
+                  bias.numel() == 2 * heads && gate.size(0) == B && gate.size(1) == heads * vdim && norm_w.is_contiguous() &&
+                  norm_w.numel() == heads * vdim && cap > 0.0, "memory_step: operands");
+  int64_t ld_keep = 0;
+  const uint8_t* kp = keep_ptr(keep, B, 1, ld_keep);
+  c10::cuda::CUDAGuard guard(q.device());
+  Tensor out = at::empty({B, heads * vdim}, q.options());
+  check_rc(oslo_memory_step(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), x.data_ptr(), x.stride(0),
+                            static_cast<int>(x.size(1)), w.data_ptr(), bias.data_ptr(), static_cast<float>(cap), gate.data_ptr(),
+                            gate.stride(0), norm_w.data_ptr(), kp, ld_keep, state.data_ptr<float>(), top.data_ptr<float>(), out.data_ptr(),
+                            static_cast<float>(q_scale), static_cast<float>(eps), static_cast<int>(B), static_cast<int>(heads),
+                            static_cast<int>(dim), static_cast<int>(vdim), dev_state(q.get_device()).sms, dt_code(q), cur_stream()),
+           "memory_step");
+  return out;
+}
+
 void check_state(const Tensor& state, int64_t n) {
   TORCH_CHECK(state.is_cuda() && state.is_contiguous() && state.scalar_type() == at::kFloat && state.numel() == n, "state: contiguous fp32 of the right size");
 }
@@ -1041,20 +1179,42 @@ Tensor sink_gate(const Tensor& o, const Tensor& lse, const Tensor& sink, const T
   return out;
 }
 
-// q [B, H, Sq, dim], k [B, G, Sk, dim], v [B, G, Sk, vdim] (any strides that TMA takes, contiguous last dim) -> [B * Sq, H * vdim]
-Tensor flash_sink_fwd(const Tensor& q, const Tensor& k, const Tensor& v, const optional<Tensor>& kpm, const Tensor& sink,
-                      const optional<Tensor>& gate, double scale, double softcap) {
+// the output gate: none, one column per head or one per output column; returns whether it is the latter
+bool check_gate(const optional<Tensor>& gate, int64_t rows, int64_t heads, int64_t vdim, const Tensor& like, const char* what) {
+  if (!(gate.has_value() && gate->defined())) return false;
+  check_rows(*gate, what);
+  TORCH_CHECK(gate->size(0) == rows && (gate->size(1) == heads || gate->size(1) == heads * vdim) && gate->scalar_type() == like.scalar_type(), what);
+  return gate->size(1) != heads;
+}
+const void* sink_ptr(const optional<Tensor>& sink, int64_t heads, const Tensor& like, const char* what) {
+  if (!(sink.has_value() && sink->defined())) return nullptr;
+  TORCH_CHECK(sink->is_contiguous() && sink->numel() == heads && sink->scalar_type() == like.scalar_type(), what);
+  return sink->data_ptr();
+}
+const int* lead_ptr(const optional<Tensor>& lead, int64_t B) {
+  if (!(lead.has_value() && lead->defined())) return nullptr;
+  TORCH_CHECK(lead->is_cuda() && lead->is_contiguous() && lead->scalar_type() == at::kInt && lead->numel() == B, "lead: int32 [batch]");
+  return lead->data_ptr<int>();
+}
+
+// q [B, H, Sq, dim], k [B, G, Sk, dim], v [B, G, Sk, vdim] (any strides that TMA takes, contiguous last dim) -> [B * Sq, H * vdim];
+// q2 [B, H, Sq, rot], k2 [B, Sk, rot]: a part of queries and keys whose keys all heads share
+Tensor flash_sink_fwd(const Tensor& q, const Tensor& k, const Tensor& v, const optional<Tensor>& kpm, const optional<Tensor>& sink,
+                      const optional<Tensor>& gate, double scale, double softcap, int64_t window, int64_t keep_first,
+                      const optional<Tensor>& lead, const optional<Tensor>& q2, const optional<Tensor>& k2) {
   TORCH_CHECK(q.is_cuda() && q.dim() == 4 && k.dim() == 4 && v.dim() == 4 && q.stride(3) == 1 && k.stride(3) == 1 && v.stride(3) == 1 &&
                   k.size(3) == q.size(3) && k.size(0) == q.size(0) && v.size(0) == q.size(0) && v.size(1) == k.size(1) &&
                   v.size(2) == k.size(2) && q.size(1) % k.size(1) == 0 && k.size(2) >= q.size(2), "flash_sink_fwd: q, k, v");
   const int64_t B = q.size(0), H = q.size(1), G = k.size(1), Sq = q.size(2), Sk = k.size(2), dim = q.size(3), vdim = v.size(3);
-  TORCH_CHECK(sink.is_contiguous() && sink.numel() == H && k.scalar_type() == q.scalar_type() && v.scalar_type() == q.scalar_type() &&
-                  sink.scalar_type() == q.scalar_type(), "flash_sink_fwd: operands");
-  const bool gated = gate.has_value() && gate->defined();
-  if (gated) {
-    check_rows(*gate, "gate");
-    TORCH_CHECK(gate->size(0) == B * Sq && gate->size(1) == H && gate->scalar_type() == q.scalar_type(), "flash_sink_fwd: gate");
-  }
+  TORCH_CHECK(k.scalar_type() == q.scalar_type() && v.scalar_type() == q.scalar_type(), "flash_sink_fwd: operands");
+  const void* sp = sink_ptr(sink, H, q, "flash_sink_fwd: sink");
+  const bool wide = check_gate(gate, B * Sq, H, vdim, q, "flash_sink_fwd: gate");
+  const bool gated = gate.has_value() && gate->defined(), parts = q2.has_value() && q2->defined();
+  TORCH_CHECK(window >= 0 && keep_first >= 0 && parts == (k2.has_value() && k2->defined()), "flash_sink_fwd: window / second parts");
+  if (parts)
+    TORCH_CHECK(q2->dim() == 4 && k2->dim() == 3 && q2->stride(3) == 1 && k2->stride(2) == 1 && q2->size(0) == B && q2->size(1) == H &&
+                    q2->size(2) == Sq && k2->size(0) == B && k2->size(1) == Sk && k2->size(2) == q2->size(3) &&
+                    q2->scalar_type() == q.scalar_type() && k2->scalar_type() == q.scalar_type(), "flash_sink_fwd: second parts");
   const uint8_t* kp = nullptr;
   if (kpm.has_value() && kpm->defined()) {
     TORCH_CHECK(kpm->is_contiguous() && kpm->scalar_type() == at::kByte && kpm->numel() == B * Sk, "flash_sink_fwd: mask");
@@ -1062,46 +1222,49 @@ Tensor flash_sink_fwd(const Tensor& q, const Tensor& k, const Tensor& v, const o
   }
   c10::cuda::CUDAGuard guard(q.device());
   Tensor out = at::empty({B * Sq, H * vdim}, q.options());
-  check_rc(oslo_flash_sink_fwd_sm100(q.data_ptr(), k.data_ptr(), v.data_ptr(), out.data_ptr(), kp, sink.data_ptr(),
+  check_rc(oslo_flash_sink_fwd_sm100(q.data_ptr(), k.data_ptr(), v.data_ptr(), out.data_ptr(), kp, sp,
                                      ptr_or_null(gate), gated ? gate->stride(0) : 0, static_cast<int>(B), static_cast<int>(H),
                                      static_cast<int>(G), static_cast<int>(Sq), static_cast<int>(Sk), static_cast<int>(dim),
                                      static_cast<int>(vdim), q.stride(0), q.stride(1), q.stride(2), k.stride(0), k.stride(1),
                                      k.stride(2), v.stride(0), v.stride(1), v.stride(2), Sq * H * vdim, vdim, H * vdim,
-                                     static_cast<float>(scale), static_cast<float>(softcap), dt_code(q),
-                                     dev_state(q.get_device()).err.data_ptr<int>(), cur_stream()), "flash_sink_fwd");
+                                     static_cast<float>(scale), static_cast<float>(softcap), static_cast<int>(window),
+                                     static_cast<int>(keep_first), lead_ptr(lead, B), wide ? 1 : 0, ptr_or_null(q2),
+                                     parts ? q2->stride(0) : 0, parts ? q2->stride(1) : 0, parts ? q2->stride(2) : 0, ptr_or_null(k2),
+                                     parts ? k2->stride(0) : 0, parts ? k2->stride(1) : 0, parts ? static_cast<int>(q2->size(3)) : 0,
+                                     dt_code(q), dev_state(q.get_device()).err.data_ptr<int>(), cur_stream()), "flash_sink_fwd");
   return out;
 }
 
-Tensor sink_attention(const Tensor& q, const Tensor& k, const Tensor& v, const optional<Tensor>& keep, const Tensor& sink,
-                      const optional<Tensor>& gate, double scale, double softcap) {
+Tensor sink_attention(const Tensor& q, const Tensor& k, const Tensor& v, const optional<Tensor>& keep, const optional<Tensor>& sink,
+                      const optional<Tensor>& gate, double scale, double softcap, int64_t window, int64_t keep_first,
+                      const optional<Tensor>& lead) {
   // [B, S, heads, D] views with contiguous D
   TORCH_CHECK(q.is_cuda() && q.dim() == 4 && k.dim() == 4 && v.dim() == 4 && q.stride(3) == 1 && k.stride(3) == 1 && v.stride(3) == 1,
               "sink_attention: q, k, v must be [B, S, H, D] with a contiguous last dim");
   const int64_t B = q.size(0), Sq = q.size(1), H = q.size(2), G = k.size(2), D = q.size(3), Sk = k.size(1), Dv = v.size(3);
   TORCH_CHECK(k.size(0) == B && v.size(0) == B && H % G == 0 && v.size(2) == G && v.size(1) == Sk && k.size(3) == D && Sk >= Sq,
               "sink_attention: sizes");
-  TORCH_CHECK(sink.is_contiguous() && sink.numel() == H && k.scalar_type() == q.scalar_type() && v.scalar_type() == q.scalar_type() &&
-                  sink.scalar_type() == q.scalar_type(), "sink_attention: operands");
+  TORCH_CHECK(k.scalar_type() == q.scalar_type() && v.scalar_type() == q.scalar_type() && window >= 0 && keep_first >= 0,
+              "sink_attention: operands");
+  const void* sp = sink_ptr(sink, H, q, "sink_attention: sink");
+  const bool wide = check_gate(gate, B * Sq, H, Dv, q, "sink_attention: gate");
   const bool gated = gate.has_value() && gate->defined();
-  if (gated) {
-    check_rows(*gate, "gate");
-    TORCH_CHECK(gate->size(0) == B * Sq && gate->size(1) == H && gate->scalar_type() == q.scalar_type(), "sink_attention: gate");
-  }
   int64_t ld_keep = 0;
   const uint8_t* kp = keep_ptr(keep, B, Sk, ld_keep);
   c10::cuda::CUDAGuard guard(q.device());
   Tensor out = at::empty({B * Sq, H * Dv}, q.options());
   check_rc(oslo_sink_attention(q.data_ptr(), q.stride(0), q.stride(1), q.stride(2), k.data_ptr(), k.stride(0), k.stride(1),
-                               k.stride(2), v.data_ptr(), v.stride(0), v.stride(1), v.stride(2), kp, ld_keep, sink.data_ptr(),
+                               k.stride(2), v.data_ptr(), v.stride(0), v.stride(1), v.stride(2), kp, ld_keep, sp,
                                ptr_or_null(gate), gated ? gate->stride(0) : 0, out.data_ptr(), static_cast<int>(B),
                                static_cast<int>(H), static_cast<int>(G), static_cast<int>(Sq), static_cast<int>(Sk),
                                static_cast<int>(D), static_cast<int>(Dv), static_cast<float>(scale), static_cast<float>(softcap),
+                               static_cast<int>(window), static_cast<int>(keep_first), lead_ptr(lead, B), wide ? 1 : 0,
                                dt_code(q), cur_stream()), "sink_attention");
   return out;
 }
 
 // ---------------------------------------------------------------------- grouped-query attention
-Tensor qkv_prep(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& wq, const Tensor& wk, double eps, const Tensor& positions,
+Tensor qkv_prep(const Tensor& q, const Tensor& k, const Tensor& v, const optional<Tensor>& wq, const optional<Tensor>& wk, double eps, const Tensor& positions,
                 const Tensor& freq, Tensor kc, Tensor vc, const Tensor& lengths) {
   check_rows(q, "q"); check_rows(k, "k"); check_rows(v, "v");
   TORCH_CHECK(kc.dim() == 4 && vc.dim() == 4 && kc.is_contiguous() && vc.is_contiguous() && vc.size(0) == kc.size(0) &&
@@ -1112,14 +1275,14 @@ Tensor qkv_prep(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor&
   const int64_t S = q.size(0) / B, H = q.size(1) / dim;
   for (const Tensor* t : {&k, &v, static_cast<const Tensor*>(&kc), static_cast<const Tensor*>(&vc)})
     TORCH_CHECK(t->scalar_type() == q.scalar_type(), "qkv_prep: dtypes");
-  check_channels(wq, dim, q, "qkv_prep: query norm weight");
-  check_channels(wk, dim, q, "qkv_prep: key norm weight");
+  if (ptr_or_null(wq)) check_channels(*wq, dim, q, "qkv_prep: query norm weight");
+  if (ptr_or_null(wk)) check_channels(*wk, dim, q, "qkv_prep: key norm weight");
   TORCH_CHECK(positions.is_cuda() && positions.dim() == 2 && positions.size(0) == B && positions.size(1) == S && positions.scalar_type() == at::kLong, "qkv_prep: positions");
   TORCH_CHECK(freq.is_cuda() && freq.is_contiguous() && freq.scalar_type() == at::kFloat && 2 * freq.numel() <= dim, "qkv_prep: frequencies");
   TORCH_CHECK(lengths.scalar_type() == at::kInt && lengths.is_contiguous() && lengths.numel() == B, "qkv_prep: lengths");
   c10::cuda::CUDAGuard guard(q.device());
   Tensor out = at::empty({B, S, H, dim}, q.options());
-  check_rc(oslo_qkv_prep(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), wq.data_ptr(), wk.data_ptr(),
+  check_rc(oslo_qkv_prep(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), ptr_or_null(wq), ptr_or_null(wk),
                          static_cast<float>(eps), reinterpret_cast<const long long*>(positions.data_ptr<int64_t>()), positions.stride(0),
                          positions.stride(1), freq.numel() ? freq.data_ptr<float>() : nullptr, static_cast<int>(freq.numel()),
                          out.data_ptr(), kc.data_ptr(), vc.data_ptr(), lengths.data_ptr<int>(), static_cast<int>(B),
@@ -1130,27 +1293,35 @@ Tensor qkv_prep(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor&
 }
 
 Tensor grouped_decode(const Tensor& q, const Tensor& kc, const Tensor& vc, const Tensor& lengths, const optional<Tensor>& keep,
-                      const Tensor& sink, double scale, double softcap) {
+                      const optional<Tensor>& sink, double scale, double softcap, const optional<Tensor>& gate, int64_t window,
+                      int64_t keep_first, const optional<Tensor>& lead) {
   TORCH_CHECK(q.is_cuda() && q.dim() == 3 && q.is_contiguous() && kc.dim() == 4 && vc.dim() == 4 && kc.is_contiguous() && vc.is_contiguous() &&
                   vc.size(0) == kc.size(0) && vc.size(1) == kc.size(1) && vc.size(2) == kc.size(2) && kc.size(0) == q.size(0) &&
                   kc.size(3) == q.size(2) && q.size(1) % kc.size(1) == 0, "grouped_decode: q [B, H, dim], caches [B, G, T, *]");
   const int64_t B = q.size(0), H = q.size(1), G = kc.size(1), T = kc.size(2), vdim = vc.size(3);
-  TORCH_CHECK(sink.is_contiguous() && sink.numel() == H && kc.scalar_type() == q.scalar_type() && vc.scalar_type() == q.scalar_type() &&
-                  sink.scalar_type() == q.scalar_type(), "grouped_decode: operands");
+  TORCH_CHECK(kc.scalar_type() == q.scalar_type() && vc.scalar_type() == q.scalar_type() && window >= 0 && keep_first >= 0, "grouped_decode: operands");
+  const void* sp = sink_ptr(sink, H, q, "grouped_decode: sink");
+  const bool gated = gate.has_value() && gate->defined();
+  if (gated) {
+    check_rows(*gate, "gate");
+    TORCH_CHECK(gate->size(0) == B && gate->size(1) == H && gate->scalar_type() == q.scalar_type(), "grouped_decode: gate");
+  }
   TORCH_CHECK(lengths.scalar_type() == at::kInt && lengths.is_contiguous() && lengths.numel() == B, "grouped_decode: lengths");
   int64_t ld_keep = 0;
   const uint8_t* kp = keep_ptr(keep, B, 0, ld_keep);
   c10::cuda::CUDAGuard guard(q.device());
   auto& st = dev_state(q.get_device());
-  const int splits = oslo_grouped_splits(static_cast<int>(B), static_cast<int>(H), static_cast<int>(G), static_cast<int>(T),
+  const int64_t most = window > 0 ? std::min(T, window + keep_first) : T;     // keys a query can see
+  const int splits = oslo_grouped_splits(static_cast<int>(B), static_cast<int>(H), static_cast<int>(G), static_cast<int>(most),
                                          static_cast<int>(q.size(2)), static_cast<int>(vdim), dt_code(q), st.sms);
   const auto f32 = q.options().dtype(at::kFloat);
   Tensor ws = at::empty({B, H, splits, (vdim + 3) / 4 * 4}, f32);
   Tensor stat = at::empty({B, H, splits, 2}, f32);
   Tensor out = at::empty({B, H * vdim}, q.options());
   check_rc(oslo_grouped_decode(q.data_ptr(), kc.data_ptr(), vc.data_ptr(), lengths.data_ptr<int>(), kp, ld_keep,
-                               kp ? static_cast<int>(keep->size(1)) : 0, sink.data_ptr(), ws.data_ptr<float>(), stat.data_ptr<float>(),
-                               out.data_ptr(), static_cast<int>(B), static_cast<int>(H), static_cast<int>(G),
+                               kp ? static_cast<int>(keep->size(1)) : 0, sp, ptr_or_null(gate), gated ? gate->stride(0) : 0,
+                               static_cast<int>(window), static_cast<int>(keep_first), lead_ptr(lead, B), ws.data_ptr<float>(),
+                               stat.data_ptr<float>(), out.data_ptr(), static_cast<int>(B), static_cast<int>(H), static_cast<int>(G),
                                static_cast<int>(q.size(2)), static_cast<int>(vdim), static_cast<int>(T), splits,
                                static_cast<float>(scale), static_cast<float>(softcap), dt_code(q), st.err.data_ptr<int>(),
                                cur_stream(2)), "grouped_decode");
@@ -1259,67 +1430,109 @@ Tensor scan_step(const Tensor& x, const Tensor& dt, const Tensor& w_dt, const Te
   return out;
 }
 
-Tensor latent_prep(const Tensor& cq, const Tensor& wq, const optional<Tensor>& ckv, const optional<Tensor>& wkv,
-                   optional<Tensor> cache, const Tensor& lengths, double eps) {
+// positions int64 [B, S] and frequencies fp32 [rot / 2] of a rotation (rot 0: none are needed)
+struct Turn {
+  const long long* pos = nullptr;
+  int64_t sb = 0, ss = 0;
+  const float* freq = nullptr;
+  Turn(const optional<Tensor>& positions, const optional<Tensor>& freqs, int64_t B, int64_t S, int64_t rot) {
+    if (rot == 0) return;
+    TORCH_CHECK(positions.has_value() && positions->defined() && freqs.has_value() && freqs->defined() && positions->is_cuda() &&
+                    positions->dim() == 2 && positions->size(0) == B && positions->size(1) == S && positions->scalar_type() == at::kLong &&
+                    freqs->is_cuda() && freqs->is_contiguous() && freqs->scalar_type() == at::kFloat && 2 * freqs->numel() == rot,
+                "rotation: positions int64 [batch, S], frequencies fp32 [dims / 2]");
+    pos = reinterpret_cast<const long long*>(positions->data_ptr<int64_t>());
+    sb = positions->stride(0);
+    ss = positions->stride(1);
+    freq = freqs->data_ptr<float>();
+  }
+};
+
+// rows b * S + t; the columns of ckv after wkv's are rotated and cached behind the latent. Returns the normed query latents and
+// (rows) the normed key-value latents
+std::tuple<Tensor, Tensor> latent_prep(const Tensor& cq, const Tensor& wq, const optional<Tensor>& ckv, const optional<Tensor>& wkv,
+                                       optional<Tensor> cache, const Tensor& lengths, double eps, const optional<Tensor>& positions,
+                                       const optional<Tensor>& freq, bool rows) {
   check_rows(cq, "cq");
-  const int64_t B = cq.size(0);
   TORCH_CHECK(wq.is_contiguous() && wq.numel() == cq.size(1) && wq.scalar_type() == cq.scalar_type(), "latent_prep: query norm weight");
-  TORCH_CHECK(lengths.scalar_type() == at::kInt && lengths.is_contiguous() && lengths.numel() == B, "latent_prep: lengths");
+  const int64_t n = cq.size(0), B = lengths.numel();
+  TORCH_CHECK(lengths.scalar_type() == at::kInt && lengths.is_contiguous() && B > 0 && n % B == 0, "latent_prep: lengths");
+  const int64_t S = n / B;
   const bool kv = ckv.has_value() && ckv->defined();
-  int64_t R = 0, T = 0;
+  int64_t R = 0, W = 0, T = 0;
   if (kv) {
     check_rows(*ckv, "ckv");
-    R = ckv->size(1);
-    TORCH_CHECK(wkv.has_value() && wkv->numel() == R && wkv->is_contiguous() && cache.has_value() && cache->dim() == 3 &&
-                    cache->is_contiguous() && cache->size(0) == B && cache->size(2) == R && ckv->size(0) == B &&
-                    cache->scalar_type() == cq.scalar_type() && ckv->scalar_type() == cq.scalar_type() &&
-                    wkv->scalar_type() == cq.scalar_type(), "latent_prep: key-value operands");
+    TORCH_CHECK(wkv.has_value() && wkv->defined() && wkv->is_contiguous() && cache.has_value() && cache->dim() == 3 && cache->is_contiguous(),
+                "latent_prep: key-value operands");
+    R = wkv->numel();
+    W = ckv->size(1);
+    TORCH_CHECK(W >= R && cache->size(0) == B && cache->size(2) == W && ckv->size(0) == n && cache->scalar_type() == cq.scalar_type() &&
+                    ckv->scalar_type() == cq.scalar_type() && wkv->scalar_type() == cq.scalar_type(), "latent_prep: key-value sizes");
     T = cache->size(1);
   }
+  const Turn turn(positions, freq, B, S, W - R);
   c10::cuda::CUDAGuard guard(cq.device());
-  Tensor out = at::empty({B, cq.size(1)}, cq.options());
+  Tensor out = at::empty({n, cq.size(1)}, cq.options());
+  Tensor c = at::empty({kv && rows ? n : 0, R}, cq.options());
   check_rc(oslo_latent_prep(cq.data_ptr(), cq.stride(0), wq.data_ptr(), static_cast<int>(cq.size(1)), out.data_ptr(),
                             ptr_or_null(ckv), kv ? ckv->stride(0) : 0, ptr_or_null(wkv), static_cast<int>(R),
                             kv ? cache->data_ptr() : nullptr, lengths.data_ptr<int>(), static_cast<int>(T),
-                            static_cast<float>(eps), static_cast<int>(B), dt_code(cq),
+                            static_cast<float>(eps), static_cast<int>(B), static_cast<int>(S), static_cast<int>(W - R), turn.pos, turn.sb,
+                            turn.ss, turn.freq, kv && rows ? c.data_ptr() : nullptr, dt_code(cq),
                             dev_state(cq.get_device()).err.data_ptr<int>(), cur_stream()), "latent_prep");
-  return out;
+  return {out, c};
+}
+
+// q [B, S, heads, dim + rot] contiguous: the last rot dims of every head are rotated in place (halves paired)
+Tensor rotate_halves_(Tensor q, const Tensor& positions, const Tensor& freq) {
+  TORCH_CHECK(q.is_cuda() && q.dim() == 4 && q.is_contiguous() && 2 * freq.numel() <= q.size(3), "rotate_halves_: q [B, S, heads, dim]");
+  const int64_t rot = 2 * freq.numel();
+  const Turn turn(positions, freq, q.size(0), q.size(1), rot);
+  c10::cuda::CUDAGuard guard(q.device());
+  check_rc(oslo_rotate_halves(q.data_ptr(), turn.pos, turn.sb, turn.ss, turn.freq, static_cast<int>(q.size(0)), static_cast<int>(q.size(1)),
+                              static_cast<int>(q.size(2)), static_cast<int>(q.size(3) - rot), static_cast<int>(rot), dt_code(q),
+                              cur_stream()), "rotate_halves_");
+  return q;
 }
 
 Tensor latent_decode(const Tensor& q, const Tensor& w_uk, const Tensor& w_uv, const Tensor& cache, const Tensor& lengths,
-                     const optional<Tensor>& keep, const Tensor& sink, const Tensor& gate, double scale, int64_t heads) {
-  check_rows(q, "q"); check_rows(w_uk, "w_uk"); check_rows(w_uv, "w_uv"); check_rows(gate, "gate");
-  TORCH_CHECK(cache.dim() == 3 && cache.is_contiguous(), "latent_decode: cache must be contiguous [B, T, rank]");
-  const int64_t B = q.size(0), R = cache.size(2), T = cache.size(1);
-  TORCH_CHECK(q.size(1) % heads == 0 && w_uk.size(0) == q.size(1) && w_uv.size(0) % heads == 0 && w_uk.size(1) == R &&
-                  w_uv.size(1) == R && cache.size(0) == B && gate.size(0) == B && gate.size(1) == heads && sink.numel() == heads,
-              "latent_decode: sizes");
-  TORCH_CHECK(w_uk.scalar_type() == q.scalar_type() && w_uv.scalar_type() == q.scalar_type() && cache.scalar_type() == q.scalar_type() &&
-                  gate.scalar_type() == q.scalar_type() && sink.scalar_type() == q.scalar_type(), "latent_decode: dtypes");
+                     const optional<Tensor>& keep, const optional<Tensor>& sink, const Tensor& gate, double scale, int64_t heads,
+                     const optional<Tensor>& positions, const optional<Tensor>& freq) {
+  check_rows(q, "q"); check_rows(w_uk, "w_uk"); check_rows(w_uv, "w_uv");
+  TORCH_CHECK(cache.dim() == 3 && cache.is_contiguous(), "latent_decode: cache must be contiguous [B, T, rank + rotated]");
+  const int64_t B = q.size(0), R = w_uk.size(1), rot = cache.size(2) - R, T = cache.size(1);
+  TORCH_CHECK(rot >= 0 && q.size(1) % heads == 0 && w_uk.size(0) == q.size(1) - heads * rot && w_uv.size(0) % heads == 0 &&
+                  w_uv.size(1) == R && cache.size(0) == B, "latent_decode: sizes");
+  TORCH_CHECK(w_uk.scalar_type() == q.scalar_type() && w_uv.scalar_type() == q.scalar_type() && cache.scalar_type() == q.scalar_type(),
+              "latent_decode: dtypes");
   TORCH_CHECK(lengths.scalar_type() == at::kInt && lengths.is_contiguous() && lengths.numel() == B, "latent_decode: lengths");
   int64_t ld_keep = 0;
   const uint8_t* kp = keep_ptr(keep, B, 0, ld_keep);
-  const int64_t dim = q.size(1) / heads, vdim = w_uv.size(0) / heads;
+  const int64_t dim = q.size(1) / heads - rot, vdim = w_uv.size(0) / heads;
+  const void* sp = sink_ptr(sink, heads, q, "latent_decode: sink");
+  const bool wide = check_gate(gate, B, heads, vdim, q, "latent_decode: gate");
+  const Turn turn(positions, freq, B, 1, rot);
   c10::cuda::CUDAGuard guard(q.device());
   auto& st = dev_state(q.get_device());
   const int splits = oslo_latent_splits(static_cast<int>(B), static_cast<int>(heads), static_cast<int>(T), st.sms);
   const auto f32 = q.options().dtype(at::kFloat);
-  Tensor qa = at::empty({B, heads, R}, f32);
+  Tensor qa = at::empty({B, heads, R + rot}, f32);
   Tensor ws = at::empty({B, heads, splits, (R + 3) / 4 * 4}, f32);
   Tensor stat = at::empty({B, heads, splits, 2}, f32);
   Tensor out = at::empty({B, heads * vdim}, q.options());
   check_rc(oslo_latent_decode(q.data_ptr(), q.stride(0), w_uk.data_ptr(), w_uk.stride(0), w_uv.data_ptr(), w_uv.stride(0),
                               cache.data_ptr(), lengths.data_ptr<int>(), kp, ld_keep, kp ? static_cast<int>(keep->size(1)) : 0,
-                              sink.data_ptr(), gate.data_ptr(), gate.stride(0), qa.data_ptr<float>(), ws.data_ptr<float>(),
+                              sp, gate.data_ptr(), gate.stride(0), qa.data_ptr<float>(), ws.data_ptr<float>(),
                               stat.data_ptr<float>(), out.data_ptr(), static_cast<int>(B), static_cast<int>(heads), static_cast<int>(dim),
-                              static_cast<int>(vdim), static_cast<int>(R), static_cast<int>(T), splits,
-                              static_cast<float>(scale), st.sms, dt_code(q), st.err.data_ptr<int>(), cur_stream(3)),
-           "latent_decode");
+                              static_cast<int>(vdim), static_cast<int>(R), static_cast<int>(rot), turn.pos, turn.sb, turn.freq,
+                              wide ? 1 : 0, static_cast<int>(T), splits, static_cast<float>(scale), st.sms, dt_code(q),
+                              st.err.data_ptr<int>(), cur_stream(3)), "latent_decode");
   return out;
 }
 
 // ---------------------------------------------------------------------- mixture of experts
-std::tuple<Tensor, Tensor> moe_route(const Tensor& h, const Tensor& w, const Tensor& bias, const optional<Tensor>& logits, int64_t top) {
+std::tuple<Tensor, Tensor> moe_route(const Tensor& h, const Tensor& w, const Tensor& bias, const optional<Tensor>& logits, int64_t top,
+                                     bool scored) {
   check_rows(h, "h");
   TORCH_CHECK(w.dim() == 2 && w.is_contiguous() && w.size(1) == h.size(1) && bias.numel() == w.size(0) &&
                   w.scalar_type() == h.scalar_type() && bias.scalar_type() == h.scalar_type(), "moe_route: router");
@@ -1333,8 +1546,8 @@ std::tuple<Tensor, Tensor> moe_route(const Tensor& h, const Tensor& w, const Ten
   Tensor idx = at::empty({n, top}, h.options().dtype(at::kInt));
   Tensor wgt = at::empty({n, top}, h.options().dtype(at::kFloat));
   check_rc(oslo_moe_route(h.data_ptr(), h.stride(0), w.data_ptr(), bias.data_ptr(), lg, idx.data_ptr<int>(), wgt.data_ptr<float>(),
-                          n, static_cast<int>(E), static_cast<int>(h.size(1)), static_cast<int>(top), dt_code(h), cur_stream()),
-           "moe_route");
+                          n, static_cast<int>(E), static_cast<int>(h.size(1)), static_cast<int>(top), scored ? 1 : 0, dt_code(h),
+                          cur_stream()), "moe_route");
   return {idx, wgt};
 }
 
@@ -1356,39 +1569,43 @@ std::tuple<Tensor, Tensor, Tensor, Tensor> moe_plan(const Tensor& h, const Tenso
   return {slots, rows, tg, nt};
 }
 
-// act(rows . w[expert of the tile]^T): [slots, N]; tcgen05 for 16-bit types with K % 8 == 0 and N % 8 == 0
-Tensor moe_grouped(const Tensor& rows, const Tensor& w, const Tensor& tile_group, const Tensor& n_tiles, bool relu2) {
+// unit(rows . w[expert of the tile]^T): [slots, N], or [slots, N / 2] for unit 2 (silu(gate) * up of column pairs); tcgen05 for
+// 16-bit types with K % 8 == 0 and 16-byte result rows
+Tensor moe_grouped(const Tensor& rows, const Tensor& w, const Tensor& tile_group, const Tensor& n_tiles, int64_t unit) {
   TORCH_CHECK(rows.is_cuda() && rows.dim() == 2 && rows.is_contiguous() && w.dim() == 3 && w.is_contiguous() &&
                   w.size(2) == rows.size(1) && w.scalar_type() == rows.scalar_type(), "moe_grouped: operands");
   TORCH_CHECK(tile_group.scalar_type() == at::kInt && tile_group.numel() * 128 == rows.size(0) && n_tiles.scalar_type() == at::kInt,
               "moe_grouped: plan");
-  const int64_t N = w.size(1), K = w.size(2);
+  const int64_t N = w.size(1), K = w.size(2), cols = unit == 2 ? N / 2 : N;
+  TORCH_CHECK(unit >= 0 && unit <= 2 && (unit != 2 || N % 2 == 0), "moe_grouped: unit");
   c10::cuda::CUDAGuard guard(rows.device());
   auto& st = dev_state(rows.get_device());
-  Tensor out = at::empty({rows.size(0), N}, rows.options());
-  if (rows.scalar_type() != at::kFloat && K % 8 == 0 && N % 8 == 0 && reinterpret_cast<uintptr_t>(w.data_ptr()) % 16 == 0) {
-    const int fl = (relu2 ? GEMM_FLAG_RELU2 : 0) | (rows.scalar_type() == at::kHalf ? GEMM_FLAG_FP16 : 0);
+  Tensor out = at::empty({rows.size(0), cols}, rows.options());
+  if (rows.scalar_type() != at::kFloat && K % 8 == 0 && cols % 8 == 0 && reinterpret_cast<uintptr_t>(w.data_ptr()) % 16 == 0) {
+    const int fl = (unit == 1 ? GEMM_FLAG_RELU2 : 0) | (unit == 2 ? GEMM_FLAG_GLU : 0) | (rows.scalar_type() == at::kHalf ? GEMM_FLAG_FP16 : 0);
     check_rc(oslo_gemm_grouped(rows.data_ptr(), w.data_ptr(), out.data_ptr(), static_cast<int>(rows.size(0)), static_cast<int>(N),
                                static_cast<int>(K), static_cast<int>(w.size(0)), tile_group.data_ptr<int>(),
                                n_tiles.data_ptr<int>(), fl, st.err.data_ptr<int>(), usable_sms(st), cur_stream()), "gemm_grouped");
   } else {
     check_rc(oslo_moe_grouped(rows.data_ptr(), w.data_ptr(), out.data_ptr(), tile_group.data_ptr<int>(), n_tiles.data_ptr<int>(),
-                              static_cast<int>(tile_group.numel()), static_cast<int>(N), static_cast<int>(K), relu2, dt_code(rows),
-                              cur_stream()), "moe_grouped");
+                              static_cast<int>(tile_group.numel()), static_cast<int>(N), static_cast<int>(K), static_cast<int>(unit),
+                              dt_code(rows), cur_stream()), "moe_grouped");
   }
   return out;
 }
 
-// one row of the result per (row, choice): act(w[idx] . x[row]); x has one row per `per_row` entries of idx
-Tensor moe_few(const Tensor& x, const Tensor& idx, const Tensor& w, int64_t per_row, bool relu2) {
+// one row of the result per (row, choice): unit(w[idx] . x[row]); x has one row per `per_row` entries of idx; rows of entries that are
+// no expert (>= w.size(0)) are not written
+Tensor moe_few(const Tensor& x, const Tensor& idx, const Tensor& w, int64_t per_row, int64_t unit) {
   check_rows(x, "x");
   TORCH_CHECK(w.dim() == 3 && w.is_contiguous() && w.size(2) == x.size(1) && w.scalar_type() == x.scalar_type(), "moe_few: weights");
   TORCH_CHECK(idx.is_contiguous() && idx.scalar_type() == at::kInt && idx.numel() == x.size(0) * per_row, "moe_few: idx");
+  TORCH_CHECK(unit >= 0 && unit <= 2 && (unit != 2 || w.size(1) % 2 == 0), "moe_few: unit");
   c10::cuda::CUDAGuard guard(x.device());
-  Tensor out = at::empty({idx.numel(), w.size(1)}, x.options());
+  Tensor out = at::empty({idx.numel(), unit == 2 ? w.size(1) / 2 : w.size(1)}, x.options());
   check_rc(oslo_moe_few(x.data_ptr(), x.stride(0), idx.data_ptr<int>(), w.data_ptr(), out.data_ptr(), static_cast<int>(idx.numel()),
-                        static_cast<int>(per_row), static_cast<int>(w.size(1)), static_cast<int>(w.size(2)), relu2, dt_code(x),
-                        cur_stream()), "moe_few");
+                        static_cast<int>(per_row), static_cast<int>(w.size(1)), static_cast<int>(w.size(2)), static_cast<int>(unit),
+                        static_cast<int>(w.size(0)), dt_code(x), cur_stream()), "moe_few");
   return out;
 }
 
@@ -1440,24 +1657,29 @@ TORCH_LIBRARY(oslo_b200, m) {
   m.def("recurrence(Tensor q, Tensor f, Tensor v, Tensor f_bias, Tensor lower, Tensor? keep, Tensor(a!)? state, int batch, int heads, int dim, int vdim, int chunks=0) -> Tensor");
   m.def("recurrence_step(Tensor q, Tensor f, Tensor v, Tensor f_bias, Tensor lower, Tensor norm_w, Tensor? keep, Tensor(a!) state, float eps, int heads, int dim, int vdim) -> Tensor");
   m.def("sink_gate(Tensor o, Tensor lse, Tensor sink, Tensor gate, int vdim) -> Tensor");
-  m.def("flash_sink_fwd(Tensor q, Tensor k, Tensor v, Tensor? kpm, Tensor sink, Tensor? gate, float scale, float softcap) -> Tensor");
-  m.def("sink_attention(Tensor q, Tensor k, Tensor v, Tensor? keep, Tensor sink, Tensor? gate, float scale, float softcap) -> Tensor");
-  m.def("latent_prep(Tensor cq, Tensor wq, Tensor? ckv, Tensor? wkv, Tensor(a!)? cache, Tensor lengths, float eps) -> Tensor");
-  m.def("latent_decode(Tensor q, Tensor w_uk, Tensor w_uv, Tensor cache, Tensor lengths, Tensor? keep, Tensor sink, Tensor gate, float scale, int heads) -> Tensor");
-  m.def("moe_route(Tensor h, Tensor w, Tensor bias, Tensor? logits, int top) -> (Tensor, Tensor)");
+  m.def("flash_sink_fwd(Tensor q, Tensor k, Tensor v, Tensor? kpm, Tensor? sink, Tensor? gate, float scale, float softcap, int window=0, int keep_first=0, Tensor? lead=None, Tensor? q2=None, Tensor? k2=None) -> Tensor");
+  m.def("sink_attention(Tensor q, Tensor k, Tensor v, Tensor? keep, Tensor? sink, Tensor? gate, float scale, float softcap, int window=0, int keep_first=0, Tensor? lead=None) -> Tensor");
+  m.def("latent_prep(Tensor cq, Tensor wq, Tensor? ckv, Tensor? wkv, Tensor(a!)? cache, Tensor lengths, float eps, Tensor? positions=None, Tensor? freq=None, bool rows=False) -> (Tensor, Tensor)");
+  m.def("rotate_halves_(Tensor(a!) q, Tensor positions, Tensor freq) -> Tensor(a!)");
+  m.def("latent_decode(Tensor q, Tensor w_uk, Tensor w_uv, Tensor cache, Tensor lengths, Tensor? keep, Tensor? sink, Tensor gate, float scale, int heads, Tensor? positions=None, Tensor? freq=None) -> Tensor");
+  m.def("moe_route(Tensor h, Tensor w, Tensor bias, Tensor? logits, int top, bool scored=False) -> (Tensor, Tensor)");
   m.def("moe_plan(Tensor h, Tensor idx, int experts) -> (Tensor, Tensor, Tensor, Tensor)");
-  m.def("moe_grouped(Tensor rows, Tensor w, Tensor tile_group, Tensor n_tiles, bool relu2) -> Tensor");
-  m.def("moe_few(Tensor x, Tensor idx, Tensor w, int per_row, bool relu2) -> Tensor");
+  m.def("moe_grouped(Tensor rows, Tensor w, Tensor tile_group, Tensor n_tiles, int unit) -> Tensor");
+  m.def("moe_few(Tensor x, Tensor idx, Tensor w, int per_row, int unit) -> Tensor");
   m.def("clamped_glu(Tensor gate, Tensor up, float limit, float alpha) -> Tensor");
   m.def("branch_join(Tensor x, Tensor y0, Tensor? n0, float f0, Tensor? y1, Tensor? n1, float f1, Tensor? y2, Tensor? n2, float f2, float mult, float eps, Tensor? w1, Tensor? w2) -> (Tensor, Tensor, Tensor)");
-  m.def("gated_rms_norm(Tensor o, Tensor w, Tensor gate, float eps, int group, int act) -> Tensor");
+  m.def("gated_rms_norm(Tensor o, Tensor w, Tensor gate, float eps, int group, int act, Tensor? z=None, Tensor? m=None) -> Tensor");
+  m.def("hyper_join(Tensor x, Tensor? y, Tensor? slots, Tensor? weights, Tensor? choice, int experts, Tensor? own, Tensor? shared, Tensor? gate, Tensor? w_out, Tensor? mix, Tensor? w_in, Tensor w_norm, float eps, float scale) -> (Tensor, Tensor)");
+  m.def("memory_gates(Tensor z, Tensor bias, float cap, Tensor? keep, Tensor(a!)? top, int batch) -> (Tensor, Tensor, Tensor, Tensor)");
+  m.def("memory_recurrence(Tensor q, Tensor k, Tensor v, Tensor read, Tensor write, Tensor start, float q_scale, Tensor? keep, Tensor(a!)? state, int batch, int heads, int dim, int vdim, int chunks=0) -> (Tensor, Tensor)");
+  m.def("memory_step(Tensor q, Tensor k, Tensor v, Tensor x, Tensor w, Tensor bias, float cap, Tensor gate, Tensor norm_w, Tensor? keep, Tensor(a!) state, Tensor(b!) top, float q_scale, float eps, int heads, int dim, int vdim) -> Tensor");
   m.def("gemv_stacked(Tensor x, Tensor w) -> Tensor");
   m.def("decayed_recurrence(Tensor q, Tensor k, Tensor v, Tensor decay, Tensor? keep, Tensor(a!)? state, int batch, int heads, int dim, int vdim, int chunks=0) -> Tensor");
   m.def("bonus_recurrence(Tensor q, Tensor k, Tensor v, Tensor z, Tensor w0, Tensor u, Tensor? keep, Tensor(a!)? state, int batch, int heads, int dim, int vdim, int chunks=0) -> Tensor");
   m.def("decayed_step(Tensor q, Tensor k, Tensor v, Tensor decay, Tensor? keep, Tensor(a!) state, int heads, int dim, int vdim) -> Tensor");
   m.def("bonus_step(Tensor r, Tensor k, Tensor v, Tensor t, Tensor w2, Tensor w0, Tensor u, Tensor norm_w, Tensor gate, Tensor? keep, Tensor(a!) state, float eps, int heads, int dim, int vdim) -> Tensor");
-  m.def("qkv_prep(Tensor q, Tensor k, Tensor v, Tensor wq, Tensor wk, float eps, Tensor positions, Tensor freq, Tensor(a!) kc, Tensor(b!) vc, Tensor lengths) -> Tensor");
-  m.def("grouped_decode(Tensor q, Tensor kc, Tensor vc, Tensor lengths, Tensor? keep, Tensor sink, float scale, float softcap) -> Tensor");
+  m.def("qkv_prep(Tensor q, Tensor k, Tensor v, Tensor? wq, Tensor? wk, float eps, Tensor positions, Tensor freq, Tensor(a!) kc, Tensor(b!) vc, Tensor lengths) -> Tensor");
+  m.def("grouped_decode(Tensor q, Tensor kc, Tensor vc, Tensor lengths, Tensor? keep, Tensor? sink, float scale, float softcap, Tensor? gate=None, int window=0, int keep_first=0, Tensor? lead=None) -> Tensor");
   m.def("token_shift(Tensor h, Tensor mu, int batch, Tensor? keep, Tensor(a!)? prev) -> Tensor");
   m.def("causal_conv_silu(Tensor x, Tensor w, Tensor bias, int batch, Tensor? keep, Tensor(a!)? prev) -> Tensor");
   m.def("selective_scan(Tensor x, Tensor dt, Tensor dt_bias, Tensor a_log, Tensor b, Tensor c, Tensor d, Tensor z, int batch, Tensor? keep, Tensor(a!)? state, int chunks=0) -> Tensor");
@@ -1508,6 +1730,11 @@ TORCH_LIBRARY_IMPL(oslo_b200, CUDA, m) {
   m.impl("flash_sink_fwd", &flash_sink_fwd);
   m.impl("sink_attention", &sink_attention);
   m.impl("latent_prep", &latent_prep);
+  m.impl("rotate_halves_", &rotate_halves_);
+  m.impl("hyper_join", &hyper_join);
+  m.impl("memory_gates", &memory_gates);
+  m.impl("memory_recurrence", &memory_recurrence);
+  m.impl("memory_step", &memory_step);
   m.impl("latent_decode", &latent_decode);
   m.impl("moe_route", &moe_route);
   m.impl("moe_plan", &moe_plan);

@@ -342,6 +342,23 @@ __device__ __forceinline__ void epilogue_chunk(const GemmParams& p, int row, int
         v[i] = x * x;
       }
     }
+    if (p.flags & GEMM_FLAG_GLU) {   // 16-bit output, no further epilogue
+      uint16_t* d = reinterpret_cast<uint16_t*>(p.D) + static_cast<size_t>(row) * p.ldd + col0 / 2;
+#pragma unroll
+      for (int i = 0; i < 16; ++i) v[i] = __fdividef(v[2 * i], 1.f + __expf(-v[2 * i])) * v[2 * i + 1];
+      if (vec) {
+#pragma unroll
+        for (int i = 0; i < 16; i += 8) {
+          uint4 o;
+          o.x = pack2(v[i], v[i + 1], fp16); o.y = pack2(v[i + 2], v[i + 3], fp16);
+          o.z = pack2(v[i + 4], v[i + 5], fp16); o.w = pack2(v[i + 6], v[i + 7], fp16);
+          *reinterpret_cast<uint4*>(d + i) = o;
+        }
+      } else {
+        _Pragma("unroll") for (int i = 0; i < 16; ++i) if (i < ncols / 2) d[i] = static_cast<uint16_t>(pack2(v[i], 0.f, fp16) & 0xffff);
+      }
+      return;
+    }
     if (p.flags & GEMM_FLAG_DGELU) {
       const uint16_t* z = reinterpret_cast<const uint16_t*>(p.aux) + static_cast<size_t>(row) * p.ld_aux + col0;
       if (vec) {

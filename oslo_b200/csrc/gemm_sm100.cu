@@ -155,7 +155,7 @@ extern "C" int oslo_gemm_16bit(const void* A, const void* B, void* D, int M, int
                                cudaStream_t stream) {
   using namespace oslo;
   if (M <= 0 || N <= 0 || K <= 0) return -1;
-  if (flags & (GEMM_FLAG_CE_STATS | GEMM_FLAG_CE_GRAD)) return -7;   // those epilogues come through oslo_gemm_ce_16bit
+  if (flags & (GEMM_FLAG_CE_STATS | GEMM_FLAG_CE_GRAD | GEMM_FLAG_GLU)) return -7;   // those epilogues come through oslo_gemm_ce_16bit
   GemmParams p;
   p.D = D; p.bias = bias; p.aux = aux; p.aux_out = aux_out;
   p.M = M; p.N = N; p.K = K; p.ldd = ldd; p.ld_aux = ld_aux; p.ld_aux_out = ld_aux_out;
@@ -254,7 +254,9 @@ extern "C" int oslo_gemm_grouped(const void* A, const void* B, void* D, int M, i
                                  const int* group_tiles, int flags, int* err_word, int num_sms, cudaStream_t stream) {
   using namespace oslo;
   if (M <= 0 || N <= 0 || K <= 0 || M % BM || groups <= 0 || group_of_tile == nullptr || group_tiles == nullptr) return -1;
-  if (flags & ~(GEMM_FLAG_RELU2 | GEMM_FLAG_FP16 | GEMM_FLAG_OUT_FP32)) return -7;
+  if (flags & ~(GEMM_FLAG_RELU2 | GEMM_FLAG_GLU | GEMM_FLAG_FP16 | GEMM_FLAG_OUT_FP32)) return -7;
+  const bool glu = (flags & GEMM_FLAG_GLU) != 0;
+  if (glu && (N % 16 || (flags & (GEMM_FLAG_RELU2 | GEMM_FLAG_OUT_FP32)))) return -7;   // 16-byte output rows
   static thread_local bool ctx_bound = false;
   if (!ctx_bound) { cudaFree(nullptr); ctx_bound = true; }
   const bool fp16 = (flags & GEMM_FLAG_FP16) != 0;
@@ -266,7 +268,7 @@ extern "C" int oslo_gemm_grouped(const void* A, const void* B, void* D, int M, i
   if (rc) return rc - 1000;
   GemmParams p;
   p.D = D; p.bias = nullptr; p.aux = nullptr; p.aux_out = nullptr;
-  p.M = M; p.N = N; p.K = K; p.ldd = N; p.ld_aux = 0; p.ld_aux_out = 0;
+  p.M = M; p.N = N; p.K = K; p.ldd = glu ? N / 2 : N; p.ld_aux = 0; p.ld_aux_out = 0;
   p.a_mn_major = 0; p.b_mn_major = 0; p.flags = flags; p.alpha = 1.f; p.err = err_word;
   p.group_of_tile = group_of_tile; p.group_tiles = group_tiles;
   p.comm = CommParams{};

@@ -1,10 +1,11 @@
-// Grouped-query attention with query / key norms, interleaved rotation, capped scores and a sink in the denominator:
+// Grouped-query attention with query / key norms, interleaved rotation, capped scores, a sink in the denominator, a window that
+// keeps the first keys and an output gate per head:
 // what comes before the scores (qkv_prep_kernel) and decoding with one query per row (grouped_decode_kernel). Prompts run
 // on the tcgen05 flash kernel (attention_sm100.cu) or, in 32-bit, on sink_attention_kernel (latent_attention.cu).
 //
 // Decode: a block scans a slice of one key / value head's cache for the query heads that share it (up to 16 on tensor cores,
-// 8 in the 32-bit version), so every cached byte is read once per block; grouped_finish_kernel merges the slices and adds the
-// sink to the denominator.
+// 8 in the 32-bit version), so every cached byte is read once per block; grouped_finish_kernel merges the slices, adds the
+// sink to the denominator and gates. With a window the slices run over the visible keys only (KeyRun).
 #include <math_constants.h>
 
 #include <algorithm>
@@ -18,7 +19,7 @@ namespace oslo {
 // ------------------------------------------------------------------ norms, rotation, cache append
 struct PrepParams {
   const void *q, *k, *v; long long ldq, ldk, ldv;     // row b * S + t
-  const void *wq, *wk;                                // [dim]
+  const void *wq, *wk;                                // [dim], or nullptr: norms without a weight
   const long long* pos; long long pos_sb, pos_ss;
   const float* freq; int n_freq;
   void *q_out, *kc, *vc;                              // [B, S, H, dim], [B, G, Tmax, dim], [B, G, Tmax, vdim]
@@ -82,8 +83,8 @@ __global__ void __launch_bounds__(256) qkv_prep_kernel(const PrepParams p) {
       for (int u = 0; u < 2; ++u) {
         const int c = 4 * (lane + 32 * u);
         if (c >= p.dim) break;
-        float g[4];
-        load_vec<T, 4>(w + c, g);
+        float g[4] = {1.f, 1.f, 1.f, 1.f};
+        if (w != nullptr) load_vec<T, 4>(w + c, g);
 #pragma unroll
         for (int i = 0; i < 4; ++i) x[u][i] *= r * g[i];
 #pragma unroll
@@ -108,8 +109,8 @@ __global__ void __launch_bounds__(256) qkv_prep_kernel(const PrepParams p) {
   const float r = 1.0f / sqrtf(warp_sum(ss) / p.dim + p.eps);
   for (int c = 2 * lane; c < p.dim; c += 64) {         // the pair (c, c + 1)
     const bool two = c + 1 < p.dim;
-    float x = Num<T>::to(src[c]) * r * Num<T>::to(w[c]);
-    float y = two ? Num<T>::to(src[c + 1]) * r * Num<T>::to(w[c + 1]) : 0.f;
+    float x = Num<T>::to(src[c]) * r * (w ? Num<T>::to(w[c]) : 1.f);
+    float y = two ? Num<T>::to(src[c + 1]) * r * (w ? Num<T>::to(w[c + 1]) : 1.f) : 0.f;
     if ((c >> 1) < p.n_freq) {
       float sn, cs;
       sincosf(at * p.freq[c >> 1], &sn, &cs);
@@ -132,7 +133,26 @@ struct GroupedParams {
   float* stat;                         // [B, H, splits, 2]: max, sum p
   int H, G, dim, vdim, ldw, Tmax, splits;
   float scale, softcap;
+  int window, keep_first;              // window > 0: the last `window` positions, and the first keep_first after lead[b]
+  const int* lead;                     // [B] padding ahead of the sequence, or nullptr
   int* err;
+};
+
+// the positions a query reads, as one run of `n` indices: `head` of them from `first`, the others up to the sequence's end
+struct KeyRun {
+  int first, head, jump, n;
+  __device__ __forceinline__ KeyRun(const GroupedParams& p, int b, int len) {
+    if (p.window <= 0 || p.window >= len) {
+      first = 0; head = n = len; jump = 0;
+      return;
+    }
+    const int tail = len - p.window;
+    first = p.lead ? max(0, min(p.lead[b], tail)) : 0;
+    head = min(p.keep_first, tail - first);
+    jump = tail - (first + head);
+    n = head + p.window;
+  }
+  __device__ __forceinline__ int at(int i) const { return first + i + (i >= head ? jump : 0); }
 };
 
 constexpr int GD_HEADS = 8, GD_KEYS = 32, GD_MAX_SPLITS = 128;
@@ -154,8 +174,9 @@ __global__ void __launch_bounds__(256) grouped_decode_kernel(const GroupedParams
     if (tid == 0) OSLO_REPORT_BOUNDS(p.err);
     len = len < 0 ? 0 : p.Tmax;
   }
-  const int span = (len + p.splits - 1) / p.splits;
-  const int t0 = sp * span, t1 = min(len, t0 + span);
+  const KeyRun run(p, b, len);
+  const int span = (run.n + p.splits - 1) / p.splits;
+  const int t0 = sp * span, t1 = min(run.n, t0 + span);
   const T* q = static_cast<const T*>(p.q) + (static_cast<long long>(b) * p.H + h0) * p.dim;
   for (int e = tid; e < GD_HEADS * p.dim; e += 256) {
     const int a = e / p.dim, c = e - a * p.dim;
@@ -174,17 +195,19 @@ __global__ void __launch_bounds__(256) grouped_decode_kernel(const GroupedParams
     __syncthreads();
     for (int e = tid; e < GD_KEYS * p.dim; e += 256) {
       const int t = e / p.dim, c = e - t * p.dim;
-      ks[t * dp + c] = t < n ? Num<T>::to(kb[static_cast<long long>(k0) * p.dim + e]) : 0.f;
+      ks[t * dp + c] = t < n ? Num<T>::to(kb[static_cast<long long>(run.at(k0 + t)) * p.dim + c]) : 0.f;
     }
-    for (int e = tid; e < GD_KEYS * p.vdim; e += 256)
-      vs[e] = e < n * p.vdim ? Num<T>::to(vb[static_cast<long long>(k0) * p.vdim + e]) : 0.f;
+    for (int e = tid; e < GD_KEYS * p.vdim; e += 256) {
+      const int t = e / p.vdim, c = e - t * p.vdim;
+      vs[e] = t < n ? Num<T>::to(vb[static_cast<long long>(run.at(k0 + t)) * p.vdim + c]) : 0.f;
+    }
     __syncthreads();
     {
       const int a = tid >> 5, t = tid & 31;              // warp = head, lane = key
       float d = 0.f;
       for (int c = 0; c < p.dim; ++c) d = fmaf(qs[a * dp + c], ks[t * dp + c], d);
       if (p.softcap > 0.f) d = p.softcap * tanhf(d / p.softcap);
-      const int pos = k0 + t;
+      const int pos = run.at(k0 + t);
       const bool vis = t < n && (p.keep == nullptr || pos >= p.n_keep || p.keep[b * p.ld_keep + pos]);
       d = vis ? d : -CUDART_INF_F;
       float mx = d;
@@ -294,8 +317,9 @@ __global__ void __launch_bounds__(128) grouped_decode_mma_kernel(const GroupedPa
     if (tid == 0) OSLO_REPORT_BOUNDS(p.err);
     len = len < 0 ? 0 : p.Tmax;
   }
-  const int span = (len + p.splits - 1) / p.splits;
-  const int t0 = sp * span, t1 = min(len, t0 + span);
+  const KeyRun run(p, b, len);
+  const int span = (run.n + p.splits - 1) / p.splits;
+  const int t0 = sp * span, t1 = min(run.n, t0 + span);
   const T* kb = static_cast<const T*>(p.kc) + (static_cast<long long>(b) * p.G + g) * p.Tmax * p.dim;
   const T* vb = static_cast<const T*>(p.vc) + (static_cast<long long>(b) * p.G + g) * p.Tmax * p.vdim;
   // columns past the head sizes are zero for good: the copies below never write them
@@ -314,7 +338,7 @@ __global__ void __launch_bounds__(128) grouped_decode_mma_kernel(const GroupedPa
       const bool ok = k0 + t < t1;
       const uint32_t d32 = smem_u32(dst + t * PITCH + c);
       const int bytes = ok ? 16 : 0;         // 0: the 16 bytes are filled with zeros
-      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d32), "l"(src + static_cast<long long>(ok ? k0 + t : t0) * width + c), "r"(bytes) : "memory");
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d32), "l"(src + static_cast<long long>(run.at(ok ? k0 + t : t0)) * width + c), "r"(bytes) : "memory");
     }
   };
   const int k_rows = 128 / (p.dim / 8), k_first = tid / (p.dim / 8), k_col = tid % (p.dim / 8) * 8;
@@ -355,8 +379,8 @@ __global__ void __launch_bounds__(128) grouped_decode_mma_kernel(const GroupedPa
     for (int nt = 0; nt < 2; ++nt) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const int pos = k0 + w * 16 + nt * 8 + (l & 3) * 2 + (e & 1);
-        const bool vis = pos < t1 && (p.keep == nullptr || pos >= p.n_keep || p.keep[b * p.ld_keep + pos]);
+        const int i = k0 + w * 16 + nt * 8 + (l & 3) * 2 + (e & 1), pos = run.at(i);
+        const bool vis = i < t1 && (p.keep == nullptr || pos >= p.n_keep || p.keep[b * p.ld_keep + pos]);
         float d = c[nt][e] * scale;                    // capped: twice the score over the cap, in log2 units
         if (p.softcap > 0.f) d = cap - __fdividef(2.f * cap, gd_exp2(d) + 1.f);   // cap * tanh(score / cap)
         c[nt][e] = vis ? d : -CUDART_INF_F;
@@ -430,15 +454,15 @@ __global__ void __launch_bounds__(128) grouped_decode_mma_kernel(const GroupedPa
   }
 }
 
-// block = (head, row): merge the slices; exp(sink) joins the denominator
+// block = (head, row): merge the slices; exp(sink) joins the denominator (sink null: nothing does)
 template <typename T>
 __global__ void __launch_bounds__(128) grouped_finish_kernel(const float* __restrict__ ws, const float* __restrict__ stat,
-                                                             const T* __restrict__ sink, T* __restrict__ out, int H, int vdim,
-                                                             int ldw, int splits) {
+                                                             const T* __restrict__ sink, const T* __restrict__ gate, long long ldg,
+                                                             T* __restrict__ out, int H, int vdim, int ldw, int splits) {
   __shared__ float red[4], fac[GD_MAX_SPLITS];
   const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x;
   const long long at = (static_cast<long long>(b) * H + h) * splits;
-  const float snk = Num<T>::to(sink[h]);
+  const float snk = sink ? Num<T>::to(sink[h]) : -CUDART_INF_F;
   const float m_mine = tid < splits ? stat[(at + tid) * 2] : -CUDART_INF_F;    // splits <= 128: a slice per thread
   float m = fmaxf(m_mine, snk);
 #pragma unroll
@@ -452,7 +476,8 @@ __global__ void __launch_bounds__(128) grouped_finish_kernel(const float* __rest
   __syncthreads();
   if ((tid & 31) == 0) red[tid >> 5] = part;
   __syncthreads();
-  const float inv = 1.0f / (red[0] + red[1] + red[2] + red[3] + expf(snk - m));
+  const float den = red[0] + red[1] + red[2] + red[3] + (sink ? expf(snk - m) : 0.f);
+  const float inv = den > 0.f ? (gate ? sigmoid_f(Num<T>::to(gate[b * ldg + h])) : 1.0f) / den : 0.f;   // no visible key: zeros
   for (int c = tid; c < vdim; c += blockDim.x) {
     float v = 0.f;
 #pragma unroll 8
@@ -510,14 +535,15 @@ extern "C" int oslo_grouped_splits(int B, int H, int G, int T, int dim, int vdim
 }
 
 extern "C" int oslo_grouped_decode(const void* q, const void* kc, const void* vc, const int* lengths, const uint8_t* keep,
-                                   long long ld_keep, int n_keep, const void* sink, float* ws, float* stat, void* out, int B,
-                                   int H, int G, int dim, int vdim, int Tmax, int splits, float scale, float softcap, int dtype,
-                                   int* err_word, cudaStream_t stream) {
+                                   long long ld_keep, int n_keep, const void* sink, const void* gate, long long ldg, int window,
+                                   int keep_first, const int* lead, float* ws, float* stat, void* out, int B, int H, int G, int dim,
+                                   int vdim, int Tmax, int splits, float scale, float softcap, int dtype, int* err_word,
+                                   cudaStream_t stream) {
   using namespace oslo;
   if (B <= 0 || H <= 0) return 0;
-  if (G <= 0 || H % G || B > 65535 || splits < 1 || splits > GD_MAX_SPLITS) return -1;
+  if (G <= 0 || H % G || B > 65535 || window < 0 || keep_first < 0 || splits < 1 || splits > GD_MAX_SPLITS) return -1;
   GroupedParams p{q, kc, vc, lengths, keep, ld_keep, n_keep, ws, stat, H, G, dim, vdim, (vdim + 3) / 4 * 4, Tmax, splits,
-                  scale, softcap, err_word};
+                  scale, softcap, window, keep_first, lead, err_word};
   const int tiles = (H / G + GD_HEADS - 1) / GD_HEADS;
   const dim3 grid(splits, G * tiles, B);
   const size_t smem = (static_cast<size_t>(GD_HEADS + GD_KEYS) * (dim + 1) + static_cast<size_t>(GD_KEYS) * vdim) * sizeof(float);
@@ -538,8 +564,8 @@ extern "C" int oslo_grouped_decode(const void* q, const void* kc, const void* vc
   rc = widest <= 64 ? gd_mma_launch<T, 64>(p, B, stream) : (widest <= 128 ? gd_mma_launch<T, 128>(p, B, stream)               \
                                                                            : gd_mma_launch<T, 256>(p, B, stream));            \
   if (rc == 0)                                                                                                                \
-    grouped_finish_kernel<T><<<dim3(H, B), 128, 0, stream>>>(ws, stat, static_cast<const T*>(sink), static_cast<T*>(out), H,  \
-                                                             vdim, p.ldw, splits);
+    grouped_finish_kernel<T><<<dim3(H, B), 128, 0, stream>>>(ws, stat, static_cast<const T*>(sink), static_cast<const T*>(gate), \
+                                                             ldg, static_cast<T*>(out), H, vdim, p.ldw, splits);
     if (dtype == OSLO_DT_BF16) { GM_GO(__nv_bfloat16) } else { GM_GO(__half) }
 #undef GM_GO
     return rc ? rc : static_cast<int>(cudaGetLastError());
@@ -549,8 +575,8 @@ extern "C" int oslo_grouped_decode(const void* q, const void* kc, const void* vc
     else if (vdim <= 512) GD_GO(2)
     else if (vdim <= 1024) GD_GO(4)
     else return -3;
-    grouped_finish_kernel<T><<<dim3(H, B), 128, 0, stream>>>(ws, stat, static_cast<const T*>(sink), static_cast<T*>(out), H, vdim,
-                                                             p.ldw, splits);
+    grouped_finish_kernel<T><<<dim3(H, B), 128, 0, stream>>>(ws, stat, static_cast<const T*>(sink), static_cast<const T*>(gate), ldg,
+                                                             static_cast<T*>(out), H, vdim, p.ldw, splits);
   });
 #undef GD_GO
   return static_cast<int>(cudaGetLastError());

@@ -1,12 +1,13 @@
-// Latent attention (one low-rank vector c per token is cached; every head's key W_uk c and value W_uv c come from it),
-// softmax with a learned sink in the denominator, one sigmoid output gate per head.
+// Latent attention (one low-rank vector c per token is cached; every head's key W_uk c and value W_uv c come from it), optionally
+// with a rotated key part that all heads share (cached behind c), a learned sink in the softmax denominator, sigmoid output
+// gates per head or per element.
 //
 // Prompts: keys and values are expanded with a GEMM. For 16-bit head sizes that the tcgen05 flash kernel takes, that
 // kernel runs and sink_gate_kernel turns its (output, log-sum-exp) pair into the result:
 //   out * exp(lse) / (exp(lse) + exp(sink)) * sigmoid(g) = out * sigmoid(lse - sink) * sigmoid(g).
 // sink_attention_kernel covers everything else (float32, any head sizes) in 32-bit.
-// Decode: keys are never expanded. latent_absorb_kernel moves W_uk to the query side (q' = W_uk^T q, 32-bit), the
-// scores are q' . c, latent_decode_*_kernel accumulates sum_t p_t c_t per head over slices of the cache, and
+// Decode: keys are never expanded. latent_absorb_kernel moves W_uk to the query side (q' = W_uk^T q, 32-bit) and rotates the
+// query's own rotated part, which follows q'; the scores are q' . (c and what is cached behind it), latent_decode_*_kernel accumulates sum_t p_t c_t per head over slices of the cache, and
 // latent_finish_kernel merges the slices, adds the sink to the denominator, applies W_uv and the gate. All heads of a
 // block share each cached vector they read.
 #include <math_constants.h>
@@ -58,6 +59,9 @@ struct SinkAttnParams {
   void* out;                           // [B * Sq, H * vdim]
   int B, H, G, Sq, Sk, dim, vdim;      // query head h reads key / value head h / (H / G)
   float scale, softcap;                // softcap > 0: scores become softcap * tanh(score / softcap)
+  int window, keep_first;              // window > 0: the last `window` keys, and the first keep_first after lead[b]
+  const int* lead;                     // [B] padding ahead of the sequence, or nullptr
+  int gate_wide;                       // the gate has a column per output column
 };
 
 constexpr int SA_Q = 16, SA_K = 32;
@@ -84,10 +88,13 @@ __global__ void __launch_bounds__(128) sink_attention_kernel(const SinkAttnParam
     qs[r * dp + c] = q0 + r < p.Sq ? Num<T>::to(q[(q0 + r) * p.q_ss + c]) : 0.f;
   }
   for (int e = tid; e < SA_Q * p.vdim; e += 128) os[(e / p.vdim) * vp + e % p.vdim] = 0.f;
-  const float sink = Num<T>::to(static_cast<const T*>(p.sink)[h]);
-  float m = sink, s = 1.0f;            // the sink is the first member of the denominator
+  // the sink is the first member of the denominator
+  float m = p.sink ? Num<T>::to(static_cast<const T*>(p.sink)[h]) : -CUDART_INF_F, s = p.sink ? 1.0f : 0.f;
   const int k_end = min(p.Sk, past + q0 + SA_Q);
+  const int kept = p.window > 0 ? (p.lead ? p.lead[b] : 0) + p.keep_first : 0;     // keys before this one are in every window
+  const int near = p.window > 0 ? past + q0 - p.window + 1 : 0;                    // no window of this block starts earlier
   for (int k0 = 0; k0 < k_end; k0 += SA_K) {
+    if (k0 + SA_K <= near && k0 >= kept) continue;     // uniform over the block
     __syncthreads();
     for (int e = tid; e < SA_K * p.dim; e += 128) {
       const int r = e / p.dim, c = e % p.dim;
@@ -104,7 +111,8 @@ __global__ void __launch_bounds__(128) sink_attention_kernel(const SinkAttnParam
       const int kj = u * 8 + l8, pos = k0 + kj;
       float d = 0.f;
       for (int c = 0; c < p.dim; ++c) d = fmaf(qs[qi * dp + c], ks[kj * dp + c], d);
-      const bool vis = pos < k_end && pos <= past + q0 + qi && (p.keep == nullptr || p.keep[b * p.ld_keep + pos]);
+      const bool in = p.window <= 0 || past + q0 + qi - pos < p.window || pos < kept;
+      const bool vis = in && pos < k_end && pos <= past + q0 + qi && (p.keep == nullptr || p.keep[b * p.ld_keep + pos]);
       d *= p.scale;
       if (p.softcap > 0.f) d = p.softcap * tanhf(d / p.softcap);
       sc[u] = vis ? d : -CUDART_INF_F;
@@ -112,11 +120,12 @@ __global__ void __launch_bounds__(128) sink_attention_kernel(const SinkAttnParam
     }
 #pragma unroll
     for (int off = 4; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
-    const float a = expf(m - mx);      // m is finite: it starts at the sink
+    const float base = mx == -CUDART_INF_F ? 0.f : mx; // nothing seen yet: every term is exp(-inf) = 0
+    const float a = expf(m - base);
     float ps_sum = 0.f;
 #pragma unroll
     for (int u = 0; u < SA_K / 8; ++u) {
-      const float e = expf(sc[u] - mx);
+      const float e = expf(sc[u] - base);
       ps[qi * (SA_K + 1) + u * 8 + l8] = e;
       ps_sum += e;
     }
@@ -134,37 +143,70 @@ __global__ void __launch_bounds__(128) sink_attention_kernel(const SinkAttnParam
   }
   if (q0 + qi < p.Sq) {
     const long long row = static_cast<long long>(b) * p.Sq + q0 + qi;
-    const float fac = (p.gate ? sigmoid_f(Num<T>::to(static_cast<const T*>(p.gate)[row * p.ldg + h])) : 1.0f) / s;
+    const T* gate = static_cast<const T*>(p.gate) + (p.gate ? row * p.ldg : 0);
+    float fac = s > 0.f ? 1.0f / s : 0.f;              // a padded query may see nothing
+    if (p.gate && !p.gate_wide) fac *= sigmoid_f(Num<T>::to(gate[h]));
     T* out = static_cast<T*>(p.out) + row * (static_cast<long long>(p.H) * p.vdim) + static_cast<long long>(h) * p.vdim;
-    for (int c = l8; c < p.vdim; c += 8) out[c] = Num<T>::from(os[qi * vp + c] * fac);
+    for (int c = l8; c < p.vdim; c += 8) {
+      const float g = p.gate && p.gate_wide ? sigmoid_f(Num<T>::to(gate[static_cast<long long>(h) * p.vdim + c])) : 1.0f;
+      out[c] = Num<T>::from(os[qi * vp + c] * fac * g);
+    }
   }
 }
 
 // ------------------------------------------------------------------ decode
-// block (0, b): RMS norm of the query latent; block (1, b): RMS norm of the key-value latent, written to the cache at
-// position lengths[b]
+// the pair (x, y) turned by the angle a
+__device__ __forceinline__ void turn(float a, float& x, float& y) {
+  float sn, cs;
+  sincosf(a, &sn, &cs);
+  const float u = x * cs - y * sn;
+  y = y * cs + x * sn;
+  x = u;
+}
+
+struct LatentPrepParams {
+  const void *cq, *wq; long long ldq; int q_rank;
+  void* cq_out;
+  const void *ckv, *wkv; long long ldkv; int kv_rank, rot;
+  void* cache;                         // [B, Tmax, kv_rank + rot]
+  void* c_out;                         // [B * S, kv_rank] or nullptr
+  const int* lengths;
+  const long long* pos; long long pos_sb, pos_ss;
+  const float* freq;                   // [rot / 2]
+  int S, Tmax;
+  float eps;
+  int* err;
+};
+
+// block (0, row b * S + t): RMS norm of the query latent; block (1, row): RMS norm of the key-value latent and rotation of the key
+// part behind it, written to the cache at position lengths[b] + t
 template <typename T>
-__global__ void __launch_bounds__(256) latent_prep_kernel(const T* __restrict__ cq, long long ldq, const T* __restrict__ wq,
-                                                          int q_rank, T* __restrict__ cq_out, const T* __restrict__ ckv,
-                                                          long long ldkv, const T* __restrict__ wkv, int kv_rank,
-                                                          T* __restrict__ cache, const int* __restrict__ lengths, int Tmax,
-                                                          float eps, int* err) {
+__global__ void __launch_bounds__(256) latent_prep_kernel(const LatentPrepParams p) {
   __shared__ float red[32];
-  const int b = blockIdx.y;
-  const bool is_q = blockIdx.x == 0;
-  const T* x = is_q ? cq + b * ldq : ckv + b * ldkv;
-  const T* w = is_q ? wq : wkv;
-  const int n = is_q ? q_rank : kv_rank;
-  T* out;
+  const long long row = blockIdx.x;
+  const bool is_q = blockIdx.y == 0;
+  const T* x = is_q ? static_cast<const T*>(p.cq) + row * p.ldq : static_cast<const T*>(p.ckv) + row * p.ldkv;
+  const T* w = static_cast<const T*>(is_q ? p.wq : p.wkv);
+  const int n = is_q ? p.q_rank : p.kv_rank;
+  T *out, *again = nullptr;
   if (is_q) {
-    out = cq_out + static_cast<long long>(b) * q_rank;
+    out = static_cast<T*>(p.cq_out) + row * p.q_rank;
   } else {
-    const int pos = lengths[b];
-    if (pos < 0 || pos >= Tmax) {      // never write outside the cache
-      if (threadIdx.x == 0) OSLO_REPORT_BOUNDS(err);
+    const long long b = row / p.S, t = row - b * p.S;
+    const long long at = p.lengths[b] + t;
+    if (at < 0 || at >= p.Tmax) {      // never write outside the cache
+      if (threadIdx.x == 0) OSLO_REPORT_BOUNDS(p.err);
       return;
     }
-    out = cache + (static_cast<long long>(b) * Tmax + pos) * kv_rank;
+    out = static_cast<T*>(p.cache) + (b * p.Tmax + at) * (p.kv_rank + p.rot);
+    if (p.c_out) again = static_cast<T*>(p.c_out) + row * p.kv_rank;
+    const int half = p.rot / 2;
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+      float u = Num<T>::to(x[n + i]), v = Num<T>::to(x[n + half + i]);
+      turn(static_cast<float>(p.pos[b * p.pos_sb + t * p.pos_ss]) * p.freq[i], u, v);
+      out[n + i] = Num<T>::from(u);
+      out[n + half + i] = Num<T>::from(v);
+    }
   }
   float ss = 0.f;
   for (int c = threadIdx.x; c < n; c += blockDim.x) {
@@ -172,24 +214,72 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const T* __restrict__ 
     ss = fmaf(v, v, ss);
   }
   ss = block_sum(ss, red);
-  const float r = 1.0f / sqrtf(ss / n + eps);
-  for (int c = threadIdx.x; c < n; c += blockDim.x) out[c] = Num<T>::from(Num<T>::to(x[c]) * r * Num<T>::to(w[c]));
+  const float r = 1.0f / sqrtf(ss / n + p.eps);
+  for (int c = threadIdx.x; c < n; c += blockDim.x) {
+    const T v = Num<T>::from(Num<T>::to(x[c]) * r * Num<T>::to(w[c]));
+    out[c] = v;
+    if (again) again[c] = v;
+  }
+}
+
+// in place, a thread per pair of the last rot dims of a head
+template <typename T>
+__global__ void __launch_bounds__(256) rotate_halves_kernel(T* __restrict__ q, const long long* __restrict__ pos, long long pos_sb,
+                                                            long long pos_ss, const float* __restrict__ freq, long long pairs, int S,
+                                                            int H, int dim, int rot) {
+  const int half = rot / 2;
+  for (long long e = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; e < pairs;
+       e += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const int i = static_cast<int>(e % half);
+    const long long head = e / half, row = head / H, b = row / S, t = row - b * S;
+    T* at = q + head * (dim + rot) + dim + i;
+    float u = Num<T>::to(at[0]), v = Num<T>::to(at[half]);
+    turn(static_cast<float>(pos[b * pos_sb + t * pos_ss]) * freq[i], u, v);
+    at[0] = Num<T>::from(u);
+    at[half] = Num<T>::from(v);
+  }
+}
+
+// what a decode step's query carries besides the part that meets W_uk
+struct QueryTail {
+  int rot;                             // 0: nothing
+  const long long* pos; long long pos_sb;
+  const float* freq;
+};
+// columns R .. R + rot of qa for rows b0 .. b0 + nb, head h: the query's rotated part, scaled
+template <typename T>
+__device__ __forceinline__ void absorb_tail(const T* q, long long ldq, float* qa, const QueryTail& x, int b0, int nb, int h, int H,
+                                            int dim, int R, float scale) {
+  const int half = x.rot / 2;
+  for (int e = threadIdx.x; e < nb * half; e += blockDim.x) {
+    const int b = b0 + e / half, i = e % half;
+    const T* src = q + b * ldq + static_cast<long long>(h) * (dim + x.rot) + dim + i;
+    float u = Num<T>::to(src[0]), v = Num<T>::to(src[half]);
+    turn(static_cast<float>(x.pos[b * x.pos_sb]) * x.freq[i], u, v);
+    float* dst = qa + (static_cast<long long>(b) * H + h) * (R + x.rot) + R + i;
+    dst[0] = u * scale;
+    dst[half] = v * scale;
+  }
 }
 
 // qa[b, h, r] = scale * sum_d q[b, h * dim + d] * w_uk[h * dim + d, r]; block = (64 columns r, head, NB rows b)
 template <typename T, int VEC, int NB>
 __global__ void __launch_bounds__(256) latent_absorb_kernel(const T* __restrict__ q, long long ldq, const T* __restrict__ w,
                                                             long long ldw, float* __restrict__ qa, int B, int H, int dim,
-                                                            int R, float scale) {
+                                                            int R, float scale, const QueryTail tail) {
   constexpr int CW = 64, CP = CW / VEC, DG = 256 / CP;   // VEC columns per thread, DG groups of rows d
   extern __shared__ float ab_smem[];
   float* qs = ab_smem;                 // [NB][dim]
   float* part = qs + NB * dim;         // [DG][CW], one row b at a time
   const int h = blockIdx.y, r0 = blockIdx.x * CW, b0 = blockIdx.z * NB;
   const int nb = min(NB, B - b0);
+  if (r0 >= R) {                       // one more block along the columns when there is a rotated part
+    absorb_tail<T>(q, ldq, qa, tail, b0, nb, h, H, dim, R, scale);
+    return;
+  }
   for (int b = 0; b < nb; ++b)
     for (int d = threadIdx.x; d < dim; d += 256)
-      qs[b * dim + d] = Num<T>::to(q[(b0 + b) * ldq + static_cast<long long>(h) * dim + d]) * scale;
+      qs[b * dim + d] = Num<T>::to(q[(b0 + b) * ldq + static_cast<long long>(h) * (dim + tail.rot) + d]) * scale;
   __syncthreads();
   const int cp = threadIdx.x % CP, dg = threadIdx.x / CP;
   const int r = r0 + cp * VEC;
@@ -223,19 +313,20 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const T* __restrict_
       float t = 0.f;
 #pragma unroll
       for (int g = 0; g < DG; ++g) t += part[g * CW + threadIdx.x];
-      qa[(static_cast<long long>(b0 + b) * H + h) * R + r0 + threadIdx.x] = t;
+      qa[(static_cast<long long>(b0 + b) * H + h) * (R + tail.rot) + r0 + threadIdx.x] = t;
     }
   }
 }
 
 struct LatentDecodeParams {
-  const float* qa;                     // [B, H, R], scaled
-  const void* cache;                   // [B, Tmax, R]
+  const float* qa;                     // [B, H, W], scaled
+  const void* cache;                   // [B, Tmax, W]
   const int* lengths;                  // [B] valid positions
   const uint8_t* keep; long long ld_keep; int n_keep;   // [B, n_keep], 0 = padded, or nullptr
   float* ws;                           // [B, H, splits, ldw]: sum p c; ldw = R rounded up to a multiple of 4
   float* stat;                         // [B, H, splits, 2]: max, sum p
-  int B, H, R, ldw, Tmax, splits;
+  int B, H, R, W, ldw, Tmax, splits;   // W = R + rotated part: the width of the scores' vectors
+  int gate_wide;                       // the output gate has a column per output column
   int* err;
 };
 
@@ -245,9 +336,9 @@ constexpr int LD_HEADS = 16, LD_KEYS = 16;
 template <typename T, int NR>
 __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentDecodeParams p) {
   extern __shared__ float ld_smem[];
-  const int rp = p.R + 1;
-  float* qs = ld_smem;                 // [LD_HEADS][R + 1]
-  float* cs = qs + LD_HEADS * rp;      // [LD_KEYS][R + 1]
+  const int rp = p.W + 1;
+  float* qs = ld_smem;                 // [LD_HEADS][W + 1]
+  float* cs = qs + LD_HEADS * rp;      // [LD_KEYS][W + 1]
   float* sc = cs + LD_KEYS * rp;       // [LD_HEADS][LD_KEYS]
   __shared__ float resc[LD_HEADS], ms[LD_HEADS], ls[LD_HEADS];
   const int b = blockIdx.z, h0 = blockIdx.y * LD_HEADS, sp = blockIdx.x, tid = threadIdx.x;
@@ -259,28 +350,28 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentDecodePa
   }
   const int per = (len + p.splits - 1) / p.splits;
   const int t0 = sp * per, t1 = min(len, t0 + per);
-  for (int e = tid; e < nh * p.R; e += 256)
-    qs[(e / p.R) * rp + e % p.R] = p.qa[(static_cast<long long>(b) * p.H + h0) * p.R + e];
-  for (int e = tid; e < (LD_HEADS - nh) * p.R; e += 256) qs[(nh + e / p.R) * rp + e % p.R] = 0.f;
+  for (int e = tid; e < nh * p.W; e += 256)
+    qs[(e / p.W) * rp + e % p.W] = p.qa[(static_cast<long long>(b) * p.H + h0) * p.W + e];
+  for (int e = tid; e < (LD_HEADS - nh) * p.W; e += 256) qs[(nh + e / p.W) * rp + e % p.W] = 0.f;
   if (tid < LD_HEADS) { ms[tid] = -CUDART_INF_F; ls[tid] = 0.f; }
   float acc[NR][LD_HEADS];
 #pragma unroll
   for (int j = 0; j < NR; ++j)
 #pragma unroll
     for (int a = 0; a < LD_HEADS; ++a) acc[j][a] = 0.f;
-  const T* c = static_cast<const T*>(p.cache) + static_cast<long long>(b) * p.Tmax * p.R;
+  const T* c = static_cast<const T*>(p.cache) + static_cast<long long>(b) * p.Tmax * p.W;
   for (int k0 = t0; k0 < t1; k0 += LD_KEYS) {
     const int n = min(LD_KEYS, t1 - k0);
     __syncthreads();
-    for (int e = tid; e < LD_KEYS * p.R; e += 256) {
-      const int t = e / p.R, r = e % p.R;
-      cs[t * rp + r] = t < n ? Num<T>::to(c[static_cast<long long>(k0 + t) * p.R + r]) : 0.f;
+    for (int e = tid; e < LD_KEYS * p.W; e += 256) {
+      const int t = e / p.W, r = e % p.W;
+      cs[t * rp + r] = t < n ? Num<T>::to(c[static_cast<long long>(k0 + t) * p.W + r]) : 0.f;
     }
     __syncthreads();
     {
       const int a = tid >> 4, t = tid & 15;
       float d = 0.f;
-      for (int r = 0; r < p.R; ++r) d = fmaf(qs[a * rp + r], cs[t * rp + r], d);
+      for (int r = 0; r < p.W; ++r) d = fmaf(qs[a * rp + r], cs[t * rp + r], d);
       const int pos = k0 + t;
       const bool vis = t < n && (p.keep == nullptr || pos >= p.n_keep || p.keep[b * p.ld_keep + pos]);
       d = vis ? d : -CUDART_INF_F;
@@ -334,9 +425,9 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentDecodePa
   }
 }
 
-// 16-bit version on the tensor cores for R % 16 == 0: MT x 16 heads are the rows of m16n8k16 tiles, so the cache streams
+// 16-bit version on the tensor cores for R % 16 == 0 and W % 16 == 0: MT x 16 heads are the rows of m16n8k16 tiles, so the cache streams
 // through shared memory once for all of them. 8 warps, LM_KT cached vectors per step:
-//   scores  warp = (16 heads) x (16 of the keys) x (a half or a quarter of R); q' as 16-bit, 32-bit sums
+//   scores  warp = (16 heads) x (16 of the keys) x (a half or a quarter of W); q' as 16-bit, 32-bit sums
 //   softmax warp w owns heads 2 MT w ..; lane = key; running max and sum in registers, P is stored as 16-bit
 //   output  a warp owns every eighth pair of 8-column blocks of R; the cached vectors are read transposed
 // The next vectors are fetched with cp.async meanwhile, and two blocks per SM overlap each other's phases.
@@ -372,7 +463,7 @@ __device__ __forceinline__ void ldsm4_t(uint32_t addr, uint32_t (&r)[4]) {
 template <typename T>
 __global__ void __launch_bounds__(256) latent_absorb_mma_kernel(const T* __restrict__ q, long long ldq, const T* __restrict__ w,
                                                                 long long ldw, float* __restrict__ qa, int B, int H, int dim,
-                                                                int R, float scale) {
+                                                                int R, float scale, const QueryTail tail) {
   constexpr int CW = 64, WP = CW + 8;
   extern __shared__ __align__(16) uint8_t am_smem[];
   const int qp = dim + 8;
@@ -380,6 +471,10 @@ __global__ void __launch_bounds__(256) latent_absorb_mma_kernel(const T* __restr
   T* wsm = qs + 16 * qp;                   // [dim][WP]
   const int h = blockIdx.y, r0 = blockIdx.x * CW, b0 = blockIdx.z * 16;
   const int nb = min(16, B - b0), nc = min(CW, R - r0) / 8;   // 16-byte pieces of a tile row
+  if (r0 >= R) {                           // one more block along the columns when there is a rotated part
+    absorb_tail<T>(q, ldq, qa, tail, b0, nb, h, H, dim, R, scale);
+    return;
+  }
   for (int e = threadIdx.x; e < dim * 8; e += 256) {
     const int d = e >> 3, v = e & 7;
     const bool in = v < nc;                // columns past R are zero-filled
@@ -390,7 +485,7 @@ __global__ void __launch_bounds__(256) latent_absorb_mma_kernel(const T* __restr
   asm volatile("cp.async.commit_group;" ::: "memory");
   for (int e = threadIdx.x; e < 16 * dim; e += 256) {
     const int b = e / dim, d = e - b * dim;
-    qs[b * qp + d] = b < nb ? q[(b0 + b) * ldq + static_cast<long long>(h) * dim + d] : Num<T>::from(0.f);
+    qs[b * qp + d] = b < nb ? q[(b0 + b) * ldq + static_cast<long long>(h) * (dim + tail.rot) + d] : Num<T>::from(0.f);
   }
   asm volatile("cp.async.wait_group 0;" ::: "memory");
   __syncthreads();
@@ -409,7 +504,7 @@ __global__ void __launch_bounds__(256) latent_absorb_mma_kernel(const T* __restr
     for (int hf = 0; hf < 2; ++hf) {
       const int b = (lane >> 2) + 8 * hf;
       if (b < nb)
-        *reinterpret_cast<float2*>(qa + (static_cast<long long>(b0 + b) * H + h) * R + col) =
+        *reinterpret_cast<float2*>(qa + (static_cast<long long>(b0 + b) * H + h) * (R + tail.rot) + col) =
             make_float2(acc[hf * 2] * scale, acc[hf * 2 + 1] * scale);
     }
   }
@@ -421,7 +516,7 @@ template <typename T, int MT, int NP>   // MT groups of 16 heads, NP pairs of 8-
 __global__ void __launch_bounds__(256, NP <= 4 ? 2 : 1) latent_decode_mma_kernel(const LatentDecodeParams p) {
   constexpr int HM = 16 * MT, PP = LM_KT + 8, SP = LM_KT + 1, KS = 4 / MT;
   extern __shared__ __align__(16) uint8_t lm_smem[];
-  const int rp = p.R + 8;               // padded row: 16-byte aligned, conflict-free ldmatrix
+  const int rp = p.W + 8;               // padded row: 16-byte aligned, conflict-free ldmatrix
   T* qs = reinterpret_cast<T*>(lm_smem);            // [HM][rp]
   T* cs = qs + HM * rp;                             // [2][LM_KT][rp]
   T* ps = cs + 2 * LM_KT * rp;                      // [HM][PP]
@@ -437,8 +532,8 @@ __global__ void __launch_bounds__(256, NP <= 4 ? 2 : 1) latent_decode_mma_kernel
   }
   const int tiles = (len + LM_KT - 1) / LM_KT, per = (tiles + p.splits - 1) / p.splits * LM_KT;
   const int t0 = sp * per, t1 = min(len, t0 + per);
-  const T* c = static_cast<const T*>(p.cache) + static_cast<long long>(b) * p.Tmax * p.R;
-  const int vr = p.R / 8;              // 16-byte pieces of a cached vector
+  const T* c = static_cast<const T*>(p.cache) + static_cast<long long>(b) * p.Tmax * p.W;
+  const int vr = p.W / 8;              // 16-byte pieces of a cached vector
   const int dt = 256 / vr, dv = 256 % vr, ft = tid / vr, fv = tid % vr;
   auto fetch = [&](int k0, int buf) {
     T* dst = cs + static_cast<size_t>(buf) * LM_KT * rp;
@@ -446,7 +541,7 @@ __global__ void __launch_bounds__(256, NP <= 4 ? 2 : 1) latent_decode_mma_kernel
     while (t < LM_KT) {
       const uint32_t d32 = smem_u32(dst + t * rp + v * 8);
       const bool in = k0 + t < t1;     // rows past the slice are zero-filled (source size 0)
-      const T* src = c + static_cast<long long>(in ? k0 + t : 0) * p.R + v * 8;
+      const T* src = c + static_cast<long long>(in ? k0 + t : 0) * p.W + v * 8;
       const int bytes = in ? 16 : 0;
       asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d32), "l"(src), "r"(bytes) : "memory");
       t += dt;
@@ -457,9 +552,9 @@ __global__ void __launch_bounds__(256, NP <= 4 ? 2 : 1) latent_decode_mma_kernel
   };
   if (t0 < t1) fetch(t0, 0);
   for (int a = warp; a < HM; a += 8) {
-    const float* src = p.qa + (static_cast<long long>(b) * p.H + h0 + a) * p.R;
+    const float* src = p.qa + (static_cast<long long>(b) * p.H + h0 + a) * p.W;
 #pragma unroll 4
-    for (int r = lane * 4; r < p.R; r += 128) {
+    for (int r = lane * 4; r < p.W; r += 128) {
       float x[4] = {0.f, 0.f, 0.f, 0.f};
       if (a < nh) load_vec<float, 4>(src + r, x);
       store_vec<T, 4>(qs + a * rp + r, x);
@@ -479,7 +574,7 @@ __global__ void __launch_bounds__(256, NP <= 4 ? 2 : 1) latent_decode_mma_kernel
   for (int u = 0; u < 2 * MT; ++u) { m_run[u] = -CUDART_INF_F; l_run[u] = 0.f; }
   const int arow = lane & 15, acol = (lane >> 4) * 8;      // ldmatrix.x4 source of an A fragment
   const int kg = warp & 1, mt = (warp >> 1) % MT, ks = (warp >> 1) / MT;
-  const int n16 = p.R / 16, s_begin = ks * n16 / KS, s_end = (ks + 1) * n16 / KS;
+  const int n16 = p.W / 16, s_begin = ks * n16 / KS, s_end = (ks + 1) * n16 / KS;
   // B fragments of 16 keys x 16 columns: matrices (keys 0-7, cols 0-7), (keys 0-7, cols 8-15), (keys 8-15, ...)
   const int brow = kg * 16 + (lane & 7) + ((lane >> 4) << 3), bcol = ((lane >> 3) & 1) * 8;
   for (int k0 = t0, it = 0; k0 < t1; k0 += LM_KT, ++it) {
@@ -607,12 +702,12 @@ __global__ void __launch_bounds__(256, NP <= 4 ? 2 : 1) latent_decode_mma_kernel
     }
   }
 }
-static size_t latent_mma_smem(int R, int mt) {
-  const size_t rp = R + 8, hm = 16 * mt;
+static size_t latent_mma_smem(int W, int mt) {
+  const size_t rp = W + 8, hm = 16 * mt;
   return (hm * rp + 2 * LM_KT * rp + hm * (LM_KT + 8)) * 2 + (4 / mt * hm * (LM_KT + 1) + hm) * sizeof(float);
 }
 
-// the slice weights of one row (all lanes of a warp): wt[s] = exp(max_s - max) * gate / denominator
+// the slice weights of one row (all lanes of a warp): wt[s] = exp(max_s - max) * gate / denominator; sink -inf: none
 template <typename T>
 __device__ __forceinline__ void slice_weights(const LatentDecodeParams& p, int b, int h, float snk, float gate, float* wt, int lane) {
   const float2* st = reinterpret_cast<const float2*>(p.stat) + (static_cast<long long>(b) * p.H + h) * p.splits;
@@ -620,6 +715,7 @@ __device__ __forceinline__ void slice_weights(const LatentDecodeParams& p, int b
   for (int s = lane; s < p.splits; s += 32) m = fmaxf(m, st[s].x);
 #pragma unroll
   for (int off = 16; off > 0; off >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, off));
+  if (m == -CUDART_INF_F) m = 0.f;     // no visible key: all terms are zero
   float tot = 0.f;
   for (int s = lane; s < p.splits; s += 32) {
     const float2 ml = st[s];
@@ -627,7 +723,8 @@ __device__ __forceinline__ void slice_weights(const LatentDecodeParams& p, int b
     tot += f * ml.y;
     wt[s] = f;
   }
-  const float g = sigmoid_f(gate) / (warp_sum(tot) + expf(snk - m));
+  const float den = warp_sum(tot) + expf(snk - m);
+  const float g = den > 0.f ? gate / den : 0.f;
   for (int s = lane; s < p.splits; s += 32) wt[s] *= g;
 }
 
@@ -642,9 +739,9 @@ __global__ void __launch_bounds__(256) latent_finish_kernel(const LatentDecodePa
   float* wt = fin_smem + NB * p.ldw;
   const int h = blockIdx.y, b0 = blockIdx.z * NB, nb = min(NB, p.B - b0), R = p.R, splits = p.splits;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const float snk = Num<T>::to(sink[h]);
+  const float snk = sink ? Num<T>::to(sink[h]) : -CUDART_INF_F;
   for (int i = warp; i < nb; i += 8)
-    slice_weights<T>(p, b0 + i, h, snk, Num<T>::to(gate[(b0 + i) * ldg + h]), wt + i * splits, lane);
+    slice_weights<T>(p, b0 + i, h, snk, p.gate_wide ? 1.f : sigmoid_f(Num<T>::to(gate[(b0 + i) * ldg + h])), wt + i * splits, lane);
   __syncthreads();
   const int quads = p.ldw / 4;
   for (int e = threadIdx.x; e < nb * quads; e += 256) {
@@ -696,7 +793,10 @@ __global__ void __launch_bounds__(256) latent_finish_kernel(const LatentDecodePa
 #pragma unroll
       for (int i = 0; i < NB; ++i) {
         const float d = warp_sum(acc[a][i]);
-        if (lane == 0 && i < nb && a < nj) out[(static_cast<long long>(b0 + i) * p.H + h) * vdim + j + a] = Num<T>::from(d);
+        if (lane == 0 && i < nb && a < nj) {
+          const float g = p.gate_wide ? sigmoid_f(Num<T>::to(gate[(b0 + i) * ldg + static_cast<long long>(h) * vdim + j + a])) : 1.f;
+          out[(static_cast<long long>(b0 + i) * p.H + h) * vdim + j + a] = Num<T>::from(d * g);
+        }
       }
   }
 }
@@ -713,9 +813,9 @@ __global__ void __launch_bounds__(256) latent_finish_mma_kernel(const LatentDeco
   float* wt = reinterpret_cast<float*>(o + 16 * op);       // [16][splits]
   const int h = blockIdx.y, b0 = blockIdx.z * 16, nb = min(16, p.B - b0);
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const float snk = Num<T>::to(sink[h]);
+  const float snk = sink ? Num<T>::to(sink[h]) : -CUDART_INF_F;
   for (int i = warp; i < nb; i += 8)
-    slice_weights<T>(p, b0 + i, h, snk, Num<T>::to(gate[(b0 + i) * ldg + h]), wt + i * p.splits, lane);
+    slice_weights<T>(p, b0 + i, h, snk, p.gate_wide ? 1.f : sigmoid_f(Num<T>::to(gate[(b0 + i) * ldg + h])), wt + i * p.splits, lane);
   __syncthreads();
 #pragma unroll 2
   for (int e = threadIdx.x; e < 16 * quads; e += 256) {
@@ -750,7 +850,12 @@ __global__ void __launch_bounds__(256) latent_finish_mma_kernel(const LatentDeco
     for (int hf = 0; hf < 2; ++hf) {
       const int b = g + 8 * hf;
       if (b < nb) {
-        const float v[2] = {acc[hf * 2], acc[hf * 2 + 1]};
+        float v[2] = {acc[hf * 2], acc[hf * 2 + 1]};
+        if (p.gate_wide) {                 // the gate's rows need not be aligned
+          const T* g = gate + (b0 + b) * ldg + static_cast<long long>(h) * vdim + j0 + t * 2;
+          v[0] *= sigmoid_f(Num<T>::to(g[0]));
+          v[1] *= sigmoid_f(Num<T>::to(g[1]));
+        }
         store_vec<T, 2>(out + (static_cast<long long>(b0 + b) * p.H + h) * vdim + j0 + t * 2, v);
       }
     }
@@ -785,12 +890,13 @@ extern "C" int oslo_sink_attention(const void* q, long long q_sb, long long q_ss
                                    long long k_ss, long long k_sh, const void* v, long long v_sb, long long v_ss,
                                    long long v_sh, const uint8_t* keep, long long ld_keep, const void* sink, const void* gate,
                                    long long ldg, void* out, int B, int H, int G, int Sq, int Sk, int dim, int vdim, float scale,
-                                   float softcap, int dtype, cudaStream_t stream) {
+                                   float softcap, int window, int keep_first, const int* lead, int gate_wide, int dtype,
+                                   cudaStream_t stream) {
   using namespace oslo;
   if (B <= 0 || H <= 0 || Sq <= 0) return 0;
   if (Sk < Sq || B > 65535 || H > 65535 || G <= 0 || H % G) return -1;
   SinkAttnParams p{q, k, v, q_sb, q_ss, q_sh, k_sb, k_ss, k_sh, v_sb, v_ss, v_sh, keep, ld_keep, sink, gate, ldg, out,
-                   B, H, G, Sq, Sk, dim, vdim, scale, softcap};
+                   B, H, G, Sq, Sk, dim, vdim, scale, softcap, window, keep_first, lead, gate_wide};
   const size_t smem = (static_cast<size_t>(SA_Q + SA_K) * (dim + 1 + vdim + 1) + SA_Q * (SA_K + 1)) * sizeof(float);
   dim3 grid((Sq + SA_Q - 1) / SA_Q, H, B);
   OSLO_DISPATCH_T(dtype, {
@@ -803,13 +909,27 @@ extern "C" int oslo_sink_attention(const void* q, long long q_sb, long long q_ss
 
 extern "C" int oslo_latent_prep(const void* cq, long long ldq, const void* wq, int q_rank, void* cq_out, const void* ckv,
                                 long long ldkv, const void* wkv, int kv_rank, void* cache, const int* lengths, int Tmax,
-                                float eps, int B, int dtype, int* err_word, cudaStream_t stream) {
+                                float eps, int B, int S, int rot, const long long* pos, long long pos_sb, long long pos_ss,
+                                const float* freq, void* c_out, int dtype, int* err_word, cudaStream_t stream) {
   using namespace oslo;
-  if (B <= 0) return 0;
+  if (B <= 0 || S <= 0) return 0;
+  const long long rows = static_cast<long long>(B) * S;
+  if (rows > 0x7fffffffll || rot < 0 || rot % 2 || (rot > 0 && (pos == nullptr || freq == nullptr))) return -1;
+  const LatentPrepParams p{cq, wq, ldq, q_rank, cq_out, ckv, wkv, ldkv, kv_rank, rot, cache, c_out, lengths, pos, pos_sb, pos_ss,
+                           freq, S, Tmax, eps, err_word};
+  const int threads = std::max(q_rank, kv_rank) <= 128 && rows > 64 ? 64 : 256;
+  OSLO_DISPATCH_T(dtype, { latent_prep_kernel<T><<<dim3(static_cast<unsigned>(rows), ckv ? 2 : 1), threads, 0, stream>>>(p); });
+  return static_cast<int>(cudaGetLastError());
+}
+
+extern "C" int oslo_rotate_halves(void* q, const long long* pos, long long pos_sb, long long pos_ss, const float* freq, int B, int S,
+                                  int H, int dim, int rot, int dtype, cudaStream_t stream) {
+  using namespace oslo;
+  const long long pairs = static_cast<long long>(B) * S * H * (rot / 2);
+  if (pairs <= 0) return 0;
+  const unsigned blocks = static_cast<unsigned>(std::min<long long>((pairs + 255) / 256, 148 * 32));
   OSLO_DISPATCH_T(dtype, {
-    latent_prep_kernel<T><<<dim3(ckv ? 2 : 1, B), 256, 0, stream>>>(
-        static_cast<const T*>(cq), ldq, static_cast<const T*>(wq), q_rank, static_cast<T*>(cq_out), static_cast<const T*>(ckv),
-        ldkv, static_cast<const T*>(wkv), kv_rank, static_cast<T*>(cache), lengths, Tmax, eps, err_word);
+    rotate_halves_kernel<T><<<blocks, 256, 0, stream>>>(static_cast<T*>(q), pos, pos_sb, pos_ss, freq, pairs, S, H, dim, rot);
   });
   return static_cast<int>(cudaGetLastError());
 }
@@ -821,7 +941,7 @@ static int latent_scan(const LatentDecodeParams& p, int use_mma, cudaStream_t st
   if constexpr (sizeof(T) == 2) {
     if (use_mma) {
       const int mt = p.H > LD_HEADS ? 2 : 1, np = (p.R + 127) / 128;
-      const size_t smem = latent_mma_smem(p.R, mt);
+      const size_t smem = latent_mma_smem(p.W, mt);
       dim3 grid(p.splits, (p.H + 16 * mt - 1) / (16 * mt), p.B);
 #define LM_GO(MT, NP)                                                                                   \
   {                                                                                                     \
@@ -844,7 +964,7 @@ static int latent_scan(const LatentDecodeParams& p, int use_mma, cudaStream_t st
     }
   }
   dim3 grid(p.splits, (p.H + LD_HEADS - 1) / LD_HEADS, p.B);
-  const size_t smem = (static_cast<size_t>(LD_HEADS + LD_KEYS) * (p.R + 1) + LD_HEADS * LD_KEYS) * sizeof(float);
+  const size_t smem = (static_cast<size_t>(LD_HEADS + LD_KEYS) * (p.W + 1) + LD_HEADS * LD_KEYS) * sizeof(float);
 #define LD_GO(NR)                                                                               \
   {                                                                                             \
     const int rc = set_smem(reinterpret_cast<const void*>(&latent_decode_kernel<T, NR>), smem); \
@@ -860,26 +980,27 @@ static int latent_scan(const LatentDecodeParams& p, int use_mma, cudaStream_t st
 
 template <typename T, int VEC>
 static int latent_absorb(const LatentDecodeParams& p, const void* q, long long ldq, const void* w, long long ldw, float* qa,
-                         int dim, float scale, cudaStream_t st) {
+                         int dim, float scale, const QueryTail& tail, cudaStream_t st) {
+  const int extra = tail.rot > 0 ? 1 : 0;  // a block of its own for the rotated part
   if constexpr (sizeof(T) == 2 && VEC == 8) {
     if (p.B > 2 && dim % 16 == 0) {
       const size_t smem = (16 * static_cast<size_t>(dim + 8) + static_cast<size_t>(dim) * 72) * 2;
       const int rc = set_smem(reinterpret_cast<const void*>(&latent_absorb_mma_kernel<T>), smem);
       if (rc) return rc;
-      latent_absorb_mma_kernel<T><<<dim3((p.R + 63) / 64, p.H, (p.B + 15) / 16), 256, smem, st>>>(
-          static_cast<const T*>(q), ldq, static_cast<const T*>(w), ldw, qa, p.B, p.H, dim, p.R, scale);
+      latent_absorb_mma_kernel<T><<<dim3((p.R + 63) / 64 + extra, p.H, (p.B + 15) / 16), 256, smem, st>>>(
+          static_cast<const T*>(q), ldq, static_cast<const T*>(w), ldw, qa, p.B, p.H, dim, p.R, scale, tail);
       return static_cast<int>(cudaGetLastError());
     }
   }
   const int nb = p.B >= 8 ? 8 : (p.B >= 2 ? 2 : 1);
   const size_t smem = (static_cast<size_t>(nb) * dim + 256 * VEC) * sizeof(float);
-  dim3 grid((p.R + 63) / 64, p.H, (p.B + nb - 1) / nb);
+  dim3 grid((p.R + 63) / 64 + extra, p.H, (p.B + nb - 1) / nb);
 #define AB_GO(NB)                                                                                                       \
   {                                                                                                                     \
     const int rc = set_smem(reinterpret_cast<const void*>(&latent_absorb_kernel<T, VEC, NB>), smem);                    \
     if (rc) return rc;                                                                                                  \
     latent_absorb_kernel<T, VEC, NB><<<grid, 256, smem, st>>>(static_cast<const T*>(q), ldq, static_cast<const T*>(w), ldw, qa, \
-                                                              p.B, p.H, dim, p.R, scale);                               \
+                                                              p.B, p.H, dim, p.R, scale, tail);                         \
   }
   if (nb == 8) AB_GO(8)
   else if (nb == 2) AB_GO(2)
@@ -939,22 +1060,26 @@ extern "C" int oslo_latent_splits(int B, int H, int T, int num_sms) {
 extern "C" int oslo_latent_decode(const void* q, long long ldq, const void* w_uk, long long ldk, const void* w_uv, long long ldv,
                                   const void* cache, const int* lengths, const uint8_t* keep, long long ld_keep, int n_keep,
                                   const void* sink, const void* gate, long long ldg, float* qa, float* ws, float* stat, void* out,
-                                  int B, int H, int dim, int vdim, int R, int Tmax, int splits, float scale, int num_sms,
-                                  int dtype, int* err_word, cudaStream_t stream) {
+                                  int B, int H, int dim, int vdim, int R, int rot, const long long* pos, long long pos_sb,
+                                  const float* freq, int gate_wide, int Tmax, int splits, float scale, int num_sms, int dtype,
+                                  int* err_word, cudaStream_t stream) {
   using namespace oslo;
   if (B <= 0 || H <= 0) return 0;
   if (R <= 0 || R > 1024 || splits < 1 || splits > 64 || B > 65535 || H > 65535) return -1;
-  LatentDecodeParams p{qa, cache, lengths, keep, ld_keep, n_keep, ws, stat, B, H, R, (R + 3) / 4 * 4, Tmax, splits, err_word};
+  if (rot < 0 || rot % 2 || (rot > 0 && (pos == nullptr || freq == nullptr))) return -1;
+  const int W = R + rot;
+  LatentDecodeParams p{qa, cache, lengths, keep, ld_keep, n_keep, ws, stat, B, H, R, W, (R + 3) / 4 * 4, Tmax, splits, gate_wide, err_word};
+  const QueryTail tail{rot, pos, pos_sb, freq};
   const size_t te = dtype == OSLO_DT_FP32 ? 4 : 2;
   const int v16 = static_cast<int>(16 / te);
   const bool kv = R % v16 == 0 && ldk % v16 == 0 && aligned_to(w_uk, 16);
   const bool vv = R % v16 == 0 && ldv % v16 == 0 && aligned_to(w_uv, 16);
   OSLO_DISPATCH_T(dtype, {
     constexpr int V = 16 / sizeof(T);
-    int rc = kv ? latent_absorb<T, V>(p, q, ldq, w_uk, ldk, qa, dim, scale, stream)
-                : latent_absorb<T, 1>(p, q, ldq, w_uk, ldk, qa, dim, scale, stream);
+    int rc = kv ? latent_absorb<T, V>(p, q, ldq, w_uk, ldk, qa, dim, scale, tail, stream)
+                : latent_absorb<T, 1>(p, q, ldq, w_uk, ldk, qa, dim, scale, tail, stream);
     if (rc) return rc;
-    rc = latent_scan<T>(p, R % 16 == 0 && aligned_to(cache, 16), stream);
+    rc = latent_scan<T>(p, R % 16 == 0 && W % 16 == 0 && aligned_to(cache, 16), stream);
     if (rc) return rc;
     return vv ? latent_finish<T, V>(p, w_uv, ldv, sink, gate, ldg, out, vdim, num_sms, stream)
               : latent_finish<T, 1>(p, w_uv, ldv, sink, gate, ldg, out, vdim, num_sms, stream);

@@ -1,4 +1,4 @@
-// Linear recurrences with a matrix state S (key channels x value channels) per head, in 32-bit floats. Three rules:
+// Linear recurrences with a matrix state S (key channels x value channels) per head, in 32-bit floats. Four rules:
 //
 // RULE_GATED (HGRN2 form): k = (1 - lower) * sigmoid(-(f + f_bias)),  forget gate = 1 - k  (= lower + (1 - lower) * sigmoid(f + f_bias))
 //   S_t = S_{t-1} + k_t (v_t - S_{t-1})   per row of the state (a key channel) and column (a value channel)
@@ -10,6 +10,9 @@
 //   state is multiplied once per period. The period is short enough for 1 / P_t to stay far from overflow, whatever d is.
 // RULE_BONUS (RWKV form): decay w_t = exp(-exp(z_t + w0)) per key channel, o_t = S_{t-1}^T r_t + (r_t . (u k_t)) v_t, then
 //   S_t = diag(w_t) S_{t-1} + k_t v_t^T.
+// RULE_MEMORY (mLSTM form): one decay and one write factor per head and token, S_t = d_t S_{t-1} + w_t k_t [v_t, 1]^T, o_t = S_t^T q_t:
+//   the column after the values is the normaliser. Periods as with RULE_DECAY; their starts, P_t and w_t / P_t come from
+//   matrix_memory.cu. The last block along the columns has little but the normaliser and lets its other warps idle.
 //
 // Prefill (recurrence_kernel): a thread keeps a 16 x 4 tile of S in registers - rows in pairs, so that every update is a
 // packed two-float FMA - and G lanes share a column group; per token it reads 16 + 16 + 4 floats from shared memory,
@@ -32,7 +35,7 @@ namespace cg = cooperative_groups;
 
 namespace oslo {
 
-enum { RULE_GATED = 0, RULE_DECAY = 1, RULE_BONUS = 2 };
+enum { RULE_GATED = 0, RULE_DECAY = 1, RULE_BONUS = 2, RULE_MEMORY = 3 };
 
 typedef unsigned long long f32x2;
 __device__ __forceinline__ f32x2 pack_f2(float lo, float hi) {
@@ -73,14 +76,18 @@ struct RecParams {
   const void *f_bias, *lower;        // [H * dim]; RULE_BONUS: w0 and u
   const float* z; long long ldz;     // RULE_BONUS: decay logits [B * S, H * dim]
   const float* head_decay;           // RULE_DECAY: [H]
+  const float *read, *write, *start; // RULE_MEMORY: [B, H, S] P_t, w_t / P_t, and what the state is multiplied by where a period starts (< 0: nowhere)
+  float q_scale;                     // RULE_MEMORY
+  float* norm;                       // RULE_MEMORY: [B, S, H] the normaliser column's outputs
   const uint8_t* keep; long long ld_keep;   // [B, S], 0 = padding, or nullptr
   const float* s_in;                 // initial states, or nullptr (zero)
   float* s_out;                      // final states, or nullptr
   float* decay;                      // STATE_ONLY: product of the forget gates or decays of the chunk
   float* out;                        // [B, S, H, vdim]
   int B, S, H, dim, vdim;
+  int ncols, lds;                    // columns of a state in use (RULE_MEMORY: vdim + 1, else vdim) and elements per state row
   int chunk, nchunks;                // tokens per chunk; chunks of this launch per batch row
-  float* s_end;                      // last chunk only: final states [B, H, dim, vdim], or nullptr
+  float* s_end;                      // last chunk only: final states [B, H, dim, lds], or nullptr
   long long s_batch, s_chunk;        // element strides of s_in / s_out over batch rows and chunks
   int dim_pad;                       // dim rounded up so that every row of a raw stage starts at a 16-byte boundary
   int vec16;                         // q, f, v (and z) rows and head slices start at 16-byte boundaries
@@ -107,7 +114,9 @@ __global__ void __launch_bounds__(RULE == RULE_BONUS ? 128 : 256, RULE == RULE_B
   float* ws = qs + (STATE_ONLY ? 0 : REC_TB * DP);            // RULE_BONUS: decays
   float* vs = ws + (RULE == RULE_BONUS ? REC_TB * DP : 0);
   __shared__ float bonus_s[RULE == RULE_BONUS && !STATE_ONLY ? REC_TB * PARTS : 1];
-  __shared__ float read_s[RULE == RULE_DECAY ? REC_TB : 1], write_s[RULE == RULE_DECAY ? REC_TB : 1];   // P_t, 1 / P_t
+  constexpr bool PERIODS = RULE == RULE_DECAY || RULE == RULE_MEMORY;
+  __shared__ float read_s[PERIODS ? REC_TB : 1], write_s[PERIODS ? REC_TB : 1];   // P_t, 1 / P_t (RULE_MEMORY: w_t / P_t)
+  __shared__ float start_s[RULE == RULE_MEMORY ? 2 * REC_TB : 1], after_s[2];     // [stage parity]: period starts, P of the last token
   __shared__ float period_s[RULE == RULE_DECAY ? 2 * REC_TB : 1];   // [stage parity][period]: d^(real tokens - 1), negative: none
   const int tid = threadIdx.x, g = tid % G, cgp = tid / G;
   const int h = blockIdx.y;
@@ -123,16 +132,16 @@ __global__ void __launch_bounds__(RULE == RULE_BONUS ? 128 : 256, RULE == RULE_B
 
   // row pair rp of this thread: rows 4 * (g + G * (rp / 2)) + 2 * (rp % 2) and the next one
   f32x2 s[REC_ROWS / 2][REC_COLS];
-  const float* sin = p.s_in ? p.s_in + b * p.s_batch + ch * p.s_chunk + static_cast<long long>(h) * p.dim * p.vdim : nullptr;
+  const float* sin = p.s_in ? p.s_in + b * p.s_batch + ch * p.s_chunk + static_cast<long long>(h) * p.dim * p.lds : nullptr;
 #pragma unroll
   for (int rp = 0; rp < REC_ROWS / 2; ++rp) {
     const int i = 4 * (g + G * (rp / 2)) + 2 * (rp % 2);
 #pragma unroll
     for (int c = 0; c < REC_COLS; ++c) {
       float a0 = 0.f, a1 = 0.f;
-      if (!STATE_ONLY && sin && my_col + c < p.vdim) {
-        if (i < p.dim) a0 = sin[static_cast<long long>(i) * p.vdim + my_col + c];
-        if (i + 1 < p.dim) a1 = sin[static_cast<long long>(i + 1) * p.vdim + my_col + c];
+      if (!STATE_ONLY && sin && my_col + c < p.ncols) {
+        if (i < p.dim) a0 = sin[static_cast<long long>(i) * p.lds + my_col + c];
+        if (i + 1 < p.dim) a1 = sin[static_cast<long long>(i + 1) * p.lds + my_col + c];
       }
       s[rp][c] = pack_f2(a0, a1);
     }
@@ -158,10 +167,15 @@ __global__ void __launch_bounds__(RULE == RULE_BONUS ? 128 : 256, RULE == RULE_B
 #pragma unroll
   for (int off = G / 2, w = REC_COLS; off > 0 && w > 1; off >>= 1, w /= 2)
     if (g & off) first += w / 2;
-  const int out_cols = (G <= REC_COLS || g % (G / REC_COLS > 0 ? G / REC_COLS : 1) == 0) ? min(WIDTH, p.vdim - my_col - first) : 0;
+  const bool writes = G <= REC_COLS || g % (G / REC_COLS > 0 ? G / REC_COLS : 1) == 0;
+  const int out_cols = writes ? min(WIDTH, p.vdim - my_col - first) : 0;
+  const int norm_col = RULE == RULE_MEMORY && writes ? p.vdim - my_col - first : -1;
+  const bool idle = RULE == RULE_MEMORY && col0 + (tid & ~31) / G * REC_COLS >= p.ncols;   // a warp without any column
   const long long out_step = static_cast<long long>(p.H) * p.vdim;
   float* out = STATE_ONLY ? nullptr
                           : p.out + ((static_cast<long long>(b) * p.S + t_begin) * p.H + h) * p.vdim + my_col + first;
+  float* norm = RULE == RULE_MEMORY && !STATE_ONLY ? p.norm + (static_cast<long long>(b) * p.S + t_begin) * p.H + h : nullptr;
+  const long long gates_at = RULE == RULE_MEMORY ? (static_cast<long long>(b) * p.H + h) * p.S : 0;
 
   // raw [REC_TB][raw_ld] stages in the storage type, fetched one step ahead: q (unless STATE_ONLY), f, v slice
   const int f_at = STATE_ONLY ? 0 : p.dim_pad, v_at = f_at + p.dim_pad, raw_ld = v_at + cols;
@@ -240,6 +254,14 @@ __global__ void __launch_bounds__(RULE == RULE_BONUS ? 128 : 256, RULE == RULE_B
         period_s[(it & 1) * REC_TB + s0 / period] = real ? pr : -1.f;
       }
     }
+    if (RULE == RULE_MEMORY && tid < n) {
+      const long long at = gates_at + t0 + tid;
+      const float pr = p.read[at];
+      read_s[tid] = pr * p.q_scale;
+      write_s[tid] = p.write[at];
+      start_s[(it & 1) * REC_TB + tid] = p.start[at];
+      if (tid == n - 1) after_s[it & 1] = pr;
+    }
     __syncthreads();
     const T* src = raw + static_cast<size_t>(it & 1) * REC_TB * raw_ld;
     for (int e = tid; e < DP * CONV; e += nt) {          // CONV threads share a channel's tokens
@@ -252,6 +274,13 @@ __global__ void __launch_bounds__(RULE == RULE_BONUS ? 128 : 256, RULE == RULE_B
           const bool on = real && (p.keep == nullptr || p.keep[b * p.ld_keep + t0 + t]);
           ks[t * DP + i] = on ? write_gate<T>(Num<T>::to(src[t * raw_ld + f_at + i]) + bias, low) : 0.f;
           if (!STATE_ONLY) qs[t * DP + i] = on ? silu_t<T>(Num<T>::to(src[t * raw_ld + i])) : 0.f;
+        }
+      } else if constexpr (RULE == RULE_MEMORY) {
+#pragma unroll 4
+        for (int t = e / DP; t < n; t += CONV) {
+          const bool on = real && (p.keep == nullptr || p.keep[b * p.ld_keep + t0 + t]);
+          ks[t * DP + i] = on ? Num<T>::to(src[t * raw_ld + f_at + i]) * write_s[t] : 0.f;
+          if (!STATE_ONLY) qs[t * DP + i] = on ? Num<T>::to(src[t * raw_ld + i]) * read_s[t] : 0.f;
         }
       } else if constexpr (RULE == RULE_DECAY) {
 #pragma unroll 4
@@ -287,10 +316,23 @@ __global__ void __launch_bounds__(RULE == RULE_BONUS ? 128 : 256, RULE == RULE_B
     for (int e = tid; e < n * cols; e += nt) {
       const int t = e / cols, c = e - t * cols;
       const float v = col0 + c < p.vdim ? Num<T>::to(src[t * raw_ld + v_at + c]) : 0.f;
-      vs[e] = RULE == RULE_DECAY ? silu_t<T>(v) : v;
+      vs[e] = RULE == RULE_DECAY ? silu_t<T>(v) : (RULE == RULE_MEMORY && col0 + c == p.vdim ? 1.f : v);
     }
     __syncthreads();
-    for (int t = 0; t < n; ++t) {
+    for (int t = 0; t < (idle ? 0 : n); ++t) {
+      if constexpr (RULE == RULE_MEMORY) {
+        float f = start_s[(it & 1) * REC_TB + t];
+        if (f >= 0.f) {
+          if (t == 0) f *= pending;                      // what the last stage left; within a stage the starts hold it already
+          const f32x2 f2 = pack_f2(f, f);
+#pragma unroll
+          for (int rp = 0; rp < REC_ROWS / 2; ++rp)
+#pragma unroll
+            for (int c = 0; c < REC_COLS; ++c) s[rp][c] = mul_f2(s[rp][c], f2);
+          if (STATE_ONLY) dec[0] *= f;
+        }
+        if (t == n - 1) pending = after_s[it & 1];
+      }
       if (RULE == RULE_DECAY && (t & (period - 1)) == 0) {    // a period begins: its first real token's decay and what is pending
         const float in_period = period_s[(it & 1) * REC_TB + t / period];
         if (in_period >= 0.f) {
@@ -346,7 +388,7 @@ __global__ void __launch_bounds__(RULE == RULE_BONUS ? 128 : 256, RULE == RULE_B
               const f32x2 d = fma_f2(st, minus1, v2[c]);
               st = fma_f2(k2[u], d, st);
               if (!STATE_ONLY) o2[c] = fma_f2(q2[u], st, o2[c]);
-            } else if (RULE == RULE_DECAY) {
+            } else if (PERIODS) {
               st = fma_f2(k2[u], v2[c], st);
               if (!STATE_ONLY) o2[c] = fma_f2(q2[u], st, o2[c]);
             } else {
@@ -387,11 +429,14 @@ __global__ void __launch_bounds__(RULE == RULE_BONUS ? 128 : 256, RULE == RULE_B
 #pragma unroll
         for (int c = 0; c < WIDTH; ++c)
           if (c < out_cols) out[c] = o[c];
+          else if (RULE == RULE_MEMORY && c == norm_col) *norm = o[c];
         out += out_step;
+        if (RULE == RULE_MEMORY) norm += p.H;
       }
     }
   }
-  if (RULE == RULE_DECAY) {
+  if (PERIODS) {
+    if (RULE == RULE_MEMORY && STATE_ONLY) dec[0] *= pending;
     const f32x2 f2 = pack_f2(pending, pending);
 #pragma unroll
     for (int rp = 0; rp < REC_ROWS / 2; ++rp)
@@ -406,18 +451,18 @@ __global__ void __launch_bounds__(RULE == RULE_BONUS ? 128 : 256, RULE == RULE_B
       for (int c = 0; c < REC_COLS; ++c) {
         float a0, a1;
         unpack_f2(s[rp][c], a0, a1);
-        if (my_col + c < p.vdim) {
-          if (i < p.dim) so[static_cast<long long>(i) * p.vdim + my_col + c] = a0;
-          if (i + 1 < p.dim) so[static_cast<long long>(i + 1) * p.vdim + my_col + c] = a1;
+        if (my_col + c < p.ncols) {
+          if (i < p.dim) so[static_cast<long long>(i) * p.lds + my_col + c] = a0;
+          if (i + 1 < p.dim) so[static_cast<long long>(i + 1) * p.lds + my_col + c] = a1;
         }
       }
     }
   };
   if (p.s_end && ch == p.nchunks - 1) {
-    store_state(p.s_end + (static_cast<long long>(b) * p.H + h) * p.dim * p.vdim);
+    store_state(p.s_end + (static_cast<long long>(b) * p.H + h) * p.dim * p.lds);
   }
   if (p.s_out) {
-    store_state(p.s_out + b * p.s_batch + ch * p.s_chunk + static_cast<long long>(h) * p.dim * p.vdim);
+    store_state(p.s_out + b * p.s_batch + ch * p.s_chunk + static_cast<long long>(h) * p.dim * p.lds);
   }
   if (STATE_ONLY && cgp == 0 && blockIdx.x == 0) {
     float* d = p.decay + ((static_cast<long long>(b) * p.nchunks + ch) * p.H + h) * p.dim;
@@ -426,7 +471,7 @@ __global__ void __launch_bounds__(RULE == RULE_BONUS ? 128 : 256, RULE == RULE_B
 #pragma unroll
       for (int u = 0; u < 4; ++u) {
         const int i = 4 * (g + G * kk) + u;
-        if (i < p.dim) d[i] = RULE == RULE_DECAY ? dec[0] : dec[4 * kk + u];
+        if (i < p.dim) d[i] = PERIODS ? dec[0] : dec[4 * kk + u];
       }
   }
 }
@@ -612,9 +657,11 @@ __global__ void __launch_bounds__(256) recurrence_step_kernel(const StepParams p
   }
 }
 
+static int rec_cols(int vdim, int rule) { return rule == RULE_MEMORY ? vdim + 1 : vdim; }
+
 // threads of a block: the column groups of a head, at most 256 (128 with the bonus rule, whose decays need more registers)
 static int rec_threads(int g, int vdim, int rule) {
-  const int groups = (vdim + REC_COLS - 1) / REC_COLS;
+  const int groups = (rec_cols(vdim, rule) + REC_COLS - 1) / REC_COLS;
   return std::min(rule == RULE_BONUS ? 128 : 256, (groups * g + 31) / 32 * 32);
 }
 
@@ -629,7 +676,7 @@ static int rec_launch(const RecParams& p, cudaStream_t st) {
                                          static_cast<int>(smem));
     if (e != cudaSuccess) return static_cast<int>(e);
   }
-  dim3 grid((p.vdim + cols - 1) / cols, p.H, p.B * p.nchunks);
+  dim3 grid((p.ncols + cols - 1) / cols, p.H, p.B * p.nchunks);
   recurrence_kernel<T, G, STATE_ONLY, RULE><<<grid, nt, smem, st>>>(p);
   return static_cast<int>(cudaGetLastError());
 }
@@ -649,6 +696,7 @@ static int rec_dispatch(const RecParams& p, int rule, cudaStream_t st) {
   if (rule == RULE_GATED) return rec_dispatch_rule<T, STATE_ONLY, RULE_GATED>(p, st);
   if (rule == RULE_DECAY) return rec_dispatch_rule<T, STATE_ONLY, RULE_DECAY>(p, st);
   if (rule == RULE_BONUS) return rec_dispatch_rule<T, STATE_ONLY, RULE_BONUS>(p, st);
+  if (rule == RULE_MEMORY) return rec_dispatch_rule<T, STATE_ONLY, RULE_MEMORY>(p, st);
   return -1;
 }
 
@@ -683,25 +731,19 @@ extern "C" int oslo_recurrence_chunks(int rule, int B, int S, int H, int dim, in
   return best;
 }
 
-// f_bias / lower: the gate bias and lower bound (RULE_GATED), or w0 and u (RULE_BONUS); z: decay logits (RULE_BONUS);
-// head_decay: RULE_DECAY
-extern "C" int oslo_recurrence(int rule, const void* q, long long ldq, const void* f, long long ldf, const void* v, long long ldv,
-                               const void* f_bias, const void* lower, const float* z, long long ldz, const float* head_decay,
-                               const uint8_t* keep, long long ld_keep, float* state, float* out, float* ws, float* decay, int nchunks,
-                               int B, int S, int H, int dim, int vdim, int dtype, cudaStream_t stream) {
+static int run_recurrence(int rule, oslo::RecParams& p, float* state, float* ws, float* decay, int nchunks, int dtype,
+                          cudaStream_t stream) {
   using namespace oslo;
+  const int B = p.B, S = p.S, H = p.H, dim = p.dim, vdim = p.vdim;
   if (B <= 0 || S <= 0 || H <= 0) return 0;
   if (dim <= 0 || vdim <= 0 || dim > 512 || H > 65535 || nchunks < 1 || static_cast<long long>(B) * nchunks > 65535) return -1;
-  RecParams p{};
-  p.q = q; p.f = f; p.v = v; p.ldq = ldq; p.ldf = ldf; p.ldv = ldv; p.f_bias = f_bias; p.lower = lower;
-  p.z = z; p.ldz = ldz; p.head_decay = head_decay;
-  p.keep = keep; p.ld_keep = ld_keep; p.out = out;
-  p.B = B; p.S = S; p.H = H; p.dim = dim; p.vdim = vdim;
-  const long long per = static_cast<long long>(H) * dim * vdim;
+  p.ncols = rec_cols(vdim, rule);
+  p.lds = rule == RULE_MEMORY ? (p.ncols + 3) / 4 * 4 : vdim;
+  const long long per = static_cast<long long>(H) * dim * p.lds;
   const int te = dtype == OSLO_DT_FP32 ? 4 : 2, v16 = 16 / te;
   p.dim_pad = (dim + 7) / 8 * 8;
-  p.vec16 = dim % v16 == 0 && vdim % v16 == 0 && ldq % v16 == 0 && ldf % v16 == 0 && ldv % v16 == 0 && aligned_to(q, 16) &&
-            aligned_to(f, 16) && aligned_to(v, 16) && (rule != RULE_BONUS || (ldz % 4 == 0 && aligned_to(z, 16)));
+  p.vec16 = dim % v16 == 0 && vdim % v16 == 0 && p.ldq % v16 == 0 && p.ldf % v16 == 0 && p.ldv % v16 == 0 && aligned_to(p.q, 16) &&
+            aligned_to(p.f, 16) && aligned_to(p.v, 16) && (rule != RULE_BONUS || (p.ldz % 4 == 0 && aligned_to(p.z, 16)));
   int rc = 0;
   if (nchunks == 1) {
     p.chunk = S; p.nchunks = 1; p.s_in = state; p.s_out = state; p.s_batch = per; p.s_chunk = 0;
@@ -717,13 +759,39 @@ extern "C" int oslo_recurrence(int rule, const void* q, long long ldq, const voi
   OSLO_DISPATCH_T(dtype, { rc = rec_dispatch<T, true>(p, rule, stream); });
   if (rc) return rc;
   recurrence_chunk_scan_kernel<<<dim3(static_cast<unsigned>((per + 255) / 256), B), 256, 0, stream>>>(ws, decay, state, nchunks, H,
-                                                                                                     dim, vdim);
+                                                                                                     dim, p.lds);
   rc = static_cast<int>(cudaGetLastError());
   if (rc) return rc;
   p.nchunks = nchunks;
   p.s_in = ws; p.s_out = nullptr; p.s_end = state;
   OSLO_DISPATCH_T(dtype, { rc = rec_dispatch<T, false>(p, rule, stream); });
   return rc;
+}
+
+// f_bias / lower: the gate bias and lower bound (RULE_GATED), or w0 and u (RULE_BONUS); z: decay logits (RULE_BONUS);
+// head_decay: RULE_DECAY
+extern "C" int oslo_recurrence(int rule, const void* q, long long ldq, const void* f, long long ldf, const void* v, long long ldv,
+                               const void* f_bias, const void* lower, const float* z, long long ldz, const float* head_decay,
+                               const uint8_t* keep, long long ld_keep, float* state, float* out, float* ws, float* decay, int nchunks,
+                               int B, int S, int H, int dim, int vdim, int dtype, cudaStream_t stream) {
+  oslo::RecParams p{};
+  if (rule == oslo::RULE_MEMORY) return -1;
+  p.q = q; p.f = f; p.v = v; p.ldq = ldq; p.ldf = ldf; p.ldv = ldv; p.f_bias = f_bias; p.lower = lower;
+  p.z = z; p.ldz = ldz; p.head_decay = head_decay;
+  p.keep = keep; p.ld_keep = ld_keep; p.out = out;
+  p.B = B; p.S = S; p.H = H; p.dim = dim; p.vdim = vdim;
+  return run_recurrence(rule, p, state, ws, decay, nchunks, dtype, stream);
+}
+
+extern "C" int oslo_memory_recurrence(const void* q, long long ldq, const void* k, long long ldk, const void* v, long long ldv,
+                                      const float* read, const float* write, const float* start, float q_scale, const uint8_t* keep,
+                                      long long ld_keep, float* state, float* out, float* norm, float* ws, float* decay, int nchunks,
+                                      int B, int S, int H, int dim, int vdim, int dtype, cudaStream_t stream) {
+  oslo::RecParams p{};
+  p.q = q; p.f = k; p.v = v; p.ldq = ldq; p.ldf = ldk; p.ldv = ldv; p.read = read; p.write = write; p.start = start; p.q_scale = q_scale;
+  p.keep = keep; p.ld_keep = ld_keep; p.out = out; p.norm = norm;
+  p.B = B; p.S = S; p.H = H; p.dim = dim; p.vdim = vdim;
+  return run_recurrence(oslo::RULE_MEMORY, p, state, ws, decay, nchunks, dtype, stream);
 }
 
 static int step_launch(int rule, oslo::StepParams p, int B, int num_sms, int dtype, cudaStream_t stream) {

@@ -1,10 +1,13 @@
 // Mixture-of-experts feed-forward: routing, the plan that turns (token, choice) pairs into expert-contiguous rows, and the
 // expert products that do not go through the tcgen05 grouped GEMM (oslo_gemm_grouped, gemm_sm100.cu).
 //
-//   route:   z = W_router h + b (32-bit), the `top` largest, softmax over those only
+//   route:   z = W_router h + b (32-bit), the `top` largest, softmax over those only; or scored: s = softmax(W_router h) over
+//            all outputs, the `top` largest s + b, weights s / sum of the chosen s. Outputs past the experts stand for the
+//            input itself: no slot and no product, the step that joins the residual stream knows them
 //   prefill: moe_plan assigns every (token, choice) a slot; an expert's slots are consecutive and start at a multiple of
 //            128, so a 128-row tile of the grouped GEMM belongs to one expert (tile_group); moe_gather copies the rows.
-//            Everything stays on the device: no counts are read back, grids are sized for the worst case.
+//            Everything stays on the device: no counts are read back, grids are sized for the worst case. Units: relu^2,
+//            or silu(gate) * up with the rows of the two matrices in turns, so that a pair of columns is one output.
 //   decode:  a few rows: one warp per output element of the chosen experts, straight from the expert's weights.
 // The down projection leaves one row per slot; the residual join adds them up with their weights.
 #include <cooperative_groups.h>
@@ -55,14 +58,64 @@ __device__ __forceinline__ void pick_top(float* z, int E, int top, int* idx, flo
   }
 }
 
+// z[0..E) become scores, the softmax over all of them; the `top` largest score + b, ties to the lower index; weights: the chosen
+// scores divided by their sum. `ch` [E] is work space. One warp.
+template <typename T>
+__device__ __forceinline__ void pick_scored(float* z, float* ch, const T* b, int E, int top, int* idx, float* wgt, int lane) {
+  float mx = -CUDART_INF_F;
+  for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
+#pragma unroll
+  for (int off = 16; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
+  float sum = 0.f;
+  for (int e = lane; e < E; e += 32) {
+    z[e] = expf(z[e] - mx);
+    sum += z[e];
+  }
+  sum = warp_sum(sum);
+  for (int e = lane; e < E; e += 32) {
+    z[e] = z[e] / sum;
+    ch[e] = z[e] + Num<T>::to(b[e]);
+  }
+  __syncwarp();
+  float tot = 0.f;
+  for (int j = 0; j < top; ++j) {
+    float best = -CUDART_INF_F;
+    int at = E;
+    for (int e = lane; e < E; e += 32) {
+      const float v = ch[e];
+      if (v > best || (at == E && v == best)) { best = v; at = e; }
+    }
+#pragma unroll
+    for (int off = 16; off > 0; off >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, best, off);
+      const int oa = __shfl_xor_sync(0xffffffffu, at, off);
+      if (ov > best || (ov == best && oa < at)) { best = ov; at = oa; }
+    }
+    if (at >= E) at = 0;                               // only NaN logits get here
+    const float s = z[at];
+    tot += s;
+    if (lane == 0) {
+      idx[j] = at;
+      wgt[j] = s;
+    }
+    __syncwarp();
+    if (lane == 0) ch[at] = -CUDART_INF_F;
+    __syncwarp();
+  }
+  if (lane == 0) {
+    const float inv = 1.0f / (tot + 1e-20f);
+    for (int j = 0; j < top; ++j) wgt[j] *= inv;
+  }
+}
+
 // logits from the kernel itself: a cluster of RT_CLUSTER blocks per row shares the experts, the first block collects the
 // logits over distributed shared memory and picks
 constexpr int RT_CLUSTER = 8;
 template <typename T, int VEC>
 __global__ void __cluster_dims__(RT_CLUSTER, 1, 1) __launch_bounds__(256)
 route_kernel(const T* __restrict__ h, long long ldh, const T* __restrict__ w, const T* __restrict__ bias, int* __restrict__ idx,
-             float* __restrict__ wgt, int E, int K, int top) {
-  extern __shared__ float z[];         // [E], used in the first block
+             float* __restrict__ wgt, int E, int K, int top, int scored) {
+  extern __shared__ float z[];         // [E] (scored: and [E] of work space), used in the first block
   cg::cluster_group cluster = cg::this_cluster();
   const int rank = static_cast<int>(cluster.block_rank());
   float* z0 = cluster.map_shared_rank(z, 0);
@@ -81,25 +134,29 @@ route_kernel(const T* __restrict__ h, long long ldh, const T* __restrict__ w, co
       for (int i = 0; i < VEC; ++i) acc = fmaf(a[i], b[i], acc);
     }
     acc = warp_sum(acc);
-    if (lane == 0) z0[e] = acc + Num<T>::to(bias[e]);
+    if (lane == 0) z0[e] = scored ? acc : acc + Num<T>::to(bias[e]);
   }
   cluster.sync();                      // also keeps the first block's shared memory alive until all have written
-  if (rank == 0 && threadIdx.x < 32) pick_top(z, E, top, idx + row * top, wgt + row * top, lane);
+  if (rank == 0 && threadIdx.x < 32) {
+    if (scored) pick_scored<T>(z, z + E, bias, E, top, idx + row * top, wgt + row * top, lane);
+    else pick_top(z, E, top, idx + row * top, wgt + row * top, lane);
+  }
 }
 
 // logits [rows, E] (32-bit, without the bias) from a GEMM: one warp per row
 template <typename T>
 __global__ void __launch_bounds__(128) route_logits_kernel(const float* __restrict__ logits, const T* __restrict__ bias,
                                                            int* __restrict__ idx, float* __restrict__ wgt, long long rows,
-                                                           int E, int top) {
+                                                           int E, int top, int scored) {
   extern __shared__ float rl_smem[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const long long row = static_cast<long long>(blockIdx.x) * 4 + warp;
   if (row >= rows) return;
-  float* z = rl_smem + warp * E;
-  for (int e = lane; e < E; e += 32) z[e] = logits[row * E + e] + Num<T>::to(bias[e]);
+  float* z = rl_smem + warp * E * (scored ? 2 : 1);
+  for (int e = lane; e < E; e += 32) z[e] = scored ? logits[row * E + e] : logits[row * E + e] + Num<T>::to(bias[e]);
   __syncwarp();
-  pick_top(z, E, top, idx + row * top, wgt + row * top, lane);
+  if (scored) pick_scored<T>(z, z + E, bias, E, top, idx + row * top, wgt + row * top, lane);
+  else pick_top(z, E, top, idx + row * top, wgt + row * top, lane);
 }
 
 // counts per expert -> start slot of every expert (multiple of MOE_TILE), expert of every tile, number of tiles
@@ -111,7 +168,8 @@ __global__ void __launch_bounds__(1024) moe_plan_kernel(const int* __restrict__ 
   __shared__ int total;
   for (int e = threadIdx.x; e < E; e += blockDim.x) count[e] = 0;
   __syncthreads();
-  for (long long i = threadIdx.x; i < pairs; i += blockDim.x) atomicAdd(&count[idx[i]], 1);
+  for (long long i = threadIdx.x; i < pairs; i += blockDim.x)
+    if (idx[i] < E) atomicAdd(&count[idx[i]], 1);      // the others are no experts
   __syncthreads();
   if (threadIdx.x == 0) {
     int t = 0;
@@ -135,9 +193,13 @@ __global__ void __launch_bounds__(1024) moe_plan_kernel(const int* __restrict__ 
 template <typename T, int VEC>
 __global__ void __launch_bounds__(128) moe_gather_kernel(const T* __restrict__ h, long long ldh, const int* __restrict__ idx,
                                                          int* __restrict__ cursor, int* __restrict__ slots, T* __restrict__ out,
-                                                         int K, int top, int max_slots) {
+                                                         int K, int top, int max_slots, int E) {
   __shared__ int slot_s;
   const long long pair = blockIdx.x;
+  if (idx[pair] >= E) {                                // no expert, no slot
+    if (threadIdx.x == 0) slots[pair] = -1;
+    return;
+  }
   if (threadIdx.x == 0) {
     slot_s = atomicAdd(&cursor[idx[pair]], 1);
     slots[pair] = slot_s;
@@ -151,11 +213,13 @@ __global__ void __launch_bounds__(128) moe_gather_kernel(const T* __restrict__ h
     *reinterpret_cast<Pack<T, VEC>*>(dst + k) = *reinterpret_cast<const Pack<T, VEC>*>(src + k);
 }
 
+enum { UNIT_NONE = 0, UNIT_RELU2 = 1, UNIT_GLU = 2 };   // GLU: columns in pairs (gate, up), half as many outputs
+
 // scalar grouped product for types and sizes outside the tensor-core path: 32 x 64 outputs per block
 template <typename T>
 __global__ void __launch_bounds__(256) moe_grouped_kernel(const T* __restrict__ a, const T* __restrict__ w, T* __restrict__ out,
                                                           const int* __restrict__ tile_group, const int* __restrict__ n_tiles,
-                                                          int N, int K, int relu2) {
+                                                          int N, int K, int unit) {
   constexpr int BMS = 32, BNS = 64, BKS = 16;
   __shared__ float as[BKS][BMS + 1];
   __shared__ float bs[BKS][BNS + 1];
@@ -192,9 +256,14 @@ __global__ void __launch_bounds__(256) moe_grouped_kernel(const T* __restrict__ 
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx + 16 * j;
-      if (n >= N) continue;
       float v = acc[i][j];
-      if (relu2) { v = fmaxf(v, 0.f); v *= v; }
+      if (unit == UNIT_GLU) {                          // N is even: a pair of columns is in one pair of lanes
+        const float up = __shfl_xor_sync(0xffffffffu, v, 1);
+        if (n < N && (n & 1) == 0) out[static_cast<long long>(m0 + ty * 2 + i) * (N / 2) + n / 2] = Num<T>::from(silu_f(v) * up);
+        continue;
+      }
+      if (n >= N) continue;
+      if (unit == UNIT_RELU2) { v = fmaxf(v, 0.f); v *= v; }
       out[static_cast<long long>(m0 + ty * 2 + i) * N + n] = Num<T>::from(v);
     }
 }
@@ -204,8 +273,9 @@ __global__ void __launch_bounds__(256) moe_grouped_kernel(const T* __restrict__ 
 template <typename T, int VEC>
 __global__ void __launch_bounds__(256, 4) moe_few_kernel(const T* __restrict__ x, long long ldx, const int* __restrict__ idx,
                                                          const T* __restrict__ w, T* __restrict__ out, int N, int K,
-                                                         int per_row, int relu2, int wg) {
+                                                         int per_row, int unit, int wg, int E) {
   __shared__ float red[2][8][4];
+  if (idx[blockIdx.y] >= E) return;                    // no expert: nobody reads the row
   const int pair = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const T* src = x + static_cast<long long>(pair / per_row) * ldx;
   const T* we = w + static_cast<long long>(idx[pair]) * N * K;
@@ -235,11 +305,17 @@ __global__ void __launch_bounds__(256, 4) moe_few_kernel(const T* __restrict__ x
       for (int j = 0; j < 4; ++j) r[warp][j] = acc[j];
     }
     __syncthreads();                   // the other half of `red` is free again: it was read before this barrier
-    if (gw == 0 && lane < nn) {
+    if (gw == 0) {                     // uniform over the warp
       float s = 0.f;
-      for (int g = 0; g < wg; ++g) s += r[warp + g][lane];
-      if (relu2) { s = fmaxf(s, 0.f); s *= s; }
-      out[static_cast<long long>(pair) * N + n0 + lane] = Num<T>::from(s);
+      if (lane < nn)
+        for (int g = 0; g < wg; ++g) s += r[warp + g][lane];
+      if (unit == UNIT_GLU) {
+        const float up = __shfl_xor_sync(0xffffffffu, s, 1);
+        if (lane < nn && (lane & 1) == 0) out[static_cast<long long>(pair) * (N / 2) + (n0 + lane) / 2] = Num<T>::from(silu_f(s) * up);
+      } else if (lane < nn) {
+        if (unit == UNIT_RELU2) { s = fmaxf(s, 0.f); s *= s; }
+        out[static_cast<long long>(pair) * N + n0 + lane] = Num<T>::from(s);
+      }
     }
   }
 }
@@ -247,15 +323,16 @@ __global__ void __launch_bounds__(256, 4) moe_few_kernel(const T* __restrict__ x
 }  // namespace oslo
 
 extern "C" int oslo_moe_route(const void* h, long long ldh, const void* w, const void* bias, const float* logits, int* idx,
-                              float* wgt, long long rows, int E, int K, int top, int dtype, cudaStream_t stream) {
+                              float* wgt, long long rows, int E, int K, int top, int scored, int dtype, cudaStream_t stream) {
   using namespace oslo;
+  const size_t per_row = (scored ? 2 : 1) * E * sizeof(float);
   if (rows <= 0) return 0;
   if (E <= 0 || E > MOE_MAX_EXPERTS || top <= 0 || top > E || rows > 0x7fffffffll) return -1;
   const size_t te = dtype == OSLO_DT_FP32 ? 4 : 2;
   if (logits) {
     OSLO_DISPATCH_T(dtype, {
-      route_logits_kernel<T><<<static_cast<unsigned>((rows + 3) / 4), 128, 4 * E * sizeof(float), stream>>>(
-          logits, static_cast<const T*>(bias), idx, wgt, rows, E, top);
+      route_logits_kernel<T><<<static_cast<unsigned>((rows + 3) / 4), 128, 4 * per_row, stream>>>(
+          logits, static_cast<const T*>(bias), idx, wgt, rows, E, top, scored);
     });
     return static_cast<int>(cudaGetLastError());
   }
@@ -266,11 +343,11 @@ extern "C" int oslo_moe_route(const void* h, long long ldh, const void* w, const
   OSLO_DISPATCH_T(dtype, {
     constexpr int V = 16 / sizeof(T);
     if (vec)
-      route_kernel<T, V><<<grid, 256, E * sizeof(float), stream>>>(static_cast<const T*>(h), ldh, static_cast<const T*>(w),
-                                                                   static_cast<const T*>(bias), idx, wgt, E, K, top);
+      route_kernel<T, V><<<grid, 256, per_row, stream>>>(static_cast<const T*>(h), ldh, static_cast<const T*>(w),
+                                                                   static_cast<const T*>(bias), idx, wgt, E, K, top, scored);
     else
-      route_kernel<T, 1><<<grid, 256, E * sizeof(float), stream>>>(static_cast<const T*>(h), ldh, static_cast<const T*>(w),
-                                                                   static_cast<const T*>(bias), idx, wgt, E, K, top);
+      route_kernel<T, 1><<<grid, 256, per_row, stream>>>(static_cast<const T*>(h), ldh, static_cast<const T*>(w),
+                                                                   static_cast<const T*>(bias), idx, wgt, E, K, top, scored);
   });
   return static_cast<int>(cudaGetLastError());
 }
@@ -289,31 +366,32 @@ extern "C" int oslo_moe_plan(const void* h, long long ldh, const int* idx, int* 
     constexpr int V = 16 / sizeof(T);
     if (vec)
       moe_gather_kernel<T, V><<<static_cast<unsigned>(pairs), 128, 0, stream>>>(
-          static_cast<const T*>(h), ldh, idx, cursor, slots, static_cast<T*>(rows_out), K, top, max_tiles * MOE_TILE);
+          static_cast<const T*>(h), ldh, idx, cursor, slots, static_cast<T*>(rows_out), K, top, max_tiles * MOE_TILE, E);
     else
       moe_gather_kernel<T, 1><<<static_cast<unsigned>(pairs), 128, 0, stream>>>(
-          static_cast<const T*>(h), ldh, idx, cursor, slots, static_cast<T*>(rows_out), K, top, max_tiles * MOE_TILE);
+          static_cast<const T*>(h), ldh, idx, cursor, slots, static_cast<T*>(rows_out), K, top, max_tiles * MOE_TILE, E);
   });
   return static_cast<int>(cudaGetLastError());
 }
 
 extern "C" int oslo_moe_grouped(const void* a, const void* w, void* out, const int* tile_group, const int* n_tiles,
-                                int max_tiles, int N, int K, int relu2, int dtype, cudaStream_t stream) {
+                                int max_tiles, int N, int K, int unit, int dtype, cudaStream_t stream) {
   using namespace oslo;
   if (max_tiles <= 0 || N <= 0) return 0;
+  if (unit == UNIT_GLU && N % 2) return -1;
   if (static_cast<long long>(max_tiles) * (MOE_TILE / 32) > 65535) return -1;
   OSLO_DISPATCH_T(dtype, {
     moe_grouped_kernel<T><<<dim3((N + 63) / 64, max_tiles * (MOE_TILE / 32)), 256, 0, stream>>>(
-        static_cast<const T*>(a), static_cast<const T*>(w), static_cast<T*>(out), tile_group, n_tiles, N, K, relu2);
+        static_cast<const T*>(a), static_cast<const T*>(w), static_cast<T*>(out), tile_group, n_tiles, N, K, unit);
   });
   return static_cast<int>(cudaGetLastError());
 }
 
 extern "C" int oslo_moe_few(const void* x, long long ldx, const int* idx, const void* w, void* out, int pairs, int per_row,
-                            int N, int K, int relu2, int dtype, cudaStream_t stream) {
+                            int N, int K, int unit, int E, int dtype, cudaStream_t stream) {
   using namespace oslo;
   if (pairs <= 0 || N <= 0) return 0;
-  if (pairs > 65535 || per_row < 1) return -1;
+  if (pairs > 65535 || per_row < 1 || (unit == UNIT_GLU && N % 2)) return -1;
   const size_t te = dtype == OSLO_DT_FP32 ? 4 : 2;
   const int v = static_cast<int>(16 / te);
   const bool vec = K % v == 0 && ldx % v == 0 && aligned_to(w, 16) && aligned_to(x, 16);
@@ -326,10 +404,10 @@ extern "C" int oslo_moe_few(const void* x, long long ldx, const int* idx, const 
     constexpr int V = 16 / sizeof(T);
     if (vec)
       moe_few_kernel<T, V><<<grid, 256, 0, stream>>>(static_cast<const T*>(x), ldx, idx, static_cast<const T*>(w),
-                                                     static_cast<T*>(out), N, K, per_row, relu2, wg);
+                                                     static_cast<T*>(out), N, K, per_row, unit, wg, E);
     else
       moe_few_kernel<T, 1><<<grid, 256, 0, stream>>>(static_cast<const T*>(x), ldx, idx, static_cast<const T*>(w),
-                                                     static_cast<T*>(out), N, K, per_row, relu2, wg);
+                                                     static_cast<T*>(out), N, K, per_row, unit, wg, E);
   });
   return static_cast<int>(cudaGetLastError());
 }

@@ -17,6 +17,7 @@
                                   // (max, sum exp(x - max), logit of the row's label if it lies in the block)
 #define GEMM_FLAG_CE_GRAD 512     // LM head + cross-entropy, backward: D = (exp(x - lse[row]) - [col == label]) * scale[row]
 #define GEMM_FLAG_RELU2 1024      // square of relu
+#define GEMM_FLAG_GLU 2048        // columns in pairs (gate, up): silu(gate) * up, half as many output columns; N is even, ldd >= N / 2
 #define GEMM_CE_BLOCK 128         // columns per statistics record
 
 #define OSLO_DT_BF16 0
@@ -125,7 +126,9 @@ int oslo_flash_sink_fwd_sm100(const void* q, const void* k, const void* v, void*
                               const void* gate, long long ldg, int B, int H, int G, int Sq, int Sk, int dim, int vdim,
                               long long q_sb, long long q_sh, long long q_ss, long long k_sb, long long k_sh, long long k_ss,
                               long long v_sb, long long v_sh, long long v_ss, long long o_sb, long long o_sh, long long o_ss,
-                              float scale, float softcap, int dtype, int* err_word, cudaStream_t stream);
+                              float scale, float softcap, int window, int keep_first, const int* lead, int gate_wide,
+                              const void* q2, long long q2_sb, long long q2_sh, long long q2_ss, const void* k2, long long k2_sb,
+                              long long k2_ss, int rot, int dtype, int* err_word, cudaStream_t stream);
 int oslo_flash_bwd(const void* q, const void* k, const void* v, const void* o, const void* dout, const float* lse,
                    float* delta, float* dq_acc, void* dq, void* dk, void* dv, const uint8_t* kpm, int B, int H,
                    int Sq, int Sk, int D, long long q_sb, long long q_sh, long long q_ss, long long k_sb,
@@ -225,8 +228,18 @@ int oslo_branch_join(const float* x, int n, const void* const* y, const long lon
                      float mult, float eps, const void* w1, const void* w2, float* x_out, void* h1, void* h2, long long rows,
                      int cols, int dtype, cudaStream_t stream);
 // out = o / rms(runs of `group` columns) * w * act(gate); act 0: sigmoid, 1: silu; o fp32 [rows, cols]
-int oslo_gated_rms_norm(const float* o, const void* w, const void* gate, long long ldg, void* out, long long rows, int cols,
-                        int group, float eps, int act, int dtype, cudaStream_t stream);
+// z, m [rows, cols / group] (or null): the runs are first divided by max(|z|, exp(-m)) + 1e-6
+int oslo_gated_rms_norm(const float* o, const void* w, const void* gate, long long ldg, void* out, const float* z, const float* m,
+                        long long rows, int cols, int group, float eps, int act, int dtype, cudaStream_t stream);
+
+// residual streams (hyper_connections.cu): x [rows, n, cols] fp32 with row and stream strides, x_out contiguous, h [rows, cols].
+// y null: the streams stay. weights null: y has one row per token, else y = sum_j weights[t, j] * row, which is y's row slots[t, j]
+// (null: t * top + j) or, where choice[t, j] >= experts, own's row t. shared null or added times sigmoid(gate). w_in null: ones
+int oslo_hyper_join(const float* x, long long x_row, long long x_stream, const void* y, long long ldy, const int* slots,
+                    const float* weights, int top, const int* choice, int experts, const void* own, long long ld_own,
+                    const void* shared, long long ld_shared, const void* gate, long long ld_gate, const void* w_out, const void* mix,
+                    const void* w_in, const void* w_norm, float* x_out, void* h, long long rows, int n, int cols, float eps,
+                    float scale, int dtype, cudaStream_t stream);
 
 // linear recurrences (linear_recurrence.cu): q, f [B * S, H * dim], v [B * S, H * vdim] with row strides; keep [B, S]
 // (0 = padding) or null; state [B, H, dim, vdim] fp32, read and updated, or null; out fp32 [B, S, H, vdim].
@@ -254,6 +267,21 @@ int oslo_bonus_step(const void* r, long long ldr, const void* k, long long ldk, 
                     long long ldg, const uint8_t* keep, long long ld_keep, float* state, void* out, float eps, int B, int H, int dim,
                     int vdim, int num_sms, int dtype, cudaStream_t stream);
 
+// rule 3 (matrix memory): state [B, H, dim, lds], lds = vdim + 1 rounded up to a multiple of 4, column vdim the normaliser; read,
+// write, start [B, H, S] of oslo_memory_gates; norm [B, S, H]; ws [B, nchunks, H, dim, lds]
+int oslo_memory_recurrence(const void* q, long long ldq, const void* k, long long ldk, const void* v, long long ldv, const float* read,
+                           const float* write, const float* start, float q_scale, const uint8_t* keep, long long ld_keep, float* state,
+                           float* out, float* norm, float* ws, float* decay, int nchunks, int B, int S, int H, int dim, int vdim,
+                           int dtype, cudaStream_t stream);
+// matrix_memory.cu: z fp32 [B * S, 2 H], bias [2 H], top [B, H] (read and updated) or null, m_out [B, S, H]
+int oslo_memory_gates(const float* z, long long ldz, const void* bias, float cap, const uint8_t* keep, long long ld_keep, float* top,
+                      float* read, float* write, float* start, float* m_out, int B, int S, int H, int dtype, cudaStream_t stream);
+// one token per row: gates from x [B, width], memory, normaliser, head norms with norm_w [H * vdim], sigmoid(gate)
+int oslo_memory_step(const void* q, long long ldq, const void* k, long long ldk, const void* v, long long ldv, const void* x, long long ldx,
+                     int width, const void* w, const void* bias, float cap, const void* gate, long long ldg, const void* norm_w,
+                     const uint8_t* keep, long long ld_keep, float* state, float* top, void* out, float q_scale, float eps, int B, int H,
+                     int dim, int vdim, int num_sms, int dtype, cudaStream_t stream);
+
 // latent attention (latent_attention.cu). sink_gate: flash output [B, S, H, *] + lse [B, H, S] -> out [B * S, H * vdim]
 int oslo_sink_gate(const void* o, long long o_sb, long long o_ss, long long o_sh, const float* lse, const void* sink,
                    const void* gate, long long ldg, void* out, int B, int S, int H, int vdim, int dtype, cudaStream_t stream);
@@ -262,33 +290,43 @@ int oslo_sink_gate(const void* o, long long o_sb, long long o_ss, long long o_sh
 int oslo_sink_attention(const void* q, long long q_sb, long long q_ss, long long q_sh, const void* k, long long k_sb,
                         long long k_ss, long long k_sh, const void* v, long long v_sb, long long v_ss, long long v_sh,
                         const uint8_t* keep, long long ld_keep, const void* sink, const void* gate, long long ldg, void* out,
-                        int B, int H, int G, int Sq, int Sk, int dim, int vdim, float scale, float softcap, int dtype,
-                        cudaStream_t stream);
-// decode: RMS norm of the query latent -> cq_out; of the key-value latent (null: none) -> cache [B, Tmax, kv_rank] at lengths[b]
+                        int B, int H, int G, int Sq, int Sk, int dim, int vdim, float scale, float softcap, int window,
+                        int keep_first, const int* lead, int gate_wide, int dtype, cudaStream_t stream);
+// rows b * S + t: RMS norm of the query latent -> cq_out; of the key-value latent (null: none) -> cache [B, Tmax, kv_rank + rot] at
+// lengths[b] + t, followed by the rot columns after it, rotated (halves) by pos[b, t] * freq; c_out (null: none) [B * S, kv_rank]
+// gets the normed latents once more
 int oslo_latent_prep(const void* cq, long long ldq, const void* wq, int q_rank, void* cq_out, const void* ckv, long long ldkv,
-                     const void* wkv, int kv_rank, void* cache, const int* lengths, int Tmax, float eps, int B, int dtype,
+                     const void* wkv, int kv_rank, void* cache, const int* lengths, int Tmax, float eps, int B, int S, int rot,
+                     const long long* pos, long long pos_sb, long long pos_ss, const float* freq, void* c_out, int dtype,
                      int* err_word, cudaStream_t stream);
-// one query per row over a latent cache; fp32 workspaces qa [B, H, R], ws [B, H, splits, R rounded up to
-// a multiple of 4] and stat [B, H, splits, 2]
+// in place: the last rot dims of every head of q [B * S, H * (dim + rot)] (contiguous) turn by pos[b, t] * freq, halves paired
+int oslo_rotate_halves(void* q, const long long* pos, long long pos_sb, long long pos_ss, const float* freq, int B, int S, int H,
+                       int dim, int rot, int dtype, cudaStream_t stream);
+// one query per row, q [B, H * (dim + rot)], over a latent cache [B, Tmax, R + rot]; the query's last rot dims are rotated by pos[b] *
+// freq; sink null: none; gate_wide: a gate per output element; fp32 workspaces qa [B, H, R + rot], ws [B, H, splits, R rounded up
+// to a multiple of 4] and stat [B, H, splits, 2]
 int oslo_latent_decode(const void* q, long long ldq, const void* w_uk, long long ldk, const void* w_uv, long long ldv,
                        const void* cache, const int* lengths, const uint8_t* keep, long long ld_keep, int n_keep,
                        const void* sink, const void* gate, long long ldg, float* qa, float* ws, float* stat, void* out,
-                       int B, int H, int dim, int vdim, int R, int Tmax, int splits, float scale, int num_sms, int dtype,
-                       int* err_word, cudaStream_t stream);
+                       int B, int H, int dim, int vdim, int R, int rot, const long long* pos, long long pos_sb, const float* freq,
+                       int gate_wide, int Tmax, int splits, float scale, int num_sms, int dtype, int* err_word,
+                       cudaStream_t stream);
 int oslo_latent_splits(int B, int H, int T, int num_sms);
 
-// grouped-query attention (grouped_attention.cu). qkv_prep: RMS norm of every query / key head (weights wq, wk [dim]), rotation of
+// grouped-query attention (grouped_attention.cu). qkv_prep: RMS norm of every query / key head (weights wq, wk [dim] or null), rotation of
 // the first 2 * n_freq dims by pos[b, t] * freq, q -> q_out [B, S, H, dim], k / v -> caches [B, G, Tmax, *] at lengths[b] + t
 int oslo_qkv_prep(const void* q, long long ldq, const void* k, long long ldk, const void* v, long long ldv, const void* wq,
                   const void* wk, float eps, const long long* pos, long long pos_sb, long long pos_ss, const float* freq, int n_freq,
                   void* q_out, void* kc, void* vc, const int* lengths, int B, int S, int H, int G, int dim, int vdim, int Tmax,
                   int dtype, int* err_word, cudaStream_t stream);
 // one query per row: q [B, H, dim], caches [B, G, Tmax, *], of which lengths[b] positions count; keep [B, n_keep] (0 = padded) or
-// null; fp32 workspaces ws [B, H, splits, vdim rounded up to a multiple of 4] and stat [B, H, splits, 2]; out [B, H * vdim]
+// null; sink null: none; gate null or [B, H]; window > 0: the last `window` positions and the first keep_first after lead[b] (null: 0)
+// are read; fp32 workspaces ws [B, H, splits, vdim rounded up to a multiple of 4] and stat [B, H, splits, 2]; out [B, H * vdim]
 int oslo_grouped_splits(int B, int H, int G, int T, int dim, int vdim, int dtype, int num_sms);
 int oslo_grouped_decode(const void* q, const void* kc, const void* vc, const int* lengths, const uint8_t* keep, long long ld_keep,
-                        int n_keep, const void* sink, float* ws, float* stat, void* out, int B, int H, int G, int dim, int vdim,
-                        int Tmax, int splits, float scale, float softcap, int dtype, int* err_word, cudaStream_t stream);
+                        int n_keep, const void* sink, const void* gate, long long ldg, int window, int keep_first, const int* lead,
+                        float* ws, float* stat, void* out, int B, int H, int G, int dim, int vdim, int Tmax, int splits,
+                        float scale, float softcap, int dtype, int* err_word, cudaStream_t stream);
 
 // token shift, causal convolution and selective scan (selective_scan.cu)
 // out[i] = h + (h' - h) * mu[i], i < P; prev fp32 [B, width] (the row before the first; read and updated) or null
@@ -311,14 +349,17 @@ int oslo_scan_step(const void* x, long long ldx, const void* dt, long long lddt,
                    cudaStream_t stream);
 
 // mixture of experts (moe.cu, grouped GEMM in gemm_sm100.cu)
+// route: idx, wgt [rows, top]; scored: scores are the softmax over all E outputs, bias only enters the choice, weights are the chosen
+// scores over their sum. Choices >= the experts of plan / few get no slot (-1) and no product. unit: 0 none, 1 relu^2, 2 silu(gate) *
+// up of column pairs (out has N / 2 columns)
 int oslo_moe_route(const void* h, long long ldh, const void* w, const void* bias, const float* logits, int* idx, float* wgt,
-                   long long rows, int E, int K, int top, int dtype, cudaStream_t stream);
+                   long long rows, int E, int K, int top, int scored, int dtype, cudaStream_t stream);
 int oslo_moe_plan(const void* h, long long ldh, const int* idx, int* cursor, int* tile_group, int* n_tiles, int* slots,
                   void* rows_out, long long pairs, int E, int K, int top, int max_tiles, int dtype, cudaStream_t stream);
 int oslo_moe_grouped(const void* a, const void* w, void* out, const int* tile_group, const int* n_tiles, int max_tiles, int N,
-                     int K, int relu2, int dtype, cudaStream_t stream);
+                     int K, int unit, int dtype, cudaStream_t stream);
 int oslo_moe_few(const void* x, long long ldx, const int* idx, const void* w, void* out, int pairs, int per_row, int N, int K,
-                 int relu2, int dtype, cudaStream_t stream);
+                 int unit, int E, int dtype, cudaStream_t stream);
 int oslo_gemm_grouped(const void* A, const void* B, void* D, int M, int N, int K, int groups, const int* group_of_tile,
                       const int* group_tiles, int flags, int* err_word, int num_sms, cudaStream_t stream);
 

@@ -1,7 +1,8 @@
 // RMS norms with 32-bit arithmetic and the step that joins a sublayer to the residual stream.
 //
 //   rms_norm:      out = x / sqrt(mean(x^2) + eps) * (offset + w)        offset 1: the weight is stored around zero
-//   gated_rms_norm: out = o / sqrt(mean(o^2 of a run of columns) + eps) * w * act(gate)
+//   gated_rms_norm: out = o / sqrt(mean(o^2 of a run of columns) + eps) * w * act(gate); the runs may first be divided by
+//                  max(|z|, exp(-m)) + 1e-6, one z and m per run
 //   branch_join:   x'  = x + mult * sum of the (possibly normed) results of parallel branches
 //                  h_i = x' / sqrt(mean(x'^2) + eps) * w_i, i = 1, 2    the inputs of the next layer's branches
 //   residual_join: z   = y * sigmoid(gate + gate_bias)
@@ -256,6 +257,7 @@ __device__ __forceinline__ void gate_run(const float* o, const T* w, const T* ga
 template <typename T, int VEC, int LANES>
 __global__ void __launch_bounds__(256) gated_rms_norm_kernel(const float* __restrict__ o, const T* __restrict__ w,
                                                              const T* __restrict__ gate, long long ldg, T* __restrict__ out,
+                                                             const float* __restrict__ z, const float* __restrict__ m,
                                                              long long runs, int cols, int group, float eps, int act) {
   __shared__ float red[32];
   constexpr bool WARP = LANES > 0;
@@ -285,7 +287,8 @@ __global__ void __launch_bounds__(256) gated_rms_norm_kernel(const float* __rest
     ss = block_sum(ss, red);
   }
   if (!real) return;
-  const float r = 1.0f / sqrtf(ss / group + eps);
+  const float inv = z ? 1.0f / (fmaxf(fabsf(z[run]), expf(-m[run])) + 1e-6f) : 1.0f;
+  const float r = inv / sqrtf(inv * inv * (ss / group) + eps);
   for (int c = lane * VEC; c < group; c += step * VEC) gate_run<T, VEC>(o, w, gate, out, c, r, act);
 }
 
@@ -433,11 +436,12 @@ extern "C" int oslo_branch_join(const float* x, int n, const void* const* y, con
   return static_cast<int>(cudaGetLastError());
 }
 
-extern "C" int oslo_gated_rms_norm(const float* o, const void* w, const void* gate, long long ldg, void* out, long long rows,
-                                   int cols, int group, float eps, int act, int dtype, cudaStream_t stream) {
+extern "C" int oslo_gated_rms_norm(const float* o, const void* w, const void* gate, long long ldg, void* out, const float* z,
+                                   const float* m, long long rows, int cols, int group, float eps, int act, int dtype,
+                                   cudaStream_t stream) {
   using namespace oslo;
   if (rows <= 0 || cols <= 0) return 0;
-  if (group <= 0 || cols % group) return -1;
+  if (group <= 0 || cols % group || (z == nullptr) != (m == nullptr)) return -1;
   const long long runs = rows * (cols / group);
   if (runs > 0x7fffffffll) return -1;
   const size_t te = dtype == OSLO_DT_FP32 ? 4 : 2;
@@ -445,7 +449,7 @@ extern "C" int oslo_gated_rms_norm(const float* o, const void* w, const void* ga
                    aligned_to(out, 4 * te);
 #define GATED_LAUNCH(V, L, BLOCKS)                                                                  \
   gated_rms_norm_kernel<T, V, L><<<static_cast<unsigned>(BLOCKS), 256, 0, stream>>>(                \
-      o, static_cast<const T*>(w), static_cast<const T*>(gate), ldg, static_cast<T*>(out), runs, cols, group, eps, act)
+      o, static_cast<const T*>(w), static_cast<const T*>(gate), ldg, static_cast<T*>(out), z, m, runs, cols, group, eps, act)
 #define GATED_GO(V)                                                         \
   if (group <= 8 * V) GATED_LAUNCH(V, 8, (runs + 31) / 32);                 \
   else if (group <= 16 * V) GATED_LAUNCH(V, 16, (runs + 15) / 16);          \

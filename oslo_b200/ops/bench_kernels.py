@@ -196,12 +196,12 @@ def bench_mixers(args, timer: _Timer) -> None:
         idx, wgt = co.moe_route(hb, rw, rb, top)
         slots, rows, tg, nt = ext.moe_plan(hb, idx, e)
         report(case, "prompt plan + gather", lambda: ext.moe_plan(hb, idx, e), gbytes=n * w * (1 + top) * 2 / 1e9, like="layer norm")
-        report(case, "prompt experts up", lambda: ext.moe_grouped(rows, up, tg, nt, True), tflop=2.0 * n * top * w * ff / 1e12,
+        report(case, "prompt experts up", lambda: ext.moe_grouped(rows, up, tg, nt, 1), tflop=2.0 * n * top * w * ff / 1e12,
                gbytes=(n * top * (w + ff) + e * w * ff) * 2 / 1e9, like="MLP GEMM (GPT-J)")
-        a = ext.moe_grouped(rows, up, tg, nt, True)
-        report(case, "prompt experts down", lambda: ext.moe_grouped(a, down, tg, nt, False), tflop=2.0 * n * top * w * ff / 1e12,
+        a = ext.moe_grouped(rows, up, tg, nt, 1)
+        report(case, "prompt experts down", lambda: ext.moe_grouped(a, down, tg, nt, 0), tflop=2.0 * n * top * w * ff / 1e12,
                gbytes=(n * top * (w + ff) + e * w * ff) * 2 / 1e9, like="MLP GEMM (GPT-J)")
-        ye = ext.moe_grouped(a, down, tg, nt, False)
+        ye = ext.moe_grouped(a, down, tg, nt, 0)
         report(case, "prompt residual join of experts", lambda: ext.residual_join(x, ye, slots, wgt, gate, vec, vec, vec, 1e-5),
                gbytes=n * w * (4 + 2 * top + 2 + 4 + 2) / 1e9, like="layer norm")
         wm = mk(top * ff, w)

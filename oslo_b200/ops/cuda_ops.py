@@ -742,8 +742,59 @@ def clamped_glu(gate: Tensor, up: Tensor, limit: float, alpha: float) -> Tensor:
     return _ext().clamped_glu(_rows(gate), _rows(up), float(limit), float(alpha))
 
 
-def gated_rms_norm(o: Tensor, w: Tensor, gate: Tensor, eps: float, group: int, act: str) -> Tensor:
-    return _ext().gated_rms_norm(o.contiguous(), w, _rows(gate), float(eps), int(group), {"sigmoid": 0, "silu": 1}[act])
+def gated_rms_norm(o: Tensor, w: Tensor, gate: Tensor, eps: float, group: int, act: str, normalizer=None) -> Tensor:
+    z, m = (None, None) if normalizer is None else (t.contiguous() for t in normalizer)
+    return _ext().gated_rms_norm(o.contiguous(), w, _rows(gate), float(eps), int(group), {"sigmoid": 0, "silu": 1}[act], z, m)
+
+
+HYPER_MAX_TOP = 64     # rows per token that the stream join adds up
+HYPER_MAX_STREAMS = 16
+
+
+def hyper_join(x: Tensor, result, w_out: Optional[Tensor], mix: Optional[Tensor], w_in: Optional[Tensor], w_norm: Tensor, eps: float,
+               scale: float):
+    r = result if result is not None else ref.SublayerResult(None)
+    if x.size(1) > HYPER_MAX_STREAMS or (r.weights is not None and r.weights.size(1) > HYPER_MAX_TOP):
+        return ref.hyper_join(x, result, w_out, mix, w_in, w_norm, eps, scale)
+    rows = lambda t: None if t is None else _rows(t)                                       # noqa: E731
+    xo, h = _ext().hyper_join(x if x.stride(-1) == 1 else x.contiguous(), rows(r.y), r.slots, r.weights, r.choice, int(r.experts),
+                              rows(r.h), rows(r.shared), rows(r.shared_gate), w_out, mix, w_in, w_norm, float(eps), float(scale))
+    return (xo if result is not None else x), h
+
+
+def matrix_memory(q: Tensor, k: Tensor, v: Tensor, z: Tensor, bias: Tensor, cap: float, keep: Optional[Tensor],
+                  state: Optional[Tensor], top: Optional[Tensor], batch: int, heads: int):
+    dim, vdim = q.size(1) // heads, v.size(1) // heads
+    q, k, v, keep, scale = _rows(q), _rows(k), _rows(v), _keep8(keep), dim ** -0.5
+    read, write, start, m = _ext().memory_gates(_rows(z), bias, float(cap), keep, top, batch)
+    run = lambda a, b, s, d: _ext().memory_recurrence(a, b, v, read, write, start, scale, keep, s, batch, heads, d, vdim)   # noqa: E731
+    if dim <= RECURRENCE_MAX_DIM:
+        o, n = run(q, k, state, dim)
+        return o, n, m
+    o = n = 0.0                                            # key channels are independent of one another
+    for a in range(0, dim, RECURRENCE_MAX_DIM):
+        b = min(dim, a + RECURRENCE_MAX_DIM)
+        cut = lambda t: t.reshape(-1, heads, dim)[:, :, a:b].reshape(t.size(0), -1)        # noqa: E731
+        part = state[:, :, a:b].contiguous() if state is not None else None
+        more_o, more_n = run(cut(q), cut(k), part, b - a)
+        o, n = o + more_o, n + more_n
+        if state is not None:
+            state[:, :, a:b] = part
+    return o, n, m
+
+
+MEMORY_STEP_MAX = 46 * 1024 - 4096   # bytes of shared memory that a step's key channels may take
+
+
+def memory_step(q: Tensor, k: Tensor, v: Tensor, x: Tensor, w: Tensor, bias: Tensor, cap: float, gate: Tensor, norm_w: Tensor,
+                keep: Optional[Tensor], state: Tensor, top: Tensor, eps: float, heads: int) -> Tensor:
+    """Decode step: gates from the mixer's input ``x``, memory, normaliser, head norms and output gate in one launch."""
+    dim, vdim = q.size(1) // heads, v.size(1) // heads
+    if 12 * dim > MEMORY_STEP_MAX:
+        o, n, m = matrix_memory(q, k, v, linear_fp32(x, w), bias, cap, keep, state, top, q.size(0), heads)
+        return gated_rms_norm(o, norm_w, gate, eps, vdim, "sigmoid", (n, m))
+    return _ext().memory_step(_rows(q), _rows(k), _rows(v), _rows(x), w, bias, float(cap), _rows(gate), norm_w, _keep8(keep), state, top,
+                              dim ** -0.5, float(eps), heads, dim, vdim)
 
 
 def token_shift(h: Tensor, mu: Tensor, batch: int, keep: Optional[Tensor], prev: Optional[Tensor]) -> Tensor:
@@ -773,17 +824,20 @@ def scan_step(x: Tensor, dt: Tensor, w_dt: Tensor, dt_bias: Tensor, a_log: Tenso
     return _ext().scan_step(_rows(x), _rows(dt), w_dt, dt_bias, a_log, _rows(b), _rows(c), d, _rows(z), _keep8(keep), state)
 
 
-def qkv_prep(q: Tensor, k: Tensor, v: Tensor, wq: Tensor, wk: Tensor, eps: float, positions: Tensor, freq: Tensor, k_store: Tensor,
-             v_store: Tensor, lengths: Tensor) -> Tensor:
-    """Head norms and rotation of queries and keys; keys and values go into the caches at ``lengths[row]``. Returns ``[B, S, H, dim]``."""
+def qkv_prep(q: Tensor, k: Tensor, v: Tensor, wq: Optional[Tensor], wk: Optional[Tensor], eps: float, positions: Tensor, freq: Tensor,
+             k_store: Tensor, v_store: Tensor, lengths: Tensor) -> Tensor:
+    """Head norms (weights or ``None``) and rotation of queries and keys; keys and values go into the caches at ``lengths[row]``. Returns
+    ``[B, S, H, dim]``."""
     return _ext().qkv_prep(_rows(q), _rows(k), _rows(v), wq, wk, float(eps), positions, freq, k_store, v_store, lengths)
 
 
-def grouped_decode(q: Tensor, k: Tensor, v: Tensor, lengths: Tensor, keep: Optional[Tensor], sink: Tensor, scale: float,
-                   softcap: float) -> Tensor:
+def grouped_decode(q: Tensor, k: Tensor, v: Tensor, lengths: Tensor, keep: Optional[Tensor], sink: Optional[Tensor], scale: float,
+                   softcap: float, gate: Optional[Tensor] = None, window: int = 0, keep_first: int = 0,
+                   lead: Optional[Tensor] = None) -> Tensor:
     if v.size(-1) > GROUPED_MAX_VDIM:
-        return ref.grouped_decode(q, k, v, lengths, keep, sink, scale, softcap)
-    return _ext().grouped_decode(q.contiguous(), k, v, lengths, _keep8(keep), sink, float(scale), float(softcap))
+        return ref.grouped_decode(q, k, v, lengths, keep, sink, scale, softcap, gate, window, keep_first, lead)
+    return _ext().grouped_decode(q.contiguous(), k, v, lengths, _keep8(keep), sink, float(scale), float(softcap),
+                                 None if gate is None else _rows(gate), int(window), int(keep_first), lead)
 
 
 def flash_head_dim(dim: int, vdim: int) -> int:
@@ -796,54 +850,83 @@ def pad_heads(t: Tensor, d: int) -> Tensor:
     return t if t.size(-1) == d else torch.nn.functional.pad(t, (0, d - t.size(-1)))
 
 
-def sink_attention(q: Tensor, k: Tensor, v: Tensor, keep: Optional[Tensor], sink: Tensor, gate: Optional[Tensor], scale: float,
-                   softcap: float = 0.0) -> Tensor:
-    """``q`` ``[B, Sq, H, dim]``, ``k``/``v`` ``[B, Sk, G, *]``. 16-bit heads run on the tcgen05 flash kernel, with sink, gate and cap
-    in its softmax and epilogue (gated value sizes that are no multiple of 8: zero-padded heads, sink and gate from its
-    log-sum-exp); everything else in the fp32 kernel."""
+def flash_parts_fit(dim: int, rot: int, vdim: int) -> bool:
+    """Whether the tcgen05 flash kernel runs heads of ``dim`` + ``rot`` query and key dimensions from two operands."""
+    return dim % 8 == 0 and rot % 8 == 0 and vdim % 8 == 0 and -(-dim // 64) + -(-rot // 64) <= 4 and vdim <= 256
+
+
+def sink_attention(q: Tensor, k: Tensor, v: Tensor, keep: Optional[Tensor], sink: Optional[Tensor], gate: Optional[Tensor], scale: float,
+                   softcap: float = 0.0, window: int = 0, keep_first: int = 0, lead: Optional[Tensor] = None,
+                   q_rot: Optional[Tensor] = None, k_rot: Optional[Tensor] = None) -> Tensor:
+    """``q`` ``[B, Sq, H, dim]``, ``k``/``v`` ``[B, Sk, G, *]``. 16-bit heads run on the tcgen05 flash kernel, with sink, gate, cap and
+    window in its softmax and epilogue, and a second operand for the key part that heads share (gated value sizes that are no
+    multiple of 8: zero-padded heads, sink and gate from its log-sum-exp); everything else in the fp32 kernel."""
     dim, vdim = q.size(-1), v.size(-1)
     d = flash_head_dim(dim, vdim)
-    if q.dtype in _16BIT and d and q.size(1) > 1:
+    mask = (int(window), int(keep_first), lead)
+    flash = q.dtype in _16BIT and d and q.size(1) > 1
+    gate = None if gate is None else _rows(gate)
+    if flash and gate is not None and gate.size(1) != q.size(2):
+        gate = _attn_operand(gate)                         # a gate per element is read in 16-byte pieces
+    if q_rot is not None:
+        if flash and not softcap and flash_parts_fit(dim, q_rot.size(-1), vdim):
+            kpm = _keep8(keep).contiguous() if keep is not None else None
+            qh, kh, vh, q2 = (_attn_operand(t.permute(0, 2, 1, 3)) for t in (q, k, v, q_rot))
+            return _ext().flash_sink_fwd(qh, kh, vh, kpm, sink, gate, float(scale), 0.0, *mask, q2, _attn_operand(k_rot))
+        q = torch.cat([q, q_rot], dim=-1)
+        k = torch.cat([k, k_rot.unsqueeze(2).expand(-1, -1, k.size(2), -1)], dim=-1)
+        return sink_attention(q, k, v, keep, sink, gate, scale, softcap, *mask)
+    if flash:
         kpm = _keep8(keep).contiguous() if keep is not None else None
         if dim % 8 == 0 and vdim % 8 == 0:
             qh, kh, vh = (_attn_operand(t.permute(0, 2, 1, 3)) for t in (q, k, v))
-            return _ext().flash_sink_fwd(qh, kh, vh, kpm, sink, None if gate is None else _rows(gate), float(scale), float(softcap))
-        if gate is not None and not softcap and k.size(2) == q.size(2):
+            return _ext().flash_sink_fwd(qh, kh, vh, kpm, sink, gate, float(scale), float(softcap), *mask)
+        if (gate is not None and sink is not None and gate.size(1) == q.size(2) and not softcap and not window
+                and k.size(2) == q.size(2)):
             qh, kh, vh = (_attn_operand(pad_heads(t, d).permute(0, 2, 1, 3)) for t in (q, k, v))
             o, lse = _ext().flash_fwd(qh, kh, vh, float(scale), True, 0, kpm, _flash_impl())
-            return _ext().sink_gate(o, lse, sink, _rows(gate), vdim)
-    return _ext().sink_attention(*(t if t.stride(-1) == 1 else t.contiguous() for t in (q, k, v)), _keep8(keep), sink,
-                                 None if gate is None else _rows(gate), float(scale), float(softcap))
+            return _ext().sink_gate(o, lse, sink, gate, vdim)
+    return _ext().sink_attention(*(t if t.stride(-1) == 1 else t.contiguous() for t in (q, k, v)), _keep8(keep), sink, gate,
+                                 float(scale), float(softcap), *mask)
 
 
 def latent_prep(cq: Tensor, wq: Tensor, ckv: Optional[Tensor], wkv: Optional[Tensor], cache: Optional[Tensor], lengths: Tensor,
-                eps: float) -> Tensor:
-    """Decode step: the normed query latent; the normed key-value latent goes into ``cache`` at position ``lengths[row]``."""
-    return _ext().latent_prep(_rows(cq), wq, None if ckv is None else _rows(ckv), wkv, cache, lengths, float(eps))
+                eps: float, positions: Optional[Tensor] = None, freq: Optional[Tensor] = None, rows: bool = False):
+    """The normed query latents; the normed key-value latents, and behind them what ``ckv`` has besides, rotated, go into ``cache`` at
+    position ``lengths[row]`` and on. ``rows``: also the normed key-value latents as rows."""
+    return _ext().latent_prep(_rows(cq), wq, None if ckv is None else _rows(ckv), wkv, cache, lengths, float(eps), positions, freq, rows)
 
 
-def latent_decode(q: Tensor, w_uk: Tensor, w_uv: Tensor, cache: Tensor, lengths: Tensor, keep: Optional[Tensor], sink: Tensor,
-                  gate: Tensor, scale: float, heads: int) -> Tensor:
+def rotate_halves_(q: Tensor, positions: Tensor, freq: Tensor) -> Tensor:
+    """The last ``2 * len(freq)`` dims of ``q`` ``[B, S, heads, dim]`` rotated in place."""
+    return _ext().rotate_halves_(q, positions, freq)
+
+
+def latent_decode(q: Tensor, w_uk: Tensor, w_uv: Tensor, cache: Tensor, lengths: Tensor, keep: Optional[Tensor],
+                  sink: Optional[Tensor], gate: Tensor, scale: float, heads: int, positions: Optional[Tensor] = None,
+                  freq: Optional[Tensor] = None) -> Tensor:
     return _ext().latent_decode(_rows(q), w_uk, w_uv, cache, lengths.to(torch.int32), _keep8(keep), sink, _rows(gate),
-                                float(scale), heads)
+                                float(scale), heads, positions, freq)
 
 
+MOE_UNITS = {None: 0, "relu2": 1, "silu": 2}
 MOE_FEW_PAIRS = 8   # (token, choice) pairs up to which the chosen experts' weights are streamed per pair
 
 
-def moe_route(h: Tensor, w: Tensor, bias: Tensor, top: int):
+def moe_route(h: Tensor, w: Tensor, bias: Tensor, top: int, scored: bool = False):
     logits = None
     if h.size(0) > SMALL_M_ROWS and gemm_ok(h, w) and h.size(1) % 8 == 0 and (w.size(0) < 32 or w.size(0) % 4 == 0):
         logits = gemm(h, w, flags=FLAG_OUT_FP32)           # 16-bit operands, exact products, fp32 sums and output
     elif h.size(0) > 65535:                                # no tensor-core path for these sizes or types: 32-bit library product
         logits = torch.matmul(h.float(), w.float().t())
-    return _ext().moe_route(_rows(h), w, bias, logits, top)
+    return _ext().moe_route(_rows(h), w, bias, logits, top, scored)
 
 
-def moe_experts(h: Tensor, idx: Tensor, up: Tensor, down: Tensor):
+def moe_experts(h: Tensor, idx: Tensor, up: Tensor, down: Tensor, unit: str = "relu2"):
+    u = MOE_UNITS[unit]
     if idx.numel() <= MOE_FEW_PAIRS:
-        a = _ext().moe_few(_rows(h), idx, up, idx.size(1), True)
-        return _ext().moe_few(a, idx, down, 1, False), None
+        a = _ext().moe_few(_rows(h), idx, up, idx.size(1), u)
+        return _ext().moe_few(a, idx, down, 1, 0), None
     slots, rows, tile_group, n_tiles = _ext().moe_plan(_rows(h), idx, up.size(0))
-    a = _ext().moe_grouped(rows, up, tile_group, n_tiles, True)
-    return _ext().moe_grouped(a, down, tile_group, n_tiles, False), slots
+    a = _ext().moe_grouped(rows, up, tile_group, n_tiles, u)
+    return _ext().moe_grouped(a, down, tile_group, n_tiles, 0), slots

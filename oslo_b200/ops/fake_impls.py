@@ -199,23 +199,27 @@ def register() -> None:
         return o.new_empty((o.size(0) * o.size(2), o.size(1) * vdim))
 
     @reg("oslo_b200::flash_sink_fwd")
-    def _(q, k, v, kpm, sink, gate, scale, softcap):
+    def _(q, k, v, kpm, sink, gate, scale, softcap, window=0, keep_first=0, lead=None, q2=None, k2=None):
         return q.new_empty((q.size(0) * q.size(2), q.size(1) * v.size(3)))
 
     @reg("oslo_b200::sink_attention")
-    def _(q, k, v, keep, sink, gate, scale, softcap):
+    def _(q, k, v, keep, sink, gate, scale, softcap, window=0, keep_first=0, lead=None):
         return q.new_empty((q.size(0) * q.size(1), q.size(2) * v.size(3)))
 
     @reg("oslo_b200::latent_prep")
-    def _(cq, wq, ckv, wkv, cache, lengths, eps):
-        return cq.new_empty(cq.shape)
+    def _(cq, wq, ckv, wkv, cache, lengths, eps, positions=None, freq=None, rows=False):
+        return cq.new_empty(cq.shape), cq.new_empty((cq.size(0) if rows and ckv is not None else 0, 0 if wkv is None else wkv.numel()))
+
+    @reg("oslo_b200::rotate_halves_")
+    def _(q, positions, freq):
+        return q
 
     @reg("oslo_b200::latent_decode")
-    def _(q, w_uk, w_uv, cache, lengths, keep, sink, gate, scale, heads):
+    def _(q, w_uk, w_uv, cache, lengths, keep, sink, gate, scale, heads, positions=None, freq=None):
         return q.new_empty((q.size(0), w_uv.size(0)))
 
     @reg("oslo_b200::moe_route")
-    def _(h, w, bias, logits, top):
+    def _(h, w, bias, logits, top, scored=False):
         return h.new_empty((h.size(0), top), dtype=torch.int32), h.new_empty((h.size(0), top), dtype=torch.float32)
 
     @reg("oslo_b200::moe_plan")
@@ -224,12 +228,12 @@ def register() -> None:
         return (torch.empty_like(idx), h.new_empty((tiles * 128, h.size(1))), idx.new_empty((tiles,)), idx.new_empty((1,)))
 
     @reg("oslo_b200::moe_grouped")
-    def _(rows, w, tile_group, n_tiles, relu2):
-        return rows.new_empty((rows.size(0), w.size(1)))
+    def _(rows, w, tile_group, n_tiles, unit):
+        return rows.new_empty((rows.size(0), w.size(1) // (2 if unit == 2 else 1)))
 
     @reg("oslo_b200::moe_few")
-    def _(x, idx, w, per_row, relu2):
-        return x.new_empty((idx.numel(), w.size(1)))
+    def _(x, idx, w, per_row, unit):
+        return x.new_empty((idx.numel(), w.size(1) // (2 if unit == 2 else 1)))
 
     @reg("oslo_b200::clamped_glu")
     def _(gate, up, limit, alpha):
@@ -242,8 +246,26 @@ def register() -> None:
                 y0.new_empty((rows if w2 is not None else 0, cols)))
 
     @reg("oslo_b200::gated_rms_norm")
-    def _(o, w, gate, eps, group, act):
+    def _(o, w, gate, eps, group, act, z=None, m=None):
         return w.new_empty(o.shape)
+
+    @reg("oslo_b200::hyper_join")
+    def _(x, y, slots, weights, choice, experts, own, shared, gate, w_out, mix, w_in, w_norm, eps, scale):
+        rows, n, cols = x.shape
+        return x.new_empty((rows if y is not None else 0, n, cols)), w_norm.new_empty((rows, cols))
+
+    @reg("oslo_b200::memory_gates")
+    def _(z, bias, cap, keep, top, batch):
+        heads, s = z.size(1) // 2, z.size(0) // batch
+        return (*(z.new_empty((batch, heads, s)) for _ in range(3)), z.new_empty((z.size(0), heads)))
+
+    @reg("oslo_b200::memory_recurrence")
+    def _(q, k, v, read, write, start, q_scale, keep, state, batch, heads, dim, vdim, chunks=0):
+        return q.new_empty((q.size(0), heads * vdim), dtype=torch.float32), q.new_empty((q.size(0), heads), dtype=torch.float32)
+
+    @reg("oslo_b200::memory_step")
+    def _(q, k, v, x, w, bias, cap, gate, norm_w, keep, state, top, q_scale, eps, heads, dim, vdim):
+        return q.new_empty((q.size(0), heads * vdim))
 
     @reg("oslo_b200::gemv_stacked")
     def _(x, w):
@@ -270,7 +292,7 @@ def register() -> None:
         return q.new_empty((kc.size(0), q.size(0) // kc.size(0), q.size(1) // kc.size(3), kc.size(3)))
 
     @reg("oslo_b200::grouped_decode")
-    def _(q, kc, vc, lengths, keep, sink, scale, softcap):
+    def _(q, kc, vc, lengths, keep, sink, scale, softcap, gate=None, window=0, keep_first=0, lead=None):
         return q.new_empty((q.size(0), q.size(1) * vc.size(3)))
 
     @reg("oslo_b200::token_shift")

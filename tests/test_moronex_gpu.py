@@ -153,7 +153,7 @@ def test_latent_prep_norms_and_appends():
         wq, wk = rnd(128, dtype=dtype), rnd(72, dtype=dtype)
         cache = torch.zeros(3, 9, 72, dtype=dtype, device="cuda")
         lengths = torch.full((3,), 4, dtype=torch.int32, device="cuda")
-        got = cuda_ops.latent_prep(p[:, 8:136], wq, p[:, 200:272], wk, cache, lengths, 1e-5)
+        got, _ = cuda_ops.latent_prep(p[:, 8:136], wq, p[:, 200:272], wk, cache, lengths, 1e-5)
         close(got, ref.rms_norm(p[:, 8:136], wq, 1e-5), dtype)
         close(cache[:, 4], ref.rms_norm(p[:, 200:272], wk, 1e-5), dtype)
         cache[:, 4] = 0

@@ -111,3 +111,15 @@ def write_model(directory, cfg, tensors):
     with open(os.path.join(directory, "config.json"), "w") as f:
         json.dump(cfg, f)
     save_file({k: v.contiguous() for k, v in tensors.items()}, os.path.join(directory, "model.safetensors"))
+
+
+def steady(tensors):
+    """The same model without a router's close calls, for comparisons in 16-bit: corrections far apart choose, scores only weigh."""
+    out = dict(tensors)
+    for name, t in tensors.items():
+        if name.endswith("mlp.correction"):
+            g = torch.Generator().manual_seed(t.numel())
+            out[name] = (1.5 * torch.randperm(t.numel(), generator=g)).to(t.dtype)
+        elif ".mlp.e" in name or ".mlp.shared." in name:
+            out[name] = 0.7 * t
+    return out

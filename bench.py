@@ -68,7 +68,7 @@ def parse_args():
     ap.add_argument("--no-e2e", action="store_true")
     ap.add_argument("--mode", default="train", choices=["train", "decode", "fusion", "serving"],
                     help="train: tokens/s of a training step; decode: ms/token of greedy generation with a KV cache; "
-                         "serving: prompt and decode throughput of Moronex and Begovik beside GPT-J at equal width, heads and layers; "
+                         "serving: prompt and decode throughput of Moronex, Begovik and Dekutar beside GPT-J at equal width, heads and layers; "
                          "fusion: seconds of one GPT-2 small beam-search generate() call before and after fuse() (the "
                          "benchmark behind the reference's published numbers)")
     ap.add_argument("--fusion-dtype", default="fp32", choices=["fp32", "bf16"],
@@ -607,10 +607,25 @@ def begovik_config(width, heads, layers, vocab=50400):
                 layers=[{"type": kinds[i % 3][0], "mixer": kinds[i % 3][1], "mlp": mlp} for i in range(layers)])
 
 
+def dekutar_config(width, heads, layers, q_rank, kv_rank, experts, vocab=50400):
+    """Layers in groups of three: attention in a window of 512 (4 query heads per key / value head), matrix memory, latent attention
+    with 64 rotated dims; four residual streams; four gated experts of the router's (4 of its outputs are the identity) and a shared
+    one, each with a fourth of GPT-J's MLP weights."""
+    dim, ff = width // heads, 2 * width // 3 // 64 * 64
+    mlp = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "identity": 4, "top": 4}, "shared": {"ff": ff}}
+    kinds = [("attention", {"heads": heads, "kv_heads": max(1, heads // 4), "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+                            "mask": {"size": 512, "keep_first": 16}, "rot": {"base": 10000.0, "dims": dim}}),
+             ("mlstm", {"heads": heads, "dim": dim, "vdim": dim, "gate_cap": 15.0}),
+             ("latent_attention", {"heads": heads, "dim": dim, "rot_dim": 64, "vdim": dim, "q_rank": q_rank, "kv_rank": kv_rank,
+                                   "scale": (dim + 64) ** -0.5, "rot": {"base": 10000.0, "dims": 64}})]
+    return dict(vocab=vocab, width=width, norm={"eps": 1e-6}, embedding={"scale": 3.0}, streams=4, logit_scale=0.5,
+                layers=[{"type": kinds[i % 3][0], "mixer": kinds[i % 3][1], "mlp": mlp} for i in range(layers)])
+
+
 def serving_main(args) -> None:
     """One GPU, random weights, bf16: prompt throughput (4 x 2048 tokens) and greedy decoding after 2048-token prompts with 1, 8
-    and 64 sequences (one CUDA-graph replay per token) of Moronex, Begovik and GPT-J with the same width, heads and number of
-    layers. A "step" is one ``GraphedGreedyDecoder.generate`` call; CUDA events around its prompt and its token loop; weights
+    and 64 sequences (one CUDA-graph replay per token) of Moronex, Begovik, Dekutar and GPT-J with the same width, heads and
+    number of layers. A "step" is one ``GraphedGreedyDecoder.generate`` call; CUDA events around its prompt and its token loop; weights
     and caches are larger than L2. ``--layers`` shortens both models (debug)."""
     import gc
 
@@ -629,8 +644,11 @@ def serving_main(args) -> None:
     l0, results = ext.launch_count(), {}
     for size, (width, heads, layers, q_rank, kv_rank, experts) in SERVING_SIZES.items():
         layers = args.layers or layers
-        for name in ("moronex", "begovik", "gptj"):
-            if name == "begovik":
+        for name in ("moronex", "begovik", "dekutar", "gptj"):
+            if name == "dekutar":
+                cls, cfg = ob.DekutarForCausalLM, ob.DekutarConfig(**dekutar_config(width, heads, layers, q_rank, kv_rank, experts),
+                                                                   torch_dtype=torch.bfloat16)
+            elif name == "begovik":
                 cls, cfg = ob.BegovikForCausalLM, ob.BegovikConfig(**begovik_config(width, heads, layers), torch_dtype=torch.bfloat16)
             elif name == "moronex":
                 cls, cfg = ob.MoronexForCausalLM, ob.MoronexConfig(**serving_config(width, heads, layers, q_rank, kv_rank, experts),
@@ -676,7 +694,7 @@ def serving_main(args) -> None:
         "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
         "ms_per_step": 4 * 2048 / main_rec["prompt_tokens_per_s"] * 1e3, "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
         "dtype": "bf16", "data": "synthetic uniform token ids, random-init weights", "impl": "oslo_b200",
-        "config": {"model": "moronex and begovik beside gptj", "global_batch": 4, "seq_len": 2048, "parallelism": "single",
+        "config": {"model": "moronex, begovik and dekutar beside gptj", "global_batch": 4, "seq_len": 2048, "parallelism": "single",
                    "sizes": {k: dict(zip(("width", "heads", "layers", "q_rank", "kv_rank", "experts"), v)) for k, v in SERVING_SIZES.items()},
                    "l2": "weights + caches per step >> 126 MB L2, no explicit flush"},
         "results": results, "clocks": clocks, "e2e": None, "gpu_launches": ext.launch_count() - l0,

@@ -240,15 +240,19 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
                              (p.causal && n0 + BN - 1 > q0 + offset) ||
                              (p.window > 0 && n0 <= q0 + FA_BM - 1 + offset - p.window);
       if (need_mask) {
+        // one bit per column: up to `last`, and from `first` on or before `kept`
         const int qpos = row + offset;
+        const int last = p.causal ? min(p.Sk - 1, qpos) : p.Sk - 1;
+        const int first = p.window > 0 ? qpos - p.window + 1 : 0, kept = p.window > 0 ? lead + p.keep_first : 0;
+        auto below = [](int n) { return n <= 0 ? 0u : (n >= 32 ? 0xffffffffu : (1u << n) - 1u); };
 #pragma unroll
-        for (int i = 0; i < BN; ++i) {
-          const int col = n0 + i;
-          bool vis = col < p.Sk;
-          if (p.causal && col > qpos) vis = false;
-          if (p.window > 0 && col <= qpos - p.window && col - lead >= p.keep_first) vis = false;
-          if (vis && kpm_row && !kpm_row[col]) vis = false;
-          if (!vis) s[i] = -CUDART_INF_F;
+        for (int c0 = 0; c0 < BN; c0 += 32) {
+          const int base = n0 + c0;
+          uint32_t vis = below(last - base + 1) & (~below(first - base) | below(kept - base));
+          if (kpm_row) vis &= __ballot_sync(0xffffffffu, base + lane < p.Sk && kpm_row[base + lane] != 0);
+#pragma unroll
+          for (int i = 0; i < 32; ++i)
+            if (!((vis >> i) & 1u)) s[c0 + i] = -CUDART_INF_F;
         }
       }
       // four independent chains: one thread per row means nothing else hides the latency of a 64-long dependent chain

@@ -179,8 +179,8 @@ struct LatentPrepParams {
 };
 
 // block (0, row b * S + t): RMS norm of the query latent; block (1, row): RMS norm of the key-value latent and rotation of the key
-// part behind it, written to the cache at position lengths[b] + t
-template <typename T>
+// part behind it, written to the cache at position lengths[b] + t. VEC 4: rows and sizes are aligned to four elements
+template <typename T, int VEC>
 __global__ void __launch_bounds__(256) latent_prep_kernel(const LatentPrepParams p) {
   __shared__ float red[32];
   const long long row = blockIdx.x;
@@ -209,34 +209,43 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const LatentPrepParams
     }
   }
   float ss = 0.f;
-  for (int c = threadIdx.x; c < n; c += blockDim.x) {
-    const float v = Num<T>::to(x[c]);
-    ss = fmaf(v, v, ss);
+  for (int c = threadIdx.x * VEC; c < n; c += blockDim.x * VEC) {
+    float v[VEC];
+    load_vec<T, VEC>(x + c, v);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) ss = fmaf(v[i], v[i], ss);
   }
   ss = block_sum(ss, red);
   const float r = 1.0f / sqrtf(ss / n + p.eps);
-  for (int c = threadIdx.x; c < n; c += blockDim.x) {
-    const T v = Num<T>::from(Num<T>::to(x[c]) * r * Num<T>::to(w[c]));
-    out[c] = v;
-    if (again) again[c] = v;
+  for (int c = threadIdx.x * VEC; c < n; c += blockDim.x * VEC) {
+    float v[VEC], g[VEC];
+    load_vec<T, VEC>(x + c, v);
+    load_vec<T, VEC>(w + c, g);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[i] *= r * g[i];
+    store_vec<T, VEC>(out + c, v);
+    if (again) store_vec<T, VEC>(again + c, v);
   }
 }
 
-// in place, a thread per pair of the last rot dims of a head
-template <typename T>
+// in place: a thread turns VEC neighbouring pairs of one head's last rot dims; block = (rows, heads x groups of pairs)
+template <typename T, int VEC>
 __global__ void __launch_bounds__(256) rotate_halves_kernel(T* __restrict__ q, const long long* __restrict__ pos, long long pos_sb,
-                                                            long long pos_ss, const float* __restrict__ freq, long long pairs, int S,
-                                                            int H, int dim, int rot) {
+                                                            long long pos_ss, const float* __restrict__ freq, int S, int H, int dim,
+                                                            int rot, int per_head) {
   const int half = rot / 2;
-  for (long long e = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; e < pairs;
-       e += static_cast<long long>(gridDim.x) * blockDim.x) {
-    const int i = static_cast<int>(e % half);
-    const long long head = e / half, row = head / H, b = row / S, t = row - b * S;
-    T* at = q + head * (dim + rot) + dim + i;
-    float u = Num<T>::to(at[0]), v = Num<T>::to(at[half]);
-    turn(static_cast<float>(pos[b * pos_sb + t * pos_ss]) * freq[i], u, v);
-    at[0] = Num<T>::from(u);
-    at[half] = Num<T>::from(v);
+  const long long row = blockIdx.x, b = row / S, t = row - b * S;
+  const float at = static_cast<float>(pos[b * pos_sb + t * pos_ss]);
+  for (int e = threadIdx.x; e < H * per_head; e += blockDim.x) {
+    const int h = e / per_head, i = (e - h * per_head) * VEC;
+    T* p = q + (row * H + h) * (dim + rot) + dim + i;
+    float u[VEC], v[VEC];
+    load_vec<T, VEC>(p, u);
+    load_vec<T, VEC>(p + half, v);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) turn(at * freq[i + j], u[j], v[j]);
+    store_vec<T, VEC>(p, u);
+    store_vec<T, VEC>(p + half, v);
   }
 }
 
@@ -917,19 +926,32 @@ extern "C" int oslo_latent_prep(const void* cq, long long ldq, const void* wq, i
   if (rows > 0x7fffffffll || rot < 0 || rot % 2 || (rot > 0 && (pos == nullptr || freq == nullptr))) return -1;
   const LatentPrepParams p{cq, wq, ldq, q_rank, cq_out, ckv, wkv, ldkv, kv_rank, rot, cache, c_out, lengths, pos, pos_sb, pos_ss,
                            freq, S, Tmax, eps, err_word};
-  const int threads = std::max(q_rank, kv_rank) <= 128 && rows > 64 ? 64 : 256;
-  OSLO_DISPATCH_T(dtype, { latent_prep_kernel<T><<<dim3(static_cast<unsigned>(rows), ckv ? 2 : 1), threads, 0, stream>>>(p); });
+  const size_t a4 = dtype == OSLO_DT_FP32 ? 16 : 8;
+  bool vec = q_rank % 4 == 0 && kv_rank % 4 == 0 && rot % 4 == 0 && ldq % 4 == 0 && ldkv % 4 == 0;
+  for (const void* t : {cq, wq, static_cast<const void*>(cq_out), ckv, wkv, static_cast<const void*>(cache), static_cast<const void*>(c_out)})
+    vec = vec && aligned_to(t, a4);        // null is aligned
+  const int widest = std::max(q_rank, kv_rank) / (vec ? 4 : 1), threads = widest <= 64 ? 64 : (widest <= 128 ? 128 : 256);
+  const dim3 grid(static_cast<unsigned>(rows), ckv ? 2 : 1);
+  OSLO_DISPATCH_T(dtype, {
+    if (vec) latent_prep_kernel<T, 4><<<grid, threads, 0, stream>>>(p);
+    else latent_prep_kernel<T, 1><<<grid, threads, 0, stream>>>(p);
+  });
   return static_cast<int>(cudaGetLastError());
 }
 
 extern "C" int oslo_rotate_halves(void* q, const long long* pos, long long pos_sb, long long pos_ss, const float* freq, int B, int S,
                                   int H, int dim, int rot, int dtype, cudaStream_t stream) {
   using namespace oslo;
-  const long long pairs = static_cast<long long>(B) * S * H * (rot / 2);
-  if (pairs <= 0) return 0;
-  const unsigned blocks = static_cast<unsigned>(std::min<long long>((pairs + 255) / 256, 148 * 32));
+  const long long rows = static_cast<long long>(B) * S;
+  if (rows <= 0 || H <= 0 || rot <= 0) return 0;
+  if (rows > 0x7fffffffll || rot % 2) return -1;
+  const size_t a4 = dtype == OSLO_DT_FP32 ? 16 : 8;
+  const bool vec = rot % 8 == 0 && dim % 4 == 0 && aligned_to(q, a4);
+  const int per_head = rot / 2 / (vec ? 4 : 1);
+  const unsigned grid = static_cast<unsigned>(rows), threads = std::min(256, (H * per_head + 31) / 32 * 32);
   OSLO_DISPATCH_T(dtype, {
-    rotate_halves_kernel<T><<<blocks, 256, 0, stream>>>(static_cast<T*>(q), pos, pos_sb, pos_ss, freq, pairs, S, H, dim, rot);
+    if (vec) rotate_halves_kernel<T, 4><<<grid, threads, 0, stream>>>(static_cast<T*>(q), pos, pos_sb, pos_ss, freq, S, H, dim, rot, per_head);
+    else rotate_halves_kernel<T, 1><<<grid, threads, 0, stream>>>(static_cast<T*>(q), pos, pos_sb, pos_ss, freq, S, H, dim, rot, per_head);
   });
   return static_cast<int>(cudaGetLastError());
 }

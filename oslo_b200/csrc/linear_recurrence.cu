@@ -12,7 +12,8 @@
 //   S_t = diag(w_t) S_{t-1} + k_t v_t^T.
 // RULE_MEMORY (mLSTM form): one decay and one write factor per head and token, S_t = d_t S_{t-1} + w_t k_t [v_t, 1]^T, o_t = S_t^T q_t:
 //   the column after the values is the normaliser. Periods as with RULE_DECAY; their starts, P_t and w_t / P_t come from
-//   matrix_memory.cu. The last block along the columns has little but the normaliser and lets its other warps idle.
+//   matrix_memory.cu. The first block along the columns also keeps the normaliser, a channel per thread in shared memory: after the
+//   conversions of a stage its n . q take two FMAs per channel and token and one reduction over the warp per eight tokens.
 //
 // Prefill (recurrence_kernel): a thread keeps a 16 x 4 tile of S in registers - rows in pairs, so that every update is a
 // packed two-float FMA - and G lanes share a column group; per token it reads 16 + 16 + 4 floats from shared memory,
@@ -85,7 +86,7 @@ struct RecParams {
   float* decay;                      // STATE_ONLY: product of the forget gates or decays of the chunk
   float* out;                        // [B, S, H, vdim]
   int B, S, H, dim, vdim;
-  int ncols, lds;                    // columns of a state in use (RULE_MEMORY: vdim + 1, else vdim) and elements per state row
+  int lds;                           // elements per state row: vdim; RULE_MEMORY: vdim + 1 and padding, column vdim the normaliser
   int chunk, nchunks;                // tokens per chunk; chunks of this launch per batch row
   float* s_end;                      // last chunk only: final states [B, H, dim, lds], or nullptr
   long long s_batch, s_chunk;        // element strides of s_in / s_out over batch rows and chunks
@@ -117,6 +118,7 @@ __global__ void __launch_bounds__(RULE == RULE_BONUS ? 128 : 256, RULE == RULE_B
   constexpr bool PERIODS = RULE == RULE_DECAY || RULE == RULE_MEMORY;
   __shared__ float read_s[PERIODS ? REC_TB : 1], write_s[PERIODS ? REC_TB : 1];   // P_t, 1 / P_t (RULE_MEMORY: w_t / P_t)
   __shared__ float start_s[RULE == RULE_MEMORY ? 2 * REC_TB : 1], after_s[2];     // [stage parity]: period starts, P of the last token
+  __shared__ float n_s[RULE == RULE_MEMORY ? DP : 1], dot_s[RULE == RULE_MEMORY && !STATE_ONLY ? 2 * 8 * REC_TB : 1];   // normaliser; [stage parity][warp][token]
   __shared__ float period_s[RULE == RULE_DECAY ? 2 * REC_TB : 1];   // [stage parity][period]: d^(real tokens - 1), negative: none
   const int tid = threadIdx.x, g = tid % G, cgp = tid / G;
   const int h = blockIdx.y;
@@ -139,7 +141,7 @@ __global__ void __launch_bounds__(RULE == RULE_BONUS ? 128 : 256, RULE == RULE_B
 #pragma unroll
     for (int c = 0; c < REC_COLS; ++c) {
       float a0 = 0.f, a1 = 0.f;
-      if (!STATE_ONLY && sin && my_col + c < p.ncols) {
+      if (!STATE_ONLY && sin && my_col + c < p.vdim) {
         if (i < p.dim) a0 = sin[static_cast<long long>(i) * p.lds + my_col + c];
         if (i + 1 < p.dim) a1 = sin[static_cast<long long>(i + 1) * p.lds + my_col + c];
       }
@@ -169,12 +171,15 @@ __global__ void __launch_bounds__(RULE == RULE_BONUS ? 128 : 256, RULE == RULE_B
     if (g & off) first += w / 2;
   const bool writes = G <= REC_COLS || g % (G / REC_COLS > 0 ? G / REC_COLS : 1) == 0;
   const int out_cols = writes ? min(WIDTH, p.vdim - my_col - first) : 0;
-  const int norm_col = RULE == RULE_MEMORY && writes ? p.vdim - my_col - first : -1;
-  const bool idle = RULE == RULE_MEMORY && col0 + (tid & ~31) / G * REC_COLS >= p.ncols;   // a warp without any column
   const long long out_step = static_cast<long long>(p.H) * p.vdim;
   float* out = STATE_ONLY ? nullptr
                           : p.out + ((static_cast<long long>(b) * p.S + t_begin) * p.H + h) * p.vdim + my_col + first;
-  float* norm = RULE == RULE_MEMORY && !STATE_ONLY ? p.norm + (static_cast<long long>(b) * p.S + t_begin) * p.H + h : nullptr;
+  // the normaliser: channel i of this head by thread i % blockDim.x; warps without a channel skip it
+  const bool has_norm = RULE == RULE_MEMORY && blockIdx.x == 0;
+  const int norm_warps = min(nt, DP + 31) / 32;
+  float* norm = has_norm && !STATE_ONLY ? p.norm + (static_cast<long long>(b) * p.S + t_begin) * p.H + h : nullptr;
+  if (has_norm)
+    for (int i = tid; i < DP; i += nt) n_s[i] = !STATE_ONLY && sin && i < p.dim ? sin[static_cast<long long>(i) * p.lds + p.vdim] : 0.f;
   const long long gates_at = RULE == RULE_MEMORY ? (static_cast<long long>(b) * p.H + h) * p.S : 0;
 
   // raw [REC_TB][raw_ld] stages in the storage type, fetched one step ahead: q (unless STATE_ONLY), f, v slice
@@ -231,7 +236,8 @@ __global__ void __launch_bounds__(RULE == RULE_BONUS ? 128 : 256, RULE == RULE_B
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   if (t_begin < t_end) fetch(t_begin, 0);
-  for (int t0 = t_begin, it = 0; t0 < t_end; t0 += REC_TB, ++it) {
+  int it = 0;
+  for (int t0 = t_begin; t0 < t_end; t0 += REC_TB, ++it) {
     const int n = min(REC_TB, t_end - t0);
     if (t0 + REC_TB < t_end) {                         // every thread read the other stage before the last barrier
       fetch(t0 + REC_TB, (it + 1) & 1);
@@ -316,10 +322,54 @@ __global__ void __launch_bounds__(RULE == RULE_BONUS ? 128 : 256, RULE == RULE_B
     for (int e = tid; e < n * cols; e += nt) {
       const int t = e / cols, c = e - t * cols;
       const float v = col0 + c < p.vdim ? Num<T>::to(src[t * raw_ld + v_at + c]) : 0.f;
-      vs[e] = RULE == RULE_DECAY ? silu_t<T>(v) : (RULE == RULE_MEMORY && col0 + c == p.vdim ? 1.f : v);
+      vs[e] = RULE == RULE_DECAY ? silu_t<T>(v) : v;
+    }
+    if (RULE == RULE_MEMORY && !STATE_ONLY && has_norm && it > 0 && tid < REC_TB) {     // the last stage's n . q
+      float a = 0.f;
+      for (int w = 0; w < norm_warps; ++w) a += dot_s[((it - 1) & 1) * 8 * REC_TB + w * REC_TB + tid];
+      norm[static_cast<long long>((it - 1) * REC_TB + tid) * p.H] = a;
     }
     __syncthreads();
-    for (int t = 0; t < (idle ? 0 : n); ++t) {
+    if (RULE == RULE_MEMORY && has_norm && tid / 32 < norm_warps) {
+#pragma unroll 1
+      for (int h0 = 0; h0 < n; h0 += 8) {
+        float a[8];
+#pragma unroll
+        for (int u = 0; u < 8; ++u) a[u] = 0.f;
+        for (int i = tid; i < DP; i += nt) {
+          float nn = n_s[i];
+#pragma unroll
+          for (int u = 0; u < 8; ++u) {
+            const int t = h0 + u;
+            if (t < n) {                                 // uniform over the block
+              const float f = start_s[(it & 1) * REC_TB + t];
+              if (f >= 0.f) nn *= t == 0 ? f * pending : f;
+              nn += ks[t * DP + i];
+              if (!STATE_ONLY) a[u] = fmaf(nn, qs[t * DP + i], a[u]);
+            }
+          }
+          n_s[i] = nn;
+        }
+        if (!STATE_ONLY) {                               // eight sums over the warp; lane 4 u ends up with token h0 + u
+          const int lane = tid & 31;
+#pragma unroll
+          for (int off = 16, w = 4; off >= 4; off >>= 1, w >>= 1) {
+            const bool upper = (lane & off) != 0;
+#pragma unroll
+            for (int u = 0; u < 4; ++u) {
+              if (u < w) {
+                const float mine = upper ? a[u + w] : a[u], give = upper ? a[u] : a[u + w];
+                a[u] = mine + __shfl_xor_sync(0xffffffffu, give, off);
+              }
+            }
+          }
+          a[0] += __shfl_xor_sync(0xffffffffu, a[0], 2);
+          a[0] += __shfl_xor_sync(0xffffffffu, a[0], 1);
+          if ((lane & 3) == 0) dot_s[(it & 1) * 8 * REC_TB + tid / 32 * REC_TB + h0 + lane / 4] = a[0];
+        }
+      }
+    }
+    for (int t = 0; t < n; ++t) {
       if constexpr (RULE == RULE_MEMORY) {
         float f = start_s[(it & 1) * REC_TB + t];
         if (f >= 0.f) {
@@ -429,9 +479,7 @@ __global__ void __launch_bounds__(RULE == RULE_BONUS ? 128 : 256, RULE == RULE_B
 #pragma unroll
         for (int c = 0; c < WIDTH; ++c)
           if (c < out_cols) out[c] = o[c];
-          else if (RULE == RULE_MEMORY && c == norm_col) *norm = o[c];
         out += out_step;
-        if (RULE == RULE_MEMORY) norm += p.H;
       }
     }
   }
@@ -443,7 +491,17 @@ __global__ void __launch_bounds__(RULE == RULE_BONUS ? 128 : 256, RULE == RULE_B
 #pragma unroll
       for (int c = 0; c < REC_COLS; ++c) s[rp][c] = mul_f2(s[rp][c], f2);
   }
+  if (RULE == RULE_MEMORY && has_norm && !STATE_ONLY) {
+    __syncthreads();
+    if (it > 0 && tid < REC_TB && t_begin + (it - 1) * REC_TB + tid < t_end) {
+      float a = 0.f;
+      for (int w = 0; w < norm_warps; ++w) a += dot_s[((it - 1) & 1) * 8 * REC_TB + w * REC_TB + tid];
+      norm[static_cast<long long>((it - 1) * REC_TB + tid) * p.H] = a;
+    }
+  }
   auto store_state = [&](float* so) {
+    if (has_norm)
+      for (int i = tid; i < p.dim; i += nt) so[static_cast<long long>(i) * p.lds + p.vdim] = n_s[i] * pending;
 #pragma unroll
     for (int rp = 0; rp < REC_ROWS / 2; ++rp) {
       const int i = 4 * (g + G * (rp / 2)) + 2 * (rp % 2);
@@ -451,7 +509,7 @@ __global__ void __launch_bounds__(RULE == RULE_BONUS ? 128 : 256, RULE == RULE_B
       for (int c = 0; c < REC_COLS; ++c) {
         float a0, a1;
         unpack_f2(s[rp][c], a0, a1);
-        if (my_col + c < p.ncols) {
+        if (my_col + c < p.vdim) {
           if (i < p.dim) so[static_cast<long long>(i) * p.lds + my_col + c] = a0;
           if (i + 1 < p.dim) so[static_cast<long long>(i + 1) * p.lds + my_col + c] = a1;
         }
@@ -657,11 +715,9 @@ __global__ void __launch_bounds__(256) recurrence_step_kernel(const StepParams p
   }
 }
 
-static int rec_cols(int vdim, int rule) { return rule == RULE_MEMORY ? vdim + 1 : vdim; }
-
 // threads of a block: the column groups of a head, at most 256 (128 with the bonus rule, whose decays need more registers)
 static int rec_threads(int g, int vdim, int rule) {
-  const int groups = (rec_cols(vdim, rule) + REC_COLS - 1) / REC_COLS;
+  const int groups = (vdim + REC_COLS - 1) / REC_COLS;
   return std::min(rule == RULE_BONUS ? 128 : 256, (groups * g + 31) / 32 * 32);
 }
 
@@ -676,7 +732,7 @@ static int rec_launch(const RecParams& p, cudaStream_t st) {
                                          static_cast<int>(smem));
     if (e != cudaSuccess) return static_cast<int>(e);
   }
-  dim3 grid((p.ncols + cols - 1) / cols, p.H, p.B * p.nchunks);
+  dim3 grid((p.vdim + cols - 1) / cols, p.H, p.B * p.nchunks);
   recurrence_kernel<T, G, STATE_ONLY, RULE><<<grid, nt, smem, st>>>(p);
   return static_cast<int>(cudaGetLastError());
 }
@@ -737,8 +793,7 @@ static int run_recurrence(int rule, oslo::RecParams& p, float* state, float* ws,
   const int B = p.B, S = p.S, H = p.H, dim = p.dim, vdim = p.vdim;
   if (B <= 0 || S <= 0 || H <= 0) return 0;
   if (dim <= 0 || vdim <= 0 || dim > 512 || H > 65535 || nchunks < 1 || static_cast<long long>(B) * nchunks > 65535) return -1;
-  p.ncols = rec_cols(vdim, rule);
-  p.lds = rule == RULE_MEMORY ? (p.ncols + 3) / 4 * 4 : vdim;
+  p.lds = rule == RULE_MEMORY ? (vdim + 1 + 3) / 4 * 4 : vdim;
   const long long per = static_cast<long long>(H) * dim * p.lds;
   const int te = dtype == OSLO_DT_FP32 ? 4 : 2, v16 = 16 / te;
   p.dim_pad = (dim + 7) / 8 * 8;

@@ -31,71 +31,94 @@ constexpr float MEMORY_FLOOR = 1e-6f;
 __device__ __forceinline__ float capped(float z, float cap) { return cap * tanhf(z / cap); }
 __device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 
+constexpr int MG_SCAN = 128;                                  // threads that scan, a stage each
+constexpr int MG_PASS = MG_SCAN * MG_STAGE, MG_PITCH = MG_STAGE + 1;
+
 template <typename T>
 __global__ void __launch_bounds__(256) memory_gates_kernel(const float* __restrict__ z, long long ldz, const T* __restrict__ bias,
                                                            float cap, const uint8_t* __restrict__ keep, long long ld_keep,
                                                            float* __restrict__ top, float* __restrict__ read, float* __restrict__ write,
                                                            float* __restrict__ start, float* __restrict__ m_out, int S, int H) {
-  __shared__ float warp_f[8], warp_m[8], carry_s;
+  __shared__ float warp_f[MG_SCAN / 32], warp_m[MG_SCAN / 32], carry_s;
+  // a pass's gates (i, f), then its results (P, w / P, start, m); token t of stage s at s * MG_PITCH + t
+  __shared__ float buf[4][MG_SCAN * MG_PITCH];
   const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const float bi = Num<T>::to(bias[h]), bf = Num<T>::to(bias[H + h]);
   float carry = top ? top[static_cast<long long>(b) * H + h] : 0.f;
-  const long long at = (static_cast<long long>(b) * H + h) * S;
-  for (int base = 0; base < S; base += 256 * MG_STAGE) {
-    const int t0 = base + tid * MG_STAGE, n = min(MG_STAGE, S - t0);      // n may be <= 0
-    float gi[MG_STAGE], gf[MG_STAGE], F = 0.f, M = -CUDART_INF_F;
-#pragma unroll
-    for (int u = 0; u < MG_STAGE; ++u) {
-      gi[u] = -CUDART_INF_F;
-      gf[u] = 0.f;
-      if (u < n && (keep == nullptr || keep[b * ld_keep + t0 + u])) {
-        const float* row = z + (static_cast<long long>(b) * S + t0 + u) * ldz;
-        gi[u] = capped(row[h] + bi, cap);
-        gf[u] = log_sigmoid(capped(row[H + h] + bf, cap));
+  const long long at = (static_cast<long long>(b) * H + h) * S, row0 = static_cast<long long>(b) * S;
+  for (int base = 0; base < S; base += MG_PASS) {
+    const int count = min(MG_PASS, S - base);
+#pragma unroll 4
+    for (int t = tid; t < MG_PASS; t += 256) {
+      float gi = -CUDART_INF_F, gf = 0.f;
+      if (t < count && (keep == nullptr || keep[b * ld_keep + base + t])) {
+        const float* row = z + (row0 + base + t) * ldz;
+        gi = capped(row[h] + bi, cap);
+        gf = log_sigmoid(capped(row[H + h] + bf, cap));
       }
-      F += gf[u];
-      M = fmaxf(M + gf[u], gi[u]);
+      const int o = t / MG_STAGE * MG_PITCH + t % MG_STAGE;
+      buf[0][o] = gi;
+      buf[1][o] = gf;
     }
-    // inclusive scan of (F, M) over the block: first this, then that: (F1 + F2, max(M1 + F2, M2))
-    float sf = F, sm = M;
-#pragma unroll
-    for (int off = 1; off < 32; off <<= 1) {
-      const float pf = __shfl_up_sync(0xffffffffu, sf, off), pm = __shfl_up_sync(0xffffffffu, sm, off);
-      if (lane >= off) { sm = fmaxf(pm + sf, sm); sf += pf; }
-    }
-    if (lane == 31) { warp_f[warp] = sf; warp_m[warp] = sm; }
-    const float ef = __shfl_up_sync(0xffffffffu, sf, 1), em = __shfl_up_sync(0xffffffffu, sm, 1);
     __syncthreads();
-    float m = carry;
-    for (int w = 0; w < warp; ++w) m = fmaxf(m + warp_f[w], warp_m[w]);
-    if (lane > 0) m = fmaxf(m + ef, em);
-    float P = 1.f;
+    const int o0 = tid * MG_PITCH, n = min(MG_STAGE, count - tid * MG_STAGE);    // n may be <= 0
+    float ef = 0.f, em = -CUDART_INF_F;
+    if (warp < MG_SCAN / 32) {
+      float sf = 0.f, sm = -CUDART_INF_F;
 #pragma unroll
-    for (int u = 0; u < MG_STAGE; ++u) {
-      if (u >= n) break;
-      const float top_t = fmaxf(gf[u] + m, gi[u]);
-      const float d = expf(gf[u] + m - top_t), w = expf(gi[u] - top_t);
-      m = top_t;
-      float s = -1.f;
-      if (u == 0) {
-        s = d;                                   // the kernel multiplies by what the last stage left
-        P = 1.f;
-      } else if (P * d < MG_MIN_PERIOD) {
-        s = P * d;
-        P = 1.f;
-      } else {
-        P *= d;
+      for (int u = 0; u < MG_STAGE; ++u) {
+        const float gf = buf[1][o0 + u];
+        sf += gf;
+        sm = fmaxf(sm + gf, buf[0][o0 + u]);
       }
-      read[at + t0 + u] = P;
-      write[at + t0 + u] = w / P;
-      start[at + t0 + u] = s;
-      m_out[(static_cast<long long>(b) * S + t0 + u) * H + h] = top_t;
+      // inclusive scan of (F, M) over the warp: first this, then that: (F1 + F2, max(M1 + F2, M2))
+#pragma unroll
+      for (int off = 1; off < 32; off <<= 1) {
+        const float pf = __shfl_up_sync(0xffffffffu, sf, off), pm = __shfl_up_sync(0xffffffffu, sm, off);
+        if (lane >= off) { sm = fmaxf(pm + sf, sm); sf += pf; }
+      }
+      if (lane == 31) { warp_f[warp] = sf; warp_m[warp] = sm; }
+      ef = __shfl_up_sync(0xffffffffu, sf, 1);
+      em = __shfl_up_sync(0xffffffffu, sm, 1);
     }
-    if (n > 0 && t0 + n == S) carry_s = m;
-    // the next pass starts from the last thread's maximum
-    if (tid == 255 && n == MG_STAGE) carry_s = m;
+    __syncthreads();
+    if (warp < MG_SCAN / 32) {
+      float m = carry;
+      for (int w = 0; w < warp; ++w) m = fmaxf(m + warp_f[w], warp_m[w]);
+      if (lane > 0) m = fmaxf(m + ef, em);
+      float P = 1.f;
+#pragma unroll
+      for (int u = 0; u < MG_STAGE; ++u) {
+        const float gi = buf[0][o0 + u], gf = buf[1][o0 + u];
+        const float top_t = fmaxf(gf + m, gi);
+        const float d = expf(gf + m - top_t), w = expf(gi - top_t);
+        m = top_t;
+        float s = -1.f;
+        if (u == 0) {
+          s = d;                                 // the kernel multiplies by what the last stage left
+        } else if (P * d < MG_MIN_PERIOD) {
+          s = P * d;
+          P = 1.f;
+        } else {
+          P *= d;
+        }
+        buf[0][o0 + u] = P;
+        buf[1][o0 + u] = w / P;
+        buf[2][o0 + u] = s;
+        buf[3][o0 + u] = m;
+        if (n > 0 && u == n - 1 && (tid == MG_SCAN - 1 || tid * MG_STAGE + n == count)) carry_s = m;   // the pass's last token
+      }
+    }
     __syncthreads();
     carry = carry_s;
+#pragma unroll 4
+    for (int t = tid; t < count; t += 256) {
+      const int o = t / MG_STAGE * MG_PITCH + t % MG_STAGE;
+      read[at + base + t] = buf[0][o];
+      write[at + base + t] = buf[1][o];
+      start[at + base + t] = buf[2][o];
+      m_out[(row0 + base + t) * H + h] = buf[3][o];
+    }
     __syncthreads();
   }
   if (top && tid == 0) top[static_cast<long long>(b) * H + h] = carry;

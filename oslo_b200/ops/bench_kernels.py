@@ -7,6 +7,10 @@
                                                            expert and norm layers, each with its bound (HBM bytes, bf16
                                                            tensor-core or fp32 FMA throughput, whichever is slowest),
                                                            beside the like kernels of GPT-J at the same sizes
+``python -m oslo_b200.ops.bench_kernels --op branches``    the same for grouped-query attention, the linear recurrences, the
+                                                           selective scan and the branch joins, beside those
+``python -m oslo_b200.ops.bench_kernels --op streams``     the same for windowed and two-part attention, matrix memory, gated and
+                                                           identity experts and the stream join, beside those
 ``--case i`` restricts the run to one shape and ``--iters n --warmup w`` bound the number of launches, which is
 what a profiler capture wants. Every line is JSON; ``frac_of_measured`` divides by the bf16 GEMM throughput in
 ``MEASURED_PEAKS.json`` at the repository root when that file exists (else by 1590 TFLOP/s).
@@ -133,6 +137,7 @@ def bench_attention(args, timer: _Timer) -> None:
 
 # width, heads, head dim, q_rank, kv_rank, experts, top, ff of an expert
 MIXER_CASES = [(2048, 16, 128, 1024, 512, 16, 2, 1024), (4096, 32, 128, 1536, 512, 32, 4, 1536)]
+SFU_TERAOPS = 148 * 16 * 1.965e9 / 1e12            # exponentials, reciprocals: 16 per cycle and SM (nominal)
 FP32_TFLOPS = 148 * 128 * 2 * 1.965e9 / 1e12       # FMA pipes at the maximum SM clock (nominal; nothing measures it)
 
 
@@ -145,21 +150,28 @@ def _measured_hbm() -> float:
         return 6650.0
 
 
-def bench_mixers(args, timer: _Timer) -> None:
-    ext = load_ext(required=True)
-    timer = _GraphTimer(args.iters, args.warmup, not args.no_flush)
+def _reporter(args, timer):
+    """``report(case, op, fn, ...)``: time ``fn`` and print it beside the slowest of its bounds (HBM bytes, bf16 products, fp32 FMAs,
+    special functions)."""
     peak, hbm = _peak_tflops(), _measured_hbm()
-    bf = torch.bfloat16
-    mk = lambda *s: (torch.randn(*s, device="cuda") * 0.5).to(bf)                                          # noqa: E731
 
-    def report(case, op, fn, gbytes=0.0, tflop=0.0, fp32_tflop=0.0, like=""):
+    def report(case, op, fn, gbytes=0.0, tflop=0.0, fp32_tflop=0.0, sfu=0.0, like=""):
         if args.only and args.only not in op:
             return
         ms = timer(fn)
-        bound = {"hbm": gbytes / hbm * 1e3, "bf16": tflop / peak * 1e3, "fp32": fp32_tflop / FP32_TFLOPS * 1e3}
+        bound = {"hbm": gbytes / hbm * 1e3, "bf16": tflop / peak * 1e3, "fp32": fp32_tflop / FP32_TFLOPS * 1e3, "sfu": sfu / SFU_TERAOPS / 1e9}
         by = max(bound, key=bound.get)
         print(json.dumps(dict(case=case, op=op, us=round(ms * 1e3, 2), bound_us=round(bound[by] * 1e3, 2), bound_by=by,
                               times_bound=round(ms / bound[by], 2), like=like)), flush=True)
+
+    return report
+
+
+def bench_mixers(args, timer: _Timer) -> None:
+    ext = load_ext(required=True)
+    report = _reporter(args, _GraphTimer(args.iters, args.warmup, not args.no_flush))
+    bf = torch.bfloat16
+    mk = lambda *s: (torch.randn(*s, device="cuda") * 0.5).to(bf)                                          # noqa: E731
 
     for case, (w, h, d, qr, kr, e, top, ff) in enumerate(MIXER_CASES):
         if args.case is not None and args.case != case:
@@ -253,26 +265,15 @@ def bench_mixers(args, timer: _Timer) -> None:
 
 # width, wkv heads x dim, decay rank, inner channels, states, dt_rank, attention heads, kv heads, head dim, linear heads x dim, ff
 BRANCH_CASES = [(2048, 32, 64, 64, 4096, 16, 128, 16, 4, 128, 16, 128, 5504), (4096, 64, 64, 128, 8192, 16, 256, 32, 8, 128, 32, 128, 11008)]
-SFU_TERAOPS = 148 * 16 * 1.965e9 / 1e12            # exponentials, reciprocals: 16 per cycle and SM (nominal)
 
 
 def bench_branches(args, timer: _Timer) -> None:
     """The kernels of grouped-query attention, the linear recurrences, the selective scan and the joins (Begovik layers) beside the
     like kernels of the other families."""
     ext = load_ext(required=True)
-    timer = _GraphTimer(args.iters, args.warmup, not args.no_flush)
-    peak, hbm = _peak_tflops(), _measured_hbm()
+    report = _reporter(args, _GraphTimer(args.iters, args.warmup, not args.no_flush))
     bf = torch.bfloat16
     mk = lambda *s: (torch.randn(*s, device="cuda") * 0.5).to(bf)                                          # noqa: E731
-
-    def report(case, op, fn, gbytes=0.0, tflop=0.0, fp32_tflop=0.0, sfu=0.0, like=""):
-        if args.only and args.only not in op:
-            return
-        ms = timer(fn)
-        bound = {"hbm": gbytes / hbm * 1e3, "bf16": tflop / peak * 1e3, "fp32": fp32_tflop / FP32_TFLOPS * 1e3, "sfu": sfu / SFU_TERAOPS / 1e9}
-        by = max(bound, key=bound.get)
-        print(json.dumps(dict(case=case, op=op, us=round(ms * 1e3, 2), bound_us=round(bound[by] * 1e3, 2), bound_by=by,
-                              times_bound=round(ms / bound[by], 2), like=like)), flush=True)
 
     for case, (w, rh, rd, rank, inner, ns, dtr, h, g, d, lh, ld, ff) in enumerate(BRANCH_CASES):
         if args.case is not None and args.case != case:
@@ -396,20 +397,188 @@ def bench_branches(args, timer: _Timer) -> None:
             del ws, wm
 
 
+# width, streams, attention heads, kv heads, head dim, window, kept, latent dim, rot, vdim, q_rank, kv_rank, memory heads x dim x vdim,
+# experts, identity, top, ff
+STREAM_CASES = [(2048, 4, 16, 4, 128, 512, 16, 128, 64, 128, 1024, 512, 16, 128, 128, 16, 4, 4, 1344),
+                (4096, 4, 32, 8, 128, 1024, 16, 128, 64, 128, 1536, 512, 32, 128, 128, 32, 4, 4, 2688)]
+
+
+def bench_streams(args, timer: _Timer) -> None:
+    """The kernels of the Dekutar layers beside the like kernels of the other families at the same sizes."""
+    ext = load_ext(required=True)
+    report = _reporter(args, _GraphTimer(args.iters, args.warmup, not args.no_flush))
+    bf, none = torch.bfloat16, None
+    mk = lambda *s: (torch.randn(*s, device="cuda") * 0.5).to(bf)                                          # noqa: E731
+    for case, (w, ns, h, g, d, win, kept, ld, rot, vd, qr, kr, mh, md, mv, e, ident, top, ff) in enumerate(STREAM_CASES):
+        if args.case is not None and args.case != case:
+            continue
+        vec, vq, vk = mk(w), mk(qr), mk(kr)
+        w_in, w_out, mix = mk(ns), mk(ns), mk(ns, ns)
+        nm, gb, wg = mk(mh * mv), mk(2 * mh), mk(2 * mh, w)
+        fb, lo = mk(mh * md), mk(mh * md).abs().clamp(max=0.9)
+        decay, sink = torch.linspace(0.5, 0.999, mh, device="cuda"), torch.zeros(h, dtype=bf, device="cuda")
+        freq, lfreq = torch.rand(d // 2, device="cuda"), torch.rand(rot // 2, device="cuda")
+        rw, rb = mk(e + ident, w) * 0.1, mk(e + ident) * 0.1
+        up, down = mk(e, 2 * ff, w), mk(e, w, ff)
+        lds = (mv + 4) // 4 * 4
+        # ------------------------------------------------ prompts: 4 x 2048 and 1 x 2048 tokens
+        for b, s in ((4, 2048), (1, 2048)):
+            n, tag = b * s, f"prompt {b} x {s} "
+            q, k, v = mk(b, h, s, d), mk(b, g, s, d), mk(b, g, s, d)
+            gate, wide = mk(n, h), mk(n, h * vd)
+            seen = sum(min(i + 1, win + kept) for i in range(s))
+            pairs = b * h * s * s / 2.0
+            report(case, tag + "windowed attention + gate", lambda: ext.flash_sink_fwd(q, k, v, none, none, gate, d ** -0.5, 0.0, win, kept),
+                   gbytes=2 * n * (h + g) * d * 2 / 1e9, tflop=4.0 * b * h * seen * d / 1e12, sfu=1.0 * b * h * seen, like="attention, window only")
+            report(case, tag + "attention, window only", lambda: ext.flash_sink_fwd(q, k, v, none, sink, gate, d ** -0.5, 0.0, win + kept, 0),
+                   gbytes=2 * n * (h + g) * d * 2 / 1e9, tflop=4.0 * b * h * seen * d / 1e12, sfu=1.0 * b * h * seen)
+            kf, vf = _every_head(k, h // g), _every_head(v, h // g)
+            report(case, tag + "attention (GPT-J)", lambda: ext.flash_fwd(q, kf, vf, d ** -0.5, True, 0, none, 1),
+                   gbytes=4 * n * h * d * 2 / 1e9, tflop=4.0 * pairs * d / 1e12, sfu=pairs)
+            qa, ka, va, kr2 = mk(b, s, h, ld + rot), mk(b, s, h, ld), mk(b, s, h, vd), mk(b, s, kr + rot)
+            flat = lambda t: t.permute(0, 2, 1, 3)                                                         # noqa: E731
+            report(case, tag + "two-part attention + gate", lambda: ext.flash_sink_fwd(flat(qa)[..., :ld], flat(ka), flat(va), none, none, wide, 0.07, 0.0,
+                                                                                       0, 0, none, flat(qa)[..., ld:], kr2[..., kr:]),
+                   gbytes=n * (h * (2 * ld + rot + 3 * vd) + rot) * 2 / 1e9, tflop=2.0 * pairs * (ld + rot + vd) / 1e12, sfu=pairs,
+                   like="attention with sink + gate (Moronex)")
+            report(case, tag + "attention with sink + gate (Moronex)", lambda: ext.flash_sink_fwd(flat(qa)[..., :ld], flat(ka), flat(va), none, sink, gate,
+                                                                                                  0.07, 0.0),
+                   gbytes=n * h * (2 * ld + 2 * vd) * 2 / 1e9, tflop=2.0 * pairs * (ld + vd) / 1e12, sfu=pairs)
+            pm = mk(n, 2 * mh * md + mh * mv)
+            mq, mkk, mvv = pm[:, :mh * md], pm[:, mh * md:2 * mh * md], pm[:, 2 * mh * md:]
+            z = torch.randn(n, 2 * mh, device="cuda") * 3.0
+            st, tp = torch.zeros(b, mh, md, lds, device="cuda"), torch.zeros(b, mh, device="cuda")
+            rd, wr, bg, mm = ext.memory_gates(z, gb, 15.0, none, tp, b)
+            report(case, tag + "memory gates", lambda: ext.memory_gates(z, gb, 15.0, none, tp, b), gbytes=n * mh * 24 / 1e9, sfu=8.0 * n * mh,
+                   like="layer norm")
+            report(case, tag + "memory recurrence", lambda: ext.memory_recurrence(mq, mkk, mvv, rd, wr, bg, md ** -0.5, none, st, b, mh, md, mv),
+                   gbytes=n * mh * (4 * md + 6 * mv) / 1e9, fp32_tflop=4.0 * n * mh * md * (mv + 1) / 1e12, like="decayed recurrence (Begovik)")
+            if md == mv:
+                s2 = torch.zeros(b, mh, md, mv, device="cuda")
+                report(case, tag + "decayed recurrence (Begovik)", lambda: ext.decayed_recurrence(mq, mkk, mvv, decay, none, s2, b, mh, md, mv),
+                       gbytes=n * mh * (4 * md + 6 * mv) / 1e9, fp32_tflop=4.0 * n * mh * md * mv / 1e12)
+                report(case, tag + "gated recurrence (Moronex)", lambda: ext.recurrence(mq, mkk, mvv, fb, lo, none, s2, b, mh, md, mv),
+                       gbytes=n * mh * (4 * md + 6 * mv) / 1e9, fp32_tflop=6.0 * n * mh * md * mv / 1e12)
+            del q, k, v, qa, ka, va, kf, vf
+            if b == 1:
+                continue
+            o, og, nq = torch.randn(n, mh * mv, device="cuda"), mk(n, mh * mv), torch.randn(n, mh, device="cuda")
+            report(case, tag + "normaliser + head norm + gate", lambda: ext.gated_rms_norm(o, nm, og, 1e-6, mv, 0, nq, mm), gbytes=n * mh * mv * 8 / 1e9,
+                   like="head norm + gate (Begovik)")
+            report(case, tag + "head norm + gate (Begovik)", lambda: ext.gated_rms_norm(o, nm, og, 1e-6, mv, 0), gbytes=n * mh * mv * 8 / 1e9)
+            hb = mk(n, w)
+            report(case, tag + "gate logits, fp32 result", lambda: co.linear_fp32(hb, wg), gbytes=n * w * 2 / 1e9, like="route (Moronex)")
+            pos, l0 = torch.arange(s, device="cuda")[None].expand(b, s), torch.zeros(b, dtype=torch.int32, device="cuda")
+            pa = mk(n, (h + g) * d)
+            kc, vc = mk(b, g, s, d), mk(b, g, s, d)
+            report(case, tag + "norms + rotation + append", lambda: ext.qkv_prep(pa[:, :h * d], pa[:, h * d:], pa[:, h * d:], none, none, 1e-6, pos, freq, kc,
+                                                                              vc, l0), gbytes=n * (2 * h + 3 * g) * d * 2 / 1e9, like="layer norm")
+            pl, lc = mk(n, qr + kr + rot), mk(b, s, kr + rot)
+            report(case, tag + "latent norms + rotation + append", lambda: ext.latent_prep(pl[:, :qr], vq, pl[:, qr:], vk, lc, l0, 1e-6, pos, lfreq, True),
+                   gbytes=n * (2 * qr + 3 * kr + 2 * rot) * 2 / 1e9, like="layer norm")
+            ql = mk(b, s, h, ld + rot)
+            report(case, tag + "query rotation in place", lambda: ext.rotate_halves_(ql, pos, lfreq), gbytes=n * h * rot * 4 / 1e9, like="layer norm")
+            x, y, sh, sg = torch.randn(n, ns, w, device="cuda"), mk(n, w), mk(n, w), mk(n, 8)[:, :1]
+            report(case, tag + f"join of {ns} streams", lambda: ext.hyper_join(x, y, none, none, none, 0, none, none, none, w_out, mix, w_in, vec, 1e-6, 1.0),
+                   gbytes=n * w * (8 * ns + 4) / 1e9, like="residual join (Moronex)")
+            x1, gt = torch.randn(n, w, device="cuda"), mk(n, w)
+            report(case, tag + "residual join (Moronex)", lambda: ext.residual_join(x1, y, none, none, gt, vec, vec, vec, 1e-5), gbytes=n * w * 14 / 1e9)
+            report(case, tag + "layer norm (GPT-J)", lambda: ext.layernorm_fwd(hb, vec, vec, 1e-5), gbytes=n * w * 4 / 1e9)
+            report(case, tag + "route, scored", lambda: co.moe_route(hb, rw, rb, top, True), gbytes=n * w * 2 / 1e9, like="route (Moronex)")
+            report(case, tag + "route (Moronex)", lambda: co.moe_route(hb, rw, rb, top), gbytes=n * w * 2 / 1e9)
+            idx, wgt = co.moe_route(hb, rw, rb, top, True)
+            real = int((idx < e).sum())
+            slots, rows, tg, nt = ext.moe_plan(hb, idx, e)
+            report(case, tag + "plan + gather", lambda: ext.moe_plan(hb, idx, e), gbytes=(n + real) * w * 2 / 1e9, like="layer norm")
+            report(case, tag + "gated experts up", lambda: ext.moe_grouped(rows, up, tg, nt, 2), tflop=4.0 * real * w * ff / 1e12,
+                   gbytes=(real * (w + ff) + 2 * e * w * ff) * 2 / 1e9, like="experts up, relu^2 (Moronex)")
+            report(case, tag + "experts up, relu^2 (Moronex)", lambda: ext.moe_grouped(rows, up, tg, nt, 1), tflop=4.0 * real * w * ff / 1e12,
+                   gbytes=(real * (w + 2 * ff) + 2 * e * w * ff) * 2 / 1e9)
+            a = ext.moe_grouped(rows, up, tg, nt, 2)
+            report(case, tag + "experts down", lambda: ext.moe_grouped(a, down, tg, nt, 0), tflop=2.0 * real * w * ff / 1e12,
+                   gbytes=(real * (w + ff) + e * w * ff) * 2 / 1e9, like="experts up, relu^2 (Moronex)")
+            ye = ext.moe_grouped(a, down, tg, nt, 0)
+            report(case, tag + f"join of {ns} streams, experts + shared",
+                   lambda: ext.hyper_join(x, ye, slots, wgt, idx, e, hb, sh, sg, w_out, mix, w_in, vec, 1e-6, 1.0),
+                   gbytes=(n * w * (8 * ns + 4) + (real + n) * w * 2) / 1e9, like="residual join of experts (Moronex)")
+            report(case, tag + "residual join of experts (Moronex)", lambda: ext.residual_join(x1, ye, slots.clamp(min=0), wgt, gt, vec, vec, vec, 1e-5),
+                   gbytes=n * w * (12 + 2 * top) / 1e9)
+            del o, og, hb, pa, x, y, sh, rows, a, ye, x1, gt
+        # ------------------------------------------------ decode over 4096 cached tokens
+        for n in (1, 8, 64):
+            t, tag = 4096, f"decode {n} "
+            lengths = torch.full((n,), t, dtype=torch.int32, device="cuda")
+            l1, pos = lengths - 1, torch.full((n, 1), t - 1, dtype=torch.long, device="cuda")
+            q3, gate, kc, vc = mk(n, h, d), mk(n, h), mk(n, g, t, d), mk(n, g, t, d)
+            report(case, tag + "windowed attention + gate (2 launches)", lambda: ext.grouped_decode(q3, kc, vc, lengths, none, none, d ** -0.5, 0.0, gate, win, kept),
+                   gbytes=2 * n * (win + kept) * g * d * 2 / 1e9, like="attention over as many keys (Begovik)")
+            ks, vs, ls = mk(n, g, win + kept, d), mk(n, g, win + kept, d), torch.full((n,), win + kept, dtype=torch.int32, device="cuda")
+            report(case, tag + "attention over as many keys (Begovik)", lambda: ext.grouped_decode(q3, ks, vs, ls, none, sink, d ** -0.5, 0.0),
+                   gbytes=2 * n * (win + kept) * g * d * 2 / 1e9)
+            pa = mk(n, (h + g) * d)
+            report(case, tag + "norms + rotation + append", lambda: ext.qkv_prep(pa[:, :h * d], pa[:, h * d:], pa[:, h * d:], none, none, 1e-6, pos, freq, kc,
+                                                                              vc, l1), gbytes=n * (2 * h + 3 * g) * d * 2 / 1e9, like="layer norm")
+            del kc, vc, ks, vs
+            uk, uv, ql, wide, lc = mk(h * ld, kr), mk(h * vd, kr), mk(n, h * (ld + rot)), mk(n, h * vd), mk(n, t, kr + rot)
+            report(case, tag + "rotated latent attention (3 launches)",
+                   lambda: ext.latent_decode(ql, uk, uv, lc, lengths, none, none, wide, 0.07, h, pos, lfreq),
+                   gbytes=(n * t * (kr + rot) + h * (ld + vd) * kr) * 2 / 1e9, tflop=2.0 * n * t * h * (2 * kr + rot) / 1e12, like="latent attention (Moronex)")
+            lm, qm = mk(n, t, kr), mk(n, h * ld)
+            report(case, tag + "latent attention (Moronex)", lambda: ext.latent_decode(qm, uk, uv, lm, lengths, none, sink, gate, 0.07, h),
+                   gbytes=(n * t * kr + h * (ld + vd) * kr) * 2 / 1e9, tflop=4.0 * n * t * h * kr / 1e12)
+            pl = mk(n, qr + kr + rot)
+            report(case, tag + "latent norms + rotation + append", lambda: ext.latent_prep(pl[:, :qr], vq, pl[:, qr:], vk, lc, l1, 1e-6, pos, lfreq),
+                   gbytes=n * (qr + kr + rot) * 4 / 1e9, like="layer norm")
+            del lc, lm
+            mq, mkk, mvv, og, hb = mk(n, mh * md), mk(n, mh * md), mk(n, mh * mv), mk(n, mh * mv), mk(n, w)
+            st, tp = torch.zeros(n, mh, md, lds, device="cuda"), torch.zeros(n, mh, device="cuda")
+            report(case, tag + "memory step", lambda: ext.memory_step(mq, mkk, mvv, hb, wg, gb, 15.0, og, nm, none, st, tp, md ** -0.5, 1e-6, mh, md, mv),
+                   gbytes=(n * mh * md * (mv + 1) * 8 + 2 * mh * w * 2) / 1e9, like="recurrence step (Moronex)")
+            if md == mv:
+                s2, nv = torch.zeros(n, mh, md, mv, device="cuda"), mk(mv)
+                report(case, tag + "recurrence step (Moronex)", lambda: ext.recurrence_step(mq, mkk, mvv, fb, lo, nv, none, s2, 1e-5, mh, md, mv),
+                       gbytes=n * mh * md * mv * 8 / 1e9)
+            x, y, sh, sg = torch.randn(n, ns, w, device="cuda"), mk(n, w), mk(n, w), mk(n, 8)[:, :1]
+            report(case, tag + f"join of {ns} streams", lambda: ext.hyper_join(x, y, none, none, none, 0, none, none, none, w_out, mix, w_in, vec, 1e-6, 1.0),
+                   gbytes=n * w * (8 * ns + 4) / 1e9, like="residual join (Moronex)")
+            x1, gt = torch.randn(n, w, device="cuda"), mk(n, w)
+            report(case, tag + "residual join (Moronex)", lambda: ext.residual_join(x1, y, none, none, gt, vec, vec, vec, 1e-5), gbytes=n * w * 14 / 1e9)
+            report(case, tag + "layer norm (GPT-J)", lambda: ext.layernorm_fwd(hb, vec, vec, 1e-5), gbytes=n * w * 4 / 1e9)
+            report(case, tag + "route, scored", lambda: co.moe_route(hb, rw, rb, top, True), gbytes=(e + ident) * w * 2 / 1e9, like="route (Moronex)")
+            report(case, tag + "route (Moronex)", lambda: co.moe_route(hb, rw, rb, top), gbytes=(e + ident) * w * 2 / 1e9)
+            idx, wgt = co.moe_route(hb, rw, rb, top, True)
+            used = int(idx[idx < e].unique().numel())
+            report(case, tag + "gated experts up + down", lambda: co.moe_experts(hb, idx, up, down, "silu"), gbytes=used * w * ff * 6 / 1e9,
+                   like="experts up + down, relu^2 (Moronex)")
+            up1 = mk(e, ff, w)
+            report(case, tag + "experts up + down, relu^2 (Moronex)", lambda: co.moe_experts(hb, idx, up1, down), gbytes=used * w * ff * 4 / 1e9)
+            ye, slots = co.moe_experts(hb, idx, up, down, "silu")
+            report(case, tag + f"join of {ns} streams, experts + shared",
+                   lambda: ext.hyper_join(x, ye, slots, wgt, idx, e, hb, sh, sg, w_out, mix, w_in, vec, 1e-6, 1.0),
+                   gbytes=n * w * (8 * ns + 6 + 2 * top) / 1e9, like="residual join (Moronex)")
+            del up1
+
+
+def _every_head(t: torch.Tensor, per: int) -> torch.Tensor:
+    """Every key / value head ``per`` times: what attention without groups reads."""
+    b, g, s, d = t.shape
+    return t[:, :, None].expand(b, g, per, s, d).reshape(b, g * per, s, d)
+
+
 def main() -> None:
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
-    ap.add_argument("--op", choices=["gemm", "attention", "mixers", "branches"], required=True)
+    ap.add_argument("--op", choices=["gemm", "attention", "mixers", "branches", "streams"], required=True)
     ap.add_argument("--case", type=int, default=None, help="index into the op's shape list")
     ap.add_argument("--iters", type=int, default=20)
     ap.add_argument("--warmup", type=int, default=5)
     ap.add_argument("--causal", type=int, default=None, help="attention: 1 / 0 to run only one mask")
     ap.add_argument("--no-baseline", action="store_true", help="skip the library / legacy-kernel baseline")
     ap.add_argument("--no-flush", action="store_true", help="do not write a 256 MB buffer between timed calls")
-    ap.add_argument("--only", default="", help="mixers, branches: only the entries whose name contains this")
+    ap.add_argument("--only", default="", help="mixers, branches, streams: only the entries whose name contains this")
     args = ap.parse_args()
     timer = _Timer(args.iters, args.warmup, not args.no_flush)
     with torch.no_grad():
-        {"gemm": bench_gemm, "attention": bench_attention, "mixers": bench_mixers, "branches": bench_branches}[args.op](args, timer)
+        {"gemm": bench_gemm, "attention": bench_attention, "mixers": bench_mixers, "branches": bench_branches, "streams": bench_streams}[args.op](args, timer)
 
 
 if __name__ == "__main__":

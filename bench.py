@@ -609,10 +609,10 @@ def begovik_config(width, heads, layers, vocab=50400):
 
 def dekutar_config(width, heads, layers, q_rank, kv_rank, experts, vocab=50400):
     """Layers in groups of three: attention in a window of 512 (4 query heads per key / value head), matrix memory, latent attention
-    with 64 rotated dims; four residual streams; four gated experts of the router's (4 of its outputs are the identity) and a shared
+    with 64 rotated dims; four residual streams; four gated experts of the router's (3 of its outputs are the identity) and a shared
     one, each with a fourth of GPT-J's MLP weights."""
     dim, ff = width // heads, 2 * width // 3 // 64 * 64
-    mlp = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "identity": 4, "top": 4}, "shared": {"ff": ff}}
+    mlp = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "identity": 3, "top": 4}, "shared": {"ff": ff}}
     kinds = [("attention", {"heads": heads, "kv_heads": max(1, heads // 4), "dim": dim, "vdim": dim, "scale": dim ** -0.5,
                             "mask": {"size": 512, "keep_first": 16}, "rot": {"base": 10000.0, "dims": dim}}),
              ("mlstm", {"heads": heads, "dim": dim, "vdim": dim, "gate_cap": 15.0}),

@@ -1538,14 +1538,17 @@ std::tuple<Tensor, Tensor> moe_route(const Tensor& h, const Tensor& w, const Ten
                   w.scalar_type() == h.scalar_type() && bias.scalar_type() == h.scalar_type(), "moe_route: router");
   const int64_t n = h.size(0), E = w.size(0);
   const float* lg = nullptr;
+  int64_t ldl = 0;
   if (logits.has_value() && logits->defined()) {
-    TORCH_CHECK(logits->scalar_type() == at::kFloat && logits->is_contiguous() && logits->numel() == n * E, "moe_route: logits");
+    check_rows(*logits, "logits");
+    TORCH_CHECK(logits->scalar_type() == at::kFloat && logits->size(0) == n && logits->size(1) == E, "moe_route: logits");
     lg = logits->data_ptr<float>();
+    ldl = logits->stride(0);
   }
   c10::cuda::CUDAGuard guard(h.device());
   Tensor idx = at::empty({n, top}, h.options().dtype(at::kInt));
   Tensor wgt = at::empty({n, top}, h.options().dtype(at::kFloat));
-  check_rc(oslo_moe_route(h.data_ptr(), h.stride(0), w.data_ptr(), bias.data_ptr(), lg, idx.data_ptr<int>(), wgt.data_ptr<float>(),
+  check_rc(oslo_moe_route(h.data_ptr(), h.stride(0), w.data_ptr(), bias.data_ptr(), lg, ldl, idx.data_ptr<int>(), wgt.data_ptr<float>(),
                           n, static_cast<int>(E), static_cast<int>(h.size(1)), static_cast<int>(top), scored ? 1 : 0, dt_code(h),
                           cur_stream()), "moe_route");
   return {idx, wgt};

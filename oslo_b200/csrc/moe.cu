@@ -143,9 +143,9 @@ route_kernel(const T* __restrict__ h, long long ldh, const T* __restrict__ w, co
   }
 }
 
-// logits [rows, E] (32-bit, without the bias) from a GEMM: one warp per row
+// logits [rows, E] (32-bit, without the bias, rows ldl apart) from a GEMM: one warp per row
 template <typename T>
-__global__ void __launch_bounds__(128) route_logits_kernel(const float* __restrict__ logits, const T* __restrict__ bias,
+__global__ void __launch_bounds__(128) route_logits_kernel(const float* __restrict__ logits, long long ldl, const T* __restrict__ bias,
                                                            int* __restrict__ idx, float* __restrict__ wgt, long long rows,
                                                            int E, int top, int scored) {
   extern __shared__ float rl_smem[];
@@ -153,7 +153,7 @@ __global__ void __launch_bounds__(128) route_logits_kernel(const float* __restri
   const long long row = static_cast<long long>(blockIdx.x) * 4 + warp;
   if (row >= rows) return;
   float* z = rl_smem + warp * E * (scored ? 2 : 1);
-  for (int e = lane; e < E; e += 32) z[e] = scored ? logits[row * E + e] : logits[row * E + e] + Num<T>::to(bias[e]);
+  for (int e = lane; e < E; e += 32) z[e] = scored ? logits[row * ldl + e] : logits[row * ldl + e] + Num<T>::to(bias[e]);
   __syncwarp();
   if (scored) pick_scored<T>(z, z + E, bias, E, top, idx + row * top, wgt + row * top, lane);
   else pick_top(z, E, top, idx + row * top, wgt + row * top, lane);
@@ -322,8 +322,8 @@ __global__ void __launch_bounds__(256, 4) moe_few_kernel(const T* __restrict__ x
 
 }  // namespace oslo
 
-extern "C" int oslo_moe_route(const void* h, long long ldh, const void* w, const void* bias, const float* logits, int* idx,
-                              float* wgt, long long rows, int E, int K, int top, int scored, int dtype, cudaStream_t stream) {
+extern "C" int oslo_moe_route(const void* h, long long ldh, const void* w, const void* bias, const float* logits, long long ldl,
+                              int* idx, float* wgt, long long rows, int E, int K, int top, int scored, int dtype, cudaStream_t stream) {
   using namespace oslo;
   const size_t per_row = (scored ? 2 : 1) * E * sizeof(float);
   if (rows <= 0) return 0;
@@ -332,7 +332,7 @@ extern "C" int oslo_moe_route(const void* h, long long ldh, const void* w, const
   if (logits) {
     OSLO_DISPATCH_T(dtype, {
       route_logits_kernel<T><<<static_cast<unsigned>((rows + 3) / 4), 128, 4 * per_row, stream>>>(
-          logits, static_cast<const T*>(bias), idx, wgt, rows, E, top, scored);
+          logits, ldl, static_cast<const T*>(bias), idx, wgt, rows, E, top, scored);
     });
     return static_cast<int>(cudaGetLastError());
   }

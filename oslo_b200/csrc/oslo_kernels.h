@@ -352,8 +352,8 @@ int oslo_scan_step(const void* x, long long ldx, const void* dt, long long lddt,
 // route: idx, wgt [rows, top]; scored: scores are the softmax over all E outputs, bias only enters the choice, weights are the chosen
 // scores over their sum. Choices >= the experts of plan / few get no slot (-1) and no product. unit: 0 none, 1 relu^2, 2 silu(gate) *
 // up of column pairs (out has N / 2 columns)
-int oslo_moe_route(const void* h, long long ldh, const void* w, const void* bias, const float* logits, int* idx, float* wgt,
-                   long long rows, int E, int K, int top, int scored, int dtype, cudaStream_t stream);
+int oslo_moe_route(const void* h, long long ldh, const void* w, const void* bias, const float* logits, long long ldl, int* idx,
+                   float* wgt, long long rows, int E, int K, int top, int scored, int dtype, cudaStream_t stream);
 int oslo_moe_plan(const void* h, long long ldh, const int* idx, int* cursor, int* tile_group, int* n_tiles, int* slots,
                   void* rows_out, long long pairs, int E, int K, int top, int max_tiles, int dtype, cudaStream_t stream);
 int oslo_moe_grouped(const void* a, const void* w, void* out, const int* tile_group, const int* n_tiles, int max_tiles, int N,

@@ -399,8 +399,8 @@ def bench_branches(args, timer: _Timer) -> None:
 
 # width, streams, attention heads, kv heads, head dim, window, kept, latent dim, rot, vdim, q_rank, kv_rank, memory heads x dim x vdim,
 # experts, identity, top, ff
-STREAM_CASES = [(2048, 4, 16, 4, 128, 512, 16, 128, 64, 128, 1024, 512, 16, 128, 128, 16, 4, 4, 1344),
-                (4096, 4, 32, 8, 128, 1024, 16, 128, 64, 128, 1536, 512, 32, 128, 128, 32, 4, 4, 2688)]
+STREAM_CASES = [(2048, 4, 16, 4, 128, 512, 16, 128, 64, 128, 1024, 512, 16, 128, 128, 16, 3, 4, 1344),
+                (4096, 4, 32, 8, 128, 1024, 16, 128, 64, 128, 1536, 512, 32, 128, 128, 32, 3, 4, 2688)]
 
 
 def bench_streams(args, timer: _Timer) -> None:

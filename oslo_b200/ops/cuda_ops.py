@@ -915,8 +915,8 @@ MOE_FEW_PAIRS = 8   # (token, choice) pairs up to which the chosen experts' weig
 
 def moe_route(h: Tensor, w: Tensor, bias: Tensor, top: int, scored: bool = False):
     logits = None
-    if h.size(0) > SMALL_M_ROWS and gemm_ok(h, w) and h.size(1) % 8 == 0 and (w.size(0) < 32 or w.size(0) % 4 == 0):
-        logits = gemm(h, w, flags=FLAG_OUT_FP32)           # 16-bit operands, exact products, fp32 sums and output
+    if h.size(0) > SMALL_M_ROWS and gemm_ok(h, w):
+        logits = linear_fp32(h, w)                         # 16-bit operands, exact products, fp32 sums and output
     elif h.size(0) > 65535:                                # no tensor-core path for these sizes or types: 32-bit library product
         logits = torch.matmul(h.float(), w.float().t())
     return _ext().moe_route(_rows(h), w, bias, logits, top, scored)

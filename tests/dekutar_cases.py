@@ -38,7 +38,7 @@ CASES = {
                 latent(3, 5, 6, 11, 13, 9, 0.4, moe(9, 5, 4, 3, 5)), attn(6, 3, 6, 0.9, 1, 5, 2, moe(11, 2, 1, 1, 3)),
                 latent(1, 3, 2, 7, 5, 17, 0.6, None), mlstm(1, 13, 3, 30.0, None), scale=1.7, logit_scale=1.3),
     # head sizes the tensor-core kernels take as they are, groups of several sizes
-    "heads64": case(128, 128, 1e-6, 2, latent(4, 64, 64, 128, 96, 64, 0.1, moe(64, 12, 4, 4, 96)), attn(4, 1, 128, 0.1, 33, 9, 64, moe(96, 8, 0, 2, 64)),
+    "heads64": case(128, 128, 1e-6, 2, latent(4, 64, 64, 128, 96, 64, 0.1, moe(64, 12, 5, 4, 88)), attn(4, 1, 128, 0.1, 33, 9, 64, moe(96, 8, 0, 2, 64)),
                     mlstm(2, 64, 128, 12.0, moe(48, 6, 2, 6, 128)), latent(2, 128, 64, 64, 64, 128, 0.08, moe(32, 4, 4, 2, 32)),
                     attn(8, 4, 64, 0.13, 24, 17, 16, None), mlstm(4, 32, 32, 6.0, None)),
     # one stream, one head, one expert, sizes of 1; windows of one position, nothing kept, no identity experts

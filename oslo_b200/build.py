@@ -86,23 +86,34 @@ def build_kernels(force: bool = False, verbose: bool = True, debug_bounds: bool 
     inc = ["-I" + CSRC, "-I" + os.path.join(cuda_home, "include")]
     tinc = ["-I" + p for p in cpp_extension.include_paths()]
     objs: List[str] = []
-    jobs = []
+    jobs, fresh = [], []
     suffix = ".bounds.o" if debug_bounds else ".o"
+
+    def queue(src: str, obj: str, cmd: List[str]) -> None:
+        """An object is compiled again when its source, a header or the command has changed."""
+        mine = _stamp([src] + headers, torch.__version__ + " ".join(cmd))
+        if force or _needs(obj, obj + ".stamp", mine):
+            jobs.append(cmd)
+            fresh.append((obj + ".stamp", mine))
+
     for src in cu:
         obj = os.path.join(BUILD, os.path.basename(src) + suffix)
         objs.append(obj)
         flags = [f for f in NVCC_FLAGS if f != "--use_fast_math" or os.path.basename(src) not in ACCURATE_SOURCES]
-        jobs.append([nvcc] + flags + extra + inc + ["-c", src, "-o", obj])
+        queue(src, obj, [nvcc] + flags + extra + inc + ["-c", src, "-o", obj])
     abi = int(torch._C._GLIBCXX_USE_CXX11_ABI)
     for src in cpp:
         obj = os.path.join(BUILD, os.path.basename(src) + suffix)
         objs.append(obj)
-        jobs.append(["g++", "-std=c++17", "-O2", "-fPIC", "-fvisibility=hidden", f"-D_GLIBCXX_USE_CXX11_ABI={abi}",
-                     "-DTORCH_EXTENSION_NAME=_C"] + inc + tinc + ["-c", src, "-o", obj])
+        queue(src, obj, ["g++", "-std=c++17", "-O2", "-fPIC", "-fvisibility=hidden", f"-D_GLIBCXX_USE_CXX11_ABI={abi}",
+                         "-DTORCH_EXTENSION_NAME=_C"] + inc + tinc + ["-c", src, "-o", obj])
     if verbose:
         print(f"[oslo_b200.build] compiling {len(jobs)} sources for sm_100a", flush=True)
-    with ThreadPoolExecutor(max_workers=min(8, len(jobs))) as ex:
+    with ThreadPoolExecutor(max_workers=max(1, min(8, len(jobs)))) as ex:
         list(ex.map(_run, jobs))
+    for path, text in fresh:
+        with open(path, "w") as f:
+            f.write(text)
     tlib = os.path.join(os.path.dirname(torch.__file__), "lib")
     link = ["g++", "-shared", "-o", out] + objs + [
         "-L" + tlib, "-L" + os.path.join(cuda_home, "lib64"), "-lc10", "-lc10_cuda", "-ltorch_cpu", "-ltorch_cuda",

@@ -54,6 +54,234 @@ struct FaParams {
   int q2_pos[3], k2_pos[3];
 };
 
+// Which blocks of BN keys the 128 query rows from q0 on read: the kept keys' blocks ahead of the window's come first
+struct FaBlocks {
+  int offset, lead, kept_lo, key_lo, nkept, n, bn;
+  __device__ __forceinline__ FaBlocks(const FaParams& p, int b, int q0, int BN) {
+    bn = BN;
+    offset = p.Sk - p.Sq;
+    int key_hi = p.Sk;
+    key_lo = 0;
+    if (p.causal) key_hi = min(p.Sk, q0 + FA_BM + offset);
+    if (p.window > 0) key_lo = max(0, q0 + offset - p.window + 1) / BN * BN;
+    lead = p.lead ? p.lead[b] : 0;
+    kept_lo = max(0, lead) / BN * BN;
+    const int kept_hi = min(key_lo, lead + p.keep_first);
+    nkept = kept_hi > kept_lo ? (kept_hi - kept_lo + BN - 1) / BN : 0;
+    n = nkept + (key_hi > key_lo ? (key_hi - key_lo + BN - 1) / BN : 0);
+  }
+  __device__ __forceinline__ int start(int j) const { return j < nkept ? kept_lo + j * bn : key_lo + (j - nkept) * bn; }
+};
+
+// The four softmax warps of both kernels: S from TMEM columns [0, BN) and [BN, 2 BN), O (D columns) from 2 BN on. Barriers by
+// number from bar0: 9,10 s_full | 11,12 s_empty | 13 p_ready[0] | 14 pv_done | 15 p_ready[1] (PT only: one per S/P buffer)
+template <int BN, bool PT, bool CAP>
+__device__ __forceinline__ void fa_softmax_warps(const FaParams& p, const int D, const FaBlocks& blocks, uint32_t tmem_base, uint32_t bar0,
+                                                 uint32_t p_s, volatile int* abort_flag, int warp, int lane, int b, int h, int q0) {
+  constexpr uint32_t Q_SUB = FA_BM * 128, O_COL = 2 * BN;
+  auto bar = [&](int i) { return bar0 + 8u * i; };
+  const int offset = blocks.offset;
+  const int quad = warp & 3;
+  const int row_l = quad * 32 + lane;
+  const int row = q0 + row_l;
+  const uint32_t t_lane = tmem_base + (static_cast<uint32_t>(quad * 32) << 16);
+  const uint8_t* kpm_row = p.kpm ? p.kpm + static_cast<long long>(b) * p.Sk : nullptr;
+  const float sc = CAP ? 2.f * FA_LOG2E * p.scale / p.softcap : p.scale * FA_LOG2E;
+  const float cap = p.softcap * FA_LOG2E;
+  const bool fp16 = p.fp16 != 0;
+  float m_ref = -CUDART_INF_F, l_sum = 0.f;
+  bool ok = true;
+  for (int j = 0; j < blocks.n && ok; ++j) {
+    const int st = j & 1;
+    const int n0 = blocks.start(j);
+    ok = mbar_wait(bar(9 + st), (j >> 1) & 1, abort_flag, p.err, ERR_WAIT_TMEM_FULL);
+    if (!ok) break;
+    tc_fence_after();
+    float s[BN];
+#pragma unroll
+    for (int c0 = 0; c0 < BN; c0 += 32) {
+      uint32_t r[32];
+      tmem_ld_32x32(t_lane + st * BN + c0, r);
+      tmem_wait_ld();
+#pragma unroll
+      for (int i = 0; i < 32; ++i) {
+        s[c0 + i] = __uint_as_float(r[i]) * sc;
+        if (CAP) s[c0 + i] = cap - __fdividef(2.f * cap, exp2f(s[c0 + i]) + 1.f);
+      }
+    }
+    tc_fence_before();
+    __syncwarp();
+    if (lane == 0) mbar_arrive(bar(11 + st));  // S buffer may be overwritten by Q K^T of block j + 2
+    // ---- mask (only blocks that touch the diagonal, the window edge, the end of the keys, or padding)
+    const bool need_mask = (n0 + BN > p.Sk) || kpm_row != nullptr ||
+                           (p.causal && n0 + BN - 1 > q0 + offset) ||
+                           (p.window > 0 && n0 <= q0 + FA_BM - 1 + offset - p.window);
+    if (need_mask) {
+      // one bit per column: up to `last`, and from `first` on or before `kept`
+      const int qpos = row + offset;
+      const int last = p.causal ? min(p.Sk - 1, qpos) : p.Sk - 1;
+      const int first = p.window > 0 ? qpos - p.window + 1 : 0, kept = p.window > 0 ? blocks.lead + p.keep_first : 0;
+      auto below = [](int n) { return n <= 0 ? 0u : (n >= 32 ? 0xffffffffu : (1u << n) - 1u); };
+#pragma unroll
+      for (int c0 = 0; c0 < BN; c0 += 32) {
+        const int base = n0 + c0;
+        uint32_t vis = below(last - base + 1) & (~below(first - base) | below(kept - base));
+        if (kpm_row) vis &= __ballot_sync(0xffffffffu, base + lane < p.Sk && kpm_row[base + lane] != 0);
+#pragma unroll
+        for (int i = 0; i < 32; ++i)
+          if (!((vis >> i) & 1u)) s[c0 + i] = -CUDART_INF_F;
+      }
+    }
+    // four independent chains: one thread per row means nothing else hides the latency of a 64-long dependent chain
+    float mx4[4] = {s[0], s[1], s[2], s[3]};
+#pragma unroll
+    for (int i = 4; i < BN; i += 4) {
+      mx4[0] = fmaxf(mx4[0], s[i]);
+      mx4[1] = fmaxf(mx4[1], s[i + 1]);
+      mx4[2] = fmaxf(mx4[2], s[i + 2]);
+      mx4[3] = fmaxf(mx4[3], s[i + 3]);
+    }
+    const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
+    const float m_new = fmaxf(m_ref, mx);
+    // rescale O only when some row of this warp outgrew its reference by 2^8 (or on the first block)
+    const bool grow = (j == 0) || (m_new - m_ref > FA_RESCALE_THRESHOLD);
+    const bool rescale = __any_sync(0xffffffffu, grow);
+    float factor = 1.f;
+    if (rescale) {
+      factor = (m_ref == -CUDART_INF_F) ? 0.f : exp2f(m_ref - m_new);
+      m_ref = m_new;
+      l_sum *= factor;
+    }
+    const float m_use = (m_ref == -CUDART_INF_F) ? 0.f : m_ref;
+    float ps4[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+    for (int i = 0; i < BN; i += 4) {
+      s[i] = exp2f(s[i] - m_use);
+      s[i + 1] = exp2f(s[i + 1] - m_use);
+      s[i + 2] = exp2f(s[i + 2] - m_use);
+      s[i + 3] = exp2f(s[i + 3] - m_use);
+      ps4[0] += s[i];
+      ps4[1] += s[i + 1];
+      ps4[2] += s[i + 2];
+      ps4[3] += s[i + 3];
+    }
+    l_sum += (ps4[0] + ps4[1]) + (ps4[2] + ps4[3]);
+    // the shared P tile is single-buffered, so P V of block j-1 must have finished before it is rewritten; the
+    // TMEM P buffers alternate, so there only a rescale of O has to wait for it
+    if (j > 0 && (!PT || rescale)) {
+      ok = mbar_wait(bar(14), (j - 1) & 1, abort_flag, p.err, ERR_WAIT_TMEM_FULL);
+      if (!ok) break;
+      tc_fence_after();
+      if (rescale) {
+#pragma unroll 1
+        for (int c0 = 0; c0 < D; c0 += 32) {
+          uint32_t r[32];
+          tmem_ld_32x32(t_lane + O_COL + c0, r);
+          tmem_wait_ld();
+#pragma unroll
+          for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * factor);
+          tmem_st_32x32(t_lane + O_COL + c0, r);
+        }
+        tmem_wait_st();
+      }
+    }
+    if constexpr (PT) {
+#pragma unroll
+      for (int c0 = 0; c0 < BN / 2; c0 += 32) {
+        uint32_t r[32];
+#pragma unroll
+        for (int i = 0; i < 32; ++i) r[i] = fa_pack2(s[2 * (c0 + i)], s[2 * (c0 + i) + 1], fp16);
+        tmem_st_32x32(t_lane + st * BN + c0, r);
+      }
+      tmem_wait_st();
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(bar(st ? 15 : 13));
+    } else {
+    // ---- P (bf16) into shared memory: K-major, 128-byte swizzle: 16-byte chunk c of row r sits at c ^ (r & 7)
+#pragma unroll
+    for (int c = 0; c < BN / 64; ++c) {
+#pragma unroll
+      for (int q = 0; q < 8; ++q) {
+        const int i0 = c * 64 + q * 8;
+        uint4 v;
+        v.x = fa_pack2(s[i0], s[i0 + 1], fp16); v.y = fa_pack2(s[i0 + 2], s[i0 + 3], fp16);
+        v.z = fa_pack2(s[i0 + 4], s[i0 + 5], fp16); v.w = fa_pack2(s[i0 + 6], s[i0 + 7], fp16);
+        const uint32_t addr = p_s + c * Q_SUB + row_l * 128 + ((q ^ (row_l & 7)) << 4);
+        asm volatile("st.shared.v4.b32 [%0], {%1, %2, %3, %4};" ::"r"(addr), "r"(v.x), "r"(v.y), "r"(v.z), "r"(v.w) : "memory");
+      }
+    }
+    fence_proxy_async_smem();   // generic-proxy writes -> visible to the tensor core's async proxy
+    tc_fence_before();
+    __syncwarp();
+    if (lane == 0) mbar_arrive(bar(13));
+    }
+  }
+  // ---- epilogue: O / l -> global, log-sum-exp
+  if (ok && blocks.n > 0) {
+    ok = mbar_wait(bar(14), (blocks.n - 1) & 1, abort_flag, p.err, ERR_WAIT_TMEM_FULL);
+    tc_fence_after();
+  }
+  float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
+  const long long gate_row = (static_cast<long long>(b) * p.Sq + row) * p.ldg;
+  const bool wide = p.gate != nullptr && p.gate_wide;
+  if ((p.sink != nullptr || p.gate != nullptr) && row < p.Sq && l_sum > 0.f) {
+    const long long gi = gate_row + h;
+    inv = l_sum;
+    if (p.sink != nullptr) {
+      const float snk = fp16 ? __half2float(static_cast<const __half*>(p.sink)[h])
+                             : __bfloat162float(static_cast<const __nv_bfloat16*>(p.sink)[h]);
+      // m_ref is the running reference in log2 units; an overflowing sink term gives 1 / inf = 0
+      inv += exp2f(snk * 1.4426950408889634f - m_ref);
+    }
+    if (p.gate != nullptr && !wide) {
+      const float gate = fp16 ? __half2float(static_cast<const __half*>(p.gate)[gi])
+                              : __bfloat162float(static_cast<const __nv_bfloat16*>(p.gate)[gi]);
+      inv *= 1.f + exp2f(-gate * 1.4426950408889634f);
+    }
+    inv = 1.f / inv;
+  }
+  uint16_t* orow = reinterpret_cast<uint16_t*>(p.out) + b * p.o_sb + h * p.o_sh + static_cast<long long>(row) * p.o_ss;
+#pragma unroll 1
+  for (int c0 = 0; c0 < D; c0 += 32) {
+    uint32_t r[32];
+    if (blocks.n > 0 && ok) {
+      tmem_ld_32x32(t_lane + O_COL + c0, r);
+      tmem_wait_ld();
+    } else {
+#pragma unroll
+      for (int i = 0; i < 32; ++i) r[i] = 0u;
+    }
+    if (row < p.Sq) {
+#pragma unroll
+      for (int i = 0; i < 32; i += 8) {
+        if (c0 + i >= p.d_out) break;
+        if (wide) {
+          const uint4 g4 = *reinterpret_cast<const uint4*>(static_cast<const uint16_t*>(p.gate) + gate_row + h * p.d_out + c0 + i);
+          const uint32_t gw[4] = {g4.x, g4.y, g4.z, g4.w};
+#pragma unroll
+          for (int u = 0; u < 4; ++u) {
+            const float2 g = fp16 ? __half22float2(*reinterpret_cast<const __half2*>(&gw[u]))
+                                  : __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gw[u]));
+            r[i + 2 * u] = __float_as_uint(__fdividef(__uint_as_float(r[i + 2 * u]), 1.f + exp2f(-g.x * 1.4426950408889634f)));
+            r[i + 2 * u + 1] = __float_as_uint(__fdividef(__uint_as_float(r[i + 2 * u + 1]), 1.f + exp2f(-g.y * 1.4426950408889634f)));
+          }
+        }
+        uint4 v;
+        v.x = fa_pack2(__uint_as_float(r[i]) * inv, __uint_as_float(r[i + 1]) * inv, fp16);
+        v.y = fa_pack2(__uint_as_float(r[i + 2]) * inv, __uint_as_float(r[i + 3]) * inv, fp16);
+        v.z = fa_pack2(__uint_as_float(r[i + 4]) * inv, __uint_as_float(r[i + 5]) * inv, fp16);
+        v.w = fa_pack2(__uint_as_float(r[i + 6]) * inv, __uint_as_float(r[i + 7]) * inv, fp16);
+        *reinterpret_cast<uint4*>(orow + c0 + i) = v;
+      }
+    }
+  }
+  if (row < p.Sq && p.lse) {
+    const float lse = l_sum > 0.f ? (m_ref + log2f(l_sum)) * FA_LN2 : 0.f;
+    p.lse[(static_cast<long long>(b) * p.H + h) * p.Sq + row] = lse;
+  }
+}
+
 // PT = true: P goes back into TMEM (over the S buffer it came from, two bf16 per 32-bit column) and is the
 // A operand of P V straight from tensor memory; PT = false: P goes through a swizzled shared-memory tile.
 // CAP = true: capped scores, tanh(u) = 1 - 2 / (exp(2u) + 1) in 32-bit (absolute error about 2^-23 of the cap).
@@ -92,16 +320,8 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int b = blockIdx.z, h = blockIdx.y;
   const int q0 = (static_cast<int>(gridDim.x) - 1 - static_cast<int>(blockIdx.x)) * FA_BM;  // long (late) rows first
-  const int offset = p.Sk - p.Sq;
-  int key_hi = p.Sk, key_lo = 0;
-  if (p.causal) key_hi = min(p.Sk, q0 + FA_BM + offset);
-  if (p.window > 0) key_lo = max(0, q0 + offset - p.window + 1) / BN * BN;
-  // the kept keys' blocks ahead of the window's come first
-  const int lead = p.lead ? p.lead[b] : 0;
-  const int kept_lo = max(0, lead) / BN * BN, kept_hi = min(key_lo, lead + p.keep_first);
-  const int nkept = kept_hi > kept_lo ? (kept_hi - kept_lo + BN - 1) / BN : 0;
-  const int nblk = nkept + (key_hi > key_lo ? (key_hi - key_lo + BN - 1) / BN : 0);
-  auto block_start = [&](int j) { return j < nkept ? kept_lo + j * BN : key_lo + (j - nkept) * BN; };
+  const FaBlocks blocks(p, b, q0, BN);
+  const int nblk = blocks.n;
 
   if (threadIdx.x == 0) {
     for (int i = 0; i < 16; ++i) {
@@ -135,7 +355,7 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
       for (int j = 0; j < nblk && ok; ++j) {
         const int st = j & 1;
         const uint32_t ph = (j >> 1) & 1;
-        const int n0 = block_start(j);
+        const int n0 = blocks.start(j);
         ok = mbar_wait(bar(3 + st), ph ^ 1, abort_flag, p.err, ERR_WAIT_EMPTY);
         if (!ok) break;
         mbar_expect_tx(bar(1 + st), K_BYTES);
@@ -204,205 +424,166 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
     }
   } else {
     // ------------------------------------------------------------------ softmax / correction / epilogue
-    const int quad = warp & 3;
-    const int row_l = quad * 32 + lane;
-    const int row = q0 + row_l;
-    const uint32_t t_lane = tmem_base + (static_cast<uint32_t>(quad * 32) << 16);
-    const uint8_t* kpm_row = p.kpm ? p.kpm + static_cast<long long>(b) * p.Sk : nullptr;
-    const float sc = CAP ? 2.f * FA_LOG2E * p.scale / p.softcap : p.scale * FA_LOG2E;
-    const float cap = p.softcap * FA_LOG2E;
-    const bool fp16 = p.fp16 != 0;
-    float m_ref = -CUDART_INF_F, l_sum = 0.f;
-    bool ok = true;
-    for (int j = 0; j < nblk && ok; ++j) {
-      const int st = j & 1;
-      const int n0 = block_start(j);
-      ok = mbar_wait(bar(9 + st), (j >> 1) & 1, abort_flag, p.err, ERR_WAIT_TMEM_FULL);
-      if (!ok) break;
-      tc_fence_after();
-      float s[BN];
-#pragma unroll
-      for (int c0 = 0; c0 < BN; c0 += 32) {
-        uint32_t r[32];
-        tmem_ld_32x32(t_lane + st * BN + c0, r);
-        tmem_wait_ld();
-#pragma unroll
-        for (int i = 0; i < 32; ++i) {
-          s[c0 + i] = __uint_as_float(r[i]) * sc;
-          if (CAP) s[c0 + i] = cap - __fdividef(2.f * cap, exp2f(s[c0 + i]) + 1.f);
+    fa_softmax_warps<BN, PT, CAP>(p, D, blocks, tmem_base, bar0, p_s, abort_flag, warp, lane, b, h, q0);
+  }
+
+  if (*abort_flag) {
+    const uint64_t t0 = globaltimer_ns();
+    while (globaltimer_ns() - t0 < 200000ull) {
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tmem_base, TMEM_COLS);
+  }
+}
+
+// ---------------------------------------------------------------------- wide keys
+// Queries and keys of any width (`chunks` sub-tiles of 64 columns), one key head for all query heads, value heads per group: attention whose
+// heads are mixed before the softmax, with the mix folded into the queries (grouped_attention.cu). All operands are sub-tiles
+// of 128 rows x 64 columns in 16 KB slots: the first FW_RESIDENT of the queries stay, everything else - keys, values, the rest of the
+// queries - passes through a ring in the order in which the MMA warp uses it, Q K^T of block j + 1 ahead of P V of block j.
+constexpr int FW_SLOTS = 14, FW_RESIDENT = 8;
+constexpr uint32_t FW_SLOT = 128 * 128;
+
+__global__ void __launch_bounds__(FA_THREADS, 1)
+fa_wide_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUtensorMap tk, const __grid_constant__ CUtensorMap tv,
+               const FaParams p, const int dim) {
+  constexpr int BN = 128;
+  constexpr uint32_t TMEM_COLS = 512, O_COL = 2 * BN;
+  extern __shared__ uint8_t fa_smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(fa_smem_raw) + 1023) & ~uintptr_t(1023));
+  const int chunks = (dim + 63) / 64, resident = min(chunks, FW_RESIDENT), ring = FW_SLOTS - resident, vc = (p.d_out + 63) / 64;
+  const uint32_t q_s = smem_u32(smem), ring_s = q_s + resident * FW_SLOT;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + FW_SLOTS * FW_SLOT);
+  const uint32_t bar0 = smem_u32(bars);
+  // 0 q_full | 9.. as in fa_softmax_warps | 16 + i slot i full | 16 + FW_SLOTS + i slot i empty
+  auto bar = [&](int i) { return bar0 + 8u * i; };
+  constexpr int BARS = 16 + 2 * FW_SLOTS;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + BARS);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int b = blockIdx.z, h = blockIdx.y;
+  const int q0 = (static_cast<int>(gridDim.x) - 1 - static_cast<int>(blockIdx.x)) * FA_BM;  // long (late) rows first
+  const FaBlocks blocks(p, b, q0, BN);
+  const int nblk = blocks.n;
+
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < BARS; ++i) {
+      const bool four = (i == 11 || i == 12 || i == 13 || i == 15);  // arrivals from the 4 softmax warps
+      mbar_init(bar(i), four ? 4 : 1);
+    }
+    *abort_flag = 0;
+    fence_barrier_init();
+  }
+  if (warp == 1) {
+    tmem_alloc(smem_u32(tmem_slot), TMEM_COLS);
+    tmem_relinquish();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_base = *tmem_slot;
+
+  // the slots in turn; `phase` is the parity of the ring's current round
+  struct Cursor {
+    int slot = 0;
+    uint32_t phase = 0;
+    __device__ __forceinline__ void next(int ring) {
+      if (++slot == ring) { slot = 0; phase ^= 1; }
+    }
+  };
+
+  if (warp == 0) {
+    // ------------------------------------------------------------------ TMA producer
+    if (lane == 0 && nblk > 0) {
+      tma_prefetch_desc(&tq); tma_prefetch_desc(&tk); tma_prefetch_desc(&tv);
+      mbar_expect_tx(bar(0), resident * FW_SLOT);
+      for (int c = 0; c < resident; ++c) tma_load_rows(q_s + c * FW_SLOT, &tq, bar(0), c * 64, q0, h, b, p.q_pos);
+      Cursor at;
+      bool ok = true;
+      auto load = [&](const CUtensorMap* map, int col, int row, int head, const int* pos) {
+        ok = mbar_wait(bar(16 + FW_SLOTS + at.slot), at.phase ^ 1, abort_flag, p.err, ERR_WAIT_EMPTY);
+        if (!ok) return;
+        mbar_expect_tx(bar(16 + at.slot), FW_SLOT);
+        tma_load_rows(ring_s + at.slot * FW_SLOT, map, bar(16 + at.slot), col, row, head, b, pos);
+        at.next(ring);
+      };
+      auto keys = [&](int j) {
+        const int n0 = blocks.start(j);
+        for (int c = 0; c < chunks && ok; ++c) {
+          if (c >= resident) load(&tq, c * 64, q0, h, p.q_pos);
+          if (ok) load(&tk, c * 64, n0, 0, p.k_pos);
         }
+      };
+      keys(0);
+      for (int j = 0; j < nblk && ok; ++j) {
+        if (j + 1 < nblk) keys(j + 1);
+        for (int c = 0; c < vc && ok; ++c) load(&tv, c * 64, blocks.start(j), h / p.group, p.v_pos);
       }
-      tc_fence_before();
-      __syncwarp();
-      if (lane == 0) mbar_arrive(bar(11 + st));  // S buffer may be overwritten by Q K^T of block j + 2
-      // ---- mask (only blocks that touch the diagonal, the window edge, the end of the keys, or padding)
-      const bool need_mask = (n0 + BN > p.Sk) || kpm_row != nullptr ||
-                             (p.causal && n0 + BN - 1 > q0 + offset) ||
-                             (p.window > 0 && n0 <= q0 + FA_BM - 1 + offset - p.window);
-      if (need_mask) {
-        // one bit per column: up to `last`, and from `first` on or before `kept`
-        const int qpos = row + offset;
-        const int last = p.causal ? min(p.Sk - 1, qpos) : p.Sk - 1;
-        const int first = p.window > 0 ? qpos - p.window + 1 : 0, kept = p.window > 0 ? lead + p.keep_first : 0;
-        auto below = [](int n) { return n <= 0 ? 0u : (n >= 32 ? 0xffffffffu : (1u << n) - 1u); };
-#pragma unroll
-        for (int c0 = 0; c0 < BN; c0 += 32) {
-          const int base = n0 + c0;
-          uint32_t vis = below(last - base + 1) & (~below(first - base) | below(kept - base));
-          if (kpm_row) vis &= __ballot_sync(0xffffffffu, base + lane < p.Sk && kpm_row[base + lane] != 0);
-#pragma unroll
-          for (int i = 0; i < 32; ++i)
-            if (!((vis >> i) & 1u)) s[c0 + i] = -CUDART_INF_F;
-        }
-      }
-      // four independent chains: one thread per row means nothing else hides the latency of a 64-long dependent chain
-      float mx4[4] = {s[0], s[1], s[2], s[3]};
-#pragma unroll
-      for (int i = 4; i < BN; i += 4) {
-        mx4[0] = fmaxf(mx4[0], s[i]);
-        mx4[1] = fmaxf(mx4[1], s[i + 1]);
-        mx4[2] = fmaxf(mx4[2], s[i + 2]);
-        mx4[3] = fmaxf(mx4[3], s[i + 3]);
-      }
-      const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
-      const float m_new = fmaxf(m_ref, mx);
-      // rescale O only when some row of this warp outgrew its reference by 2^8 (or on the first block)
-      const bool grow = (j == 0) || (m_new - m_ref > FA_RESCALE_THRESHOLD);
-      const bool rescale = __any_sync(0xffffffffu, grow);
-      float factor = 1.f;
-      if (rescale) {
-        factor = (m_ref == -CUDART_INF_F) ? 0.f : exp2f(m_ref - m_new);
-        m_ref = m_new;
-        l_sum *= factor;
-      }
-      const float m_use = (m_ref == -CUDART_INF_F) ? 0.f : m_ref;
-      float ps4[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll
-      for (int i = 0; i < BN; i += 4) {
-        s[i] = exp2f(s[i] - m_use);
-        s[i + 1] = exp2f(s[i + 1] - m_use);
-        s[i + 2] = exp2f(s[i + 2] - m_use);
-        s[i + 3] = exp2f(s[i + 3] - m_use);
-        ps4[0] += s[i];
-        ps4[1] += s[i + 1];
-        ps4[2] += s[i + 2];
-        ps4[3] += s[i + 3];
-      }
-      l_sum += (ps4[0] + ps4[1]) + (ps4[2] + ps4[3]);
-      // the shared P tile is single-buffered, so P V of block j-1 must have finished before it is rewritten; the
-      // TMEM P buffers alternate, so there only a rescale of O has to wait for it
-      if (j > 0 && (!PT || rescale)) {
-        ok = mbar_wait(bar(14), (j - 1) & 1, abort_flag, p.err, ERR_WAIT_TMEM_FULL);
-        if (!ok) break;
+    }
+  } else if (warp == 1) {
+    // ------------------------------------------------------------------ MMA issuer
+    if (lane == 0 && nblk > 0) {
+      const int fmt = p.fp16 ? 0 : 1;
+      const uint32_t idesc_qk = make_idesc_f16(FA_BM, BN, fmt, 0, 0);
+      const uint32_t idesc_pv = make_idesc_f16(FA_BM, 64, fmt, 0, 1);
+      Cursor at;
+      bool ok = mbar_wait(bar(0), 0, abort_flag, p.err, ERR_WAIT_FULL);
+      auto issue_qk = [&](int j) -> bool {
+        const int st = j & 1;
+        if (!mbar_wait(bar(11 + st), ((j >> 1) & 1) ^ 1, abort_flag, p.err, ERR_WAIT_TMEM_EMPTY)) return false;
         tc_fence_after();
-        if (rescale) {
-#pragma unroll 1
-          for (int c0 = 0; c0 < D; c0 += 32) {
-            uint32_t r[32];
-            tmem_ld_32x32(t_lane + O_COL + c0, r);
-            tmem_wait_ld();
-#pragma unroll
-            for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * factor);
-            tmem_st_32x32(t_lane + O_COL + c0, r);
+        for (int c = 0; c < chunks; ++c) {
+          uint32_t a = q_s + c * FW_SLOT;
+          int a_slot = -1;
+          if (c >= resident) {
+            if (!mbar_wait(bar(16 + at.slot), at.phase, abort_flag, p.err, ERR_WAIT_FULL)) return false;
+            a_slot = at.slot;
+            a = ring_s + at.slot * FW_SLOT;
+            at.next(ring);
           }
-          tmem_wait_st();
+          if (!mbar_wait(bar(16 + at.slot), at.phase, abort_flag, p.err, ERR_WAIT_FULL)) return false;
+          tc_fence_after();
+          const uint32_t k_s = ring_s + at.slot * FW_SLOT;
+          const int steps = min(4, (dim - c * 64 + 15) / 16);
+          for (int kk = 0; kk < steps; ++kk)
+            umma_f16(tmem_base + st * BN, make_smem_desc(a + kk * 32, 16, 1024), make_smem_desc(k_s + kk * 32, 16, 1024), idesc_qk,
+                     (c | kk) != 0);
+          if (a_slot >= 0) umma_commit(bar(16 + FW_SLOTS + a_slot));   // the slots may be refilled once these MMAs have read them
+          umma_commit(bar(16 + FW_SLOTS + at.slot));
+          at.next(ring);
         }
-      }
-      if constexpr (PT) {
-#pragma unroll
-        for (int c0 = 0; c0 < BN / 2; c0 += 32) {
-          uint32_t r[32];
-#pragma unroll
-          for (int i = 0; i < 32; ++i) r[i] = fa_pack2(s[2 * (c0 + i)], s[2 * (c0 + i) + 1], fp16);
-          tmem_st_32x32(t_lane + st * BN + c0, r);
+        umma_commit(bar(9 + st));   // S_j is ready for the softmax warps
+        return true;
+      };
+      if (ok) ok = issue_qk(0);
+      for (int j = 0; j < nblk && ok; ++j) {
+        if (j + 1 < nblk) {
+          ok = issue_qk(j + 1);
+          if (!ok) break;
         }
-        tmem_wait_st();
-        tc_fence_before();
-        __syncwarp();
-        if (lane == 0) mbar_arrive(bar(st ? 15 : 13));
-      } else {
-      // ---- P (bf16) into shared memory: K-major, 128-byte swizzle: 16-byte chunk c of row r sits at c ^ (r & 7)
+        const int st = j & 1;
+        ok = mbar_wait(bar(st ? 15 : 13), (j >> 1) & 1, abort_flag, p.err, ERR_WAIT_FULL);
+        for (int c = 0; c < vc && ok; ++c) {
+          ok = mbar_wait(bar(16 + at.slot), at.phase, abort_flag, p.err, ERR_WAIT_FULL);
+          if (!ok) break;
+          tc_fence_after();
 #pragma unroll
-      for (int c = 0; c < BN / 64; ++c) {
-#pragma unroll
-        for (int q = 0; q < 8; ++q) {
-          const int i0 = c * 64 + q * 8;
-          uint4 v;
-          v.x = fa_pack2(s[i0], s[i0 + 1], fp16); v.y = fa_pack2(s[i0 + 2], s[i0 + 3], fp16);
-          v.z = fa_pack2(s[i0 + 4], s[i0 + 5], fp16); v.w = fa_pack2(s[i0 + 6], s[i0 + 7], fp16);
-          const uint32_t addr = p_s + c * Q_SUB + row_l * 128 + ((q ^ (row_l & 7)) << 4);
-          asm volatile("st.shared.v4.b32 [%0], {%1, %2, %3, %4};" ::"r"(addr), "r"(v.x), "r"(v.y), "r"(v.z), "r"(v.w) : "memory");
+          for (int ks = 0; ks < BN / 16; ++ks)
+            umma_f16_ts(tmem_base + O_COL + c * 64, tmem_base + st * BN + ks * 8,
+                        make_smem_desc(ring_s + at.slot * FW_SLOT + ks * 2048, FW_SLOT, 1024), idesc_pv, (j | ks) != 0);
+          umma_commit(bar(16 + FW_SLOTS + at.slot));
+          at.next(ring);
         }
-      }
-      fence_proxy_async_smem();   // generic-proxy writes -> visible to the tensor core's async proxy
-      tc_fence_before();
-      __syncwarp();
-      if (lane == 0) mbar_arrive(bar(13));
+        if (ok) umma_commit(bar(14));   // O updated, P buffer reusable
       }
     }
-    // ---- epilogue: O / l -> global, log-sum-exp
-    if (ok && nblk > 0) {
-      ok = mbar_wait(bar(14), (nblk - 1) & 1, abort_flag, p.err, ERR_WAIT_TMEM_FULL);
-      tc_fence_after();
-    }
-    float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
-    const long long gate_row = (static_cast<long long>(b) * p.Sq + row) * p.ldg;
-    const bool wide = p.gate != nullptr && p.gate_wide;
-    if ((p.sink != nullptr || p.gate != nullptr) && row < p.Sq && l_sum > 0.f) {
-      const long long gi = gate_row + h;
-      inv = l_sum;
-      if (p.sink != nullptr) {
-        const float snk = fp16 ? __half2float(static_cast<const __half*>(p.sink)[h])
-                               : __bfloat162float(static_cast<const __nv_bfloat16*>(p.sink)[h]);
-        // m_ref is the running reference in log2 units; an overflowing sink term gives 1 / inf = 0
-        inv += exp2f(snk * 1.4426950408889634f - m_ref);
-      }
-      if (p.gate != nullptr && !wide) {
-        const float gate = fp16 ? __half2float(static_cast<const __half*>(p.gate)[gi])
-                                : __bfloat162float(static_cast<const __nv_bfloat16*>(p.gate)[gi]);
-        inv *= 1.f + exp2f(-gate * 1.4426950408889634f);
-      }
-      inv = 1.f / inv;
-    }
-    uint16_t* orow = reinterpret_cast<uint16_t*>(p.out) + b * p.o_sb + h * p.o_sh + static_cast<long long>(row) * p.o_ss;
-#pragma unroll 1
-    for (int c0 = 0; c0 < D; c0 += 32) {
-      uint32_t r[32];
-      if (nblk > 0 && ok) {
-        tmem_ld_32x32(t_lane + O_COL + c0, r);
-        tmem_wait_ld();
-      } else {
-#pragma unroll
-        for (int i = 0; i < 32; ++i) r[i] = 0u;
-      }
-      if (row < p.Sq) {
-#pragma unroll
-        for (int i = 0; i < 32; i += 8) {
-          if (c0 + i >= p.d_out) break;
-          if (wide) {
-            const uint4 g4 = *reinterpret_cast<const uint4*>(static_cast<const uint16_t*>(p.gate) + gate_row + h * p.d_out + c0 + i);
-            const uint32_t gw[4] = {g4.x, g4.y, g4.z, g4.w};
-#pragma unroll
-            for (int u = 0; u < 4; ++u) {
-              const float2 g = fp16 ? __half22float2(*reinterpret_cast<const __half2*>(&gw[u]))
-                                    : __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gw[u]));
-              r[i + 2 * u] = __float_as_uint(__fdividef(__uint_as_float(r[i + 2 * u]), 1.f + exp2f(-g.x * 1.4426950408889634f)));
-              r[i + 2 * u + 1] = __float_as_uint(__fdividef(__uint_as_float(r[i + 2 * u + 1]), 1.f + exp2f(-g.y * 1.4426950408889634f)));
-            }
-          }
-          uint4 v;
-          v.x = fa_pack2(__uint_as_float(r[i]) * inv, __uint_as_float(r[i + 1]) * inv, fp16);
-          v.y = fa_pack2(__uint_as_float(r[i + 2]) * inv, __uint_as_float(r[i + 3]) * inv, fp16);
-          v.z = fa_pack2(__uint_as_float(r[i + 4]) * inv, __uint_as_float(r[i + 5]) * inv, fp16);
-          v.w = fa_pack2(__uint_as_float(r[i + 6]) * inv, __uint_as_float(r[i + 7]) * inv, fp16);
-          *reinterpret_cast<uint4*>(orow + c0 + i) = v;
-        }
-      }
-    }
-    if (row < p.Sq && p.lse) {
-      const float lse = l_sum > 0.f ? (m_ref + log2f(l_sum)) * FA_LN2 : 0.f;
-      p.lse[(static_cast<long long>(b) * p.H + h) * p.Sq + row] = lse;
-    }
+  } else {
+    fa_softmax_warps<BN, true, false>(p, vc * 64, blocks, tmem_base, bar0, 0u, abort_flag, warp, lane, b, h, q0);
   }
 
   if (*abort_flag) {
@@ -545,4 +726,45 @@ extern "C" int oslo_flash_sink_fwd_sm100(const void* q, const void* k, const voi
   x.q2_sb = q2_sb; x.q2_sh = q2_sh; x.q2_ss = q2_ss; x.k2_sb = k2_sb; x.k2_ss = k2_ss;
   return oslo::flash_fwd_entry(q, k, v, o, nullptr, kpm, sink, gate, ldg, B, H, G, Sq, Sk, dim, vdim, q_sb, q_sh, q_ss, k_sb, k_sh,
                                k_ss, v_sb, v_sh, v_ss, o_sb, o_sh, o_ss, scale, softcap, 1, window, dtype, err_word, stream, x);
+}
+
+// q [B, H, Sq, dim], k [B, Sk, dim] (one head for all), v [B, G, Sk, vdim]
+extern "C" int oslo_flash_wide_fwd_sm100(const void* q, const void* k, const void* v, void* o, const uint8_t* kpm, const void* sink,
+                                         const void* gate, long long ldg, int gate_wide, int B, int H, int G, int Sq, int Sk, int dim,
+                                         int vdim, long long q_sb, long long q_sh, long long q_ss, long long k_sb, long long k_ss,
+                                         long long v_sb, long long v_sh, long long v_ss, long long o_sb, long long o_sh,
+                                         long long o_ss, float scale, int window, int keep_first, const int* lead, int dtype,
+                                         int* err_word, cudaStream_t stream) {
+  using namespace oslo;
+  if (B <= 0 || H <= 0 || Sq <= 0 || Sk < Sq || G <= 0 || H % G) return -1;
+  if (dim <= 0 || vdim <= 0 || vdim > 256 || dim % 8 || vdim % 8) return -2;
+  if (dtype != OSLO_DT_BF16 && dtype != OSLO_DT_FP16) return -3;
+  if ((reinterpret_cast<uintptr_t>(o) & 15) || (o_sb % 8) || (o_sh % 8) || (o_ss % 8)) return -4;
+  if (gate_wide && (ldg % 8 || (reinterpret_cast<uintptr_t>(gate) & 15))) return -4;
+  static thread_local bool ctx_bound = false;
+  if (!ctx_bound) { cudaFree(nullptr); ctx_bound = true; }
+  const bool fp16 = dtype == OSLO_DT_FP16;
+  FaParams p{};
+  p.out = o; p.lse = nullptr; p.kpm = kpm; p.B = B; p.H = H; p.Sq = Sq; p.Sk = Sk;
+  p.o_sb = o_sb; p.o_sh = o_sh; p.o_ss = o_ss;
+  p.scale = scale; p.causal = 1; p.window = window; p.fp16 = fp16 ? 1 : 0; p.err = err_word; p.group = H / G; p.softcap = 0.f;
+  p.sink = sink; p.gate = gate; p.ldg = ldg; p.d_out = vdim; p.gate_wide = gate_wide;
+  p.keep_first = window > 0 ? keep_first : 0; p.lead = lead;
+  FaMaps t;
+  int rc = make_qkv_map(&t.q, q, B, H, Sq, dim, q_sb, q_sh, q_ss, FA_BM, fp16, p.q_pos);
+  if (rc) return rc;
+  rc = make_qkv_map(&t.k, k, B, 1, Sk, dim, k_sb, k_ss, k_ss, 128, fp16, p.k_pos);   // one head: its stride only has to be valid
+  if (rc) return rc - 1000;
+  rc = make_qkv_map(&t.v, v, B, G, Sk, vdim, v_sb, v_sh, v_ss, 128, fp16, p.v_pos);
+  if (rc) return rc - 2000;
+  constexpr size_t smem = FW_SLOTS * FW_SLOT + (16 + 2 * FW_SLOTS) * 8 + 16 + 1024;
+  static_assert(smem <= 232448, "shared memory budget of one CTA");
+  static bool configured = false;
+  if (!configured) {
+    cudaError_t e = cudaFuncSetAttribute(fa_wide_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
+    if (e != cudaSuccess) return static_cast<int>(e);
+    configured = true;
+  }
+  fa_wide_kernel<<<dim3((Sq + FA_BM - 1) / FA_BM, H, B), FA_THREADS, smem, stream>>>(t.q, t.k, t.v, p, dim);
+  return static_cast<int>(cudaGetLastError());
 }

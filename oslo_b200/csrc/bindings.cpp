@@ -219,7 +219,7 @@ Tensor gemm_small_m(const Tensor& a, const Tensor& b, int64_t b_mn, const option
   if (has_bias)
     TORCH_CHECK(bias->numel() == N && bias->scalar_type() == a.scalar_type() && bias->is_contiguous(), "bad bias");
   if (split <= 1 && gelu_from <= 0) {
-    const int64_t fl = (has_bias ? GEMM_FLAG_BIAS : 0) | (gelu_from == 0 ? GEMM_FLAG_GELU : 0);
+    const int64_t fl = (has_bias ? GEMM_FLAG_BIAS : 0) | (gelu_from == 0 ? GEMM_FLAG_GELU : 0) | (gelu_from == OSLO_ACT_RELU2 ? GEMM_FLAG_RELU2 : 0);
     return gemm(a, b, 0, b_mn, bias, optional<Tensor>(), optional<Tensor>(), optional<Tensor>(), fl, 1.0);
   }
   Tensor ws = at::empty({split, M, N}, a.options().dtype(at::kFloat));
@@ -736,12 +736,12 @@ const uint8_t* keep_ptr(const optional<Tensor>& keep, int64_t rows, int64_t cols
 
 Tensor rms_norm(const Tensor& x, const Tensor& w, double eps, double offset) {
   check_rows(x, "x");
-  TORCH_CHECK(w.is_contiguous() && w.numel() == x.size(1), "rms_norm: weight size");
+  TORCH_CHECK(w.is_cuda() && w.is_contiguous() && (w.numel() == x.size(1) || w.numel() == 1), "rms_norm: weight size");
   TORCH_CHECK(x.scalar_type() == w.scalar_type() || x.scalar_type() == at::kFloat, "rms_norm: x is fp32 or has the weight's type");
   c10::cuda::CUDAGuard guard(x.device());
   Tensor out = at::empty({x.size(0), x.size(1)}, w.options());
-  check_rc(oslo_rms_norm(x.data_ptr(), x.stride(0), x.scalar_type() == at::kFloat, w.data_ptr(), out.data_ptr(), out.stride(0),
-                         x.size(0), static_cast<int>(x.size(1)), static_cast<float>(eps), static_cast<float>(offset), dt_code(w),
+  check_rc(oslo_rms_norm(x.data_ptr(), x.stride(0), x.scalar_type() == at::kFloat, w.data_ptr(), w.numel() != x.size(1), out.data_ptr(),
+                         out.stride(0), x.size(0), static_cast<int>(x.size(1)), static_cast<float>(eps), static_cast<float>(offset), dt_code(w),
                          cur_stream()), "rms_norm");
   return out;
 }
@@ -806,38 +806,83 @@ Tensor clamped_glu(const Tensor& gate, const Tensor& up, double limit, double al
 }
 
 // up to three results join the stream; h1 / h2: the sum normed with w1 / w2 (empty without them)
-std::tuple<Tensor, Tensor, Tensor> branch_join(const Tensor& x, const Tensor& y0, const optional<Tensor>& n0, double f0,
-                                               const optional<Tensor>& y1, const optional<Tensor>& n1, double f1,
-                                               const optional<Tensor>& y2, const optional<Tensor>& n2, double f2, double mult,
-                                               double eps, const optional<Tensor>& w1, const optional<Tensor>& w2) {
+void check_state(const Tensor& state, int64_t n);
+using OptList = c10::List<optional<Tensor>>;
+
+// up to three branches y[i] with weights w[i] (normed[i] or elementwise), the sums of top[i] rows slots[i] where top[i] > 0; two norms of
+// the sum, or a copy of it; for single tokens also the convolution of the first norm (conv_w, prev). See oslo_kernels.h
+std::tuple<Tensor, Tensor, Tensor, Tensor> branch_join(const Tensor& x, at::TensorList y, const OptList& w, at::ArrayRef<double> factor,
+                                                       at::IntArrayRef normed, const OptList& slots, at::IntArrayRef top, double mult,
+                                                       double eps, const optional<Tensor>& w1, const optional<Tensor>& w2, bool copy,
+                                                       const optional<Tensor>& conv_w, optional<Tensor> prev,
+                                                       const optional<Tensor>& keep) {
   check_rows(x, "x");
-  const int64_t rows = x.size(0), cols = x.size(1);
+  const int64_t rows = x.size(0), cols = x.size(1), n = y.size();
   TORCH_CHECK(x.scalar_type() == at::kFloat && x.is_contiguous(), "branch_join: the residual stream is contiguous fp32");
-  const void *y[3], *w[3];
-  long long ldy[3];
-  float f[3];
-  int n = 0;
-  auto vec_ok = [&](const optional<Tensor>& v) {
-    return !(v.has_value() && v->defined()) || (v->is_contiguous() && v->numel() == cols && v->scalar_type() == y0.scalar_type());
+  TORCH_CHECK(n >= 1 && n <= 3 && w.size() == static_cast<size_t>(n) && slots.size() == static_cast<size_t>(n) && static_cast<int64_t>(factor.size()) == n &&
+                  static_cast<int64_t>(normed.size()) == n && static_cast<int64_t>(top.size()) == n, "branch_join: one to three branches");
+  const auto type = y[0].scalar_type();
+  OsloBranchJoin a{};
+  a.x = x.data_ptr<float>();
+  a.n = static_cast<int>(n);
+  const auto has = [](const optional<Tensor>& t) { return t.has_value() && t->defined(); };
+  const auto vec_ok = [&](const optional<Tensor>& v, bool one) {
+    return !has(v) || (v->is_cuda() && v->is_contiguous() && (v->numel() == cols || (one && v->numel() == 1)) && v->scalar_type() == type);
   };
-  auto add = [&](const Tensor& t, const optional<Tensor>& norm, double factor) {
-    check_rows(t, "y");
-    TORCH_CHECK(t.size(0) == rows && t.size(1) == cols && t.scalar_type() == y0.scalar_type() && vec_ok(norm), "branch_join: branch");
-    y[n] = t.data_ptr(); ldy[n] = t.stride(0); w[n] = ptr_or_null(norm); f[n] = static_cast<float>(factor);
-    ++n;
-  };
-  add(y0, n0, f0);
-  if (y1.has_value() && y1->defined()) add(*y1, n1, f1);
-  if (y2.has_value() && y2->defined()) add(*y2, n2, f2);
-  TORCH_CHECK(vec_ok(w1) && vec_ok(w2) && (ptr_or_null(w1) || !ptr_or_null(w2)), "branch_join: norm weights");
+  for (int64_t i = 0; i < n; ++i) {
+    const optional<Tensor> wi = w.get(i), si = slots.get(i);
+    check_rows(y[i], "y");
+    TORCH_CHECK(y[i].size(1) == cols && y[i].scalar_type() == type && vec_ok(wi, false) && top[i] >= 0, "branch_join: branch");
+    TORCH_CHECK(top[i] == 0 ? y[i].size(0) == rows : (has(si) || y[i].size(0) == rows * top[i]), "branch_join: rows of a branch");
+    if (top[i] > 0 && has(si)) {
+      TORCH_CHECK(si->is_cuda() && si->is_contiguous() && si->scalar_type() == at::kInt && si->numel() == rows * top[i], "branch_join: slots");
+      a.slots[i] = si->data_ptr<int>();
+    }
+    a.y[i] = y[i].data_ptr(); a.ldy[i] = y[i].stride(0); a.w[i] = ptr_or_null(wi); a.normed[i] = normed[i] != 0;
+    a.top[i] = static_cast<int>(top[i]); a.factor[i] = static_cast<float>(factor[i]);
+  }
+  TORCH_CHECK(vec_ok(w1, true) && vec_ok(w2, true) && (has(w1) || !has(w2)) && !(copy && has(w1)), "branch_join: norm weights");
+  a.mult = static_cast<float>(mult); a.eps = static_cast<float>(eps);
+  a.w1 = ptr_or_null(w1); a.w2 = ptr_or_null(w2); a.copy = copy;
+  a.one1 = has(w1) && w1->numel() != cols; a.one2 = has(w2) && w2->numel() != cols;
+  if (has(conv_w)) {
+    TORCH_CHECK(conv_w->dim() == 2 && conv_w->is_contiguous() && conv_w->size(0) == cols && conv_w->scalar_type() == type && has(w1), "branch_join: convolution");
+    a.conv_w = conv_w->data_ptr();
+    a.taps = static_cast<int>(conv_w->size(1));
+    if (has(prev) && a.taps > 1) {
+      check_state(*prev, rows * (a.taps - 1) * cols);
+      a.prev = prev->data_ptr<float>();
+    }
+    int64_t ld_keep = 0;
+    a.keep = keep_ptr(keep, rows, 1, ld_keep);
+    a.ld_keep = ld_keep;
+  }
   c10::cuda::CUDAGuard guard(x.device());
+  const auto out = y[0].options();
   Tensor xo = at::empty_like(x);
-  Tensor h1 = at::empty({ptr_or_null(w1) ? rows : 0, cols}, y0.options()), h2 = at::empty({ptr_or_null(w2) ? rows : 0, cols}, y0.options());
-  check_rc(oslo_branch_join(x.data_ptr<float>(), n, y, ldy, w, f, static_cast<float>(mult), static_cast<float>(eps), ptr_or_null(w1),
-                            ptr_or_null(w2), xo.data_ptr<float>(), ptr_or_null(w1) ? h1.data_ptr() : nullptr,
-                            ptr_or_null(w2) ? h2.data_ptr() : nullptr, rows, static_cast<int>(cols), dt_code(y0), cur_stream()),
-           "branch_join");
-  return {xo, h1, h2};
+  Tensor h1 = at::empty({has(w1) || copy ? rows : 0, cols}, out), h2 = at::empty({has(w2) ? rows : 0, cols}, out);
+  Tensor co = at::empty({has(conv_w) ? rows : 0, cols}, out);
+  a.x_out = xo.data_ptr<float>();
+  a.h1 = has(w1) || copy ? h1.data_ptr() : nullptr;
+  a.h2 = has(w2) ? h2.data_ptr() : nullptr;
+  a.conv_out = has(conv_w) ? co.data_ptr() : nullptr;
+  check_rc(oslo_branch_join(&a, rows, static_cast<int>(cols), dt_code(y[0]), cur_stream()), "branch_join");
+  return {xo, h1, h2, co};
+}
+
+// gelu_tanh(z) times the tokens' columns `first` and on of table [vocab, *]
+Tensor token_gate(const Tensor& z, const Tensor& ids, const Tensor& table, int64_t first) {
+  check_rows(z, "z");
+  TORCH_CHECK(ids.is_cuda() && ids.dim() == 1 && ids.scalar_type() == at::kLong && ids.size(0) == z.size(0), "token_gate: ids");
+  TORCH_CHECK(table.dim() == 2 && table.stride(1) == 1 && table.scalar_type() == z.scalar_type() && first >= 0 &&
+                  first + z.size(1) <= table.size(1), "token_gate: table");
+  c10::cuda::CUDAGuard guard(z.device());
+  Tensor out = at::empty({z.size(0), z.size(1)}, z.options());
+  check_rc(oslo_token_gate(z.data_ptr(), z.stride(0), reinterpret_cast<const long long*>(ids.data_ptr<int64_t>()), ids.stride(0), table.data_ptr(),
+                           table.stride(0), table.size(0), static_cast<int>(first), out.data_ptr(), z.size(0),
+                           static_cast<int>(z.size(1)), dt_code(z), dev_state(z.get_device()).err.data_ptr<int>(), cur_stream()),
+           "token_gate");
+  return out;
 }
 
 Tensor gated_rms_norm(const Tensor& o, const Tensor& w, const Tensor& gate, double eps, int64_t group, int64_t act,
@@ -1235,14 +1280,42 @@ Tensor flash_sink_fwd(const Tensor& q, const Tensor& k, const Tensor& v, const o
   return out;
 }
 
+// q [B, H, Sq, dim], k [B, 1, Sk, dim] (one key head of any width for all), v [B, G, Sk, vdim] -> [B * Sq, H * vdim]
+Tensor flash_wide_fwd(const Tensor& q, const Tensor& k, const Tensor& v, const optional<Tensor>& kpm, const optional<Tensor>& sink,
+                      const optional<Tensor>& gate, double scale, int64_t window, int64_t keep_first, const optional<Tensor>& lead) {
+  TORCH_CHECK(q.is_cuda() && q.dim() == 4 && k.dim() == 4 && v.dim() == 4 && q.stride(3) == 1 && k.stride(3) == 1 && v.stride(3) == 1 &&
+                  k.size(1) == 1 && k.size(3) == q.size(3) && k.size(0) == q.size(0) && v.size(0) == q.size(0) && v.size(2) == k.size(2) &&
+                  q.size(1) % v.size(1) == 0 && k.size(2) >= q.size(2), "flash_wide_fwd: q, k, v");
+  const int64_t B = q.size(0), H = q.size(1), G = v.size(1), Sq = q.size(2), Sk = k.size(2), dim = q.size(3), vdim = v.size(3);
+  TORCH_CHECK(k.scalar_type() == q.scalar_type() && v.scalar_type() == q.scalar_type() && window >= 0 && keep_first >= 0, "flash_wide_fwd: operands");
+  const void* sp = sink_ptr(sink, H, q, "flash_wide_fwd: sink");
+  const bool wide = check_gate(gate, B * Sq, H, vdim, q, "flash_wide_fwd: gate");
+  const bool gated = gate.has_value() && gate->defined();
+  const uint8_t* kp = nullptr;
+  if (kpm.has_value() && kpm->defined()) {
+    TORCH_CHECK(kpm->is_contiguous() && kpm->scalar_type() == at::kByte && kpm->numel() == B * Sk, "flash_wide_fwd: mask");
+    kp = kpm->data_ptr<uint8_t>();
+  }
+  c10::cuda::CUDAGuard guard(q.device());
+  Tensor out = at::empty({B * Sq, H * vdim}, q.options());
+  check_rc(oslo_flash_wide_fwd_sm100(q.data_ptr(), k.data_ptr(), v.data_ptr(), out.data_ptr(), kp, sp, ptr_or_null(gate),
+                                     gated ? gate->stride(0) : 0, wide ? 1 : 0, static_cast<int>(B), static_cast<int>(H),
+                                     static_cast<int>(G), static_cast<int>(Sq), static_cast<int>(Sk), static_cast<int>(dim),
+                                     static_cast<int>(vdim), q.stride(0), q.stride(1), q.stride(2), k.stride(0), k.stride(2),
+                                     v.stride(0), v.stride(1), v.stride(2), Sq * H * vdim, vdim, H * vdim, static_cast<float>(scale),
+                                     static_cast<int>(window), static_cast<int>(keep_first), lead_ptr(lead, B), dt_code(q),
+                                     dev_state(q.get_device()).err.data_ptr<int>(), cur_stream()), "flash_wide_fwd");
+  return out;
+}
+
 Tensor sink_attention(const Tensor& q, const Tensor& k, const Tensor& v, const optional<Tensor>& keep, const optional<Tensor>& sink,
                       const optional<Tensor>& gate, double scale, double softcap, int64_t window, int64_t keep_first,
                       const optional<Tensor>& lead) {
   // [B, S, heads, D] views with contiguous D
   TORCH_CHECK(q.is_cuda() && q.dim() == 4 && k.dim() == 4 && v.dim() == 4 && q.stride(3) == 1 && k.stride(3) == 1 && v.stride(3) == 1,
               "sink_attention: q, k, v must be [B, S, H, D] with a contiguous last dim");
-  const int64_t B = q.size(0), Sq = q.size(1), H = q.size(2), G = k.size(2), D = q.size(3), Sk = k.size(1), Dv = v.size(3);
-  TORCH_CHECK(k.size(0) == B && v.size(0) == B && H % G == 0 && v.size(2) == G && v.size(1) == Sk && k.size(3) == D && Sk >= Sq,
+  const int64_t B = q.size(0), Sq = q.size(1), H = q.size(2), G = v.size(2), KG = k.size(2), D = q.size(3), Sk = k.size(1), Dv = v.size(3);
+  TORCH_CHECK(k.size(0) == B && v.size(0) == B && G > 0 && KG > 0 && H % G == 0 && H % KG == 0 && v.size(1) == Sk && k.size(3) == D && Sk >= Sq,
               "sink_attention: sizes");
   TORCH_CHECK(k.scalar_type() == q.scalar_type() && v.scalar_type() == q.scalar_type() && window >= 0 && keep_first >= 0,
               "sink_attention: operands");
@@ -1256,7 +1329,7 @@ Tensor sink_attention(const Tensor& q, const Tensor& k, const Tensor& v, const o
   check_rc(oslo_sink_attention(q.data_ptr(), q.stride(0), q.stride(1), q.stride(2), k.data_ptr(), k.stride(0), k.stride(1),
                                k.stride(2), v.data_ptr(), v.stride(0), v.stride(1), v.stride(2), kp, ld_keep, sp,
                                ptr_or_null(gate), gated ? gate->stride(0) : 0, out.data_ptr(), static_cast<int>(B),
-                               static_cast<int>(H), static_cast<int>(G), static_cast<int>(Sq), static_cast<int>(Sk),
+                               static_cast<int>(H), static_cast<int>(G), static_cast<int>(KG), static_cast<int>(Sq), static_cast<int>(Sk),
                                static_cast<int>(D), static_cast<int>(Dv), static_cast<float>(scale), static_cast<float>(softcap),
                                static_cast<int>(window), static_cast<int>(keep_first), lead_ptr(lead, B), wide ? 1 : 0,
                                dt_code(q), cur_stream()), "sink_attention");
@@ -1292,37 +1365,75 @@ Tensor qkv_prep(const Tensor& q, const Tensor& k, const Tensor& v, const optiona
   return out;
 }
 
+// caches kc [B, G, T, dim], vc [B, G, T, vdim] of any strides with contiguous heads; talk [H, H]: the queries of mixed scores, [B, S, H, G * dim]
+Tensor head_prep(const Tensor& q, const Tensor& k, const Tensor& v, const optional<Tensor>& wq, const optional<Tensor>& wk, double eps,
+                 const Tensor& positions, const Tensor& freq, bool halves, double amplitude, const optional<Tensor>& talk, Tensor kc,
+                 Tensor vc, const Tensor& lengths) {
+  check_rows(q, "q"); check_rows(k, "k"); check_rows(v, "v");
+  TORCH_CHECK(kc.is_cuda() && kc.dim() == 4 && vc.dim() == 4 && kc.stride(3) == 1 && vc.stride(3) == 1 && vc.size(0) == kc.size(0) &&
+                  vc.size(1) == kc.size(1) && vc.size(2) == kc.size(2), "head_prep: caches");
+  const int64_t B = kc.size(0), G = kc.size(1), T = kc.size(2), dim = kc.size(3), vdim = vc.size(3);
+  TORCH_CHECK(q.size(0) % B == 0 && q.size(1) % dim == 0 && k.size(0) == q.size(0) && v.size(0) == q.size(0) && k.size(1) == G * dim &&
+                  v.size(1) == G * vdim, "head_prep: projections");
+  const int64_t S = q.size(0) / B, H = q.size(1) / dim;
+  for (const Tensor* t : {&k, &v, static_cast<const Tensor*>(&kc), static_cast<const Tensor*>(&vc)})
+    TORCH_CHECK(t->scalar_type() == q.scalar_type(), "head_prep: dtypes");
+  if (ptr_or_null(wq)) check_channels(*wq, dim, q, "head_prep: query norm weight");
+  if (ptr_or_null(wk)) check_channels(*wk, dim, q, "head_prep: key norm weight");
+  const bool mixed = talk.has_value() && talk->defined();
+  if (mixed) check_channels(*talk, H * H, q, "head_prep: mix of the heads");
+  TORCH_CHECK(positions.is_cuda() && positions.dim() == 2 && positions.size(0) == B && positions.size(1) == S && positions.scalar_type() == at::kLong, "head_prep: positions");
+  TORCH_CHECK(freq.is_cuda() && freq.is_contiguous() && freq.scalar_type() == at::kFloat && 2 * freq.numel() <= dim, "head_prep: frequencies");
+  TORCH_CHECK(lengths.scalar_type() == at::kInt && lengths.is_contiguous() && lengths.numel() == B, "head_prep: lengths");
+  c10::cuda::CUDAGuard guard(q.device());
+  auto& st = dev_state(q.get_device());
+  Tensor out = at::empty({B, S, H, mixed ? G * dim : dim}, q.options());
+  check_rc(oslo_head_prep(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), ptr_or_null(wq), ptr_or_null(wk),
+                          static_cast<float>(eps), reinterpret_cast<const long long*>(positions.data_ptr<int64_t>()), positions.stride(0),
+                          positions.stride(1), freq.numel() ? freq.data_ptr<float>() : nullptr, static_cast<int>(freq.numel()),
+                          halves ? 1 : 0, static_cast<float>(amplitude), ptr_or_null(talk), out.data_ptr(), kc.data_ptr(), kc.stride(0),
+                          kc.stride(1), kc.stride(2), vc.data_ptr(), vc.stride(0), vc.stride(1), vc.stride(2), lengths.data_ptr<int>(),
+                          static_cast<int>(B), static_cast<int>(S), static_cast<int>(H), static_cast<int>(G), static_cast<int>(dim),
+                          static_cast<int>(vdim), static_cast<int>(T), st.sms, dt_code(q), st.err.data_ptr<int>(), cur_stream()), "head_prep");
+  return out;
+}
+
+// whether grouped_decode has a kernel for wide keys of these sizes
+bool wide_decode_fits(const Tensor& like, int64_t heads, int64_t value_heads, int64_t dim, int64_t vdim) {
+  return oslo_wide_decode_fits(static_cast<int>(heads), static_cast<int>(value_heads), static_cast<int>(dim), static_cast<int>(vdim), dt_code(like)) != 0;
+}
+
+// value_heads > 1: kc [B, 1, T, dim] (wide keys), vc [B, 1, T, value_heads * vdim]; query heads read value heads in equal groups
 Tensor grouped_decode(const Tensor& q, const Tensor& kc, const Tensor& vc, const Tensor& lengths, const optional<Tensor>& keep,
                       const optional<Tensor>& sink, double scale, double softcap, const optional<Tensor>& gate, int64_t window,
-                      int64_t keep_first, const optional<Tensor>& lead) {
+                      int64_t keep_first, const optional<Tensor>& lead, int64_t value_heads) {
   TORCH_CHECK(q.is_cuda() && q.dim() == 3 && q.is_contiguous() && kc.dim() == 4 && vc.dim() == 4 && kc.is_contiguous() && vc.is_contiguous() &&
                   vc.size(0) == kc.size(0) && vc.size(1) == kc.size(1) && vc.size(2) == kc.size(2) && kc.size(0) == q.size(0) &&
                   kc.size(3) == q.size(2) && q.size(1) % kc.size(1) == 0, "grouped_decode: q [B, H, dim], caches [B, G, T, *]");
-  const int64_t B = q.size(0), H = q.size(1), G = kc.size(1), T = kc.size(2), vdim = vc.size(3);
+  const int64_t B = q.size(0), H = q.size(1), G = kc.size(1), T = kc.size(2), row = vc.size(3);
+  TORCH_CHECK(value_heads >= 1 && (value_heads == 1 || (G == 1 && H % value_heads == 0 && row % value_heads == 0)), "grouped_decode: value heads");
+  const int64_t vdim = row / value_heads;
   TORCH_CHECK(kc.scalar_type() == q.scalar_type() && vc.scalar_type() == q.scalar_type() && window >= 0 && keep_first >= 0, "grouped_decode: operands");
   const void* sp = sink_ptr(sink, H, q, "grouped_decode: sink");
+  const bool wide = check_gate(gate, B, H, vdim, q, "grouped_decode: gate");
   const bool gated = gate.has_value() && gate->defined();
-  if (gated) {
-    check_rows(*gate, "gate");
-    TORCH_CHECK(gate->size(0) == B && gate->size(1) == H && gate->scalar_type() == q.scalar_type(), "grouped_decode: gate");
-  }
   TORCH_CHECK(lengths.scalar_type() == at::kInt && lengths.is_contiguous() && lengths.numel() == B, "grouped_decode: lengths");
   int64_t ld_keep = 0;
   const uint8_t* kp = keep_ptr(keep, B, 0, ld_keep);
   c10::cuda::CUDAGuard guard(q.device());
   auto& st = dev_state(q.get_device());
   const int64_t most = window > 0 ? std::min(T, window + keep_first) : T;     // keys a query can see
-  const int splits = oslo_grouped_splits(static_cast<int>(B), static_cast<int>(H), static_cast<int>(G), static_cast<int>(most),
-                                         static_cast<int>(q.size(2)), static_cast<int>(vdim), dt_code(q), st.sms);
+  const int splits = oslo_grouped_splits(static_cast<int>(B), static_cast<int>(H), static_cast<int>(G), static_cast<int>(value_heads),
+                                         static_cast<int>(most), static_cast<int>(q.size(2)), static_cast<int>(row), dt_code(q), st.sms);
   const auto f32 = q.options().dtype(at::kFloat);
   Tensor ws = at::empty({B, H, splits, (vdim + 3) / 4 * 4}, f32);
   Tensor stat = at::empty({B, H, splits, 2}, f32);
   Tensor out = at::empty({B, H * vdim}, q.options());
   check_rc(oslo_grouped_decode(q.data_ptr(), kc.data_ptr(), vc.data_ptr(), lengths.data_ptr<int>(), kp, ld_keep,
-                               kp ? static_cast<int>(keep->size(1)) : 0, sp, ptr_or_null(gate), gated ? gate->stride(0) : 0,
+                               kp ? static_cast<int>(keep->size(1)) : 0, sp, ptr_or_null(gate), gated ? gate->stride(0) : 0, wide ? 1 : 0,
                                static_cast<int>(window), static_cast<int>(keep_first), lead_ptr(lead, B), ws.data_ptr<float>(),
                                stat.data_ptr<float>(), out.data_ptr(), static_cast<int>(B), static_cast<int>(H), static_cast<int>(G),
-                               static_cast<int>(q.size(2)), static_cast<int>(vdim), static_cast<int>(T), splits,
+                               static_cast<int>(value_heads), static_cast<int>(q.size(2)), static_cast<int>(row), static_cast<int>(T), splits,
                                static_cast<float>(scale), static_cast<float>(softcap), dt_code(q), st.err.data_ptr<int>(),
                                cur_stream(2)), "grouped_decode");
   return out;
@@ -1350,22 +1461,22 @@ Tensor token_shift(const Tensor& h, const Tensor& mu, int64_t batch, const optio
   return out;
 }
 
-Tensor causal_conv_silu(const Tensor& x, const Tensor& w, const Tensor& bias, int64_t batch, const optional<Tensor>& keep,
-                        optional<Tensor> prev) {
+Tensor causal_conv(const Tensor& x, const Tensor& w, const optional<Tensor>& bias, int64_t batch, const optional<Tensor>& keep,
+                   optional<Tensor> prev, bool silu, bool residual) {
   check_rows(x, "x");
   const int64_t C = x.size(1);
-  TORCH_CHECK(batch > 0 && x.size(0) % batch == 0 && w.dim() == 2 && w.is_contiguous() && w.size(0) == C && w.scalar_type() == x.scalar_type(),
-              "causal_conv_silu: operands");
-  check_channels(bias, C, x, "causal_conv_silu: bias");
+  TORCH_CHECK(batch > 0 && x.size(0) % batch == 0 && w.dim() == 2 && w.is_contiguous() && w.size(0) == C && w.scalar_type() == x.scalar_type() &&
+                  !(silu && residual), "causal_conv: operands");
+  if (ptr_or_null(bias)) check_channels(*bias, C, x, "causal_conv: bias");
   const int64_t S = x.size(0) / batch, taps = w.size(1);
   int64_t ld_keep = 0;
   const uint8_t* kp = keep_ptr(keep, batch, S, ld_keep);
   c10::cuda::CUDAGuard guard(x.device());
   Tensor out = at::empty({x.size(0), C}, x.options());
-  check_rc(oslo_causal_conv_silu(x.data_ptr(), x.stride(0), w.data_ptr(), bias.data_ptr(), kp, ld_keep,
-                                 carried_ptr(prev, batch * (taps - 1) * C), out.data_ptr(), static_cast<int>(batch),
-                                 static_cast<int>(S), static_cast<int>(C), static_cast<int>(taps), dt_code(x), cur_stream()),
-           "causal_conv_silu");
+  check_rc(oslo_causal_conv(x.data_ptr(), x.stride(0), w.data_ptr(), ptr_or_null(bias), kp, ld_keep,
+                            taps > 1 ? carried_ptr(prev, batch * (taps - 1) * C) : nullptr, out.data_ptr(), static_cast<int>(batch),
+                            static_cast<int>(S), static_cast<int>(C), static_cast<int>(taps), silu ? 1 : 0, residual ? 1 : 0,
+                            dt_code(x), cur_stream()), "causal_conv");
   return out;
 }
 
@@ -1531,11 +1642,12 @@ Tensor latent_decode(const Tensor& q, const Tensor& w_uk, const Tensor& w_uv, co
 }
 
 // ---------------------------------------------------------------------- mixture of experts
-std::tuple<Tensor, Tensor> moe_route(const Tensor& h, const Tensor& w, const Tensor& bias, const optional<Tensor>& logits, int64_t top,
-                                     bool scored) {
+std::tuple<Tensor, Tensor> moe_route(const Tensor& h, const Tensor& w, const optional<Tensor>& bias, const optional<Tensor>& logits,
+                                     int64_t top, int64_t scored) {
   check_rows(h, "h");
-  TORCH_CHECK(w.dim() == 2 && w.is_contiguous() && w.size(1) == h.size(1) && bias.numel() == w.size(0) &&
-                  w.scalar_type() == h.scalar_type() && bias.scalar_type() == h.scalar_type(), "moe_route: router");
+  TORCH_CHECK(w.dim() == 2 && w.is_contiguous() && w.size(1) == h.size(1) && w.scalar_type() == h.scalar_type() && scored >= 0 && scored <= 2,
+              "moe_route: router");
+  if (ptr_or_null(bias)) check_channels(*bias, w.size(0), h, "moe_route: bias");
   const int64_t n = h.size(0), E = w.size(0);
   const float* lg = nullptr;
   int64_t ldl = 0;
@@ -1548,14 +1660,20 @@ std::tuple<Tensor, Tensor> moe_route(const Tensor& h, const Tensor& w, const Ten
   c10::cuda::CUDAGuard guard(h.device());
   Tensor idx = at::empty({n, top}, h.options().dtype(at::kInt));
   Tensor wgt = at::empty({n, top}, h.options().dtype(at::kFloat));
-  check_rc(oslo_moe_route(h.data_ptr(), h.stride(0), w.data_ptr(), bias.data_ptr(), lg, ldl, idx.data_ptr<int>(), wgt.data_ptr<float>(),
-                          n, static_cast<int>(E), static_cast<int>(h.size(1)), static_cast<int>(top), scored ? 1 : 0, dt_code(h),
+  check_rc(oslo_moe_route(h.data_ptr(), h.stride(0), w.data_ptr(), ptr_or_null(bias), lg, ldl, idx.data_ptr<int>(), wgt.data_ptr<float>(),
+                          n, static_cast<int>(E), static_cast<int>(h.size(1)), static_cast<int>(top), static_cast<int>(scored), dt_code(h),
                           cur_stream()), "moe_route");
   return {idx, wgt};
 }
 
 // (slots [n, top], rows sorted by expert, expert of every 128-row tile, tiles in use)
-std::tuple<Tensor, Tensor, Tensor, Tensor> moe_plan(const Tensor& h, const Tensor& idx, int64_t experts) {
+// scale [pairs] (fp32, or none) multiplies the rows
+const float* pair_scale(const optional<Tensor>& scale, int64_t pairs) {
+  if (!(scale.has_value() && scale->defined())) return nullptr;
+  TORCH_CHECK(scale->is_cuda() && scale->is_contiguous() && scale->scalar_type() == at::kFloat && scale->numel() == pairs, "weights of (token, choice) pairs");
+  return scale->data_ptr<float>();
+}
+std::tuple<Tensor, Tensor, Tensor, Tensor> moe_plan(const Tensor& h, const Tensor& idx, int64_t experts, const optional<Tensor>& scale) {
   check_rows(h, "h");
   TORCH_CHECK(idx.is_contiguous() && idx.scalar_type() == at::kInt && idx.dim() == 2 && idx.size(0) == h.size(0), "moe_plan: idx");
   const int64_t pairs = idx.numel(), K = h.size(1);
@@ -1566,49 +1684,53 @@ std::tuple<Tensor, Tensor, Tensor, Tensor> moe_plan(const Tensor& h, const Tenso
   Tensor slots = at::empty({idx.size(0), idx.size(1)}, i32);
   Tensor rows = at::empty({tiles * 128, K}, h.options());
   check_rc(oslo_moe_plan(h.data_ptr(), h.stride(0), idx.data_ptr<int>(), cursor.data_ptr<int>(), tg.data_ptr<int>(),
-                         nt.data_ptr<int>(), slots.data_ptr<int>(), rows.data_ptr(), pairs, static_cast<int>(experts),
+                         nt.data_ptr<int>(), slots.data_ptr<int>(), rows.data_ptr(), pair_scale(scale, pairs), pairs, static_cast<int>(experts),
                          static_cast<int>(K), static_cast<int>(idx.size(1)), static_cast<int>(tiles), dt_code(h), cur_stream(2)),
            "moe_plan");
   return {slots, rows, tg, nt};
 }
 
-// unit(rows . w[expert of the tile]^T): [slots, N], or [slots, N / 2] for unit 2 (silu(gate) * up of column pairs); tcgen05 for
-// 16-bit types with K % 8 == 0 and 16-byte result rows
-Tensor moe_grouped(const Tensor& rows, const Tensor& w, const Tensor& tile_group, const Tensor& n_tiles, int64_t unit) {
+// unit(rows . w[expert of the tile]^T): [slots, N], or [slots, N / 2] for units 2 and 3 (silu(gate) * up of column pairs, its clamped
+// form); tcgen05 for 16-bit types with K % 8 == 0 and 16-byte result rows
+Tensor moe_grouped(const Tensor& rows, const Tensor& w, const Tensor& tile_group, const Tensor& n_tiles, int64_t unit, double limit,
+                   double alpha) {
   TORCH_CHECK(rows.is_cuda() && rows.dim() == 2 && rows.is_contiguous() && w.dim() == 3 && w.is_contiguous() &&
                   w.size(2) == rows.size(1) && w.scalar_type() == rows.scalar_type(), "moe_grouped: operands");
   TORCH_CHECK(tile_group.scalar_type() == at::kInt && tile_group.numel() * 128 == rows.size(0) && n_tiles.scalar_type() == at::kInt,
               "moe_grouped: plan");
-  const int64_t N = w.size(1), K = w.size(2), cols = unit == 2 ? N / 2 : N;
-  TORCH_CHECK(unit >= 0 && unit <= 2 && (unit != 2 || N % 2 == 0), "moe_grouped: unit");
+  const int64_t N = w.size(1), K = w.size(2), cols = unit >= 2 ? N / 2 : N;
+  TORCH_CHECK(unit >= 0 && unit <= 3 && (unit < 2 || N % 2 == 0), "moe_grouped: unit");
   c10::cuda::CUDAGuard guard(rows.device());
   auto& st = dev_state(rows.get_device());
   Tensor out = at::empty({rows.size(0), cols}, rows.options());
   if (rows.scalar_type() != at::kFloat && K % 8 == 0 && cols % 8 == 0 && reinterpret_cast<uintptr_t>(w.data_ptr()) % 16 == 0) {
-    const int fl = (unit == 1 ? GEMM_FLAG_RELU2 : 0) | (unit == 2 ? GEMM_FLAG_GLU : 0) | (rows.scalar_type() == at::kHalf ? GEMM_FLAG_FP16 : 0);
+    const int fl = (unit == 1 ? GEMM_FLAG_RELU2 : 0) | (unit >= 2 ? GEMM_FLAG_GLU : 0) | (rows.scalar_type() == at::kHalf ? GEMM_FLAG_FP16 : 0);
     check_rc(oslo_gemm_grouped(rows.data_ptr(), w.data_ptr(), out.data_ptr(), static_cast<int>(rows.size(0)), static_cast<int>(N),
                                static_cast<int>(K), static_cast<int>(w.size(0)), tile_group.data_ptr<int>(),
-                               n_tiles.data_ptr<int>(), fl, st.err.data_ptr<int>(), usable_sms(st), cur_stream()), "gemm_grouped");
+                               n_tiles.data_ptr<int>(), fl, unit == 3 ? 1 : 0, static_cast<float>(limit), static_cast<float>(alpha),
+                               st.err.data_ptr<int>(), usable_sms(st), cur_stream()), "gemm_grouped");
   } else {
     check_rc(oslo_moe_grouped(rows.data_ptr(), w.data_ptr(), out.data_ptr(), tile_group.data_ptr<int>(), n_tiles.data_ptr<int>(),
                               static_cast<int>(tile_group.numel()), static_cast<int>(N), static_cast<int>(K), static_cast<int>(unit),
-                              dt_code(rows), cur_stream()), "moe_grouped");
+                              static_cast<float>(limit), static_cast<float>(alpha), dt_code(rows), cur_stream()), "moe_grouped");
   }
   return out;
 }
 
 // one row of the result per (row, choice): unit(w[idx] . x[row]); x has one row per `per_row` entries of idx; rows of entries that are
-// no expert (>= w.size(0)) are not written
-Tensor moe_few(const Tensor& x, const Tensor& idx, const Tensor& w, int64_t per_row, int64_t unit) {
+// no expert (>= w.size(0)) are not written; scale [pairs] (or none) multiplies the rows of x
+Tensor moe_few(const Tensor& x, const Tensor& idx, const Tensor& w, int64_t per_row, int64_t unit, double limit, double alpha,
+               const optional<Tensor>& scale) {
   check_rows(x, "x");
   TORCH_CHECK(w.dim() == 3 && w.is_contiguous() && w.size(2) == x.size(1) && w.scalar_type() == x.scalar_type(), "moe_few: weights");
   TORCH_CHECK(idx.is_contiguous() && idx.scalar_type() == at::kInt && idx.numel() == x.size(0) * per_row, "moe_few: idx");
-  TORCH_CHECK(unit >= 0 && unit <= 2 && (unit != 2 || w.size(1) % 2 == 0), "moe_few: unit");
+  TORCH_CHECK(unit >= 0 && unit <= 3 && (unit < 2 || w.size(1) % 2 == 0), "moe_few: unit");
   c10::cuda::CUDAGuard guard(x.device());
-  Tensor out = at::empty({idx.numel(), unit == 2 ? w.size(1) / 2 : w.size(1)}, x.options());
+  Tensor out = at::empty({idx.numel(), unit >= 2 ? w.size(1) / 2 : w.size(1)}, x.options());
   check_rc(oslo_moe_few(x.data_ptr(), x.stride(0), idx.data_ptr<int>(), w.data_ptr(), out.data_ptr(), static_cast<int>(idx.numel()),
                         static_cast<int>(per_row), static_cast<int>(w.size(1)), static_cast<int>(w.size(2)), static_cast<int>(unit),
-                        static_cast<int>(w.size(0)), dt_code(x), cur_stream()), "moe_few");
+                        static_cast<float>(limit), static_cast<float>(alpha), pair_scale(scale, idx.numel()), static_cast<int>(w.size(0)),
+                        dt_code(x), cur_stream()), "moe_few");
   return out;
 }
 
@@ -1665,12 +1787,12 @@ TORCH_LIBRARY(oslo_b200, m) {
   m.def("latent_prep(Tensor cq, Tensor wq, Tensor? ckv, Tensor? wkv, Tensor(a!)? cache, Tensor lengths, float eps, Tensor? positions=None, Tensor? freq=None, bool rows=False) -> (Tensor, Tensor)");
   m.def("rotate_halves_(Tensor(a!) q, Tensor positions, Tensor freq) -> Tensor(a!)");
   m.def("latent_decode(Tensor q, Tensor w_uk, Tensor w_uv, Tensor cache, Tensor lengths, Tensor? keep, Tensor? sink, Tensor gate, float scale, int heads, Tensor? positions=None, Tensor? freq=None) -> Tensor");
-  m.def("moe_route(Tensor h, Tensor w, Tensor bias, Tensor? logits, int top, bool scored=False) -> (Tensor, Tensor)");
-  m.def("moe_plan(Tensor h, Tensor idx, int experts) -> (Tensor, Tensor, Tensor, Tensor)");
-  m.def("moe_grouped(Tensor rows, Tensor w, Tensor tile_group, Tensor n_tiles, int unit) -> Tensor");
-  m.def("moe_few(Tensor x, Tensor idx, Tensor w, int per_row, int unit) -> Tensor");
+  m.def("moe_route(Tensor h, Tensor w, Tensor? bias, Tensor? logits, int top, int scored=0) -> (Tensor, Tensor)");
+  m.def("moe_plan(Tensor h, Tensor idx, int experts, Tensor? scale=None) -> (Tensor, Tensor, Tensor, Tensor)");
+  m.def("moe_grouped(Tensor rows, Tensor w, Tensor tile_group, Tensor n_tiles, int unit, float limit=0., float alpha=1.) -> Tensor");
+  m.def("moe_few(Tensor x, Tensor idx, Tensor w, int per_row, int unit, float limit=0., float alpha=1., Tensor? scale=None) -> Tensor");
   m.def("clamped_glu(Tensor gate, Tensor up, float limit, float alpha) -> Tensor");
-  m.def("branch_join(Tensor x, Tensor y0, Tensor? n0, float f0, Tensor? y1, Tensor? n1, float f1, Tensor? y2, Tensor? n2, float f2, float mult, float eps, Tensor? w1, Tensor? w2) -> (Tensor, Tensor, Tensor)");
+  m.def("branch_join(Tensor x, Tensor[] y, Tensor?[] w, float[] factor, int[] normed, Tensor?[] slots, int[] top, float mult, float eps, Tensor? w1, Tensor? w2, bool copy=False, Tensor? conv_w=None, Tensor(a!)? prev=None, Tensor? keep=None) -> (Tensor, Tensor, Tensor, Tensor)");
   m.def("gated_rms_norm(Tensor o, Tensor w, Tensor gate, float eps, int group, int act, Tensor? z=None, Tensor? m=None) -> Tensor");
   m.def("hyper_join(Tensor x, Tensor? y, Tensor? slots, Tensor? weights, Tensor? choice, int experts, Tensor? own, Tensor? shared, Tensor? gate, Tensor? w_out, Tensor? mix, Tensor? w_in, Tensor w_norm, float eps, float scale) -> (Tensor, Tensor)");
   m.def("memory_gates(Tensor z, Tensor bias, float cap, Tensor? keep, Tensor(a!)? top, int batch) -> (Tensor, Tensor, Tensor, Tensor)");
@@ -1682,9 +1804,13 @@ TORCH_LIBRARY(oslo_b200, m) {
   m.def("decayed_step(Tensor q, Tensor k, Tensor v, Tensor decay, Tensor? keep, Tensor(a!) state, int heads, int dim, int vdim) -> Tensor");
   m.def("bonus_step(Tensor r, Tensor k, Tensor v, Tensor t, Tensor w2, Tensor w0, Tensor u, Tensor norm_w, Tensor gate, Tensor? keep, Tensor(a!) state, float eps, int heads, int dim, int vdim) -> Tensor");
   m.def("qkv_prep(Tensor q, Tensor k, Tensor v, Tensor? wq, Tensor? wk, float eps, Tensor positions, Tensor freq, Tensor(a!) kc, Tensor(b!) vc, Tensor lengths) -> Tensor");
-  m.def("grouped_decode(Tensor q, Tensor kc, Tensor vc, Tensor lengths, Tensor? keep, Tensor? sink, float scale, float softcap, Tensor? gate=None, int window=0, int keep_first=0, Tensor? lead=None) -> Tensor");
+  m.def("head_prep(Tensor q, Tensor k, Tensor v, Tensor? wq, Tensor? wk, float eps, Tensor positions, Tensor freq, bool halves, float amplitude, Tensor? talk, Tensor(a!) kc, Tensor(b!) vc, Tensor lengths) -> Tensor");
+  m.def("wide_decode_fits(Tensor like, int heads, int value_heads, int dim, int vdim) -> bool");
+  m.def("flash_wide_fwd(Tensor q, Tensor k, Tensor v, Tensor? kpm, Tensor? sink, Tensor? gate, float scale, int window=0, int keep_first=0, Tensor? lead=None) -> Tensor");
+  m.def("token_gate(Tensor z, Tensor ids, Tensor table, int first) -> Tensor");
+  m.def("grouped_decode(Tensor q, Tensor kc, Tensor vc, Tensor lengths, Tensor? keep, Tensor? sink, float scale, float softcap, Tensor? gate=None, int window=0, int keep_first=0, Tensor? lead=None, int value_heads=1) -> Tensor");
   m.def("token_shift(Tensor h, Tensor mu, int batch, Tensor? keep, Tensor(a!)? prev) -> Tensor");
-  m.def("causal_conv_silu(Tensor x, Tensor w, Tensor bias, int batch, Tensor? keep, Tensor(a!)? prev) -> Tensor");
+  m.def("causal_conv(Tensor x, Tensor w, Tensor? bias, int batch, Tensor? keep, Tensor(a!)? prev, bool silu=False, bool residual=False) -> Tensor");
   m.def("selective_scan(Tensor x, Tensor dt, Tensor dt_bias, Tensor a_log, Tensor b, Tensor c, Tensor d, Tensor z, int batch, Tensor? keep, Tensor(a!)? state, int chunks=0) -> Tensor");
   m.def("scan_step(Tensor x, Tensor dt, Tensor w_dt, Tensor dt_bias, Tensor a_log, Tensor b, Tensor c, Tensor d, Tensor z, Tensor? keep, Tensor(a!) state) -> Tensor");
 }
@@ -1752,9 +1878,13 @@ TORCH_LIBRARY_IMPL(oslo_b200, CUDA, m) {
   m.impl("decayed_step", &decayed_step);
   m.impl("bonus_step", &bonus_step);
   m.impl("qkv_prep", &qkv_prep);
+  m.impl("head_prep", &head_prep);
+  m.impl("wide_decode_fits", &wide_decode_fits);
+  m.impl("flash_wide_fwd", &flash_wide_fwd);
+  m.impl("token_gate", &token_gate);
   m.impl("grouped_decode", &grouped_decode);
   m.impl("token_shift", &token_shift);
-  m.impl("causal_conv_silu", &causal_conv_silu);
+  m.impl("causal_conv", &causal_conv);
   m.impl("selective_scan", &selective_scan);
   m.impl("scan_step", &scan_step);
 }

@@ -134,6 +134,7 @@ __global__ void __launch_bounds__(GV_THREADS) gemv_rows_kernel(const T* __restri
         const int n = n0 + c;
         if (bias) v += DCvt<T>::to(bias[n]);
         if (gelu_from >= 0 && n >= gelu_from) v = gelu_tanh_dec(v);
+        if (gelu_from == OSLO_ACT_RELU2) { v = fmaxf(v, 0.f); v *= v; }
         if (res) v += DCvt<T>::to(res[static_cast<size_t>(m) * ldr + n]);
         out[static_cast<size_t>(m) * ldo + n] = DCvt<T>::from(v);
       }

@@ -648,6 +648,7 @@ __global__ void splitk_finalize_kernel(const float* __restrict__ ws, const T* __
     const int c = static_cast<int>(i % cols);
     if (bias) v += Cvt<T>::to(bias[c]);
     if (gelu_from >= 0 && c >= gelu_from) v = gelu_f(v);
+    if (gelu_from == OSLO_ACT_RELU2) { v = fmaxf(v, 0.f); v *= v; }
     out[i] = Cvt<T>::from(v);
   }
 }

@@ -62,6 +62,9 @@ struct GemmParams {
   // group; B stacks the groups' [N, K] matrices. Both arrays are device data written by an earlier kernel.
   const int* group_of_tile = nullptr;     // [tiles_m] group of every row tile, or nullptr
   const int* group_tiles = nullptr;       // [1] row tiles in use (<= tiles_m)
+  // GEMM_FLAG_GLU, clamped: g sigmoid(glu_alpha g) (u + 1) of g = min(gate, limit), u = clamp(up, -limit, limit)
+  int glu_clamped = 0;
+  float glu_limit = 0.f, glu_alpha = 1.f;
   CommParams comm;
 };
 
@@ -344,8 +347,17 @@ __device__ __forceinline__ void epilogue_chunk(const GemmParams& p, int row, int
     }
     if (p.flags & GEMM_FLAG_GLU) {   // 16-bit output, no further epilogue
       uint16_t* d = reinterpret_cast<uint16_t*>(p.D) + static_cast<size_t>(row) * p.ldd + col0 / 2;
+      if (p.glu_clamped) {
+        const float lim = p.glu_limit, al = p.glu_alpha;
 #pragma unroll
-      for (int i = 0; i < 16; ++i) v[i] = __fdividef(v[2 * i], 1.f + __expf(-v[2 * i])) * v[2 * i + 1];
+        for (int i = 0; i < 16; ++i) {
+          const float g = fminf(v[2 * i], lim), u = fminf(fmaxf(v[2 * i + 1], -lim), lim);
+          v[i] = __fdividef(g, 1.f + __expf(-al * g)) * (u + 1.f);
+        }
+      } else {
+#pragma unroll
+        for (int i = 0; i < 16; ++i) v[i] = __fdividef(v[2 * i], 1.f + __expf(-v[2 * i])) * v[2 * i + 1];
+      }
       if (vec) {
 #pragma unroll
         for (int i = 0; i < 16; i += 8) {

@@ -251,7 +251,8 @@ extern "C" int oslo_gemm_splitk_16bit(const void* A, const void* B, float* D, in
 
 // D[slot, N] = act(A[slot, :] . B[group of the slot's 128-row tile]^T) for rows sorted by group (see GemmParams)
 extern "C" int oslo_gemm_grouped(const void* A, const void* B, void* D, int M, int N, int K, int groups, const int* group_of_tile,
-                                 const int* group_tiles, int flags, int* err_word, int num_sms, cudaStream_t stream) {
+                                 const int* group_tiles, int flags, int glu_clamped, float glu_limit, float glu_alpha, int* err_word, int num_sms,
+                                 cudaStream_t stream) {
   using namespace oslo;
   if (M <= 0 || N <= 0 || K <= 0 || M % BM || groups <= 0 || group_of_tile == nullptr || group_tiles == nullptr) return -1;
   if (flags & ~(GEMM_FLAG_RELU2 | GEMM_FLAG_GLU | GEMM_FLAG_FP16 | GEMM_FLAG_OUT_FP32)) return -7;
@@ -271,6 +272,7 @@ extern "C" int oslo_gemm_grouped(const void* A, const void* B, void* D, int M, i
   p.M = M; p.N = N; p.K = K; p.ldd = glu ? N / 2 : N; p.ld_aux = 0; p.ld_aux_out = 0;
   p.a_mn_major = 0; p.b_mn_major = 0; p.flags = flags; p.alpha = 1.f; p.err = err_word;
   p.group_of_tile = group_of_tile; p.group_tiles = group_tiles;
+  p.glu_clamped = glu_clamped; p.glu_limit = glu_limit; p.glu_alpha = glu_alpha;
   p.comm = CommParams{};
   return wide ? launch<256, 4>(ta, tb, p, num_sms, stream) : launch<128, 6>(ta, tb, p, num_sms, stream);
 }

@@ -1,7 +1,12 @@
-// Grouped-query attention with query / key norms, interleaved rotation, capped scores, a sink in the denominator, a window that
-// keeps the first keys and an output gate per head:
-// what comes before the scores (qkv_prep_kernel) and decoding with one query per row (grouped_decode_kernel). Prompts run
-// on the tcgen05 flash kernel (attention_sm100.cu) or, in 32-bit, on sink_attention_kernel (latent_attention.cu).
+// Grouped-query attention with query / key norms, rotation, capped scores, a sink in the denominator, a window that
+// keeps the first keys and an output gate per head or element:
+// what comes before the scores (qkv_prep_kernel, head_prep_kernel) and decoding with one query per row (grouped_decode_kernel). Prompts
+// run on the tcgen05 flash kernels (attention_sm100.cu) or, in 32-bit, on sink_attention_kernel (latent_attention.cu).
+//
+// Talking heads: scores mixed over the heads before the softmax, score_h <- sum_g talk[h, g] q_g . k_{group(g)}, are products of one
+// wide key per token (all key heads in a row) with the query [sum_{g in group 0} talk[h, g] q_g | the same of group 1 | ...].
+// head_prep_kernel writes these queries from normed and rotated heads in 32-bit, rounding once; from there on it is attention
+// with one key head for all query heads and value heads per group (wide_decode_kernel; fa_wide_kernel for prompts).
 //
 // Decode: a block scans a slice of one key / value head's cache for the query heads that share it (up to 16 on tensor cores,
 // 8 in the 32-bit version), so every cached byte is read once per block; grouped_finish_kernel merges the slices, adds the
@@ -123,6 +128,157 @@ __global__ void __launch_bounds__(256) qkv_prep_kernel(const PrepParams p) {
   }
 }
 
+// ------------------------------------------------------------------ rotation by halves, queries of talking heads
+struct HeadPrepParams {
+  const void *q, *k, *v; long long ldq, ldk, ldv;     // row b * S + t
+  const void *wq, *wk;                                // [dim], or nullptr
+  const long long* pos; long long pos_sb, pos_ss;
+  const float* freq; int n_freq, halves;
+  float amplitude;                                    // of sines and cosines
+  const void* talk;                                   // [H, H], or nullptr: the heads as they are
+  void* q_out;                                        // [B, S, H, talk ? G * dim : dim]
+  void *kc, *vc;                                      // heads g, position t at b * sb + g * sg + t * st
+  long long k_sb, k_sg, k_st, v_sb, v_sg, v_st;
+  const int* lengths;
+  int S, H, G, dim, vdim, Tmax;
+  float eps;
+  int* err;
+};
+
+constexpr int HP_WARPS = 8, HP_PER = 8;               // query heads per key head that a thread keeps in registers
+
+// block = (token, share of the query heads that are written); the first share also does keys and values. Angles are
+// computed once per token. VEC 4: everything is aligned to four elements
+template <typename T, int VEC>
+__global__ void __launch_bounds__(32 * HP_WARPS) head_prep_kernel(const HeadPrepParams p) {
+  extern __shared__ float hp_smem[];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, H = p.H, dim = p.dim;
+  float* cs = hp_smem;                                 // [n_freq]
+  float* sn = cs + p.n_freq;                           // [n_freq]
+  float* qs = sn + p.n_freq + (2 * p.n_freq % 4 ? 4 - 2 * p.n_freq % 4 : 0);   // [talk ? H : HP_WARPS][dim], 16-byte aligned
+  float* kb = qs + (p.talk ? H : HP_WARPS) * dim;      // [HP_WARPS][dim]
+  float* ts = kb + HP_WARPS * dim;                     // [share][H]
+  const long long row = blockIdx.x;
+  const long long b = row / p.S, t = row - b * p.S;
+  const int share = (H + gridDim.y - 1) / gridDim.y, h0 = blockIdx.y * share, h1 = min(H, h0 + share);
+  const float at = static_cast<float>(p.pos[b * p.pos_sb + t * p.pos_ss]);
+  for (int i = tid; i < p.n_freq; i += blockDim.x) {
+    float s, c;
+    sincosf(at * p.freq[i], &s, &c);
+    cs[i] = c * p.amplitude;
+    sn[i] = s * p.amplitude;
+  }
+  if (p.talk != nullptr)
+    for (int e = tid; e < (h1 - h0) * H; e += blockDim.x) ts[e] = Num<T>::to(static_cast<const T*>(p.talk)[static_cast<long long>(h0) * H + e]);
+  __syncthreads();
+  // one head, normed and rotated, in `buf`
+  auto head = [&](const T* src, const T* w, float* buf) {
+    float ss = 0.f;
+    for (int c = lane * VEC; c < dim; c += 32 * VEC) {
+      float x[VEC];
+      load_vec<T, VEC>(src + c, x);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) {
+        ss = fmaf(x[i], x[i], ss);
+        buf[c + i] = x[i];
+      }
+    }
+    const float r = 1.0f / sqrtf(warp_sum(ss) / dim + p.eps);
+    __syncwarp();
+    const int n = p.n_freq;
+    for (int i = lane; i < n; i += 32) {               // pairs
+      const int a = p.halves ? i : 2 * i, c = p.halves ? i + n : 2 * i + 1;
+      const float x = buf[a] * r * (w ? Num<T>::to(w[a]) : 1.f), y = buf[c] * r * (w ? Num<T>::to(w[c]) : 1.f);
+      buf[a] = x * cs[i] - y * sn[i];
+      buf[c] = y * cs[i] + x * sn[i];
+    }
+    for (int c = 2 * n + lane; c < dim; c += 32) buf[c] *= r * (w ? Num<T>::to(w[c]) : 1.f);
+    __syncwarp();
+  };
+  auto put = [&](T* dst, const float* buf) {
+    for (int c = lane * VEC; c < dim; c += 32 * VEC) {
+      float x[VEC];
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) x[i] = buf[c + i];
+      store_vec<T, VEC>(dst + c, x);
+    }
+  };
+  const T* q = static_cast<const T*>(p.q) + row * p.ldq;
+  const int q0 = p.talk ? 0 : h0, q1 = p.talk ? H : h1;
+  for (int h = q0 + warp; h < q1; h += HP_WARPS) {
+    float* buf = qs + (p.talk ? h : warp) * dim;
+    head(q + static_cast<long long>(h) * dim, static_cast<const T*>(p.wq), buf);
+    if (p.talk == nullptr) {
+      put(static_cast<T*>(p.q_out) + (row * H + h) * dim, buf);
+      __syncwarp();
+    }
+  }
+  if (blockIdx.y == 0) {
+    const long long to = p.lengths[b] + t;
+    if (to < 0 || to >= p.Tmax) {                      // never write outside the cache
+      if (tid == 0) OSLO_REPORT_BOUNDS(p.err);
+    } else {
+      for (int g = warp; g < 2 * p.G; g += HP_WARPS) {
+        if (g < p.G) {
+          float* buf = kb + warp * dim;
+          head(static_cast<const T*>(p.k) + row * p.ldk + static_cast<long long>(g) * dim, static_cast<const T*>(p.wk), buf);
+          put(static_cast<T*>(p.kc) + b * p.k_sb + g * p.k_sg + to * p.k_st, buf);
+          __syncwarp();
+        } else {
+          const T* src = static_cast<const T*>(p.v) + row * p.ldv + static_cast<long long>(g - p.G) * p.vdim;
+          T* dst = static_cast<T*>(p.vc) + b * p.v_sb + (g - p.G) * p.v_sg + to * p.v_st;
+          for (int c = lane * VEC; c < p.vdim; c += 32 * VEC)
+            *reinterpret_cast<Pack<T, VEC>*>(dst + c) = *reinterpret_cast<const Pack<T, VEC>*>(src + c);
+        }
+      }
+    }
+  }
+  if (p.talk == nullptr) return;
+  __syncthreads();
+  const int per = H / p.G, cols = p.G * dim, groups = cols / VEC;
+  T* out = static_cast<T*>(p.q_out) + row * H * cols;
+  // a thread owns VEC columns; with fewer columns than threads several threads share them, each with heads of its own
+  const int lanes = groups < static_cast<int>(blockDim.x) ? static_cast<int>(blockDim.x) / groups : 1;
+  if (tid / groups >= lanes && groups < static_cast<int>(blockDim.x)) return;
+  const int first = groups < static_cast<int>(blockDim.x) ? tid / groups : 0;
+  for (int u = groups < static_cast<int>(blockDim.x) ? tid % groups : tid; u < groups; u += groups < static_cast<int>(blockDim.x) ? groups : static_cast<int>(blockDim.x)) {
+    const int c = u * VEC, g = c / dim, d = c - g * dim;
+    const float* src = qs + g * per * dim + d;
+    if (per <= HP_PER) {
+      float x[HP_PER][VEC];
+#pragma unroll
+      for (int r = 0; r < HP_PER; ++r)
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) x[r][i] = r < per ? src[r * dim + i] : 0.f;
+      for (int h = first; h < h1 - h0; h += lanes) {
+        const float* tw = ts + h * H + g * per;
+        float o[VEC];
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) o[i] = 0.f;
+#pragma unroll
+        for (int r = 0; r < HP_PER; ++r) {
+          if (r >= per) break;
+          const float m = tw[r];
+#pragma unroll
+          for (int i = 0; i < VEC; ++i) o[i] = fmaf(m, x[r][i], o[i]);
+        }
+        store_vec<T, VEC>(out + static_cast<long long>(h0 + h) * cols + c, o);
+      }
+    } else {
+      for (int h = first; h < h1 - h0; h += lanes) {
+        const float* tw = ts + h * H + g * per;
+        float o[VEC];
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) o[i] = 0.f;
+        for (int r = 0; r < per; ++r)
+#pragma unroll
+          for (int i = 0; i < VEC; ++i) o[i] = fmaf(tw[r], src[r * dim + i], o[i]);
+        store_vec<T, VEC>(out + static_cast<long long>(h0 + h) * cols + c, o);
+      }
+    }
+  }
+}
+
 // ------------------------------------------------------------------ decode
 struct GroupedParams {
   const void* q;                       // [B, H, dim]
@@ -132,6 +288,7 @@ struct GroupedParams {
   float* ws;                           // [B, H, splits, ldw]: sum p v; ldw = vdim rounded up to a multiple of 4
   float* stat;                         // [B, H, splits, 2]: max, sum p
   int H, G, dim, vdim, ldw, Tmax, splits;
+  int VG;                              // value heads in a cached value row (wide keys: G = 1, all value heads in a row); else 1
   float scale, softcap;
   int window, keep_first;              // window > 0: the last `window` positions, and the first keep_first after lead[b]
   const int* lead;                     // [B] padding ahead of the sequence, or nullptr
@@ -242,12 +399,14 @@ __global__ void __launch_bounds__(256) grouped_decode_kernel(const GroupedParams
     }
   }
   __syncthreads();
+  const int vd = p.vdim / p.VG;
   for (int a = 0; a < nh; ++a) {
     const long long at = (static_cast<long long>(b) * p.H + h0 + a) * p.splits + sp;
+    const int own = p.VG > 1 ? (h0 + a) / (p.H / p.VG) * vd : 0;          // the head's own columns
 #pragma unroll
     for (int j = 0; j < NR; ++j) {
-      const int c = tid + j * 256;
-      if (c < p.vdim) {
+      const int c = tid + j * 256 - own;
+      if (c >= 0 && c < vd) {
         float v = 0.f;
 #pragma unroll
         for (int u = 0; u < GD_HEADS; ++u) v = u == a ? acc[j][u] : v;
@@ -454,11 +613,299 @@ __global__ void __launch_bounds__(128) grouped_decode_mma_kernel(const GroupedPa
   }
 }
 
+// ------------------------------------------------------------------ decode, wide keys on tensor cores
+// One cached key row (dim columns) for all query heads, value heads side by side in a cached value row: block = (slice, up to 16 MT
+// query heads, row). A stage of KEYS keys and values is on its way while the one before is used: (1) scores of 16 heads x 16 keys per
+// warp (over a share of the columns when there are fewer tiles than warps), (2) softmax, a warp per head row, (3) 16 heads x 64 value
+// columns per item, only the columns of these heads' groups.
+constexpr int WD_WARPS = 8;
+
+struct WideLayout {
+  int kp, vp;                          // row pitches of the key and value stages
+  size_t q, k, v, s, p, total;         // byte offsets
+};
+template <int MT, int KEYS, int NBUF>
+__host__ __device__ inline WideLayout wide_layout(int dim, int vdim) {
+  WideLayout l;
+  l.kp = (dim + 15) / 16 * 16 + 8;     // 16-byte rows whose starts fall on different banks
+  l.vp = (vdim + 15) / 16 * 16 + 8;
+  constexpr int TILES = MT * KEYS / 16, KSPLIT = WD_WARPS / (TILES < WD_WARPS ? TILES : WD_WARPS);
+  l.q = 0;
+  l.k = l.q + static_cast<size_t>(MT) * 16 * l.kp * 2;
+  l.v = l.k + static_cast<size_t>(NBUF) * KEYS * l.kp * 2;
+  l.s = l.v + static_cast<size_t>(NBUF) * KEYS * l.vp * 2;
+  l.p = l.s + static_cast<size_t>(KSPLIT) * MT * 16 * (KEYS + 1) * 4;
+  l.p = (l.p + 15) / 16 * 16;
+  l.total = l.p + static_cast<size_t>(MT) * 16 * (KEYS + 8) * 2;
+  return l;
+}
+
+template <typename T, int MT, int KEYS, int NBUF, int ITEMS>
+__global__ void __launch_bounds__(32 * WD_WARPS) wide_decode_kernel(const GroupedParams p) {
+  constexpr int ROWS = MT * 16, TILES = MT * KEYS / 16, KSPLIT = WD_WARPS / (TILES < WD_WARPS ? TILES : WD_WARPS);
+  constexpr int RW = ROWS / WD_WARPS;                  // head rows of a warp in step 2
+  static_assert(TILES <= WD_WARPS, "a warp has one tile of scores");
+  extern __shared__ uint4 gm_smem[];
+  const WideLayout lay = wide_layout<MT, KEYS, NBUF>(p.dim, p.vdim);
+  uint8_t* base = reinterpret_cast<uint8_t*>(gm_smem);
+  T* qs = reinterpret_cast<T*>(base + lay.q);          // [ROWS][kp]
+  T* ks = reinterpret_cast<T*>(base + lay.k);          // [NBUF][KEYS][kp]
+  T* vs = reinterpret_cast<T*>(base + lay.v);          // [NBUF][KEYS][vp]
+  float* sc = reinterpret_cast<float*>(base + lay.s);  // [KSPLIT][ROWS][KEYS + 1]
+  T* ps = reinterpret_cast<T*>(base + lay.p);          // [ROWS][KEYS + 8]
+  __shared__ float alpha_s[ROWS];
+  const int b = blockIdx.z, sp = blockIdx.x, tid = threadIdx.x, w = tid >> 5, l = tid & 31;
+  const int h0 = blockIdx.y * ROWS, nh = min(ROWS, p.H - h0);
+  const int vd = p.vdim / p.VG, per = p.H / p.VG;      // columns of a value head, query heads that read it
+  int len = p.lengths[b];
+  if (len < 0 || len > p.Tmax) {             // a length that does not fit the cache: never read past it
+    if (tid == 0) OSLO_REPORT_BOUNDS(p.err);
+    len = len < 0 ? 0 : p.Tmax;
+  }
+  const KeyRun run(p, b, len);
+  const int span = (run.n + p.splits - 1) / p.splits;
+  const int t0 = sp * span, t1 = min(run.n, t0 + span);
+  const T* kb = static_cast<const T*>(p.kc) + static_cast<long long>(b) * p.Tmax * p.dim;
+  const T* vb = static_cast<const T*>(p.vc) + static_cast<long long>(b) * p.Tmax * p.vdim;
+  const T* q = static_cast<const T*>(p.q) + (static_cast<long long>(b) * p.H + h0) * p.dim;
+  const int kc8 = p.dim / 8, vc8 = p.vdim / 8;
+  // columns past the rows' ends and rows past the heads are zero for good: the copies below never write them
+  for (int e = tid; e < ROWS * (lay.kp / 8); e += blockDim.x) {
+    const int a = e / (lay.kp / 8), c = e % (lay.kp / 8);
+    uint4 v = make_uint4(0, 0, 0, 0);
+    if (a < nh && c < kc8) v = *reinterpret_cast<const uint4*>(q + static_cast<long long>(a) * p.dim + c * 8);
+    *reinterpret_cast<uint4*>(qs + a * lay.kp + c * 8) = v;
+  }
+  for (int t = tid; t < NBUF * KEYS; t += blockDim.x) {
+    for (int c = kc8; c < lay.kp / 8; ++c) *reinterpret_cast<uint4*>(ks + t * lay.kp + c * 8) = make_uint4(0, 0, 0, 0);
+    for (int c = vc8; c < lay.vp / 8; ++c) *reinterpret_cast<uint4*>(vs + t * lay.vp + c * 8) = make_uint4(0, 0, 0, 0);
+  }
+  // a warp copies whole rows
+  auto fetch = [&](int k0, int buf) {
+    for (int t = w; t < KEYS; t += WD_WARPS) {
+      const bool ok = k0 + t < t1;
+      const long long pos = run.at(ok ? k0 + t : t0);
+      const int bytes = ok ? 16 : 0;                   // 0: the 16 bytes are filled with zeros
+      T* kd = ks + (buf * KEYS + t) * lay.kp;
+      T* vdst = vs + (buf * KEYS + t) * lay.vp;
+#pragma unroll 4
+      for (int c = l; c < kc8; c += 32)
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(kd + c * 8)), "l"(kb + pos * p.dim + c * 8), "r"(bytes) : "memory");
+#pragma unroll 4
+      for (int c = l; c < vc8; c += 32)
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(vdst + c * 8)), "l"(vb + pos * p.vdim + c * 8), "r"(bytes) : "memory");
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  // step 1: tile of this warp and its share of the columns
+  const int tile = w % TILES, mt = tile % MT, kt = tile / MT, part = w / TILES;
+  const int steps = (p.dim + 15) / 16, step0 = steps * part / KSPLIT, step1 = steps * (part + 1) / KSPLIT;
+  // step 3: items (16 heads, 64 of the columns of their groups), dealt out to the warps
+  int item_mt[ITEMS], item_c0[ITEMS], item_c1[ITEMS];
+#pragma unroll
+  for (int i = 0; i < ITEMS; ++i) { item_mt[i] = -1; item_c0[i] = item_c1[i] = 0; }
+  {
+    int n = 0;
+#pragma unroll
+    for (int m = 0; m < MT; ++m) {
+      if (m * 16 >= nh) break;
+      const int lo = (h0 + m * 16) / per * vd, hi = ((h0 + min(nh, m * 16 + 16) - 1) / per + 1) * vd;
+      for (int c = lo; c < hi; c += 64, ++n)
+        if (n % WD_WARPS == w) {
+#pragma unroll
+          for (int i = 0; i < ITEMS; ++i)
+            if (i == n / WD_WARPS) { item_mt[i] = m; item_c0[i] = c; item_c1[i] = min(hi, c + 64); }
+        }
+    }
+  }
+  float o[ITEMS][8][4];
+#pragma unroll
+  for (int i = 0; i < ITEMS; ++i)
+#pragma unroll
+    for (int j = 0; j < 8; ++j) o[i][j][0] = o[i][j][1] = o[i][j][2] = o[i][j][3] = 0.f;
+  float m_row[RW], l_row[RW];                          // of the warp's head rows, the same in every lane; scores in log2 units
+#pragma unroll
+  for (int r = 0; r < RW; ++r) { m_row[r] = -CUDART_INF_F; l_row[r] = 0.f; }
+  const float scale = p.scale * GD_LOG2E;
+  if (t0 < t1) fetch(t0, 0);
+  for (int k0 = t0, it = 0; k0 < t1; k0 += KEYS, ++it) {
+    const int buf = NBUF > 1 ? it & 1 : 0;
+    if (NBUF > 1 && k0 + KEYS < t1) {
+      fetch(k0 + KEYS, buf ^ 1);
+      asm volatile("cp.async.wait_group 1;" ::: "memory");
+    } else {
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
+    }
+    __syncthreads();
+    {
+      float c[2][4] = {};
+      const T* kw = ks + (buf * KEYS + kt * 16) * lay.kp;
+      const T* qw = qs + mt * 16 * lay.kp;
+#pragma unroll 4
+      for (int kk = step0; kk < step1; ++kk) {
+        uint32_t a[4], bb[4];
+        gd_ldsm4(a, smem_u32(qw + ((l & 7) + ((l >> 3) & 1) * 8) * lay.kp + kk * 16 + (l >> 4) * 8));
+        gd_ldsm4(bb, smem_u32(kw + ((l & 7) + (l >> 4) * 8) * lay.kp + kk * 16 + ((l >> 3) & 1) * 8));
+        GdMma<T>::run(c[0], a, bb[0], bb[1]);
+        GdMma<T>::run(c[1], a, bb[2], bb[3]);
+      }
+      float* dst = sc + (part * ROWS + mt * 16) * (KEYS + 1) + kt * 16;
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) dst[((l >> 2) + (e >> 1) * 8) * (KEYS + 1) + nt * 8 + (l & 3) * 2 + (e & 1)] = c[nt][e];
+    }
+    __syncthreads();
+    {
+      constexpr int KL = (KEYS + 31) / 32;             // keys per lane
+      bool vis[KL];
+#pragma unroll
+      for (int u = 0; u < KL; ++u) {
+        const int j = l + 32 * u, pos = run.at(k0 + j);
+        vis[u] = j < KEYS && k0 + j < t1 && (p.keep == nullptr || pos >= p.n_keep || p.keep[b * p.ld_keep + pos]);
+      }
+#pragma unroll
+      for (int r = 0; r < RW; ++r) {
+        const int row = w * RW + r;
+        float d[KL], mx = m_row[r];
+#pragma unroll
+        for (int u = 0; u < KL; ++u) {
+          const int j = l + 32 * u;
+          float x = 0.f;
+          if (j < KEYS) {
+#pragma unroll
+            for (int s = 0; s < KSPLIT; ++s) x += sc[(s * ROWS + row) * (KEYS + 1) + j];
+          }
+          d[u] = vis[u] ? x * scale : -CUDART_INF_F;
+          mx = fmaxf(mx, d[u]);
+        }
+#pragma unroll
+        for (int off = 16; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
+        const float ref = mx == -CUDART_INF_F ? 0.f : mx, al = gd_exp2(m_row[r] - ref);     // 2^-inf = 0
+        float sum = 0.f;
+#pragma unroll
+        for (int u = 0; u < KL; ++u) {
+          const int j = l + 32 * u;
+          const float e = gd_exp2(d[u] - ref);
+          sum += e;
+          if (j < KEYS) ps[row * (KEYS + 8) + j] = Num<T>::from(e);
+        }
+        l_row[r] = l_row[r] * al + warp_sum(sum);
+        m_row[r] = mx;
+        if (l == 0) alpha_s[row] = al;
+      }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < ITEMS; ++i) {
+      if (item_mt[i] < 0) continue;                    // uniform over the warp
+      const float a0 = alpha_s[item_mt[i] * 16 + (l >> 2)], a1 = alpha_s[item_mt[i] * 16 + (l >> 2) + 8];
+      if (__any_sync(0xffffffffu, a0 != 1.f || a1 != 1.f)) {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) { o[i][j][0] *= a0; o[i][j][1] *= a0; o[i][j][2] *= a1; o[i][j][3] *= a1; }
+      }
+      const T* pw = ps + item_mt[i] * 16 * (KEYS + 8);
+#pragma unroll
+      for (int kk = 0; kk < KEYS / 16; ++kk) {
+        uint32_t a[4];
+        gd_ldsm4(a, smem_u32(pw + ((l & 7) + ((l >> 3) & 1) * 8) * (KEYS + 8) + kk * 16 + (l >> 4) * 8));
+        const T* vw = vs + (buf * KEYS + kk * 16 + (l & 7) + ((l >> 3) & 1) * 8) * lay.vp + item_c0[i] + (l >> 4) * 8;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          if (item_c0[i] + j * 16 >= item_c1[i]) break;
+          uint32_t bb[4];
+          gd_ldsm4_t(bb, smem_u32(vw + j * 16));
+          GdMma<T>::run(o[i][2 * j], a, bb[0], bb[1]);
+          GdMma<T>::run(o[i][2 * j + 1], a, bb[2], bb[3]);
+        }
+      }
+    }
+    __syncthreads();                                   // the stage may be fetched over
+    if (NBUF == 1 && k0 + KEYS < t1) fetch(k0 + KEYS, 0);
+  }
+#pragma unroll
+  for (int i = 0; i < ITEMS; ++i) {
+    if (item_mt[i] < 0) continue;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const int c = item_c0[i] + j * 8 + (l & 3) * 2;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int a = item_mt[i] * 16 + (l >> 2) + (e >> 1) * 8, col = c + (e & 1);
+        if (a >= nh || col >= item_c1[i] || col / vd != (h0 + a) / per) continue;
+        p.ws[((static_cast<long long>(b) * p.H + h0 + a) * p.splits + sp) * p.ldw + col % vd] = o[i][j][e];
+      }
+    }
+  }
+  if (l == 0) {
+#pragma unroll
+    for (int r = 0; r < RW; ++r) {
+      const int a = w * RW + r;
+      if (a >= nh) continue;
+      const long long at = (static_cast<long long>(b) * p.H + h0 + a) * p.splits + sp;
+      p.stat[at * 2] = m_row[r] * GD_LN2;
+      p.stat[at * 2 + 1] = l_row[r];
+    }
+  }
+}
+
+constexpr size_t WD_SMEM = 220 * 1024;
+// how the wide kernel runs these sizes: MT, KEYS, NBUF and ITEMS; keys 0: not at all
+struct WidePlan { int mt, keys, nbuf, items; size_t smem; };
+static WidePlan wide_plan(int H, int VG, int dim, int vdim, int dtype) {
+  WidePlan w{0, 0, 0, 0, 0};
+  if (dtype == OSLO_DT_FP32 || dim % 8 || vdim % VG || (vdim / VG) % 8) return w;
+  w.mt = H > 16 ? 2 : 1;
+  const int vd = vdim / VG, per = H / VG;
+  int worst = 0;
+  for (int h0 = 0; h0 < H; h0 += 16 * w.mt) {
+    int n = 0;
+    for (int m = 0; m < w.mt && h0 + m * 16 < H; ++m) {
+      const int a = h0 + m * 16, z = std::min(H, a + 16) - 1;
+      n += ((z / per - a / per + 1) * vd + 63) / 64;
+    }
+    worst = std::max(worst, n);
+  }
+  const int items = (worst + WD_WARPS - 1) / WD_WARPS;
+  if (items > 4) return w;
+  w.items = items <= 1 ? 1 : (items <= 2 ? 2 : 4);
+  auto fits = [&](size_t bytes, int keys, int nbuf) {
+    if (bytes > WD_SMEM) return false;
+    w.keys = keys; w.nbuf = nbuf; w.smem = bytes;
+    return true;
+  };
+#define WD_TRY(K, N) (w.mt == 2 ? fits(wide_layout<2, K, N>(dim, vdim).total, K, N) : fits(wide_layout<1, K, N>(dim, vdim).total, K, N))
+  if (WD_TRY(32, 2) || WD_TRY(16, 2) || WD_TRY(16, 1)) return w;
+#undef WD_TRY
+  return w;
+}
+
+template <typename T, int MT, int KEYS, int NBUF, int ITEMS>
+static int wide_launch(const GroupedParams& p, int B, size_t smem, cudaStream_t st) {
+  cudaError_t e = cudaFuncSetAttribute(wide_decode_kernel<T, MT, KEYS, NBUF, ITEMS>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                       static_cast<int>(smem));
+  if (e != cudaSuccess) return static_cast<int>(e);
+  wide_decode_kernel<T, MT, KEYS, NBUF, ITEMS><<<dim3(p.splits, (p.H + 16 * MT - 1) / (16 * MT), B), 32 * WD_WARPS, smem, st>>>(p);
+  return static_cast<int>(cudaGetLastError());
+}
+template <typename T, int MT, int KEYS, int NBUF>
+static int wide_items(const GroupedParams& p, int B, const WidePlan& w, cudaStream_t st) {
+  if (w.items == 1) return wide_launch<T, MT, KEYS, NBUF, 1>(p, B, w.smem, st);
+  if (w.items == 2) return wide_launch<T, MT, KEYS, NBUF, 2>(p, B, w.smem, st);
+  return wide_launch<T, MT, KEYS, NBUF, 4>(p, B, w.smem, st);
+}
+template <typename T, int MT>
+static int wide_keys(const GroupedParams& p, int B, const WidePlan& w, cudaStream_t st) {
+  if (w.keys == 32) return wide_items<T, MT, 32, 2>(p, B, w, st);
+  if (w.nbuf == 2) return wide_items<T, MT, 16, 2>(p, B, w, st);
+  return wide_items<T, MT, 16, 1>(p, B, w, st);
+}
+
 // block = (head, row): merge the slices; exp(sink) joins the denominator (sink null: nothing does)
 template <typename T>
 __global__ void __launch_bounds__(128) grouped_finish_kernel(const float* __restrict__ ws, const float* __restrict__ stat,
                                                              const T* __restrict__ sink, const T* __restrict__ gate, long long ldg,
-                                                             T* __restrict__ out, int H, int vdim, int ldw, int splits) {
+                                                             int gate_wide, T* __restrict__ out, int H, int vdim, int ldw, int splits) {
   __shared__ float red[4], fac[GD_MAX_SPLITS];
   const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x;
   const long long at = (static_cast<long long>(b) * H + h) * splits;
@@ -477,11 +924,13 @@ __global__ void __launch_bounds__(128) grouped_finish_kernel(const float* __rest
   if ((tid & 31) == 0) red[tid >> 5] = part;
   __syncthreads();
   const float den = red[0] + red[1] + red[2] + red[3] + (sink ? expf(snk - m) : 0.f);
-  const float inv = den > 0.f ? (gate ? sigmoid_f(Num<T>::to(gate[b * ldg + h])) : 1.0f) / den : 0.f;   // no visible key: zeros
+  const bool narrow = gate != nullptr && !gate_wide;
+  const float inv = den > 0.f ? (narrow ? sigmoid_f(Num<T>::to(gate[b * ldg + h])) : 1.0f) / den : 0.f;   // no visible key: zeros
   for (int c = tid; c < vdim; c += blockDim.x) {
     float v = 0.f;
 #pragma unroll 8
     for (int s = 0; s < splits; ++s) v = fmaf(ws[(at + s) * ldw + c], fac[s], v);
+    if (gate != nullptr && gate_wide) v *= sigmoid_f(Num<T>::to(gate[b * ldg + static_cast<long long>(h) * vdim + c]));
     out[(static_cast<long long>(b) * H + h) * vdim + c] = Num<T>::from(v * inv);
   }
 }
@@ -525,8 +974,66 @@ extern "C" int oslo_qkv_prep(const void* q, long long ldq, const void* k, long l
   return static_cast<int>(cudaGetLastError());
 }
 
-extern "C" int oslo_grouped_splits(int B, int H, int G, int T, int dim, int vdim, int dtype, int num_sms) {
+extern "C" int oslo_head_prep(const void* q, long long ldq, const void* k, long long ldk, const void* v, long long ldv,
+                              const void* wq, const void* wk, float eps, const long long* pos, long long pos_sb, long long pos_ss,
+                              const float* freq, int n_freq, int halves, float amplitude, const void* talk, void* q_out, void* kc,
+                              long long k_sb, long long k_sg, long long k_st, void* vc, long long v_sb, long long v_sg,
+                              long long v_st, const int* lengths, int B, int S, int H, int G, int dim, int vdim, int Tmax,
+                              int num_sms, int dtype, int* err_word, cudaStream_t stream) {
   using namespace oslo;
+  if (B <= 0 || S <= 0) return 0;
+  if (H <= 0 || G <= 0 || H % G || dim <= 0 || vdim <= 0 || 2 * n_freq > dim) return -1;
+  const long long tokens = static_cast<long long>(B) * S;
+  if (tokens > 0x7fffffffll) return -1;
+  HeadPrepParams p{q, k, v, ldq, ldk, ldv, wq, wk, pos, pos_sb, pos_ss, freq, n_freq, halves, amplitude, talk, q_out, kc, vc,
+                   k_sb, k_sg, k_st, v_sb, v_sg, v_st, lengths, S, H, G, dim, vdim, Tmax, eps, err_word};
+  // few tokens: several blocks write the heads of one (each norms all of them first where heads are mixed)
+  const int shares = static_cast<int>(std::max<long long>(1, std::min<long long>(talk ? (H + 3) / 4 : (H + HP_WARPS - 1) / HP_WARPS, num_sms / tokens)));
+  const int share = (H + shares - 1) / shares;
+  const size_t smem = (2 * static_cast<size_t>(n_freq) + 4 + static_cast<size_t>(talk ? H : HP_WARPS) * dim + static_cast<size_t>(HP_WARPS) * dim +
+                       (talk ? static_cast<size_t>(share) * H : 0)) * sizeof(float);
+  if (smem > 220 * 1024) return -3;
+  const size_t a4 = dtype == OSLO_DT_FP32 ? 16 : 8;
+  bool vec = dim % 4 == 0 && vdim % 4 == 0;
+  for (long long s : {ldq, ldk, ldv, k_sb, k_sg, k_st, v_sb, v_sg, v_st}) vec = vec && s % 4 == 0;
+  for (const void* t : {q, k, v, static_cast<const void*>(q_out), static_cast<const void*>(kc), static_cast<const void*>(vc)})
+    vec = vec && aligned_to(t, a4);
+#define HP_GO(V)                                                                                                               \
+  {                                                                                                                            \
+    if (smem > 48 * 1024) {                                                                                                    \
+      cudaError_t e = cudaFuncSetAttribute(head_prep_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)); \
+      if (e != cudaSuccess) return static_cast<int>(e);                                                                        \
+    }                                                                                                                          \
+    head_prep_kernel<T, V><<<dim3(static_cast<unsigned>(tokens), shares), 32 * HP_WARPS, smem, stream>>>(p);                   \
+  }
+  OSLO_DISPATCH_T(dtype, { if (vec) HP_GO(4) else HP_GO(1) });
+#undef HP_GO
+  return static_cast<int>(cudaGetLastError());
+}
+
+// whether oslo_grouped_decode runs wide keys (one key head, VG value heads in a cached row) of these sizes
+extern "C" int oslo_wide_decode_fits(int H, int VG, int dim, int vdim, int dtype) {
+  using namespace oslo;
+  if (wide_plan(H, VG, dim, vdim, dtype).keys) return 1;
+  const size_t smem = (static_cast<size_t>(GD_HEADS + GD_KEYS) * (dim + 1) + static_cast<size_t>(GD_KEYS) * vdim) * sizeof(float);
+  return vdim <= 1024 && smem <= 220 * 1024 ? 1 : 0;
+}
+
+extern "C" int oslo_grouped_splits(int B, int H, int G, int VG, int T, int dim, int vdim, int dtype, int num_sms) {
+  using namespace oslo;
+  const WidePlan wide = VG > 1 ? wide_plan(H, VG, dim, vdim, dtype) : WidePlan{};
+  if (wide.keys) {
+    // whole waves of blocks: a block costs its share of the keys and some for its start
+    const long long blocks = static_cast<long long>(B) * ((H + 16 * wide.mt - 1) / (16 * wide.mt));
+    const long long room = static_cast<long long>(num_sms) * std::max<size_t>(1, std::min<size_t>(4, WD_SMEM / (wide.smem + 2048)));
+    int best = 1;
+    double best_cost = 1e30;
+    for (int n = 1; n <= GD_MAX_SPLITS && (n == 1 || n * 64 <= T); ++n) {
+      const double cost = static_cast<double>((blocks * n + room - 1) / room) * (static_cast<double>(T) / n + 96.0);
+      if (cost < best_cost * 0.999) { best_cost = cost; best = n; }
+    }
+    return best;
+  }
   const int per = gd_use_mma(dim, vdim, dtype) ? GM_HEADS : GD_HEADS;
   const long long blocks = static_cast<long long>(B) * G * ((H / G + per - 1) / per);
   long long s = (3ll * num_sms + blocks - 1) / blocks;
@@ -535,15 +1042,30 @@ extern "C" int oslo_grouped_splits(int B, int H, int G, int T, int dim, int vdim
 }
 
 extern "C" int oslo_grouped_decode(const void* q, const void* kc, const void* vc, const int* lengths, const uint8_t* keep,
-                                   long long ld_keep, int n_keep, const void* sink, const void* gate, long long ldg, int window,
-                                   int keep_first, const int* lead, float* ws, float* stat, void* out, int B, int H, int G, int dim,
-                                   int vdim, int Tmax, int splits, float scale, float softcap, int dtype, int* err_word,
-                                   cudaStream_t stream) {
+                                   long long ld_keep, int n_keep, const void* sink, const void* gate, long long ldg, int gate_wide,
+                                   int window, int keep_first, const int* lead, float* ws, float* stat, void* out, int B, int H,
+                                   int G, int VG, int dim, int vdim, int Tmax, int splits, float scale, float softcap, int dtype,
+                                   int* err_word, cudaStream_t stream) {
   using namespace oslo;
   if (B <= 0 || H <= 0) return 0;
   if (G <= 0 || H % G || B > 65535 || window < 0 || keep_first < 0 || splits < 1 || splits > GD_MAX_SPLITS) return -1;
-  GroupedParams p{q, kc, vc, lengths, keep, ld_keep, n_keep, ws, stat, H, G, dim, vdim, (vdim + 3) / 4 * 4, Tmax, splits,
+  if (VG < 1 || (VG > 1 && (G != 1 || H % VG || vdim % VG))) return -1;
+  const int vd = vdim / VG;
+  GroupedParams p{q, kc, vc, lengths, keep, ld_keep, n_keep, ws, stat, H, G, dim, vdim, (vd + 3) / 4 * 4, Tmax, splits, VG,
                   scale, softcap, window, keep_first, lead, err_word};
+#define GD_FINISH(T)                                                                                                               \
+  grouped_finish_kernel<T><<<dim3(H, B), 128, 0, stream>>>(ws, stat, static_cast<const T*>(sink), static_cast<const T*>(gate), ldg, \
+                                                           gate_wide, static_cast<T*>(out), H, vd, p.ldw, splits)
+  const WidePlan wide = VG > 1 && softcap <= 0.f ? wide_plan(H, VG, dim, vdim, dtype) : WidePlan{};
+  if (wide.keys && aligned_to(q, 16) && aligned_to(kc, 16) && aligned_to(vc, 16)) {
+    int rc = 0;
+#define WD_GO(T)                                                                                                       \
+  rc = wide.mt == 2 ? wide_keys<T, 2>(p, B, wide, stream) : wide_keys<T, 1>(p, B, wide, stream);                       \
+  if (rc == 0) GD_FINISH(T);
+    if (dtype == OSLO_DT_BF16) { WD_GO(__nv_bfloat16) } else { WD_GO(__half) }
+#undef WD_GO
+    return rc ? rc : static_cast<int>(cudaGetLastError());
+  }
   const int tiles = (H / G + GD_HEADS - 1) / GD_HEADS;
   const dim3 grid(splits, G * tiles, B);
   const size_t smem = (static_cast<size_t>(GD_HEADS + GD_KEYS) * (dim + 1) + static_cast<size_t>(GD_KEYS) * vdim) * sizeof(float);
@@ -557,15 +1079,13 @@ extern "C" int oslo_grouped_decode(const void* q, const void* kc, const void* vc
     }                                                                                                              \
     grouped_decode_kernel<T, NR><<<grid, 256, smem, stream>>>(p);                                                  \
   }
-  if (gd_use_mma(dim, vdim, dtype) && aligned_to(q, 16) && aligned_to(kc, 16) && aligned_to(vc, 16)) {
+  if (VG == 1 && gd_use_mma(dim, vdim, dtype) && aligned_to(q, 16) && aligned_to(kc, 16) && aligned_to(vc, 16)) {
     const int widest = std::max(dim, vdim);
     int rc = 0;
 #define GM_GO(T)                                                                                                              \
   rc = widest <= 64 ? gd_mma_launch<T, 64>(p, B, stream) : (widest <= 128 ? gd_mma_launch<T, 128>(p, B, stream)               \
                                                                            : gd_mma_launch<T, 256>(p, B, stream));            \
-  if (rc == 0)                                                                                                                \
-    grouped_finish_kernel<T><<<dim3(H, B), 128, 0, stream>>>(ws, stat, static_cast<const T*>(sink), static_cast<const T*>(gate), \
-                                                             ldg, static_cast<T*>(out), H, vdim, p.ldw, splits);
+  if (rc == 0) GD_FINISH(T);
     if (dtype == OSLO_DT_BF16) { GM_GO(__nv_bfloat16) } else { GM_GO(__half) }
 #undef GM_GO
     return rc ? rc : static_cast<int>(cudaGetLastError());
@@ -575,9 +1095,9 @@ extern "C" int oslo_grouped_decode(const void* q, const void* kc, const void* vc
     else if (vdim <= 512) GD_GO(2)
     else if (vdim <= 1024) GD_GO(4)
     else return -3;
-    grouped_finish_kernel<T><<<dim3(H, B), 128, 0, stream>>>(ws, stat, static_cast<const T*>(sink), static_cast<const T*>(gate), ldg,
-                                                             static_cast<T*>(out), H, vdim, p.ldw, splits);
+    GD_FINISH(T);
   });
+#undef GD_FINISH
 #undef GD_GO
   return static_cast<int>(cudaGetLastError());
 }

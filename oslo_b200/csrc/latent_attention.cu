@@ -57,7 +57,7 @@ struct SinkAttnParams {
   const void* sink;
   const void* gate; long long ldg;     // row b * Sq + s; nullptr: no output gate
   void* out;                           // [B * Sq, H * vdim]
-  int B, H, G, Sq, Sk, dim, vdim;      // query head h reads key / value head h / (H / G)
+  int B, H, G, KG, Sq, Sk, dim, vdim;  // query head h reads key head h / (H / KG) and value head h / (H / G)
   float scale, softcap;                // softcap > 0: scores become softcap * tanh(score / softcap)
   int window, keep_first;              // window > 0: the last `window` keys, and the first keep_first after lead[b]
   const int* lead;                     // [B] padding ahead of the sequence, or nullptr
@@ -80,9 +80,8 @@ __global__ void __launch_bounds__(128) sink_attention_kernel(const SinkAttnParam
   const int tid = threadIdx.x, qi = tid >> 3, l8 = tid & 7;
   const int past = p.Sk - p.Sq;
   const T* q = static_cast<const T*>(p.q) + b * p.q_sb + h * p.q_sh;
-  const int kv = h / (p.H / p.G);
-  const T* k = static_cast<const T*>(p.k) + b * p.k_sb + kv * p.k_sh;
-  const T* v = static_cast<const T*>(p.v) + b * p.v_sb + kv * p.v_sh;
+  const T* k = static_cast<const T*>(p.k) + b * p.k_sb + h / (p.H / p.KG) * p.k_sh;
+  const T* v = static_cast<const T*>(p.v) + b * p.v_sb + h / (p.H / p.G) * p.v_sh;
   for (int e = tid; e < SA_Q * p.dim; e += 128) {
     const int r = e / p.dim, c = e % p.dim;
     qs[r * dp + c] = q0 + r < p.Sq ? Num<T>::to(q[(q0 + r) * p.q_ss + c]) : 0.f;
@@ -898,14 +897,14 @@ extern "C" int oslo_sink_gate(const void* o, long long o_sb, long long o_ss, lon
 extern "C" int oslo_sink_attention(const void* q, long long q_sb, long long q_ss, long long q_sh, const void* k, long long k_sb,
                                    long long k_ss, long long k_sh, const void* v, long long v_sb, long long v_ss,
                                    long long v_sh, const uint8_t* keep, long long ld_keep, const void* sink, const void* gate,
-                                   long long ldg, void* out, int B, int H, int G, int Sq, int Sk, int dim, int vdim, float scale,
+                                   long long ldg, void* out, int B, int H, int G, int KG, int Sq, int Sk, int dim, int vdim, float scale,
                                    float softcap, int window, int keep_first, const int* lead, int gate_wide, int dtype,
                                    cudaStream_t stream) {
   using namespace oslo;
   if (B <= 0 || H <= 0 || Sq <= 0) return 0;
-  if (Sk < Sq || B > 65535 || H > 65535 || G <= 0 || H % G) return -1;
+  if (Sk < Sq || B > 65535 || H > 65535 || G <= 0 || H % G || KG <= 0 || H % KG) return -1;
   SinkAttnParams p{q, k, v, q_sb, q_ss, q_sh, k_sb, k_ss, k_sh, v_sb, v_ss, v_sh, keep, ld_keep, sink, gate, ldg, out,
-                   B, H, G, Sq, Sk, dim, vdim, scale, softcap, window, keep_first, lead, gate_wide};
+                   B, H, G, KG, Sq, Sk, dim, vdim, scale, softcap, window, keep_first, lead, gate_wide};
   const size_t smem = (static_cast<size_t>(SA_Q + SA_K) * (dim + 1 + vdim + 1) + SA_Q * (SA_K + 1)) * sizeof(float);
   dim3 grid((Sq + SA_Q - 1) / SA_Q, H, B);
   OSLO_DISPATCH_T(dtype, {

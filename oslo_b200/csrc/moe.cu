@@ -3,11 +3,13 @@
 //
 //   route:   z = W_router h + b (32-bit), the `top` largest, softmax over those only; or scored: s = softmax(W_router h) over
 //            all outputs, the `top` largest s + b, weights s / sum of the chosen s. Outputs past the experts stand for the
-//            input itself: no slot and no product, the step that joins the residual stream knows them
+//            input itself: no slot and no product, the step that joins the residual stream knows them. Or sigmoid scores: the
+//            `top` largest z, weights sigmoid(z)
 //   prefill: moe_plan assigns every (token, choice) a slot; an expert's slots are consecutive and start at a multiple of
 //            128, so a 128-row tile of the grouped GEMM belongs to one expert (tile_group); moe_gather copies the rows.
 //            Everything stays on the device: no counts are read back, grids are sized for the worst case. Units: relu^2,
-//            or silu(gate) * up with the rows of the two matrices in turns, so that a pair of columns is one output.
+//            or silu(gate) * up or its clamped form with the rows of the two matrices in turns, so that a pair of columns is one
+//            output. Where a token's weight belongs to what the expert reads, it goes in with the copy.
 //   decode:  a few rows: one warp per output element of the chosen experts, straight from the expert's weights.
 // The down projection leaves one row per slot; the residual join adds them up with their weights.
 #include <cooperative_groups.h>
@@ -25,8 +27,11 @@ namespace oslo {
 constexpr int MOE_TILE = 128;          // rows per grouped-GEMM tile
 constexpr int MOE_MAX_EXPERTS = 2048;
 
-// the `top` largest of z[0..E) (shared memory, overwritten), ties to the lower index; softmax over them. One warp.
-__device__ __forceinline__ void pick_top(float* z, int E, int top, int* idx, float* wgt, int lane) {
+enum { ROUTE_CHOSEN = 0, ROUTE_SCORED = 1, ROUTE_SIGMOID = 2 };   // softmax over the chosen; over all; sigmoids
+
+// the `top` largest of z[0..E) (shared memory, overwritten), ties to the lower index; softmax over them, or (sig) the sigmoid
+// of each. One warp.
+__device__ __forceinline__ void pick_top(float* z, int E, int top, int* idx, float* wgt, int lane, bool sig) {
   float first = 0.f, sum = 0.f;
   for (int j = 0; j < top; ++j) {
     float best = -CUDART_INF_F;
@@ -43,7 +48,7 @@ __device__ __forceinline__ void pick_top(float* z, int E, int top, int* idx, flo
     }
     if (at >= E) { at = 0; best = 0.f; }               // only NaN logits get here
     if (j == 0) first = best;
-    const float ex = expf(best - first);
+    const float ex = sig ? 1.0f / (1.0f + expf(-best)) : expf(best - first);
     sum += ex;
     if (lane == 0) {
       idx[j] = at;
@@ -52,7 +57,7 @@ __device__ __forceinline__ void pick_top(float* z, int E, int top, int* idx, flo
     }
     __syncwarp();
   }
-  if (lane == 0) {
+  if (lane == 0 && !sig) {
     const float inv = 1.0f / sum;
     for (int j = 0; j < top; ++j) wgt[j] *= inv;
   }
@@ -115,7 +120,7 @@ template <typename T, int VEC>
 __global__ void __cluster_dims__(RT_CLUSTER, 1, 1) __launch_bounds__(256)
 route_kernel(const T* __restrict__ h, long long ldh, const T* __restrict__ w, const T* __restrict__ bias, int* __restrict__ idx,
              float* __restrict__ wgt, int E, int K, int top, int scored) {
-  extern __shared__ float z[];         // [E] (scored: and [E] of work space), used in the first block
+  extern __shared__ float z[];         // [E] (ROUTE_SCORED: and [E] of work space), used in the first block
   cg::cluster_group cluster = cg::this_cluster();
   const int rank = static_cast<int>(cluster.block_rank());
   float* z0 = cluster.map_shared_rank(z, 0);
@@ -134,12 +139,12 @@ route_kernel(const T* __restrict__ h, long long ldh, const T* __restrict__ w, co
       for (int i = 0; i < VEC; ++i) acc = fmaf(a[i], b[i], acc);
     }
     acc = warp_sum(acc);
-    if (lane == 0) z0[e] = scored ? acc : acc + Num<T>::to(bias[e]);
+    if (lane == 0) z0[e] = bias == nullptr || scored == ROUTE_SCORED ? acc : acc + Num<T>::to(bias[e]);
   }
   cluster.sync();                      // also keeps the first block's shared memory alive until all have written
   if (rank == 0 && threadIdx.x < 32) {
-    if (scored) pick_scored<T>(z, z + E, bias, E, top, idx + row * top, wgt + row * top, lane);
-    else pick_top(z, E, top, idx + row * top, wgt + row * top, lane);
+    if (scored == ROUTE_SCORED) pick_scored<T>(z, z + E, bias, E, top, idx + row * top, wgt + row * top, lane);
+    else pick_top(z, E, top, idx + row * top, wgt + row * top, lane, scored == ROUTE_SIGMOID);
   }
 }
 
@@ -152,11 +157,12 @@ __global__ void __launch_bounds__(128) route_logits_kernel(const float* __restri
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const long long row = static_cast<long long>(blockIdx.x) * 4 + warp;
   if (row >= rows) return;
-  float* z = rl_smem + warp * E * (scored ? 2 : 1);
-  for (int e = lane; e < E; e += 32) z[e] = scored ? logits[row * ldl + e] : logits[row * ldl + e] + Num<T>::to(bias[e]);
+  float* z = rl_smem + warp * E * (scored == ROUTE_SCORED ? 2 : 1);
+  const bool add = bias != nullptr && scored != ROUTE_SCORED;
+  for (int e = lane; e < E; e += 32) z[e] = add ? logits[row * ldl + e] + Num<T>::to(bias[e]) : logits[row * ldl + e];
   __syncwarp();
-  if (scored) pick_scored<T>(z, z + E, bias, E, top, idx + row * top, wgt + row * top, lane);
-  else pick_top(z, E, top, idx + row * top, wgt + row * top, lane);
+  if (scored == ROUTE_SCORED) pick_scored<T>(z, z + E, bias, E, top, idx + row * top, wgt + row * top, lane);
+  else pick_top(z, E, top, idx + row * top, wgt + row * top, lane, scored == ROUTE_SIGMOID);
 }
 
 // counts per expert -> start slot of every expert (multiple of MOE_TILE), expert of every tile, number of tiles
@@ -189,11 +195,11 @@ __global__ void __launch_bounds__(1024) moe_plan_kernel(const int* __restrict__ 
   }
 }
 
-// one block per (token, choice): take the next slot of its expert and copy the token's row there
+// one block per (token, choice): take the next slot of its expert and copy the token's row there, times `scale` [pairs] if given
 template <typename T, int VEC>
 __global__ void __launch_bounds__(128) moe_gather_kernel(const T* __restrict__ h, long long ldh, const int* __restrict__ idx,
                                                          int* __restrict__ cursor, int* __restrict__ slots, T* __restrict__ out,
-                                                         int K, int top, int max_slots, int E) {
+                                                         const float* __restrict__ scale, int K, int top, int max_slots, int E) {
   __shared__ int slot_s;
   const long long pair = blockIdx.x;
   if (idx[pair] >= E) {                                // no expert, no slot
@@ -209,17 +215,35 @@ __global__ void __launch_bounds__(128) moe_gather_kernel(const T* __restrict__ h
   if (slot >= max_slots) return;
   const T* src = h + pair / top * ldh;
   T* dst = out + static_cast<long long>(slot) * K;
+  if (scale != nullptr) {
+    const float f = scale[pair];
+    for (int k = threadIdx.x * VEC; k < K; k += blockDim.x * VEC) {
+      float v[VEC];
+      load_vec<T, VEC>(src + k, v);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) v[i] *= f;
+      store_vec<T, VEC>(dst + k, v);
+    }
+    return;
+  }
   for (int k = threadIdx.x * VEC; k < K; k += blockDim.x * VEC)
     *reinterpret_cast<Pack<T, VEC>*>(dst + k) = *reinterpret_cast<const Pack<T, VEC>*>(src + k);
 }
 
-enum { UNIT_NONE = 0, UNIT_RELU2 = 1, UNIT_GLU = 2 };   // GLU: columns in pairs (gate, up), half as many outputs
+// GLU, CLAMPED: columns in pairs (gate, up), half as many outputs
+enum { UNIT_NONE = 0, UNIT_RELU2 = 1, UNIT_GLU = 2, UNIT_CLAMPED = 3 };
+__device__ __forceinline__ float pair_unit(float g, float u, int unit, float limit, float alpha) {
+  if (unit == UNIT_GLU) return silu_f(g) * u;
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return g * sigmoid_f(alpha * g) * (u + 1.0f);
+}
 
 // scalar grouped product for types and sizes outside the tensor-core path: 32 x 64 outputs per block
 template <typename T>
 __global__ void __launch_bounds__(256) moe_grouped_kernel(const T* __restrict__ a, const T* __restrict__ w, T* __restrict__ out,
                                                           const int* __restrict__ tile_group, const int* __restrict__ n_tiles,
-                                                          int N, int K, int unit) {
+                                                          int N, int K, int unit, float limit, float alpha) {
   constexpr int BMS = 32, BNS = 64, BKS = 16;
   __shared__ float as[BKS][BMS + 1];
   __shared__ float bs[BKS][BNS + 1];
@@ -257,9 +281,10 @@ __global__ void __launch_bounds__(256) moe_grouped_kernel(const T* __restrict__ 
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx + 16 * j;
       float v = acc[i][j];
-      if (unit == UNIT_GLU) {                          // N is even: a pair of columns is in one pair of lanes
+      if (unit >= UNIT_GLU) {                          // N is even: a pair of columns is in one pair of lanes
         const float up = __shfl_xor_sync(0xffffffffu, v, 1);
-        if (n < N && (n & 1) == 0) out[static_cast<long long>(m0 + ty * 2 + i) * (N / 2) + n / 2] = Num<T>::from(silu_f(v) * up);
+        if (n < N && (n & 1) == 0)
+          out[static_cast<long long>(m0 + ty * 2 + i) * (N / 2) + n / 2] = Num<T>::from(pair_unit(v, up, unit, limit, alpha));
         continue;
       }
       if (n >= N) continue;
@@ -268,12 +293,13 @@ __global__ void __launch_bounds__(256) moe_grouped_kernel(const T* __restrict__ 
     }
 }
 
-// few rows: out[pair, n] = act(w[idx[pair]][n, :] . x[row of pair, :]); groups of `wg` warps share the k range of 4 outputs
+// few rows: out[pair, n] = act(w[idx[pair]][n, :] . x[row of pair, :] * scale[pair]); groups of `wg` warps share the k range of 4 outputs
 // and walk over the output groups, so that the chosen expert is looked up once per block
 template <typename T, int VEC>
 __global__ void __launch_bounds__(256, 4) moe_few_kernel(const T* __restrict__ x, long long ldx, const int* __restrict__ idx,
                                                          const T* __restrict__ w, T* __restrict__ out, int N, int K,
-                                                         int per_row, int unit, int wg, int E) {
+                                                         int per_row, int unit, int wg, int E, float limit, float alpha,
+                                                         const float* __restrict__ scale) {
   __shared__ float red[2][8][4];
   if (idx[blockIdx.y] >= E) return;                    // no expert: nobody reads the row
   const int pair = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -309,9 +335,11 @@ __global__ void __launch_bounds__(256, 4) moe_few_kernel(const T* __restrict__ x
       float s = 0.f;
       if (lane < nn)
         for (int g = 0; g < wg; ++g) s += r[warp + g][lane];
-      if (unit == UNIT_GLU) {
+      if (scale != nullptr) s *= scale[pair];
+      if (unit >= UNIT_GLU) {
         const float up = __shfl_xor_sync(0xffffffffu, s, 1);
-        if (lane < nn && (lane & 1) == 0) out[static_cast<long long>(pair) * (N / 2) + (n0 + lane) / 2] = Num<T>::from(silu_f(s) * up);
+        if (lane < nn && (lane & 1) == 0)
+          out[static_cast<long long>(pair) * (N / 2) + (n0 + lane) / 2] = Num<T>::from(pair_unit(s, up, unit, limit, alpha));
       } else if (lane < nn) {
         if (unit == UNIT_RELU2) { s = fmaxf(s, 0.f); s *= s; }
         out[static_cast<long long>(pair) * N + n0 + lane] = Num<T>::from(s);
@@ -325,9 +353,10 @@ __global__ void __launch_bounds__(256, 4) moe_few_kernel(const T* __restrict__ x
 extern "C" int oslo_moe_route(const void* h, long long ldh, const void* w, const void* bias, const float* logits, long long ldl,
                               int* idx, float* wgt, long long rows, int E, int K, int top, int scored, int dtype, cudaStream_t stream) {
   using namespace oslo;
-  const size_t per_row = (scored ? 2 : 1) * E * sizeof(float);
+  const size_t per_row = (scored == ROUTE_SCORED ? 2 : 1) * E * sizeof(float);
   if (rows <= 0) return 0;
   if (E <= 0 || E > MOE_MAX_EXPERTS || top <= 0 || top > E || rows > 0x7fffffffll) return -1;
+  if (scored < ROUTE_CHOSEN || scored > ROUTE_SIGMOID || (scored == ROUTE_SCORED && bias == nullptr)) return -1;
   const size_t te = dtype == OSLO_DT_FP32 ? 4 : 2;
   if (logits) {
     OSLO_DISPATCH_T(dtype, {
@@ -353,7 +382,7 @@ extern "C" int oslo_moe_route(const void* h, long long ldh, const void* w, const
 }
 
 extern "C" int oslo_moe_plan(const void* h, long long ldh, const int* idx, int* cursor, int* tile_group, int* n_tiles, int* slots,
-                             void* rows_out, long long pairs, int E, int K, int top, int max_tiles, int dtype,
+                             void* rows_out, const float* scale, long long pairs, int E, int K, int top, int max_tiles, int dtype,
                              cudaStream_t stream) {
   using namespace oslo;
   if (pairs <= 0) return 0;
@@ -366,32 +395,33 @@ extern "C" int oslo_moe_plan(const void* h, long long ldh, const int* idx, int* 
     constexpr int V = 16 / sizeof(T);
     if (vec)
       moe_gather_kernel<T, V><<<static_cast<unsigned>(pairs), 128, 0, stream>>>(
-          static_cast<const T*>(h), ldh, idx, cursor, slots, static_cast<T*>(rows_out), K, top, max_tiles * MOE_TILE, E);
+          static_cast<const T*>(h), ldh, idx, cursor, slots, static_cast<T*>(rows_out), scale, K, top, max_tiles * MOE_TILE, E);
     else
       moe_gather_kernel<T, 1><<<static_cast<unsigned>(pairs), 128, 0, stream>>>(
-          static_cast<const T*>(h), ldh, idx, cursor, slots, static_cast<T*>(rows_out), K, top, max_tiles * MOE_TILE, E);
+          static_cast<const T*>(h), ldh, idx, cursor, slots, static_cast<T*>(rows_out), scale, K, top, max_tiles * MOE_TILE, E);
   });
   return static_cast<int>(cudaGetLastError());
 }
 
 extern "C" int oslo_moe_grouped(const void* a, const void* w, void* out, const int* tile_group, const int* n_tiles,
-                                int max_tiles, int N, int K, int unit, int dtype, cudaStream_t stream) {
+                                int max_tiles, int N, int K, int unit, float limit, float alpha, int dtype, cudaStream_t stream) {
   using namespace oslo;
   if (max_tiles <= 0 || N <= 0) return 0;
-  if (unit == UNIT_GLU && N % 2) return -1;
+  if (unit >= UNIT_GLU && N % 2) return -1;
   if (static_cast<long long>(max_tiles) * (MOE_TILE / 32) > 65535) return -1;
   OSLO_DISPATCH_T(dtype, {
     moe_grouped_kernel<T><<<dim3((N + 63) / 64, max_tiles * (MOE_TILE / 32)), 256, 0, stream>>>(
-        static_cast<const T*>(a), static_cast<const T*>(w), static_cast<T*>(out), tile_group, n_tiles, N, K, unit);
+        static_cast<const T*>(a), static_cast<const T*>(w), static_cast<T*>(out), tile_group, n_tiles, N, K, unit, limit, alpha);
   });
   return static_cast<int>(cudaGetLastError());
 }
 
 extern "C" int oslo_moe_few(const void* x, long long ldx, const int* idx, const void* w, void* out, int pairs, int per_row,
-                            int N, int K, int unit, int E, int dtype, cudaStream_t stream) {
+                            int N, int K, int unit, float limit, float alpha, const float* scale, int E, int dtype,
+                            cudaStream_t stream) {
   using namespace oslo;
   if (pairs <= 0 || N <= 0) return 0;
-  if (pairs > 65535 || per_row < 1 || (unit == UNIT_GLU && N % 2)) return -1;
+  if (pairs > 65535 || per_row < 1 || (unit >= UNIT_GLU && N % 2)) return -1;
   const size_t te = dtype == OSLO_DT_FP32 ? 4 : 2;
   const int v = static_cast<int>(16 / te);
   const bool vec = K % v == 0 && ldx % v == 0 && aligned_to(w, 16) && aligned_to(x, 16);
@@ -404,10 +434,10 @@ extern "C" int oslo_moe_few(const void* x, long long ldx, const int* idx, const 
     constexpr int V = 16 / sizeof(T);
     if (vec)
       moe_few_kernel<T, V><<<grid, 256, 0, stream>>>(static_cast<const T*>(x), ldx, idx, static_cast<const T*>(w),
-                                                     static_cast<T*>(out), N, K, per_row, unit, wg, E);
+                                                     static_cast<T*>(out), N, K, per_row, unit, wg, E, limit, alpha, scale);
     else
       moe_few_kernel<T, 1><<<grid, 256, 0, stream>>>(static_cast<const T*>(x), ldx, idx, static_cast<const T*>(w),
-                                                     static_cast<T*>(out), N, K, per_row, unit, wg, E);
+                                                     static_cast<T*>(out), N, K, per_row, unit, wg, E, limit, alpha, scale);
   });
   return static_cast<int>(cudaGetLastError());
 }

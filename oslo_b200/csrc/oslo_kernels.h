@@ -17,6 +17,7 @@
                                   // (max, sum exp(x - max), logit of the row's label if it lies in the block)
 #define GEMM_FLAG_CE_GRAD 512     // LM head + cross-entropy, backward: D = (exp(x - lse[row]) - [col == label]) * scale[row]
 #define GEMM_FLAG_RELU2 1024      // square of relu
+#define OSLO_ACT_RELU2 (-2)       // `gelu_from` of the few-row products: square of relu on all columns
 #define GEMM_FLAG_GLU 2048        // columns in pairs (gate, up): silu(gate) * up, half as many output columns; N is even, ldd >= N / 2
 #define GEMM_CE_BLOCK 128         // columns per statistics record
 
@@ -129,6 +130,12 @@ int oslo_flash_sink_fwd_sm100(const void* q, const void* k, const void* v, void*
                               float scale, float softcap, int window, int keep_first, const int* lead, int gate_wide,
                               const void* q2, long long q2_sb, long long q2_sh, long long q2_ss, const void* k2, long long k2_sb,
                               long long k2_ss, int rot, int dtype, int* err_word, cudaStream_t stream);
+// the same with one key head of any width for all query heads, k [B, Sk, dim], and value heads per group
+int oslo_flash_wide_fwd_sm100(const void* q, const void* k, const void* v, void* o, const uint8_t* kpm, const void* sink,
+                              const void* gate, long long ldg, int gate_wide, int B, int H, int G, int Sq, int Sk, int dim, int vdim,
+                              long long q_sb, long long q_sh, long long q_ss, long long k_sb, long long k_ss, long long v_sb,
+                              long long v_sh, long long v_ss, long long o_sb, long long o_sh, long long o_ss, float scale, int window,
+                              int keep_first, const int* lead, int dtype, int* err_word, cudaStream_t stream);
 int oslo_flash_bwd(const void* q, const void* k, const void* v, const void* o, const void* dout, const float* lse,
                    float* delta, float* dq_acc, void* dq, void* dk, void* dv, const uint8_t* kpm, int B, int H,
                    int Sq, int Sk, int D, long long q_sb, long long q_sh, long long q_ss, long long k_sb,
@@ -210,8 +217,9 @@ int oslo_allreduce_oneshot(const void* in, void* out, void* const* peer_ptrs_dev
                            long long half_bytes, int rank, int world, int dtype, int use_multimem, int* err_word,
                            cudaStream_t stream);
 
-// RMS norms and the residual join (rms_norm.cu). x is fp32 when x_fp32, else the storage type; rows have strides
-int oslo_rms_norm(const void* x, long long ldx, int x_fp32, const void* w, void* out, long long ldo, long long rows, int cols,
+// RMS norms and the residual join (rms_norm.cu). x is fp32 when x_fp32, else the storage type; rows have strides;
+// one: the weight is one number
+int oslo_rms_norm(const void* x, long long ldx, int x_fp32, const void* w, int one, void* out, long long ldo, long long rows, int cols,
                   float eps, float offset, int dtype, cudaStream_t stream);
 // x_out = x + rms(y * sigmoid(gate + gate_bias)) * (1 + w_post); h_out = rms(x_out) * (1 + w_next) unless w_next is null.
 // slot_weights null: y has one row per token, else y = sum_j slot_weights[t, j] * y[slots[t, j]] (slots null: t * top + j)
@@ -223,10 +231,22 @@ int oslo_silu_mul(const void* gate, long long ldg, const void* up, long long ldu
 // g sigmoid(alpha g) (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit)
 int oslo_clamped_glu(const void* gate, long long ldg, const void* up, long long ldu, void* out, long long rows, int cols,
                      float limit, float alpha, int dtype, cudaStream_t stream);
-// x_out = x + mult * sum_i factor[i] * (w[i] ? rms(y[i]) * w[i] : y[i]), n <= 3; h1 = rms(x_out) * w1, h2 = rms(x_out) * w2 (or null)
-int oslo_branch_join(const float* x, int n, const void* const* y, const long long* ldy, const void* const* w, const float* factor,
-                     float mult, float eps, const void* w1, const void* w2, float* x_out, void* h1, void* h2, long long rows,
-                     int cols, int dtype, cudaStream_t stream);
+// x_out = x + mult * sum_i factor[i] * b_i, i < n <= 3, with b_i = y[i], rms(y[i]) * w[i] (normed) or y[i] * w[i]; top[i] > 0: y[i] of a
+// row is the sum of the rows slots[i][row, j] (null: row * top + j), j < top. h1 = rms(x_out) * w1, h2 = rms(x_out) * w2 (w2 or both null:
+// not written; one1, one2: the weight is one number); copy (w1 null): h1 = x_out. conv_w [cols, taps] (rows are single tokens):
+// conv_out = h1 + the causal convolution of prev fp32 [rows, taps - 1, cols] and h1, prev moves on (null: zeros); keep 0: h1 counts as 0
+struct OsloBranchJoin {
+  const float* x; int n;
+  const void* y[3]; long long ldy[3]; const void* w[3]; int normed[3]; const int* slots[3]; int top[3]; float factor[3];
+  float mult, eps;
+  const void *w1, *w2; int one1, one2, copy;
+  float* x_out; void *h1, *h2;
+  const void* conv_w; float* prev; int taps; const uint8_t* keep; long long ld_keep; void* conv_out;
+};
+int oslo_branch_join(const struct OsloBranchJoin* a, long long rows, int cols, int dtype, cudaStream_t stream);
+// out [rows, cols] = gelu_tanh(z) * table[ids[row * id_step], first + column]
+int oslo_token_gate(const void* z, long long ldz, const long long* ids, long long id_step, const void* table, long long ldt,
+                    long long vocab, int first, void* out, long long rows, int cols, int dtype, int* err_word, cudaStream_t stream);
 // out = o / rms(runs of `group` columns) * w * act(gate); act 0: sigmoid, 1: silu; o fp32 [rows, cols]
 // z, m [rows, cols / group] (or null): the runs are first divided by max(|z|, exp(-m)) + 1e-6
 int oslo_gated_rms_norm(const float* o, const void* w, const void* gate, long long ldg, void* out, const float* z, const float* m,
@@ -285,12 +305,12 @@ int oslo_memory_step(const void* q, long long ldq, const void* k, long long ldk,
 // latent attention (latent_attention.cu). sink_gate: flash output [B, S, H, *] + lse [B, H, S] -> out [B * S, H * vdim]
 int oslo_sink_gate(const void* o, long long o_sb, long long o_ss, long long o_sh, const float* lse, const void* sink,
                    const void* gate, long long ldg, void* out, int B, int S, int H, int vdim, int dtype, cudaStream_t stream);
-// causal attention with sink and output gate (or null) in 32-bit, any head sizes; strides of (batch, position, head); G key /
+// causal attention with sink and output gate (or null) in 32-bit, any head sizes; strides of (batch, position, head); KG key and G
 // value heads; softcap > 0: scores become softcap * tanh(score / softcap)
 int oslo_sink_attention(const void* q, long long q_sb, long long q_ss, long long q_sh, const void* k, long long k_sb,
                         long long k_ss, long long k_sh, const void* v, long long v_sb, long long v_ss, long long v_sh,
                         const uint8_t* keep, long long ld_keep, const void* sink, const void* gate, long long ldg, void* out,
-                        int B, int H, int G, int Sq, int Sk, int dim, int vdim, float scale, float softcap, int window,
+                        int B, int H, int G, int KG, int Sq, int Sk, int dim, int vdim, float scale, float softcap, int window,
                         int keep_first, const int* lead, int gate_wide, int dtype, cudaStream_t stream);
 // rows b * S + t: RMS norm of the query latent -> cq_out; of the key-value latent (null: none) -> cache [B, Tmax, kv_rank + rot] at
 // lengths[b] + t, followed by the rot columns after it, rotated (halves) by pos[b, t] * freq; c_out (null: none) [B * S, kv_rank]
@@ -319,22 +339,31 @@ int oslo_qkv_prep(const void* q, long long ldq, const void* k, long long ldk, co
                   const void* wk, float eps, const long long* pos, long long pos_sb, long long pos_ss, const float* freq, int n_freq,
                   void* q_out, void* kc, void* vc, const int* lengths, int B, int S, int H, int G, int dim, int vdim, int Tmax,
                   int dtype, int* err_word, cudaStream_t stream);
+// the same with interleaved pairs or (halves) dims i and i + n_freq, sines and cosines times amplitude; caches by strides of (batch,
+// head, position); talk [H, H] or null: the queries of mixed scores for keys of all heads in a row, q_out [B, S, H, G * dim]
+int oslo_head_prep(const void* q, long long ldq, const void* k, long long ldk, const void* v, long long ldv, const void* wq,
+                   const void* wk, float eps, const long long* pos, long long pos_sb, long long pos_ss, const float* freq, int n_freq,
+                   int halves, float amplitude, const void* talk, void* q_out, void* kc, long long k_sb, long long k_sg, long long k_st,
+                   void* vc, long long v_sb, long long v_sg, long long v_st, const int* lengths, int B, int S, int H, int G, int dim,
+                   int vdim, int Tmax, int num_sms, int dtype, int* err_word, cudaStream_t stream);
 // one query per row: q [B, H, dim], caches [B, G, Tmax, *], of which lengths[b] positions count; keep [B, n_keep] (0 = padded) or
-// null; sink null: none; gate null or [B, H]; window > 0: the last `window` positions and the first keep_first after lead[b] (null: 0)
+// null; sink null: none; gate null, [B, H] or (gate_wide) [B, H * vdim / VG]; VG > 1 (G = 1): a cached value row holds VG value heads
+// side by side and a query head's result is that of its own; window > 0: the last `window` positions and the first keep_first after lead[b] (null: 0)
 // are read; fp32 workspaces ws [B, H, splits, vdim rounded up to a multiple of 4] and stat [B, H, splits, 2]; out [B, H * vdim]
-int oslo_grouped_splits(int B, int H, int G, int T, int dim, int vdim, int dtype, int num_sms);
+int oslo_grouped_splits(int B, int H, int G, int VG, int T, int dim, int vdim, int dtype, int num_sms);
+int oslo_wide_decode_fits(int H, int VG, int dim, int vdim, int dtype);
 int oslo_grouped_decode(const void* q, const void* kc, const void* vc, const int* lengths, const uint8_t* keep, long long ld_keep,
-                        int n_keep, const void* sink, const void* gate, long long ldg, int window, int keep_first, const int* lead,
-                        float* ws, float* stat, void* out, int B, int H, int G, int dim, int vdim, int Tmax, int splits,
-                        float scale, float softcap, int dtype, int* err_word, cudaStream_t stream);
+                        int n_keep, const void* sink, const void* gate, long long ldg, int gate_wide, int window, int keep_first,
+                        const int* lead, float* ws, float* stat, void* out, int B, int H, int G, int VG, int dim, int vdim, int Tmax,
+                        int splits, float scale, float softcap, int dtype, int* err_word, cudaStream_t stream);
 
 // token shift, causal convolution and selective scan (selective_scan.cu)
 // out[i] = h + (h' - h) * mu[i], i < P; prev fp32 [B, width] (the row before the first; read and updated) or null
 int oslo_token_shift(const void* h, long long ldh, const void* mu, const uint8_t* keep, long long ld_keep, float* prev, void* out,
                      int B, int S, int width, int P, int dtype, cudaStream_t stream);
-// out [B * S, C] = silu(conv(x) + bias); prev fp32 [B, taps - 1, C] (read and updated) or null
-int oslo_causal_conv_silu(const void* x, long long ldx, const void* w, const void* bias, const uint8_t* keep, long long ld_keep,
-                          float* prev, void* out, int B, int S, int C, int taps, int dtype, cudaStream_t stream);
+// out [B * S, C] = y = conv(x) + bias (or null), silu(y) or y + x; prev fp32 [B, taps - 1, C] (read and updated) or null
+int oslo_causal_conv(const void* x, long long ldx, const void* w, const void* bias, const uint8_t* keep, long long ld_keep, float* prev,
+                     void* out, int B, int S, int C, int taps, int silu, int residual, int dtype, cudaStream_t stream);
 // dt fp32 logits [B * S, C]; state fp32 [B, C, N] (read and updated) or null; out [B * S, C]. nchunks > 1 (oslo_scan_chunks) needs
 // ws [B, nchunks, C, N] and steps [B, nchunks, C] fp32
 int oslo_scan_chunks(int B, int S, int C, int N, int num_sms);
@@ -349,19 +378,21 @@ int oslo_scan_step(const void* x, long long ldx, const void* dt, long long lddt,
                    cudaStream_t stream);
 
 // mixture of experts (moe.cu, grouped GEMM in gemm_sm100.cu)
-// route: idx, wgt [rows, top]; scored: scores are the softmax over all E outputs, bias only enters the choice, weights are the chosen
-// scores over their sum. Choices >= the experts of plan / few get no slot (-1) and no product. unit: 0 none, 1 relu^2, 2 silu(gate) *
-// up of column pairs (out has N / 2 columns)
+// route: idx, wgt [rows, top]; scored 1: scores are the softmax over all E outputs, bias only enters the choice, weights are the chosen
+// scores over their sum; 2: the weights are the sigmoids of the largest logits; bias null: none. Choices >= the experts of plan / few
+// get no slot (-1) and no product. unit: 0 none, 1 relu^2, 2 silu(gate) * up of column pairs (out has N / 2 columns), 3 the clamped
+// form of that (limit, alpha). scale [pairs] (or null) multiplies what an expert reads
 int oslo_moe_route(const void* h, long long ldh, const void* w, const void* bias, const float* logits, long long ldl, int* idx,
                    float* wgt, long long rows, int E, int K, int top, int scored, int dtype, cudaStream_t stream);
-int oslo_moe_plan(const void* h, long long ldh, const int* idx, int* cursor, int* tile_group, int* n_tiles, int* slots,
-                  void* rows_out, long long pairs, int E, int K, int top, int max_tiles, int dtype, cudaStream_t stream);
+int oslo_moe_plan(const void* h, long long ldh, const int* idx, int* cursor, int* tile_group, int* n_tiles, int* slots, void* rows_out,
+                  const float* scale, long long pairs, int E, int K, int top, int max_tiles, int dtype, cudaStream_t stream);
 int oslo_moe_grouped(const void* a, const void* w, void* out, const int* tile_group, const int* n_tiles, int max_tiles, int N,
-                     int K, int unit, int dtype, cudaStream_t stream);
+                     int K, int unit, float limit, float alpha, int dtype, cudaStream_t stream);
 int oslo_moe_few(const void* x, long long ldx, const int* idx, const void* w, void* out, int pairs, int per_row, int N, int K,
-                 int unit, int E, int dtype, cudaStream_t stream);
+                 int unit, float limit, float alpha, const float* scale, int E, int dtype, cudaStream_t stream);
 int oslo_gemm_grouped(const void* A, const void* B, void* D, int M, int N, int K, int groups, const int* group_of_tile,
-                      const int* group_tiles, int flags, int* err_word, int num_sms, cudaStream_t stream);
+                      const int* group_tiles, int flags, int glu_clamped, float glu_limit, float glu_alpha, int* err_word, int num_sms,
+                      cudaStream_t stream);
 
 #ifdef __cplusplus
 }

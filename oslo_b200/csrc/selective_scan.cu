@@ -1,7 +1,7 @@
 // Token shift, causal convolution per channel and selective scan (Mamba form), arithmetic and states in 32-bit floats.
 //
 //   token shift:  out_i = h_t + (h_{t-1} - h_t) * mu_i           h_{-1}: the state (zero for a new sequence)
-//   convolution:  y_t = silu(bias + sum_j w_j x_{t - taps + 1 + j})
+//   convolution:  y_t = bias + sum_j w_j x_{t - taps + 1 + j}, then silu(y_t), or y_t + x_t, or as it is
 //   scan:         s_t = softplus(dt_t + dt_bias),  S[n] <- exp(s_t A[n]) S[n] + s_t x_t B_t[n],  A = -exp(a_log)
 //                 out_t = (sum_n S[n] C_t[n] + d x_t) * silu(z_t)
 //
@@ -80,11 +80,12 @@ __global__ void __launch_bounds__(128) token_shift_kernel(const ShiftParams p) {
 // ------------------------------------------------------------------ causal convolution
 struct ConvParams {
   const void* x; long long ldx;
-  const void *w, *bias;                      // [C, taps], [C]
+  const void *w, *bias;                      // [C, taps], [C] or nullptr
   const uint8_t* keep; long long ld_keep;
   float* prev;                               // [B, taps - 1, C] or nullptr
   void* out;                                 // [B * S, C]
   int S, C, taps, run;                       // run: tokens per thread, at least taps
+  int silu, residual;
 };
 
 // TAPS 0: any number of taps, the window is read again for every token
@@ -110,8 +111,15 @@ __global__ void __launch_bounds__(128) causal_conv_kernel(const ConvParams p) {
     }
   };
   float bias[VEC];
-  load_vec<T, VEC>(static_cast<const T*>(p.bias) + c, bias);
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) bias[i] = 0.f;
+  if (p.bias != nullptr) load_vec<T, VEC>(static_cast<const T*>(p.bias) + c, bias);
   T* out = static_cast<T*>(p.out) + static_cast<long long>(b) * p.S * p.C + c;
+  auto finish = [&](float y, float x) {
+    if (p.residual) return y + x;
+    if (!p.silu) return y;
+    return sizeof(T) == 4 ? silu_f(y) : y * __fdividef(1.0f, 1.0f + __expf(-y));
+  };
   if constexpr (TAPS > 0) {
     float wr[TAPS][VEC], win[TAPS][VEC];
 #pragma unroll
@@ -140,24 +148,23 @@ __global__ void __launch_bounds__(128) causal_conv_kernel(const ConvParams p) {
           y[i] = bias[i];
 #pragma unroll
           for (int j = 0; j < TAPS; ++j) y[i] = fmaf(wr[j][i], win[j][i], y[i]);
-          y[i] = sizeof(T) == 4 ? silu_f(y[i]) : y[i] * __fdividef(1.0f, 1.0f + __expf(-y[i]));
+          y[i] = finish(y[i], now[a][i]);
         }
         store_vec<T, VEC>(out + static_cast<long long>(tb + a) * p.C, y);
       }
     }
   } else {
     for (int t = t0; t < t1; ++t) {
-      float y[VEC];
+      float y[VEC], v[VEC];
 #pragma unroll
       for (int i = 0; i < VEC; ++i) y[i] = bias[i];
-      for (int j = 0; j < taps; ++j) {
-        float v[VEC];
+      for (int j = 0; j < taps; ++j) {                 // the last one leaves the token's own input in v
         input(t - taps + 1 + j, v);
 #pragma unroll
         for (int i = 0; i < VEC; ++i) y[i] = fmaf(Num<T>::to(w[i * taps + j]), v[i], y[i]);
       }
 #pragma unroll
-      for (int i = 0; i < VEC; ++i) y[i] = silu_f(y[i]);
+      for (int i = 0; i < VEC; ++i) y[i] = finish(y[i], v[i]);
       store_vec<T, VEC>(out + static_cast<long long>(t) * p.C, y);
     }
   }
@@ -616,13 +623,13 @@ extern "C" int oslo_token_shift(const void* h, long long ldh, const void* mu, co
   return static_cast<int>(cudaGetLastError());
 }
 
-extern "C" int oslo_causal_conv_silu(const void* x, long long ldx, const void* w, const void* bias, const uint8_t* keep,
-                                     long long ld_keep, float* prev, void* out, int B, int S, int C, int taps, int dtype,
-                                     cudaStream_t stream) {
+extern "C" int oslo_causal_conv(const void* x, long long ldx, const void* w, const void* bias, const uint8_t* keep,
+                                long long ld_keep, float* prev, void* out, int B, int S, int C, int taps, int silu, int residual,
+                                int dtype, cudaStream_t stream) {
   using namespace oslo;
   if (B <= 0 || S <= 0 || C <= 0) return 0;
-  if (taps < 1) return -1;
-  ConvParams p{x, ldx, w, bias, keep, ld_keep, prev, out, S, C, taps, std::max(16, taps)};
+  if (taps < 1 || (silu && residual)) return -1;
+  ConvParams p{x, ldx, w, bias, keep, ld_keep, prev, out, S, C, taps, std::max(16, taps), silu, residual};
   const int runs = (S + p.run - 1) / p.run;
   if (B > 65535 || runs > 65535) return -1;
   const size_t te = dtype == OSLO_DT_FP32 ? 4 : 2;

@@ -23,10 +23,11 @@ from torch.utils.checkpoint import checkpoint
 
 from ... import ops
 from ...modeling_utils import PretrainedConfig, PreTrainedModel
+from ...ops.reference import Branch
 from ...parallel.layers import Embedding, Linear, RMSNorm
 from ...parallel.mpu import Layer, LayerPolicy
 from ..common import CausalLMHeadMixin, DecoderBackbone, SequenceClassificationMixin, StaticKVCache
-from ..mixers import BonusRecurrence, Branch, GatedMLP, SelectiveScan, SideBySide
+from ..mixers import BonusRecurrence, GatedMLP, SelectiveScan, SideBySide
 
 _MIXER_KEYS = {
     "parallel.left": ("heads", "kv_heads", "dim", "vdim", "scale"),

@@ -102,7 +102,7 @@ def _mixer(kind: str, m: Dict[str, Any], width: int, eps: float) -> nn.Module:
     if kind == "attention":
         return GroupedQueryAttention(width, m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["scale"], eps, rot_dims=m["rot"]["dims"],
                                      rot_base=m["rot"]["base"], norm_weights=False, sink=False, window=m["mask"]["size"],
-                                     keep_first=m["mask"]["keep_first"], value_is_key=True, gate=True)
+                                     keep_first=m["mask"]["keep_first"], value_is_key=True, gate="head")
     if kind == "latent_attention":
         return LatentAttention(width, m["heads"], m["dim"], m["vdim"], m["q_rank"], m["kv_rank"], m["scale"], eps, rot_dim=m["rot_dim"],
                                rot_base=m["rot"]["base"], sink=False, gate="element")

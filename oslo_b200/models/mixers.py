@@ -1,7 +1,8 @@
 """Token mixers and feed-forwards that are not tied to one model family: latent attention (with or without a sink and a rotated
-part), grouped-query attention with query / key norms, capped scores, windows and gates, gated linear recurrence (HGRN2),
+part), grouped-query attention with query / key norms, capped or mixed scores, windows and gates, gated linear recurrence (HGRN2),
 linear attention with constant decays, linear recurrence with a bonus (WKV), matrix memory (mLSTM), selective scan (Mamba), two
-mixers side by side; gated MLPs, mixtures of experts; residual streams with hyper-connections.
+mixers side by side; dense and gated MLPs, mixtures of experts; causal convolutions of a mixer's input, per-token inputs of a layer; residual
+streams with hyper-connections.
 
 They take their sizes and constants as arguments and work on token rows ``[batch * positions, width]``. A mixer or
 feed-forward can carry ``side`` projections: further linear maps of the same input (a block's residual gate, say) that
@@ -19,15 +20,9 @@ import torch.nn as nn
 from torch import Tensor
 
 from .. import ops
+from ..ops.reference import Branch
 from ..parallel.layers import Linear, PackedLinear, RMSNorm, StackedLinear
 from .common import StaticKVCache
-
-
-class Branch(NamedTuple):
-    """A result on its way to the residual stream: ``factor * y``, or ``factor * norm(y) * norm_weight``."""
-    y: Tensor                              # [rows, width]
-    norm_weight: Optional[Tensor] = None
-    factor: float = 1.0
 
 
 class MixerOutput(NamedTuple):
@@ -221,34 +216,42 @@ class GroupedQueryAttention(nn.Module, _Constants):
     """Causal softmax attention with ``heads`` query heads over ``kv_heads`` key / value heads.
 
     Queries and keys are RMS-normed per head (weights ``[dim]``, shared by the heads; ``norm_weights=False``: without weights), then
-    the first ``rot_dims`` dims are rotated (interleaved pairs, ``rot_base``); scores ``(q . k) * scale`` pass through ``softcap *
-    tanh(score / softcap)`` (0: they do not). With ``sink`` the softmax denominator holds an additional 1 (a sink with score 0). With a
-    ``window`` > 0 a position reads the last ``window`` positions and the first ``keep_first`` of the sequence. ``value_is_key``: values
-    are the projected keys, before norm and rotation. ``gate``: head ``h``'s output is multiplied by ``sigmoid(W_g x)[h]``. Keys (after
-    norm and rotation) and values are cached. ``in_proj=False``: the projections come from the caller's packed GEMM (``parts``)."""
+    the first ``rot_dims`` dims are rotated (interleaved pairs, or ``halves``: dim ``i`` with dim ``i + rot_dims / 2``; ``rot_base``, YaRN
+    ``rot_scaling``); scores ``(q . k) * scale`` pass through ``softcap * tanh(score / softcap)`` (0: they do not). With ``sink`` the softmax
+    denominator holds an additional 1 (a sink with score 0). With a ``window`` > 0 a position reads the last ``window`` positions and the
+    first ``keep_first`` of the sequence. ``value_is_key``: values are the projected keys, before norm and rotation. ``gate``: ``"head"``
+    (head ``h``'s output is multiplied by ``sigmoid(W_g x)[h]``), ``"element"`` (one factor per element) or ``None``. ``talk``: before the
+    softmax the heads' scores are mixed, ``score_h <- sum_g talk[h, g] score_g``; the mix is folded into the queries
+    (``reference.norm_rotate_fold``) and the keys of all key heads are cached as one row per token. Keys (after norm and rotation)
+    and values are cached. ``in_proj=False``: the projections come from the caller's packed GEMM (``parts``)."""
 
     oslo_fused = False
 
     def __init__(self, width: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, eps: float, rot_dims: int = 0,
                  rot_base: float = 10000.0, softcap: float = 0.0, in_proj: bool = True, norm_weights: bool = True, sink: bool = True,
-                 window: int = 0, keep_first: int = 0, value_is_key: bool = False, gate: bool = False) -> None:
+                 window: int = 0, keep_first: int = 0, value_is_key: bool = False, gate: Optional[str] = None, halves: bool = False,
+                 rot_scaling: Optional[Dict[str, float]] = None, talk: bool = False) -> None:
         super().__init__()
         if heads % kv_heads:
             raise ValueError(f"{heads} query heads do not divide into {kv_heads} groups")
         if value_is_key and vdim != dim:
             raise ValueError(f"values are the keys, but have size {vdim} and not {dim}")
+        if gate not in (None, "head", "element"):
+            raise ValueError(f"output gate per {gate!r}")
         self.heads, self.kv_heads, self.dim, self.vdim, self.eps = heads, kv_heads, dim, vdim, float(eps)
         self.scale, self.softcap = float(scale), float(softcap)
         self.sink, self.window, self.keep_first = bool(sink), int(window), int(keep_first)
-        self.frequencies = ops.reference.rotary_frequencies(rot_dims, rot_base)
+        self.frequencies = ops.reference.rotary_frequencies(rot_dims, rot_base, rot_scaling)
+        self.halves, self.amplitude = bool(halves), ops.reference.rotary_amplitude(rot_scaling)
         self.parts = {"q": heads * dim, "k": kv_heads * dim}
         if not value_is_key:
             self.parts["v"] = kv_heads * vdim
-        if gate:
-            self.parts["g"] = heads
+        if gate is not None:
+            self.parts["g"] = heads if gate == "head" else heads * vdim
         self.in_proj = PackedLinear(width, self.parts) if in_proj else None
         self.q_norm = RMSNorm(dim, eps) if norm_weights else None
         self.k_norm = RMSNorm(dim, eps) if norm_weights else None
+        self.talk = nn.Parameter(torch.eye(heads)) if talk else None
         self.out_proj = Linear(heads * vdim, width, bias=False)
 
     def forward(self, h: Tensor, batch: int, layer_id: int, cache: Optional[StaticKVCache], keep: Optional[Tensor],
@@ -268,17 +271,29 @@ class GroupedQueryAttention(nn.Module, _Constants):
         if (self.oslo_fused and not output_attentions and _inference(p["q"], self.out_proj.weight) and ops.use_kernels(p["q"])):
             o = self._kernels(p, values, batch, s, layer_id, cache, keep, positions, freq, sink, gate, mask)
             return MixerOutput(self.out_proj(o), {})
-        q = ops.reference.norm_rotate(p["q"].reshape(batch, s, self.heads, self.dim), wq, self.eps, positions, freq)
-        k = ops.reference.norm_rotate(p["k"].reshape(batch, s, self.kv_heads, self.dim), wk, self.eps, positions, freq)
+        q, turn = p["q"].reshape(batch, s, self.heads, self.dim), (self.halves, self.amplitude)
+        if self.talk is None:
+            q = ops.reference.norm_rotate(q, wq, self.eps, positions, freq, *turn)
+        else:
+            q = ops.reference.norm_rotate_fold(q, wq, self.eps, positions, freq, self.talk, self.kv_heads, *turn)
+        k = ops.reference.norm_rotate(p["k"].reshape(batch, s, self.kv_heads, self.dim), wk, self.eps, positions, freq, *turn)
         v = values.reshape(batch, s, self.kv_heads, self.vdim)
+        if self.talk is not None:
+            k = k.flatten(2).unsqueeze(2)
         if cache is not None:
-            k, v, end = cache.append(layer_id, k.transpose(1, 2), v.transpose(1, 2))
+            kc, vc = (k, v) if self.talk is None else (k, v.flatten(2).unsqueeze(2))
+            k, v, end = cache.append(layer_id, kc.transpose(1, 2), vc.transpose(1, 2))
+            v = v if self.talk is None else self._heads(v, self.vdim)
             if s == 1 and not output_attentions:
                 o = ops.reference.grouped_decode(q[:, 0], k, v, cache.lengths_next, keep, sink, self.scale, self.softcap, gate, *mask)
                 return MixerOutput(self.out_proj(o), {})
             k, v = k[:, :, :end].transpose(1, 2), v[:, :, :end].transpose(1, 2)
         o, probs = ops.reference.sink_attention(q, k, v, keep, sink, gate, self.scale, self.softcap, *mask)
         return MixerOutput(self.out_proj(o), {}, probs=probs if output_attentions else None)
+
+    def _heads(self, store: Tensor, dim: int) -> Tensor:
+        """A cache with all key heads in a row, ``[B, 1, T, kv_heads * dim]``, as ``[B, kv_heads, T, dim]`` (a view)."""
+        return store.view(store.size(0), store.size(2), self.kv_heads, dim).transpose(1, 2)
 
     def _sink(self, like: Tensor) -> Optional[Tensor]:
         if not self.sink:
@@ -294,9 +309,17 @@ class GroupedQueryAttention(nn.Module, _Constants):
         from ..ops import cuda_ops
         q = p["q"]
         holder = cache if cache is not None else StaticKVCache(s)
-        ks, vs = holder.kv_storage(layer_id, batch, self.kv_heads, self.dim, self.vdim, q.dtype, q.device, s)
+        wide = self.talk is not None
+        sizes = (1, self.kv_heads * self.dim, self.kv_heads * self.vdim) if wide else (self.kv_heads, self.dim, self.vdim)
+        ks, vs = holder.kv_storage(layer_id, batch, *sizes, q.dtype, q.device, s)
         wq, wk = (None, None) if self.q_norm is None else (self.q_norm.weight, self.k_norm.weight)
-        q = cuda_ops.qkv_prep(q, p["k"], values, wq, wk, self.eps, positions, freq, ks, vs, holder.lengths_dev)
+        if wide or self.halves or self.amplitude != 1.0:
+            kh, vh = (self._heads(ks, self.dim), self._heads(vs, self.vdim)) if wide else (ks, vs)
+            q = cuda_ops.head_prep(q, p["k"], values, wq, wk, self.eps, positions, freq, self.halves, self.amplitude, self.talk, kh, vh,
+                                   holder.lengths_dev)
+            vs = vh
+        else:
+            q = cuda_ops.qkv_prep(q, p["k"], values, wq, wk, self.eps, positions, freq, ks, vs, holder.lengths_dev)
         if s == 1 and cache is not None:
             return cuda_ops.grouped_decode(q[:, 0], ks, vs, holder.lengths_next, keep, sink, self.scale, self.softcap, gate, *mask)
         end = holder.length + s
@@ -470,7 +493,7 @@ class SelectiveScan(nn.Module):
             prev = cache.recurrent_state(layer_id, (batch, self.taps - 1, self.inner), h.device, "conv")
             state = cache.recurrent_state(layer_id, (batch, self.inner, self.state), h.device)
         p = self.in_proj(h)
-        x = ops.causal_conv_silu(p["x"], self.conv_weight, self.conv_bias, batch, keep, prev, fused=self.oslo_fused)
+        x = ops.causal_conv(p["x"], self.conv_weight, self.conv_bias, batch, keep, prev, silu=True, fused=self.oslo_fused)
         sel = self.x_proj(x)
         if s == 1 and state is not None and self.oslo_fused and _inference(h, self.a_log) and ops.use_kernels(h):
             from ..ops import cuda_ops
@@ -506,47 +529,112 @@ class GatedMLP(nn.Module):
         return FeedForwardOutput(self.down(a), {n: p[n] for n in self.side})
 
 
+class DenseMLP(nn.Module):
+    """``W_down act(W_up h)``, ``act`` ``"relu2"`` (the square of relu) or a GeLU."""
+
+    oslo_fused = False
+
+    def __init__(self, width: int, ff: int, act: str = "relu2") -> None:
+        super().__init__()
+        self.act = act
+        self.up = Linear(width, ff, bias=False)
+        self.down = Linear(ff, width, bias=False)
+
+    def forward(self, h: Tensor) -> FeedForwardOutput:
+        return FeedForwardOutput(self.down(self.up(h, self.act)), {})
+
+
 class MixtureOfExperts(nn.Module):
     """``experts`` small feed-forwards, of which a token uses ``top``. No capacity limit: every choice is computed. The result keeps one
     row per (token, choice); whoever adds it to the residual stream sums the rows.
 
-    ``unit="relu2"``: ``W_down relu(W_up h)^2``; ``"silu"``: ``W_down (silu(W_gate h) * W_up h)``. The router's logits are fp32: ``W_r h + b``
-    choose, weighted by the softmax over the chosen ones; ``scored``: scores are the softmax of ``W_r h`` over all outputs, ``score +
-    correction`` choose, the weights are the chosen scores divided by their sum. ``identity`` further router outputs stand for the
-    input itself. ``shared``: size of an expert that every token uses, weighted by a sigmoid projection of its own."""
+    ``unit="relu2"``: ``W_down relu(W_up h)^2``; ``"silu"``: ``W_down (silu(W_gate h) * W_up h)``; ``"clamped"``: ``GatedMLP``'s unit with
+    ``limit`` and ``alpha``. The router's logits are fp32: ``W_r h + b`` choose, weighted by the softmax over the chosen ones; ``scored``:
+    scores are the softmax of ``W_r h`` over all outputs, ``score + correction`` choose, the weights are the chosen scores divided by
+    their sum; ``scored="sigmoid"``: the largest ``sigmoid(W_r h)`` choose and are the weights as they are. ``identity`` further router
+    outputs stand for the input itself. ``scale_input``: a weight multiplies what its expert reads, and the rows are summed without
+    weights. ``shared``: size of an expert that every token uses, weighted by a sigmoid projection of its own (``shared_gate=False``:
+    added as it is), with ``shared_limit`` where it is clamped."""
 
     oslo_fused = False
 
     def __init__(self, width: int, ff: int, experts: int, top: int, side: Optional[Dict[str, int]] = None, unit: str = "relu2",
-                 scored: bool = False, identity: int = 0, shared: Optional[int] = None) -> None:
+                 scored=False, identity: int = 0, shared: Optional[int] = None, limit: float = 0.0, alpha: float = 1.702,
+                 scale_input: bool = False, shared_gate: bool = True, shared_limit: Optional[float] = None) -> None:
         super().__init__()
-        if unit not in ("relu2", "silu"):
+        if unit not in ("relu2", "silu", "clamped"):
             raise ValueError(f"unknown expert unit {unit!r}")
+        if scored not in (False, True, "sigmoid"):
+            raise ValueError(f"unknown scores {scored!r}")
         self.experts, self.top, self.unit, self.scored, self.identity = experts, top, unit, scored, identity
+        self.limit, self.alpha, self.scale_input, self.shared_gate = float(limit), float(alpha), bool(scale_input), bool(shared_gate)
         self.side = dict(side or {})
         self.in_proj = PackedLinear(width, self.side) if self.side else None
         outputs = experts + identity
         self.router = Linear(width, outputs, bias=not scored)
-        self.correction = nn.Parameter(torch.zeros(outputs)) if scored else None
-        self.up = nn.Parameter(torch.empty(experts, ff * (2 if unit == "silu" else 1), width).normal_(std=0.02))
+        self.correction = nn.Parameter(torch.zeros(outputs)) if scored is True else None
+        self.up = nn.Parameter(torch.empty(experts, ff * (1 if unit == "relu2" else 2), width).normal_(std=0.02))
         self.down = nn.Parameter(torch.empty(experts, width, ff).normal_(std=0.02))
-        self.shared = GatedMLP(width, shared, side={"sg": 1}) if shared is not None else None
+        self.shared = None
+        if shared is not None:
+            self.shared = GatedMLP(width, shared, side={"sg": 1} if shared_gate else None, limit=shared_limit, alpha=alpha)
 
     @staticmethod
     def interleave(gate: Tensor, up: Tensor) -> Tensor:
-        """``up`` of a ``"silu"`` expert from its two matrices ``[ff, width]``: rows in turns, so that one tile holds both factors."""
+        """``up`` of a gated expert from its two matrices ``[ff, width]``: rows in turns, so that one tile holds both factors."""
         return torch.stack([gate, up], dim=1).reshape(2 * gate.size(0), gate.size(1))
 
     def forward(self, h: Tensor) -> FeedForwardOutput:
         side = self.in_proj(h) if self.in_proj is not None else {}
         bias = self.correction if self.scored else self.router.bias
         idx, weights = ops.moe_route(h, self.router.weight, bias, self.top, self.scored, fused=self.oslo_fused)
-        y, slots = ops.moe_experts(h, idx, self.up, self.down, self.unit, fused=self.oslo_fused)
+        y, slots = ops.moe_experts(h, idx, self.up, self.down, self.unit, self.limit, self.alpha, weights if self.scale_input else None,
+                                   fused=self.oslo_fused)
         shared, gate = None, None
         if self.shared is not None:
             out = self.shared(h)
-            shared, gate = out.y, out.side["sg"]
-        return FeedForwardOutput(y, side, slots, weights, idx if self.identity else None, shared, gate)
+            shared, gate = out.y, out.side.get("sg")
+        return FeedForwardOutput(y, side, slots, None if self.scale_input else weights, idx if self.identity else None, shared, gate)
+
+
+class InputConvolution(nn.Module):
+    """What a mixer reads is its input plus a causal convolution of it over time, per channel and without a bias: ``h + conv(h)``. The
+    last ``taps - 1`` inputs are part of a sequence's state."""
+
+    oslo_fused = False
+
+    def __init__(self, width: int, taps: int) -> None:
+        super().__init__()
+        self.taps = taps
+        self.weight = nn.Parameter(torch.empty(width, taps).normal_(std=taps ** -0.5))
+
+    def state(self, batch: int, layer_id: int, cache: Optional[StaticKVCache], device) -> Optional[Tensor]:
+        if cache is None:
+            return None
+        return cache.recurrent_state(layer_id, (batch, self.taps - 1, self.weight.size(0)), device, "inputs")
+
+    def forward(self, h: Tensor, batch: int, layer_id: int, cache: Optional[StaticKVCache], keep: Optional[Tensor]) -> Tensor:
+        s = h.size(0) // batch
+        return ops.causal_conv(h, self.weight, None, batch, _last(keep, s), self.state(batch, layer_id, cache, h.device), residual=True,
+                               fused=self.oslo_fused)
+
+
+class TokenInput(nn.Module):
+    """A layer's input from the token itself: ``norm(W_proj (gelu(W_gate x) * e))`` with ``e`` the columns ``first`` to ``first + dim`` of the
+    token's row of a table that the model's layers share. The result is a ``Branch`` of the residual stream ``x``."""
+
+    oslo_fused = False
+
+    def __init__(self, width: int, dim: int, first: int, eps: float) -> None:
+        super().__init__()
+        self.first = first
+        self.gate = Linear(width, dim, bias=False)
+        self.proj = Linear(dim, width, bias=False)
+        self.norm = RMSNorm(width, eps)
+
+    def forward(self, x: Tensor, ids: Tensor, table: Tensor) -> Branch:
+        """``x`` ``[rows, width]`` in the weights' dtype, ``ids`` ``[rows]``, ``table`` ``[vocab, *]``."""
+        return Branch(self.proj(ops.token_gate(self.gate(x), ids, table, self.first, fused=self.oslo_fused)), self.norm.weight)
 
 
 class HyperConnections(nn.Module):

@@ -15,6 +15,7 @@ from .dekutar import DekutarConfig, DekutarForCausalLM
 from .gpt2 import GPT2Config, GPT2LMHeadModel
 from .gpt_neo import GPTNeoConfig, GPTNeoForCausalLM
 from .gptj import GPTJConfig, GPTJForCausalLM
+from .masezen import MasezenConfig, MasezenForCausalLM
 from .moronex import MoronexConfig, MoronexForCausalLM
 
 
@@ -30,6 +31,7 @@ MODELS: Dict[str, ModelEntry] = {
     "moronex": ModelEntry(MoronexConfig, MoronexForCausalLM),
     "begovik": ModelEntry(BegovikConfig, BegovikForCausalLM),
     "dekutar": ModelEntry(DekutarConfig, DekutarForCausalLM),
+    "masezen": ModelEntry(MasezenConfig, MasezenForCausalLM),
 }
 
 

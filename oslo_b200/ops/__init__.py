@@ -72,7 +72,8 @@ from .functional import (  # noqa: E402
     scaled_upper_triang_masked_softmax, scaled_masked_softmax, cross_entropy, linear_cross_entropy,
     ban_repeated_ngrams, decode_attention, rms_norm, residual_join, silu_mul, gated_recurrence, sink_attention,
     latent_decode, moe_route, moe_experts, linear_fp32, stacked_linear, branch_join, clamped_glu, gated_rms_norm,
-    decayed_attention, bonus_recurrence, token_shift, causal_conv_silu, selective_scan, matrix_memory, hyper_join,
+    decayed_attention, bonus_recurrence, token_shift, causal_conv, selective_scan, matrix_memory, hyper_join,
+    token_gate,
 )
 
 __all__ = [
@@ -81,6 +82,6 @@ __all__ = [
     "scaled_masked_softmax", "cross_entropy", "linear_cross_entropy", "ban_repeated_ngrams",
     "decode_attention", "rms_norm", "residual_join", "silu_mul", "gated_recurrence", "sink_attention", "latent_decode",
     "moe_route", "moe_experts", "linear_fp32", "stacked_linear", "branch_join", "clamped_glu", "gated_rms_norm",
-    "decayed_attention", "bonus_recurrence", "token_shift", "causal_conv_silu", "selective_scan", "matrix_memory",
-    "hyper_join",
+    "decayed_attention", "bonus_recurrence", "token_shift", "causal_conv", "selective_scan", "matrix_memory",
+    "hyper_join", "token_gate",
 ]

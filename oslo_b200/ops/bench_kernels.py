@@ -323,16 +323,16 @@ def bench_branches(args, timer: _Timer) -> None:
                    like="layer norm")
             hb = mk(n, w)
             report(case, tag + "token shift", lambda: ext.token_shift(hb, mu, b, None, None), gbytes=n * w * 12 / 1e9, like="layer norm")
-            report(case, tag + "convolution", lambda: ext.causal_conv_silu(x, conv, convb, b, None, None), gbytes=n * inner * 4 / 1e9, like="layer norm")
+            report(case, tag + "convolution", lambda: ext.causal_conv(x, conv, convb, b, None, None, True), gbytes=n * inner * 4 / 1e9, like="layer norm")
             p = mk(n, (h + 2 * g) * d)
             kc, vc, l0 = mk(b, g, s, d), mk(b, g, s, d), torch.zeros(b, dtype=torch.int32, device="cuda")
             pos = torch.arange(s, device="cuda")[None].expand(b, s)
             report(case, tag + "norms + rotation + append", lambda: ext.qkv_prep(p[:, :h * d], p[:, h * d:(h + g) * d], p[:, (h + g) * d:], hw, hw, 1e-5,
                                                                               pos, freq, kc, vc, l0), gbytes=n * (h + 2 * g) * d * 4 / 1e9, like="layer norm")
             xs, y1, y2, y3 = torch.randn(n, w, device="cuda"), mk(n, w), mk(n, w), mk(n, w)
-            report(case, tag + "join, 2 branches", lambda: ext.branch_join(xs, y1, None, 1.0, y2, None, 1.0, None, None, 1.0, 0.3, 1e-5, vec, vec),
+            report(case, tag + "join, 2 branches", lambda: co.branch_join(xs, [(y1,), (y2,)], 0.3, 1e-5, [vec, vec]),
                    gbytes=n * w * 16 / 1e9, like="residual join (Moronex)")
-            report(case, tag + "join, 3 branches, 2 normed", lambda: ext.branch_join(xs, y1, vec, 0.5, y2, vec, 0.5, y3, None, 1.0, 0.3, 1e-5, vec, vec),
+            report(case, tag + "join, 3 branches, 2 normed", lambda: co.branch_join(xs, [(y1, vec, 0.5), (y2, vec, 0.5), (y3,)], 0.3, 1e-5, [vec, vec]),
                    gbytes=n * w * 18 / 1e9, like="residual join (Moronex)")
             report(case, tag + "residual join (Moronex)", lambda: ext.residual_join(xs, y1, None, None, y2, vec, vec, vec, 1e-5), gbytes=n * w * 14 / 1e9)
             report(case, tag + "layer norm (GPT-J)", lambda: ext.layernorm_fwd(hb, vec, vec, 1e-5), gbytes=n * w * 4 / 1e9)
@@ -369,7 +369,7 @@ def bench_branches(args, timer: _Timer) -> None:
             report(case, tag + "scan step", lambda: ext.scan_step(x, dl, w_dt, dtb, a_log, bc[:, :ns], bc[:, ns:], dd, zz, None, st3),
                    gbytes=(n * inner * ns * 8 + inner * (dtr + ns) * 2) / 1e9, like="recurrence step (Moronex)")
             cst = torch.zeros(n, 3, inner, device="cuda")
-            report(case, tag + "convolution step", lambda: ext.causal_conv_silu(x, conv, convb, n, None, cst), gbytes=n * inner * 28 / 1e9, like="layer norm")
+            report(case, tag + "convolution step", lambda: ext.causal_conv(x, conv, convb, n, None, cst, True), gbytes=n * inner * 28 / 1e9, like="layer norm")
             hb, sh = mk(n, w), torch.zeros(n, w, device="cuda")
             report(case, tag + "token shift step", lambda: ext.token_shift(hb, mu, n, None, sh), gbytes=n * w * 20 / 1e9, like="layer norm")
             q3 = mk(n, h, d)
@@ -387,7 +387,7 @@ def bench_branches(args, timer: _Timer) -> None:
                 report(case, tag + "attention (GPT-J, 2 launches)", lambda: ext.decode_attn(q3, kf, vf, lengths, d ** -0.5, 0), gbytes=2 * n * t * h * d * 2 / 1e9)
                 del kf, vf
             xs, y1, y2, y3 = torch.randn(n, w, device="cuda"), mk(n, w), mk(n, w), mk(n, w)
-            report(case, tag + "join, 3 branches, 2 normed", lambda: ext.branch_join(xs, y1, vec, 0.5, y2, vec, 0.5, y3, None, 1.0, 0.3, 1e-5, vec, vec),
+            report(case, tag + "join, 3 branches, 2 normed", lambda: co.branch_join(xs, [(y1, vec, 0.5), (y2, vec, 0.5), (y3,)], 0.3, 1e-5, [vec, vec]),
                    gbytes=n * w * 18 / 1e9, like="layer norm")
             report(case, tag + "layer norm (GPT-J)", lambda: ext.layernorm_fwd(hb, vec, vec, 1e-5), gbytes=n * w * 4 / 1e9)
             ws, xm, wx, wm = mk(4, nr, w), mk(4, n, w), mk(dtr + 2 * ns, inner), mk(4 * w, w)

@@ -19,6 +19,7 @@ from ..config import get_config as _get_config
 from . import reference as ref
 
 FLAG_BIAS, FLAG_GELU, FLAG_SAVE_PREACT, FLAG_DGELU, FLAG_RESIDUAL, FLAG_OUT_FP32, FLAG_ACCUMULATE = 1, 2, 4, 8, 16, 32, 64
+FLAG_RELU2, ACT_RELU2 = 1024, -2   # square of relu: in a GEMM's epilogue; as `gelu_from` of the few-row products
 _GELU = ("gelu", "gelu_new", "gelu_tanh", "gelu_pytorch_tanh")
 _16BIT = (torch.bfloat16, torch.float16)
 _dropout_calls = itertools.count()
@@ -297,7 +298,7 @@ def linear(x: Tensor, weight: Tensor, bias: Optional[Tensor], reversed_: bool, a
         if big:
             return _Linear.apply(x, weight, bias, reversed_, False, residual)
         return linear(x, weight, bias, reversed_, activation) + residual
-    if activation is not None and activation not in _GELU:
+    if activation is not None and activation not in _GELU + ("relu2",):
         raise ValueError(f"unsupported fused activation {activation!r}")
     n = weight.size(1) if reversed_ else weight.size(0)
     ok = (x.dtype in _16BIT and weight.dtype == x.dtype and x.size(-1) % 8 == 0 and n % 8 == 0 and x.numel() > 0
@@ -308,12 +309,17 @@ def linear(x: Tensor, weight: Tensor, bias: Optional[Tensor], reversed_: bool, a
     if rows <= SMALL_M_ROWS and not (torch.is_grad_enabled() and (x.requires_grad or weight.requires_grad)):
         # decode steps: weight-streaming split-K GEMM so that every SM pulls weights, not just N / 128 of them
         x2 = _as_operand(x.reshape(rows, x.size(-1)))
-        gelu_from = 0 if activation is not None else -1
+        gelu_from = -1 if activation is None else (ACT_RELU2 if activation == "relu2" else 0)
         if rows <= GEMV_ROWS and not reversed_ and n % 4 == 0:
             y = _ext().gemv_rows(x2, None, _as_operand(weight), bias, gelu_from)   # no tensor-core tile to pad
         else:
             y = _ext().gemm_small_m(x2, _as_operand(weight), int(reversed_), bias, gelu_from)
         return y.view(*x.shape[:-1], n)
+    if activation == "relu2":
+        if torch.is_grad_enabled() and (x.requires_grad or weight.requires_grad):      # no backward of its own
+            return torch.relu(_Linear.apply(x, weight, bias, reversed_, False, None)).pow(2)
+        flags = FLAG_RELU2 | (FLAG_BIAS if bias is not None else 0)
+        return gemm(x.reshape(rows, x.size(-1)), weight, False, reversed_, bias=bias, flags=flags).view(*x.shape[:-1], n)
     return _Linear.apply(x, weight, bias, reversed_, activation is not None, None)
 
 
@@ -730,12 +736,20 @@ def stacked_linear(x: Tensor, weight: Tensor):
     return tuple(gemm(x[i], weight[i]) for i in range(parts))
 
 
-def branch_join(x: Tensor, branches, mult: float, eps: float, w_next):
-    args = [a for y, w, factor in branches for a in (_rows(y), w, float(factor))]
-    args += [None, None, 1.0] * (3 - len(branches))
+def branch_join(x: Tensor, branches, mult: float, eps: float, w_next, copy: Optional[torch.dtype] = None, conv=None):
+    """``reference.branch_join``. ``conv`` ``(weight, state, keep)``, for rows that are single tokens: a second result, the first norm plus its
+    causal convolution (``reference.causal_conv`` with ``residual``), whose state moves on."""
+    bs = [ref.Branch(*b) for b in branches]
     w = list(w_next) + [None] * (2 - len(w_next))
-    xo, h1, h2 = _ext().branch_join(x.contiguous(), *args, float(mult), float(eps), w[0], w[1])
-    return xo, [h1, h2][:len(w_next)]
+    conv_w, state, keep = (None, None, None) if conv is None else conv
+    xo, h1, h2, co = _ext().branch_join(x.contiguous(), [_rows(b.y) for b in bs], [b.weight for b in bs], [float(b.factor) for b in bs],
+                                        [int(b.normed) for b in bs], [b.slots for b in bs], [int(b.top) for b in bs], float(mult),
+                                        float(eps), w[0], w[1], copy is not None, conv_w, state, _keep8(keep))
+    return xo, [h1, co] if conv is not None else [h1, h2][:1 if copy is not None else len(w_next)]
+
+
+def token_gate(z: Tensor, ids: Tensor, table: Tensor, first: int) -> Tensor:
+    return _ext().token_gate(_rows(z), ids.reshape(-1), table, int(first))
 
 
 def clamped_glu(gate: Tensor, up: Tensor, limit: float, alpha: float) -> Tensor:
@@ -801,8 +815,9 @@ def token_shift(h: Tensor, mu: Tensor, batch: int, keep: Optional[Tensor], prev:
     return _ext().token_shift(_rows(h), mu, batch, _keep8(keep), prev)
 
 
-def causal_conv_silu(x: Tensor, w: Tensor, bias: Tensor, batch: int, keep: Optional[Tensor], prev: Optional[Tensor]) -> Tensor:
-    return _ext().causal_conv_silu(_rows(x), w, bias, batch, _keep8(keep), prev)
+def causal_conv(x: Tensor, w: Tensor, bias: Optional[Tensor], batch: int, keep: Optional[Tensor], prev: Optional[Tensor],
+                silu: bool = False, residual: bool = False) -> Tensor:
+    return _ext().causal_conv(_rows(x), w, bias, batch, _keep8(keep), prev, bool(silu), bool(residual))
 
 
 SCAN_MAX_STATES = 256   # states per channel that one launch of the prompt scan covers
@@ -831,13 +846,29 @@ def qkv_prep(q: Tensor, k: Tensor, v: Tensor, wq: Optional[Tensor], wk: Optional
     return _ext().qkv_prep(_rows(q), _rows(k), _rows(v), wq, wk, float(eps), positions, freq, k_store, v_store, lengths)
 
 
+def head_prep(q: Tensor, k: Tensor, v: Tensor, wq: Optional[Tensor], wk: Optional[Tensor], eps: float, positions: Tensor, freq: Tensor,
+              halves: bool, amplitude: float, talk: Optional[Tensor], k_store: Tensor, v_store: Tensor, lengths: Tensor) -> Tensor:
+    """``qkv_prep`` with either rotation, scaled sines and cosines, and caches of any strides ``[B, G, T, *]``. ``talk``: the queries of mixed
+    scores instead (``reference.norm_rotate_fold``), ``[B, S, H, G * dim]``."""
+    return _ext().head_prep(_rows(q), _rows(k), _rows(v), wq, wk, float(eps), positions, freq, bool(halves), float(amplitude), talk, k_store,
+                            v_store, lengths)
+
+
 def grouped_decode(q: Tensor, k: Tensor, v: Tensor, lengths: Tensor, keep: Optional[Tensor], sink: Optional[Tensor], scale: float,
                    softcap: float, gate: Optional[Tensor] = None, window: int = 0, keep_first: int = 0,
                    lead: Optional[Tensor] = None) -> Tensor:
-    if v.size(-1) > GROUPED_MAX_VDIM:
+    """``v`` may have more heads than ``k`` when ``k`` has one and ``v`` is a view of rows that hold all its heads."""
+    heads = v.size(1) // k.size(1)
+    if heads == 1:
+        fits = v.size(-1) <= GROUPED_MAX_VDIM
+    else:
+        fits = _ext().wide_decode_fits(q, q.size(1), heads, k.size(-1), heads * v.size(-1))
+    if not fits:
         return ref.grouped_decode(q, k, v, lengths, keep, sink, scale, softcap, gate, window, keep_first, lead)
+    if heads > 1:
+        v = v.transpose(1, 2).flatten(2).unsqueeze(1)      # a view again
     return _ext().grouped_decode(q.contiguous(), k, v, lengths, _keep8(keep), sink, float(scale), float(softcap),
-                                 None if gate is None else _rows(gate), int(window), int(keep_first), lead)
+                                 None if gate is None else _rows(gate), int(window), int(keep_first), lead, heads)
 
 
 def flash_head_dim(dim: int, vdim: int) -> int:
@@ -858,7 +889,7 @@ def flash_parts_fit(dim: int, rot: int, vdim: int) -> bool:
 def sink_attention(q: Tensor, k: Tensor, v: Tensor, keep: Optional[Tensor], sink: Optional[Tensor], gate: Optional[Tensor], scale: float,
                    softcap: float = 0.0, window: int = 0, keep_first: int = 0, lead: Optional[Tensor] = None,
                    q_rot: Optional[Tensor] = None, k_rot: Optional[Tensor] = None) -> Tensor:
-    """``q`` ``[B, Sq, H, dim]``, ``k``/``v`` ``[B, Sk, G, *]``. 16-bit heads run on the tcgen05 flash kernel, with sink, gate, cap and
+    """``q`` ``[B, Sq, H, dim]``, ``k``/``v`` ``[B, Sk, G, *]`` (``k`` may have one head where ``v`` has several). 16-bit heads run on the tcgen05 flash kernel, with sink, gate, cap and
     window in its softmax and epilogue, and a second operand for the key part that heads share (gated value sizes that are no
     multiple of 8: zero-padded heads, sink and gate from its log-sum-exp); everything else in the fp32 kernel."""
     dim, vdim = q.size(-1), v.size(-1)
@@ -866,6 +897,14 @@ def sink_attention(q: Tensor, k: Tensor, v: Tensor, keep: Optional[Tensor], sink
     mask = (int(window), int(keep_first), lead)
     flash = q.dtype in _16BIT and d and q.size(1) > 1
     gate = None if gate is None else _rows(gate)
+    if k.size(2) == 1 and (v.size(2) > 1 or not d):
+        flash = False
+        if q.dtype in _16BIT and q.size(1) > 1 and not softcap and q_rot is None and dim % 8 == 0 and vdim % 8 == 0 and vdim <= 256:
+            if gate is not None and gate.size(1) != q.size(2):
+                gate = _attn_operand(gate)                 # a gate per element is read in 16-byte pieces
+            kpm = _keep8(keep).contiguous() if keep is not None else None
+            qh, kh, vh = (_attn_operand(t.permute(0, 2, 1, 3)) for t in (q, k, v))
+            return _ext().flash_wide_fwd(qh, kh, vh, kpm, sink, gate, float(scale), *mask)
     if flash and gate is not None and gate.size(1) != q.size(2):
         gate = _attn_operand(gate)                         # a gate per element is read in 16-byte pieces
     if q_rot is not None:
@@ -909,24 +948,26 @@ def latent_decode(q: Tensor, w_uk: Tensor, w_uv: Tensor, cache: Tensor, lengths:
                                 float(scale), heads, positions, freq)
 
 
-MOE_UNITS = {None: 0, "relu2": 1, "silu": 2}
+MOE_UNITS = {None: 0, "relu2": 1, "silu": 2, "clamped": 3}
+MOE_SCORES = {False: 0, True: 1, "sigmoid": 2}
 MOE_FEW_PAIRS = 8   # (token, choice) pairs up to which the chosen experts' weights are streamed per pair
 
 
-def moe_route(h: Tensor, w: Tensor, bias: Tensor, top: int, scored: bool = False):
+def moe_route(h: Tensor, w: Tensor, bias: Optional[Tensor], top: int, scored=False):
     logits = None
     if h.size(0) > SMALL_M_ROWS and gemm_ok(h, w):
         logits = linear_fp32(h, w)                         # 16-bit operands, exact products, fp32 sums and output
     elif h.size(0) > 65535:                                # no tensor-core path for these sizes or types: 32-bit library product
         logits = torch.matmul(h.float(), w.float().t())
-    return _ext().moe_route(_rows(h), w, bias, logits, top, scored)
+    return _ext().moe_route(_rows(h), w, bias, logits, top, MOE_SCORES[scored])
 
 
-def moe_experts(h: Tensor, idx: Tensor, up: Tensor, down: Tensor, unit: str = "relu2"):
+def moe_experts(h: Tensor, idx: Tensor, up: Tensor, down: Tensor, unit: str = "relu2", limit: float = 0.0, alpha: float = 1.702,
+                scale: Optional[Tensor] = None):
     u = MOE_UNITS[unit]
     if idx.numel() <= MOE_FEW_PAIRS:
-        a = _ext().moe_few(_rows(h), idx, up, idx.size(1), u)
+        a = _ext().moe_few(_rows(h), idx, up, idx.size(1), u, float(limit), float(alpha), scale)
         return _ext().moe_few(a, idx, down, 1, 0), None
-    slots, rows, tile_group, n_tiles = _ext().moe_plan(_rows(h), idx, up.size(0))
-    a = _ext().moe_grouped(rows, up, tile_group, n_tiles, u)
+    slots, rows, tile_group, n_tiles = _ext().moe_plan(_rows(h), idx, up.size(0), scale)
+    a = _ext().moe_grouped(rows, up, tile_group, n_tiles, u, float(limit), float(alpha))
     return _ext().moe_grouped(a, down, tile_group, n_tiles, 0), slots

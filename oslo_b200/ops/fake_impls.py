@@ -219,31 +219,35 @@ def register() -> None:
         return q.new_empty((q.size(0), w_uv.size(0)))
 
     @reg("oslo_b200::moe_route")
-    def _(h, w, bias, logits, top, scored=False):
+    def _(h, w, bias, logits, top, scored=0):
         return h.new_empty((h.size(0), top), dtype=torch.int32), h.new_empty((h.size(0), top), dtype=torch.float32)
 
     @reg("oslo_b200::moe_plan")
-    def _(h, idx, experts):
+    def _(h, idx, experts, scale=None):
         tiles = (idx.numel() + 127) // 128 + min(experts, idx.numel())
         return (torch.empty_like(idx), h.new_empty((tiles * 128, h.size(1))), idx.new_empty((tiles,)), idx.new_empty((1,)))
 
     @reg("oslo_b200::moe_grouped")
-    def _(rows, w, tile_group, n_tiles, unit):
-        return rows.new_empty((rows.size(0), w.size(1) // (2 if unit == 2 else 1)))
+    def _(rows, w, tile_group, n_tiles, unit, limit=0.0, alpha=1.0):
+        return rows.new_empty((rows.size(0), w.size(1) // (2 if unit >= 2 else 1)))
 
     @reg("oslo_b200::moe_few")
-    def _(x, idx, w, per_row, unit):
-        return x.new_empty((idx.numel(), w.size(1) // (2 if unit == 2 else 1)))
+    def _(x, idx, w, per_row, unit, limit=0.0, alpha=1.0, scale=None):
+        return x.new_empty((idx.numel(), w.size(1) // (2 if unit >= 2 else 1)))
 
     @reg("oslo_b200::clamped_glu")
     def _(gate, up, limit, alpha):
         return gate.new_empty(gate.shape)
 
     @reg("oslo_b200::branch_join")
-    def _(x, y0, n0, f0, y1, n1, f1, y2, n2, f2, mult, eps, w1, w2):
+    def _(x, y, w, factor, normed, slots, top, mult, eps, w1, w2, copy=False, conv_w=None, prev=None, keep=None):
         rows, cols = x.shape
-        return (torch.empty_like(x), y0.new_empty((rows if w1 is not None else 0, cols)),
-                y0.new_empty((rows if w2 is not None else 0, cols)))
+        outs = (w1 is not None or copy, w2 is not None, conv_w is not None)
+        return (torch.empty_like(x), *(y[0].new_empty((rows if there else 0, cols)) for there in outs))
+
+    @reg("oslo_b200::token_gate")
+    def _(z, ids, table, first):
+        return z.new_empty(z.shape)
 
     @reg("oslo_b200::gated_rms_norm")
     def _(o, w, gate, eps, group, act, z=None, m=None):
@@ -291,16 +295,29 @@ def register() -> None:
     def _(q, k, v, wq, wk, eps, positions, freq, kc, vc, lengths):
         return q.new_empty((kc.size(0), q.size(0) // kc.size(0), q.size(1) // kc.size(3), kc.size(3)))
 
+    @reg("oslo_b200::head_prep")
+    def _(q, k, v, wq, wk, eps, positions, freq, halves, amplitude, talk, kc, vc, lengths):
+        b, g, _, d = kc.shape
+        return q.new_empty((b, q.size(0) // b, q.size(1) // d, d if talk is None else g * d))
+
+    @reg("oslo_b200::wide_decode_fits")
+    def _(like, heads, value_heads, dim, vdim):
+        return True
+
+    @reg("oslo_b200::flash_wide_fwd")
+    def _(q, k, v, kpm, sink, gate, scale, window=0, keep_first=0, lead=None):
+        return q.new_empty((q.size(0) * q.size(2), q.size(1) * v.size(3)))
+
     @reg("oslo_b200::grouped_decode")
-    def _(q, kc, vc, lengths, keep, sink, scale, softcap, gate=None, window=0, keep_first=0, lead=None):
-        return q.new_empty((q.size(0), q.size(1) * vc.size(3)))
+    def _(q, kc, vc, lengths, keep, sink, scale, softcap, gate=None, window=0, keep_first=0, lead=None, value_heads=1):
+        return q.new_empty((q.size(0), q.size(1) * (vc.size(3) // value_heads)))
 
     @reg("oslo_b200::token_shift")
     def _(h, mu, batch, keep, prev):
         return h.new_empty((mu.size(0), h.size(0), h.size(1)))
 
-    @reg("oslo_b200::causal_conv_silu")
-    def _(x, w, bias, batch, keep, prev):
+    @reg("oslo_b200::causal_conv")
+    def _(x, w, bias, batch, keep, prev, silu=False, residual=False):
         return x.new_empty(x.shape)
 
     @reg("oslo_b200::selective_scan")

@@ -214,21 +214,21 @@ def latent_decode(q: Tensor, w_uk: Tensor, w_uv: Tensor, cache: Tensor, lengths:
     return ref.latent_decode(q, w_uk, w_uv, cache, lengths, keep, sink, gate, scale, heads, positions, freq)
 
 
-def moe_route(h: Tensor, w: Tensor, bias: Tensor, top: int, scored: bool = False, fused: bool = True) -> Tuple[Tensor, Tensor]:
+def moe_route(h: Tensor, w: Tensor, bias: Optional[Tensor], top: int, scored=False, fused: bool = True) -> Tuple[Tensor, Tensor]:
     if fused and _kn(h, w, bias):
         from . import cuda_ops
         return cuda_ops.moe_route(h, w, bias, top, scored)
     return ref.moe_route(h, w, bias, top, scored)
 
 
-def moe_experts(h: Tensor, idx: Tensor, up: Tensor, down: Tensor, unit: str = "relu2",
-                fused: bool = True) -> Tuple[Tensor, Optional[Tensor]]:
+def moe_experts(h: Tensor, idx: Tensor, up: Tensor, down: Tensor, unit: str = "relu2", limit: float = 0.0, alpha: float = 1.702,
+                scale: Optional[Tensor] = None, fused: bool = True) -> Tuple[Tensor, Optional[Tensor]]:
     """The chosen experts' results (``reference.moe_experts``), one row per (token, choice), and where those rows are (``None``: row
     ``token * top + choice``); the step that joins the residual stream adds them up. Rows of choices that are no expert hold anything."""
-    if fused and _kn(h, up, down):
+    if fused and _kn(h, up, down, scale):
         from . import cuda_ops
-        return cuda_ops.moe_experts(h, idx, up, down, unit)
-    return ref.moe_experts(h, idx, up, down, unit), None
+        return cuda_ops.moe_experts(h, idx, up, down, unit, limit, alpha, scale)
+    return ref.moe_experts(h, idx, up, down, unit, limit, alpha, scale), None
 
 
 def hyper_join(x: Tensor, result: Optional[ref.SublayerResult], w_out: Optional[Tensor], mix: Optional[Tensor],
@@ -258,13 +258,20 @@ def stacked_linear(x: Tensor, weight: Tensor, fused: bool = True) -> Tuple[Tenso
     return torch.matmul(x, weight.transpose(1, 2)).unbind(0)
 
 
-def branch_join(x: Tensor, branches, mult: float, eps: float, w_next, fused: bool = True):
-    """Add the results of parallel branches to the fp32 residual stream and norm the sum once per weight of ``w_next``: one pass
-    over the rows. See ``reference.branch_join``."""
+def branch_join(x: Tensor, branches, mult: float, eps: float, w_next, copy: Optional[torch.dtype] = None, fused: bool = True):
+    """Add the results of parallel branches to the fp32 residual stream and norm the sum once per weight of ``w_next``, or copy it: one
+    pass over the rows. See ``reference.branch_join``."""
     if fused and _kn(x, *(t for b in branches for t in b[:2]), *w_next):
         from . import cuda_ops
-        return cuda_ops.branch_join(x, branches, mult, eps, w_next)
-    return ref.branch_join(x, branches, mult, eps, w_next)
+        return cuda_ops.branch_join(x, branches, mult, eps, w_next, copy)
+    return ref.branch_join(x, branches, mult, eps, w_next, copy)
+
+
+def token_gate(z: Tensor, ids: Tensor, table: Tensor, first: int, fused: bool = True) -> Tensor:
+    if fused and _kn(z, table):
+        from . import cuda_ops
+        return cuda_ops.token_gate(z, ids, table, first)
+    return ref.token_gate(z, ids, table, first)
 
 
 def clamped_glu(gate: Tensor, up: Tensor, limit: float, alpha: float, fused: bool = True) -> Tensor:
@@ -331,12 +338,12 @@ def token_shift(h: Tensor, mu: Tensor, batch: int, keep: Optional[Tensor], prev:
     return mixed
 
 
-def causal_conv_silu(x: Tensor, w: Tensor, bias: Tensor, batch: int, keep: Optional[Tensor], prev: Optional[Tensor],
-                     fused: bool = True) -> Tensor:
+def causal_conv(x: Tensor, w: Tensor, bias: Optional[Tensor], batch: int, keep: Optional[Tensor], prev: Optional[Tensor],
+                silu: bool = False, residual: bool = False, fused: bool = True) -> Tensor:
     if fused and _kn(x, w, bias):
         from . import cuda_ops
-        return cuda_ops.causal_conv_silu(x, w, bias, batch, keep, prev)
-    y, last = ref.causal_conv_silu(x, w, bias, batch, keep, prev)
+        return cuda_ops.causal_conv(x, w, bias, batch, keep, prev, silu, residual)
+    y, last = ref.causal_conv(x, w, bias, batch, keep, prev, silu, residual)
     if prev is not None:
         prev.copy_(last.detach())
     return y

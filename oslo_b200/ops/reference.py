@@ -9,7 +9,7 @@ includes/fused_softmax.h:111-229; n-gram ban: fused_ngram_repeat_block.cu:18-49)
 from __future__ import annotations
 
 import math
-from typing import NamedTuple, Optional, Tuple
+from typing import Dict, NamedTuple, Optional, Tuple
 
 import torch
 import torch.nn.functional as F
@@ -28,6 +28,8 @@ def linear(x: Tensor, weight: Tensor, bias: Optional[Tensor] = None, reversed: b
         y = y + bias
     if activation in ("gelu", "gelu_new", "gelu_tanh", "gelu_pytorch_tanh"):
         y = gelu_tanh(y)
+    elif activation == "relu2":
+        y = torch.relu(y).pow(2)
     elif activation is not None:
         raise ValueError(f"unsupported fused activation {activation!r}")
     return y
@@ -258,14 +260,13 @@ def sink_attention(q: Tensor, k: Tensor, v: Tensor, keep: Optional[Tensor], sink
                    q_rot: Optional[Tensor] = None, k_rot: Optional[Tensor] = None):
     """Causal softmax attention; with ``sink`` the denominator also holds ``exp(sink[head])``; with ``gate`` ``[B * Sq, H]`` or
     ``[B * Sq, H * Dv]`` the output is multiplied by its sigmoid, with ``softcap`` scores become ``softcap * tanh(score / softcap)``.
-    ``q`` ``[B, Sq, H, D]`` are the last positions of ``k``/``v`` ``[B, Sk, G, *]``; query head ``h`` reads key head ``h // (H / G)``;
-    ``keep`` ``[B, Sk]``; ``window``, ``keep_first``, ``lead`` ``[B]``: ``visible_keys``. ``q_rot`` ``[B, Sq, H, R]`` and ``k_rot`` ``[B, Sk,
+    ``q`` ``[B, Sq, H, D]`` are the last positions of ``k``/``v`` ``[B, Sk, G, *]``; query head ``h`` reads key head ``h // (H / G)``
+    (keys and values may differ in ``G``); ``keep`` ``[B, Sk]``; ``window``, ``keep_first``, ``lead`` ``[B]``: ``visible_keys``. ``q_rot`` ``[B, Sq, H, R]`` and ``k_rot`` ``[B, Sk,
     R]``, a part of the keys that all heads share, add ``q_rot . k_rot`` to the scores before the scale. Returns ``[B * Sq, H * Dv]``
     and the weights ``[B, H, Sq, Sk]``."""
     b, sq, h, _ = q.shape
-    sk, per = k.size(1), h // k.size(2)
-    if per > 1:
-        k, v = k.repeat_interleave(per, dim=2), v.repeat_interleave(per, dim=2)
+    sk = k.size(1)
+    k, v = (t if t.size(2) == h else t.repeat_interleave(h // t.size(2), dim=2) for t in (k, v))
     s = torch.einsum("bqhd,bkhd->bhqk", q.to(torch.float32), k.to(torch.float32))
     if q_rot is not None:
         s = s + torch.einsum("bqhd,bkd->bhqk", q_rot.to(torch.float32), k_rot.to(torch.float32))
@@ -329,11 +330,15 @@ def latent_decode(q: Tensor, w_uk: Tensor, w_uv: Tensor, cache: Tensor, lengths:
     return output_gate(o, gate).reshape(b, -1).to(q.dtype)
 
 
-def moe_route(h: Tensor, w: Tensor, bias: Tensor, top: int, scored: bool = False) -> Tuple[Tensor, Tensor]:
+def moe_route(h: Tensor, w: Tensor, bias: Optional[Tensor], top: int, scored=False) -> Tuple[Tensor, Tensor]:
     """The ``top`` experts with the largest ``W h + b`` per token (``[tokens, top]``, int32) and the softmax over those logits.
     ``scored``: scores are the softmax of ``W h`` over all experts, the largest ``score + b`` are chosen, and the weights are the
-    chosen scores without ``b``, divided by their sum."""
+    chosen scores without ``b``, divided by their sum. ``scored="sigmoid"``: the largest ``W h`` are chosen (no ``b``), their weights are
+    ``sigmoid(W h)``."""
     z = torch.matmul(h.to(torch.float32), w.to(torch.float32).t())
+    if scored == "sigmoid":
+        picked, idx = torch.topk(z, top, dim=-1)
+        return idx.to(torch.int32), torch.sigmoid(picked)
     if scored:
         score = torch.softmax(z, dim=-1)
         idx = torch.topk(score + bias.to(torch.float32), top, dim=-1).indices
@@ -343,20 +348,29 @@ def moe_route(h: Tensor, w: Tensor, bias: Tensor, top: int, scored: bool = False
     return idx.to(torch.int32), torch.softmax(picked, dim=-1)
 
 
-def moe_experts(h: Tensor, idx: Tensor, up: Tensor, down: Tensor, unit: str = "relu2") -> Tensor:
+def moe_experts(h: Tensor, idx: Tensor, up: Tensor, down: Tensor, unit: str = "relu2", limit: float = 0.0, alpha: float = 1.702,
+                scale: Optional[Tensor] = None) -> Tensor:
     """Every (token, choice): ``[tokens * top, width]``; ``down`` ``[experts, width, ff]``. ``unit`` ``"relu2"``: ``W_down relu(W_up h)^2``
     with ``up`` ``[experts, ff, width]``; ``"silu"``: ``W_down (silu(W_gate h) * W_up h)`` with ``up`` ``[experts, 2 ff, width]``, rows of the
-    two matrices in turns. Rows of choices that are no expert (``idx >= experts``) are zeros."""
+    two matrices in turns; ``"clamped"``: the same with ``clamped_glu(limit, alpha)`` for ``silu``. ``scale`` ``[tokens, top]`` multiplies what
+    an expert reads. Rows of choices that are no expert (``idx >= experts``) are zeros."""
     n, top = idx.shape
     flat = idx.reshape(-1).to(torch.long)
     rows = h.repeat_interleave(top, dim=0)
+    if scale is not None:
+        rows = (rows.to(torch.float32) * scale.reshape(-1, 1)).to(h.dtype)
     out = h.new_zeros(n * top, down.size(1))
     for e in flat.unique().tolist():
         if e >= up.size(0):
             continue
         at = (flat == e).nonzero(as_tuple=True)[0]
         a = torch.matmul(rows[at], up[e].t())
-        a = silu_mul(a[:, 0::2], a[:, 1::2]) if unit == "silu" else torch.relu(a).pow(2)
+        if unit == "relu2":
+            a = torch.relu(a).pow(2)
+        elif unit == "clamped":
+            a = clamped_glu(a[:, 0::2], a[:, 1::2], limit, alpha)
+        else:
+            a = silu_mul(a[:, 0::2], a[:, 1::2])
         out = out.index_copy(0, at, torch.matmul(a, down[e].t()).to(out.dtype))
     return out
 
@@ -411,18 +425,43 @@ def hyper_join(x: Tensor, result: Optional[SublayerResult], w_out: Optional[Tens
 # ---------------------------------------------------------------------------------------------------------------
 # Residual joins of parallel branches, grouped-query attention, linear recurrences with decays of their own, token shift,
 # causal convolution, selective scan, clamped gated units.
-def branch_join(x: Tensor, branches, mult: float, eps: float, w_next) -> Tuple[Tensor, list]:
-    """``x + mult * sum(factor * y)`` over ``branches`` ``[(y, w, factor), ...]`` in fp32, ``y`` first RMS-normed with weight ``w``
-    unless that is ``None``; and the RMS norms of the sum with every weight of ``w_next``."""
+class Branch(NamedTuple):
+    """A result on its way to the residual stream: ``factor * y``, with a ``weight`` ``[width]`` ``factor * norm(y) * weight``, or
+    (``normed=False``) ``factor * y * weight``. With ``top`` > 0 a token's ``y`` is the sum of ``top`` rows: those that ``slots`` ``[rows,
+    top]`` names, or (``None``) rows ``top * token`` and on."""
+    y: Tensor                              # [rows, width], or more rows with ``top``
+    weight: Optional[Tensor] = None
+    factor: float = 1.0
+    normed: bool = True
+    slots: Optional[Tensor] = None
+    top: int = 0
+
+
+def branch_join(x: Tensor, branches, mult: float, eps: float, w_next, copy: Optional[torch.dtype] = None) -> Tuple[Tensor, list]:
+    """``x + mult`` times the sum of the ``branches`` (``Branch``) in fp32, and the RMS norms of that with every weight of ``w_next``
+    (``[width]``, or one number). ``copy`` (without ``w_next``): instead of norms the sum itself in that dtype."""
     total = None
-    for y, w, factor in branches:
-        yf = y.to(torch.float32)
-        if w is not None:
-            yf = yf * torch.rsqrt(yf.pow(2).mean(-1, keepdim=True) + eps) * w.to(torch.float32)
-        yf = yf if factor == 1.0 else yf * factor
+    for b in branches:
+        b = Branch(*b)
+        yf = b.y.to(torch.float32)
+        if b.top:
+            yf = (yf if b.slots is None else yf[b.slots.reshape(-1).to(torch.long)]).view(x.size(0), b.top, -1).sum(1)
+        if b.weight is not None:
+            if b.normed:
+                yf = yf * torch.rsqrt(yf.pow(2).mean(-1, keepdim=True) + eps)
+            yf = yf * b.weight.to(torch.float32)
+        yf = yf if b.factor == 1.0 else yf * b.factor
         total = yf if total is None else total + yf
-    x = x + mult * total
-    return x, [rms_norm(x, w, eps) for w in w_next]
+    if total is not None:
+        x = x + mult * total
+    return x, [x.to(copy)] if copy is not None else [rms_norm(x, w, eps) for w in w_next]
+
+
+def token_gate(z: Tensor, ids: Tensor, table: Tensor, first: int) -> Tensor:
+    """``gelu_tanh(z)`` times the columns ``first`` and on of the tokens' rows of ``table`` ``[vocab, *]``: ``z`` ``[rows, dim]``, ``ids``
+    ``[rows]``."""
+    e = table[ids.reshape(-1), first:first + z.size(1)]
+    return (gelu_tanh(z.to(torch.float32)) * e.to(torch.float32)).to(z.dtype)
 
 
 def clamped_glu(gate: Tensor, up: Tensor, limit: float, alpha: float) -> Tensor:
@@ -432,15 +471,36 @@ def clamped_glu(gate: Tensor, up: Tensor, limit: float, alpha: float) -> Tensor:
     return (g * torch.sigmoid(alpha * g) * (u + 1.0)).to(up.dtype)
 
 
-def rotary_frequencies(rot_dims: int, base: float):
-    """``base^(-2i / rot_dims)`` for the pairs of the rotated dims, as 32-bit floats rounded once."""
-    return [base ** (-2.0 * i / rot_dims) for i in range(rot_dims // 2)]
+def rotary_frequencies(rot_dims: int, base: float, scaling: Optional[Dict[str, float]] = None):
+    """``base^(-2i / rot_dims)`` for the pairs of the rotated dims, as 32-bit floats rounded once. ``scaling`` (YaRN): pairs that turn
+    less than ``slow`` times over ``original`` positions are slowed down by ``factor``, those that turn more than ``fast`` times keep
+    their frequency, with a linear ramp in between."""
+    freq = [base ** (-2.0 * i / rot_dims) for i in range(rot_dims // 2)]
+    if scaling is None:
+        return freq
+    factor, original = float(scaling["factor"]), float(scaling["original"])
+    pair = lambda turns: rot_dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))   # noqa: E731
+    lo = max(math.floor(pair(float(scaling["fast"]))), 0)
+    hi = min(math.ceil(pair(float(scaling["slow"]))), rot_dims - 1)
+    ramp = [min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0) for i in range(len(freq))]
+    return [f / factor * r + f * (1.0 - r) for f, r in zip(freq, ramp)]
 
 
-def norm_rotate(x: Tensor, w: Optional[Tensor], eps: float, positions: Tensor, freq: Optional[Tensor]) -> Tensor:
+def rotary_amplitude(scaling: Optional[Dict[str, float]] = None) -> float:
+    """What YaRN multiplies sines and cosines by."""
+    return 1.0 if scaling is None else 0.1 * math.log(float(scaling["factor"])) + 1.0
+
+
+def norm_rotate(x: Tensor, w: Optional[Tensor], eps: float, positions: Tensor, freq: Optional[Tensor], halves: bool = False,
+                amplitude: float = 1.0) -> Tensor:
     """Per head of ``x`` ``[B, S, heads, D]``: RMS norm with weight ``w`` ``[D]`` (shared by the heads; ``None``: without a weight, and
-    then before or after the rotation is the same), then the interleaved rotation of the first ``2 * len(freq)`` dims by
-    ``positions * freq`` (fp32); ``positions`` ``[B, S]``."""
+    then before or after the rotation is the same), then the rotation of the first ``2 * len(freq)`` dims by ``positions * freq``
+    (fp32), interleaved pairs or (``halves``) dim ``i`` with dim ``i + len(freq)``, sines and cosines times ``amplitude``; ``positions``
+    ``[B, S]``."""
+    return _norm_rotate(x, w, eps, positions, freq, halves, amplitude).to(x.dtype)
+
+
+def _norm_rotate(x, w, eps, positions, freq, halves, amplitude) -> Tensor:
     y = x.to(torch.float32)
     y = y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + eps)
     if w is not None:
@@ -448,26 +508,44 @@ def norm_rotate(x: Tensor, w: Optional[Tensor], eps: float, positions: Tensor, f
     if freq is not None and freq.numel():
         r = 2 * freq.numel()
         ang = (positions.to(torch.float32).unsqueeze(-1) * freq).unsqueeze(2)
-        sin, cos = torch.sin(ang), torch.cos(ang)
-        a, b = y[..., :r:2], y[..., 1:r:2]
-        y = torch.cat((torch.stack((a * cos - b * sin, b * cos + a * sin), dim=-1).flatten(-2), y[..., r:]), dim=-1)
-    return y.to(x.dtype)
+        sin, cos = amplitude * torch.sin(ang), amplitude * torch.cos(ang)
+        a, b = (y[..., :r // 2], y[..., r // 2:r]) if halves else (y[..., :r:2], y[..., 1:r:2])
+        turned = (a * cos - b * sin, b * cos + a * sin)
+        y = torch.cat((*(turned if halves else (torch.stack(turned, dim=-1).flatten(-2),)), y[..., r:]), dim=-1)
+    return y
+
+
+def norm_rotate_fold(q: Tensor, w: Optional[Tensor], eps: float, positions: Tensor, freq: Optional[Tensor], talk: Tensor, groups: int,
+                     halves: bool = False, amplitude: float = 1.0) -> Tensor:
+    """Queries of attention whose heads' scores are mixed before the softmax (talking heads), ``score_h <- sum_g talk[h, g] score_g``,
+    with ``groups`` key heads: since head ``g`` reads key head ``g // (H / groups)``, the mixed score is one product of the keys of
+    all key heads together with the query ``[sum over the heads g of key head 0 of talk[h, g] q_g | the same of key head 1 | ...]``.
+    Returns that, ``[B, S, H, groups * D]``, for ``q`` ``[B, S, H, D]``, normed and rotated first (``norm_rotate``; rounded once)."""
+    b, s, h, d = q.shape
+    y = _norm_rotate(q, w, eps, positions, freq, halves, amplitude).view(b, s, groups, h // groups, d)
+    t = talk.to(torch.float32).view(h, groups, h // groups)
+    return torch.einsum("hgr,bsgrd->bshgd", t, y).reshape(b, s, h, groups * d).to(q.dtype)
 
 
 def grouped_decode(q: Tensor, k: Tensor, v: Tensor, lengths: Tensor, keep: Optional[Tensor], sink: Optional[Tensor], scale: float,
                    softcap: float = 0.0, gate: Optional[Tensor] = None, window: int = 0, keep_first: int = 0,
                    lead: Optional[Tensor] = None) -> Tensor:
     """One query per row: ``q`` ``[B, H, D]`` over caches ``[B, G, T, *]`` of which the first ``lengths[b]`` positions count;
-    ``keep`` ``[B, <= T]``. Sink, gate ``[B, H]`` and window as in ``sink_attention``. Returns ``[B, H * Dv]``."""
+    ``keep`` ``[B, <= T]``. Sink, gate ``[B, H]`` or ``[B, H * Dv]`` and window as in ``sink_attention``; keys and values may differ in
+    ``G``. Returns ``[B, H * Dv]``."""
     b, h, _ = q.shape
-    g, t = k.size(1), k.size(2)
+    g, t = v.size(1), k.size(2)
+    if k.size(1) != g:
+        k = k.repeat_interleave(h // k.size(1), dim=1).view(b, g, h // g, t, -1)
+    else:
+        k = k.unsqueeze(2)
     at = torch.arange(t, device=q.device)[None, :]
     vis = visible_keys(lengths[:, None] - 1, at, window, keep_first, None if lead is None else lead[:, None])
     if keep is not None:
         n = min(t, keep.size(1))
         vis[:, :n] &= keep[:, :n] != 0
     qg = q.to(torch.float32).view(b, g, h // g, -1)
-    s = torch.einsum("bgrd,bgtd->bgrt", qg, k.to(torch.float32)) * scale
+    s = torch.matmul(k.to(torch.float32), qg.unsqueeze(-1)).squeeze(-1) * scale
     if softcap:
         s = softcap * torch.tanh(s / softcap)
     s = s.masked_fill(~vis[:, None, None, :], float("-inf"))
@@ -578,10 +656,11 @@ def token_shift(h: Tensor, mu: Tensor, batch: int, keep: Optional[Tensor], prev:
     return (hb + (before - hb) * m).to(h.dtype).view(mu.size(0), h.size(0), -1), hb[:, -1]
 
 
-def causal_conv_silu(x: Tensor, w: Tensor, bias: Tensor, batch: int, keep: Optional[Tensor],
-                     prev: Optional[Tensor]) -> Tuple[Tensor, Tensor]:
-    """``silu`` of a causal convolution per channel: ``x`` ``[B * S, C]``, ``w`` ``[C, taps]`` with the current token's tap last,
-    ``prev`` ``[B, taps - 1, C]`` the inputs before (zeros when ``None``). Returns the result and the last ``taps - 1`` inputs."""
+def causal_conv(x: Tensor, w: Tensor, bias: Optional[Tensor], batch: int, keep: Optional[Tensor], prev: Optional[Tensor],
+                silu: bool = False, residual: bool = False) -> Tuple[Tensor, Tensor]:
+    """A causal convolution per channel: ``x`` ``[B * S, C]``, ``w`` ``[C, taps]`` with the current token's tap last, ``prev`` ``[B, taps -
+    1, C]`` the inputs before (zeros when ``None``). ``silu``: of the result; ``residual``: the input is added to it. Returns the
+    result and the last ``taps - 1`` inputs."""
     taps = w.size(1)
     xb = x.view(batch, -1, x.size(-1)).to(torch.float32)
     if keep is not None:
@@ -589,8 +668,11 @@ def causal_conv_silu(x: Tensor, w: Tensor, bias: Tensor, batch: int, keep: Optio
     s = xb.size(1)
     head = xb.new_zeros(batch, taps - 1, xb.size(-1)) if prev is None else prev
     full = torch.cat([head, xb], dim=1)
-    y = bias.to(torch.float32) + sum(w[:, j].to(torch.float32) * full[:, j:j + s] for j in range(taps))
-    return F.silu(y).to(x.dtype).reshape(x.shape), full[:, s:]
+    y = sum(w[:, j].to(torch.float32) * full[:, j:j + s] for j in range(taps))
+    if bias is not None:
+        y = bias.to(torch.float32) + y
+    y = F.silu(y) if silu else y
+    return (y + xb if residual else y).to(x.dtype).reshape(x.shape), full[:, s:]
 
 
 def selective_scan(x: Tensor, dt: Tensor, dt_bias: Tensor, a_log: Tensor, b: Tensor, c: Tensor, d: Tensor, z: Tensor, batch: int,

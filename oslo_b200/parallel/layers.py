@@ -78,14 +78,14 @@ class LayerNorm(nn.LayerNorm):
 
 class RMSNorm(nn.Module):
     """``x / sqrt(mean(x^2) + eps) * (offset + weight)``, fp32 arithmetic, result in the weight's dtype. ``offset=1``: the
-    weight is stored around zero."""
+    weight is stored around zero. ``dim`` ``None``: the weight is one number for all coordinates."""
 
     oslo_fused = False
 
-    def __init__(self, dim: int, eps: float, offset: float = 0.0) -> None:
+    def __init__(self, dim: Optional[int], eps: float, offset: float = 0.0) -> None:
         super().__init__()
         self.eps, self.offset = float(eps), float(offset)
-        self.weight = nn.Parameter(torch.full((dim,), 1.0 - offset))
+        self.weight = nn.Parameter(torch.full(() if dim is None else (dim,), 1.0 - offset))
 
     def forward(self, x: Tensor) -> Tensor:
         fn = ops.rms_norm if self.oslo_fused else ops.reference.rms_norm

@@ -144,7 +144,7 @@ def test_token_shift_and_convolution_look_back_to_the_state():
     w, bias, back = torch.randn(width, taps), torch.randn(width), torch.randn(batch, taps - 1, width)
     for m in (n, 2, 1):                                   # also fewer tokens than the convolution is wide
         x = torch.randn(batch * m, width)
-        got, last = ops.reference.causal_conv_silu(x, w, bias, batch, None, back)
+        got, last = ops.reference.causal_conv(x, w, bias, batch, None, back, silu=True)
         for b in range(batch):
             want = plain.silu(plain.causal_conv(x.double().view(batch, m, width)[b], w.double(), bias.double(), back[b].double()))
             assert err(got.view(batch, m, width)[b], want) < TOL
@@ -221,7 +221,7 @@ def test_mixers_alone():
         assert err(s(h, 1, 0, None, None).y, plain.mamba1(h.double(), get, m, eps)[0]) < TOL
         two = SideBySide(width, dict(heads=4, kv_heads=2, dim=8, vdim=6, scale=0.4), dict(heads=3, dim=5, vdim=4, decay=[0.5] * 3), eps)
         out = two(h, 1, 0, None, None, pos)
-        assert out.y is None and [b.factor for b in out.branches] == [0.5, 0.5] and all(b.norm_weight is not None for b in out.branches)
+        assert out.y is None and [b.factor for b in out.branches] == [0.5, 0.5] and all(b.weight is not None for b in out.branches)
 
 
 # ---------------------------------------------------------------------------------------------------- the whole model

@@ -166,9 +166,9 @@ def test_causal_conv(dtype, batch, s, channels, taps):
     start = rnd(batch, taps - 1, channels)
     for kp in (None, some_padding(batch, s)):
         for prev in (None, start):
-            want, last = ref.causal_conv_silu(x, w, b, batch, kp, prev)
+            want, last = ref.causal_conv(x, w, b, batch, kp, prev, silu=True)
             st = prev.clone() if prev is not None else torch.zeros_like(start)
-            close(ops.causal_conv_silu(x, w, b, batch, kp, st), want, dtype)
+            close(ops.causal_conv(x, w, b, batch, kp, st, silu=True), want, dtype)
             if taps > 1:
                 close(st, last, torch.float32)
 

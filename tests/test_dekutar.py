@@ -222,7 +222,7 @@ def test_mixers_alone():
     with torch.no_grad():
         m = attn(4, 2, 8, 0.4, 6, 2, 4, None, 100.0)["mixer"]
         a = randomise(GroupedQueryAttention(width, 4, 2, 8, 8, 0.4, eps, rot_dims=4, rot_base=100.0, norm_weights=False, sink=False, window=6,
-                                            keep_first=2, value_is_key=True, gate=True))
+                                            keep_first=2, value_is_key=True, gate="head"))
         get = getter({**{s: a.in_proj.part(s) for s in "qkg"}, "o": a.out_proj.weight})
         assert err(a(h, 1, 0, None, None, pos).y, plain.windowed_attention(h.double(), get, m, eps)) < TOL
         m = latent(3, 4, 6, 5, 7, 8, 0.3, None, 50.0)["mixer"]

@@ -68,9 +68,10 @@ def parse_args():
     ap.add_argument("--no-e2e", action="store_true")
     ap.add_argument("--mode", default="train", choices=["train", "decode", "fusion", "serving"],
                     help="train: tokens/s of a training step; decode: ms/token of greedy generation with a KV cache; "
-                         "serving: prompt and decode throughput of Moronex, Begovik and Dekutar beside GPT-J at equal width, heads and layers; "
+                         "serving: prompt and decode throughput of Moronex, Begovik, Dekutar and Masezen beside GPT-J at equal width, heads and layers; "
                          "fusion: seconds of one GPT-2 small beam-search generate() call before and after fuse() (the "
                          "benchmark behind the reference's published numbers)")
+    ap.add_argument("--serving-models", default="moronex,begovik,dekutar,masezen,gptj", help="serving: which models, the first one named in the metric")
     ap.add_argument("--fusion-dtype", default="fp32", choices=["fp32", "bf16"],
                     help="fusion: parameter dtype (the reference's script runs the fp32 checkpoint)")
     ap.add_argument("--prompt", type=int, default=512, help="decode: prompt length")
@@ -622,10 +623,22 @@ def dekutar_config(width, heads, layers, q_rank, kv_rank, experts, vocab=50400):
                 layers=[{"type": kinds[i % 3][0], "mixer": kinds[i % 3][1], "mlp": mlp} for i in range(layers)])
 
 
+def masezen_config(width, heads, layers, experts, vocab=50400):
+    """Attention with mixed heads over four key / value heads; the first feed-forward is dense with GPT-J's weights, the others
+    are three clamped experts of the router's and a shared one, each with a fourth of them; token inputs of 256 dims."""
+    dim, ff = width // heads, 2 * width // 3 // 64 * 64
+    mixer = {"heads": heads, "kv_heads": 4, "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+             "rot": {"base": 500000.0, "dims": dim, "scaling": {"factor": 8.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}
+    dense = {"kind": "dense", "ff": 4 * width}
+    moe = {"kind": "moe", "expert": {"ff": ff, "limit": 7.0}, "router": {"experts": experts, "top": 3}, "shared": {"ff": ff, "limit": 7.0}}
+    return dict(vocab=vocab, width=width, norm={"eps": 1e-6}, canon={"taps": 4}, token_side={"dim": 256},
+                layers=[{"type": "attention", "mixer": mixer, "mlp": moe if i else dense} for i in range(layers)])
+
+
 def serving_main(args) -> None:
     """One GPU, random weights, bf16: prompt throughput (4 x 2048 tokens) and greedy decoding after 2048-token prompts with 1, 8
-    and 64 sequences (one CUDA-graph replay per token) of Moronex, Begovik, Dekutar and GPT-J with the same width, heads and
-    number of layers. A "step" is one ``GraphedGreedyDecoder.generate`` call; CUDA events around its prompt and its token loop; weights
+    and 64 sequences (one CUDA-graph replay per token) of Moronex, Begovik, Dekutar, Masezen and GPT-J with the same width, heads and
+    number of layers (``--serving-models`` selects some). A "step" is one ``GraphedGreedyDecoder.generate`` call; CUDA events around its prompt and its token loop; weights
     and caches are larger than L2. ``--layers`` shortens both models (debug)."""
     import gc
 
@@ -644,8 +657,10 @@ def serving_main(args) -> None:
     l0, results = ext.launch_count(), {}
     for size, (width, heads, layers, q_rank, kv_rank, experts) in SERVING_SIZES.items():
         layers = args.layers or layers
-        for name in ("moronex", "begovik", "dekutar", "gptj"):
-            if name == "dekutar":
+        for name in args.serving_models.split(","):
+            if name == "masezen":
+                cls, cfg = ob.MasezenForCausalLM, ob.MasezenConfig(**masezen_config(width, heads, layers, experts), torch_dtype=torch.bfloat16)
+            elif name == "dekutar":
                 cls, cfg = ob.DekutarForCausalLM, ob.DekutarConfig(**dekutar_config(width, heads, layers, q_rank, kv_rank, experts),
                                                                    torch_dtype=torch.bfloat16)
             elif name == "begovik":
@@ -688,13 +703,14 @@ def serving_main(args) -> None:
             gc.collect()
             torch.cuda.empty_cache()
     clocks = sampler.stop()
-    main_rec = results["w2048_moronex"]
+    first = args.serving_models.split(",")[0]
+    main_rec = results[f"w2048_{first}"]
     print(json.dumps({
-        "metric": "Moronex prompt tokens/sec (width 2048)" + (" (debug)" if args.layers else ""), "value": main_rec["prompt_tokens_per_s"],
+        "metric": f"{first.capitalize()} prompt tokens/sec (width 2048)" + (" (debug)" if args.layers else ""), "value": main_rec["prompt_tokens_per_s"],
         "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
         "ms_per_step": 4 * 2048 / main_rec["prompt_tokens_per_s"] * 1e3, "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
         "dtype": "bf16", "data": "synthetic uniform token ids, random-init weights", "impl": "oslo_b200",
-        "config": {"model": "moronex, begovik and dekutar beside gptj", "global_batch": 4, "seq_len": 2048, "parallelism": "single",
+        "config": {"model": args.serving_models, "global_batch": 4, "seq_len": 2048, "parallelism": "single",
                    "sizes": {k: dict(zip(("width", "heads", "layers", "q_rank", "kv_rank", "experts"), v)) for k, v in SERVING_SIZES.items()},
                    "l2": "weights + caches per step >> 126 MB L2, no explicit flush"},
         "results": results, "clocks": clocks, "e2e": None, "gpu_launches": ext.launch_count() - l0,

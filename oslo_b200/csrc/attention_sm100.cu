@@ -442,11 +442,12 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
 
 // ---------------------------------------------------------------------- wide keys
 // Queries and keys of any width (`chunks` sub-tiles of 64 columns), one key head for all query heads, value heads per group: attention whose
-// heads are mixed before the softmax, with the mix folded into the queries (grouped_attention.cu). All operands are sub-tiles
-// of 128 rows x 64 columns in 16 KB slots: the first FW_RESIDENT of the queries stay, everything else - keys, values, the rest of the
-// queries - passes through a ring in the order in which the MMA warp uses it, Q K^T of block j + 1 ahead of P V of block j.
-constexpr int FW_SLOTS = 14, FW_RESIDENT = 8;
-constexpr uint32_t FW_SLOT = 128 * 128;
+// heads are mixed before the softmax, with the mix folded into the queries (grouped_attention.cu). All operands are sub-tiles of
+// 128 rows x 64 columns, two of them to a 32 KB slot (a slot's hand-over costs the issuing thread about as much as four
+// products take): the first FW_RESIDENT slots hold queries for good, everything else - keys, values, the rest of the queries -
+// passes through a ring in the order in which the MMA warp uses it, Q K^T of block j + 1 ahead of P V of block j.
+constexpr int FW_SLOTS = 7, FW_RESIDENT = 4;
+constexpr uint32_t FW_SUB = 128 * 128, FW_SLOT = 2 * FW_SUB;
 
 __global__ void __launch_bounds__(FA_THREADS, 1)
 fa_wide_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUtensorMap tk, const __grid_constant__ CUtensorMap tv,
@@ -455,7 +456,8 @@ fa_wide_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ C
   constexpr uint32_t TMEM_COLS = 512, O_COL = 2 * BN;
   extern __shared__ uint8_t fa_smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(fa_smem_raw) + 1023) & ~uintptr_t(1023));
-  const int chunks = (dim + 63) / 64, resident = min(chunks, FW_RESIDENT), ring = FW_SLOTS - resident, vc = (p.d_out + 63) / 64;
+  const int chunks = (dim + 63) / 64, pairs = (chunks + 1) / 2, resident = min(pairs, FW_RESIDENT), ring = FW_SLOTS - resident;
+  const int vc = (p.d_out + 63) / 64;
   const uint32_t q_s = smem_u32(smem), ring_s = q_s + resident * FW_SLOT;
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + FW_SLOTS * FW_SLOT);
   const uint32_t bar0 = smem_u32(bars);
@@ -501,63 +503,85 @@ fa_wide_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ C
     // ------------------------------------------------------------------ TMA producer
     if (lane == 0 && nblk > 0) {
       tma_prefetch_desc(&tq); tma_prefetch_desc(&tk); tma_prefetch_desc(&tv);
-      mbar_expect_tx(bar(0), resident * FW_SLOT);
-      for (int c = 0; c < resident; ++c) tma_load_rows(q_s + c * FW_SLOT, &tq, bar(0), c * 64, q0, h, b, p.q_pos);
+      const int first = min(chunks, 2 * resident);
+      mbar_expect_tx(bar(0), first * FW_SUB);
+      for (int c = 0; c < first; ++c) tma_load_rows(q_s + c * FW_SUB, &tq, bar(0), c * 64, q0, h, b, p.q_pos);
       Cursor at;
       bool ok = true;
-      auto load = [&](const CUtensorMap* map, int col, int row, int head, const int* pos) {
+      // sub-tiles c and (below `end`) c + 1 into the next slot
+      auto load = [&](const CUtensorMap* map, int c, int end, int row, int head, const int* pos) {
         ok = mbar_wait(bar(16 + FW_SLOTS + at.slot), at.phase ^ 1, abort_flag, p.err, ERR_WAIT_EMPTY);
         if (!ok) return;
-        mbar_expect_tx(bar(16 + at.slot), FW_SLOT);
-        tma_load_rows(ring_s + at.slot * FW_SLOT, map, bar(16 + at.slot), col, row, head, b, pos);
+        const uint32_t full = bar(16 + at.slot), dst = ring_s + at.slot * FW_SLOT;
+        const bool two = c + 1 < end;
+        mbar_expect_tx(full, two ? FW_SLOT : FW_SUB);
+        tma_load_rows(dst, map, full, c * 64, row, head, b, pos);
+        if (two) tma_load_rows(dst + FW_SUB, map, full, c * 64 + 64, row, head, b, pos);
         at.next(ring);
       };
       auto keys = [&](int j) {
         const int n0 = blocks.start(j);
-        for (int c = 0; c < chunks && ok; ++c) {
-          if (c >= resident) load(&tq, c * 64, q0, h, p.q_pos);
-          if (ok) load(&tk, c * 64, n0, 0, p.k_pos);
+        for (int g = 0; g < pairs && ok; ++g) {
+          if (g >= resident) load(&tq, 2 * g, chunks, q0, h, p.q_pos);
+          if (ok) load(&tk, 2 * g, chunks, n0, 0, p.k_pos);
         }
       };
       keys(0);
       for (int j = 0; j < nblk && ok; ++j) {
         if (j + 1 < nblk) keys(j + 1);
-        for (int c = 0; c < vc && ok; ++c) load(&tv, c * 64, blocks.start(j), h / p.group, p.v_pos);
+        for (int c = 0; c < vc && ok; c += 2) load(&tv, c, vc, blocks.start(j), h / p.group, p.v_pos);
       }
     }
   } else if (warp == 1) {
     // ------------------------------------------------------------------ MMA issuer
-    if (lane == 0 && nblk > 0) {
+    // The whole warp runs the loops, so that addresses and descriptors are warp-uniform; one lane issues.
+    if (nblk > 0) {
       const int fmt = p.fp16 ? 0 : 1;
       const uint32_t idesc_qk = make_idesc_f16(FA_BM, BN, fmt, 0, 0);
-      const uint32_t idesc_pv = make_idesc_f16(FA_BM, 64, fmt, 0, 1);
+      const uint32_t idesc_pv = make_idesc_f16(FA_BM, 128, fmt, 0, 1), idesc_pv1 = make_idesc_f16(FA_BM, 64, fmt, 0, 1);
+      const uint64_t desc_k = make_smem_desc(0, 16, 1024), desc_v = make_smem_desc(0, FW_SUB, 1024);   // plus (address >> 4)
+      const uint32_t q_at = q_s >> 4, ring_at = ring_s >> 4;
+      constexpr uint32_t SLOT_AT = FW_SLOT >> 4, SUB_AT = FW_SUB >> 4;
+      const bool issuer = elect_one();
       Cursor at;
       bool ok = mbar_wait(bar(0), 0, abort_flag, p.err, ERR_WAIT_FULL);
       auto issue_qk = [&](int j) -> bool {
         const int st = j & 1;
         if (!mbar_wait(bar(11 + st), ((j >> 1) & 1) ^ 1, abort_flag, p.err, ERR_WAIT_TMEM_EMPTY)) return false;
         tc_fence_after();
-        for (int c = 0; c < chunks; ++c) {
-          uint32_t a = q_s + c * FW_SLOT;
+        const uint32_t dst = tmem_base + st * BN;
+        for (int g = 0; g < pairs; ++g) {
+          uint32_t a = q_at + g * SLOT_AT;
           int a_slot = -1;
-          if (c >= resident) {
+          if (g >= resident) {
             if (!mbar_wait(bar(16 + at.slot), at.phase, abort_flag, p.err, ERR_WAIT_FULL)) return false;
             a_slot = at.slot;
-            a = ring_s + at.slot * FW_SLOT;
+            a = ring_at + at.slot * SLOT_AT;
             at.next(ring);
           }
           if (!mbar_wait(bar(16 + at.slot), at.phase, abort_flag, p.err, ERR_WAIT_FULL)) return false;
-          tc_fence_after();
-          const uint32_t k_s = ring_s + at.slot * FW_SLOT;
-          const int steps = min(4, (dim - c * 64 + 15) / 16);
-          for (int kk = 0; kk < steps; ++kk)
-            umma_f16(tmem_base + st * BN, make_smem_desc(a + kk * 32, 16, 1024), make_smem_desc(k_s + kk * 32, 16, 1024), idesc_qk,
-                     (c | kk) != 0);
-          if (a_slot >= 0) umma_commit(bar(16 + FW_SLOTS + a_slot));   // the slots may be refilled once these MMAs have read them
-          umma_commit(bar(16 + FW_SLOTS + at.slot));
+          const uint64_t da = desc_k + a, db = desc_k + (ring_at + at.slot * SLOT_AT);
+          const int left = dim - g * 128;              // columns from this slot on
+          if (issuer) {
+            if (left >= 128) {
+#pragma unroll
+              for (int kk = 0; kk < 8; ++kk) {
+                const uint32_t off = (kk >> 2) * SUB_AT + (kk & 3) * 2;
+                umma_f16(dst, da + off, db + off, idesc_qk, (g | kk) != 0);
+              }
+            } else {
+              for (int kk = 0; kk * 16 < left; ++kk) {
+                const uint32_t off = (kk >> 2) * SUB_AT + (kk & 3) * 2;
+                umma_f16(dst, da + off, db + off, idesc_qk, (g | kk) != 0);
+              }
+            }
+            if (a_slot >= 0) umma_commit(bar(16 + FW_SLOTS + a_slot));   // the slots may be refilled once these MMAs have read them
+            umma_commit(bar(16 + FW_SLOTS + at.slot));
+            if (g + 1 == pairs) umma_commit(bar(9 + st));                // S_j is ready for the softmax warps
+          }
+          __syncwarp();
           at.next(ring);
         }
-        umma_commit(bar(9 + st));   // S_j is ready for the softmax warps
         return true;
       };
       if (ok) ok = issue_qk(0);
@@ -568,18 +592,23 @@ fa_wide_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ C
         }
         const int st = j & 1;
         ok = mbar_wait(bar(st ? 15 : 13), (j >> 1) & 1, abort_flag, p.err, ERR_WAIT_FULL);
-        for (int c = 0; c < vc && ok; ++c) {
+        if (!ok) break;
+        tc_fence_after();
+        for (int c = 0; c < vc && ok; c += 2) {
           ok = mbar_wait(bar(16 + at.slot), at.phase, abort_flag, p.err, ERR_WAIT_FULL);
           if (!ok) break;
-          tc_fence_after();
+          const uint64_t db = desc_v + (ring_at + at.slot * SLOT_AT);
+          const uint32_t dst = tmem_base + O_COL + c * 64, src = tmem_base + st * BN;
+          const uint32_t idesc = c + 1 < vc ? idesc_pv : idesc_pv1;
+          if (issuer) {
 #pragma unroll
-          for (int ks = 0; ks < BN / 16; ++ks)
-            umma_f16_ts(tmem_base + O_COL + c * 64, tmem_base + st * BN + ks * 8,
-                        make_smem_desc(ring_s + at.slot * FW_SLOT + ks * 2048, FW_SLOT, 1024), idesc_pv, (j | ks) != 0);
-          umma_commit(bar(16 + FW_SLOTS + at.slot));
+            for (int ks = 0; ks < BN / 16; ++ks) umma_f16_ts(dst, src + ks * 8, db + ks * 128, idesc, (j | ks) != 0);
+            umma_commit(bar(16 + FW_SLOTS + at.slot));
+            if (c + 2 >= vc) umma_commit(bar(14));                       // O updated, P buffer reusable
+          }
+          __syncwarp();
           at.next(ring);
         }
-        if (ok) umma_commit(bar(14));   // O updated, P buffer reusable
       }
     }
   } else {

@@ -91,13 +91,14 @@ __device__ __forceinline__ bool mbar_try_wait(uint32_t bar, uint32_t parity) {
 // first; every other role then leaves its own wait loop too.
 __device__ __forceinline__ bool mbar_wait(uint32_t bar, uint32_t parity, volatile int* abort_flag, int* err_word,
                                           int code) {
-  if (mbar_try_wait(bar, parity)) return true;
-  const uint64_t t0 = globaltimer_ns();
+  uint64_t t0 = 0;                     // the timer is slow to read: not before the wait has lasted a while
   uint32_t spins = 0;
   while (!mbar_try_wait(bar, parity)) {
     if ((++spins & 0x3f) == 0) {
       if (*abort_flag) return false;
-      if (globaltimer_ns() - t0 > OSLO_WAIT_LIMIT_NS) {
+      const uint64_t now = globaltimer_ns();
+      if (t0 == 0) t0 = now;
+      if (now - t0 > OSLO_WAIT_LIMIT_NS) {
         *abort_flag = 1;
         if (err_word) atomicCAS(err_word, 0, code);
         return false;

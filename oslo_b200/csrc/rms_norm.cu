@@ -223,8 +223,9 @@ __device__ __forceinline__ void load_branch(const BranchParams& p, int b, long l
   }
 }
 
-template <typename T, int VEC>
-__global__ void __launch_bounds__(256) branch_join_kernel(const BranchParams p) {
+// THREADS: at most; few rows get large blocks, so that a row's loads are on their way together
+template <typename T, int VEC, int THREADS>
+__global__ void __launch_bounds__(THREADS) branch_join_kernel(const BranchParams p) {
   extern __shared__ float row_s[];
   __shared__ float red[32];
   const long long row = blockIdx.x;
@@ -524,16 +525,21 @@ extern "C" int oslo_branch_join(const OsloBranchJoin* a, long long rows, int col
   const size_t smem = a->w1 ? static_cast<size_t>(cols) * sizeof(float) : 0;
   if (smem > 200 * 1024) return -3;
   const int threads = cols >= 1024 ? 256 : (cols >= 512 ? 128 : 64);
-#define BRANCH_GO(V)                                                                                             \
+  const bool few = rows <= 296 && cols > 1024;         // at most two blocks per SM
+#define BRANCH_GO(V, N, THREADS)                                                                                 \
   {                                                                                                              \
     if (smem > 48 * 1024) {                                                                                      \
-      cudaError_t e = cudaFuncSetAttribute(branch_join_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
+      cudaError_t e = cudaFuncSetAttribute(branch_join_kernel<T, V, N>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
                                            static_cast<int>(smem));                                              \
       if (e != cudaSuccess) return static_cast<int>(e);                                                          \
     }                                                                                                            \
-    branch_join_kernel<T, V><<<static_cast<unsigned>(rows), threads, smem, stream>>>(p);                         \
+    branch_join_kernel<T, V, N><<<static_cast<unsigned>(rows), THREADS, smem, stream>>>(p);                      \
   }
-  OSLO_DISPATCH_T(dtype, { if (vec) BRANCH_GO(4) else BRANCH_GO(1) });
+  OSLO_DISPATCH_T(dtype, {
+    if (vec && few) BRANCH_GO(4, 1024, std::min(1024, (cols / 4 + 31) / 32 * 32))
+    else if (vec) BRANCH_GO(4, 256, threads)
+    else BRANCH_GO(1, 256, threads)
+  });
 #undef BRANCH_GO
   return static_cast<int>(cudaGetLastError());
 }

@@ -14,7 +14,7 @@ Checkpoints use flat names (``l3.mix.q``, ``l3.mlp.e0.up``, ``l3.canon1``, ...);
 """
 from __future__ import annotations
 
-from typing import Any, Dict, List, Optional
+from typing import Any, Dict, List, NamedTuple, Optional
 
 import torch
 import torch.nn as nn
@@ -26,6 +26,7 @@ from ...modeling_utils import PretrainedConfig, PreTrainedModel
 from ...ops.reference import Branch
 from ...parallel.layers import Embedding, Linear, RMSNorm
 from ...parallel.mpu import Layer, LayerPolicy
+from ...utils.streams import beside
 from ..common import CausalLMHeadMixin, DecoderBackbone, SequenceClassificationMixin, StaticKVCache
 from ..mixers import DenseMLP, GroupedQueryAttention, InputConvolution, MixtureOfExperts, TokenInput
 
@@ -109,6 +110,12 @@ def _feed_forward(mlp: Optional[Dict[str, Any]], width: int) -> Optional[nn.Modu
                             limit=expert["limit"], scale_input=True, shared_gate=False, **sizes)
 
 
+class After(NamedTuple):
+    """What reads the residual stream after a block: the next block's norm and input convolution, or the final norm."""
+    norm: RMSNorm
+    canon: Optional[InputConvolution] = None
+
+
 class MasezenBlock(nn.Module):
     oslo_fused = False
 
@@ -125,26 +132,35 @@ class MasezenBlock(nn.Module):
         self.ls2 = nn.Parameter(torch.ones(w)) if self.mlp is not None else None
         self.side = TokenInput(w, dim, layer_id * dim, eps)
 
-    def forward(self, x: Tensor, normed: Optional[Tensor], after: RMSNorm, ids: Tensor, table: Tensor,
+    def forward(self, x: Tensor, normed: Optional[Tensor], convolved: Optional[Tensor], after: "After", ids: Tensor, table: Tensor,
                 cache: Optional[StaticKVCache] = None, keep: Optional[Tensor] = None, positions: Optional[Tensor] = None,
                 output_attentions: bool = False):
-        """``x`` ``[batch, S, width]`` fp32. ``normed``: ``x`` through this block's norm when the previous block computed that;
-        ``after``: the norm that follows this block; ``ids`` ``[batch * S]`` tokens and ``table`` ``[vocab, *]`` of their inputs. Returns ``(x, x
-        through after, attention weights or None)``."""
+        """``x`` ``[batch, S, width]`` fp32. ``normed``, ``convolved``: ``x`` through this block's norm, and that through its convolution, when
+        the previous block computed them; ``after``: what follows this block; ``ids`` ``[batch * S]`` tokens and ``table`` ``[vocab, *]`` of
+        their inputs. Returns ``(x, x through the norm that follows, that through the convolution that follows or None, attention
+        weights or None)``."""
         batch, s, w = x.shape
         rows = x.reshape(batch * s, w)
         h = (self.norm1(rows) if normed is None else normed).reshape(batch * s, w)
-        out = self.mixer(self.canon1(h, batch, self.layer_id, cache, keep), batch, self.layer_id, cache, keep, positions, output_attentions)
+
+        def attend():
+            c = self.canon1(h, batch, self.layer_id, cache, keep) if convolved is None else convolved
+            return self.mixer(c, batch, self.layer_id, cache, keep, positions, output_attentions)
+
+        out, f = beside(attend, lambda: None if self.mlp is None else self.mlp(h), h)
         branches = [Branch(out.y, self.ls1, normed=False)]
-        if self.mlp is not None:
-            f = self.mlp(h)
+        if f is not None:
             top = self.mlp.top if isinstance(self.mlp, MixtureOfExperts) else 0
             branches.append(Branch(f.y, self.ls2, normed=False, slots=f.slots, top=top))
             if f.shared is not None:
                 branches.append(Branch(f.shared, self.ls2, normed=False))
         rows, (copy,) = ops.branch_join(rows, branches, 1.0, self.eps, [], copy=self.ls1.dtype, fused=self.oslo_fused)
-        rows, (h,) = ops.branch_join(rows, [self.side(copy, ids, table)], 1.0, self.eps, [after.weight], fused=self.oslo_fused)
-        return rows.view(batch, s, w), h.view(batch, s, w), out.probs
+        conv = None
+        if s == 1 and cache is not None and after.canon is not None:          # single tokens: the join does the next convolution too
+            conv = after.canon.step(batch, self.layer_id + 1, cache, keep, x.device)
+        rows, (h, *more) = ops.branch_join(rows, [self.side(copy, ids, table)], 1.0, self.eps, [after.norm.weight], conv=conv,
+                                           fused=self.oslo_fused)
+        return rows.view(batch, s, w), h.view(batch, s, w), more[0] if more else None, out.probs
 
 
 class MasezenPreTrainedModel(PreTrainedModel):
@@ -247,7 +263,7 @@ class MasezenModel(DecoderBackbone, MasezenPreTrainedModel):
             past_key_values = StaticKVCache(input_ids.shape[-1], grow=True)
         kw = super().prepare_fn(input_ids=input_ids, past_key_values=past_key_values, use_cache=use_cache, **kw)
         kw["presents"] = None
-        kw["_normed"] = None
+        kw["_normed"] = kw["_convolved"] = None
         kw["_ids"] = kw["input_ids"].reshape(-1)
         if kw["attention_mask"] is not None:
             kw["attention_mask"] = (kw["attention_mask"] != 0).to(torch.uint8)
@@ -258,14 +274,14 @@ class MasezenModel(DecoderBackbone, MasezenPreTrainedModel):
         hs = kw["hidden_states"]
         if kw["all_hidden_states"] is not None:
             kw["all_hidden_states"].append(hs)
-        args = dict(after=self.ln_f if layer_id + 1 == len(self.h) else self.h[layer_id + 1].norm1, ids=kw["_ids"],
-                    table=self.side_table.weight, cache=kw["cache"], keep=kw["attention_mask"], positions=kw["position_ids"],
-                    output_attentions=kw["output_attentions"])
+        after = After(self.ln_f) if layer_id + 1 == len(self.h) else After(self.h[layer_id + 1].norm1, self.h[layer_id + 1].canon1)
+        args = dict(convolved=kw["_convolved"], after=after, ids=kw["_ids"], table=self.side_table.weight, cache=kw["cache"], keep=kw["attention_mask"],
+                    positions=kw["position_ids"], output_attentions=kw["output_attentions"])
         if self.gradient_checkpointing and self.training and torch.is_grad_enabled():
-            hs, normed, probs = checkpoint(lambda x, n: block(x, n, **args), hs, kw["_normed"], use_reentrant=False)
+            hs, normed, convolved, probs = checkpoint(lambda x, n: block(x, n, **args), hs, kw["_normed"], use_reentrant=False)
         else:
-            hs, normed, probs = block(hs, kw["_normed"], **args)
-        kw["hidden_states"], kw["_normed"] = hs, normed
+            hs, normed, convolved, probs = block(hs, kw["_normed"], **args)
+        kw["hidden_states"], kw["_normed"], kw["_convolved"] = hs, normed, convolved
         if kw["all_attentions"] is not None:
             kw["all_attentions"].append(probs)
         return kw

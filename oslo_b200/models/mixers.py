@@ -613,6 +613,10 @@ class InputConvolution(nn.Module):
             return None
         return cache.recurrent_state(layer_id, (batch, self.taps - 1, self.weight.size(0)), device, "inputs")
 
+    def step(self, batch: int, layer_id: int, cache: Optional[StaticKVCache], keep: Optional[Tensor], device):
+        """What the join kernel needs to do the convolution of single tokens on its way (``conv`` of ``cuda_ops.branch_join``)."""
+        return self.weight, self.state(batch, layer_id, cache, device), _last(keep, 1)
+
     def forward(self, h: Tensor, batch: int, layer_id: int, cache: Optional[StaticKVCache], keep: Optional[Tensor]) -> Tensor:
         s = h.size(0) // batch
         return ops.causal_conv(h, self.weight, None, batch, _last(keep, s), self.state(batch, layer_id, cache, h.device), residual=True,

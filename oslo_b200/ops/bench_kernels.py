@@ -11,6 +11,8 @@
                                                            selective scan and the branch joins, beside those
 ``python -m oslo_b200.ops.bench_kernels --op streams``     the same for windowed and two-part attention, matrix memory, gated and
                                                            identity experts and the stream join, beside those
+``python -m oslo_b200.ops.bench_kernels --op talk``        the same for attention with mixed heads, clamped experts with scaled inputs,
+                                                           input convolutions and per-token layer inputs, beside those
 ``--case i`` restricts the run to one shape and ``--iters n --warmup w`` bound the number of launches, which is
 what a profiler capture wants. Every line is JSON; ``frac_of_measured`` divides by the bf16 GEMM throughput in
 ``MEASURED_PEAKS.json`` at the repository root when that file exists (else by 1590 TFLOP/s).
@@ -559,6 +561,128 @@ def bench_streams(args, timer: _Timer) -> None:
             del up1
 
 
+# width, heads, kv heads, head dim, experts, top, ff of an expert, token dim, taps
+TALK_CASES = [(2048, 16, 4, 128, 16, 3, 1344, 256, 4), (4096, 32, 8, 128, 32, 3, 2688, 256, 4), (4096, 32, 4, 128, 32, 3, 2688, 256, 4)]
+
+
+def bench_talk(args, timer: _Timer) -> None:
+    """The kernels of the Masezen layers beside the like kernels of the other families at the same sizes."""
+    ext = load_ext(required=True)
+    report = _reporter(args, _GraphTimer(args.iters, args.warmup, not args.no_flush))
+    bf, none = torch.bfloat16, None
+    mk = lambda *s: (torch.randn(*s, device="cuda") * 0.5).to(bf)                                          # noqa: E731
+    for case, (w, h, g, d, e, top, ff, td, taps) in enumerate(TALK_CASES):
+        if args.case is not None and args.case != case:
+            continue
+        vec, vd, talk, conv, one = mk(w), mk(d), mk(h, h), mk(w, taps), mk(1)
+        sink, freq = torch.zeros(h, dtype=bf, device="cuda"), torch.rand(d // 2, device="cuda")
+        rw, rb = mk(e, w) * 0.1, mk(e) * 0.1
+        up, down, dense, wg, wp, table = mk(e, 2 * ff, w), mk(e, w, ff), mk(4 * w, w), mk(td, w), mk(w, td), mk(50400, 8 * td)
+        clamped = lambda rows, tg, nt: ext.moe_grouped(rows, up, tg, nt, 3, 7.0, 1.702)                    # noqa: E731
+        # ------------------------------------------------ prompts: 4 x 2048 and 1 x 2048 tokens
+        for b, s in ((4, 2048), (1, 2048)):
+            n, tag = b * s, f"prompt {b} x {s} "
+            q, k, v, gate = mk(b, s, h, g * d), mk(b, 1, s, g * d), mk(b, s, g, d), mk(n, h * d)
+            flat = lambda t: t.permute(0, 2, 1, 3)                                                         # noqa: E731
+            pairs = b * h * s * s / 2.0
+            report(case, tag + "attention, mixed heads + gate", lambda: ext.flash_wide_fwd(flat(q), k, flat(v), none, none, gate, d ** -0.5),
+                   gbytes=n * (3 * h + 2 * g) * d * 2 / 1e9, tflop=2.0 * pairs * (2 * d + h) / 1e12, sfu=pairs, like="attention, heads alone (Begovik)")
+            qg, kg = mk(b, s, h, d), mk(b, s, g, d)
+            report(case, tag + "attention, heads alone (Begovik)", lambda: ext.flash_sink_fwd(flat(qg), flat(kg), flat(v), none, sink, none, d ** -0.5, 0.0),
+                   gbytes=n * (2 * h + 2 * g) * d * 2 / 1e9, tflop=4.0 * pairs * d / 1e12, sfu=pairs)
+            pos, l0 = torch.arange(s, device="cuda")[None].expand(b, s), torch.zeros(b, dtype=torch.int32, device="cuda")
+            pa = mk(n, (h + g) * d)
+            ks, vs = mk(b, s, g, d), mk(b, s, g, d)
+            report(case, tag + "norms + rotation + mix + append",
+                   lambda: ext.head_prep(pa[:, :h * d], pa[:, h * d:], pa[:, h * d:], vd, vd, 1e-6, pos, freq, True, 1.1, talk, flat(ks), flat(vs), l0),
+                   gbytes=n * (h + h * g + 3 * g) * d * 2 / 1e9, fp32_tflop=2.0 * n * h * h * d / 1e12, like="norms + rotation + append (Begovik)")
+            kc, vc = mk(b, g, s, d), mk(b, g, s, d)
+            report(case, tag + "norms + rotation by halves + append",
+                   lambda: ext.head_prep(pa[:, :h * d], pa[:, h * d:], pa[:, h * d:], vd, vd, 1e-6, pos, freq, True, 1.1, none, kc, vc, l0),
+                   gbytes=n * (2 * h + 3 * g) * d * 2 / 1e9, like="norms + rotation + append (Begovik)")
+            report(case, tag + "norms + rotation + append (Begovik)",
+                   lambda: ext.qkv_prep(pa[:, :h * d], pa[:, h * d:], pa[:, h * d:], vd, vd, 1e-6, pos, freq, kc, vc, l0),
+                   gbytes=n * (2 * h + 3 * g) * d * 2 / 1e9, like="layer norm")
+            del q, k, v, qg, kg, pa, ks, vs, kc, vc
+            hb, x, y, sh = mk(n, w), torch.randn(n, w, device="cuda"), mk(n, w), mk(n, w)
+            report(case, tag + "input convolution", lambda: ext.causal_conv(hb, conv, none, b, none, none, False, True), gbytes=n * w * 4 / 1e9,
+                   like="layer norm (GPT-J)")
+            report(case, tag + "join of mixer + dense, copy", lambda: co.branch_join(x, [(y, vec, 1.0, False), (sh, vec, 1.0, False)], 1.0, 1e-6, [], bf),
+                   gbytes=n * w * 14 / 1e9, like="residual join (Moronex)")
+            report(case, tag + "join of token input + norm", lambda: co.branch_join(x, [(y, vec)], 1.0, 1e-6, [one]), gbytes=n * w * 12 / 1e9,
+                   like="residual join (Moronex)")
+            report(case, tag + "residual join (Moronex)", lambda: ext.residual_join(x, y, none, none, sh, vec, vec, vec, 1e-5), gbytes=n * w * 14 / 1e9)
+            report(case, tag + "layer norm (GPT-J)", lambda: ext.layernorm_fwd(hb, vec, vec, 1e-5), gbytes=n * w * 4 / 1e9)
+            z, ids = mk(n, td), torch.randint(0, 50400, (n,), device="cuda")
+            report(case, tag + "token input: gate product", lambda: co.linear(hb, wg, none, False, none), gbytes=n * (w + td) * 2 / 1e9,
+                   tflop=2.0 * n * w * td / 1e12, like="MLP GEMM (GPT-J)")
+            report(case, tag + "token input: gelu * entry", lambda: ext.token_gate(z, ids, table, td), gbytes=n * td * 6 / 1e9, like="layer norm (GPT-J)")
+            report(case, tag + "token input: product", lambda: co.linear(z, wp, none, False, none), gbytes=n * (w + td) * 2 / 1e9,
+                   tflop=2.0 * n * w * td / 1e12, like="MLP GEMM (GPT-J)")
+            report(case, tag + "dense up, relu^2", lambda: co.linear(hb, dense, none, False, "relu2"), tflop=8.0 * n * w * w / 1e12, like="MLP GEMM (GPT-J)")
+            report(case, tag + "MLP GEMM (GPT-J)", lambda: co.linear(hb, dense, none, False, "gelu_new"), tflop=8.0 * n * w * w / 1e12)
+            report(case, tag + "route, sigmoid", lambda: co.moe_route(hb, rw, none, top, "sigmoid"), gbytes=n * w * 2 / 1e9, like="route (Moronex)")
+            report(case, tag + "route (Moronex)", lambda: co.moe_route(hb, rw, rb, top), gbytes=n * w * 2 / 1e9)
+            idx, wgt = co.moe_route(hb, rw, none, top, "sigmoid")
+            real = n * top
+            slots, rows, tg, nt = ext.moe_plan(hb, idx, e, wgt)
+            report(case, tag + "plan + scaled gather", lambda: ext.moe_plan(hb, idx, e, wgt), gbytes=(n + real) * w * 2 / 1e9, like="plan + gather (Moronex)")
+            report(case, tag + "plan + gather (Moronex)", lambda: ext.moe_plan(hb, idx, e), gbytes=(n + real) * w * 2 / 1e9)
+            report(case, tag + "clamped experts up", lambda: clamped(rows, tg, nt), tflop=4.0 * real * w * ff / 1e12,
+                   gbytes=(real * (w + ff) + 2 * e * w * ff) * 2 / 1e9, like="gated experts up (Dekutar)")
+            report(case, tag + "gated experts up (Dekutar)", lambda: ext.moe_grouped(rows, up, tg, nt, 2), tflop=4.0 * real * w * ff / 1e12,
+                   gbytes=(real * (w + ff) + 2 * e * w * ff) * 2 / 1e9)
+            a = clamped(rows, tg, nt)
+            ye = ext.moe_grouped(a, down, tg, nt, 0)
+            report(case, tag + "join of mixer + experts + shared, copy",
+                   lambda: co.branch_join(x, [(y, vec, 1.0, False), (ye, vec, 1.0, False, slots, top), (sh, vec, 1.0, False)], 1.0, 1e-6, [], bf),
+                   gbytes=n * w * (14 + 2 * top) / 1e9, like="residual join of experts (Moronex)")
+            report(case, tag + "residual join of experts (Moronex)", lambda: ext.residual_join(x, ye, slots, wgt, sh, vec, vec, vec, 1e-5),
+                   gbytes=n * w * (12 + 2 * top) / 1e9)
+            del hb, x, y, sh, rows, a, ye
+        # ------------------------------------------------ decode over 4096 cached tokens
+        for n in (1, 8, 64):
+            t, tag = 4096, f"decode {n} "
+            lengths = torch.full((n,), t, dtype=torch.int32, device="cuda")
+            l1, pos = lengths - 1, torch.full((n, 1), t - 1, dtype=torch.long, device="cuda")
+            q, gate, ks, vs = mk(n, h, g * d), mk(n, h * d), mk(n, 1, t, g * d), mk(n, 1, t, g * d)
+            report(case, tag + "attention, mixed heads + gate (2 launches)",
+                   lambda: ext.grouped_decode(q, ks, vs, lengths, none, none, d ** -0.5, 0.0, gate, 0, 0, none, g),
+                   gbytes=2 * n * t * g * d * 2 / 1e9, like="attention, heads alone (Begovik, 2 launches)")
+            pa = mk(n, (h + g) * d)
+            heads = lambda c: c.view(n, t, g, d).transpose(1, 2)                                           # noqa: E731
+            report(case, tag + "norms + rotation + mix + append",
+                   lambda: ext.head_prep(pa[:, :h * d], pa[:, h * d:], pa[:, h * d:], vd, vd, 1e-6, pos, freq, True, 1.1, talk, heads(ks), heads(vs), l1),
+                   gbytes=n * (h + h * g + 3 * g) * d * 2 / 1e9, like="norms + rotation + append (Begovik)")
+            q3, kc, vc = mk(n, h, d), ks.view(n, g, t, d), vs.view(n, g, t, d)
+            report(case, tag + "attention, heads alone (Begovik, 2 launches)", lambda: ext.grouped_decode(q3, kc, vc, lengths, none, sink, d ** -0.5, 0.0),
+                   gbytes=2 * n * t * g * d * 2 / 1e9)
+            report(case, tag + "norms + rotation + append (Begovik)",
+                   lambda: ext.qkv_prep(pa[:, :h * d], pa[:, h * d:], pa[:, h * d:], vd, vd, 1e-6, pos, freq, kc, vc, l1),
+                   gbytes=n * (2 * h + 3 * g) * d * 2 / 1e9)
+            del ks, vs, kc, vc
+            hb, x, y, sh, state = mk(n, w), torch.randn(n, w, device="cuda"), mk(n, w), mk(n, w), torch.zeros(n, taps - 1, w, device="cuda")
+            report(case, tag + "join of token input + norm + convolution", lambda: co.branch_join(x, [(y, vec)], 1.0, 1e-6, [one], none, (conv, state, none)),
+                   gbytes=n * w * (14 + 8 * (taps - 1)) / 1e9, like="residual join (Moronex)")
+            report(case, tag + "residual join (Moronex)", lambda: ext.residual_join(x, y, none, none, sh, vec, vec, vec, 1e-5), gbytes=n * w * 14 / 1e9)
+            z, ids = mk(n, td), torch.randint(0, 50400, (n,), device="cuda")
+            report(case, tag + "token input (3 launches)", lambda: co.linear(ext.token_gate(co.linear(hb, wg, none, False, none), ids, table, td), wp, none, False, none),
+                   gbytes=2 * w * td * 2 / 1e9, like="route (Moronex)")
+            report(case, tag + "dense up, relu^2", lambda: co.linear(hb, dense, none, False, "relu2"), gbytes=8 * w * w / 1e9, like="MLP GEMV (GPT-J)")
+            report(case, tag + "MLP GEMV (GPT-J)", lambda: co.linear(hb, dense, none, False, "gelu_new"), gbytes=8 * w * w / 1e9)
+            report(case, tag + "route, sigmoid", lambda: co.moe_route(hb, rw, none, top, "sigmoid"), gbytes=e * w * 2 / 1e9, like="route (Moronex)")
+            report(case, tag + "route (Moronex)", lambda: co.moe_route(hb, rw, rb, top), gbytes=e * w * 2 / 1e9)
+            idx, wgt = co.moe_route(hb, rw, none, top, "sigmoid")
+            used = int(idx.unique().numel())
+            report(case, tag + "clamped experts up + down", lambda: co.moe_experts(hb, idx, up, down, "clamped", 7.0, 1.702, wgt), gbytes=used * w * ff * 6 / 1e9,
+                   like="gated experts up + down (Dekutar)")
+            report(case, tag + "gated experts up + down (Dekutar)", lambda: co.moe_experts(hb, idx, up, down, "silu"), gbytes=used * w * ff * 6 / 1e9)
+            ye, slots = co.moe_experts(hb, idx, up, down, "clamped", 7.0, 1.702, wgt)
+            report(case, tag + "join of mixer + experts + shared, copy",
+                   lambda: co.branch_join(x, [(y, vec, 1.0, False), (ye, vec, 1.0, False, slots, top), (sh, vec, 1.0, False)], 1.0, 1e-6, [], bf),
+                   gbytes=n * w * (14 + 2 * top) / 1e9, like="residual join (Moronex)")
+
+
 def _every_head(t: torch.Tensor, per: int) -> torch.Tensor:
     """Every key / value head ``per`` times: what attention without groups reads."""
     b, g, s, d = t.shape
@@ -567,18 +691,19 @@ def _every_head(t: torch.Tensor, per: int) -> torch.Tensor:
 
 def main() -> None:
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
-    ap.add_argument("--op", choices=["gemm", "attention", "mixers", "branches", "streams"], required=True)
+    ap.add_argument("--op", choices=["gemm", "attention", "mixers", "branches", "streams", "talk"], required=True)
     ap.add_argument("--case", type=int, default=None, help="index into the op's shape list")
     ap.add_argument("--iters", type=int, default=20)
     ap.add_argument("--warmup", type=int, default=5)
     ap.add_argument("--causal", type=int, default=None, help="attention: 1 / 0 to run only one mask")
     ap.add_argument("--no-baseline", action="store_true", help="skip the library / legacy-kernel baseline")
     ap.add_argument("--no-flush", action="store_true", help="do not write a 256 MB buffer between timed calls")
-    ap.add_argument("--only", default="", help="mixers, branches, streams: only the entries whose name contains this")
+    ap.add_argument("--only", default="", help="mixers, branches, streams, talk: only the entries whose name contains this")
     args = ap.parse_args()
     timer = _Timer(args.iters, args.warmup, not args.no_flush)
     with torch.no_grad():
-        {"gemm": bench_gemm, "attention": bench_attention, "mixers": bench_mixers, "branches": bench_branches, "streams": bench_streams}[args.op](args, timer)
+        {"gemm": bench_gemm, "attention": bench_attention, "mixers": bench_mixers, "branches": bench_branches, "streams": bench_streams,
+         "talk": bench_talk}[args.op](args, timer)
 
 
 if __name__ == "__main__":

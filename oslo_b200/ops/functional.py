@@ -258,13 +258,18 @@ def stacked_linear(x: Tensor, weight: Tensor, fused: bool = True) -> Tuple[Tenso
     return torch.matmul(x, weight.transpose(1, 2)).unbind(0)
 
 
-def branch_join(x: Tensor, branches, mult: float, eps: float, w_next, copy: Optional[torch.dtype] = None, fused: bool = True):
+def branch_join(x: Tensor, branches, mult: float, eps: float, w_next, copy: Optional[torch.dtype] = None, conv=None, fused: bool = True):
     """Add the results of parallel branches to the fp32 residual stream and norm the sum once per weight of ``w_next``, or copy it: one
-    pass over the rows. See ``reference.branch_join``."""
+    pass over the rows. See ``reference.branch_join``. ``conv`` ``(weight, state, keep)``, with one norm and rows that are single tokens:
+    a second result, ``reference.causal_conv`` of the norm with ``residual`` (``state``, or ``None``, is updated)."""
     if fused and _kn(x, *(t for b in branches for t in b[:2]), *w_next):
         from . import cuda_ops
-        return cuda_ops.branch_join(x, branches, mult, eps, w_next, copy)
-    return ref.branch_join(x, branches, mult, eps, w_next, copy)
+        return cuda_ops.branch_join(x, branches, mult, eps, w_next, copy, conv)
+    x, out = ref.branch_join(x, branches, mult, eps, w_next, copy)
+    if conv is not None:
+        weight, state, keep = conv
+        out.append(causal_conv(out[0], weight, None, x.size(0), keep, state, residual=True, fused=False))
+    return x, out
 
 
 def token_gate(z: Tensor, ids: Tensor, table: Tensor, first: int, fused: bool = True) -> Tensor:

@@ -292,10 +292,10 @@ fa_bwd_kernel(const __grid_constant__ CUtensorMap tr1, const __grid_constant__ C
     for (int j = 0; j < nblk && ok; ++j) {
       const int buf = j & 1;
       const int c0 = c_lo + j * BN;
-      ok = mbar_wait(bar(B_SPF + buf), (j >> 1) & 1, abort_flag, p.err, ERR_WAIT_TMEM_FULL);
+      ok = mbar_wait_warp(bar(B_SPF + buf), (j >> 1) & 1, abort_flag, p.err, ERR_WAIT_TMEM_FULL);
       if (!ok) break;
       if (KEY_ROWS) {
-        ok = mbar_wait(bar(B_STF + buf), (j >> 1) & 1, abort_flag, p.err, ERR_WAIT_FULL);
+        ok = mbar_wait_warp(bar(B_STF + buf), (j >> 1) & 1, abort_flag, p.err, ERR_WAIT_FULL);
         if (!ok) break;
       }
       tc_fence_after();
@@ -364,7 +364,7 @@ fa_bwd_kernel(const __grid_constant__ CUtensorMap tr1, const __grid_constant__ C
     }
     // ---- epilogue: accumulator (x scale for dK, dQ) -> global
     if (ok && nblk > 0) {
-      ok = mbar_wait(bar(B_ACC), 0, abort_flag, p.err, ERR_WAIT_TMEM_FULL);
+      ok = mbar_wait_warp(bar(B_ACC), 0, abort_flag, p.err, ERR_WAIT_TMEM_FULL);
       tc_fence_after();
     }
     const float mult = TWO ? p.scale : 1.f;

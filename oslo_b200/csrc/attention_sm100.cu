@@ -74,7 +74,7 @@ struct FaBlocks {
 };
 
 // The four softmax warps of both kernels: S from TMEM columns [0, BN) and [BN, 2 BN), O (D columns) from 2 BN on. Barriers by
-// number from bar0: 9,10 s_full | 11,12 s_empty | 13 p_ready[0] | 14 pv_done | 15 p_ready[1] (PT only: one per S/P buffer)
+// number from bar0: 0 q_full, then (second phase) the last P V is done | 9,10 s_full | 11,12 s_empty | 13 p_ready[0] | 14 pv_done | 15 p_ready[1] (PT only: one per S/P buffer)
 template <int BN, bool PT, bool CAP>
 __device__ __forceinline__ void fa_softmax_warps(const FaParams& p, const int D, const FaBlocks& blocks, uint32_t tmem_base, uint32_t bar0,
                                                  uint32_t p_s, volatile int* abort_flag, int warp, int lane, int b, int h, int q0) {
@@ -94,7 +94,7 @@ __device__ __forceinline__ void fa_softmax_warps(const FaParams& p, const int D,
   for (int j = 0; j < blocks.n && ok; ++j) {
     const int st = j & 1;
     const int n0 = blocks.start(j);
-    ok = mbar_wait(bar(9 + st), (j >> 1) & 1, abort_flag, p.err, ERR_WAIT_TMEM_FULL);
+    ok = mbar_wait_warp(bar(9 + st), (j >> 1) & 1, abort_flag, p.err, ERR_WAIT_TMEM_FULL);
     if (!ok) break;
     tc_fence_after();
     float s[BN];
@@ -169,7 +169,7 @@ __device__ __forceinline__ void fa_softmax_warps(const FaParams& p, const int D,
     // the shared P tile is single-buffered, so P V of block j-1 must have finished before it is rewritten; the
     // TMEM P buffers alternate, so there only a rescale of O has to wait for it
     if (j > 0 && (!PT || rescale)) {
-      ok = mbar_wait(bar(14), (j - 1) & 1, abort_flag, p.err, ERR_WAIT_TMEM_FULL);
+      ok = mbar_wait_warp(bar(14), (j - 1) & 1, abort_flag, p.err, ERR_WAIT_TMEM_FULL);
       if (!ok) break;
       tc_fence_after();
       if (rescale) {
@@ -219,7 +219,8 @@ __device__ __forceinline__ void fa_softmax_warps(const FaParams& p, const int D,
   }
   // ---- epilogue: O / l -> global, log-sum-exp
   if (ok && blocks.n > 0) {
-    ok = mbar_wait(bar(14), (blocks.n - 1) & 1, abort_flag, p.err, ERR_WAIT_TMEM_FULL);
+    // not pv_done: a warp that has rescaled nothing lately may be two of its phases behind, which have the same parity
+    ok = mbar_wait_warp(bar(0), 1, abort_flag, p.err, ERR_WAIT_TMEM_FULL);
     tc_fence_after();
   }
   float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
@@ -311,7 +312,7 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
   const uint32_t p_s = v_s + 2 * V_BYTES;
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + Q_BYTES + 2 * (K_BYTES + V_BYTES) + P_BYTES);
   const uint32_t bar0 = smem_u32(bars);
-  // 0 q_full | 1,2 k_full | 3,4 k_empty | 5,6 v_full | 7,8 v_empty | 9,10 s_full | 11,12 s_empty | 13 p_ready[0] |
+  // 0 q_full, then the last P V | 1,2 k_full | 3,4 k_empty | 5,6 v_full | 7,8 v_empty | 9,10 s_full | 11,12 s_empty | 13 p_ready[0] |
   // 14 pv_done | 15 p_ready[1] (PT only: one per S/P buffer)
   auto bar = [&](int i) { return bar0 + 8u * i; };
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 16);
@@ -420,6 +421,7 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CU
         }
         umma_commit(bar(7 + st));   // V stage free
         umma_commit(bar(14));       // O updated, P buffer reusable
+        if (j + 1 == nblk) umma_commit(bar(0));
       }
     }
   } else {
@@ -544,22 +546,22 @@ fa_wide_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ C
       constexpr uint32_t SLOT_AT = FW_SLOT >> 4, SUB_AT = FW_SUB >> 4;
       const bool issuer = elect_one();
       Cursor at;
-      bool ok = mbar_wait(bar(0), 0, abort_flag, p.err, ERR_WAIT_FULL);
+      bool ok = mbar_wait_warp(bar(0), 0, abort_flag, p.err, ERR_WAIT_FULL);
       auto issue_qk = [&](int j) -> bool {
         const int st = j & 1;
-        if (!mbar_wait(bar(11 + st), ((j >> 1) & 1) ^ 1, abort_flag, p.err, ERR_WAIT_TMEM_EMPTY)) return false;
+        if (!mbar_wait_warp(bar(11 + st), ((j >> 1) & 1) ^ 1, abort_flag, p.err, ERR_WAIT_TMEM_EMPTY)) return false;
         tc_fence_after();
         const uint32_t dst = tmem_base + st * BN;
         for (int g = 0; g < pairs; ++g) {
           uint32_t a = q_at + g * SLOT_AT;
           int a_slot = -1;
           if (g >= resident) {
-            if (!mbar_wait(bar(16 + at.slot), at.phase, abort_flag, p.err, ERR_WAIT_FULL)) return false;
+            if (!mbar_wait_warp(bar(16 + at.slot), at.phase, abort_flag, p.err, ERR_WAIT_FULL)) return false;
             a_slot = at.slot;
             a = ring_at + at.slot * SLOT_AT;
             at.next(ring);
           }
-          if (!mbar_wait(bar(16 + at.slot), at.phase, abort_flag, p.err, ERR_WAIT_FULL)) return false;
+          if (!mbar_wait_warp(bar(16 + at.slot), at.phase, abort_flag, p.err, ERR_WAIT_FULL)) return false;
           const uint64_t da = desc_k + a, db = desc_k + (ring_at + at.slot * SLOT_AT);
           const int left = dim - g * 128;              // columns from this slot on
           if (issuer) {
@@ -591,11 +593,11 @@ fa_wide_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ C
           if (!ok) break;
         }
         const int st = j & 1;
-        ok = mbar_wait(bar(st ? 15 : 13), (j >> 1) & 1, abort_flag, p.err, ERR_WAIT_FULL);
+        ok = mbar_wait_warp(bar(st ? 15 : 13), (j >> 1) & 1, abort_flag, p.err, ERR_WAIT_FULL);
         if (!ok) break;
         tc_fence_after();
         for (int c = 0; c < vc && ok; c += 2) {
-          ok = mbar_wait(bar(16 + at.slot), at.phase, abort_flag, p.err, ERR_WAIT_FULL);
+          ok = mbar_wait_warp(bar(16 + at.slot), at.phase, abort_flag, p.err, ERR_WAIT_FULL);
           if (!ok) break;
           const uint64_t db = desc_v + (ring_at + at.slot * SLOT_AT);
           const uint32_t dst = tmem_base + O_COL + c * 64, src = tmem_base + st * BN;
@@ -605,6 +607,7 @@ fa_wide_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ C
             for (int ks = 0; ks < BN / 16; ++ks) umma_f16_ts(dst, src + ks * 8, db + ks * 128, idesc, (j | ks) != 0);
             umma_commit(bar(16 + FW_SLOTS + at.slot));
             if (c + 2 >= vc) umma_commit(bar(14));                       // O updated, P buffer reusable
+            if (c + 2 >= vc && j + 1 == nblk) umma_commit(bar(0));
           }
           __syncwarp();
           at.next(ring);

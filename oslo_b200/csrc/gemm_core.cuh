@@ -653,7 +653,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_cons
       const int buf = local & 1;
       int tm, tn;
       coords(tile, tm, tn);
-      ok = mbar_wait(tfull_bar(buf), acc_phase[buf], abort_flag, p.err, ERR_WAIT_TMEM_FULL);
+      ok = mbar_wait_warp(tfull_bar(buf), acc_phase[buf], abort_flag, p.err, ERR_WAIT_TMEM_FULL);
       if (!ok) break;
       acc_phase[buf] ^= 1;
       tc_fence_after();

@@ -164,7 +164,7 @@ gemm_pair_tcgen05_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid
       const int buf = local & 1;
       int tm, tn;
       tile_coords(tile, p.tiles_m, p.tiles_n, tm, tn, p.group_m);
-      ok = mbar_wait(tfull_bar(buf), acc_phase[buf], abort_flag, p.err, ERR_WAIT_TMEM_FULL);
+      ok = mbar_wait_warp(tfull_bar(buf), acc_phase[buf], abort_flag, p.err, ERR_WAIT_TMEM_FULL);
       if (!ok) break;
       acc_phase[buf] ^= 1;
       tc_fence_after();

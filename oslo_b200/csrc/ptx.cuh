@@ -108,6 +108,14 @@ __device__ __forceinline__ bool mbar_wait(uint32_t bar, uint32_t parity, volatil
   return true;
 }
 
+// The same for a whole warp (all 32 lanes): its lanes leave together, with one answer. Lanes that poll one by one may see
+// the barrier in different rounds of their loop, and a warp that is not whole must not execute the .sync.aligned
+// instructions (tcgen05.ld / st / wait) that follow such a wait.
+__device__ __forceinline__ bool mbar_wait_warp(uint32_t bar, uint32_t parity, volatile int* abort_flag, int* err_word,
+                                               int code) {
+  return __all_sync(0xffffffffu, mbar_wait(bar, parity, abort_flag, err_word, code)) != 0;
+}
+
 // ------------------------------------------------------------------ TMA (tile mode, this CTA only)
 __device__ __forceinline__ void tma_load_2d(uint32_t dst, const CUtensorMap* map, uint32_t bar, int x, int y) {
   asm volatile(

@@ -657,6 +657,7 @@ RECURRENCE_MAX_DIM = 512   # key channels per head that one launch of the prompt
 BONUS_MAX_DIM = 256        # ... under the rule with a decay per channel
 LATENT_MAX_RANK = 1024     # latent sizes that the decode kernel covers
 GROUPED_MAX_VDIM = 1024    # value sizes that the grouped decode kernel covers
+SINK_SMEM = 227 * 1024     # bytes of shared memory of a block of the 32-bit prompt kernel
 
 
 def _channel_blocks(run, dim: int, limit: int, heads: int, state: Optional[Tensor], rows, vectors) -> Tensor:
@@ -925,6 +926,8 @@ def sink_attention(q: Tensor, k: Tensor, v: Tensor, keep: Optional[Tensor], sink
             qh, kh, vh = (_attn_operand(pad_heads(t, d).permute(0, 2, 1, 3)) for t in (q, k, v))
             o, lse = _ext().flash_fwd(qh, kh, vh, float(scale), True, 0, kpm, _flash_impl())
             return _ext().sink_gate(o, lse, sink, gate, vdim)
+    if 4 * (48 * (dim + vdim + 2) + 528) > SINK_SMEM:      # 16 queries and 32 keys and values of the kernel do not fit
+        return ref.sink_attention(q, k, v, keep, sink, gate, scale, softcap, *mask)[0]
     return _ext().sink_attention(*(t if t.stride(-1) == 1 else t.contiguous() for t in (q, k, v)), _keep8(keep), sink, gate,
                                  float(scale), float(softcap), *mask)
 

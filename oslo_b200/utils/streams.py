@@ -13,7 +13,7 @@ def beside(main: Callable[[], Any], side: Callable[[], Any], like: Tensor) -> Tu
     """``(main(), side())``. While ``like``'s device captures a graph ``side`` is captured on a stream of its own, so that a replay runs the two
     next to each other; what either returns may be used once both have been. Memory: the side stream starts from where the
     capturing one is and is joined before this returns, so a block that one of them gives back is never reused under the other."""
-    if not (like.is_cuda and torch.cuda.is_current_stream_capturing()):
+    if not (like.is_cuda and torch.cuda.is_initialized() and torch.cuda.is_current_stream_capturing()):
         return main(), side()
     current = torch.cuda.current_stream(like.device)
     stream = _SIDE.setdefault(current.device_index, torch.cuda.Stream(like.device))

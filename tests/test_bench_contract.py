@@ -41,6 +41,9 @@ def test_serving_sizes_are_valid_configurations():
         assert any(l["mixer"].get("kv_from") is not None for l in cfg.layers)
         cfg = ob.BegovikConfig(**bench.begovik_config(*size[:3]))
         assert cfg.num_hidden_layers == size[2] and {l["type"] for l in cfg.layers} == {"wkv", "mamba1", "parallel"}
+        width, heads, layers, experts = size[0], size[1], size[2], size[5]
+        cfg = ob.MasezenConfig(**bench.masezen_config(width, heads, layers, experts))
+        assert cfg.num_hidden_layers == layers and [l["mlp"]["kind"] for l in cfg.layers] == ["dense"] + ["moe"] * (layers - 1)
 
 
 def _reference_installed() -> bool:

@@ -152,6 +152,28 @@ def test_dekutar_inference_paths_run_on_fake_cuda_tensors(kernels, dtype):
                 model(input_ids=ids, use_cache=False, output_attentions=True)
 
 
+@pytest.mark.parametrize("dtype", [torch.bfloat16, torch.float32])
+def test_masezen_inference_paths_run_on_fake_cuda_tensors(kernels, dtype):
+    """Prompt, padded batch, decode step and portion through the kernel wrappers of mixed heads, input convolutions, scaled experts and
+    token inputs."""
+    from oslo_b200.models.common import StaticKVCache
+    from .masezen_cases import CASES
+    with FakeTensorMode():
+        with torch.device("cuda"):
+            model = ob.MasezenForCausalLM._from_config(ob.MasezenConfig(**CASES["heads64"]), torch_dtype=dtype)
+        model.fuse().eval()
+        for rows in (2, 7):
+            ids = torch.randint(0, 128, (rows, 96), device="cuda")
+            with torch.no_grad():
+                mask = torch.ones(rows, 96, dtype=torch.long, device="cuda")
+                out = model(input_ids=ids, attention_mask=mask, past_key_values=StaticKVCache(160), use_cache=True)
+                assert out.logits.shape == (rows, 96, 128) and out.logits.dtype == dtype
+                out = model(input_ids=ids[:, :1], past_key_values=out.past_key_values, use_cache=True)
+                out = model(input_ids=ids[:, :40], past_key_values=out.past_key_values, use_cache=True, output_hidden_states=True)
+                assert out.logits.shape == (rows, 40, 128) and all(h.dtype == torch.float32 for h in out.hidden_states)
+                model(input_ids=ids, use_cache=False, output_attentions=True)
+
+
 def test_optimizer_and_elementwise_wrappers_on_fake_cuda_tensors(kernels):
     from oslo_b200.optim import FusedAdamW
     with FakeTensorMode():

@@ -118,6 +118,21 @@ def test_prompt_attention_finds_one_key_among_many():
         assert float(o[at:].min()) > 0.99 and not o[:at].any(), at
 
 
+def test_prompt_attention_is_the_same_every_time():
+    """Bit for bit, with operands in L2 and not: the roles of a block meet in whatever order loads arrive."""
+    ext, other = ops.load_ext(required=True), torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
+    for b, s, t, h, g, d in ((3, 257, 260, 20, 10, 104), (2, 300, 300, 16, 4, 128)):
+        q = rnd(b, h, s, g * d, dtype=torch.bfloat16, scale=2.0 * (g * d) ** -0.25)
+        k, v = rnd(b, 1, t, g * d, dtype=torch.bfloat16, scale=(g * d) ** -0.25), rnd(b, g, t, d, dtype=torch.bfloat16)
+        kq, kk = rnd(b, h, s, 128, dtype=torch.bfloat16), rnd(b, g, t, 128, dtype=torch.bfloat16)
+        for run in (lambda: ext.flash_wide_fwd(q, k, v, None, None, None, 0.7), lambda: ext.flash_sink_fwd(kq, kk, v, None, None, None, 0.2, 0.0)):
+            first = run()
+            for i in range(20):
+                if i % 2:
+                    other.zero_()
+                assert torch.equal(run(), first), i
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("heads,groups,dim", HEADS + RAGGED)
 def test_decode_attention_with_wide_keys(dtype, heads, groups, dim):

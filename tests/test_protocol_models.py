@@ -293,3 +293,65 @@ def test_signal_word_model_catches_a_put_that_does_not_wait_for_an_empty_word():
         if exposed:
             break
     assert exposed, "the model failed to expose the overwritten signal"
+
+
+def _flash_order(blocks, warps, rescales, own_barrier, rnd):
+    """The flash kernels' hand-overs as a random walk over their roles' next steps. Barriers are ``[phases completed]``, a wait for parity
+    ``p`` passes while the phase after the last completed one has the other parity, as on the device. Returns whether some
+    softmax warp read the output before the last P V was done."""
+    s_full, s_empty, p_ready = [0, 0], [[0] * warps, [0] * warps], [[0] * warps, [0] * warps]
+    pv_done, last = 0, 0
+    issued = []                                           # products in issue order; they complete in that order
+    done = 0
+    mma = [("qk", 0)] + [x for j in range(blocks) for x in ([("qk", j + 1)] if j + 1 < blocks else []) + [("pv", j)]]
+    at_mma, at = 0, [(0, "wait")] * warps
+    passed = lambda completed, parity: completed % 2 != parity                                  # noqa: E731
+    early = False
+    while any(step != (blocks, "out") for step in at):
+        who = rnd.randrange(warps + 2)
+        if who == warps:                                  # the issuing thread
+            if at_mma < len(mma):
+                kind, j = mma[at_mma]
+                st, n = j & 1, j >> 1
+                ready = min(s_empty[st]) >= n if kind == "qk" else min(p_ready[st]) > n
+                if ready:
+                    issued.append((kind, j))
+                    at_mma += 1
+        elif who == warps + 1:                            # the tensor core
+            if done < len(issued):
+                kind, j = issued[done]
+                done += 1
+                if kind == "qk":
+                    s_full[j & 1] += 1
+                else:
+                    pv_done += 1
+                    last += j + 1 == blocks
+        else:
+            j, where = at[who]
+            st = j & 1
+            if where == "wait" and j < blocks and passed(s_full[st], (j >> 1) & 1):
+                s_empty[st][who] += 1
+                at[who] = (j, "rescale" if j and rescales(who, j) else "store")
+            elif where == "rescale" and passed(pv_done, (j - 1) & 1):
+                early = early or ("pv", j - 1) not in issued[:done]
+                at[who] = (j, "store")
+            elif where == "store":
+                p_ready[st][who] += 1
+                at[who] = (j + 1, "wait")
+            elif where == "wait" and j == blocks and (last if own_barrier else passed(pv_done, (blocks - 1) & 1)):
+                early = early or done < len(mma)
+                at[who] = (blocks, "out")
+    return early
+
+
+@pytest.mark.parametrize("blocks", [1, 2, 3, 6])
+def test_flash_epilogue_waits_for_the_last_product(blocks):
+    for seed in range(150):
+        rnd = random.Random(seed)
+        rescales = lambda w, j: (w * 7 + j * 5 + seed) % 3 == 0                                 # noqa: E731
+        assert not _flash_order(blocks, 4, rescales, True, rnd), seed
+
+
+def test_flash_epilogue_on_the_shared_barrier_is_caught_by_the_model():
+    never = lambda w, j: False                                                                  # noqa: E731
+    assert any(_flash_order(3, 4, never, False, random.Random(seed)) for seed in range(150))

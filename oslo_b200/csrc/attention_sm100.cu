@@ -546,22 +546,22 @@ fa_wide_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ C
       constexpr uint32_t SLOT_AT = FW_SLOT >> 4, SUB_AT = FW_SUB >> 4;
       const bool issuer = elect_one();
       Cursor at;
-      bool ok = mbar_wait_warp(bar(0), 0, abort_flag, p.err, ERR_WAIT_FULL);
+      bool ok = mbar_wait(bar(0), 0, abort_flag, p.err, ERR_WAIT_FULL);
       auto issue_qk = [&](int j) -> bool {
         const int st = j & 1;
-        if (!mbar_wait_warp(bar(11 + st), ((j >> 1) & 1) ^ 1, abort_flag, p.err, ERR_WAIT_TMEM_EMPTY)) return false;
+        if (!mbar_wait(bar(11 + st), ((j >> 1) & 1) ^ 1, abort_flag, p.err, ERR_WAIT_TMEM_EMPTY)) return false;
         tc_fence_after();
         const uint32_t dst = tmem_base + st * BN;
         for (int g = 0; g < pairs; ++g) {
           uint32_t a = q_at + g * SLOT_AT;
           int a_slot = -1;
           if (g >= resident) {
-            if (!mbar_wait_warp(bar(16 + at.slot), at.phase, abort_flag, p.err, ERR_WAIT_FULL)) return false;
+            if (!mbar_wait(bar(16 + at.slot), at.phase, abort_flag, p.err, ERR_WAIT_FULL)) return false;
             a_slot = at.slot;
             a = ring_at + at.slot * SLOT_AT;
             at.next(ring);
           }
-          if (!mbar_wait_warp(bar(16 + at.slot), at.phase, abort_flag, p.err, ERR_WAIT_FULL)) return false;
+          if (!mbar_wait(bar(16 + at.slot), at.phase, abort_flag, p.err, ERR_WAIT_FULL)) return false;
           const uint64_t da = desc_k + a, db = desc_k + (ring_at + at.slot * SLOT_AT);
           const int left = dim - g * 128;              // columns from this slot on
           if (issuer) {
@@ -593,11 +593,11 @@ fa_wide_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ C
           if (!ok) break;
         }
         const int st = j & 1;
-        ok = mbar_wait_warp(bar(st ? 15 : 13), (j >> 1) & 1, abort_flag, p.err, ERR_WAIT_FULL);
+        ok = mbar_wait(bar(st ? 15 : 13), (j >> 1) & 1, abort_flag, p.err, ERR_WAIT_FULL);
         if (!ok) break;
         tc_fence_after();
         for (int c = 0; c < vc && ok; c += 2) {
-          ok = mbar_wait_warp(bar(16 + at.slot), at.phase, abort_flag, p.err, ERR_WAIT_FULL);
+          ok = mbar_wait(bar(16 + at.slot), at.phase, abort_flag, p.err, ERR_WAIT_FULL);
           if (!ok) break;
           const uint64_t db = desc_v + (ring_at + at.slot * SLOT_AT);
           const uint32_t dst = tmem_base + O_COL + c * 64, src = tmem_base + st * BN;

@@ -178,10 +178,8 @@ __global__ void __launch_bounds__(32 * HP_WARPS) head_prep_kernel(const HeadPrep
       float x[VEC];
       load_vec<T, VEC>(src + c, x);
 #pragma unroll
-      for (int i = 0; i < VEC; ++i) {
-        ss = fmaf(x[i], x[i], ss);
-        buf[c + i] = x[i];
-      }
+      for (int i = 0; i < VEC; ++i) ss = fmaf(x[i], x[i], ss);
+      store_vec<float, VEC>(buf + c, x);
     }
     const float r = 1.0f / sqrtf(warp_sum(ss) / dim + p.eps);
     __syncwarp();
@@ -198,8 +196,7 @@ __global__ void __launch_bounds__(32 * HP_WARPS) head_prep_kernel(const HeadPrep
   auto put = [&](T* dst, const float* buf) {
     for (int c = lane * VEC; c < dim; c += 32 * VEC) {
       float x[VEC];
-#pragma unroll
-      for (int i = 0; i < VEC; ++i) x[i] = buf[c + i];
+      load_vec<float, VEC>(buf + c, x);
       store_vec<T, VEC>(dst + c, x);
     }
   };
@@ -247,9 +244,14 @@ __global__ void __launch_bounds__(32 * HP_WARPS) head_prep_kernel(const HeadPrep
     if (per <= HP_PER) {
       float x[HP_PER][VEC];
 #pragma unroll
-      for (int r = 0; r < HP_PER; ++r)
+      for (int r = 0; r < HP_PER; ++r) {
+        if (r < per) {
+          load_vec<float, VEC>(src + r * dim, x[r]);
+        } else {
 #pragma unroll
-        for (int i = 0; i < VEC; ++i) x[r][i] = r < per ? src[r * dim + i] : 0.f;
+          for (int i = 0; i < VEC; ++i) x[r][i] = 0.f;
+        }
+      }
       for (int h = first; h < h1 - h0; h += lanes) {
         const float* tw = ts + h * H + g * per;
         float o[VEC];

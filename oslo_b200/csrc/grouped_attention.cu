@@ -145,7 +145,57 @@ struct HeadPrepParams {
   int* err;
 };
 
-constexpr int HP_WARPS = 8, HP_PER = 8;               // query heads per key head that a thread keeps in registers
+constexpr int HP_WARPS = 8;
+
+// what heads h0..h1 of a token ask of the keys of all key heads: sums of the heads `qs` [H][dim] weighted by `ts` [h1 - h0][H]. PER: query
+// heads per key head, 0: any number
+template <typename T, int VEC, int PER>
+__device__ __forceinline__ void head_mix(const HeadPrepParams& p, const float* qs, const float* ts, long long row, int h0, int h1) {
+  const int H = p.H, dim = p.dim, per = PER > 0 ? PER : H / p.G, cols = p.G * dim, groups = cols / VEC;
+  const int threads = static_cast<int>(blockDim.x), tid = threadIdx.x;
+  T* out = static_cast<T*>(p.q_out) + (row * H + h0) * cols;
+  // a thread owns VEC columns; with fewer columns than threads several threads share them, each with heads of its own
+  const int lanes = groups < threads ? threads / groups : 1, step = groups < threads ? groups : threads;
+  const int first = groups < threads ? tid / groups : 0;
+  if (first >= lanes) return;
+  for (int u = groups < threads ? tid - first * groups : tid; u < groups; u += step) {
+    const int c = u * VEC, g = c / dim;
+    const float* src = qs + g * per * dim + (c - g * dim);
+    float x[PER > 0 ? PER : 1][VEC];
+    if constexpr (PER > 0) {
+#pragma unroll
+      for (int r = 0; r < PER; ++r) load_vec<float, VEC>(src + r * dim, x[r]);
+    }
+    const float* tw = ts + first * H + g * per;
+    T* dst = out + static_cast<long long>(first) * cols + c;
+#pragma unroll 2
+    for (int h = first; h < h1 - h0; h += lanes, tw += lanes * H, dst += static_cast<long long>(lanes) * cols) {
+      float o[VEC];
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) o[i] = 0.f;
+      if constexpr (PER > 0) {
+        constexpr int W = PER % 4 == 0 ? 4 : 1;        // weights read at a time; H is a multiple of PER
+#pragma unroll
+        for (int r = 0; r < PER; r += W) {
+          float m[W];
+          load_vec<float, W>(tw + r, m);
+#pragma unroll
+          for (int k = 0; k < W; ++k)
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) o[i] = fmaf(m[k], x[r + k][i], o[i]);
+        }
+      } else {
+        for (int r = 0; r < per; ++r) {
+          float y[VEC];
+          load_vec<float, VEC>(src + r * dim, y);
+#pragma unroll
+          for (int i = 0; i < VEC; ++i) o[i] = fmaf(tw[r], y[i], o[i]);
+        }
+      }
+      store_vec<T, VEC>(dst, o);
+    }
+  }
+}
 
 // block = (token, share of the query heads that are written); the first share also does keys and values. Angles are
 // computed once per token. VEC 4: everything is aligned to four elements
@@ -184,6 +234,7 @@ __global__ void __launch_bounds__(32 * HP_WARPS) head_prep_kernel(const HeadPrep
     const float r = 1.0f / sqrtf(warp_sum(ss) / dim + p.eps);
     __syncwarp();
     const int n = p.n_freq;
+#pragma unroll 2
     for (int i = lane; i < n; i += 32) {               // pairs
       const int a = p.halves ? i : 2 * i, c = p.halves ? i + n : 2 * i + 1;
       const float x = buf[a] * r * (w ? Num<T>::to(w[a]) : 1.f), y = buf[c] * r * (w ? Num<T>::to(w[c]) : 1.f);
@@ -232,53 +283,12 @@ __global__ void __launch_bounds__(32 * HP_WARPS) head_prep_kernel(const HeadPrep
   }
   if (p.talk == nullptr) return;
   __syncthreads();
-  const int per = H / p.G, cols = p.G * dim, groups = cols / VEC;
-  T* out = static_cast<T*>(p.q_out) + row * H * cols;
-  // a thread owns VEC columns; with fewer columns than threads several threads share them, each with heads of its own
-  const int lanes = groups < static_cast<int>(blockDim.x) ? static_cast<int>(blockDim.x) / groups : 1;
-  if (tid / groups >= lanes && groups < static_cast<int>(blockDim.x)) return;
-  const int first = groups < static_cast<int>(blockDim.x) ? tid / groups : 0;
-  for (int u = groups < static_cast<int>(blockDim.x) ? tid % groups : tid; u < groups; u += groups < static_cast<int>(blockDim.x) ? groups : static_cast<int>(blockDim.x)) {
-    const int c = u * VEC, g = c / dim, d = c - g * dim;
-    const float* src = qs + g * per * dim + d;
-    if (per <= HP_PER) {
-      float x[HP_PER][VEC];
-#pragma unroll
-      for (int r = 0; r < HP_PER; ++r) {
-        if (r < per) {
-          load_vec<float, VEC>(src + r * dim, x[r]);
-        } else {
-#pragma unroll
-          for (int i = 0; i < VEC; ++i) x[r][i] = 0.f;
-        }
-      }
-      for (int h = first; h < h1 - h0; h += lanes) {
-        const float* tw = ts + h * H + g * per;
-        float o[VEC];
-#pragma unroll
-        for (int i = 0; i < VEC; ++i) o[i] = 0.f;
-#pragma unroll
-        for (int r = 0; r < HP_PER; ++r) {
-          if (r >= per) break;
-          const float m = tw[r];
-#pragma unroll
-          for (int i = 0; i < VEC; ++i) o[i] = fmaf(m, x[r][i], o[i]);
-        }
-        store_vec<T, VEC>(out + static_cast<long long>(h0 + h) * cols + c, o);
-      }
-    } else {
-      for (int h = first; h < h1 - h0; h += lanes) {
-        const float* tw = ts + h * H + g * per;
-        float o[VEC];
-#pragma unroll
-        for (int i = 0; i < VEC; ++i) o[i] = 0.f;
-        for (int r = 0; r < per; ++r)
-#pragma unroll
-          for (int i = 0; i < VEC; ++i) o[i] = fmaf(tw[r], src[r * dim + i], o[i]);
-        store_vec<T, VEC>(out + static_cast<long long>(h0 + h) * cols + c, o);
-      }
-    }
-  }
+  const int per = H / p.G;
+  if (per == 4 && VEC == 4) head_mix<T, VEC, 4>(p, qs, ts, row, h0, h1);
+  else if (per == 8 && VEC == 4) head_mix<T, VEC, 8>(p, qs, ts, row, h0, h1);
+  else if (per == 2) head_mix<T, VEC, 2>(p, qs, ts, row, h0, h1);
+  else if (per == 1) head_mix<T, VEC, 1>(p, qs, ts, row, h0, h1);
+  else head_mix<T, VEC, 0>(p, qs, ts, row, h0, h1);
 }
 
 // ------------------------------------------------------------------ decode
@@ -618,9 +628,9 @@ __global__ void __launch_bounds__(128) grouped_decode_mma_kernel(const GroupedPa
 // ------------------------------------------------------------------ decode, wide keys on tensor cores
 // One cached key row (dim columns) for all query heads, value heads side by side in a cached value row: block = (slice, up to 16 MT
 // query heads, row). A stage of KEYS keys and values is on its way while the one before is used: (1) scores of 16 heads x 16 keys per
-// warp (over a share of the columns when there are fewer tiles than warps), (2) softmax, a warp per head row, (3) 16 heads x 64 value
-// columns per item, only the columns of these heads' groups.
-constexpr int WD_WARPS = 8;
+// warp (over a share of the columns when there are fewer tiles than warps), (2) softmax, head rows dealt out to the warps, (3) 16 heads x
+// 32 value columns per item, only the columns of these heads' groups.
+constexpr int WD_WARPS = 16, WD_COLS = 32;
 
 struct WideLayout {
   int kp, vp;                          // row pitches of the key and value stages
@@ -631,7 +641,7 @@ __host__ __device__ inline WideLayout wide_layout(int dim, int vdim) {
   WideLayout l;
   l.kp = (dim + 15) / 16 * 16 + 8;     // 16-byte rows whose starts fall on different banks
   l.vp = (vdim + 15) / 16 * 16 + 8;
-  constexpr int TILES = MT * KEYS / 16, KSPLIT = WD_WARPS / (TILES < WD_WARPS ? TILES : WD_WARPS);
+  constexpr int TILES = MT * KEYS / 16, KSPLIT = WD_WARPS / TILES;
   l.q = 0;
   l.k = l.q + static_cast<size_t>(MT) * 16 * l.kp * 2;
   l.v = l.k + static_cast<size_t>(NBUF) * KEYS * l.kp * 2;
@@ -644,9 +654,9 @@ __host__ __device__ inline WideLayout wide_layout(int dim, int vdim) {
 
 template <typename T, int MT, int KEYS, int NBUF, int ITEMS>
 __global__ void __launch_bounds__(32 * WD_WARPS) wide_decode_kernel(const GroupedParams p) {
-  constexpr int ROWS = MT * 16, TILES = MT * KEYS / 16, KSPLIT = WD_WARPS / (TILES < WD_WARPS ? TILES : WD_WARPS);
+  constexpr int ROWS = MT * 16, TILES = MT * KEYS / 16, KSPLIT = WD_WARPS / TILES;
   constexpr int RW = ROWS / WD_WARPS;                  // head rows of a warp in step 2
-  static_assert(TILES <= WD_WARPS, "a warp has one tile of scores");
+  static_assert(TILES * KSPLIT == WD_WARPS && RW * WD_WARPS == ROWS && KEYS <= 32, "a warp has one share of a tile of scores, a lane one key");
   extern __shared__ uint4 gm_smem[];
   const WideLayout lay = wide_layout<MT, KEYS, NBUF>(p.dim, p.vdim);
   uint8_t* base = reinterpret_cast<uint8_t*>(gm_smem);
@@ -702,7 +712,7 @@ __global__ void __launch_bounds__(32 * WD_WARPS) wide_decode_kernel(const Groupe
   // step 1: tile of this warp and its share of the columns
   const int tile = w % TILES, mt = tile % MT, kt = tile / MT, part = w / TILES;
   const int steps = (p.dim + 15) / 16, step0 = steps * part / KSPLIT, step1 = steps * (part + 1) / KSPLIT;
-  // step 3: items (16 heads, 64 of the columns of their groups), dealt out to the warps
+  // step 3: items (16 heads, WD_COLS of the columns of their groups), dealt out to the warps
   int item_mt[ITEMS], item_c0[ITEMS], item_c1[ITEMS];
 #pragma unroll
   for (int i = 0; i < ITEMS; ++i) { item_mt[i] = -1; item_c0[i] = item_c1[i] = 0; }
@@ -712,23 +722,26 @@ __global__ void __launch_bounds__(32 * WD_WARPS) wide_decode_kernel(const Groupe
     for (int m = 0; m < MT; ++m) {
       if (m * 16 >= nh) break;
       const int lo = (h0 + m * 16) / per * vd, hi = ((h0 + min(nh, m * 16 + 16) - 1) / per + 1) * vd;
-      for (int c = lo; c < hi; c += 64, ++n)
+      for (int c = lo; c < hi; c += WD_COLS, ++n)
         if (n % WD_WARPS == w) {
 #pragma unroll
           for (int i = 0; i < ITEMS; ++i)
-            if (i == n / WD_WARPS) { item_mt[i] = m; item_c0[i] = c; item_c1[i] = min(hi, c + 64); }
+            if (i == n / WD_WARPS) { item_mt[i] = m; item_c0[i] = c; item_c1[i] = min(hi, c + WD_COLS); }
         }
     }
   }
-  float o[ITEMS][8][4];
+  float o[ITEMS][WD_COLS / 8][4];
 #pragma unroll
   for (int i = 0; i < ITEMS; ++i)
 #pragma unroll
-    for (int j = 0; j < 8; ++j) o[i][j][0] = o[i][j][1] = o[i][j][2] = o[i][j][3] = 0.f;
+    for (int j = 0; j < WD_COLS / 8; ++j) o[i][j][0] = o[i][j][1] = o[i][j][2] = o[i][j][3] = 0.f;
   float m_row[RW], l_row[RW];                          // of the warp's head rows, the same in every lane; scores in log2 units
 #pragma unroll
   for (int r = 0; r < RW; ++r) { m_row[r] = -CUDART_INF_F; l_row[r] = 0.f; }
   const float scale = p.scale * GD_LOG2E;
+  const uint32_t qa = smem_u32(qs + mt * 16 * lay.kp + ((l & 7) + ((l >> 3) & 1) * 8) * lay.kp + (l >> 4) * 8);
+  const uint32_t ka = smem_u32(ks + kt * 16 * lay.kp + ((l & 7) + (l >> 4) * 8) * lay.kp + ((l >> 3) & 1) * 8);
+  const uint32_t k_stage = KEYS * lay.kp * 2;
   if (t0 < t1) fetch(t0, 0);
   for (int k0 = t0, it = 0; k0 < t1; k0 += KEYS, ++it) {
     const int buf = NBUF > 1 ? it & 1 : 0;
@@ -741,60 +754,44 @@ __global__ void __launch_bounds__(32 * WD_WARPS) wide_decode_kernel(const Groupe
     __syncthreads();
     {
       float c[2][4] = {};
-      const T* kw = ks + (buf * KEYS + kt * 16) * lay.kp;
-      const T* qw = qs + mt * 16 * lay.kp;
+      const uint32_t kaddr = ka + buf * k_stage;
 #pragma unroll 4
       for (int kk = step0; kk < step1; ++kk) {
         uint32_t a[4], bb[4];
-        gd_ldsm4(a, smem_u32(qw + ((l & 7) + ((l >> 3) & 1) * 8) * lay.kp + kk * 16 + (l >> 4) * 8));
-        gd_ldsm4(bb, smem_u32(kw + ((l & 7) + (l >> 4) * 8) * lay.kp + kk * 16 + ((l >> 3) & 1) * 8));
+        gd_ldsm4(a, qa + kk * 32);
+        gd_ldsm4(bb, kaddr + kk * 32);
         GdMma<T>::run(c[0], a, bb[0], bb[1]);
         GdMma<T>::run(c[1], a, bb[2], bb[3]);
       }
-      float* dst = sc + (part * ROWS + mt * 16) * (KEYS + 1) + kt * 16;
+      float* dst = sc + (part * ROWS + mt * 16 + (l >> 2)) * (KEYS + 1) + kt * 16 + (l & 3) * 2;
 #pragma unroll
       for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) dst[((l >> 2) + (e >> 1) * 8) * (KEYS + 1) + nt * 8 + (l & 3) * 2 + (e & 1)] = c[nt][e];
+        for (int e = 0; e < 4; ++e) dst[(e >> 1) * 8 * (KEYS + 1) + nt * 8 + (e & 1)] = c[nt][e];
     }
     __syncthreads();
     {
-      constexpr int KL = (KEYS + 31) / 32;             // keys per lane
-      bool vis[KL];
-#pragma unroll
-      for (int u = 0; u < KL; ++u) {
-        const int j = l + 32 * u, pos = run.at(k0 + j);
-        vis[u] = j < KEYS && k0 + j < t1 && (p.keep == nullptr || pos >= p.n_keep || p.keep[b * p.ld_keep + pos]);
-      }
+      const int pos = run.at(k0 + l);
+      const bool vis = l < KEYS && k0 + l < t1 && (p.keep == nullptr || pos >= p.n_keep || p.keep[b * p.ld_keep + pos]);
 #pragma unroll
       for (int r = 0; r < RW; ++r) {
         const int row = w * RW + r;
-        float d[KL], mx = m_row[r];
+        float x = 0.f;
+        if (l < KEYS) {
 #pragma unroll
-        for (int u = 0; u < KL; ++u) {
-          const int j = l + 32 * u;
-          float x = 0.f;
-          if (j < KEYS) {
-#pragma unroll
-            for (int s = 0; s < KSPLIT; ++s) x += sc[(s * ROWS + row) * (KEYS + 1) + j];
-          }
-          d[u] = vis[u] ? x * scale : -CUDART_INF_F;
-          mx = fmaxf(mx, d[u]);
+          for (int s = 0; s < KSPLIT; ++s) x += sc[(s * ROWS + row) * (KEYS + 1) + l];
         }
+        const float d = vis ? x * scale : -CUDART_INF_F;
+        float mx = d;
 #pragma unroll
         for (int off = 16; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
+        mx = fmaxf(mx, m_row[r]);
         const float ref = mx == -CUDART_INF_F ? 0.f : mx, al = gd_exp2(m_row[r] - ref);     // 2^-inf = 0
-        float sum = 0.f;
-#pragma unroll
-        for (int u = 0; u < KL; ++u) {
-          const int j = l + 32 * u;
-          const float e = gd_exp2(d[u] - ref);
-          sum += e;
-          if (j < KEYS) ps[row * (KEYS + 8) + j] = Num<T>::from(e);
-        }
-        l_row[r] = l_row[r] * al + warp_sum(sum);
-        m_row[r] = mx;
+        const float e = gd_exp2(d - ref);
+        if (l < KEYS) ps[row * (KEYS + 8) + l] = Num<T>::from(e);
         if (l == 0) alpha_s[row] = al;
+        l_row[r] = l_row[r] * al + warp_sum(e);
+        m_row[r] = mx;
       }
     }
     __syncthreads();
@@ -804,7 +801,7 @@ __global__ void __launch_bounds__(32 * WD_WARPS) wide_decode_kernel(const Groupe
       const float a0 = alpha_s[item_mt[i] * 16 + (l >> 2)], a1 = alpha_s[item_mt[i] * 16 + (l >> 2) + 8];
       if (__any_sync(0xffffffffu, a0 != 1.f || a1 != 1.f)) {
 #pragma unroll
-        for (int j = 0; j < 8; ++j) { o[i][j][0] *= a0; o[i][j][1] *= a0; o[i][j][2] *= a1; o[i][j][3] *= a1; }
+        for (int j = 0; j < WD_COLS / 8; ++j) { o[i][j][0] *= a0; o[i][j][1] *= a0; o[i][j][2] *= a1; o[i][j][3] *= a1; }
       }
       const T* pw = ps + item_mt[i] * 16 * (KEYS + 8);
 #pragma unroll
@@ -813,7 +810,7 @@ __global__ void __launch_bounds__(32 * WD_WARPS) wide_decode_kernel(const Groupe
         gd_ldsm4(a, smem_u32(pw + ((l & 7) + ((l >> 3) & 1) * 8) * (KEYS + 8) + kk * 16 + (l >> 4) * 8));
         const T* vw = vs + (buf * KEYS + kk * 16 + (l & 7) + ((l >> 3) & 1) * 8) * lay.vp + item_c0[i] + (l >> 4) * 8;
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
+        for (int j = 0; j < WD_COLS / 16; ++j) {
           if (item_c0[i] + j * 16 >= item_c1[i]) break;
           uint32_t bb[4];
           gd_ldsm4_t(bb, smem_u32(vw + j * 16));
@@ -829,7 +826,7 @@ __global__ void __launch_bounds__(32 * WD_WARPS) wide_decode_kernel(const Groupe
   for (int i = 0; i < ITEMS; ++i) {
     if (item_mt[i] < 0) continue;
 #pragma unroll
-    for (int j = 0; j < 8; ++j) {
+    for (int j = 0; j < WD_COLS / 8; ++j) {
       const int c = item_c0[i] + j * 8 + (l & 3) * 2;
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
@@ -864,7 +861,7 @@ static WidePlan wide_plan(int H, int VG, int dim, int vdim, int dtype) {
     int n = 0;
     for (int m = 0; m < w.mt && h0 + m * 16 < H; ++m) {
       const int a = h0 + m * 16, z = std::min(H, a + 16) - 1;
-      n += ((z / per - a / per + 1) * vd + 63) / 64;
+      n += ((z / per - a / per + 1) * vd + WD_COLS - 1) / WD_COLS;
     }
     worst = std::max(worst, n);
   }
@@ -884,10 +881,10 @@ static WidePlan wide_plan(int H, int VG, int dim, int vdim, int dtype) {
 
 template <typename T, int MT, int KEYS, int NBUF, int ITEMS>
 static int wide_launch(const GroupedParams& p, int B, size_t smem, cudaStream_t st) {
-  cudaError_t e = cudaFuncSetAttribute(wide_decode_kernel<T, MT, KEYS, NBUF, ITEMS>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                       static_cast<int>(smem));
+  const auto kernel = wide_decode_kernel<T, MT, KEYS, NBUF, ITEMS>;
+  cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
   if (e != cudaSuccess) return static_cast<int>(e);
-  wide_decode_kernel<T, MT, KEYS, NBUF, ITEMS><<<dim3(p.splits, (p.H + 16 * MT - 1) / (16 * MT), B), 32 * WD_WARPS, smem, st>>>(p);
+  kernel<<<dim3(p.splits, (p.H + 16 * MT - 1) / (16 * MT), B), 32 * WD_WARPS, smem, st>>>(p);
   return static_cast<int>(cudaGetLastError());
 }
 template <typename T, int MT, int KEYS, int NBUF>
@@ -1027,7 +1024,7 @@ extern "C" int oslo_grouped_splits(int B, int H, int G, int VG, int T, int dim, 
   if (wide.keys) {
     // whole waves of blocks: a block costs its share of the keys and some for its start
     const long long blocks = static_cast<long long>(B) * ((H + 16 * wide.mt - 1) / (16 * wide.mt));
-    const long long room = static_cast<long long>(num_sms) * std::max<size_t>(1, std::min<size_t>(4, WD_SMEM / (wide.smem + 2048)));
+    const long long room = static_cast<long long>(num_sms) * std::max<size_t>(1, std::min<size_t>(wide.items > 1 ? 1 : 2, WD_SMEM / (wide.smem + 2048)));
     int best = 1;
     double best_cost = 1e30;
     for (int n = 1; n <= GD_MAX_SPLITS && (n == 1 || n * 64 <= T); ++n) {

@@ -36,7 +36,7 @@ CASES = {
     "odd": case(51, 35, 1e-3, 5, 9, attn(5, 5, 7, 0.4, 4, moe(13, 3, 3, 0.9, 17, 2.1), 50.0, {**YARN, "fast": 30.0}), attn(6, 3, 9, 0.3, 6, dense(21)),
                 attn(6, 2, 5, 0.5, 2, moe(7, 7, 5, 3.0, 11, 0.5), 300.0), attn(1, 1, 11, 0.3, 10, None, 20.0, YARN)),
     # head sizes the tensor-core kernels take as they are, keys of several widths
-    "heads64": case(128, 128, 1e-6, 4, 24, attn(4, 2, 64, 0.15, 64, moe(64, 12, 1, 1.5, 88, 1.0), 5e5, {"factor": 4.0, "original": 64, "fast": 16.0, "slow": 1.0}),
+    "heads64": case(128, 128, 2e-6, 3, 40, attn(6, 3, 64, 0.15, 48, moe(80, 10, 2, 1.5, 88, 1.0), 3e5, {"factor": 6.0, "original": 48, "fast": 16.0, "slow": 2.0}),
                     attn(8, 4, 32, 0.2, 16, dense(160)), attn(4, 1, 128, 0.1, 96, moe(96, 8, 2, 2.5, 64), 1e5, YARN), attn(6, 6, 16, 0.3, 16, None)),
     # one head, one expert, one tap, sizes of 1; nothing rotated, factor 1
     "ones": case(17, 16, 1e-6, 1, 1, attn(1, 1, 8, 1.0, 0, moe(8, 1, 1, 1.0, 1, 1.0)), attn(2, 1, 2, 1.0, 2, dense(1), 10.0, {**YARN, "factor": 1.0}),
